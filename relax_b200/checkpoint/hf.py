@@ -516,8 +516,13 @@ def config_from_hf(path: str) -> ModelConfig:
     the reference cross-checks its Megatron flags against this file, relax/backends/megatron/arguments.py)."""
     import json
 
+    from ..models.architectures import architecture_of
+
     with open(os.path.join(path, "config.json")) as f:
         d = json.load(f)
+    own = architecture_of(d)
+    if own is not None:
+        return own.config_from_dict(d, os.path.basename(os.path.normpath(path)) or "model")
     arch = (d.get("architectures") or [""])[0]
     heads = d["num_attention_heads"]
     kw = dict(name=os.path.basename(os.path.normpath(path)) or "hf", num_layers=d["num_hidden_layers"], hidden_size=d["hidden_size"],
@@ -563,6 +568,12 @@ def validate_against_hf(cfg: ModelConfig, path: str) -> None:
     if not os.path.isfile(os.path.join(path, "config.json")):
         return
     hf = config_from_hf(path)
+    if cfg.is_composed or hf.is_composed:
+        names = ("layer_specs", "hidden_size", "vocab_size", "norm_groups", "rms_norm_eps")
+        diff = [f"{n}: {getattr(cfg, n)} here, {getattr(hf, n)} in the checkpoint" for n in names if getattr(cfg, n) != getattr(hf, n)]
+        if diff:
+            raise ValueError("the model configuration does not match the checkpoint: " + "; ".join(diff))
+        return
     fields = ["hidden_size", "num_attention_heads", "num_query_groups", "num_layers", "head_dim", "vocab_size",
               "tie_word_embeddings", "rope_theta", "rms_norm_eps"]
     if cfg.is_moe or hf.is_moe:
@@ -581,7 +592,16 @@ def validate_against_hf(cfg: ModelConfig, path: str) -> None:
 
 def load_hf_into_rollout(path: str, cfg: ModelConfig, rollout_weights) -> None:
     """Fill a rollout engine's parameter buffer straight from a Hugging Face checkpoint (a grader or any serving-only
-    model that has no trainer): HF names -> Megatron layout -> the block-copy plan the weight sync uses."""
+    model that has no trainer): HF names -> Megatron layout -> the block-copy plan the weight sync uses.  Designs with
+    their own tensor names (:mod:`relax_b200.models.architectures`) fill the buffer themselves."""
+    if cfg.is_composed:
+        from ..models.architectures import architecture_of
+
+        with open(os.path.join(path, "config.json")) as f:
+            own = architecture_of(json.load(f))
+        if own is None:
+            raise ValueError(f"{path} holds no checkpoint of a composed stack")
+        return own.load_tensors(cfg, load_hf_checkpoint(path, dequantize=False), rollout_weights)
     from ..weight_sync.plan import TrainerLayout, build_plan
     from ..weight_sync.sync import apply_block
 

@@ -28,6 +28,30 @@ class VisionConfig:
     rms_norm_eps: "float | None" = None
 
 
+@dataclass(frozen=True)
+class LayerSpec:
+    """One layer of a composed stack (``ModelConfig.layer_specs``): its token mixer with the mixer's sizes and its
+    feed-forward.  ``hgrn2``: gated linear recurrence with ``heads`` states of ``dim x vdim``.  ``latent_attention``:
+    softmax attention whose keys and values are projections of one cached latent row of ``kv_rank`` features per token."""
+    mixer: str
+    heads: int
+    dim: int                     # query (and key / forget-gate) features per head
+    vdim: int                    # value features per head
+    kv_rank: int = 0             # latent_attention only
+    scale: float = 1.0           # latent_attention only: factor on q . k
+    ff: int = 0                  # width of the gated feed-forward; 0 = the layer has none
+    act: str = "gelu_tanh"       # activation of the feed-forward's gate half
+
+    def __post_init__(self):
+        if self.mixer not in MIXERS:
+            raise ValueError(f"unknown mixer {self.mixer!r}; known: {MIXERS}")
+        if min(self.heads, self.dim, self.vdim) < 1 or (self.mixer == "latent_attention" and self.kv_rank < 1) or self.ff < 0:
+            raise ValueError(f"bad layer sizes: {self}")
+
+
+MIXERS = ("hgrn2", "latent_attention")
+
+
 @dataclass
 class ModelConfig:
     name: str = "tiny"
@@ -91,7 +115,20 @@ class ModelConfig:
     dsa_index_heads: int = 4
     dsa_index_dim: int = 16
     dsa_indexer_loss_coef: float = 1.0
+    # composed stacks (Talizen): every layer is spelled out - mixer, sizes, feed-forward.  The sublayers read the fp32
+    # residual stream itself and their OUTPUT is normed (RMS over each of `norm_groups` equal parts) before it is added.
+    # The fields above that describe one uniform layer (heads, head_dim, ffn, rotary, MoE, ...) do not apply then.
+    layer_specs: Optional[tuple] = None
+    norm_groups: int = 1
     dtype: str = "bf16"
+
+    @property
+    def is_composed(self) -> bool:
+        return self.layer_specs is not None
+
+    def layers_with(self, mixer: str) -> list:
+        """Indices of the layers of a composed stack that use ``mixer``."""
+        return [i for i, s in enumerate(self.layer_specs or ()) if s.mixer == mixer]
 
     @property
     def is_moe(self) -> bool:
@@ -115,6 +152,15 @@ class ModelConfig:
 
     def num_parameters(self) -> int:
         h, L = self.hidden_size, self.num_layers
+        if self.is_composed:
+            n = 2 * self.vocab_size * h + h
+            for s in self.layer_specs:
+                n += h + 3 * s.ff * h + (h if s.ff else 0) + s.heads * s.vdim * h
+                if s.mixer == "hgrn2":
+                    n += s.heads * (2 * s.dim + s.vdim) * h + 2 * s.heads * s.dim + s.vdim
+                else:
+                    n += (s.heads * (s.dim + 1) + s.kv_rank) * h + s.kv_rank * (1 + s.heads * (s.dim + s.vdim))
+            return n
         attn = h * (self.q_size * (2 if self.attention_output_gate else 1) + 2 * self.kv_size) + self.q_size * h
         if self.qk_layernorm:
             attn += 2 * self.head_dim
@@ -137,6 +183,22 @@ PRESETS: dict[str, ModelConfig] = {}
 def _reg(c: ModelConfig):
     PRESETS[c.name] = c
     return c
+
+
+def composed_config(name: str, layers, hidden_size: int, vocab_size: int, norm_groups: int = 1, eps: float = 1e-5, **kw) -> ModelConfig:
+    """A composed stack from its list of :class:`LayerSpec`."""
+    layers = tuple(layers)
+    if not layers:
+        raise ValueError("a composed stack needs at least one layer")
+    if norm_groups < 1 or hidden_size % norm_groups:
+        raise ValueError(f"{norm_groups} norm groups do not divide the width {hidden_size}")
+    return ModelConfig(name=name, num_layers=len(layers), hidden_size=hidden_size, vocab_size=vocab_size, rms_norm_eps=eps,
+                       layer_specs=layers, norm_groups=norm_groups, qk_layernorm=False, **kw)
+
+
+def talizen_layers(n_layers: int, every: int, rec: LayerSpec, att: LayerSpec) -> tuple:
+    """``every - 1`` recurrent layers, then one latent-attention layer, repeated."""
+    return tuple(att if (i + 1) % every == 0 else rec for i in range(n_layers))
 
 
 # BASELINE config 0 ("tiny Qwen-style decoder")
@@ -232,6 +294,20 @@ _reg(ModelConfig(name="qwen2.5-vl-7b", num_layers=28, hidden_size=3584, num_atte
 _reg(ModelConfig(name="llama3-8b", num_layers=32, hidden_size=4096, num_attention_heads=32, num_query_groups=8,
                  head_dim=128, ffn_hidden_size=14336, vocab_size=128256, qk_layernorm=False, rope_theta=5e5,
                  rms_norm_eps=1e-5))
+
+
+# Talizen: HGRN2 recurrent layers with a latent-attention layer among every few of them
+_reg(composed_config("tiny-talizen", [LayerSpec("hgrn2", heads=3, dim=16, vdim=24), LayerSpec("hgrn2", heads=3, dim=16, vdim=24, ff=160),
+                                      LayerSpec("latent_attention", heads=4, dim=32, vdim=16, kv_rank=48, scale=0.2, ff=224)],
+                     hidden_size=192, vocab_size=384, norm_groups=2, dtype="fp32"))
+_reg(composed_config("talizen-1b", talizen_layers(32, 4, LayerSpec("hgrn2", heads=16, dim=128, vdim=128),
+                                                  LayerSpec("latent_attention", heads=16, dim=128, vdim=128, kv_rank=512,
+                                                            scale=128 ** -0.5, ff=8192)),
+                     hidden_size=2048, vocab_size=64000, norm_groups=8))
+_reg(composed_config("talizen-5b", talizen_layers(36, 4, LayerSpec("hgrn2", heads=32, dim=128, vdim=128),
+                                                  LayerSpec("latent_attention", heads=32, dim=128, vdim=128, kv_rank=512,
+                                                            scale=128 ** -0.5, ff=12288)),
+                     hidden_size=4096, vocab_size=151936, norm_groups=8))
 
 
 def get_config(name: str, **overrides) -> ModelConfig:

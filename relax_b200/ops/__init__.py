@@ -51,6 +51,61 @@ def swiglu(gate_up):
     return ref.swiglu(gate_up)
 
 
+def glu(gate_up, act: str = "silu"):
+    """Gated unit ``act(gate) * up`` on ``[gate | up]`` rows; ``act``: ``silu`` or ``gelu_tanh``."""
+    return _cuda().glu(gate_up, act) if _use_cuda(gate_up) else ref.glu(gate_up, act)
+
+
+def linear_glu(x, w, act: str = "silu"):
+    """``glu(x @ w.T)`` with ``w = [gate; up]``: one fused kernel for decode shapes."""
+    return _cuda().linear_glu(x, w, act) if _use_cuda(x) else ref.glu(ref.linear(x, w), act)
+
+
+def embed_rows(tokens, w):
+    return _cuda().embed_rows(tokens, w) if _use_cuda(w) else ref.embed_rows(tokens, w)
+
+
+def norm_add(res, y, w, width, groups, eps, next_w=None):
+    """Output norm in groups + add to the fp32 residual stream (in place) + the next sublayer's input, one kernel."""
+    return (_cuda() if _use_cuda(y) else ref).norm_add(res, y, w, width, groups, eps, next_w)
+
+
+def hgrn2(qfv, f_bias, lower, norm_w, state, state_slot, ctx_lens, cu, heads, dim, vdim, eps):
+    """HGRN2 token mixing (gates, recurrence, per-head norm) on packed rows with the state carried in slots."""
+    return (_cuda() if _use_cuda(qfv) else ref).hgrn2(qfv, f_bias, lower, norm_w, state, state_slot, ctx_lens, cu, heads, dim, vdim, eps)
+
+
+def latent_write(raw, w, rank, eps, pool, slots):
+    """Norm of the latent projection + write of the new rows into the paged latent cache."""
+    (_cuda() if _use_cuda(raw) else ref).latent_write(raw, w, rank, eps, pool, slots)
+
+
+def head_linear(x, w, transposed):
+    """One small linear map per head (folds a latent up-projection into the queries / applies it to attended latents)."""
+    return (_cuda() if _use_cuda(x) else ref).head_linear(x, w, transposed)
+
+
+def latent_attention(q, pool, batch, block_size, scale, gate):
+    """Attention of absorbed queries over paged latent rows for the short segments of a
+    :class:`relax_b200.rollout.composed.SegmentBatch`, head outputs scaled by ``sigmoid(gate)``."""
+    if _use_cuda(q):
+        return _cuda().latent_attention(q, pool, batch, block_size, scale, gate)
+    n = batch.long_segs
+    cu = batch.short_cu if n else batch.cu
+    return ref.latent_attention(q, pool, batch.block_tables[n:], block_size, batch.ctx[n:], cu, scale, gate)
+
+
+def flash_serves_dims(dtype, dk: int, dv: int) -> bool:
+    """Whether the flash kernel takes heads of ``dk`` query / key and ``dv`` value features (zero-padded to 128)."""
+    return not _force_ref() and dtype == torch.bfloat16 and max(dk, dv) <= 128
+
+
+def flash_gated(q, k, v, cu_q, cu_k, scale, max_q, gate):
+    """Causal varlen attention on per-head keys / values whose widths may differ, every head's output scaled by
+    ``sigmoid(gate)``; returns ``[T, H * dv]``."""
+    return _cuda().flash_gated(q, k, v, cu_q, cu_k, scale, max_q, gate)
+
+
 def linear(x, w, bias=None):
     return _cuda().linear(x, w, bias) if _use_cuda(x) else ref.linear(x, w, bias)
 

@@ -32,8 +32,100 @@ def swiglu(gate_up):
     return (F.silu(g.float()) * u.float()).to(gate_up.dtype)
 
 
+def glu(gate_up, act: str = "silu"):
+    """``act(gate) * up`` for ``gate_up = [gate | up]``; ``act``: ``silu`` or ``gelu_tanh``."""
+    g, u = gate_up.chunk(2, dim=-1)
+    g = g.float()
+    a = F.silu(g) if act == "silu" else F.gelu(g, approximate="tanh")
+    return (a * u.float()).to(gate_up.dtype)
+
+
 def linear(x, w, bias=None):
     return F.linear(x, w, bias)
+
+
+# --------------------------------------------------------------------------- composed stacks (fp32 residual, grouped output norms)
+
+
+def group_rms(x, w, width: int, groups: int, eps: float):
+    """RMS norm over each of ``groups`` equal parts of the first ``width`` columns; the columns behind them are padding
+    and come out zero (their weights are).  fp32 in, fp32 out."""
+    y = torch.zeros_like(x, dtype=torch.float32)
+    p = x[:, :width].float().reshape(x.shape[0], groups, width // groups)
+    p = p / torch.sqrt(p.pow(2).mean(-1, keepdim=True) + eps)
+    y[:, :width] = p.reshape(x.shape[0], width) * w[:width].float()
+    return y
+
+
+def embed_rows(tokens, w):
+    """``(fp32 residual stream, its copy in the weights' type)`` of embedded tokens."""
+    h = w[tokens]
+    return h.float(), h
+
+
+def norm_add(res, y, w, width: int, groups: int, eps: float, next_w=None):
+    """``res += group_rms(y) * w`` in place (fp32); returns the next sublayer's input in ``w``'s type: the new stream
+    itself, or its own group norm with ``next_w`` when given."""
+    res += group_rms(y, w, width, groups, eps)
+    return (res if next_w is None else group_rms(res, next_w, width, groups, eps)).to(w.dtype)
+
+
+def hgrn2(qfv, f_bias, lower, norm_w, state, state_slot, ctx_lens, cu, heads: int, dim: int, vdim: int, eps: float):
+    """HGRN2 recurrence on packed rows ``[q | f | v]`` (raw projections), state carried in ``state[slot, h, dim, >= vdim]``.
+    Segment ``s`` owns rows ``cu[s]:cu[s+1]`` (``cu`` None: one row each), the last of them at position ``ctx_lens[s] - 1``;
+    a segment that starts at position 0 starts from a zero state whatever its slot holds.
+
+    ``g = lower + (1 - lower) sigmoid(f + bias)``;  ``S <- diag(g) S + (1 - g) v^T``;  ``o = S^T silu(q)``, RMS-normed."""
+    T, qd = qfv.shape[0], heads * dim
+    q = F.silu(qfv[:, :qd].float()).view(T, heads, dim)
+    lo = lower.float()
+    g = (lo + (1 - lo) * torch.sigmoid(qfv[:, qd:2 * qd].float() + f_bias.float())).view(T, heads, dim)
+    v = qfv[:, 2 * qd:2 * qd + heads * vdim].float().reshape(T, heads, vdim)
+    o = torch.zeros(T, (heads * vdim + 7) // 8 * 8, dtype=torch.float32, device=qfv.device)
+    bounds = list(range(T + 1)) if cu is None else cu.tolist()
+    for s, (a, b) in enumerate(zip(bounds, bounds[1:])):
+        S = state[int(state_slot[s])][:, :, :vdim]
+        cur = torch.zeros_like(S) if int(ctx_lens[s]) - (b - a) == 0 else S.clone()
+        for t in range(a, b):
+            cur = cur * g[t][:, :, None] + (1 - g[t])[:, :, None] * v[t][:, None, :]
+            r = (cur * q[t][:, :, None]).sum(1)
+            r = r / torch.sqrt(r.pow(2).mean(-1, keepdim=True) + eps) * norm_w[:vdim].float()
+            o[t, : heads * vdim] = r.reshape(-1)
+        S.copy_(cur)
+    return o.to(qfv.dtype)
+
+
+def latent_write(raw, w, rank: int, eps: float, pool, slots):
+    """RMS-normed latent rows -> ``pool[slots]`` (columns behind ``rank`` zero)."""
+    c = torch.zeros(raw.shape[0], pool.shape[1], dtype=torch.float32, device=raw.device)
+    x = raw[:, :rank].float()
+    c[:, :rank] = x / torch.sqrt(x.pow(2).mean(-1, keepdim=True) + eps) * w[:rank].float()
+    pool[slots] = c.to(pool.dtype)
+
+
+def head_linear(x, w, transposed: bool):
+    """Per-head product ``x[T, H, a] -> [T, H, b]`` with ``w[H, a, b]`` (``transposed``: ``w[H, b, a]``)."""
+    return torch.einsum("tha,hba->thb" if transposed else "tha,hab->thb", x.float(), w.float()).to(w.dtype)
+
+
+def latent_attention(q, pool, block_tables, block_size: int, ctx_lens, cu, scale: float, gate=None):
+    """Softmax attention of absorbed queries ``q[T, H, R]`` over the paged latent rows of their sequence (each row is key
+    and value of every head); row ``i`` of a segment of ``n`` rows sees the first ``ctx - n + i + 1`` of them.
+    ``gate[T, H]``: every head's output is multiplied by its sigmoid."""
+    T, H, R = q.shape
+    out = torch.zeros(T, H, R, dtype=torch.float32, device=q.device)
+    bounds = list(range(T + 1)) if cu is None else cu.tolist()
+    for s, (a, b) in enumerate(zip(bounds, bounds[1:])):
+        L = int(ctx_lens[s])
+        pos = torch.arange(L, device=q.device)
+        c = pool[block_tables[s].long()[pos // block_size] * block_size + pos % block_size].float()
+        sc = torch.einsum("thr,lr->thl", q[a:b].float(), c) * scale
+        lim = L - (b - a) + torch.arange(b - a, device=q.device)
+        sc = sc.masked_fill(pos[None, None, :] > lim[:, None, None], float("-inf"))
+        out[a:b] = torch.einsum("thl,lr->thr", torch.softmax(sc, -1), c)
+    if gate is not None:
+        out = out * torch.sigmoid(gate.float())[..., None]
+    return out.to(q.dtype)
 
 
 # --------------------------------------------------------------------------- rotary embedding

@@ -1,0 +1,391 @@
+"""Composed stacks in the rollout engine: cache, batch description, forward and scheduling.
+
+A composed stack (``ModelConfig.layer_specs``) mixes layers whose memory of the past differs in kind:
+
+* recurrent layers keep one fp32 matrix per head and sequence, in a STATE SLOT of a fixed pool (:class:`StackCache.state`);
+* latent-attention layers keep one row per token in PAGES of the engine's block manager (:class:`StackCache.latent`).
+
+One forward (:meth:`ComposedForward.forward_segments`) runs a batch of SEGMENTS - the next ``n >= 1`` tokens of several
+sequences, prompt portions beside single decoded tokens - from what earlier forwards left in slots and pages.  The engine's
+scheduler cuts prompts into portions with it; pure decode batches take the same layers through the engine's captured
+windows (:meth:`ComposedForward.forward_step`).
+"""
+from __future__ import annotations
+
+import math
+from collections import deque
+from dataclasses import dataclass
+from typing import Optional, Sequence
+
+import torch
+
+from .. import ops
+from ..models.config import ModelConfig
+
+LONG_PORTION = 192     # portions of at least this many rows attend through projected keys / values (flash attention)
+
+
+def pad_to(n: int, m: int) -> int:
+    return (n + m - 1) // m * m
+
+
+class SlotManager:
+    """Fixed pool of state slots, one per live sequence."""
+
+    def __init__(self, n: int):
+        self.n, self.free, self.used = n, deque(range(n)), set()
+
+    @property
+    def num_free(self) -> int:
+        return len(self.free)
+
+    def alloc(self) -> int:
+        if not self.free:
+            raise RuntimeError("no state slot is free")
+        s = self.free.popleft()
+        self.used.add(s)
+        return s
+
+    def release(self, s: int):
+        if s not in self.used:
+            raise RuntimeError(f"state slot {s} released twice")
+        self.used.remove(s)
+        self.free.append(s)
+
+
+class StackCache:
+    """The two pools of a composed stack.  ``latent[layer]``: ``[blocks * block_size, padded rank]`` rows in the model's
+    type; ``state[layer]``: ``[slots, heads, dim, padded vdim]`` fp32.  All of it lives in ONE buffer."""
+
+    def __init__(self, cfg: ModelConfig, num_blocks: int, block_size: int, num_slots: int, dtype, device, memory_saver: bool):
+        self.block_size = block_size
+        views, n = [], 0
+        es = torch.empty(0, dtype=dtype).element_size()
+        for i, s in enumerate(cfg.layer_specs):
+            if s.mixer == "hgrn2":
+                shape, dt, size = (num_slots, s.heads, s.dim, pad_to(s.vdim, 4)), torch.float32, 4
+            else:
+                shape, dt, size = (num_blocks * block_size, pad_to(s.kv_rank, 64)), dtype, es
+            views.append((i, s.mixer, shape, dt, n))
+            n += pad_to(math.prod(shape) * size, 1024)
+        self.nbytes = n
+        self.buf = None
+        if memory_saver:
+            from ..utils.memory_saver import PausableBuffer
+
+            self.buf = PausableBuffer(n, device)
+            make = lambda shape, dt, off: self.buf.tensor(shape, dt, off)
+        else:
+            flat = torch.zeros(n, dtype=torch.uint8, device=device)
+            make = lambda shape, dt, off: flat[off:off + math.prod(shape) * torch.empty(0, dtype=dt).element_size()].view(dt).view(shape)
+        self.latent, self.state = {}, {}
+        for i, kind, shape, dt, off in views:
+            (self.state if kind == "hgrn2" else self.latent)[i] = make(shape, dt, off)
+
+    def copy_sequence(self, src_blocks: Sequence[int], dst_blocks: Sequence[int], src_slot: int, dst_slot: int):
+        """Pages ``src -> dst`` pairwise and the whole state slot."""
+        bs = self.block_size
+        for pool in self.latent.values():
+            v = pool.view(-1, bs, pool.shape[1])
+            for a, b in zip(src_blocks, dst_blocks):
+                v[b] = v[a]
+        for st in self.state.values():
+            st[dst_slot] = st[src_slot]
+
+
+@dataclass
+class SegmentBatch:
+    """Device description of a batch of segments; the first ``long_segs`` of them (``long_rows`` rows) are long portions.
+    ``cu`` is None when every segment is a single row.  ``short_*`` describe the segments behind the long ones, with row
+    numbers counted from ``long_rows``; ``items[heads]`` are their column groups (see :func:`attention_items`)."""
+    tokens: torch.Tensor
+    slots: torch.Tensor                      # [T] row of the latent pools that each token's row goes to
+    ctx: torch.Tensor                        # [S] int32: tokens of the sequence including this segment
+    block_tables: torch.Tensor               # [S, max blocks] int32
+    state_slot: torch.Tensor                 # [S] int32
+    cu: Optional[torch.Tensor] = None        # [S + 1] int32
+    long_segs: int = 0
+    long_rows: int = 0
+    long_cu: Optional[torch.Tensor] = None   # [long + 1] int32 rows / context rows of the long segments
+    long_cu_k: Optional[torch.Tensor] = None
+    long_max: int = 0
+    ctx_slots: Optional[torch.Tensor] = None  # pool rows of the long segments' whole contexts
+    short_cu: Optional[torch.Tensor] = None
+    row_seg: Optional[torch.Tensor] = None   # [short rows] int32: segment (among the short ones) and last visible position
+    row_pos: Optional[torch.Tensor] = None
+    max_ctx: int = 0                         # host upper bound of the short segments' contexts
+    items: Optional[dict] = None
+
+
+def attention_items(lens: Sequence[int], ctx: Sequence[int], heads: int, width: int = 64) -> list:
+    """Cut the (row, head) columns of consecutive segments into groups of at most ``width`` that never span two segments:
+    ``[segment, first column, columns, base]``; the column ``c`` belongs to row ``c // heads`` and sees the first
+    ``base + c // heads`` positions."""
+    out, row0 = [], 0
+    for s, (n, L) in enumerate(zip(lens, ctx)):
+        step = width // heads * heads if heads <= width else width     # whole rows per group when a row fits
+        for c in range(row0 * heads, (row0 + n) * heads, step):
+            out.append([s, c, min(step, (row0 + n) * heads - c), L - n - row0 + 1])
+        row0 += n
+    return out
+
+
+class ComposedForward:
+    """The forward of composed stacks (mixed into :class:`relax_b200.rollout.weights.RolloutWeights`).
+
+    The residual stream is fp32.  A sublayer reads its copy in the model's type, and one kernel norms the sublayer's
+    output, adds it and writes the next copy; at the last sublayer that kernel also applies the final norm."""
+
+    def latent_dims(self, i: int) -> tuple:
+        """Padded ``(dim, vdim, rank)`` of latent layer ``i`` (16-byte rows per head, 64-column latent chunks)."""
+        s = self.cfg.layer_specs[i]
+        return pad_to(s.dim, 8), pad_to(s.vdim, 8), pad_to(s.kv_rank, 64)
+
+    @staticmethod
+    def composed_param_shapes(cfg: ModelConfig) -> dict:
+        """Every projection's output features are padded to 64 and its input features to the pitch of the rows it reads;
+        padding is zero and stays zero through every layer."""
+        Wp, Vp = pad_to(cfg.hidden_size, 64), pad_to(cfg.vocab_size, 64)
+        shapes = {"embed": (Vp, Wp)}
+        for i, s in enumerate(cfg.layer_specs):
+            p, H = f"layers.{i}.", s.heads
+            if s.mixer == "hgrn2":
+                qd, vd = H * s.dim, H * s.vdim
+                shapes[p + "rec_qfv"] = (pad_to(2 * qd + vd, 64), Wp)
+                shapes[p + "rec_f_bias"], shapes[p + "rec_lower"], shapes[p + "rec_norm"] = (qd,), (qd,), (s.vdim,)
+                shapes[p + "rec_o"] = (Wp, pad_to(vd, 8))
+            else:
+                dp, vp, Rp = pad_to(s.dim, 8), pad_to(s.vdim, 8), pad_to(s.kv_rank, 64)
+                shapes[p + "lat_qcg"] = (pad_to(H * dp + Rp + H, 64), Wp)
+                shapes[p + "lat_norm"] = (Rp,)
+                shapes[p + "lat_uk"], shapes[p + "lat_uv"] = (H * dp, Rp), (H * vp, Rp)
+                shapes[p + "lat_o"] = (Wp, H * vp)
+            shapes[p + "post_attn_norm"] = (Wp,)
+            if s.ff:
+                Fp = pad_to(s.ff, 64)
+                shapes[p + "gate_up"], shapes[p + "down"], shapes[p + "post_mlp_norm"] = (2 * Fp, Wp), (Wp, Fp), (Wp,)
+        shapes["final_norm"], shapes["lm_head"] = (Wp,), (Vp, Wp)
+        return shapes
+
+    # ------------------------------------------------------------------ mixers
+    def _hgrn2(self, i, h, b: SegmentBatch, cache: StackCache):
+        s, p, pre = self.cfg.layer_specs[i], self.p, f"layers.{i}."
+        qfv = ops.linear(h, p[pre + "rec_qfv"])
+        o = ops.hgrn2(qfv, p[pre + "rec_f_bias"], p[pre + "rec_lower"], p[pre + "rec_norm"], cache.state[i], b.state_slot,
+                      b.ctx, b.cu, s.heads, s.dim, s.vdim, self.cfg.rms_norm_eps)
+        return ops.linear(o, p[pre + "rec_o"])
+
+    def _latent(self, i, h, b: SegmentBatch, cache: StackCache):
+        """Keys and values are products of the cached latent row ``c``: ``q . (W_uk c) = (W_uk^T q) . c`` and
+        ``sum p (W_uv c) = W_uv (sum p c)``.  Single tokens and short portions therefore attend to the latent rows in
+        place, with the up-projections folded around the attention; long portions project keys and values of their whole
+        context once and run the flash kernel on them."""
+        s, p, pre = self.cfg.layer_specs[i], self.p, f"layers.{i}."
+        H, (dp, vp, Rp), pool = s.heads, self.latent_dims(i), cache.latent[i]
+        T = h.shape[0]
+        qcg = ops.linear(h, p[pre + "lat_qcg"])
+        q, gate = qcg[:, : H * dp].view(T, H, dp), qcg[:, H * dp + Rp: H * dp + Rp + H]
+        ops.latent_write(qcg[:, H * dp: H * dp + Rp], p[pre + "lat_norm"], s.kv_rank, self.cfg.rms_norm_eps, pool, b.slots)
+        uk, uv = p[pre + "lat_uk"], p[pre + "lat_uv"]
+        n = b.long_rows
+        parts = []
+        if n:
+            c = pool[b.ctx_slots]
+            k, v = ops.linear(c, uk).view(-1, H, dp), ops.linear(c, uv).view(-1, H, vp)
+            parts.append(ops.flash_gated(q[:n], k, v, b.long_cu, b.long_cu_k, s.scale, b.long_max, gate[:n]))
+        if n < T:
+            ql = ops.head_linear(q[n:], uk.view(H, dp, Rp), False)
+            o = ops.latent_attention(ql, pool, b, cache.block_size, s.scale, gate[n:])
+            parts.append(ops.head_linear(o, uv.view(H, vp, Rp), True).reshape(T - n, H * vp))
+        return ops.linear(parts[0] if len(parts) == 1 else torch.cat(parts), p[pre + "lat_o"])
+
+    # ------------------------------------------------------------------ trunk
+    def _run_composed(self, b: SegmentBatch, cache: StackCache, taps: Optional[list] = None):
+        """Final-norm output of every row.  ``taps``: a list that receives the fp32 residual stream after every layer."""
+        cfg, p = self.cfg, self.p
+        W, G, eps = cfg.hidden_size, cfg.norm_groups, cfg.rms_norm_eps
+        res, h = ops.embed_rows(b.tokens, p["embed"])
+        for i, s in enumerate(cfg.layer_specs):
+            pre = f"layers.{i}."
+            final = p["final_norm"] if i + 1 == cfg.num_layers else None
+            a = self._hgrn2(i, h, b, cache) if s.mixer == "hgrn2" else self._latent(i, h, b, cache)
+            h = ops.norm_add(res, a, p[pre + "post_attn_norm"], W, G, eps, None if s.ff else final)
+            if s.ff:
+                m = ops.linear(ops.linear_glu(h, p[pre + "gate_up"], s.act), p[pre + "down"])
+                h = ops.norm_add(res, m, p[pre + "post_mlp_norm"], W, G, eps, final)
+            if taps is not None:
+                taps.append(res[:, :W].clone())
+        return h
+
+    def forward_segments(self, b: SegmentBatch, cache: StackCache, rows: Optional[torch.Tensor], tp, taps: Optional[list] = None):
+        """Logits of the given rows (None: no row is asked for, only slots and pages are advanced)."""
+        h = self._run_composed(b, cache, taps)
+        return None if rows is None else self._logits(h[rows], tp)
+
+    def forward_step(self, tokens, block_tables, context_lens, slots, state_slot, cache: StackCache, tp):
+        """One decoded token per sequence (the captured step): everything is read from device arrays."""
+        b = SegmentBatch(tokens, slots, context_lens, block_tables, state_slot,
+                         max_ctx=block_tables.shape[1] * cache.block_size)
+        return self._logits(self._run_composed(b, cache), tp)
+
+
+class ComposedScheduler:
+    """Scheduling of composed stacks (mixed into :class:`relax_b200.rollout.engine.RolloutEngine`).
+
+    Every running request has ``fed`` tokens in its pages and state slot.  A step feeds the newest token of the requests
+    that decode and, within ``max_prefill_tokens``, the next portions of the prompts, all in one batch; a request whose
+    last known token has been fed is sampled.  When only decoding is left the engine's windowed loop takes over."""
+
+    def _release_request(self, r):
+        self.bm.release(r.blocks)
+        r.blocks = []
+        if r.state_slot is not None:
+            self.sm.release(r.state_slot)
+            r.state_slot = None
+
+    # ------------------------------------------------------------------ the step function
+    def run_segments(self, parts: Sequence[tuple], want: Sequence[Sequence[int]], taps: Optional[list] = None):
+        """One batch: ``parts[j] = (request, n)`` feeds the request's tokens ``fed .. fed + n``; ``want[j]`` are the places
+        among them whose logits are returned, ``[sum(len(w)), vocab]`` in the order of ``parts`` (None when nothing is
+        wanted).  Pages are taken as needed."""
+        if not parts or any(n < 1 for _, n in parts):
+            raise ValueError("a batch is made of segments of at least one token")
+        bs = self.block_size
+        for r, n in parts:
+            if r.state_slot is None:
+                r.state_slot = self.sm.alloc()
+            need = self.bm.blocks_for(r.fed + n)
+            while len(r.blocks) < need:
+                r.blocks.append(self.bm.alloc())
+                r._reserve = max(0, getattr(r, "_reserve", 0) - 1)
+        long_ok = self._long_portions
+        order = sorted(range(len(parts)), key=lambda j: not (long_ok and parts[j][1] >= LONG_PORTION))      # stable: long ones first
+        n_long = sum(1 for r, n in parts if long_ok and n >= LONG_PORTION)
+        toks, slots, cu, ctx, sslot, bt, rows_of = [], [], [0], [], [], [], {}
+        for j in order:
+            r, n = parts[j]
+            seq = r.prompt + r.output
+            toks += seq[r.fed:r.fed + n]
+            slots += self._slots(r, r.fed, r.fed + n)
+            rows_of[j] = cu[-1]
+            cu.append(cu[-1] + n)
+            ctx.append(r.fed + n)
+            sslot.append(r.state_slot)
+        maxb = pad_to(max(len(parts[j][0].blocks) for j in order), 8)
+        bt = [parts[j][0].blocks + [0] * (maxb - len(parts[j][0].blocks)) for j in order]
+        rows = [rows_of[j] + w for j in range(len(parts)) for w in want[j]]
+        single = all(n == 1 for _, n in parts)
+        i32, i64 = torch.int32, torch.int64
+        arrays = {"tokens": (toks, i64), "slots": (slots, i64), "ctx": (ctx, i32), "block_tables": (bt, i32), "state_slot": (sslot, i32)}
+        host = {"long_segs": n_long, "long_rows": cu[n_long], "max_ctx": max(ctx[n_long:], default=0)}
+        heads = []
+        if not single:
+            arrays["cu"] = (cu, i32)
+            lens = [b - a for a, b in zip(cu, cu[1:])]
+            sl, sc = lens[n_long:], ctx[n_long:]
+            if n_long:
+                arrays["long_cu"] = (cu[:n_long + 1], i32)
+                ck = [0]
+                for c in ctx[:n_long]:
+                    ck.append(ck[-1] + c)
+                arrays["long_cu_k"] = (ck, i32)
+                arrays["ctx_slots"] = ([x for j in order[:n_long] for x in self._slots(parts[j][0], 0, parts[j][0].fed + parts[j][1])], i64)
+                host["long_max"] = max(lens[:n_long])
+            if sl:
+                arrays["short_cu"] = ([c - cu[n_long] for c in cu[n_long:]], i32)
+                arrays["row_seg"] = ([s for s, n in enumerate(sl) for _ in range(n)], i32)
+                arrays["row_pos"] = ([c - n + k for n, c in zip(sl, sc) for k in range(n)], i32)
+                heads = sorted({self.cfg.layer_specs[i].heads for i in self.cfg.layers_with("latent_attention")})
+                for H in heads:
+                    arrays[f"items{H}"] = (attention_items(sl, sc, H), i32)
+        if rows:
+            arrays["rows"] = (rows, i64)
+        dev = dict(zip(arrays, self._stage(list(arrays.values()))))
+        want_t = dev.pop("rows", None)
+        items = {H: dev.pop(f"items{H}") for H in heads}
+        batch = SegmentBatch(**dev, **host, items=items or None)
+        logits = self.weights.forward_segments(batch, self.kv, want_t, self.tp, taps)
+        for r, n in parts:
+            r.fed += n
+        return logits
+
+    # ------------------------------------------------------------------ sequences driven from outside (trace replay)
+    def open_sequence(self):
+        """A sequence whose tokens are given step by step (:meth:`feed`) instead of being sampled."""
+        from .engine import Request, SamplingParams
+
+        r = Request(self._next_rid, [], SamplingParams())
+        self._next_rid += 1
+        r.status = "running"
+        return r
+
+    @torch.no_grad()
+    def feed(self, entries: Sequence[tuple]):
+        """``entries[j] = (sequence, its next tokens, wanted places)``; returns the wanted rows of logits (or None)."""
+        for r, tokens, _ in entries:
+            bad = [t for t in tokens if not 0 <= t < self.cfg.vocab_size]
+            if bad:
+                raise ValueError(f"token {bad[0]} is outside the vocabulary of {self.cfg.vocab_size}")
+            r.prompt.extend(tokens)
+        z = self.run_segments([(r, len(t)) for r, t, _ in entries], [w for _, _, w in entries])
+        return None if z is None else z[:, : self.cfg.vocab_size]
+
+    def close_sequence(self, r):
+        self._release_request(r)
+        r.status = "finished"
+
+    # ------------------------------------------------------------------ generation
+    def _step_composed(self):
+        for r in self._admit():
+            r.state_slot = self.sm.alloc()
+            self.running.append(r)
+        live = [r for r in self.running if r._lead is None or r.fed > 0]      # followers wait for their leader's prompt
+        if not live:
+            return
+        if all(r.num_tokens - r.fed == 1 and r.output for r in self.running):
+            if self.windowed_decode and self._decode_window():
+                for r in self.running:
+                    if r.status == "running":
+                        r.fed = r.num_tokens - 1
+                return
+        budget = self.max_prefill_tokens
+        parts = []
+        for r in live:      # decoding requests first, then prompt portions in order of arrival
+            if r.num_tokens - r.fed == 1:
+                parts.append((r, 1))
+                budget -= 1
+        budget = max(budget, self.block_size)      # prompts advance however many requests decode
+        for r in live:
+            left = r.num_tokens - r.fed
+            if left > 1 and budget > 0:
+                n = min(left, budget)
+                parts.append((r, n))
+                budget -= n
+        done = [(r, n) for r, n in parts if r.fed + n == r.num_tokens]
+        want = [[n - 1] if r.fed + n == r.num_tokens else [] for r, n in parts]
+        first = {id(r) for r, _ in done if not r.output}
+        logits = self.run_segments(parts, want)
+        self.stats["prefill_tokens"] += sum(n for r, n in parts if not (r.output and n == 1))
+        self.stats["decode_tokens"] += sum(1 for r, n in parts if r.output and n == 1)
+        if not done:
+            return
+        reqs, pick = [r for r, _ in done], list(range(len(done)))
+        for k, (r, _) in enumerate(done):
+            for f in [f for f in self.running if f._lead is r and f.fed == 0]:
+                # same prompt: same latent rows (full pages are shared already) and same states; sampled from the same row
+                shared = f.cached_tokens // self.block_size
+                self.kv.copy_sequence(r.blocks[shared:len(f.blocks)], f.blocks[shared:], r.state_slot, f.state_slot)
+                f.fed = r.fed
+                self.stats["cached_tokens"] += len(f.prompt)
+                first.add(id(f))
+                reqs.append(f)
+                pick.append(k)
+        if len(pick) > len(done):
+            logits = logits[torch.tensor(pick, device=self.device)]
+        import time
+
+        now = time.perf_counter()
+        for r in reqs:
+            if id(r) in first:
+                r.t_first = now
+        self._sample_and_append(reqs, logits)

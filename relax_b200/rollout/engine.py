@@ -25,6 +25,7 @@ import torch.distributed as dist
 from .. import ops
 from ..models.config import ModelConfig
 from ..parallel.state import GroupInfo
+from .composed import ComposedScheduler, SlotManager, StackCache
 from .speculative import SpeculativeMixin
 from .weights import RolloutWeights
 
@@ -53,6 +54,9 @@ class Request:
     finish_reason: Optional[str] = None
     weight_versions: list = field(default_factory=list)
     cached_tokens: int = 0
+    # composed stacks: tokens whose latent rows / states are in the cache, and the slot of the recurrent states
+    fed: int = 0
+    state_slot: Optional[int] = None
     # with ``return_routed_experts``: per context position that was fed to the model, the expert ids every MoE layer
     # chose - a list of ``[L_moe, k]`` int lists (positions 0 .. num_tokens - 2; the last token is never fed)
     routed_experts: list = field(default_factory=list)
@@ -112,15 +116,21 @@ class BlockManager:
         return (ntokens + self.block_size - 1) // self.block_size
 
 
-class RolloutEngine(SpeculativeMixin):
+class RolloutEngine(SpeculativeMixin, ComposedScheduler):
     def __init__(self, cfg: ModelConfig, tp: Optional[GroupInfo] = None, device="cpu", dtype=None,
                  num_kv_blocks: int = 256, block_size: int = 16, max_running: int = 256,
                  max_prefill_tokens: int = 16384, seed: int = 42, eos_token_id: Optional[int] = None,
                  use_cuda_graph: bool = True, max_model_len: int = 4096, memory_saver: Optional[bool] = None,
                  decode_window: Optional[int] = None, windowed_decode: Optional[bool] = None,
                  weights_shared_path: Optional[str] = None, ep: Optional[GroupInfo] = None,
-                 return_routed_experts: bool = False, speculative: bool = False, speculative_steps: int = 1):
+                 return_routed_experts: bool = False, speculative: bool = False, speculative_steps: int = 1,
+                 state_slots: Optional[int] = None):
+        """``state_slots``: most sequences that may be live at once in a composed stack (recurrent states; default
+        ``max_running``)."""
         self.cfg = cfg
+        self.composed = cfg.is_composed
+        if self.composed and (speculative or return_routed_experts):
+            raise NotImplementedError("composed stacks serve without speculative decoding and have no routed experts")
         # speculative decoding drafted by the model's multi-token-prediction block (rollout/speculative.py)
         self.speculative = bool(speculative)
         self.speculative_steps = max(1, int(speculative_steps))      # proposals per verify pass (the block is chained)
@@ -160,6 +170,13 @@ class RolloutEngine(SpeculativeMixin):
         self.weight_version = 0
         self.gen = torch.Generator(device="cpu").manual_seed(seed)
         self.kv = None
+        if self.composed:
+            self.max_running = min(max_running, state_slots or max_running)
+            self.sm = SlotManager(self.max_running + 1)
+            self._scratch_slot = self.sm.alloc()      # padding rows of a graph bucket; never handed to a request
+            # flash attention on projected keys / values: the tensor-core kernel takes bf16 heads of up to 128 features
+            self._long_portions = self.device.type == "cuda" and all(
+                ops.flash_serves_dims(self.dtype, *self.weights.latent_dims(i)[:2]) for i in cfg.layers_with("latent_attention"))
         self._alloc_kv()
         self.use_cuda_graph = use_cuda_graph and self.device.type == "cuda"
         self.max_model_len = max_model_len
@@ -191,6 +208,13 @@ class RolloutEngine(SpeculativeMixin):
     # ------------------------------------------------------------------ memory
     def _alloc_kv(self):
         c = self.cfg
+        if self.composed:
+            if self._kv_buf is not None:
+                self._kv_buf.resume()
+            else:
+                self.kv = StackCache(c, self.bm.num_blocks, self.block_size, self.sm.n, self.dtype, self.device, self.memory_saver)
+                self._kv_buf = self.kv.buf
+            return
         hkv = c.num_query_groups // self.tp.size
         # with speculative decoding the draft block keeps its own cache as one more layer under the same block tables
         shape = (c.num_layers + (1 if self.speculative else 0), 2, self.bm.num_blocks, self.block_size, hkv, c.head_dim)
@@ -256,6 +280,9 @@ class RolloutEngine(SpeculativeMixin):
         if self.running:
             raise RuntimeError("flush_cache with running requests")
         self.bm = BlockManager(self.bm.num_blocks, self.block_size)
+        if self.composed:
+            self.sm = SlotManager(self.sm.n)
+            self._scratch_slot = self.sm.alloc()
         if self.use_cuda_graph or self.windowed_decode:
             self._scratch_block = self.bm.alloc()
         for st in self._graphs.values():     # device-resident batch state refers to blocks of the old manager
@@ -310,8 +337,7 @@ class RolloutEngine(SpeculativeMixin):
         """Stop every request; running ones are returned with their partial output."""
         out = []
         for r in self.running:
-            self.bm.release(r.blocks)
-            r.blocks = []
+            self._release_request(r)
             r.status, r.finish_reason = "aborted", "abort"
             out.append(r)
         for r in self.waiting:
@@ -331,6 +357,8 @@ class RolloutEngine(SpeculativeMixin):
         admitted, budget = [], self.max_prefill_tokens
         leaders: dict = {}
         while self.waiting and len(self.running) + len(admitted) < self.max_running:
+            if self.composed and self.sm.num_free <= len(admitted):
+                break      # sequences driven from outside hold state slots too
             r = self.waiting[0]
             ctx = r.num_tokens
             need_total = self.bm.blocks_for(len(r.prompt) + r.params.max_new_tokens)
@@ -340,7 +368,7 @@ class RolloutEngine(SpeculativeMixin):
             reserved = sum(getattr(x, "_reserve", 0) for x in self.running) + sum(getattr(x, "_reserve", 0) for x in admitted)
             if need > self.bm.num_free - reserved:
                 break
-            if lead is None and ctx > budget and admitted:
+            if lead is None and ctx > budget and admitted and not self.composed:      # composed stacks cut prompts into portions
                 break
             self.waiting.popleft()
             r._lead = lead
@@ -372,8 +400,10 @@ class RolloutEngine(SpeculativeMixin):
         if self.paused:
             return []
         self.stats["steps"] += 1
-        new = self._admit()
-        if new:
+        new = [] if self.composed else self._admit()
+        if self.composed:
+            self._step_composed()
+        elif new:
             self._prefill(new)
             self.running.extend(new)
         elif self.running:
@@ -382,8 +412,7 @@ class RolloutEngine(SpeculativeMixin):
         if done:
             self.running = [r for r in self.running if r.status != "finished"]
             for r in done:
-                self.bm.release(r.blocks)
-                r.blocks = []
+                self._release_request(r)
                 r._reserve = 0
                 r.t_done = time.perf_counter()
         return done
@@ -600,7 +629,7 @@ class RolloutEngine(SpeculativeMixin):
         per_batch = [("tok", i64, (bucket,)), ("pos", i64, (bucket,)), ("slots", i64, (bucket,)), ("topk", i64, (bucket,)),
                      ("eos", i64, (bucket,)), ("stop", i64, (bucket, self.N_STOP)), ("ctx", i32, (bucket,)),
                      ("active", i32, (bucket,)), ("remain", i32, (bucket,)), ("bt", i32, (bucket, maxb)),
-                     ("temp", f32, (bucket,)), ("topp", f32, (bucket,)), ("delta", i64, (bucket,))]
+                     ("temp", f32, (bucket,)), ("topp", f32, (bucket,)), ("delta", i64, (bucket,)), ("sslot", i32, (bucket,))]
         offs, n = {}, 0
         for name, dt, shp in per_window + per_batch:
             if name == "tok":
@@ -641,7 +670,8 @@ class RolloutEngine(SpeculativeMixin):
             # rotary position = cache position + the row's offset (non-zero after an image: M-RoPE advances by the
             # largest grid side, not by the number of placeholder tokens)
             rope_pos = d["pos"] + d["delta"] if self.cfg.mrope_section is not None else d["pos"]
-            logits = self.weights.forward_decode(d["tok"], rope_pos, d["bt"], d["ctx"], d["slots"], self.kv, self.tp)
+            logits = self.weights.forward_step(d["tok"], d["bt"], d["ctx"], d["slots"], d["sslot"], self.kv, self.tp) \
+                if self.composed else self.weights.forward_decode(d["tok"], rope_pos, d["bt"], d["ctx"], d["slots"], self.kv, self.tp)
             if self.return_routed_experts:      # ring slot = the step counter, read on the device (before it advances)
                 routed = torch.stack(self.weights.routing_capture, 1).to(torch.int32)
                 self.weights.routing_capture = None
@@ -669,6 +699,7 @@ class RolloutEngine(SpeculativeMixin):
         h["tok"][lo:hi] = 0
         h["pos"][lo:hi] = 0
         h["delta"][lo:hi] = 0
+        h["sslot"][lo:hi] = self._scratch_slot if self.composed else 0
         h["ctx"][lo:hi] = 1
         h["bt"][lo:hi] = self._scratch_block
         h["slots"][lo:hi] = self._scratch_block * bs
@@ -714,6 +745,8 @@ class RolloutEngine(SpeculativeMixin):
             h["delta"][:B] = torch.tensor([r.pos_delta for r in reqs], dtype=torch.int64)
             h["slots"][:B] = torch.tensor([r.blocks[p // bs] * bs + p % bs for r, p in zip(reqs, npos)], dtype=torch.int64)
             h["bt"][:B] = torch.tensor([r.blocks + [self._scratch_block] * (maxb - len(r.blocks)) for r in reqs], dtype=torch.int32)
+            if self.composed:
+                h["sslot"][:B] = torch.tensor([r.state_slot for r in reqs], dtype=torch.int32)
             h["temp"][:B] = torch.tensor([r.params.temperature for r in reqs], dtype=torch.float32)
             h["topk"][:B] = torch.tensor([r.params.top_k for r in reqs], dtype=torch.int64)
             h["topp"][:B] = torch.tensor([r.params.top_p for r in reqs], dtype=torch.float32)

@@ -26,6 +26,7 @@ import torch.distributed as dist
 from .. import ops
 from ..models.config import ModelConfig
 from ..parallel.state import GroupInfo
+from .composed import ComposedForward
 
 
 GDN_CONV_KERNEL = 4      # taps of the Gated-DeltaNet depth-wise convolution (relax_b200/models/gdn.py)
@@ -35,6 +36,8 @@ def rollout_param_shapes(cfg: ModelConfig, tp: int, ep: int = 1, mtp: bool = Fal
     """``mtp``: the buffer also holds the first multi-token-prediction block (draft model of speculative decoding) -
     its transformer layer as layer ``num_layers`` and ``mtp.enorm / mtp.hnorm / mtp.eh_proj / mtp.final_norm`` - AFTER
     everything else, so that the offsets of the policy's own tensors do not depend on the switch."""
+    if cfg.is_composed:
+        return ComposedForward.composed_param_shapes(cfg)
     hd, H = cfg.head_dim, cfg.hidden_size
     nq, nkv = cfg.num_attention_heads // tp, cfg.num_query_groups // tp
     v_pad = (cfg.vocab_size + tp - 1) // tp * tp
@@ -122,9 +125,11 @@ def rollout_layout(cfg: ModelConfig, tp: int, ep: int = 1, mtp: bool = False):
     return shapes, offsets, n
 
 
-class RolloutWeights:
+class RolloutWeights(ComposedForward):
     def __init__(self, cfg: ModelConfig, tp_size: int, tp_rank: int, device, dtype, ep_size: int = 1, ep_rank: int = 0,
                  memory_saver: bool = False, shared_path: Optional[str] = None, mtp: bool = False):
+        if cfg.is_composed and (tp_size > 1 or ep_size > 1 or mtp):
+            raise NotImplementedError("composed stacks run on one rank per engine, without speculative decoding")
         if (cfg.linear_attention_freq > 0 or cfg.attention_output_gate or cfg.dsa_topk > 0 or cfg.multi_latent_attention) \
                 and (tp_size > 1 or ep_size > 1 or mtp):
             raise NotImplementedError("stacks with Gated-DeltaNet, gated-attention or latent-attention (MLA / DSA) layers run on "
