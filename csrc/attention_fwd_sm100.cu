@@ -219,9 +219,12 @@ fa_fwd_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant__
         if (!mbar_wait(bar_o, static_cast<uint32_t>(j - 1) & 1, abort_flag, p.err)) { ok = false; break; }
         tc_fence_after();
       }
-      if (mx > m_ref + 8.f) {
-        const float alpha = exp2f(m_ref - mx);
-        m_ref = mx;
+      // rows grow independently, but the TMEM accesses below are warp-wide (.sync.aligned): the branch is taken by the
+      // whole warp when any of its rows needs it, and rows that do not are scaled by one
+      const bool grow = mx > m_ref + 8.f;
+      if (__any_sync(0xffffffffu, grow)) {
+        const float alpha = grow ? exp2f(m_ref - mx) : 1.f;
+        if (grow) m_ref = mx;
         l *= alpha;
         if (j > 0) {
 #pragma unroll 1

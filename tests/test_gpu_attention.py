@@ -48,6 +48,22 @@ def test_flash_attention_forward(lens, Hq, Hkv, causal):
     C.check_error_flag()
 
 
+def test_flash_attention_rows_whose_maximum_jumps_late():
+    """Single rows of a warp meet a score far above their running maximum in a late block (the accumulator is rescaled in
+    TMEM for those rows only), others never do."""
+    from relax_b200 import ops
+    from relax_b200.ops import reference as R
+
+    C = _C()
+    q, k, v, cu, _ = _mk([700], [700], 2, 2, 11)
+    for row, key in ((400, 300), (401, 20), (517, 500), (699, 650), (640, 10)):
+        k[key] = q[row] * 3
+    o = ops.attention_varlen(q, k, v, cu, causal=True)
+    ref = R.attention_varlen(q.float(), k.float(), v.float(), cu, causal=True)
+    _close(o, ref, 2e-2, 2e-2, "fwd late maximum")
+    C.check_error_flag()
+
+
 def test_flash_attention_query_shorter_than_keys():
     """Chunked prefill / CP layout: queries are the tail of the key sequence (bottom-right causal)."""
     from relax_b200 import ops
