@@ -44,6 +44,7 @@ int rb_fp8_block_dequant(const void* q, const float* scale, void* out, int M, in
 #ifdef TORCH_EXTENSION_NAME
 #include <pybind11/pybind11.h>
 void register_more(pybind11::module_& m);
+void register_serving(pybind11::module_& m);
 #endif
 
 // ---- attention / decode / sampling / fused LM head (declared again for C callers)
@@ -118,7 +119,7 @@ int rb_grouped_gemm_dgrad(const void* dY, const void* W, void* dX, const int* ti
 int rb_grouped_gemm_wgrad(const void* dY, const void* X, void* dW, const int* expert_rows, int rows_cap, int Nw, int Kw,
                           int E, int out_fp32, int accumulate, int* err, cudaStream_t st);
 int rb_decode_gemm_splits(int tiles, int k_iters);
-int rb_decode_gemm(const void* x, const void* W, void* y, int Mt, int N, int K, int ldx, int ldw, int swiglu, int splits,
+int rb_decode_gemm(const void* x, const void* W, void* y, int Mt, int N, int K, int ldx, int ldw, int glu, int splits,
                    int* err, cudaStream_t st);
 int rb_policy_loss(const float* ppo_kl, const float* adv, float* loss, float* clipfrac, float* dkl, long long n, float eps_clip,
                    float eps_clip_high, float eps_clip_c, cudaStream_t st);
@@ -128,6 +129,22 @@ int rb_lm_head_logprob(const void* h, const void* W, const long long* targets, f
 int rb_lm_head_dlogits(const void* h, const void* W, const long long* targets, const float* row_stats, const float* g_lp,
                        const float* g_ent, void* dlogits, int M, int N, int K, int ldh, int ldw, int ldd, int vocab_start,
                        float inv_temp, int* err, cudaStream_t stream);
+// ---- composed stacks (stack_sm100.cu); fp32 = 1: 32-bit operands, 0: bf16
+int rb_embed_rows(const long long* tok, const void* w, float* res, void* h, int rows, int vocab, int pitch, int fp32, cudaStream_t st);
+int rb_norm_add(float* res, const void* y, const void* w, const void* next_w, void* h, int rows, int ldy, int pitch, int width,
+                int groups, float eps, int fp32, cudaStream_t st);
+int rb_hgrn2(const void* qfv, const void* f_bias, const void* lower, const void* norm_w, float* state, const int* slot, const int* ctx,
+             const int* cu, float* o_raw, void* out, int rows, int segs, int H, int dim, int vdim, int vp, int ld, int ldo, float eps,
+             int fp32, cudaStream_t st);
+int rb_latent_write(const void* raw, int ld_raw, const void* w, void* pool, const long long* slots, long long pool_rows, int rows,
+                    int rank, int pitch, float eps, int fp32, cudaStream_t st);
+int rb_latent_attn(const void* q, const void* pool, const int* block_tables, const int* row_seg, const int* row_pos, const int* ctx,
+                   const void* gate, void* out, int rows, int H, int R, int max_blocks, int block_size, int ld_gate, float scale,
+                   int fp32, cudaStream_t st);
+int rb_gate_heads(const void* o, const void* gate, int ld_gate, void* out, int rows, int H, int dv, cudaStream_t st);
+int rb_glu(const void* in, void* out, long long rows, int F, int ld_in, int act, int fp32, cudaStream_t st);
+int rb_simt_gemm(const void* A, const void* B, void* C, int M, int N, int K, int lda, int ldb, int ldc, int b_kn, int batch, long long sa,
+                 long long sb, long long sc, int fp32, cudaStream_t st);
 #ifdef __cplusplus
 }
 #endif

@@ -59,34 +59,7 @@ inline const void* optptr(const c10::optional<torch::Tensor>& t) { return t.has_
 
 #define CHECK_CUDA_CONTIG(t) TORCH_CHECK((t).is_cuda() && (t).is_contiguous(), #t " must be a contiguous CUDA tensor")
 
-void gemm(torch::Tensor A, torch::Tensor B, torch::Tensor C, c10::optional<torch::Tensor> bias, int64_t M, int64_t N,
-          int64_t K, int64_t lda, int64_t ldb, int64_t ldc, bool a_mn, bool b_mn, bool accumulate, int64_t force_bn,
-          int64_t lbo_a, int64_t sbo_a, int64_t lbo_b, int64_t sbo_b, torch::Tensor err) {
-  const c10::cuda::CUDAGuard guard(A.device());
-  TORCH_CHECK(A.scalar_type() == B.scalar_type(), "A/B dtype mismatch");
-  const bool fp16 = A.scalar_type() == at::kHalf;
-  TORCH_CHECK(fp16 || A.scalar_type() == at::kBFloat16, "gemm inputs must be bf16 or fp16");
-  const bool out_fp32 = C.scalar_type() == at::kFloat;
-  TORCH_CHECK(out_fp32 || C.scalar_type() == A.scalar_type(), "output must be fp32 or the input dtype");
-  check(rb_gemm(A.data_ptr(), B.data_ptr(), C.data_ptr(), optptr(bias), (int)M, (int)N, (int)K, (int)lda, (int)ldb,
-                (int)ldc, a_mn, b_mn, out_fp32, accumulate, fp16, (int)force_bn, (int)lbo_a, (int)sbo_a, (int)lbo_b,
-                (int)sbo_b, err.data_ptr<int>(), cur_stream()),
-        "rb_gemm");
-}
 
-// CTA-pair kernel; returns false when the problem does not qualify (the caller then uses `gemm`).
-bool gemm_pair(torch::Tensor A, torch::Tensor B, torch::Tensor C, int64_t M, int64_t N, int64_t K, int64_t lda, int64_t ldb,
-               int64_t ldc, bool a_mn, bool b_mn, bool accumulate, int64_t force_bn, torch::Tensor err) {
-  const c10::cuda::CUDAGuard guard(A.device());
-  TORCH_CHECK(A.scalar_type() == at::kBFloat16 && B.scalar_type() == at::kBFloat16, "gemm_pair inputs must be bf16");
-  const bool out_fp32 = C.scalar_type() == at::kFloat;
-  TORCH_CHECK(out_fp32 || C.scalar_type() == at::kBFloat16, "output must be fp32 or bf16");
-  const int rc = rb_gemm_pair(A.data_ptr(), B.data_ptr(), C.data_ptr(), (int)M, (int)N, (int)K, (int)lda, (int)ldb, (int)ldc,
-                              a_mn, b_mn, out_fp32, accumulate, (int)force_bn, err.data_ptr<int>(), cur_stream());
-  if (rc == -20) return false;
-  check(rc, "rb_gemm_pair");
-  return true;
-}
 
 void rmsnorm_fwd(torch::Tensor x, c10::optional<torch::Tensor> res, torch::Tensor w, torch::Tensor y,
                  c10::optional<torch::Tensor> r_out, int64_t rows, int64_t cols, double eps) {
@@ -171,10 +144,6 @@ void fp8_block_dequant(torch::Tensor q, torch::Tensor scale, torch::Tensor out, 
 
 PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("install_crash_handler", &install_crash_handler);
-  m.def("launch_count", []() { return (int64_t)rb_launch_count(); });
-  m.def("reset_launch_count", []() { rb_reset_launch_count(); });
-  m.def("gemm", &gemm);
-  m.def("gemm_pair", &gemm_pair);
   m.def("rmsnorm_fwd", &rmsnorm_fwd);
   m.def("rmsnorm_bwd_parts", &rmsnorm_bwd_parts);
   m.def("rmsnorm_bwd", &rmsnorm_bwd);
@@ -188,5 +157,6 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("int4_fake_quant", &int4_fake_quant);
   m.def("fp8_block_cast", &fp8_block_cast);
   m.def("fp8_block_dequant", &fp8_block_dequant);
+  register_serving(m);
   register_more(m);
 }

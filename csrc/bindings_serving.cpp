@@ -1,0 +1,252 @@
+// Bindings of what the rollout engine's serving path launches: matrix products, prefill attention, sampling, the decode
+// advance, and the kernels of composed stacks.  They are part of the full extension and, alone, of the small
+// serving extension (module_serving.cpp).
+#include <ATen/cuda/CUDAContext.h>
+#include <c10/cuda/CUDAGuard.h>
+#include <torch/extension.h>
+
+#include "api.h"
+#include "host_utils.h"
+
+namespace {
+// Also clears this thread's "last error" slot (an unrelated, already handled status must not look like a launch failure).
+inline cudaStream_t cur_stream() {
+  (void)cudaGetLastError();
+  return at::cuda::getCurrentCUDAStream().stream();
+}
+inline void check(int rc, const char* what) {
+  if (rc != 0) {
+    char buf[160];
+    snprintf(buf, sizeof(buf), "%s failed with code %d (%s)", what, rc, rc > 0 ? cudaGetErrorString((cudaError_t)rc) : "argument check");
+    fprintf(stderr, "[relax_b200] %s\n", buf);
+    throw std::runtime_error(buf);
+  }
+}
+inline const void* optptr(const c10::optional<torch::Tensor>& t) { return t.has_value() ? t->data_ptr() : nullptr; }
+inline const int* optint(const c10::optional<torch::Tensor>& t) { return t.has_value() ? t->data_ptr<int>() : nullptr; }
+// composed stacks run in bf16 or in fp32
+inline int is_fp32(const torch::Tensor& t) {
+  TORCH_CHECK(t.scalar_type() == at::kFloat || t.scalar_type() == at::kBFloat16, "bf16 or fp32 expected, got ", t.scalar_type());
+  return t.scalar_type() == at::kFloat;
+}
+inline void check_same(const torch::Tensor& a, const torch::Tensor& b, const char* what) {
+  TORCH_CHECK(a.scalar_type() == b.scalar_type() && a.device() == b.device(), what, ": operands differ in type or device");
+}
+
+void gemm(torch::Tensor A, torch::Tensor B, torch::Tensor C, c10::optional<torch::Tensor> bias, int64_t M, int64_t N,
+          int64_t K, int64_t lda, int64_t ldb, int64_t ldc, bool a_mn, bool b_mn, bool accumulate, int64_t force_bn,
+          int64_t lbo_a, int64_t sbo_a, int64_t lbo_b, int64_t sbo_b, torch::Tensor err) {
+  const c10::cuda::CUDAGuard guard(A.device());
+  TORCH_CHECK(A.scalar_type() == B.scalar_type(), "A/B dtype mismatch");
+  const bool fp16 = A.scalar_type() == at::kHalf;
+  TORCH_CHECK(fp16 || A.scalar_type() == at::kBFloat16, "gemm inputs must be bf16 or fp16");
+  const bool out_fp32 = C.scalar_type() == at::kFloat;
+  TORCH_CHECK(out_fp32 || C.scalar_type() == A.scalar_type(), "output must be fp32 or the input dtype");
+  check(rb_gemm(A.data_ptr(), B.data_ptr(), C.data_ptr(), optptr(bias), (int)M, (int)N, (int)K, (int)lda, (int)ldb,
+                (int)ldc, a_mn, b_mn, out_fp32, accumulate, fp16, (int)force_bn, (int)lbo_a, (int)sbo_a, (int)lbo_b,
+                (int)sbo_b, err.data_ptr<int>(), cur_stream()),
+        "rb_gemm");
+}
+// CTA-pair kernel; returns false when the problem does not qualify (the caller then uses `gemm`).
+bool gemm_pair(torch::Tensor A, torch::Tensor B, torch::Tensor C, int64_t M, int64_t N, int64_t K, int64_t lda, int64_t ldb,
+               int64_t ldc, bool a_mn, bool b_mn, bool accumulate, int64_t force_bn, torch::Tensor err) {
+  const c10::cuda::CUDAGuard guard(A.device());
+  TORCH_CHECK(A.scalar_type() == at::kBFloat16 && B.scalar_type() == at::kBFloat16, "gemm_pair inputs must be bf16");
+  const bool out_fp32 = C.scalar_type() == at::kFloat;
+  TORCH_CHECK(out_fp32 || C.scalar_type() == at::kBFloat16, "output must be fp32 or bf16");
+  const int rc = rb_gemm_pair(A.data_ptr(), B.data_ptr(), C.data_ptr(), (int)M, (int)N, (int)K, (int)lda, (int)ldb, (int)ldc,
+                              a_mn, b_mn, out_fp32, accumulate, (int)force_bn, err.data_ptr<int>(), cur_stream());
+  if (rc == -20) return false;
+  check(rc, "rb_gemm_pair");
+  return true;
+}
+void fa_fwd(torch::Tensor q, torch::Tensor k, torch::Tensor v, torch::Tensor o, torch::Tensor lse, torch::Tensor cu_q,
+            torch::Tensor cu_k, int64_t max_q_blocks, bool causal, double scale, torch::Tensor err) {
+  const c10::cuda::CUDAGuard guard(q.device());
+  TORCH_CHECK(q.scalar_type() == at::kBFloat16 && q.size(2) == 128, "flash attention: bf16, head_dim 128");
+  TORCH_CHECK(q.stride(2) == 1 && k.stride(2) == 1 && v.stride(2) == 1, "head dimension must be contiguous");
+  check(rb_fa_fwd(q.data_ptr(), k.data_ptr(), v.data_ptr(), o.data_ptr(), lse.data_ptr<float>(), cu_q.data_ptr<int>(),
+                  cu_k.data_ptr<int>(), (int)cu_q.numel() - 1, (int)q.size(0), (int)k.size(0), (int)q.size(1),
+                  (int)k.size(1), q.stride(0), q.stride(1), k.stride(0), k.stride(1), v.stride(0), v.stride(1), causal,
+                  (float)scale, (int)max_q_blocks, err.data_ptr<int>(), cur_stream()),
+        "rb_fa_fwd");
+}
+void sample_v2(torch::Tensor logits, torch::Tensor temperature, torch::Tensor top_k, torch::Tensor top_p,
+               torch::Tensor uniform, torch::Tensor tok, torch::Tensor logp, int64_t V) {
+  const c10::cuda::CUDAGuard guard(logits.device());
+  TORCH_CHECK(logits.dim() == 2 && logits.stride(1) == 1, "sample: logits rows must be contiguous");
+  const bool bf = logits.scalar_type() == at::kBFloat16;
+  TORCH_CHECK(bf || logits.scalar_type() == at::kFloat, "sample: bf16 or fp32 logits");
+  check(rb_sample_v2(logits.data_ptr(), bf ? 1 : 0, (int)logits.size(0), (int)V, (long long)logits.stride(0),
+                     temperature.data_ptr<float>(), (const long long*)top_k.data_ptr<int64_t>(), top_p.data_ptr<float>(),
+                     uniform.data_ptr<float>(), (long long*)tok.data_ptr<int64_t>(), logp.data_ptr<float>(), cur_stream()),
+        "rb_sample_v2");
+}
+void decode_advance(torch::Tensor tok_new, torch::Tensor lp_new, torch::Tensor tok_in, torch::Tensor pos, torch::Tensor ctx,
+                    torch::Tensor slot, torch::Tensor block_table, int64_t block_size, torch::Tensor active,
+                    torch::Tensor remain, torch::Tensor eos, torch::Tensor stop_ids, torch::Tensor out_tok,
+                    torch::Tensor out_lp, torch::Tensor counter, torch::Tensor u_all, torch::Tensor u_next) {
+  const c10::cuda::CUDAGuard guard(tok_new.device());
+  const int B = (int)tok_in.size(0);
+  TORCH_CHECK(block_table.dim() == 2 && block_table.size(0) == B && block_table.is_contiguous(), "block table [B, max_blocks]");
+  TORCH_CHECK(out_tok.dim() == 2 && out_tok.size(1) == B && out_tok.is_contiguous() && out_lp.is_contiguous(), "window ring [W, B]");
+  TORCH_CHECK(u_all.dim() == 2 && u_all.size(0) == out_tok.size(0) && u_all.size(1) == B && u_all.is_contiguous(), "u_all [W, B]");
+  TORCH_CHECK(stop_ids.dim() == 2 && stop_ids.size(0) == B && stop_ids.is_contiguous(), "stop ids [B, n]");
+  check(rb_decode_advance((const long long*)tok_new.data_ptr<int64_t>(), lp_new.data_ptr<float>(),
+                          (long long*)tok_in.data_ptr<int64_t>(), (long long*)pos.data_ptr<int64_t>(), ctx.data_ptr<int>(),
+                          (long long*)slot.data_ptr<int64_t>(), block_table.data_ptr<int>(), (int)block_table.size(1),
+                          (int)block_size, active.data_ptr<int>(), remain.data_ptr<int>(),
+                          (const long long*)eos.data_ptr<int64_t>(), (const long long*)stop_ids.data_ptr<int64_t>(),
+                          (int)stop_ids.size(1), (long long*)out_tok.data_ptr<int64_t>(), out_lp.data_ptr<float>(),
+                          counter.data_ptr<int>(), (int)out_tok.size(0), u_all.data_ptr<float>(), u_next.data_ptr<float>(), B,
+                          cur_stream()),
+        "rb_decode_advance");
+}
+// Weight-streaming decode GEMM; returns false when the shape is outside its range (the caller uses the split-K path).
+bool decode_gemm(torch::Tensor x, torch::Tensor W, torch::Tensor y, int64_t glu, int64_t splits, torch::Tensor err) {
+  const c10::cuda::CUDAGuard guard(x.device());
+  TORCH_CHECK(x.scalar_type() == at::kBFloat16 && W.scalar_type() == at::kBFloat16 && y.scalar_type() == at::kBFloat16, "bf16 only");
+  TORCH_CHECK(x.dim() == 2 && W.dim() == 2 && x.stride(1) == 1 && W.stride(1) == 1 && y.is_contiguous(), "row-major operands");
+  const int rc = rb_decode_gemm(x.data_ptr(), W.data_ptr(), y.data_ptr(), (int)x.size(0), (int)W.size(0), (int)x.size(1),
+                                (int)x.stride(0), (int)W.stride(0), (int)glu, (int)splits, err.data_ptr<int>(), cur_stream());
+  if (rc == -20) return false;
+  check(rc, "rb_decode_gemm");
+  return true;
+}
+std::tuple<int64_t, int64_t> gemm_splitk_plan(int64_t M, int64_t N, int64_t K) {
+  int bn = 0;
+  const int s = rb_gemm_splitk_plan((int)M, (int)N, (int)K, &bn);
+  return {s, bn};
+}
+void gemm_splitk(torch::Tensor A, torch::Tensor B, torch::Tensor C, c10::optional<torch::Tensor> bias,
+                 c10::optional<torch::Tensor> residual, torch::Tensor workspace, int64_t splits, int64_t bn,
+                 torch::Tensor err) {
+  const c10::cuda::CUDAGuard guard(A.device());
+  check(rb_gemm_splitk(A.data_ptr(), B.data_ptr(), C.data_ptr(), bias.has_value() ? bias->data_ptr() : nullptr,
+                       residual.has_value() ? residual->data_ptr() : nullptr, workspace.data_ptr<float>(), (int)A.size(0),
+                       (int)B.size(0), (int)A.size(1), (int)A.stride(0), (int)B.stride(0), (int)C.stride(0), (int)splits,
+                       (int)bn, A.scalar_type() == at::kHalf, err.data_ptr<int>(), cur_stream()),
+        "rb_gemm_splitk");
+}
+
+// ---- composed stacks
+void embed_rows(torch::Tensor tok, torch::Tensor w, torch::Tensor res, torch::Tensor h) {
+  const c10::cuda::CUDAGuard guard(w.device());
+  check_same(w, h, "embed_rows");
+  TORCH_CHECK(tok.scalar_type() == at::kLong && tok.is_contiguous() && w.is_contiguous() && res.is_contiguous() && h.is_contiguous());
+  TORCH_CHECK(res.scalar_type() == at::kFloat && res.sizes() == h.sizes() && h.size(0) == tok.numel() && h.size(1) == w.size(1));
+  check(rb_embed_rows((const long long*)tok.data_ptr<int64_t>(), w.data_ptr(), res.data_ptr<float>(), h.data_ptr(), (int)tok.numel(),
+                      (int)w.size(0), (int)w.size(1), is_fp32(w), cur_stream()),
+        "rb_embed_rows");
+}
+void norm_add(torch::Tensor res, torch::Tensor y, torch::Tensor w, c10::optional<torch::Tensor> next_w, torch::Tensor h, int64_t width,
+              int64_t groups, double eps) {
+  const c10::cuda::CUDAGuard guard(res.device());
+  check_same(y, w, "norm_add");
+  check_same(y, h, "norm_add");
+  TORCH_CHECK(res.scalar_type() == at::kFloat && res.is_contiguous() && h.is_contiguous() && res.sizes() == h.sizes());
+  TORCH_CHECK(y.dim() == 2 && y.stride(1) == 1 && y.size(0) == res.size(0) && y.size(1) >= width && w.numel() == res.size(1));
+  TORCH_CHECK(!next_w.has_value() || (next_w->numel() == w.numel() && next_w->scalar_type() == w.scalar_type()));
+  TORCH_CHECK(reinterpret_cast<uintptr_t>(y.data_ptr()) % 16 == 0, "norm_add: unaligned input");
+  check(rb_norm_add(res.data_ptr<float>(), y.data_ptr(), w.data_ptr(), optptr(next_w), h.data_ptr(), (int)res.size(0), (int)y.stride(0),
+                    (int)res.size(1), (int)width, (int)groups, (float)eps, is_fp32(y), cur_stream()),
+        "rb_norm_add");
+}
+void hgrn2(torch::Tensor qfv, torch::Tensor f_bias, torch::Tensor lower, torch::Tensor norm_w, torch::Tensor state, torch::Tensor slot,
+           torch::Tensor ctx, c10::optional<torch::Tensor> cu, c10::optional<torch::Tensor> o_raw, torch::Tensor out, int64_t dim,
+           int64_t vdim, double eps) {
+  const c10::cuda::CUDAGuard guard(qfv.device());
+  for (const auto& t : {f_bias, lower, norm_w, out}) check_same(qfv, t, "hgrn2");
+  const int64_t H = state.size(1), rows = qfv.size(0), segs = slot.numel();
+  TORCH_CHECK(state.dim() == 4 && state.scalar_type() == at::kFloat && state.is_contiguous() && state.size(2) == dim, "hgrn2: state");
+  TORCH_CHECK(qfv.dim() == 2 && qfv.stride(1) == 1 && out.is_contiguous() && out.size(0) == rows, "hgrn2: rows");
+  TORCH_CHECK(f_bias.numel() == H * dim && lower.numel() == H * dim && norm_w.numel() == vdim && f_bias.is_contiguous() && lower.is_contiguous());
+  TORCH_CHECK(slot.scalar_type() == at::kInt && ctx.scalar_type() == at::kInt && ctx.numel() == segs && slot.is_contiguous() && ctx.is_contiguous());
+  if (cu.has_value()) {
+    TORCH_CHECK(cu->scalar_type() == at::kInt && cu->numel() == segs + 1 && cu->is_contiguous());
+    TORCH_CHECK(o_raw.has_value() && o_raw->scalar_type() == at::kFloat && o_raw->numel() >= rows * H * vdim);
+  } else {
+    TORCH_CHECK(segs == rows, "hgrn2: one row per segment");
+  }
+  check(rb_hgrn2(qfv.data_ptr(), f_bias.data_ptr(), lower.data_ptr(), norm_w.data_ptr(), state.data_ptr<float>(), slot.data_ptr<int>(),
+                 ctx.data_ptr<int>(), optint(cu), o_raw.has_value() ? o_raw->data_ptr<float>() : nullptr, out.data_ptr(), (int)rows, (int)segs,
+                 (int)H, (int)dim, (int)vdim, (int)state.size(3), (int)qfv.stride(0), (int)out.size(1), (float)eps, is_fp32(qfv), cur_stream()),
+        "rb_hgrn2");
+}
+void latent_write(torch::Tensor raw, torch::Tensor w, torch::Tensor pool, torch::Tensor slots, int64_t rank, double eps) {
+  const c10::cuda::CUDAGuard guard(raw.device());
+  check_same(raw, w, "latent_write");
+  check_same(raw, pool, "latent_write");
+  TORCH_CHECK(raw.dim() == 2 && raw.stride(1) == 1 && raw.size(1) >= rank && w.numel() >= rank && pool.dim() == 2 && pool.is_contiguous());
+  TORCH_CHECK(slots.scalar_type() == at::kLong && slots.is_contiguous() && slots.numel() == raw.size(0));
+  check(rb_latent_write(raw.data_ptr(), (int)raw.stride(0), w.data_ptr(), pool.data_ptr(), (const long long*)slots.data_ptr<int64_t>(), pool.size(0),
+                        (int)raw.size(0), (int)rank, (int)pool.size(1), (float)eps, is_fp32(raw), cur_stream()),
+        "rb_latent_write");
+}
+void latent_attn(torch::Tensor q, torch::Tensor pool, torch::Tensor bt, c10::optional<torch::Tensor> row_seg, c10::optional<torch::Tensor> row_pos,
+                 torch::Tensor ctx, c10::optional<torch::Tensor> gate, torch::Tensor out, int64_t block_size, double scale) {
+  const c10::cuda::CUDAGuard guard(q.device());
+  check_same(q, pool, "latent_attn");
+  check_same(q, out, "latent_attn");
+  const int64_t T = q.size(0);
+  TORCH_CHECK(q.dim() == 3 && q.is_contiguous() && out.is_contiguous() && out.sizes() == q.sizes() && pool.is_contiguous() && pool.size(1) == q.size(2));
+  TORCH_CHECK(bt.scalar_type() == at::kInt && bt.is_contiguous() && ctx.scalar_type() == at::kInt && ctx.is_contiguous());
+  TORCH_CHECK(row_seg.has_value() == row_pos.has_value());
+  TORCH_CHECK(row_seg.has_value() ? (row_seg->numel() == T && row_pos->numel() == T && row_seg->scalar_type() == at::kInt &&
+                                     row_pos->scalar_type() == at::kInt)
+                                  : (ctx.numel() == T && bt.size(0) == T), "latent_attn: row description");
+  TORCH_CHECK(!gate.has_value() || (gate->scalar_type() == q.scalar_type() && gate->stride(1) == 1 && gate->size(0) == T));
+  check(rb_latent_attn(q.data_ptr(), pool.data_ptr(), bt.data_ptr<int>(), optint(row_seg), optint(row_pos), ctx.data_ptr<int>(), optptr(gate),
+                       out.data_ptr(), (int)T, (int)q.size(1), (int)q.size(2), (int)bt.size(1), (int)block_size,
+                       gate.has_value() ? (int)gate->stride(0) : 0, (float)scale, is_fp32(q), cur_stream()),
+        "rb_latent_attn");
+}
+void gate_heads(torch::Tensor o, torch::Tensor gate, torch::Tensor out, int64_t dv) {
+  const c10::cuda::CUDAGuard guard(o.device());
+  TORCH_CHECK(o.scalar_type() == at::kBFloat16 && gate.scalar_type() == at::kBFloat16 && out.scalar_type() == at::kBFloat16);
+  TORCH_CHECK(o.dim() == 3 && o.size(2) == 128 && o.is_contiguous() && out.is_contiguous() && gate.stride(1) == 1 && gate.size(0) == o.size(0));
+  TORCH_CHECK(out.numel() == o.size(0) * o.size(1) * dv);
+  check(rb_gate_heads(o.data_ptr(), gate.data_ptr(), (int)gate.stride(0), out.data_ptr(), (int)o.size(0), (int)o.size(1), (int)dv, cur_stream()),
+        "rb_gate_heads");
+}
+void glu(torch::Tensor in, torch::Tensor out, int64_t act) {
+  const c10::cuda::CUDAGuard guard(in.device());
+  check_same(in, out, "glu");
+  TORCH_CHECK(in.dim() == 2 && in.stride(1) == 1 && out.is_contiguous() && in.size(1) == 2 * out.size(1) && in.size(0) == out.size(0));
+  check(rb_glu(in.data_ptr(), out.data_ptr(), in.size(0), (int)out.size(1), (int)in.stride(0), (int)act, is_fp32(in), cur_stream()), "rb_glu");
+}
+// C[z] = A[z] op(B[z]) on CUDA cores; every operand [batch, rows, cols] with unit inner stride.
+void simt_gemm(torch::Tensor A, torch::Tensor B, torch::Tensor C, bool b_kn) {
+  const c10::cuda::CUDAGuard guard(A.device());
+  check_same(A, B, "simt_gemm");
+  check_same(A, C, "simt_gemm");
+  TORCH_CHECK(A.dim() == 3 && B.dim() == 3 && C.dim() == 3 && A.stride(2) == 1 && B.stride(2) == 1 && C.stride(2) == 1);
+  const int64_t K = A.size(2), N = C.size(2);
+  TORCH_CHECK(A.size(0) == C.size(0) && B.size(0) == C.size(0) && A.size(1) == C.size(1) && B.size(1) == (b_kn ? K : N) && B.size(2) == (b_kn ? N : K),
+              "simt_gemm: shapes");
+  check(rb_simt_gemm(A.data_ptr(), B.data_ptr(), C.data_ptr(), (int)A.size(1), (int)N, (int)K, (int)A.stride(1), (int)B.stride(1), (int)C.stride(1),
+                     b_kn, (int)A.size(0), A.stride(0), B.stride(0), C.stride(0), is_fp32(A), cur_stream()),
+        "rb_simt_gemm");
+}
+}  // namespace
+
+void register_serving(pybind11::module_& m) {
+  m.def("launch_count", []() { return (int64_t)rb_launch_count(); });
+  m.def("reset_launch_count", []() { rb_reset_launch_count(); });
+  m.def("gemm", &gemm);
+  m.def("gemm_pair", &gemm_pair);
+  m.def("fa_fwd", &fa_fwd);
+  m.def("sample_v2", &sample_v2);
+  m.def("decode_advance", &decode_advance);
+  m.def("decode_gemm", &decode_gemm);
+  m.def("gemm_splitk_plan", &gemm_splitk_plan);
+  m.def("gemm_splitk", &gemm_splitk);
+  m.def("embed_rows", &embed_rows);
+  m.def("norm_add", &norm_add);
+  m.def("hgrn2", &hgrn2);
+  m.def("latent_write", &latent_write);
+  m.def("latent_attn", &latent_attn);
+  m.def("gate_heads", &gate_heads);
+  m.def("glu", &glu);
+  m.def("simt_gemm", &simt_gemm);
+}

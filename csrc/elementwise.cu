@@ -517,12 +517,6 @@ static inline int grid_for(long long work_items, int threads) {
 
 using namespace rb;
 
-#include <atomic>
-static std::atomic<long long> g_launches{0};
-extern "C" void rb_note_launch(int n) { g_launches.fetch_add(n, std::memory_order_relaxed); }
-extern "C" long long rb_launch_count() { return g_launches.load(std::memory_order_relaxed); }
-extern "C" void rb_reset_launch_count() { g_launches.store(0, std::memory_order_relaxed); }
-
 #define RB_DISPATCH(dtype, ...)                                       \
   switch (dtype) {                                                    \
     case 0: { using T = __nv_bfloat16; __VA_ARGS__; break; }          \

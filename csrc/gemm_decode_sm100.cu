@@ -25,7 +25,7 @@ constexpr int CHUNK = 64;   // token columns reduced per pass
 struct Params {
   int Mt, N, K;             // tokens, output features of W (rows), reduction length
   int S;                    // cluster size = k splits
-  int swiglu;               // W rows are [gate (N/2); up (N/2)], output is [Mt, N/2]
+  int glu;                  // W rows are [gate (N/2); up (N/2)], output is [Mt, N/2]: 1 silu(g) u, 2 gelu_tanh(g) u
   void* out;
   int* err;
 };
@@ -62,6 +62,10 @@ __device__ __forceinline__ float4 ld_cluster_f32x4(uint32_t cluster_addr) {
                : "=f"(v.x), "=f"(v.y), "=f"(v.z), "=f"(v.w)
                : "r"(cluster_addr));
   return v;
+}
+// both activations are x sigmoid(z): z = x (silu), z = 2 sqrt(2 / pi) (x + 0.044715 x^3) (tanh form of gelu)
+__device__ __forceinline__ float gate_arg(float x, bool gelu) {
+  return gelu ? 1.5957691216057308f * (x + 0.044715f * x * x * x) : x;
 }
 __device__ __forceinline__ void store_bf16x4(__nv_bfloat16* dst, const float4& v) {   // dst 8-byte aligned
   const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
@@ -142,7 +146,7 @@ decode_gemm_kernel(const __grid_constant__ CUtensorMap tma_w, const __grid_const
       auto load_w = [&](int s, int k) {
         uint8_t* sw = smem + s * C::kStageBytes;
         mbar_expect_tx(&full_bar[s], C::kStageBytes);
-        if (!p.swiglu) {
+        if (!p.glu) {
           tma_load_2d(sw, &tma_w, &full_bar[s], k * BK, tile * BM);
         } else {   // 64 gate rows, then the 64 up rows of the same features
           tma_load_2d(sw, &tma_w, &full_bar[s], k * BK, tile * 64);
@@ -205,7 +209,7 @@ decode_gemm_kernel(const __grid_constant__ CUtensorMap tma_w, const __grid_const
     // slice of the tile this CTA reduces: feature rows (plain) or gate/up pairs (SwiGLU).  S is a power of two, so
     // the slice is a power of two >= 8 and splits into float4 groups with shifts.
     const int lgS = 31 - __clz(S);
-    const int units = p.swiglu ? 64 : BM;
+    const int units = p.glu ? 64 : BM;
     const int u_n = units >> lgS;
     const int u_lo = q * u_n;
     const int lgG = 31 - __clz(u_n >> 2);
@@ -251,7 +255,7 @@ decode_gemm_kernel(const __grid_constant__ CUtensorMap tma_w, const __grid_const
 #pragma unroll
           for (int z = 1; z < 8; ++z)
             if (z < S) { acc.x += a[z].x; acc.y += a[z].y; acc.z += a[z].z; acc.w += a[z].w; }
-          if (!p.swiglu) {
+          if (!p.glu) {
             const int f = tile * BM + u_lo + 4 * g;
             __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(p.out) + static_cast<size_t>(tok) * p.N + f;
             if (f + 3 < p.N) {
@@ -272,10 +276,11 @@ decode_gemm_kernel(const __grid_constant__ CUtensorMap tma_w, const __grid_const
               if (z < S) { up.x += b[z].x; up.y += b[z].y; up.z += b[z].z; up.w += b[z].w; }
             const int f = tile * 64 + u_lo + 4 * g;      // F is a multiple of 64: always inside
             float4 r;
-            r.x = acc.x / (1.f + __expf(-acc.x)) * up.x;
-            r.y = acc.y / (1.f + __expf(-acc.y)) * up.y;
-            r.z = acc.z / (1.f + __expf(-acc.z)) * up.z;
-            r.w = acc.w / (1.f + __expf(-acc.w)) * up.w;
+            const bool gelu = p.glu == 2;
+            r.x = acc.x / (1.f + __expf(-gate_arg(acc.x, gelu))) * up.x;
+            r.y = acc.y / (1.f + __expf(-gate_arg(acc.y, gelu))) * up.y;
+            r.z = acc.z / (1.f + __expf(-gate_arg(acc.z, gelu))) * up.z;
+            r.w = acc.w / (1.f + __expf(-gate_arg(acc.w, gelu))) * up.w;
             store_bf16x4(reinterpret_cast<__nv_bfloat16*>(p.out) + static_cast<size_t>(tok) * F + f, r);
           }
         }
@@ -343,27 +348,28 @@ extern "C" int rb_decode_gemm_splits(int tiles, int k_iters) {
   return s;
 }
 
-// y = x W^T (swiglu = 0, y [Mt, N]) or y = silu(x Wg^T) * (x Wu^T) with W = [Wg; Wu] (swiglu = 1, y [Mt, N / 2]).
+// y = x W^T (glu = 0, y [Mt, N]) or y = act(x Wg^T) * (x Wu^T) with W = [Wg; Wu] (glu = 1: silu, 2: tanh form of gelu;
+// y [Mt, N / 2]).
 // x [Mt <= 256, K], W [N, K], all bf16 row-major; returns -20 when the shape is outside what this kernel covers.
-extern "C" int rb_decode_gemm(const void* x, const void* W, void* y, int Mt, int N, int K, int ldx, int ldw, int swiglu,
+extern "C" int rb_decode_gemm(const void* x, const void* W, void* y, int Mt, int N, int K, int ldx, int ldw, int glu,
                               int splits, int* err, cudaStream_t st) {
   using namespace rb;
   using namespace rb::dg;
   if (Mt <= 0 || N <= 0 || K <= 0) return 0;
   if (Mt > 256 || (ldx % 8) || (ldw % 8) || (K % 8)) return -20;
   if ((reinterpret_cast<uintptr_t>(x) % 16) || (reinterpret_cast<uintptr_t>(W) % 16)) return -20;
-  if (swiglu && ((N / 2) % 64)) return -20;
+  if (glu && ((N / 2) % 64)) return -20;
   if ((N % 4) || (reinterpret_cast<uintptr_t>(y) % 8)) return -20;   // 4 features per store
   const int nt = Mt <= 64 ? 64 : (Mt <= 128 ? 128 : 256);
-  const int tiles = swiglu ? (N / 2) / 64 : (N + BM - 1) / BM;
+  const int tiles = glu ? (N / 2) / 64 : (N + BM - 1) / BM;
   const int k_iters = (K + BK - 1) / BK;
   Params p{};
-  p.Mt = Mt; p.N = N; p.K = K; p.swiglu = swiglu; p.out = y; p.err = err;
+  p.Mt = Mt; p.N = N; p.K = K; p.glu = glu; p.out = y; p.err = err;
   p.S = splits > 0 ? splits : rb_decode_gemm_splits(tiles, k_iters);
   if (p.S > 8) p.S = 8;
   while (p.S & (p.S - 1)) p.S &= p.S - 1;       // the reduction slices the tile in powers of two
   CUtensorMap tw, tx;
-  int rc = encode_tma_2d_bf16(&tw, W, K, N, ldw, BK, swiglu ? 64 : BM);
+  int rc = encode_tma_2d_bf16(&tw, W, K, N, ldw, BK, glu ? 64 : BM);
   if (rc) return rc;
   rc = encode_tma_2d_bf16(&tx, x, K, Mt, ldx, BK, nt);
   if (rc) return rc;

@@ -17,6 +17,13 @@ ROOT = os.path.dirname(os.path.dirname(os.path.dirname(os.path.abspath(__file__)
 CSRC = os.path.join(ROOT, "csrc")
 OBJ = os.path.join(ROOT, "build", "obj")
 SO_PATH = os.path.join(ROOT, "relax_b200", "_C.so")
+# The serving extension: the kernels and bindings a composed stack's engine launches, and nothing else.  It is built where
+# only such an engine runs and the full extension has not been built (a fresh checkout); the ops load whichever exists.
+SERVING_SO_PATH = os.path.join(ROOT, "relax_b200", "_C_serving.so")
+SERVING_SOURCES = ["attention_fwd_sm100.cu", "decode_step_sm100.cu", "gemm2_sm100.cu", "gemm_decode_sm100.cu", "gemm_sm100.cu",
+                   "stack_sm100.cu", "bindings_serving.cpp", "launch_count.cpp", "module_serving.cpp"]
+# fp32 results of these kernels are compared at fp32 rounding: IEEE division, square root and library exponentials
+PRECISE_SOURCES = {"stack_sm100.cu"}
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17", "--use_fast_math",
@@ -46,21 +53,39 @@ def _run(cmd: list, log_path: str | None = None):
     return p.stdout
 
 
-def build_extension(verbose: bool = False, force: bool = False) -> str:
+def ensure_serving(verbose: bool = False) -> str:
+    """The extension a serving process needs: the full one when it is there and newer than the sources, else the serving
+    subset (built if missing or stale).  Concurrent callers take turns."""
+    import fcntl
+
+    srcs = [os.path.join(CSRC, f) for f in os.listdir(CSRC)]
+    if not _stale(SO_PATH, srcs):
+        return SO_PATH
+    os.makedirs(OBJ, exist_ok=True)
+    with open(os.path.join(OBJ, ".lock"), "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        return build_extension(verbose, serving=True)
+
+
+def build_extension(verbose: bool = False, force: bool = False, serving: bool = False) -> str:
+    """Compile what is stale and link the full extension, or (``serving``) the serving subset."""
     import torch
     from torch.utils import cpp_extension as ce
 
     os.makedirs(OBJ, exist_ok=True)
     headers = [os.path.join(CSRC, f) for f in os.listdir(CSRC) if f.endswith((".h", ".cuh"))]
-    cus = sorted(f for f in os.listdir(CSRC) if f.endswith(".cu"))
-    cpps = sorted(f for f in os.listdir(CSRC) if f.endswith(".cpp"))
+    names = SERVING_SOURCES if serving else [f for f in os.listdir(CSRC) if f != "module_serving.cpp"]
+    so_path = SERVING_SO_PATH if serving else SO_PATH
+    cus = sorted(f for f in names if f.endswith(".cu"))
+    cpps = sorted(f for f in names if f.endswith(".cpp"))
     jobs = []
     objs = []
     for f in cus:
         src, out = os.path.join(CSRC, f), os.path.join(OBJ, f + ".o")
         objs.append(out)
         if force or _stale(out, [src] + headers):
-            jobs.append(([_nvcc()] + NVCC_FLAGS + ["-I", CSRC, "-c", src, "-o", out], out + ".log"))
+            flags = [x for x in NVCC_FLAGS if not (f in PRECISE_SOURCES and x == "--use_fast_math")]
+            jobs.append(([_nvcc()] + flags + ["-I", CSRC, "-c", src, "-o", out], out + ".log"))
     abi = int(getattr(torch._C, "_GLIBCXX_USE_CXX11_ABI", True))
     inc = []
     for p in ce.include_paths("cuda") if "device_type" in ce.include_paths.__code__.co_varnames else ce.include_paths(True):
@@ -78,18 +103,18 @@ def build_extension(verbose: bool = False, force: bool = False) -> str:
         if verbose:
             print(f"[relax_b200.build] compiling {len(jobs)} translation unit(s) for sm_100a", flush=True)
         with ThreadPoolExecutor(max_workers=min(8, len(jobs))) as ex:
-            list(ex.map(lambda j: _run(*j), jobs))
-    if jobs or force or _stale(SO_PATH, objs):
+            list(ex.map(lambda j: _run(*j), sorted(jobs, key=lambda j: -os.path.getsize(j[0][j[0].index("-c") + 1]))))
+    if jobs or force or _stale(so_path, objs):
         tlib = os.path.join(os.path.dirname(torch.__file__), "lib")
         cuda_lib = os.path.join(os.environ.get("CUDA_HOME", "/usr/local/cuda"), "lib64")
-        cmd = [cxx, "-shared", "-o", SO_PATH] + objs + [
+        cmd = [cxx, "-shared", "-o", so_path] + objs + [
             f"-L{tlib}", "-lc10", "-ltorch", "-ltorch_cpu", "-ltorch_python", "-lc10_cuda", "-ltorch_cuda",
             f"-L{cuda_lib}", "-lcudart", f"-Wl,-rpath,{tlib}", f"-Wl,-rpath,{cuda_lib}",
         ]
         _run(cmd)
         if verbose:
-            print(f"[relax_b200.build] linked {SO_PATH}", flush=True)
-    return SO_PATH
+            print(f"[relax_b200.build] linked {so_path}", flush=True)
+    return so_path
 
 
 def ptxas_report() -> str:

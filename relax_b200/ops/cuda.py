@@ -13,18 +13,21 @@ from typing import Optional
 import torch
 
 _SO = os.path.join(os.path.dirname(os.path.dirname(os.path.abspath(__file__))), "_C.so")
+_SO_SERVING = _SO.replace("_C.so", "_C_serving.so")      # serving subset (ops/build.py)
 _C = None
 _ERR: dict = {}
 _MN_OK: Optional[bool] = None
 
 
-def _load():
+def _load(path: Optional[str] = None):
+    """The extension module: the full one, else the serving subset (whose missing operators raise when called)."""
     global _C
     if _C is not None:
         return _C
-    if not os.path.exists(_SO):
+    so = path or (_SO if os.path.exists(_SO) else _SO_SERVING)
+    if not os.path.exists(so):
         raise RuntimeError(f"{_SO} is missing: build it with `python __graft_entry__.py` (nvcc, sm_100a)")
-    spec = importlib.util.spec_from_file_location("relax_b200._C", _SO)
+    spec = importlib.util.spec_from_file_location("relax_b200." + os.path.basename(so)[:-3], so)
     mod = importlib.util.module_from_spec(spec)
     spec.loader.exec_module(mod)
     if os.environ.get("RELAX_B200_CRASH_TRACE", "0") == "1":
@@ -178,8 +181,12 @@ class _Linear(torch.autograd.Function):
 def linear(x, w, bias=None):
     shp = x.shape
     x2 = x.reshape(-1, shp[-1])
+    if x2.dtype == torch.float32 and w.dtype == torch.float32 and not torch.is_grad_enabled():
+        y = torch.empty(x2.shape[0], w.shape[0], dtype=torch.float32, device=x.device)      # 32-bit inference: CUDA cores, true fp32
+        _load().simt_gemm(x2[None], w[None], y[None], False)
+        return (y if bias is None else y + bias).reshape(*shp[:-1], w.shape[0])
     if x2.dtype not in (torch.bfloat16, torch.float16):
-        raise TypeError("the sm_100a GEMM takes bf16/fp16 inputs")
+        raise TypeError("the sm_100a GEMM takes bf16/fp16 inputs (fp32 in inference only)")
     if w.dim() != 2:
         raise ValueError("weight must be 2-D")
     if x2.shape[0] <= 256 and not (torch.is_grad_enabled() and (x2.requires_grad or w.requires_grad)) \
@@ -200,15 +207,18 @@ def linear(x, w, bias=None):
 _DECODE_GEMM = os.environ.get("RELAX_B200_DECODE_GEMM", "1") == "1"
 
 
-def _decode_gemm(x, w, swiglu: bool):
+GLU_ACT = {"silu": 1, "gelu_tanh": 2}
+
+
+def _decode_gemm(x, w, glu_act: int):
     """Weight-streaming decode GEMM (csrc/gemm_decode_sm100.cu) when the shape is in its range, else None."""
     if not _DECODE_GEMM or x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 or x.shape[0] > 128:
         return None     # above 128 rows the 2-stage ring of the 256-column variant loses to the other paths (measured)
     if w.stride(1) != 1 or w.stride(0) % 8 or w.data_ptr() % 16:
         return None
     N = w.shape[0]
-    out = torch.empty(x.shape[0], N // 2 if swiglu else N, dtype=x.dtype, device=x.device)
-    if _load().decode_gemm(x, w, out, swiglu, 0, err_flag(x.device)):
+    out = torch.empty(x.shape[0], N // 2 if glu_act else N, dtype=x.dtype, device=x.device)
+    if _load().decode_gemm(x, w, out, glu_act, 0, err_flag(x.device)):
         return out
     return None
 
@@ -237,7 +247,7 @@ def matmul_nt_skinny(x, w, bias=None, residual=None):
     N = w.shape[0]
     C = _load()
     if bias is None and residual is None:
-        y = _decode_gemm(x, w, False)
+        y = _decode_gemm(x, w, 0)
         if y is None:
             y = _wide_pair_gemm(x, w)
         if y is not None:
@@ -259,7 +269,7 @@ def linear_swiglu_skinny(x, w):
     M, K = x.shape
     N = w.shape[0]
     C = _load()
-    y = _decode_gemm(x, w, True)
+    y = _decode_gemm(x, w, 1)
     if y is not None:
         return y
     y = _wide_pair_gemm(x, w)
@@ -272,6 +282,78 @@ def linear_swiglu_skinny(x, w):
     C.gemm_splitk_partial(x, w, ws, splits, bn, err_flag(x.device))
     out = torch.empty(M, N // 2, dtype=x.dtype, device=x.device)
     C.splitk_swiglu(ws, out, splits)
+    return out
+
+
+def glu(gate_up, act: str = "silu"):
+    """``act(gate) * up`` on ``[gate | up]`` rows (inference only)."""
+    gu = gate_up.reshape(-1, gate_up.shape[-1])
+    out = torch.empty(gu.shape[0], gu.shape[1] // 2, dtype=gu.dtype, device=gu.device)
+    _load().glu(gu, out, GLU_ACT[act] - 1)
+    return out.reshape(*gate_up.shape[:-1], out.shape[1])
+
+
+def linear_glu(x, w, act: str = "silu"):
+    """``glu(x @ w.T)``: the activation joins the decode GEMM's reduction for up to 128 rows."""
+    if x.dtype == torch.bfloat16 and x.shape[0] <= 128:
+        x, _ = _rowmajor_2d(x)
+        y = _decode_gemm(x, w, GLU_ACT[act])
+        if y is not None:
+            return y
+    return glu(linear(x, w), act)
+
+
+# --------------------------------------------------------------------------- composed stacks (inference)
+
+
+def embed_rows(tokens, w):
+    res = torch.empty(tokens.shape[0], w.shape[1], dtype=torch.float32, device=w.device)
+    h = torch.empty(tokens.shape[0], w.shape[1], dtype=w.dtype, device=w.device)
+    _load().embed_rows(tokens, w, res, h)
+    return res, h
+
+
+def norm_add(res, y, w, width, groups, eps, next_w=None):
+    h = torch.empty(res.shape, dtype=w.dtype, device=w.device)
+    _load().norm_add(res, y, w, next_w, h, int(width), int(groups), float(eps))
+    return h
+
+
+def hgrn2(qfv, f_bias, lower, norm_w, state, state_slot, ctx_lens, cu, heads, dim, vdim, eps):
+    T = qfv.shape[0]
+    out = torch.empty(T, (heads * vdim + 7) // 8 * 8, dtype=qfv.dtype, device=qfv.device)
+    raw = None if cu is None else torch.empty(T, heads, vdim, dtype=torch.float32, device=qfv.device)
+    _load().hgrn2(qfv, f_bias, lower, norm_w, state, state_slot, ctx_lens, cu, raw, out, int(dim), int(vdim), float(eps))
+    return out
+
+
+def latent_write(raw, w, rank, eps, pool, slots):
+    _load().latent_write(raw, w, pool, slots, int(rank), float(eps))
+
+
+def head_linear(x, w, transposed):
+    T, H, _ = x.shape
+    out = torch.empty(T, H, w.shape[1] if transposed else w.shape[2], dtype=x.dtype, device=x.device)
+    _load().simt_gemm(x.transpose(0, 1), w, out.transpose(0, 1), not transposed)
+    return out
+
+
+def latent_attention(q, pool, b, block_size, scale, gate):
+    q = q.contiguous()
+    out = torch.empty_like(q)
+    n = b.long_segs
+    _load().latent_attn(q, pool, b.block_tables[n:], b.row_seg, b.row_pos, b.ctx[n:], gate, out, int(block_size), float(scale))
+    return out
+
+
+def flash_gated(q, k, v, cu_q, cu_k, scale, max_q, gate):
+    F = torch.nn.functional
+    dk, dv = q.shape[-1], v.shape[-1]
+    q, k = (t if dk == 128 else F.pad(t, (0, 128 - dk)) for t in (q, k))
+    v = v if dv == 128 else F.pad(v, (0, 128 - dv))
+    o = attention_varlen(q, k, v, cu_q, True, scale, cu_k, max_q)
+    out = torch.empty(q.shape[0], q.shape[1] * dv, dtype=q.dtype, device=q.device)
+    _load().gate_heads(o, gate, out, int(dv))
     return out
 
 
