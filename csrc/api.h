@@ -141,6 +141,11 @@ int rb_latent_write(const void* raw, int ld_raw, const void* w, void* pool, cons
 int rb_latent_attn(const void* q, const void* pool, const int* block_tables, const int* row_seg, const int* row_pos, const int* ctx,
                    const void* gate, void* out, int rows, int H, int R, int max_blocks, int block_size, int ld_gate, float scale,
                    int fp32, cudaStream_t st);
+int rb_latent_attn_tc(const void* q, const void* pool, const int* block_tables, const int* items, const int* ctx, const void* gate,
+                      void* out, float* part_o, float* part_ml, int rows, int H, int R, long long pool_rows, int max_blocks, int page,
+                      int n_items, int width, int splits, int ld_gate, float scale, int* err, cudaStream_t st);
+int rb_head_gemm(const void* x, const void* w, void* out, int T, int H, int N, int K, long long x_tok, long long x_head, int kn, int* err,
+                 cudaStream_t st);
 int rb_gate_heads(const void* o, const void* gate, int ld_gate, void* out, int rows, int H, int dv, cudaStream_t st);
 int rb_glu(const void* in, void* out, long long rows, int F, int ld_in, int act, int fp32, cudaStream_t st);
 int rb_simt_gemm(const void* A, const void* B, void* C, int M, int N, int K, int lda, int ldb, int ldc, int b_kn, int batch, long long sa,

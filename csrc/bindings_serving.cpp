@@ -201,6 +201,44 @@ void latent_attn(torch::Tensor q, torch::Tensor pool, torch::Tensor bt, c10::opt
                        gate.has_value() ? (int)gate->stride(0) : 0, (float)scale, is_fp32(q), cur_stream()),
         "rb_latent_attn");
 }
+// Tensor-core form (bf16); returns false for shapes it does not take (the caller then uses latent_attn).
+bool latent_attn_tc(torch::Tensor q, torch::Tensor pool, torch::Tensor bt, c10::optional<torch::Tensor> items, torch::Tensor ctx,
+                    c10::optional<torch::Tensor> gate, torch::Tensor out, c10::optional<torch::Tensor> part_o,
+                    c10::optional<torch::Tensor> part_ml, int64_t block_size, int64_t width, int64_t splits, double scale, torch::Tensor err) {
+  const c10::cuda::CUDAGuard guard(q.device());
+  const int64_t T = q.size(0), H = q.size(1), R = q.size(2);
+  TORCH_CHECK(q.scalar_type() == at::kBFloat16 && pool.scalar_type() == at::kBFloat16 && out.scalar_type() == at::kBFloat16);
+  TORCH_CHECK(q.dim() == 3 && q.is_contiguous() && out.is_contiguous() && out.sizes() == q.sizes() && pool.is_contiguous() && pool.size(1) == R);
+  TORCH_CHECK(bt.scalar_type() == at::kInt && bt.is_contiguous() && ctx.scalar_type() == at::kInt && ctx.is_contiguous());
+  if (items.has_value()) {
+    TORCH_CHECK(items->scalar_type() == at::kInt && items->dim() == 2 && items->size(1) == 4 && items->is_contiguous());
+  } else {
+    TORCH_CHECK(ctx.numel() == T && bt.size(0) == T, "latent_attn_tc: one row per segment");
+  }
+  TORCH_CHECK(!gate.has_value() || (gate->scalar_type() == at::kBFloat16 && gate->stride(1) == 1 && gate->size(0) == T));
+  TORCH_CHECK(splits == 1 || (part_o.has_value() && part_o->numel() >= splits * T * H * R && part_ml.has_value() &&
+                              part_ml->numel() >= splits * T * H * 2), "latent_attn_tc: scratch");
+  const int rc = rb_latent_attn_tc(q.data_ptr(), pool.data_ptr(), bt.data_ptr<int>(), optint(items), ctx.data_ptr<int>(), optptr(gate), out.data_ptr(),
+                                   part_o.has_value() ? part_o->data_ptr<float>() : nullptr, part_ml.has_value() ? part_ml->data_ptr<float>() : nullptr,
+                                   (int)T, (int)H, (int)R, pool.size(0), (int)bt.size(1), (int)block_size,
+                                   items.has_value() ? (int)items->size(0) : 0, (int)width, (int)splits,
+                                   gate.has_value() ? (int)gate->stride(0) : 0, (float)scale, err.data_ptr<int>(), cur_stream());
+  if (rc == -20) return false;
+  check(rc, "rb_latent_attn_tc");
+  return true;
+}
+bool head_gemm(torch::Tensor x, torch::Tensor w, torch::Tensor out, bool kn, torch::Tensor err) {
+  const c10::cuda::CUDAGuard guard(x.device());
+  TORCH_CHECK(x.scalar_type() == at::kBFloat16 && w.scalar_type() == at::kBFloat16 && out.scalar_type() == at::kBFloat16);
+  TORCH_CHECK(x.dim() == 3 && w.dim() == 3 && out.dim() == 3 && x.stride(2) == 1 && w.is_contiguous() && out.is_contiguous());
+  TORCH_CHECK(w.size(0) == x.size(1) && w.size(kn ? 1 : 2) == x.size(2) && out.size(0) == x.size(0) && out.size(1) == x.size(1) &&
+              out.size(2) == w.size(kn ? 2 : 1), "head_gemm: shapes");
+  const int rc = rb_head_gemm(x.data_ptr(), w.data_ptr(), out.data_ptr(), (int)x.size(0), (int)x.size(1), (int)out.size(2), (int)x.size(2), x.stride(0),
+                              x.stride(1), kn, err.data_ptr<int>(), cur_stream());
+  if (rc == -20) return false;
+  check(rc, "rb_head_gemm");
+  return true;
+}
 void gate_heads(torch::Tensor o, torch::Tensor gate, torch::Tensor out, int64_t dv) {
   const c10::cuda::CUDAGuard guard(o.device());
   TORCH_CHECK(o.scalar_type() == at::kBFloat16 && gate.scalar_type() == at::kBFloat16 && out.scalar_type() == at::kBFloat16);
@@ -246,6 +284,8 @@ void register_serving(pybind11::module_& m) {
   m.def("hgrn2", &hgrn2);
   m.def("latent_write", &latent_write);
   m.def("latent_attn", &latent_attn);
+  m.def("latent_attn_tc", &latent_attn_tc);
+  m.def("head_gemm", &head_gemm);
   m.def("gate_heads", &gate_heads);
   m.def("glu", &glu);
   m.def("simt_gemm", &simt_gemm);

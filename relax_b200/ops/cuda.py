@@ -334,15 +334,36 @@ def latent_write(raw, w, rank, eps, pool, slots):
 def head_linear(x, w, transposed):
     T, H, _ = x.shape
     out = torch.empty(T, H, w.shape[1] if transposed else w.shape[2], dtype=x.dtype, device=x.device)
-    _load().simt_gemm(x.transpose(0, 1), w, out.transpose(0, 1), not transposed)
+    if x.dtype == torch.bfloat16 and _load().head_gemm(x, w, out, not transposed, err_flag(x.device)):
+        return out
+    _load().simt_gemm(x.transpose(0, 1), w, out.transpose(0, 1), not transposed)      # 32-bit mode
     return out
 
 
+LATENT_TILE = 128      # positions per tile of the tensor-core latent attention
+
+
 def latent_attention(q, pool, b, block_size, scale, gate):
+    """Tensor cores for bf16 with ranks up to 512 and pages of 16 to 128 tokens, CUDA cores otherwise (32-bit mode)."""
     q = q.contiguous()
     out = torch.empty_like(q)
+    T, H, R = q.shape
     n = b.long_segs
-    _load().latent_attn(q, pool, b.block_tables[n:], b.row_seg, b.row_pos, b.ctx[n:], gate, out, int(block_size), float(scale))
+    bt, ctx = b.block_tables[n:], b.ctx[n:]
+    if q.dtype == torch.bfloat16 and R <= 512 and block_size in (16, 32, 64, 128):
+        items = b.items[H] if b.items is not None else None
+        if items is None and b.cu is not None:
+            raise ValueError("a batch of segments needs its column groups (attention_items)")
+        width = 64 if items is not None or H > 32 else (16 if H <= 16 else 32)
+        groups = items.shape[0] if items is not None else T * ((H + width - 1) // width)
+        splits = max(1, min(148 // groups, (b.max_ctx + LATENT_TILE - 1) // LATENT_TILE, 32))
+        po = ml = None
+        if splits > 1:
+            po = torch.empty(splits * T * H * R, dtype=torch.float32, device=q.device)
+            ml = torch.empty(splits * T * H * 2, dtype=torch.float32, device=q.device)
+        if _load().latent_attn_tc(q, pool, bt, items, ctx, gate, out, po, ml, int(block_size), width, splits, float(scale), err_flag(q.device)):
+            return out
+    _load().latent_attn(q, pool, bt, b.row_seg, b.row_pos, ctx, gate, out, int(block_size), float(scale))
     return out
 
 
