@@ -75,6 +75,9 @@ def parse():
     ap.add_argument("--profile-kernels", type=int, default=0,
                     help="debug: after the timed steps run ONE more step under torch.profiler and print rank 0's top N kernels "
                          "by device time to stderr (the extra step is not part of any reported number)")
+    ap.add_argument("--stack-bench", choices=["1b", "5b"], default=None,
+                    help="instead of the headline workload: serving kernels and engine throughput of a composed stack (Talizen) "
+                         "beside the engine's existing models at the same layer sizes (1 GPU; plain-text table)")
     return ap.parse_args()
 
 
@@ -138,6 +141,10 @@ def main():
     args = parse()
     if args.impl == "reference":
         return reference_arm(args)
+    if args.stack_bench:
+        from relax_b200.rollout.bench_stack import main as stack_bench
+
+        return stack_bench(args.stack_bench, os.path.join(ROOT, "MEASURED_PEAKS.json"))
     os.environ.setdefault("PYTORCH_CUDA_ALLOC_CONF", "expandable_segments:True")
     if os.environ.get("RELAX_B200_HANG_DUMP_S"):
         # debugging aid: print every thread's Python stack and exit if the run is still going after this many seconds

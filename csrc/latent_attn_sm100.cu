@@ -24,6 +24,7 @@ constexpr int TILE = 128;                 // positions per tile
 constexpr int SLOT = 32768;               // ring slot: two 64-feature chunks of a tile
 constexpr int MAX_SLOTS = 5;
 constexpr int THREADS = 192;
+constexpr int SCRATCH = 2560;               // barriers (256 B), then 8 N + 2 words
 
 struct Params {
   const int* items;          // [n][4]: segment, first column, columns, base; null: one row per segment (decode)
@@ -47,7 +48,7 @@ __device__ __forceinline__ float redux_max(float v) {
 template <int N>
 struct Layout {
   static constexpr int kP = 2 * N * 128;                     // one P buffer: two 64-position halves of N rows
-  static int total(int slots, int NC) { return slots * SLOT + NC * N * 128 + 2 * kP + 4096; }
+  static int total(int slots, int NC) { return slots * SLOT + NC * N * 128 + 2 * kP + SCRATCH; }
 };
 
 template <int N>
@@ -414,7 +415,7 @@ extern "C" int rb_latent_attn_tc(const void* q, const void* pool, const int* blo
   p.H = H; p.R = R; p.NC = R / 64; p.NP = (p.NC + 1) / 2; p.max_blocks = max_blocks; p.page = page; p.splits = splits;
   p.columns = rows * H; p.groups_per_row = (H + width - 1) / width; p.ld_gate = ld_gate;
   p.scale_log2 = scale * 1.4426950408889634f; p.err = err;
-  const int fixed = p.NC * width * 128 + 2 * (2 * width * 128) + 4096;
+  const int fixed = p.NC * width * 128 + 2 * (2 * width * 128) + SCRATCH;
   p.slots = p.NP == 1 ? 3 : MAX_SLOTS;       // one pair: a small CTA, so that two share an SM
   while (p.slots * SLOT + fixed > 227 * 1024) --p.slots;
   if (p.slots < p.NP) return -20;
