@@ -24,7 +24,7 @@ constexpr int TILE = 128;                 // positions per tile
 constexpr int SLOT = 32768;               // ring slot: two 64-feature chunks of a tile
 constexpr int MAX_SLOTS = 5;
 constexpr int THREADS = 192;
-constexpr int SCRATCH = 2560;               // barriers (256 B), then 8 N + 2 words
+constexpr int SCRATCH = 2560;               // barriers (256 B), then 8 N words
 
 struct Params {
   const int* items;          // [n][4]: segment, first column, columns, base; null: one row per segment (decode)
@@ -43,6 +43,17 @@ __device__ __forceinline__ float redux_max(float v) {
   float r;
   asm("redux.sync.max.f32 %0, %1, 0xffffffff;" : "=f"(r) : "f"(v));
   return r;
+}
+
+// barrier `id` of `threads` threads that also ORs a predicate over them
+__device__ __forceinline__ bool named_bar_or(int id, int threads, bool v) {
+  uint32_t r;
+  asm volatile(
+      "{\n\t.reg .pred p, q;\n\tsetp.ne.u32 p, %1, 0;\n\tbar.red.or.pred q, %2, %3, p;\n\tselp.u32 %0, 1, 0, q;\n\t}"
+      : "=r"(r)
+      : "r"(static_cast<uint32_t>(v)), "r"(id), "r"(threads)
+      : "memory");
+  return r != 0;
 }
 
 template <int N>
@@ -71,7 +82,6 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
   float* s_alpha = s_m + N;                                   // [N]
   float* s_gate = s_alpha + N;                                // [N]
   int* s_lim = reinterpret_cast<int*>(s_gate + N);            // [N] positions a column sees
-  int* s_flag = s_lim + N;                                    // [2]
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   constexpr int kTmemCols = N == 16 ? 128 : (N == 32 ? 256 : 512);      // (2 + NP) * N columns, NP <= 4
@@ -137,26 +147,37 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
 
   if (warp == 4) {
     // ================================================================ TMA producer (page gather)
-    if (lane == 0 && !dead && n_tiles > 0) {
-      mbar_expect_tx(bar_q, p.NC * N * 128);
-      for (int c = 0; c < p.NC; ++c) tma_load_2d(sq + c * N * 128, &tma_q, bar_q, c * 64, col0);
+    // lane i gathers page i of every tile: the page number is looked up once per tile and the copies of a slot are issued
+    // by all lanes together
+    if (!dead && n_tiles > 0) {
+      if (lane == 0) {
+        mbar_expect_tx(bar_q, p.NC * N * 128);
+        for (int c = 0; c < p.NC; ++c) tma_load_2d(sq + c * N * 128, &tma_q, bar_q, c * 64, col0);
+      }
       const int pages = TILE / p.page, page_bytes = p.page * 128;
+      // pages behind the context: any row, masked
+      auto page_row = [&](int j) { return lane < pages ? bt[min((tile0 + j) * pages + lane, p.max_blocks - 1)] * p.page : 0; };
+      int row = page_row(0);
       int s = 0;
       uint32_t ph = 1;
       bool ok = true;
       for (int j = 0; j < n_tiles && ok; ++j) {
-        const int page0 = (tile0 + j) * pages;
+        const int next = j + 1 < n_tiles ? page_row(j + 1) : 0;
         for (int pr = 0; pr < p.NP; ++pr) {
-          if (!mbar_wait(&empty[s], ph, abort_flag, p.err)) { ok = false; break; }
+          ok = mbar_wait(&empty[s], ph, abort_flag, p.err);
+          ok = __all_sync(0xffffffffu, ok);
+          if (!ok) break;
           const int nch = min(2, p.NC - 2 * pr);
-          mbar_expect_tx(&full[s], nch * (SLOT / 2));
-          uint8_t* dst = smem + s * SLOT;
-          for (int pg = 0; pg < pages; ++pg) {
-            const int row = bt[min(page0 + pg, p.max_blocks - 1)] * p.page;      // pages behind the context: any row, masked
-            for (int c = 0; c < nch; ++c) tma_load_2d(dst + c * (SLOT / 2) + pg * page_bytes, &tma_c, &full[s], (2 * pr + c) * 64, row);
+          if (lane == 0) mbar_expect_tx(&full[s], nch * (SLOT / 2));
+          __syncwarp();
+          uint8_t* dst = smem + s * SLOT + lane * page_bytes;
+          if (lane < pages) {
+            tma_load_2d(dst, &tma_c, &full[s], pr * 128, row);
+            if (nch == 2) tma_load_2d(dst + SLOT / 2, &tma_c, &full[s], pr * 128 + 64, row);
           }
           if (++s == p.slots) { s = 0; ph ^= 1; }
         }
+        row = next;
       }
     }
   } else if (warp == 5) {
@@ -229,37 +250,40 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
       tmem_wait_ld();
       const int tok = (tile0 + j) * TILE + r;
       const bool masked = (tile0 + j + 1) * TILE > first_lim || ncols < N;      // uniform: some column ends inside this tile
-      float mine[(N + 31) / 32];
+      if (masked) {
 #pragma unroll
-      for (int n = 0; n < N; ++n) {
-        float v = s[n] * p.scale_log2;
-        if (masked && tok >= s_lim[n]) v = -1e30f;
-        s[n] = v;
-        const float wm = redux_max(v);
-        if (lane == (n & 31)) mine[n >> 5] = wm;
+        for (int n = 0; n < N; ++n)
+          if (tok >= s_lim[n]) s[n] = -INFINITY;
       }
+      // distances to the reference maxima; the maxima themselves are reduced only when a score outgrows its reference
+      float top = -1e30f;
 #pragma unroll
-      for (int k = 0; k < (N + 31) / 32; ++k)
-        if (k * 32 + lane < N) red[warp * N + k * 32 + lane] = mine[k];
-      named_bar_sync(1, 128);
-      if (warp < (N + 31) / 32) {
-        bool up = false;
+      for (int n = 0; n < N; n += 4) {
+        const float4 m = *reinterpret_cast<const float4*>(s_m + n);
+        top = fmaxf(top, fmaxf(fmaxf(s[n] * p.scale_log2 - m.x, s[n + 1] * p.scale_log2 - m.y),
+                               fmaxf(s[n + 2] * p.scale_log2 - m.z, s[n + 3] * p.scale_log2 - m.w)));
+      }
+      const bool outgrown = named_bar_or(1, 128, top > 8.f);
+      if (j >= 2 && ok) ok = mbar_wait(&bar_o[j & 1], static_cast<uint32_t>((j - 2) >> 1) & 1, abort_flag, p.err);
+      if (outgrown) {
+        __syncwarp();
+        float mine[(N + 31) / 32];
+#pragma unroll
+        for (int n = 0; n < N; ++n) {
+          const float wm = redux_max(s[n] * p.scale_log2);
+          if (lane == (n & 31)) mine[n >> 5] = wm;
+        }
+#pragma unroll
+        for (int k = 0; k < (N + 31) / 32; ++k)
+          if (k * 32 + lane < N) red[warp * N + k * 32 + lane] = mine[k];
+        named_bar_sync(1, 128);
         if (r < N) {
           const float tm = fmaxf(fmaxf(red[r], red[N + r]), fmaxf(red[2 * N + r], red[3 * N + r]));
           const float m = s_m[r];
-          up = tm > m + 8.f;
-          s_alpha[r] = up ? exp2f(m - tm) : 1.f;
-          if (up) s_m[r] = tm;
+          s_alpha[r] = tm > m + 8.f ? exp2f(m - tm) : 1.f;
+          if (tm > m + 8.f) s_m[r] = tm;
         }
-        const bool any = __any_sync(0xffffffffu, up);
-        if (lane == 0) s_flag[warp] = any;
-      } else if (warp == 1 && lane == 0) {
-        s_flag[1] = 0;
-      }
-      named_bar_sync(1, 128);
-      const bool rescale = (s_flag[0] | s_flag[1]) != 0;
-      if (j >= 2 && ok) ok = mbar_wait(&bar_o[j & 1], static_cast<uint32_t>((j - 2) >> 1) & 1, abort_flag, p.err);
-      if (rescale) {
+        named_bar_sync(1, 128);
 #pragma unroll
         for (int n = 0; n < N; ++n) l_part[n] *= s_alpha[n];
         if (j > 0) {       // O^T may be rescaled only when the product of tile j - 1 has landed
@@ -285,10 +309,15 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
       const int half = r >> 6, col = r & 63;
       uint8_t* prow = sp + (j & 1) * Layout<N>::kP + half * N * 128 + ((col & 7) << 1);
 #pragma unroll
-      for (int n = 0; n < N; ++n) {
-        const float pv = s[n] > -1e29f ? exp2f(s[n] - s_m[n]) : 0.f;
-        l_part[n] += pv;
-        *reinterpret_cast<__nv_bfloat16*>(prow + n * 128 + (((col >> 3) ^ (n & 7)) << 4)) = __float2bfloat16(pv);
+      for (int n = 0; n < N; n += 4) {
+        const float4 m = *reinterpret_cast<const float4*>(s_m + n);
+        const float mm[4] = {m.x, m.y, m.z, m.w};
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const float pv = exp2f(s[n + i] * p.scale_log2 - mm[i]);      // masked: exp2(-inf) = 0
+          l_part[n + i] += pv;
+          *reinterpret_cast<__nv_bfloat16*>(prow + (n + i) * 128 + (((col >> 3) ^ ((n + i) & 7)) << 4)) = __float2bfloat16(pv);
+        }
       }
       fence_proxy_async();
       tc_fence_before();
@@ -406,6 +435,7 @@ extern "C" int rb_latent_attn_tc(const void* q, const void* pool, const int* blo
   using namespace rb;
   using namespace rb::la;
   if (rows <= 0) return 0;
+  if (!(scale > 0.f)) return -20;            // masking relies on the sign
   if (R % 64 || R > 512 || R < 64 || (page != 16 && page != 32 && page != 64 && page != 128)) return -20;
   if ((width != 16 && width != 32 && width != 64) || splits < 1 || (splits > 1 && (!part_o || !part_ml))) return -2;
   if ((reinterpret_cast<uintptr_t>(q) % 16) || (reinterpret_cast<uintptr_t>(pool) % 16)) return -2;

@@ -48,7 +48,7 @@ def _graph(fn):
 
 
 @torch.no_grad()
-def kernel_rows(H=32, d=128, R=512, W=4096, F=12288, groups=8):
+def kernel_rows(H=32, d=128, R=512, W=4096, F=12288, groups=8, only=""):
     """``(kernel, case, ms, bytes, flops)`` for decode batches and prompts of one real-sized layer."""
     from .. import ops
     from .composed import SegmentBatch
@@ -57,30 +57,32 @@ def kernel_rows(H=32, d=128, R=512, W=4096, F=12288, groups=8):
     rows = []
     mk = lambda *s: torch.randn(*s, device=dev).to(bf)
     i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
+    want = lambda section: not only or section in only.split(",")
     for B in (16, 128):
         # recurrent step: the state is read and written once
         sbytes = B * H * d * d * 4
         fb, lo, nw = mk(H * d), torch.rand(H * d, device=dev).to(bf), mk(d)
         ctx = torch.full((B,), 9, dtype=torch.int32, device=dev)
         fns = []
-        for _ in range(_copies(2 * sbytes)):
+        for _ in range(_copies(2 * sbytes) if want("step") else 0):
             st, x, sl = torch.randn(B, H, d, d, device=dev), mk(B, 3 * H * d), torch.randperm(B, device=dev).to(torch.int32)
             fns.append(_graph(lambda st=st, x=x, sl=sl: ops.hgrn2(x, fb, lo, nw, st, sl, ctx, None, H, d, d, 1e-5)))
-        rows.append(("hgrn2_step", f"batch {B}", _time(fns), 2 * sbytes + B * 4 * H * d * 2, None))
+        if fns:
+            rows.append(("hgrn2_step", f"batch {B}", _time(fns), 2 * sbytes + B * 4 * H * d * 2, None))
         del fns
-        for L in (2048, 8192):
-            if B * L * R * 2 > 3e9:
-                continue
-            nb = L // 16
+        for L, page in () if not want("attn") else ((2048, 16), (2048, 64), (8192, 16), (8192, 64)):
+            nb = L // page
             bt = torch.randperm(B * nb, device=dev).to(torch.int32).view(B, nb)
             cl = torch.full((B,), L, dtype=torch.int32, device=dev)
             fns = []
             for _ in range(_copies(B * L * R * 2)):
                 pool, q, g = mk(B * L, R), mk(B, H, R), mk(B, H)
                 b = SegmentBatch(None, None, cl, bt, None, max_ctx=L)
-                fns.append(_graph(lambda pool=pool, q=q, g=g, b=b: ops.latent_attention(q, pool, b, 16, 0.05, g)))
-            rows.append(("latent_attn decode", f"batch {B}, context {L}", _time(fns), B * L * R * 2, 4.0 * B * L * R * H))
+                fns.append(_graph(lambda pool=pool, q=q, g=g, b=b: ops.latent_attention(q, pool, b, page, 0.05, g)))
+            rows.append(("latent_attn decode", f"batch {B}, context {L}, pages of {page}", _time(fns), B * L * R * 2, 4.0 * B * L * R * H))
             del fns
+            if page != 16:
+                continue
             kvh = 8
             fns = []
             for _ in range(_copies(B * L * kvh * d * 4)):
@@ -88,7 +90,8 @@ def kernel_rows(H=32, d=128, R=512, W=4096, F=12288, groups=8):
                 fns.append(_graph(lambda kc=kc, vc=vc, q=q: ops.paged_decode_attention(q, kc, vc, bt, cl)))
             rows.append(("  like: paged decode attention", f"batch {B}, context {L}", _time(fns), B * L * kvh * d * 4, None))
             del fns
-        wuk, wuv = mk(H, d, R), mk(H, d, R)
+        if not want("gemm"):
+            continue
         q, o = mk(B, H, d), mk(B, H, R)
         ukc = [mk(H, d, R) for _ in range(_copies(H * d * R * 2))]
         rows.append(("head_gemm fold", f"batch {B}", _time([_graph(lambda w=w: ops.head_linear(q, w, False)) for w in ukc]),
@@ -102,8 +105,7 @@ def kernel_rows(H=32, d=128, R=512, W=4096, F=12288, groups=8):
         rows.append(("decode GEMM + gelu unit", f"batch {B}", _time([_graph(lambda w=w: ops.linear_glu(x, w, "gelu_tanh")) for w in wc]), 2 * F * W * 2, None))
         rows.append(("  like: decode GEMM + SwiGLU", f"batch {B}", _time([_graph(lambda w=w: ops.linear_swiglu(x, w)) for w in wc]), 2 * F * W * 2, None))
         del wc
-    T = 8192
-    for T in (128, 8192):
+    for T in (128, 8192) if want("norm") else ():
         n = _copies(T * W * 12)
         w = mk(W)
         buf = [(torch.randn(T, W, device=dev), mk(T, W)) for _ in range(n)]
@@ -112,7 +114,7 @@ def kernel_rows(H=32, d=128, R=512, W=4096, F=12288, groups=8):
         rows.append(("  like: add_rmsnorm (bf16 stream)", f"{T} rows", _time([_graph(lambda r=r, y=y: ops.add_rmsnorm(y, r, w, 1e-5)) for r, y in b2]), T * W * 8, None))
         del buf, b2
     fb, lo, nw = mk(H * d), torch.rand(H * d, device=dev).to(bf), mk(d)
-    for S, L in ((1, 8192), (4, 2048), (32, 256)):
+    for S, L in ((1, 8192), (4, 2048), (32, 256)) if want("prompt") else ():
         T = S * L
         x, st = mk(T, 3 * H * d), torch.zeros(S, H, d, d, device=dev)
         cu, ctx, sl = i32([i * L for i in range(S + 1)]), i32([L] * S), i32(list(range(S)))
@@ -120,7 +122,7 @@ def kernel_rows(H=32, d=128, R=512, W=4096, F=12288, groups=8):
         q, k, v, g = mk(T, H, d), mk(T, H, d), mk(T, H, d), mk(T, H)
         rows.append(("flash + gate (prompt)", f"{S} x {L}", _time([lambda: ops.flash_gated(q, k, v, cu, cu, 0.08, L, g)], 10), T * H * d * 8, 2.0 * T * L * H * d))
         rows.append(("  like: flash attention", f"{S} x {L}", _time([lambda: ops.attention_varlen(q, k, v, cu, True, 0.08, cu, L)], 10), T * H * d * 8, 2.0 * T * L * H * d))
-    for n, L in ((4, 2048), (64, 2048)):
+    for n, L in ((4, 2048), (64, 2048)) if want("attn") else ():
         from .composed import attention_items
 
         S, R_ = 16, R
@@ -196,7 +198,7 @@ def model_rows(size: str, only=None, decode_batches=(1, 32, 128), prompt=2048):
     return out
 
 
-def main(size: str = "5b", peaks: str = "MEASURED_PEAKS.json", kernels: bool = True, models: bool = True) -> int:
+def main(size: str = "5b", peaks: str = "MEASURED_PEAKS.json", kernels: bool = True, models: bool = True, only: str = "") -> int:
     from ..ops import cuda as C
 
     assert C.available()
@@ -204,7 +206,7 @@ def main(size: str = "5b", peaks: str = "MEASURED_PEAKS.json", kernels: bool = T
     hbm, tf = pk.get("hbm_gbs"), pk.get("bf16_tflops")
     if kernels:
         print("kernel | case | us | GB/s (of measured copy) | TFLOP/s (of measured GEMM)")
-        for k, case, ms, nb, fl in kernel_rows():
+        for k, case, ms, nb, fl in kernel_rows(only=only):
             gb = nb / ms / 1e6
             t = f"{gb:7.0f}" + (f" ({gb / hbm:.2f})" if hbm else "")
             if fl:
@@ -216,3 +218,12 @@ def main(size: str = "5b", peaks: str = "MEASURED_PEAKS.json", kernels: bool = T
             print(f"[{size}] {name} | {what} | {tps:,.0f} tokens/s | {ms:.3f} ms", flush=True)
     C.check_error_flag()
     return 0
+
+
+if __name__ == "__main__":
+    import argparse
+
+    ap = argparse.ArgumentParser(description="kernel table of composed stacks")
+    ap.add_argument("--only", default="", help="sections, with commas: step, attn, gemm, norm, prompt")
+    ap.add_argument("--peaks", default="MEASURED_PEAKS.json")
+    raise SystemExit(main(peaks=ap.parse_args().peaks, models=False, only=ap.parse_args().only))
