@@ -383,22 +383,25 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
 __global__ void __launch_bounds__(128) latent_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                                              const __nv_bfloat16* __restrict__ gate, __nv_bfloat16* __restrict__ out,
                                                              int splits, int columns, int H, int R, int ld_gate) {
-  const int col = blockIdx.x;
+  const int col = blockIdx.x, lane = threadIdx.x & 31;
+  // lane s holds the weight of split s (at most 32 splits; splits without positions weigh nothing)
   float m = -1e30f, l = 0.f;
-  for (int s = 0; s < splits; ++s) {
-    const float* ml = part_ml + (static_cast<size_t>(s) * columns + col) * 2;
-    if (ml[1] > 0.f) m = fmaxf(m, ml[0]);
+  if (lane < splits) {
+    const float2 ml = *reinterpret_cast<const float2*>(part_ml + (static_cast<size_t>(lane) * columns + col) * 2);
+    l = ml.y;
+    if (l > 0.f) m = ml.x;
   }
+  const float top = warp_max(m);
+  const float w = l > 0.f ? exp2f(m - top) : 0.f;
+  l = warp_sum(w * l);
   float acc[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 4
   for (int s = 0; s < splits; ++s) {
-    const float* ml = part_ml + (static_cast<size_t>(s) * columns + col) * 2;
-    if (!(ml[1] > 0.f)) continue;
-    const float w = exp2f(ml[0] - m);
-    l += w * ml[1];
+    const float ws = __shfl_sync(0xffffffffu, w, s);
     const float* o = part_o + (static_cast<size_t>(s) * columns + col) * R;
 #pragma unroll
     for (int k = 0; k < 4; ++k)
-      if (threadIdx.x + k * 128 < R) acc[k] += w * o[threadIdx.x + k * 128];
+      if (ws > 0.f && threadIdx.x + k * 128 < R) acc[k] += ws * o[threadIdx.x + k * 128];
   }
   float f = l > 0.f ? 1.f / l : 0.f;
   if (gate) {
@@ -437,7 +440,7 @@ extern "C" int rb_latent_attn_tc(const void* q, const void* pool, const int* blo
   if (rows <= 0) return 0;
   if (!(scale > 0.f)) return -20;            // masking relies on the sign
   if (R % 64 || R > 512 || R < 64 || (page != 16 && page != 32 && page != 64 && page != 128)) return -20;
-  if ((width != 16 && width != 32 && width != 64) || splits < 1 || (splits > 1 && (!part_o || !part_ml))) return -2;
+  if ((width != 16 && width != 32 && width != 64) || splits < 1 || splits > 32 || (splits > 1 && (!part_o || !part_ml))) return -2;
   if ((reinterpret_cast<uintptr_t>(q) % 16) || (reinterpret_cast<uintptr_t>(pool) % 16)) return -2;
   Params p{};
   p.items = items; p.block_tables = block_tables; p.ctx = ctx;

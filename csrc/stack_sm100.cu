@@ -375,14 +375,15 @@ __global__ void __launch_bounds__(512) hgrn2_scan_kernel(const HgrnParams p, int
         else x[r][c].f.y = tf[c];
       }
     }
-  // raw data of the next chunk: token t of unit u = tid + k * nthr is u / NG, features (u % NG) * 8 ..
+  // raw data of the next chunk: this thread prepares features dpre .. dpre + 7 of the tokens tpre and tpre + 8
+  const int tpre = tid / NG, dpre = (tid - tpre * NG) * 8;
   Raw8<T> rq[2], rf[2], rv;
   auto fetch = [&](int t0) {
 #pragma unroll
     for (int k = 0; k < 2; ++k) {
-      const int u = tid + k * nthr, t = u / NG, d = (u - t * NG) * 8;
-      const int valid = t0 + t < hi ? p.dim - d : 0;
-      const T* a = base + static_cast<long long>(t0 + t) * p.ld + hd * p.dim + d;
+      const int t = tpre + 8 * k;
+      const int valid = t0 + t < hi ? p.dim - dpre : 0;
+      const T* a = base + static_cast<long long>(t0 + t) * p.ld + hd * p.dim + dpre;
       rq[k] = raw_load<T, kVec>(a, valid);
       rf[k] = raw_load<T, kVec>(a + qd, valid);
     }
@@ -391,9 +392,6 @@ __global__ void __launch_bounds__(512) hgrn2_scan_kernel(const HgrnParams p, int
       rv = raw_load<T, kVec>(base + static_cast<long long>(t0 + t) * p.ld + 2 * qd + hd * p.vdim + v0 + j, t0 + t < hi ? nv - j : 0);
     }
   };
-  // the biases and bounds of the eight features this thread prepares (the same for both of its units when NG divides
-  // the thread count, which it does: nthr = 8 NG)
-  const int dpre = (tid % NG) * 8;
   float fb[8], fl[8];
 #pragma unroll
   for (int i = 0; i < 8; ++i) {
@@ -406,7 +404,7 @@ __global__ void __launch_bounds__(512) hgrn2_scan_kernel(const HgrnParams p, int
     const int n = min(SC_CH, hi - t0);
 #pragma unroll
     for (int k = 0; k < 2; ++k) {
-      const int t = (tid + k * nthr) / NG;
+      const int t = tpre + 8 * k;
       F8 a, b, c;
 #pragma unroll
       for (int i = 0; i < 8; ++i) {
@@ -461,11 +459,24 @@ __global__ void __launch_bounds__(512) hgrn2_scan_kernel(const HgrnParams p, int
       *reinterpret_cast<float4*>(part + (t * NG + g) * SC_V + c4) = o;
     }
     __syncthreads();
-    for (int i = tid; i < n * SC_V; i += nthr) {
-      const int t = i / SC_V, j = i - t * SC_V;
-      float o = 0.f;
-      for (int k = 0; k < NG; ++k) o += part[(t * NG + k) * SC_V + j];
-      if (j < nv) p.o_raw[(static_cast<long long>(t0 + t) * p.H + hd) * p.vdim + v0 + j] = o;
+    for (int i = tid; i < n * (SC_V / 4); i += nthr) {      // four columns of one token
+      const int t = i >> 3, j = (i & 7) * 4;
+      const float4* a = reinterpret_cast<const float4*>(part + t * NG * SC_V + j);
+      float4 o = a[0];
+#pragma unroll 4
+      for (int k = 1; k < NG; ++k) {
+        const float4 b = a[k * (SC_V / 4)];
+        o.x += b.x; o.y += b.y; o.z += b.z; o.w += b.w;
+      }
+      float* d = p.o_raw + (static_cast<long long>(t0 + t) * p.H + hd) * p.vdim + v0 + j;
+      if (p.vdim % 4 == 0) {
+        if (j < nv) *reinterpret_cast<float4*>(d) = o;
+      } else {
+        const float of[4] = {o.x, o.y, o.z, o.w};
+#pragma unroll
+        for (int c = 0; c < 4; ++c)
+          if (j + c < nv) d[c] = of[c];
+      }
     }
   }
   if (cols) {
@@ -697,7 +708,8 @@ static int launch_latent_attn(const LatentParams& p, int rows, cudaStream_t stm)
 
 template <typename T>
 static int launch_scan(const HgrnParams& p, int segs, int rows, bool vec, cudaStream_t stm) {
-  const int NG = (p.dim + 31) / 32 * 4;           // row groups of 8; whole warps (8 lanes per group)
+  int NG = (p.dim + 31) / 32 * 4;                 // row groups of 8; whole warps (8 lanes per group)
+  if (NG < 8) NG = 8;                             // at least 64 threads: they also fetch the values of a chunk
   if (NG * 8 > 512) return -2;
   const size_t smem = (static_cast<size_t>(SC_CH) * (3 * NG * 8 + 2 * SC_V + NG * SC_V)) * 4;
   if (smem > 227 * 1024) return -2;
