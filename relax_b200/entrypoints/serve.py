@@ -7,7 +7,8 @@
 * ``viewer``      - the rollout result viewer (relax/entrypoints/visualize.py);
 * ``engine``      - one rollout engine behind HTTP (``/generate``, ``/flush_cache``, ``/pause_generation``,
   ``/continue_generation``, ``/abort_request``, ``/get_server_info``; relax/backends/sglang/sglang_engine.py talks to
-  its engines over the same surface); weights from ``--hf-checkpoint``;
+  its engines over the same surface); weights from ``--hf-checkpoint`` (a Hugging Face layout of the preset, or a model that
+  describes itself, e.g. a Talizen folder);
 * ``router``      - the request router as an HTTP proxy in front of engine servers (least loaded / sticky by key,
   health probes, ``/add_worker`` ``/remove_worker`` ``/list_workers``; relax/engine/router/router.py);
 * ``teacher``     - an on-policy-distillation teacher: ``POST /score`` returns the teacher's log-probs of the response
@@ -22,10 +23,32 @@ import sys
 import time
 
 
+def engine_config(model_name: str, checkpoint=None):
+    """The preset, or the model a checkpoint describes itself when its ``config.json`` names a design of its own
+    (:mod:`relax_b200.models.architectures`)."""
+    import json
+    import os
+
+    from ..checkpoint.hf import config_from_hf
+    from ..models.architectures import architecture_of
+    from ..models.config import get_config
+
+    cj = os.path.join(checkpoint, "config.json") if checkpoint else None
+    if cj and os.path.isfile(cj):
+        with open(cj) as f:
+            if architecture_of(json.load(f)) is not None:
+                return config_from_hf(checkpoint)
+    return get_config(model_name)
+
+
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser(description="relax_b200 control-plane services")
     ap.add_argument("service", choices=["metrics", "coordinator", "viewer", "teacher", "router", "engine"])
     ap.add_argument("--kv-blocks", type=int, default=4096, help="engine: KV-cache blocks of 16 tokens")
+    ap.add_argument("--dtype", choices=["bfloat16", "float32"], default=None, help="engine: default bfloat16 on a GPU, float32 on the CPU")
+    ap.add_argument("--state-slots", type=int, default=None, help="engine: most live requests of a composed stack (recurrent states)")
+    ap.add_argument("--max-model-len", type=int, default=4096, help="engine: longest request the captured decode windows take")
+    ap.add_argument("--eos-token-id", type=int, default=None, help="engine: token that ends a request")
     ap.add_argument("--speculative-steps", type=int, default=0,
                     help="engine: proposals per pass drafted by the model's multi-token-prediction block (0 = off)")
     ap.add_argument("--workers", nargs="*", default=None, help="router: base URLs of the engine servers to start with")
@@ -61,15 +84,15 @@ def main(argv=None) -> int:
     elif a.service == "engine":
         import torch
 
-        from ..models.config import get_config
         from ..rollout.engine import RolloutEngine
         from ..rollout.http_server import EngineServer
 
         dev = a.device or ("cuda" if torch.cuda.is_available() else "cpu")
-        cfg = get_config(a.model_name)
-        eng = RolloutEngine(cfg, device=dev, dtype=torch.bfloat16 if dev.startswith("cuda") else torch.float32,
-                            num_kv_blocks=a.kv_blocks, block_size=16, seed=a.seed, speculative=a.speculative_steps > 0,
-                            speculative_steps=max(1, a.speculative_steps))
+        cfg = engine_config(a.model_name, a.hf_checkpoint)
+        dtype = {"bfloat16": torch.bfloat16, "float32": torch.float32}.get(a.dtype) or (torch.bfloat16 if dev.startswith("cuda") else torch.float32)
+        eng = RolloutEngine(cfg, device=dev, dtype=dtype, num_kv_blocks=a.kv_blocks, block_size=16, seed=a.seed,
+                            speculative=a.speculative_steps > 0, speculative_steps=max(1, a.speculative_steps),
+                            state_slots=a.state_slots, max_model_len=a.max_model_len, eos_token_id=a.eos_token_id)
         if a.hf_checkpoint:
             from ..checkpoint import hf as H
 

@@ -271,6 +271,8 @@ class GPTModel(nn.Module):
     def __init__(self, cfg: ModelConfig, ps: Optional[ParallelState] = None, device="cpu", seed: int = 0,
                  dtype: Optional[torch.dtype] = None, recompute: bool = False, pp_layers: Optional[range] = None):
         super().__init__()
+        if cfg.is_composed:
+            raise NotImplementedError(f"{cfg.name}: composed stacks are served by the rollout engine; there is no trainer model of them")
         self.cfg = cfg
         self.ps = ps or single_process_state()
         self.dtype = dtype or _DTYPES[cfg.dtype]

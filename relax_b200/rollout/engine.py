@@ -304,6 +304,8 @@ class RolloutEngine(SpeculativeMixin, ComposedScheduler):
         (an attached vision tower embeds them at prefill) or ready ``image_embeds``.  Requests that share a
         ``group_key`` must carry the same prompt AND the same images: followers reuse the leader's prompt KV."""
         r = Request(self._next_rid, list(prompt), params, group_key, t_arrive=time.perf_counter())
+        if self.composed and not r.prompt:
+            raise ValueError("an empty prompt")
         if grid_thw is not None:
             from ..models.vision import mrope_positions
 

@@ -53,6 +53,8 @@ def detach(engine: RolloutEngine, reqs: Sequence[Request]) -> List[PrefilledRequ
     """Take ``reqs`` (running on ``engine``, prefilled) out of it together with their KV rows; frees their blocks."""
     if getattr(engine, "hybrid", False):
         raise NotImplementedError("the hand-over moves paged K/V; the recurrent state of Gated-DeltaNet layers does not travel yet")
+    if engine.composed:
+        raise NotImplementedError("the hand-over moves paged K/V; latent rows and state slots of composed stacks do not travel yet")
     out = []
     bs = engine.block_size
     for r in reqs:
