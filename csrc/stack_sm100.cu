@@ -215,11 +215,12 @@ constexpr int HS_THREADS = 256;
 template <typename T>
 __global__ void __launch_bounds__(HS_THREADS) hgrn2_step_kernel(const HgrnParams p) {
   constexpr bool kExact = IsExact<T>::v;
-  extern __shared__ float sm[];
+  extern __shared__ __align__(16) float sm[];
+  const int dp = (p.dim + 3) & ~3;      // the rows behind are read four values at a time
   float* sq = sm;                       // [dim]
-  float* sg = sq + p.dim;               // [dim] forget gate
-  float* sk = sg + p.dim;               // [dim] 1 - gate
-  float* sv = sk + p.dim;               // [vp]
+  float* sg = sq + dp;                  // [dim] forget gate
+  float* sk = sg + dp;                  // [dim] 1 - gate
+  float* sv = sk + dp;                  // [vp]
   float* red = sv + p.vp;               // [ng][vp]
   __shared__ float wred[HS_THREADS / 32];
   const int s = blockIdx.x, hd = blockIdx.y, tid = threadIdx.x;
@@ -772,7 +773,7 @@ extern "C" int rb_hgrn2(const void* qfv, const void* f_bias, const void* lower, 
     return fp32 ? launch_scan<float>(p, segs, rows, vec, stm) : launch_scan<bf16>(p, segs, rows, vec, stm);
   }
   const int lpr = vp / 4, ng = HS_THREADS / lpr;
-  const size_t smem = (3 * static_cast<size_t>(dim) + vp + static_cast<size_t>(ng) * vp) * 4;
+  const size_t smem = (3 * static_cast<size_t>((dim + 3) & ~3) + vp + static_cast<size_t>(ng) * vp) * 4;
   if (smem > 48 * 1024) return -2;
   if (fp32) hgrn2_step_kernel<float><<<dim3(segs, H), HS_THREADS, smem, stm>>>(p);
   else hgrn2_step_kernel<bf16><<<dim3(segs, H), HS_THREADS, smem, stm>>>(p);

@@ -143,8 +143,12 @@ def tokens(cfg, n, seed):
     return torch.randint(0, cfg["vocab"], (n,), generator=g).tolist()
 
 
-def distance(got, want):
-    """Largest over the positions of the root-mean-square difference of logits (means removed), in units of their spread."""
+def distances(got, want):
+    """Per position the root-mean-square difference of logits (means removed), in units of their spread."""
     d = got.to(F64).cpu() - want
     d = d - d.mean(-1, keepdim=True)
-    return float((d ** 2).mean(-1).sqrt().max() / (want - want.mean(-1, keepdim=True)).pow(2).mean().sqrt())
+    return (d ** 2).mean(-1).sqrt() / (want - want.mean(-1, keepdim=True)).pow(2).mean().sqrt()
+
+
+def distance(got, want):
+    return float(distances(got, want).max())
