@@ -136,6 +136,9 @@ int rb_norm_add(float* res, const void* y, const void* w, const void* next_w, vo
 int rb_hgrn2(const void* qfv, const void* f_bias, const void* lower, const void* norm_w, float* state, const int* slot, const int* ctx,
              const int* cu, float* o_raw, void* out, int rows, int segs, int H, int dim, int vdim, int vp, int ld, int ldo, float eps,
              int fp32, cudaStream_t st);
+int rb_hgrn2_chunk(const void* qfv, const void* f_bias, const void* lower, const void* norm_w, float* state, const int* slot, const int* ctx,
+                   const int* cu, const int* spans, const int* first, float* span_state, float* span_gate, void* out, int rows, int segs,
+                   int n_spans, int H, int dim, int vdim, int vp, int ld, int ldo, float eps, cudaStream_t st);
 int rb_latent_write(const void* raw, int ld_raw, const void* w, void* pool, const long long* slots, long long pool_rows, int rows,
                     int rank, int pitch, float eps, int fp32, cudaStream_t st);
 int rb_latent_attn(const void* q, const void* pool, const int* block_tables, const int* row_seg, const int* row_pos, const int* ctx,

@@ -152,9 +152,11 @@ void norm_add(torch::Tensor res, torch::Tensor y, torch::Tensor w, c10::optional
                     (int)res.size(1), (int)width, (int)groups, (float)eps, is_fp32(y), cur_stream()),
         "rb_norm_add");
 }
-void hgrn2(torch::Tensor qfv, torch::Tensor f_bias, torch::Tensor lower, torch::Tensor norm_w, torch::Tensor state, torch::Tensor slot,
-           torch::Tensor ctx, c10::optional<torch::Tensor> cu, c10::optional<torch::Tensor> o_raw, torch::Tensor out, int64_t dim,
-           int64_t vdim, double eps) {
+// Returns false when `o_raw` is not given and the shape is outside what the tensor-core kernel takes.
+bool hgrn2(torch::Tensor qfv, torch::Tensor f_bias, torch::Tensor lower, torch::Tensor norm_w, torch::Tensor state, torch::Tensor slot,
+           torch::Tensor ctx, c10::optional<torch::Tensor> cu, c10::optional<torch::Tensor> o_raw, c10::optional<torch::Tensor> spans,
+           c10::optional<torch::Tensor> first, c10::optional<torch::Tensor> span_state, c10::optional<torch::Tensor> span_gate,
+           torch::Tensor out, int64_t dim, int64_t vdim, double eps) {
   const c10::cuda::CUDAGuard guard(qfv.device());
   for (const auto& t : {f_bias, lower, norm_w, out}) check_same(qfv, t, "hgrn2");
   const int64_t H = state.size(1), rows = qfv.size(0), segs = slot.numel();
@@ -164,6 +166,23 @@ void hgrn2(torch::Tensor qfv, torch::Tensor f_bias, torch::Tensor lower, torch::
   TORCH_CHECK(slot.scalar_type() == at::kInt && ctx.scalar_type() == at::kInt && ctx.numel() == segs && slot.is_contiguous() && ctx.is_contiguous());
   if (cu.has_value()) {
     TORCH_CHECK(cu->scalar_type() == at::kInt && cu->numel() == segs + 1 && cu->is_contiguous());
+    if (!o_raw.has_value()) {      // tensor-core chunks (bf16)
+      TORCH_CHECK(qfv.scalar_type() == at::kBFloat16, "hgrn2: the 32-bit scan needs its scratch");
+      const int64_t n = spans.has_value() ? spans->size(0) : 0;
+      if (n) {
+        TORCH_CHECK(spans->scalar_type() == at::kInt && spans->dim() == 2 && spans->size(1) == 2 && spans->is_contiguous());
+        TORCH_CHECK(first.has_value() && first->scalar_type() == at::kInt && first->numel() == segs + 1 && first->is_contiguous());
+        TORCH_CHECK(span_state.has_value() && span_state->scalar_type() == at::kFloat && span_state->numel() >= n * state.stride(0));
+        TORCH_CHECK(span_gate.has_value() && span_gate->scalar_type() == at::kFloat && span_gate->numel() >= n * H * dim);
+      }
+      const int rc = rb_hgrn2_chunk(qfv.data_ptr(), f_bias.data_ptr(), lower.data_ptr(), norm_w.data_ptr(), state.data_ptr<float>(),
+                                    slot.data_ptr<int>(), ctx.data_ptr<int>(), cu->data_ptr<int>(), n ? spans->data_ptr<int>() : nullptr,
+                                    n ? first->data_ptr<int>() : nullptr, n ? span_state->data_ptr<float>() : nullptr,
+                                    n ? span_gate->data_ptr<float>() : nullptr, out.data_ptr(), (int)rows, (int)segs, (int)n, (int)H, (int)dim, (int)vdim, (int)state.size(3), (int)qfv.stride(0), (int)out.size(1), (float)eps, cur_stream());
+      if (rc == -20) return false;
+      check(rc, "rb_hgrn2_chunk");
+      return true;
+    }
     TORCH_CHECK(o_raw.has_value() && o_raw->scalar_type() == at::kFloat && o_raw->numel() >= rows * H * vdim);
   } else {
     TORCH_CHECK(segs == rows, "hgrn2: one row per segment");
@@ -172,6 +191,7 @@ void hgrn2(torch::Tensor qfv, torch::Tensor f_bias, torch::Tensor lower, torch::
                  ctx.data_ptr<int>(), optint(cu), o_raw.has_value() ? o_raw->data_ptr<float>() : nullptr, out.data_ptr(), (int)rows, (int)segs,
                  (int)H, (int)dim, (int)vdim, (int)state.size(3), (int)qfv.stride(0), (int)out.size(1), (float)eps, is_fp32(qfv), cur_stream()),
         "rb_hgrn2");
+  return true;
 }
 void latent_write(torch::Tensor raw, torch::Tensor w, torch::Tensor pool, torch::Tensor slots, int64_t rank, double eps) {
   const c10::cuda::CUDAGuard guard(raw.device());

@@ -70,9 +70,12 @@ def norm_add(res, y, w, width, groups, eps, next_w=None):
     return (_cuda() if _use_cuda(y) else ref).norm_add(res, y, w, width, groups, eps, next_w)
 
 
-def hgrn2(qfv, f_bias, lower, norm_w, state, state_slot, ctx_lens, cu, heads, dim, vdim, eps):
-    """HGRN2 token mixing (gates, recurrence, per-head norm) on packed rows with the state carried in slots."""
-    return (_cuda() if _use_cuda(qfv) else ref).hgrn2(qfv, f_bias, lower, norm_w, state, state_slot, ctx_lens, cu, heads, dim, vdim, eps)
+def hgrn2(qfv, f_bias, lower, norm_w, state, state_slot, ctx_lens, cu, heads, dim, vdim, eps, spans=None):
+    """HGRN2 token mixing (gates, recurrence, per-head norm) on packed rows with the state carried in slots.  ``spans``:
+    ``(row ranges [n, 2], first span of every segment [S + 1])`` lets long segments run in parts side by side."""
+    if _use_cuda(qfv):
+        return _cuda().hgrn2(qfv, f_bias, lower, norm_w, state, state_slot, ctx_lens, cu, heads, dim, vdim, eps, spans)
+    return ref.hgrn2(qfv, f_bias, lower, norm_w, state, state_slot, ctx_lens, cu, heads, dim, vdim, eps)
 
 
 def latent_write(raw, w, rank, eps, pool, slots):

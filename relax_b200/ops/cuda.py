@@ -319,11 +319,19 @@ def norm_add(res, y, w, width, groups, eps, next_w=None):
     return h
 
 
-def hgrn2(qfv, f_bias, lower, norm_w, state, state_slot, ctx_lens, cu, heads, dim, vdim, eps):
+def hgrn2(qfv, f_bias, lower, norm_w, state, state_slot, ctx_lens, cu, heads, dim, vdim, eps, spans=None):
     T = qfv.shape[0]
+    sp, first = spans if spans is not None else (None, None)
     out = torch.empty(T, (heads * vdim + 7) // 8 * 8, dtype=qfv.dtype, device=qfv.device)
-    raw = None if cu is None else torch.empty(T, heads, vdim, dtype=torch.float32, device=qfv.device)
-    _load().hgrn2(qfv, f_bias, lower, norm_w, state, state_slot, ctx_lens, cu, raw, out, int(dim), int(vdim), float(eps))
+    st = gt = None
+    if sp is not None and qfv.dtype == torch.bfloat16:
+        st = torch.empty(sp.shape[0], *state.shape[1:], dtype=torch.float32, device=qfv.device)
+        gt = torch.empty(sp.shape[0], heads, dim, dtype=torch.float32, device=qfv.device)
+    run = lambda raw: _load().hgrn2(qfv, f_bias, lower, norm_w, state, state_slot, ctx_lens, cu, raw, sp, first, st, gt, out, int(dim),
+                                    int(vdim), float(eps))
+    if (cu is None or qfv.dtype == torch.bfloat16) and run(None):      # decode step, or segments on the tensor cores
+        return out
+    run(torch.empty(T, heads, vdim, dtype=torch.float32, device=qfv.device))      # 32-bit mode and head sizes of odd shape
     return out
 
 

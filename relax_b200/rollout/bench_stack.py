@@ -51,7 +51,7 @@ def _graph(fn):
 def kernel_rows(H=32, d=128, R=512, W=4096, F=12288, groups=8, only=""):
     """``(kernel, case, ms, bytes, flops)`` for decode batches and prompts of one real-sized layer."""
     from .. import ops
-    from .composed import SegmentBatch
+    from .composed import SegmentBatch, recurrent_spans
 
     dev, bf = "cuda", torch.bfloat16
     rows = []
@@ -117,8 +117,10 @@ def kernel_rows(H=32, d=128, R=512, W=4096, F=12288, groups=8, only=""):
     for S, L in ((1, 8192), (4, 2048), (32, 256)) if want("prompt") else ():
         T = S * L
         x, st = mk(T, 3 * H * d), torch.zeros(S, H, d, d, device=dev)
+        spans = recurrent_spans([L] * S, H)
+        spans = None if spans is None else (i32(spans[0]), i32(spans[1]))
         cu, ctx, sl = i32([i * L for i in range(S + 1)]), i32([L] * S), i32(list(range(S)))
-        rows.append(("hgrn2 prompt", f"{S} x {L}", _time([lambda: ops.hgrn2(x, fb, lo, nw, st, sl, ctx, cu, H, d, d, 1e-5)], 10), T * H * d * 4 * 2, 6.0 * T * H * d * d))
+        rows.append(("hgrn2 prompt", f"{S} x {L}", _time([lambda: ops.hgrn2(x, fb, lo, nw, st, sl, ctx, cu, H, d, d, 1e-5, spans)], 10), T * H * d * 4 * 2, 6.0 * T * H * d * d))
         q, k, v, g = mk(T, H, d), mk(T, H, d), mk(T, H, d), mk(T, H)
         rows.append(("flash + gate (prompt)", f"{S} x {L}", _time([lambda: ops.flash_gated(q, k, v, cu, cu, 0.08, L, g)], 10), T * H * d * 8, 2.0 * T * L * H * d))
         rows.append(("  like: flash attention", f"{S} x {L}", _time([lambda: ops.attention_varlen(q, k, v, cu, True, 0.08, cu, L)], 10), T * H * d * 8, 2.0 * T * L * H * d))

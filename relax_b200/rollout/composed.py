@@ -115,6 +115,7 @@ class SegmentBatch:
     row_pos: Optional[torch.Tensor] = None
     max_ctx: int = 0                         # host upper bound of the short segments' contexts
     items: Optional[dict] = None
+    spans: Optional[tuple] = None            # row ranges of recurrent spans and the first span of every segment
 
 
 def attention_items(lens: Sequence[int], ctx: Sequence[int], heads: int, width: int = 64) -> list:
@@ -128,6 +129,20 @@ def attention_items(lens: Sequence[int], ctx: Sequence[int], heads: int, width: 
             out.append([s, c, min(step, (row0 + n) * heads - c), L - n - row0 + 1])
         row0 += n
     return out
+
+
+def recurrent_spans(lens: Sequence[int], heads: int, ctas: int = 296, shortest: int = 128) -> Optional[tuple]:
+    """Cut long segments into spans so that (spans x heads) fills the machine (``ctas`` at a time); spans are multiples of
+    the kernel's 16-token chunks.  ``(row ranges, first span of every segment)``, None when no segment is worth cutting."""
+    size = max(shortest, pad_to(-(-sum(lens) * heads // ctas), 16))
+    spans, first, row = [], [0], 0
+    for n in lens:
+        k = max(1, round(n / size))
+        step = pad_to(-(-n // k), 16)
+        spans += [[row + a, row + min(n, a + step)] for a in range(0, n, step)]
+        first.append(len(spans))
+        row += n
+    return (spans, first) if len(spans) > len(lens) else None
 
 
 class ComposedForward:
@@ -172,7 +187,7 @@ class ComposedForward:
         s, p, pre = self.cfg.layer_specs[i], self.p, f"layers.{i}."
         qfv = ops.linear(h, p[pre + "rec_qfv"])
         o = ops.hgrn2(qfv, p[pre + "rec_f_bias"], p[pre + "rec_lower"], p[pre + "rec_norm"], cache.state[i], b.state_slot,
-                      b.ctx, b.cu, s.heads, s.dim, s.vdim, self.cfg.rms_norm_eps)
+                      b.ctx, b.cu, s.heads, s.dim, s.vdim, self.cfg.rms_norm_eps, b.spans)
         return ops.linear(o, p[pre + "rec_o"])
 
     def _latent(self, i, h, b: SegmentBatch, cache: StackCache):
@@ -291,6 +306,10 @@ class ComposedScheduler:
                 arrays["long_cu_k"] = (ck, i32)
                 arrays["ctx_slots"] = ([x for j in order[:n_long] for x in self._slots(parts[j][0], 0, parts[j][0].fed + parts[j][1])], i64)
                 host["long_max"] = max(lens[:n_long])
+            rec = [self.cfg.layer_specs[i].heads for i in self.cfg.layers_with("hgrn2")]
+            cuts = recurrent_spans(lens, max(rec)) if rec and self.device.type == "cuda" else None
+            if cuts is not None:
+                arrays["spans"], arrays["span_first"] = (cuts[0], i32), (cuts[1], i32)
             if sl:
                 arrays["short_cu"] = ([c - cu[n_long] for c in cu[n_long:]], i32)
                 arrays["row_seg"] = ([s for s, n in enumerate(sl) for _ in range(n)], i32)
@@ -302,8 +321,9 @@ class ComposedScheduler:
             arrays["rows"] = (rows, i64)
         dev = dict(zip(arrays, self._stage(list(arrays.values()))))
         want_t = dev.pop("rows", None)
+        spans = (dev.pop("spans"), dev.pop("span_first")) if "spans" in dev else None
         items = {H: dev.pop(f"items{H}") for H in heads}
-        batch = SegmentBatch(**dev, **host, items=items or None)
+        batch = SegmentBatch(**dev, **host, items=items or None, spans=spans)
         logits = self.weights.forward_segments(batch, self.kv, want_t, self.tp, taps)
         for r, n in parts:
             r.fed += n

@@ -196,6 +196,21 @@ def test_attention_items_cover_every_column_once():
         assert seen == list(range(sum(lens) * heads))
 
 
+def test_recurrent_spans_cover_every_row_in_whole_chunks():
+    from relax_b200.rollout.composed import recurrent_spans
+
+    assert recurrent_spans([5, 1, 100], 2) is None
+    for lens, heads in (([8192], 32), ([1, 700, 3, 2049], 16), ([260], 1), ([4000, 4000, 1], 64)):
+        spans, first = recurrent_spans(lens, heads, shortest=64)
+        row = 0
+        for s, n in enumerate(lens):
+            part = spans[first[s]:first[s + 1]]
+            assert part[0][0] == row and part[-1][1] == row + n
+            assert all(a[1] == b[0] and (a[1] - a[0]) % 16 == 0 for a, b in zip(part, part[1:])) and all(b > a for a, b in part)
+            row += n
+        assert first[-1] == len(spans) > len(lens)
+
+
 def test_trace_replay_writes_the_wanted_logits(tmp_path):
     from relax_b200.entrypoints import trace
     from relax_b200.models import talizen

@@ -139,7 +139,7 @@ def test_hgrn2_segments_and_steps(dtype, H, dim, vdim):
     for s in range(len(lens)):
         want, S1 = _hgrn_plain(x[cu[s]:cu[s + 1]], fb, lo, nw, H, dim, vdim, eps, S0[s])
         _close(out[cu[s]:cu[s + 1], :H * vdim].cpu(), want, _tol(dtype) if dtype == torch.bfloat16 else 2e-5)
-        _close(state[slots[s], :, :, :vdim].cpu(), S1, 2e-4 if dtype == torch.bfloat16 else 1e-5)
+        _close(state[slots[s], :, :, :vdim].cpu(), S1, 2e-5)
         S0[s] = S1
     assert not out[:, H * vdim:].any() and not state[slots][..., vdim:].any()
     for _ in range(2):
@@ -154,6 +154,31 @@ def test_hgrn2_segments_and_steps(dtype, H, dim, vdim):
     out = ops.hgrn2(x1, fb, lo, nw, state, i32(slots), i32([1] * len(lens)), None, H, dim, vdim, eps)
     want, S1 = _hgrn_plain(x1[2:3], fb, lo, nw, H, dim, vdim, eps, torch.zeros(H, dim, vdim, dtype=F64))
     _close(state[slots[2], :, :, :vdim].cpu(), S1, 1e-5)
+
+
+@pytest.mark.parametrize("H,dim,vdim", [(2, 128, 128), (3, 48, 40), (1, 16, 128)])
+def test_hgrn2_spans_side_by_side(H, dim, vdim):
+    """Long segments cut into spans that run in parallel, beside segments of one span and of one token."""
+    from relax_b200 import ops
+    from relax_b200.rollout.composed import recurrent_spans
+
+    eps, lens, before = 1e-5, [1, 230, 16, 97], [4, 11, 0, 0]
+    x, fb, lo, nw = _hgrn_case(torch.bfloat16, H, dim, vdim, sum(lens), 31)
+    lo = 1 - lo * 0.05                                 # gates near one: what a span inherits matters to its end
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device="cuda")
+    cu = [0]
+    for n in lens:
+        cu.append(cu[-1] + n)
+    cuts = recurrent_spans(lens, H, ctas=10 ** 6, shortest=32)
+    assert [b - a for a, b in zip(cuts[1], cuts[1][1:])] == [1, 5, 1, 3]
+    state = _rand(9, 6, H, dim, (vdim + 3) // 4 * 4)
+    slots = [3, 1, 5, 0]
+    S0 = [torch.zeros(H, dim, vdim, dtype=F64) if b == 0 else state[s, :, :, :vdim].to(F64).cpu() for s, b in zip(slots, before)]
+    out = ops.hgrn2(x, fb, lo, nw, state, i32(slots), i32([b + n for b, n in zip(before, lens)]), i32(cu), H, dim, vdim, eps, (i32(cuts[0]), i32(cuts[1])))
+    for s in range(len(lens)):
+        want, S1 = _hgrn_plain(x[cu[s]:cu[s + 1]], fb, lo, nw, H, dim, vdim, eps, S0[s])
+        _close(out[cu[s]:cu[s + 1], :H * vdim].cpu(), want, 2e-2)
+        _close(state[slots[s], :, :, :vdim].cpu(), S1, 2e-5)
 
 
 @BOTH
@@ -175,7 +200,7 @@ def test_hgrn2_gates_at_their_ends(dtype):
     out = ops.hgrn2(x, fb, lo, nw, state, i32([1]), i32([T + 4]), i32([0, T]), H, dim, vdim, 1e-5)
     want, S1 = _hgrn_plain(x, fb, lo, nw, H, dim, vdim, 1e-5, keep.to(F64).cpu())
     _close(out.cpu(), want, _tol(dtype) if dtype == torch.bfloat16 else 2e-5)
-    _close(state[1].cpu(), S1, 2e-4 if dtype == torch.bfloat16 else 1e-5)
+    _close(state[1].cpu(), S1, 2e-5)
     assert torch.equal(state[1, 0, 16:32], keep[0, 16:32]) and torch.equal(state[1, 0, 48:], keep[0, 48:])
 
 
