@@ -10,8 +10,8 @@
 // The columns of a group belong to one sequence: the heads of one decoded token, or of several consecutive tokens of a
 // prompt portion, each with its own causal limit.  Rows are gathered page by page with TMA into the 128-byte swizzled
 // layout; a ring of 32 KB slots (128 positions x 128 latent features) keeps loads in flight while a tile is processed: a
-// slot is free again when the O product has read it.  One thread owns one position of S^T (and one latent feature of
-// O^T); maxima are shared by the CTA, the accumulator is rescaled lazily (threshold 2^8, decided for the whole CTA).
+// slot is free again when the O product has read it.  Two threads share a position of S^T (and a latent feature of
+// O^T), each with half of the columns; maxima are shared by the CTA, the accumulator is rescaled lazily (threshold 2^8, decided for the whole CTA).
 // CTA = (column group, split of the positions); partial results of several splits are merged by a second kernel, which
 // also applies the output gate.  Every wait is bounded; no load uses cluster multicast.
 #include "common.cuh"
@@ -23,7 +23,8 @@ namespace la {
 constexpr int TILE = 128;                 // positions per tile
 constexpr int SLOT = 32768;               // ring slot: two 64-feature chunks of a tile
 constexpr int MAX_SLOTS = 5;
-constexpr int THREADS = 192;
+constexpr int SOFTMAX = 256;               // eight warps: positions by warp % 4, columns by halves
+constexpr int THREADS = SOFTMAX + 64;      // and a TMA and an MMA warp
 constexpr int SCRATCH = 2560;               // barriers (256 B), then 8 N words
 
 struct Params {
@@ -54,6 +55,18 @@ __device__ __forceinline__ bool named_bar_or(int id, int threads, bool v) {
       : "r"(static_cast<uint32_t>(v)), "r"(id), "r"(threads)
       : "memory");
   return r != 0;
+}
+
+// W consecutive accumulator columns of this warp's 32 lanes
+template <int W>
+__device__ __forceinline__ void tmem_get(uint32_t addr, uint32_t* r) {
+  if constexpr (W == 8) tmem_ld_32x32b_x8(addr, r);
+  else tmem_ld_32x32b_x16(addr, r);
+}
+template <int W>
+__device__ __forceinline__ void tmem_put(uint32_t addr, const uint32_t* r) {
+  if constexpr (W == 8) tmem_st_32x32b_x8(addr, r);
+  else tmem_st_32x32b_x16(addr, r);
 }
 
 template <int N>
@@ -111,7 +124,7 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
     mbar_init(bar_q, 1);
     for (int i = 0; i < 2; ++i) {
       mbar_init(&bar_s[i], 1);
-      mbar_init(&bar_p[i], 128);
+      mbar_init(&bar_p[i], SOFTMAX);
       mbar_init(&bar_o[i], 1);
     }
     for (int s = 0; s < p.slots; ++s) {
@@ -135,7 +148,7 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
     if (live && p.gate) g = 1.f / (1.f + __expf(-__bfloat162float(p.gate[static_cast<size_t>(row) * p.ld_gate + (c - row * p.H)])));
     s_gate[n] = g;
   }
-  if (warp == 5) {
+  if (warp == 9) {
     tmem_alloc<kTmemCols>(tmem_slot);
     tmem_relinquish();
   }
@@ -145,7 +158,7 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
   const uint32_t tmem_base = *tmem_slot;
   const bool dead = (*abort_flag != 0);
 
-  if (warp == 4) {
+  if (warp == 8) {
     // ================================================================ TMA producer (page gather)
     // lane i gathers page i of every tile: the page number is looked up once per tile and the copies of a slot are issued
     // by all lanes together
@@ -180,7 +193,7 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
         row = next;
       }
     }
-  } else if (warp == 5) {
+  } else if (warp == 9) {
     // ================================================================ MMA issuer
     if (lane == 0 && !dead && n_tiles > 0) {
       const uint32_t id_s = make_idesc_f16(TILE, N, true, false, false);
@@ -232,60 +245,62 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
       }
     }
   } else {
-    // ================================================================ softmax + epilogue (warps 0..3)
-    const int r = warp * 32 + lane;          // position of the tile, latent feature of a pair
-    const uint32_t lane_addr = static_cast<uint32_t>(warp * 32) << 16;
-    float l_part[N];
+    // ================================================================ softmax + epilogue (warps 0..7)
+    constexpr int NH = N / 2, CW = NH < 16 ? NH : 16;
+    const int quad = warp & 3;
+    const int r = quad * 32 + lane;          // position of the tile, latent feature of a pair
+    const int n0 = (warp >> 2) * NH;         // this warp's columns
+    const uint32_t lane_addr = (static_cast<uint32_t>(quad * 32) << 16) + n0;
+    float l_part[NH];
 #pragma unroll
-    for (int n = 0; n < N; ++n) l_part[n] = 0.f;
+    for (int n = 0; n < NH; ++n) l_part[n] = 0.f;
     bool ok = !dead;
-    // A wait that runs out only clears `ok`; the loop keeps its shape so that all 128 threads meet at the barriers.
+    // A wait that runs out only clears `ok`; the loop keeps its shape so that all threads meet at the barriers.
     for (int j = 0; j < n_tiles; ++j) {
       if (ok) ok = mbar_wait(&bar_s[j & 1], static_cast<uint32_t>(j >> 1) & 1, abort_flag, p.err);
       __syncwarp();
       tc_fence_after();
-      float s[N];
+      float s[NH];
 #pragma unroll
-      for (int c = 0; c < N; c += 16) tmem_ld_32x32b_x16(tmem_base + T_S + (j & 1) * N + c + lane_addr, reinterpret_cast<uint32_t*>(s) + c);
+      for (int c = 0; c < NH; c += CW) tmem_get<CW>(tmem_base + T_S + (j & 1) * N + c + lane_addr, reinterpret_cast<uint32_t*>(s) + c);
       tmem_wait_ld();
       const int tok = (tile0 + j) * TILE + r;
       const bool masked = (tile0 + j + 1) * TILE > first_lim || ncols < N;      // uniform: some column ends inside this tile
       if (masked) {
 #pragma unroll
-        for (int n = 0; n < N; ++n)
-          if (tok >= s_lim[n]) s[n] = -INFINITY;
+        for (int n = 0; n < NH; ++n)
+          if (tok >= s_lim[n0 + n]) s[n] = -INFINITY;
       }
       // distances to the reference maxima; the maxima themselves are reduced only when a score outgrows its reference
       float top = -1e30f;
 #pragma unroll
-      for (int n = 0; n < N; n += 4) {
-        const float4 m = *reinterpret_cast<const float4*>(s_m + n);
+      for (int n = 0; n < NH; n += 4) {
+        const float4 m = *reinterpret_cast<const float4*>(s_m + n0 + n);
         top = fmaxf(top, fmaxf(fmaxf(s[n] * p.scale_log2 - m.x, s[n + 1] * p.scale_log2 - m.y),
                                fmaxf(s[n + 2] * p.scale_log2 - m.z, s[n + 3] * p.scale_log2 - m.w)));
       }
-      const bool outgrown = named_bar_or(1, 128, top > 8.f);
+      const bool outgrown = named_bar_or(1, SOFTMAX, top > 8.f);
       if (j >= 2 && ok) ok = mbar_wait(&bar_o[j & 1], static_cast<uint32_t>((j - 2) >> 1) & 1, abort_flag, p.err);
       if (outgrown) {
         __syncwarp();
-        float mine[(N + 31) / 32];
+        float mine = 0.f;
 #pragma unroll
-        for (int n = 0; n < N; ++n) {
+        for (int n = 0; n < NH; ++n) {
           const float wm = redux_max(s[n] * p.scale_log2);
-          if (lane == (n & 31)) mine[n >> 5] = wm;
+          if (lane == n) mine = wm;
         }
-#pragma unroll
-        for (int k = 0; k < (N + 31) / 32; ++k)
-          if (k * 32 + lane < N) red[warp * N + k * 32 + lane] = mine[k];
-        named_bar_sync(1, 128);
-        if (r < N) {
-          const float tm = fmaxf(fmaxf(red[r], red[N + r]), fmaxf(red[2 * N + r], red[3 * N + r]));
-          const float m = s_m[r];
-          s_alpha[r] = tm > m + 8.f ? exp2f(m - tm) : 1.f;
-          if (tm > m + 8.f) s_m[r] = tm;
+        if (lane < NH) red[quad * N + n0 + lane] = mine;
+        named_bar_sync(1, SOFTMAX);
+        if (threadIdx.x < N) {
+          const int c = threadIdx.x;
+          const float tm = fmaxf(fmaxf(red[c], red[N + c]), fmaxf(red[2 * N + c], red[3 * N + c]));
+          const float m = s_m[c];
+          s_alpha[c] = tm > m + 8.f ? exp2f(m - tm) : 1.f;
+          if (tm > m + 8.f) s_m[c] = tm;
         }
-        named_bar_sync(1, 128);
+        named_bar_sync(1, SOFTMAX);
 #pragma unroll
-        for (int n = 0; n < N; ++n) l_part[n] *= s_alpha[n];
+        for (int n = 0; n < NH; ++n) l_part[n] *= s_alpha[n0 + n];
         if (j > 0) {       // O^T may be rescaled only when the product of tile j - 1 has landed
           if (ok) ok = mbar_wait(&bar_o[(j - 1) & 1], static_cast<uint32_t>((j - 1) >> 1) & 1, abort_flag, p.err);
           __syncwarp();
@@ -293,13 +308,13 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
 #pragma unroll 1
           for (int pr = 0; pr < p.NP; ++pr) {
 #pragma unroll
-            for (int c = 0; c < N; c += 16) {
-              uint32_t o[16];
-              tmem_ld_32x32b_x16(tmem_base + T_O + pr * N + c + lane_addr, o);
+            for (int c = 0; c < NH; c += CW) {
+              uint32_t o[CW];
+              tmem_get<CW>(tmem_base + T_O + pr * N + c + lane_addr, o);
               tmem_wait_ld();
 #pragma unroll
-              for (int i = 0; i < 16; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * s_alpha[c + i]);
-              tmem_st_32x32b_x16(tmem_base + T_O + pr * N + c + lane_addr, o);
+              for (int i = 0; i < CW; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * s_alpha[n0 + c + i]);
+              tmem_put<CW>(tmem_base + T_O + pr * N + c + lane_addr, o);
             }
           }
           tmem_wait_st();
@@ -307,10 +322,10 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
       }
       // P[n][position]: K-major, two 64-position halves
       const int half = r >> 6, col = r & 63;
-      uint8_t* prow = sp + (j & 1) * Layout<N>::kP + half * N * 128 + ((col & 7) << 1);
+      uint8_t* prow = sp + (j & 1) * Layout<N>::kP + half * N * 128 + n0 * 128 + ((col & 7) << 1);      // n0 is a multiple of 8
 #pragma unroll
-      for (int n = 0; n < N; n += 4) {
-        const float4 m = *reinterpret_cast<const float4*>(s_m + n);
+      for (int n = 0; n < NH; n += 4) {
+        const float4 m = *reinterpret_cast<const float4*>(s_m + n0 + n);
         const float mm[4] = {m.x, m.y, m.z, m.w};
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
@@ -328,36 +343,37 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
     __syncwarp();
     tc_fence_after();
 #pragma unroll
-    for (int n = 0; n < N; ++n) {
+    for (int n = 0; n < NH; ++n) {
       const float ws = warp_sum(l_part[n]);
-      if (lane == 0) red[warp * N + n] = ws;
+      if (lane == 0) red[quad * N + n0 + n] = ws;
     }
-    named_bar_sync(1, 128);
+    named_bar_sync(1, SOFTMAX);
 #pragma unroll
-    for (int n = 0; n < N; ++n) l_part[n] = red[n] + red[N + n] + red[2 * N + n] + red[3 * N + n];
+    for (int n = 0; n < NH; ++n) l_part[n] = red[n0 + n] + red[N + n0 + n] + red[2 * N + n0 + n] + red[3 * N + n0 + n];
     const bool have = n_tiles > 0;           // uniform
-    if (p.splits > 1 && r < ncols) {
-      float* ml = p.part_ml + (static_cast<size_t>(split) * p.columns + col0 + r) * 2;
-      ml[0] = s_m[r];
-      ml[1] = have && ok ? red[r] + red[N + r] + red[2 * N + r] + red[3 * N + r] : 0.f;
+    if (p.splits > 1 && static_cast<int>(threadIdx.x) < ncols) {
+      const int c = threadIdx.x;
+      float* ml = p.part_ml + (static_cast<size_t>(split) * p.columns + col0 + c) * 2;
+      ml[0] = s_m[c];
+      ml[1] = have && ok ? red[c] + red[N + c] + red[2 * N + c] + red[3 * N + c] : 0.f;
     }
     if (have) {
 #pragma unroll 1
       for (int pr = 0; pr < p.NP; ++pr) {
         const int d = pr * 128 + r;
 #pragma unroll
-        for (int c = 0; c < N; c += 16) {
-          uint32_t o[16];
-          tmem_ld_32x32b_x16(tmem_base + T_O + pr * N + c + lane_addr, o);
+        for (int c = 0; c < NH; c += CW) {
+          uint32_t o[CW];
+          tmem_get<CW>(tmem_base + T_O + pr * N + c + lane_addr, o);
           tmem_wait_ld();
           if (d < p.R) {
 #pragma unroll
-            for (int i = 0; i < 16; ++i) {
-              const int n = c + i;
+            for (int i = 0; i < CW; ++i) {
+              const int n = n0 + c + i;
               if (n < ncols) {
                 const float v = __uint_as_float(o[i]);
                 if (p.splits == 1)
-                  p.out[static_cast<size_t>(col0 + n) * p.R + d] = __float2bfloat16(ok && l_part[n] > 0.f ? v / l_part[n] * s_gate[n] : 0.f);
+                  p.out[static_cast<size_t>(col0 + n) * p.R + d] = __float2bfloat16(ok && l_part[c + i] > 0.f ? v / l_part[c + i] * s_gate[n] : 0.f);
                 else
                   p.part_o[(static_cast<size_t>(split) * p.columns + col0 + n) * p.R + d] = v;
               }
@@ -366,14 +382,14 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
         }
       }
     } else if (p.splits == 1) {
-      for (int i = r; i < ncols * p.R; i += 128) p.out[static_cast<size_t>(col0) * p.R + i] = __float2bfloat16(0.f);
+      for (int i = threadIdx.x; i < ncols * p.R; i += SOFTMAX) p.out[static_cast<size_t>(col0) * p.R + i] = __float2bfloat16(0.f);
     }
   }
 
   if (*abort_flag) __nanosleep(50000);
   tc_fence_before();
   __syncthreads();
-  if (warp == 5) {
+  if (warp == 9) {
     tc_fence_after();
     tmem_dealloc<kTmemCols>(tmem_base);
   }
