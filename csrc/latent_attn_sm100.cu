@@ -196,24 +196,31 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
   } else if (warp == 9) {
     // ================================================================ MMA issuer
     if (lane == 0 && !dead && n_tiles > 0) {
-      const uint32_t id_s = make_idesc_f16(TILE, N, true, false, false);
-      const uint32_t id_o = make_idesc_f16(TILE, N, true, true, false);
-      const uint32_t aq = smem_u32(sq), ap = smem_u32(sp), ring = smem_u32(smem);
-      // slot of (tile j, pair pr) is (j * NP + pr) % slots, its phase the parity of the quotient
+      constexpr uint32_t id_s = make_idesc_f16(TILE, N, true, false, false);
+      constexpr uint32_t id_o = make_idesc_f16(TILE, N, true, true, false);
+      // One thread issues everything, so it must spend few instructions per product: descriptors are formed once and
+      // advanced by adding to their address field (units of 16 bytes).
+      const uint64_t ring_k = make_smem_desc(smem_u32(smem), 16, 1024, kSwizzle128B);            // tile rows as K-major A
+      const uint64_t ring_mn = make_smem_desc(smem_u32(smem), SLOT / 2, 1024, kSwizzle128B);     // the same tile as C^T, MN-major A
+      const uint64_t q0 = make_smem_desc(smem_u32(sq), 16, 1024, kSwizzle128B), p0 = make_smem_desc(smem_u32(sp), 16, 1024, kSwizzle128B);
+      int ss = 0, so = 0;              // ring slots of the next S and O products
+      uint32_t phase = 0;
       auto issue_s = [&](int j) -> bool {
+        const uint32_t d = tmem_base + T_S + (j & 1) * N;
+        uint64_t db = q0;
         for (int pr = 0; pr < p.NP; ++pr) {
-          const int u = j * p.NP + pr, s = u % p.slots;
-          if (!mbar_wait(&full[s], static_cast<uint32_t>(u / p.slots) & 1, abort_flag, p.err)) return false;
+          if (!mbar_wait(&full[ss], phase, abort_flag, p.err)) return false;
           tc_fence_after();
-          const int nch = min(2, p.NC - 2 * pr);
-          for (int c = 0; c < nch; ++c) {
+          const uint64_t da = ring_k + static_cast<uint32_t>(ss) * (SLOT >> 4);
+          umma_f16(d, da, db, id_s, pr > 0 ? 1u : 0u);
 #pragma unroll
-            for (int kk = 0; kk < 4; ++kk) {
-              const uint64_t da = make_smem_desc(ring + s * SLOT + c * (SLOT / 2) + kk * 32, 16, 1024, kSwizzle128B);
-              const uint64_t db = make_smem_desc(aq + (2 * pr + c) * N * 128 + kk * 32, 16, 1024, kSwizzle128B);
-              umma_f16(tmem_base + T_S + (j & 1) * N, da, db, id_s, (pr > 0 || c > 0 || kk > 0) ? 1u : 0u);
-            }
+          for (int kk = 1; kk < 4; ++kk) umma_f16(d, da + kk * 2, db + kk * 2, id_s, 1u);
+          if (2 * pr + 1 < p.NC) {
+#pragma unroll
+            for (int kk = 0; kk < 4; ++kk) umma_f16(d, da + (SLOT >> 5) + kk * 2, db + (N * 128 >> 4) + kk * 2, id_s, 1u);
           }
+          db += 2 * (N * 128 >> 4);
+          if (++ss == p.slots) { ss = 0; phase ^= 1; }
         }
         umma_commit(&bar_s[j & 1]);
         return true;
@@ -228,17 +235,18 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
         if (p.ahead && j + 1 < n_tiles && !issue_s(j + 1)) break;
         if (!mbar_wait(&bar_p[j & 1], static_cast<uint32_t>(j >> 1) & 1, abort_flag, p.err)) break;
         tc_fence_after();
+        const uint64_t db = p0 + static_cast<uint32_t>(j & 1) * (Layout<N>::kP >> 4);
+        const uint32_t first = j > 0 ? 1u : 0u;
         for (int pr = 0; pr < p.NP; ++pr) {
-          const int s = (j * p.NP + pr) % p.slots;
+          // A: M = 128 latent features (two chunks SLOT / 2 apart), K = 16 positions (2048 bytes).  In the last slot of an odd
+          // chunk count the upper 64 rows of the product come from stale data and are never read
+          const uint64_t da = ring_mn + static_cast<uint32_t>(so) * (SLOT >> 4);
+          const uint32_t d = tmem_base + T_O + pr * N;
+          umma_f16(d, da, db, id_o, first);
 #pragma unroll
-          for (int kk = 0; kk < TILE / 16; ++kk) {
-            // A = C^T: M = 128 latent features (two chunks SLOT/2 apart), K = 16 positions (2048 bytes).  In the last slot
-            // of an odd chunk count the upper 64 rows of the product come from stale data and are never read
-            const uint64_t da = make_smem_desc(ring + s * SLOT + kk * 2048, SLOT / 2, 1024, kSwizzle128B);
-            const uint64_t db = make_smem_desc(ap + (j & 1) * Layout<N>::kP + (kk >> 2) * N * 128 + (kk & 3) * 32, 16, 1024, kSwizzle128B);
-            umma_f16(tmem_base + T_O + pr * N, da, db, id_o, (j > 0 || kk > 0) ? 1u : 0u);
-          }
-          umma_commit(&empty[s]);
+          for (int kk = 1; kk < TILE / 16; ++kk) umma_f16(d, da + kk * 128, db + (kk >> 2) * (N * 128 >> 4) + (kk & 3) * 2, id_o, 1u);
+          umma_commit(&empty[so]);
+          if (++so == p.slots) so = 0;
         }
         umma_commit(&bar_o[j & 1]);
         if (!p.ahead && j + 1 < n_tiles && !issue_s(j + 1)) break;

@@ -90,7 +90,8 @@ def main(argv=None) -> int:
         dev = a.device or ("cuda" if torch.cuda.is_available() else "cpu")
         cfg = engine_config(a.model_name, a.hf_checkpoint)
         dtype = {"bfloat16": torch.bfloat16, "float32": torch.float32}.get(a.dtype) or (torch.bfloat16 if dev.startswith("cuda") else torch.float32)
-        eng = RolloutEngine(cfg, device=dev, dtype=dtype, num_kv_blocks=a.kv_blocks, block_size=16, seed=a.seed,
+        page = 64 if cfg.is_composed else 16          # latent rows are gathered fastest in longer pages
+        eng = RolloutEngine(cfg, device=dev, dtype=dtype, num_kv_blocks=max(1, a.kv_blocks * 16 // page), block_size=page, seed=a.seed,
                             speculative=a.speculative_steps > 0, speculative_steps=max(1, a.speculative_steps),
                             state_slots=a.state_slots, max_model_len=a.max_model_len, eos_token_id=a.eos_token_id)
         if a.hf_checkpoint:

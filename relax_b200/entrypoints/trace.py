@@ -6,7 +6,7 @@ import json
 import os
 import sys
 
-PAGE = 16           # tokens per page of the engine's block manager
+PAGE = 64           # tokens per page of the engine's block manager
 MAX_LIVE = 4        # requests that may be live at once
 
 

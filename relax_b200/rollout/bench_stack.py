@@ -160,7 +160,9 @@ def model_rows(size: str, only=None, decode_batches=(1, 32, 128), prompt=2048):
         if only and name not in only:
             continue
         slow = name == "gdn hybrid"
-        eng = RolloutEngine(cfg, device="cuda", dtype=torch.bfloat16, num_kv_blocks=(max(decode_batches) + 8) * (prompt + 256) // 16, max_running=136,
+        page = 64 if cfg.is_composed else 16
+        eng = RolloutEngine(cfg, device="cuda", dtype=torch.bfloat16, num_kv_blocks=(max(decode_batches) + 8) * (prompt + 256) // page,
+                            block_size=page, max_running=136,
                             max_model_len=prompt + 256, memory_saver=False)
         eng.weights.flat.normal_(0, 0.02)
         g = torch.Generator().manual_seed(0)
@@ -176,7 +178,7 @@ def model_rows(size: str, only=None, decode_batches=(1, 32, 128), prompt=2048):
             return a.elapsed_time(b)
 
         for S, L in ((1, 8192 if not slow else 2048), (4, 2048), (32, 256)):
-            if L > eng.max_model_len and S * L > eng.bm.num_free * 16:
+            if L > eng.max_model_len and S * L > eng.bm.num_free * page:
                 continue
             ps = [prm(L) for _ in range(S)]
             go = lambda: eng.generate(ps, SamplingParams(max_new_tokens=1, ignore_eos=True))

@@ -224,7 +224,7 @@ def test_trace_replay_writes_the_wanted_logits(tmp_path):
              {"step": 1, "entries": [{"id": "b", "tokens": b[2:], "want": []}], "end": ["b"]},
              {"step": 2, "entries": [{"id": "c", "tokens": b, "want": [5]}, {"id": "a", "tokens": a[9:], "want": [10]}], "end": ["a", "c"]}]
     eng = trace.build_engine(str(model_dir), torch.float32, 128, device="cpu")
-    assert eng.bm.num_blocks == 8 and eng.sm.num_free == 4
+    assert eng.bm.num_blocks == 2 and eng.sm.num_free == 4
     done = []
     trace.replay(eng, io.StringIO("".join(json.dumps(s) + "\n" for s in steps)), str(tmp_path), done.append)
     assert done == [0, 1, 2] and not (tmp_path / "1.f32").exists()
