@@ -133,7 +133,13 @@ def attention_items(lens: Sequence[int], ctx: Sequence[int], heads: int, width: 
 
 def recurrent_spans(lens: Sequence[int], heads: int, ctas: int = 296, shortest: int = 128) -> Optional[tuple]:
     """Cut long segments into spans so that (spans x heads) fills the machine (``ctas`` at a time); spans are multiples of
-    the kernel's 16-token chunks.  ``(row ranges, first span of every segment)``, None when no segment is worth cutting."""
+    the kernel's 16-token chunks.  ``(row ranges, first span of every segment)``, None when no segment is worth cutting:
+    a CTA alone takes 1.25 times the time per chunk that a full machine needs for one chunk per SM, and spans add 0.57 for the
+    pass over their states (measured on a B200)."""
+    chunks = [-(-n // 16) for n in lens]
+    full = sum(chunks) * heads / 148
+    if max(1.25 * max(chunks), full) <= 1.57 * full:
+        return None
     size = max(shortest, pad_to(-(-sum(lens) * heads // ctas), 16))
     spans, first, row = [], [0], 0
     for n in lens:

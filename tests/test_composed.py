@@ -199,8 +199,8 @@ def test_attention_items_cover_every_column_once():
 def test_recurrent_spans_cover_every_row_in_whole_chunks():
     from relax_b200.rollout.composed import recurrent_spans
 
-    assert recurrent_spans([5, 1, 100], 2) is None
-    for lens, heads in (([8192], 32), ([1, 700, 3, 2049], 16), ([260], 1), ([4000, 4000, 1], 64)):
+    assert recurrent_spans([5, 1, 100], 2) is None and recurrent_spans([2048] * 4, 32) is None
+    for lens, heads in (([8192], 32), ([1, 700, 3, 2049], 16), ([260], 1), ([4000, 4000, 1], 8)):
         spans, first = recurrent_spans(lens, heads, shortest=64)
         row = 0
         for s, n in enumerate(lens):
