@@ -188,7 +188,7 @@ __global__ void __launch_bounds__(NA_WARPS * 32) norm_add_kernel(const NormAddPa
         stv<V>(h + c, x);
       }
     }
-    if (wpg > 1) __syncthreads();      // the next round rewrites the sums
+    if (wpg > 1) __syncthreads();      // the next pass rewrites the sums
   }
   for (int c = p.width + threadIdx.x; c < p.pitch; c += blockDim.x) st(h + c, 0.f);
 }

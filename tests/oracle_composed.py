@@ -102,7 +102,7 @@ CONFIGS = {
     # every padding rule at once: nothing is a multiple of anything
     "odd": {"width": 90, "vocab": 131, "norm": {"eps": 3e-5, "groups": 3},
             "layers": [att(3, 20, 12, 36, 0.31, 50), rec(5, 12, 7), rec(1, 33, 18, 70), att(2, 9, 30, 100, 0.4), rec(2, 8, 8, 24)]},
-    "round": {"width": 128, "vocab": 256, "norm": {"eps": 1e-4, "groups": 1},
+    "even": {"width": 128, "vocab": 256, "norm": {"eps": 1e-4, "groups": 1},
               "layers": [rec(2, 64, 64, 192), att(4, 32, 32, 64, 0.2, 192), att(16, 16, 48, 192, 0.25, 64), rec(4, 32, 32)]},
     # sizes that often coincide differ; one head; one group per eight features
     "single": {"width": 64, "vocab": 65, "norm": {"eps": 1e-6, "groups": 8}, "layers": [rec(1, 16, 40), att(1, 24, 8, 16, 0.7, 8)]},

@@ -84,7 +84,7 @@ def test_greedy_generation_through_the_scheduler(windowed):
 def test_group_members_share_the_prompt_and_partial_rollouts_resume():
     from relax_b200.rollout.engine import SamplingParams
 
-    cfg = O.CONFIGS["round"]
+    cfg = O.CONFIGS["even"]
     t = O.random_model(cfg, 5)
     p = O.tokens(cfg, 37, 3)
     want = D.greedy(cfg, t, p, 4)

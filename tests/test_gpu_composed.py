@@ -62,7 +62,7 @@ def _ok():
 
 
 @BOTH
-@pytest.mark.parametrize("width,groups", [(4096, 8), (4096, 1), (90, 3), (320, 5), (200, 25), (64, 64)])
+@pytest.mark.parametrize("width,groups", [(4096, 8), (4096, 1), (90, 3), (360, 5), (200, 25), (64, 64)])
 def test_norm_add(dtype, width, groups):
     from relax_b200 import ops
 
@@ -115,7 +115,7 @@ def _hgrn_plain(x, fb, lo, nw, H, dim, vdim, eps, S):
 
 
 @BOTH
-@pytest.mark.parametrize("H,dim,vdim", [(2, 128, 128), (3, 48, 32), (1, 16, 40), (2, 33, 18), (5, 12, 7), (1, 200, 72), (2, 64, 130)])
+@pytest.mark.parametrize("H,dim,vdim", [(2, 128, 128), (3, 40, 24), (1, 16, 40), (2, 33, 18), (5, 12, 7), (1, 200, 72), (2, 64, 130)])
 def test_hgrn2_segments_and_steps(dtype, H, dim, vdim):
     """Segments of unequal length (one token to several chunks) in one launch, then single tokens, from states in shuffled
     slots; a segment at position 0 ignores what its slot holds."""
@@ -323,7 +323,7 @@ def test_flash_with_unequal_widths_and_gate():
     from relax_b200 import ops
 
     bf = torch.bfloat16
-    for H, dk, dv in ((3, 24, 16), (2, 128, 128), (4, 64, 80)):
+    for H, dk, dv in ((3, 24, 16), (2, 128, 128), (4, 56, 72)):
         lens, ctx = [200, 300], [450, 300]
         q, k, v = _rand(1, 500, H, dk, dtype=bf), _rand(2, 750, H, dk, dtype=bf), _rand(3, 750, H, dv, dtype=bf)
         g = _rand(4, 500, H, dtype=bf)
@@ -362,7 +362,7 @@ def test_schedules_agree_with_the_plain_model(name, dtype):
 def test_long_prompts_in_portions_beside_other_requests(dtype):
     """Portions above and below the length from which keys and values are projected, contexts of several tiles, requests
     that join and leave, few pages and slots."""
-    cfg = O.CONFIGS["round"]
+    cfg = O.CONFIGS["even"]
     t = O.random_model(cfg, 2, sharp=2.0)
     seqs = [O.tokens(cfg, n, n) for n in (420, 30, 260, 3, 199)]
     want = [O.model(cfg, t, s) for s in seqs]
