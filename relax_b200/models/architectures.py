@@ -3,9 +3,9 @@ tensor names: ``name -> module`` with ``config_from_dict(d, name, dtype)`` and `
 Checkpoints without the key are read as Hugging Face layouts (:mod:`relax_b200.checkpoint.hf`)."""
 from __future__ import annotations
 
-from . import talizen
+from . import ketolorn, talizen
 
-ARCHITECTURES = {talizen.ARCHITECTURE: talizen}
+ARCHITECTURES = {m.ARCHITECTURE: m for m in (talizen, ketolorn)}
 
 
 def architecture_of(config_json: dict):

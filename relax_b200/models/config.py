@@ -29,27 +29,76 @@ class VisionConfig:
 
 
 @dataclass(frozen=True)
+class MoESpec:
+    """Routed feed-forward of a composed layer: ``experts`` ungated feed-forwards ``down(act(up h))`` of width ``ff``, of which
+    every token takes ``top`` by the sigmoid of its router logits.  The experts form ``groups`` equal groups of neighbours; only
+    those of the ``keep`` groups with the largest sums of their two best scores can be taken.  ``shared_ff``: width of one
+    more feed-forward of the same form that every token takes with weight one (0 = none)."""
+    experts: int
+    top: int
+    ff: int
+    groups: int = 1
+    keep: int = 1
+    shared_ff: int = 0
+    act: str = "relu2"
+    renormalize: bool = False    # weights divided by their sum over the taken experts
+    weight_scale: float = 1.0    # factor on the weights
+
+    def __post_init__(self):
+        if min(self.experts, self.top, self.ff, self.groups, self.keep) < 1 or self.shared_ff < 0 or self.act not in ACTIVATIONS:
+            raise ValueError(f"bad expert layer: {self}")
+        if self.experts % self.groups or self.keep > self.groups or self.top > self.experts // self.groups * self.keep:
+            raise ValueError(f"{self.top} of {self.experts} experts cannot be taken from {self.keep} of {self.groups} groups")
+
+
+@dataclass(frozen=True)
 class LayerSpec:
     """One layer of a composed stack (``ModelConfig.layer_specs``): its token mixer with the mixer's sizes and its
     feed-forward.  ``hgrn2``: gated linear recurrence with ``heads`` states of ``dim x vdim``.  ``latent_attention``:
-    softmax attention whose keys and values are projections of one cached latent row of ``kv_rank`` features per token."""
+    softmax attention whose keys and values are projections of one cached latent row of ``kv_rank`` features per token.
+    ``attention``: softmax attention over cached keys and values of ``kv_heads`` heads."""
     mixer: str
     heads: int
     dim: int                     # query (and key / forget-gate) features per head
     vdim: int                    # value features per head
     kv_rank: int = 0             # latent_attention only
-    scale: float = 1.0           # latent_attention only: factor on q . k
+    scale: float = 1.0           # attention mixers: factor on q . k
     ff: int = 0                  # width of the gated feed-forward; 0 = the layer has none
     act: str = "gelu_tanh"       # activation of the feed-forward's gate half
+    # attention only
+    kv_heads: int = 0            # query head h reads key / value head h // (heads / kv_heads)
+    rot_dims: int = 0            # leading features of queries and keys that are rotated, in neighbouring pairs
+    rot_base: float = 0.0        # pair i turns by position * rot_base ** (-2 i / rot_dims)
+    qk_norm: bool = False        # rotated queries and keys divided by their root mean square
+    sink: bool = False           # one learned logit per head in the softmax denominator, without key or value
+    kv_from: int = -1            # >= 0: reads the keys and values that this earlier layer has cached, and has none of its own
+    moe: Optional[MoESpec] = None  # routed feed-forward instead of the gated one
 
     def __post_init__(self):
         if self.mixer not in MIXERS:
             raise ValueError(f"unknown mixer {self.mixer!r}; known: {MIXERS}")
         if min(self.heads, self.dim, self.vdim) < 1 or (self.mixer == "latent_attention" and self.kv_rank < 1) or self.ff < 0:
             raise ValueError(f"bad layer sizes: {self}")
+        if self.act not in ACTIVATIONS[:2] or (self.moe is not None and self.ff):
+            raise ValueError(f"bad feed-forward: {self}")
+        if self.mixer == "attention":
+            if self.kv_heads < 1 or self.heads % self.kv_heads:
+                raise ValueError(f"{self.kv_heads} key / value heads do not divide {self.heads} heads")
+            if self.rot_dims % 2 or not 0 <= self.rot_dims <= self.dim or (self.rot_dims and self.rot_base <= 0):
+                raise ValueError(f"bad rotation: {self.rot_dims} of {self.dim} features, base {self.rot_base}")
+
+    @property
+    def has_ff(self) -> bool:
+        return self.ff > 0 or self.moe is not None
+
+    @property
+    def own_kv(self) -> bool:
+        """An attention layer that projects and caches keys and values."""
+        return self.mixer == "attention" and self.kv_from < 0
 
 
-MIXERS = ("hgrn2", "latent_attention")
+MIXERS = ("hgrn2", "latent_attention", "attention")
+ACTIVATIONS = ("silu", "gelu_tanh", "relu2")
 
 
 @dataclass
@@ -115,11 +164,12 @@ class ModelConfig:
     dsa_index_heads: int = 4
     dsa_index_dim: int = 16
     dsa_indexer_loss_coef: float = 1.0
-    # composed stacks (Talizen): every layer is spelled out - mixer, sizes, feed-forward.  The sublayers read the fp32
+    # composed stacks (Talizen, Ketolorn): every layer is spelled out - mixer, sizes, feed-forward.  The sublayers read the fp32
     # residual stream itself and their OUTPUT is normed (RMS over each of `norm_groups` equal parts) before it is added.
     # The fields above that describe one uniform layer (heads, head_dim, ffn, rotary, MoE, ...) do not apply then.
     layer_specs: Optional[tuple] = None
     norm_groups: int = 1
+    embed_norm: bool = False               # the embedded tokens are normed before the first layer
     dtype: str = "bf16"
 
     @property
@@ -153,11 +203,15 @@ class ModelConfig:
     def num_parameters(self) -> int:
         h, L = self.hidden_size, self.num_layers
         if self.is_composed:
-            n = 2 * self.vocab_size * h + h
+            n = (1 if self.tie_word_embeddings else 2) * self.vocab_size * h + h + (h if self.embed_norm else 0)
             for s in self.layer_specs:
-                n += h + 3 * s.ff * h + (h if s.ff else 0) + s.heads * s.vdim * h
+                n += h + 3 * s.ff * h + (h if s.has_ff else 0) + s.heads * s.vdim * h
+                if s.moe is not None:
+                    n += s.moe.experts * (h + 2 * s.moe.ff * h) + 2 * s.moe.shared_ff * h
                 if s.mixer == "hgrn2":
                     n += s.heads * (2 * s.dim + s.vdim) * h + 2 * s.heads * s.dim + s.vdim
+                elif s.mixer == "attention":
+                    n += s.heads * s.dim * h + (s.heads if s.sink else 0) + (s.kv_heads * (s.dim + s.vdim) * h if s.own_kv else 0)
                 else:
                     n += (s.heads * (s.dim + 1) + s.kv_rank) * h + s.kv_rank * (1 + s.heads * (s.dim + s.vdim))
             return n
@@ -192,6 +246,13 @@ def composed_config(name: str, layers, hidden_size: int, vocab_size: int, norm_g
         raise ValueError("a composed stack needs at least one layer")
     if norm_groups < 1 or hidden_size % norm_groups:
         raise ValueError(f"{norm_groups} norm groups do not divide the width {hidden_size}")
+    for i, s in enumerate(layers):
+        if s.mixer == "attention" and s.kv_from >= 0:
+            if s.kv_from >= i or not layers[s.kv_from].own_kv:
+                raise ValueError(f"layer {i} reads keys and values of layer {s.kv_from}, which has none before it")
+            what = ("kv_heads", "dim", "vdim", "rot_dims", "rot_base", "qk_norm")
+            if any(getattr(s, f) != getattr(layers[s.kv_from], f) for f in what):
+                raise ValueError(f"layer {i} and the layer {s.kv_from} whose keys and values it reads differ in {what}")
     return ModelConfig(name=name, num_layers=len(layers), hidden_size=hidden_size, vocab_size=vocab_size, rms_norm_eps=eps,
                        layer_specs=layers, norm_groups=norm_groups, qk_layernorm=False, **kw)
 
@@ -199,6 +260,14 @@ def composed_config(name: str, layers, hidden_size: int, vocab_size: int, norm_g
 def talizen_layers(n_layers: int, every: int, rec: LayerSpec, att: LayerSpec) -> tuple:
     """``every - 1`` recurrent layers, then one latent-attention layer, repeated."""
     return tuple(att if (i + 1) % every == 0 else rec for i in range(n_layers))
+
+
+def shared_kv_layers(n_layers: int, own: int, att: LayerSpec, dense_ff: int, moe: MoESpec, first_dense: int = 1) -> tuple:
+    """Attention layers of which the first ``own`` cache keys and values and the others read those of layer ``own - 1``; the
+    first ``first_dense`` have a gated feed-forward, the others routed experts."""
+    kv = lambda i: {} if i < own else {"kv_from": own - 1}
+    ff = lambda i: {"ff": dense_ff} if i < first_dense else {"moe": moe}
+    return tuple(replace(att, **kv(i), **ff(i)) for i in range(n_layers))
 
 
 # BASELINE config 0 ("tiny Qwen-style decoder")
@@ -308,6 +377,17 @@ _reg(composed_config("talizen-5b", talizen_layers(36, 4, LayerSpec("hgrn2", head
                                                   LayerSpec("latent_attention", heads=32, dim=128, vdim=128, kv_rank=512,
                                                             scale=128 ** -0.5, ff=12288)),
                      hidden_size=4096, vocab_size=151936, norm_groups=8))
+
+# Ketolorn: attention with sinks and normed rotated keys, upper layers on the keys and values of a lower one, grouped experts
+_reg(composed_config("tiny-ketolorn", shared_kv_layers(
+    4, 2, LayerSpec("attention", heads=6, dim=32, vdim=24, kv_heads=2, scale=0.3, rot_dims=16, rot_base=1e4, qk_norm=True, sink=True, act="silu"),
+    160, MoESpec(experts=8, top=2, ff=48, groups=4, keep=2, shared_ff=96)), hidden_size=160, vocab_size=320, eps=1e-6, embed_norm=True,
+    tie_word_embeddings=True, dtype="fp32"))
+_reg(composed_config("ketolorn-16b", shared_kv_layers(
+    24, 12, LayerSpec("attention", heads=32, dim=128, vdim=128, kv_heads=4, scale=128 ** -0.5, rot_dims=64, rot_base=5e5, qk_norm=True, sink=True,
+                      act="silu"),
+    8192, MoESpec(experts=128, top=8, ff=1024, groups=8, keep=4, shared_ff=2048)), hidden_size=2048, vocab_size=64000, eps=1e-6, embed_norm=True,
+    tie_word_embeddings=True))
 
 
 def get_config(name: str, **overrides) -> ModelConfig:

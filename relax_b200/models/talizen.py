@@ -7,12 +7,10 @@ embedding and head.  This module only translates names and layouts; the layers a
 """
 from __future__ import annotations
 
-import json
-import os
-
 import torch
 
 from .config import LayerSpec, ModelConfig, composed_config
+from .native import check_tensors, put, save_folder
 
 ARCHITECTURE = "Talizen"
 
@@ -68,16 +66,8 @@ def tensor_shapes(cfg: ModelConfig) -> dict:
 def load_tensors(cfg: ModelConfig, tensors: dict, weights) -> None:
     """Copy a checkpoint's tensors into a :class:`relax_b200.rollout.weights.RolloutWeights` buffer (zero-filled there, so
     every padded row and column stays zero).  Names and shapes must match exactly."""
-    want = tensor_shapes(cfg)
-    extra, missing = sorted(set(tensors) - set(want)), sorted(set(want) - set(tensors))
-    bad = [f"{k}: {tuple(tensors[k].shape)} instead of {want[k]}" for k in want if k in tensors and tuple(tensors[k].shape) != want[k]]
-    if extra or missing or bad:
-        raise ValueError(f"checkpoint does not fit the configuration: missing {missing[:8]}, unknown {extra[:8]}, shapes {bad[:8]}")
+    check_tensors(tensor_shapes(cfg), tensors)
     p, W = weights.p, cfg.hidden_size
-
-    def put(dst, src):          # dst: a view whose leading corner takes src
-        dst[tuple(slice(0, n) for n in src.shape)].copy_(src)
-
     put(p["embed"], tensors["embed"])
     put(p["lm_head"], tensors["head"])
     put(p["final_norm"], tensors["final.norm"])
@@ -110,9 +100,4 @@ def load_tensors(cfg: ModelConfig, tensors: dict, weights) -> None:
 
 
 def save(directory: str, cfg: ModelConfig, tensors: dict) -> None:
-    from safetensors.torch import save_file
-
-    os.makedirs(directory, exist_ok=True)
-    with open(os.path.join(directory, "config.json"), "w") as f:
-        json.dump(config_to_dict(cfg), f, indent=1)
-    save_file({k: v.contiguous() for k, v in tensors.items()}, os.path.join(directory, "model.safetensors"))
+    save_folder(directory, config_to_dict(cfg), tensors)

@@ -61,13 +61,55 @@ def linear_glu(x, w, act: str = "silu"):
     return _cuda().linear_glu(x, w, act) if _use_cuda(x) else ref.glu(ref.linear(x, w), act)
 
 
-def embed_rows(tokens, w):
-    return _cuda().embed_rows(tokens, w) if _use_cuda(w) else ref.embed_rows(tokens, w)
+def linear_act(x, w, act: str):
+    """``act(x @ w.T)`` without a gate (``act``: ``relu2``); joins the decode GEMM's reduction for decode shapes."""
+    if act != "relu2":
+        raise ValueError(f"no ungated activation {act!r}")
+    return _cuda().linear_relu2(x, w) if _use_cuda(x) else ref.relu2(ref.linear(x, w))
 
 
-def norm_add(res, y, w, width, groups, eps, next_w=None):
-    """Output norm in groups + add to the fp32 residual stream (in place) + the next sublayer's input, one kernel."""
-    return (_cuda() if _use_cuda(y) else ref).norm_add(res, y, w, width, groups, eps, next_w)
+def linear_fp32(x, w):
+    """``x @ w.T`` with fp32 results (router logits): products of 16-bit operands are exact in the fp32 accumulator."""
+    return _cuda().linear_fp32(x, w) if _use_cuda(x) else ref.linear(x.float(), w.float())
+
+
+def embed_rows(tokens, w, norm_w=None, width=0, groups=1, eps=0.0):
+    """Embedded tokens as the fp32 residual stream and its copy in the weights' type, normed in groups with ``norm_w``."""
+    return (_cuda() if _use_cuda(w) else ref).embed_rows(tokens, w, norm_w, width, groups, eps)
+
+
+def norm_add(res, y, w, width, groups, eps, next_w=None, experts=None):
+    """Output norm in groups + add to the fp32 residual stream (in place) + the next sublayer's input, one kernel.
+    ``experts``: ``(rows, plan)`` of :func:`moe_experts`, whose weighted sum joins ``y`` in the same pass."""
+    return (_cuda() if _use_cuda(res) else ref).norm_add(res, y, w, width, groups, eps, next_w, experts)
+
+
+def rope_table(positions, offset, inv_freq):
+    """cos / sin of every row's angles, computed once per forward for all layers that turn alike."""
+    return (_cuda() if _use_cuda(positions) else ref).rope_table(positions, offset, inv_freq)
+
+
+def attention_inputs(qkv, table, heads, kv_heads, dim, vdim, dp, rot_dims, eps, k_pool, v_pool, slots):
+    """Rotation and weightless norm of queries and keys, and the write of keys and values into their pages, one kernel."""
+    return (_cuda() if _use_cuda(qkv) else ref).attention_inputs(qkv, table, heads, kv_heads, dim, vdim, dp, rot_dims, eps, k_pool, v_pool, slots)
+
+
+def paged_attention(q, k_pool, v_pool, batch, block_size, scale, sink, out_width):
+    """Grouped-query attention over paged keys and values for every segment of a
+    :class:`relax_b200.rollout.composed.SegmentBatch`, with an optional sink logit per head."""
+    if _use_cuda(q):
+        return _cuda().paged_attention(q, k_pool, v_pool, batch, block_size, scale, sink, out_width)
+    return ref.paged_attention(q, k_pool, v_pool, batch.block_tables, block_size, batch.ctx, batch.cu, scale, sink, out_width)
+
+
+def moe_route(logits, spec):
+    """Expert choice of every row (:class:`relax_b200.models.config.MoESpec`)."""
+    return (_cuda() if _use_cuda(logits) else ref).moe_route(logits, spec)
+
+
+def moe_experts(h, plan, up, down, act):
+    """The chosen experts' outputs, unweighted, in an order :func:`norm_add` understands."""
+    return (_cuda() if _use_cuda(h) else ref).moe_experts(h, plan, up, down, act)
 
 
 def hgrn2(qfv, f_bias, lower, norm_w, state, state_slot, ctx_lens, cu, heads, dim, vdim, eps, spans=None):

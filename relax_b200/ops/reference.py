@@ -57,15 +57,23 @@ def group_rms(x, w, width: int, groups: int, eps: float):
     return y
 
 
-def embed_rows(tokens, w):
-    """``(fp32 residual stream, its copy in the weights' type)`` of embedded tokens."""
+def embed_rows(tokens, w, norm_w=None, width: int = 0, groups: int = 1, eps: float = 0.0):
+    """``(fp32 residual stream, its copy in the weights' type)`` of embedded tokens, group-normed when ``norm_w`` is given."""
     h = w[tokens]
-    return h.float(), h
+    if norm_w is None:
+        return h.float(), h
+    res = group_rms(h.float(), norm_w, width, groups, eps)
+    return res, res.to(w.dtype)
 
 
-def norm_add(res, y, w, width: int, groups: int, eps: float, next_w=None):
+def norm_add(res, y, w, width: int, groups: int, eps: float, next_w=None, experts=None):
     """``res += group_rms(y) * w`` in place (fp32); returns the next sublayer's input in ``w``'s type: the new stream
-    itself, or its own group norm with ``next_w`` when given."""
+    itself, or its own group norm with ``next_w`` when given.  ``experts = (rows, plan)``: the weighted rows of
+    :func:`moe_experts` join ``y`` (which may be None) first."""
+    if experts is not None:
+        rows, plan = experts
+        z = (rows.float() * plan.weight[..., None]).sum(1)
+        y = z if y is None else y.float() + z
     res += group_rms(y, w, width, groups, eps)
     return (res if next_w is None else group_rms(res, next_w, width, groups, eps)).to(w.dtype)
 
@@ -126,6 +134,97 @@ def latent_attention(q, pool, block_tables, block_size: int, ctx_lens, cu, scale
     if gate is not None:
         out = out * torch.sigmoid(gate.float())[..., None]
     return out.to(q.dtype)
+
+
+def rope_table(positions, offset: int, inv_freq):
+    """cos / sin ``[T, pairs, 2]`` (fp32) of the angles ``(position + offset) * inv_freq`` (fp64, so that late positions keep
+    their low bits)."""
+    a = (positions.double() + offset)[:, None] * inv_freq[None, :]
+    return torch.stack([torch.cos(a), torch.sin(a)], -1).float()
+
+
+def attention_inputs(qkv, table, heads: int, kv_heads: int, dim: int, vdim: int, dp: int, rot_dims: int, eps: float, k_pool, v_pool, slots):
+    """Raw projections ``[q heads | k heads | v heads]`` -> queries ``[T, heads, dp]`` and rows of the paged key / value pools
+    ``[rows, kv_heads, >= dim]``; ``k_pool`` None: the rows hold queries only.  The first ``rot_dims`` features of queries and
+    keys turn in neighbouring pairs; ``eps`` > 0: they are then divided by their root mean square."""
+    def head(x, norm_and_turn=True):
+        x = x.float()
+        if norm_and_turn:
+            if rot_dims:
+                c, s = table[:, None, :, 0], table[:, None, :, 1]
+                u, v = x[..., 0:rot_dims:2], x[..., 1:rot_dims:2]
+                x = torch.cat([torch.stack([u * c - v * s, v * c + u * s], -1).flatten(-2), x[..., rot_dims:]], -1)
+            if eps > 0:
+                x = x / torch.sqrt(x.pow(2).mean(-1, keepdim=True) + eps)
+        return x
+
+    T, qd, kd = qkv.shape[0], heads * dim, kv_heads * dim
+    q = torch.zeros(T, heads, dp, dtype=qkv.dtype, device=qkv.device)
+    q[..., :dim] = head(qkv[:, :qd].view(T, heads, dim)).to(qkv.dtype)
+    if k_pool is not None:
+        k_pool[slots, :, :dim] = head(qkv[:, qd:qd + kd].view(T, kv_heads, dim)).to(k_pool.dtype)
+        v_pool[slots, :, :vdim] = qkv[:, qd + kd:qd + kd + kv_heads * vdim].view(T, kv_heads, vdim).to(v_pool.dtype)
+    return q
+
+
+def paged_attention(q, k_pool, v_pool, block_tables, block_size: int, ctx_lens, cu, scale: float, sink, out_width: int):
+    """Softmax attention of ``q[T, H, dp]`` over paged keys and values ``[rows, kv_heads, ...]`` of their sequence; row ``i`` of
+    a segment of ``n`` rows sees the first ``ctx - n + i + 1`` positions.  ``sink[H]``: a logit per head that only joins the
+    denominator.  Returns ``[T, H * out_width]``."""
+    T, H, _ = q.shape
+    G, rep = k_pool.shape[1], H // k_pool.shape[1]
+    out = torch.zeros(T, H, out_width, dtype=torch.float32, device=q.device)
+    w = min(out_width, v_pool.shape[2])
+    bounds = list(range(T + 1)) if cu is None else cu.tolist()
+    for s, (a, b) in enumerate(zip(bounds, bounds[1:])):
+        L = int(ctx_lens[s])
+        pos = torch.arange(L, device=q.device)
+        rows = block_tables[s].long()[pos // block_size] * block_size + pos % block_size
+        k, v = k_pool[rows].float(), v_pool[rows].float()[..., :w]
+        sc = torch.einsum("tgrd,lgd->tgrl", q[a:b].float().view(b - a, G, rep, -1), k).reshape(b - a, H, L) * scale
+        lim = L - (b - a) + torch.arange(b - a, device=q.device)
+        sc = sc.masked_fill(pos[None, None, :] > lim[:, None, None], float("-inf"))
+        if sink is not None:
+            sc = torch.cat([sc, sink.float()[None, :, None].expand(b - a, H, 1)], -1)
+        p = torch.softmax(sc, -1)[..., :L].reshape(b - a, G, rep, L)
+        out[a:b, :, :w] = torch.einsum("tgrl,lgd->tgrd", p, v).reshape(b - a, H, w)
+    return out.reshape(T, H * out_width).to(q.dtype)
+
+
+class ExpertPlan:
+    """Which experts every row takes, ``index [T, top]``, and with which ``weight [T, top]``."""
+
+    def __init__(self, index, weight):
+        self.index, self.weight = index, weight
+
+
+def moe_route(logits, spec):
+    """Sigmoid scores; the ``spec.keep`` groups with the largest sums of their two best scores stay; of their experts the
+    ``spec.top`` best are taken."""
+    s = torch.sigmoid(logits[:, : spec.experts].float())
+    T, n = s.shape[0], spec.experts // spec.groups
+    best = s.view(T, spec.groups, n).topk(min(2, n), -1).values.sum(-1)
+    open_ = torch.zeros(T, spec.groups, dtype=torch.bool, device=s.device).scatter_(1, best.topk(spec.keep, -1).indices, True)
+    idx = s.masked_fill(~open_.repeat_interleave(n, 1), -1.0).topk(spec.top, -1).indices
+    w = s.gather(-1, idx)
+    if spec.renormalize:
+        w = w / w.sum(-1, keepdim=True)
+    return ExpertPlan(idx, w * spec.weight_scale)
+
+
+def relu2(x):
+    return torch.relu(x.float()).pow(2).to(x.dtype)
+
+
+def moe_experts(h, plan, up, down, act: str):
+    """Outputs ``down_e act(up_e h)`` of every row's experts, unweighted: ``[T, top, W]``."""
+    assert act == "relu2"
+    T, k = plan.index.shape
+    out = torch.zeros(T, k, down.shape[1], dtype=h.dtype, device=h.device)
+    for e in plan.index.unique().tolist():
+        t, j = (plan.index == e).nonzero(as_tuple=True)
+        out[t, j] = F.linear(relu2(F.linear(h[t], up[e])), down[e])
+    return out
 
 
 # --------------------------------------------------------------------------- rotary embedding

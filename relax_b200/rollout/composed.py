@@ -3,7 +3,9 @@
 A composed stack (``ModelConfig.layer_specs``) mixes layers whose memory of the past differs in kind:
 
 * recurrent layers keep one fp32 matrix per head and sequence, in a STATE SLOT of a fixed pool (:class:`StackCache.state`);
-* latent-attention layers keep one row per token in PAGES of the engine's block manager (:class:`StackCache.latent`).
+* latent-attention layers keep one row per token in PAGES of the engine's block manager (:class:`StackCache.latent`);
+* attention layers keep a key and a value row per token and key / value head in the same pages (:class:`StackCache.kv`), unless
+  they read the rows of an earlier layer.
 
 One forward (:meth:`ComposedForward.forward_segments`) runs a batch of SEGMENTS - the next ``n >= 1`` tokens of several
 sequences, prompt portions beside single decoded tokens - from what earlier forwards left in slots and pages.  The engine's
@@ -27,6 +29,12 @@ LONG_PORTION = 192     # portions of at least this many rows attend through proj
 
 def pad_to(n: int, m: int) -> int:
     return (n + m - 1) // m * m
+
+
+def head_pitch(n: int) -> int:
+    """Columns a head of ``n`` features takes in the key / value pools and in the queries: the widths of the tensor-core kernels,
+    beyond them 16-byte rows.  Padding stays zero."""
+    return 64 if n <= 64 else (128 if n <= 128 else pad_to(n, 8))
 
 
 class SlotManager:
@@ -54,20 +62,25 @@ class SlotManager:
 
 
 class StackCache:
-    """The two pools of a composed stack.  ``latent[layer]``: ``[blocks * block_size, padded rank]`` rows in the model's
-    type; ``state[layer]``: ``[slots, heads, dim, padded vdim]`` fp32.  All of it lives in ONE buffer."""
+    """The pools of a composed stack.  ``latent[layer]``: ``[blocks * block_size, padded rank]`` rows in the model's type;
+    ``kv[layer]``: keys and values ``[blocks * block_size, kv heads, padded width]``, one pair for the layer that computes them and
+    all that read them; ``state[layer]``: ``[slots, heads, dim, padded vdim]`` fp32.  All of it lives in ONE buffer."""
 
     def __init__(self, cfg: ModelConfig, num_blocks: int, block_size: int, num_slots: int, dtype, device, memory_saver: bool):
         self.block_size = block_size
         views, n = [], 0
         es = torch.empty(0, dtype=dtype).element_size()
+        rows = num_blocks * block_size
         for i, s in enumerate(cfg.layer_specs):
             if s.mixer == "hgrn2":
-                shape, dt, size = (num_slots, s.heads, s.dim, pad_to(s.vdim, 4)), torch.float32, 4
+                pools = [("state", (num_slots, s.heads, s.dim, pad_to(s.vdim, 4)), torch.float32, 4)]
+            elif s.mixer == "latent_attention":
+                pools = [("latent", (rows, pad_to(s.kv_rank, 64)), dtype, es)]
             else:
-                shape, dt, size = (num_blocks * block_size, pad_to(s.kv_rank, 64)), dtype, es
-            views.append((i, s.mixer, shape, dt, n))
-            n += pad_to(math.prod(shape) * size, 1024)
+                pools = [(k, (rows, s.kv_heads, head_pitch(d)), dtype, es) for k, d in (("k", s.dim), ("v", s.vdim))] if s.own_kv else []
+            for kind, shape, dt, size in pools:
+                views.append((i, kind, shape, dt, n))
+                n += pad_to(math.prod(shape) * size, 1024)
         self.nbytes = n
         self.buf = None
         if memory_saver:
@@ -76,17 +89,22 @@ class StackCache:
             self.buf = PausableBuffer(n, device)
             make = lambda shape, dt, off: self.buf.tensor(shape, dt, off)
         else:
-            flat = torch.zeros(n, dtype=torch.uint8, device=device)
+            flat = torch.zeros(max(n, 1), dtype=torch.uint8, device=device)
             make = lambda shape, dt, off: flat[off:off + math.prod(shape) * torch.empty(0, dtype=dt).element_size()].view(dt).view(shape)
-        self.latent, self.state = {}, {}
+        made = {"latent": {}, "state": {}, "k": {}, "v": {}}
         for i, kind, shape, dt, off in views:
-            (self.state if kind == "hgrn2" else self.latent)[i] = make(shape, dt, off)
+            made[kind][i] = make(shape, dt, off)
+        self.latent, self.state = made["latent"], made["state"]
+        self.kv = {i: (made["k"][i], made["v"][i]) for i in made["k"]}
+        for i, s in enumerate(cfg.layer_specs):
+            if s.kv_from >= 0:
+                self.kv[i] = self.kv[s.kv_from]
+        self.paged = list(made["latent"].values()) + list(made["k"].values()) + list(made["v"].values())
 
     def copy_sequence(self, src_blocks: Sequence[int], dst_blocks: Sequence[int], src_slot: int, dst_slot: int):
         """Pages ``src -> dst`` pairwise and the whole state slot."""
-        bs = self.block_size
-        for pool in self.latent.values():
-            v = pool.view(-1, bs, pool.shape[1])
+        for pool in self.paged:
+            v = pool.view(-1, self.block_size, *pool.shape[1:])
             for a, b in zip(src_blocks, dst_blocks):
                 v[b] = v[a]
         for st in self.state.values():
@@ -95,7 +113,8 @@ class StackCache:
 
 @dataclass
 class SegmentBatch:
-    """Device description of a batch of segments; the first ``long_segs`` of them (``long_rows`` rows) are long portions.
+    """Device description of a batch of segments; the first ``long_segs`` of them (``long_rows`` rows) are long portions, those
+    from ``multi_segs`` (row ``multi_rows``) on have a single row.
     ``cu`` is None when every segment is a single row.  ``short_*`` describe the segments behind the long ones, with row
     numbers counted from ``long_rows``; ``items[heads]`` are their column groups (see :func:`attention_items`)."""
     tokens: torch.Tensor
@@ -116,6 +135,13 @@ class SegmentBatch:
     max_ctx: int = 0                         # host upper bound of the short segments' contexts
     items: Optional[dict] = None
     spans: Optional[tuple] = None            # row ranges of recurrent spans and the first span of every segment
+    # attention layers
+    multi_segs: int = 0
+    multi_rows: int = 0
+    max_ctx_one: int = 0                     # host upper bound of the single-row segments' contexts
+    pos: Optional[torch.Tensor] = None       # [T] int32 position of every row; None: ctx - 1
+    seg_of: Optional[torch.Tensor] = None    # [T] int32 segment of every row
+    blocks: Optional[dict] = None            # tokens per query tile -> [n, 4] int32 (see :func:`query_blocks`)
 
 
 def attention_items(lens: Sequence[int], ctx: Sequence[int], heads: int, width: int = 64) -> list:
@@ -129,6 +155,24 @@ def attention_items(lens: Sequence[int], ctx: Sequence[int], heads: int, width: 
             out.append([s, c, min(step, (row0 + n) * heads - c), L - n - row0 + 1])
         row0 += n
     return out
+
+
+def query_blocks(lens: Sequence[int], ctx: Sequence[int], tokens: int) -> list:
+    """Cut segments into query tiles of at most ``tokens`` rows: ``[segment, first row, rows, position of the first row]``, those
+    that see the most positions first (the last tiles to start are then the short ones)."""
+    out, row = [], 0
+    for s, (n, L) in enumerate(zip(lens, ctx)):
+        out += [[s, row + a, min(tokens, n - a), L - n + a] for a in range(0, n, tokens)]
+        row += n
+    return sorted(out, key=lambda b: -(b[2] + b[3]))
+
+
+QUERY_ROWS = 128       # (token, head) rows of a query tile
+
+
+def tile_tokens(spec) -> int:
+    """Tokens of one query tile of an attention layer: the heads of a key / value head's group lie side by side."""
+    return max(1, QUERY_ROWS // (spec.heads // spec.kv_heads))
 
 
 def recurrent_spans(lens: Sequence[int], heads: int, ctas: int = 296, shortest: int = 128) -> Optional[tuple]:
@@ -162,6 +206,20 @@ class ComposedForward:
         s = self.cfg.layer_specs[i]
         return pad_to(s.dim, 8), pad_to(s.vdim, 8), pad_to(s.kv_rank, 64)
 
+    def attention_dims(self, i: int) -> tuple:
+        """Pitch of a head's queries and keys, of its values, and of its output in attention layer ``i``."""
+        s = self.cfg.layer_specs[i]
+        return head_pitch(s.dim), head_pitch(s.vdim), pad_to(s.vdim, 8)
+
+    def rope_frequencies(self, spec) -> torch.Tensor:
+        """``rot_base ** (-2 i / rot_dims)`` in fp64, kept on the device."""
+        made = self.__dict__.setdefault("_rope_freq", {})
+        key = (spec.rot_base, spec.rot_dims)
+        if key not in made:
+            i = torch.arange(spec.rot_dims // 2, dtype=torch.float64)
+            made[key] = (float(spec.rot_base) ** (-2.0 * i / spec.rot_dims)).to(self.device)
+        return made[key]
+
     @staticmethod
     def composed_param_shapes(cfg: ModelConfig) -> dict:
         """Every projection's output features are padded to 64 and its input features to the pitch of the rows it reads;
@@ -175,6 +233,11 @@ class ComposedForward:
                 shapes[p + "rec_qfv"] = (pad_to(2 * qd + vd, 64), Wp)
                 shapes[p + "rec_f_bias"], shapes[p + "rec_lower"], shapes[p + "rec_norm"] = (qd,), (qd,), (s.vdim,)
                 shapes[p + "rec_o"] = (Wp, pad_to(vd, 8))
+            elif s.mixer == "attention":
+                shapes[p + "attn_qkv"] = (pad_to(H * s.dim + (s.kv_heads * (s.dim + s.vdim) if s.own_kv else 0), 64), Wp)
+                if s.sink:
+                    shapes[p + "attn_sink"] = (H,)
+                shapes[p + "attn_o"] = (Wp, H * pad_to(s.vdim, 8))
             else:
                 dp, vp, Rp = pad_to(s.dim, 8), pad_to(s.vdim, 8), pad_to(s.kv_rank, 64)
                 shapes[p + "lat_qcg"] = (pad_to(H * dp + Rp + H, 64), Wp)
@@ -182,10 +245,22 @@ class ComposedForward:
                 shapes[p + "lat_uk"], shapes[p + "lat_uv"] = (H * dp, Rp), (H * vp, Rp)
                 shapes[p + "lat_o"] = (Wp, H * vp)
             shapes[p + "post_attn_norm"] = (Wp,)
+            if s.has_ff:
+                shapes[p + "post_mlp_norm"] = (Wp,)
             if s.ff:
                 Fp = pad_to(s.ff, 64)
-                shapes[p + "gate_up"], shapes[p + "down"], shapes[p + "post_mlp_norm"] = (2 * Fp, Wp), (Wp, Fp), (Wp,)
-        shapes["final_norm"], shapes["lm_head"] = (Wp,), (Vp, Wp)
+                shapes[p + "gate_up"], shapes[p + "down"] = (2 * Fp, Wp), (Wp, Fp)
+            if s.moe is not None:
+                E, Fp, Fs = s.moe.experts, pad_to(s.moe.ff, 64), pad_to(s.moe.shared_ff, 64)
+                shapes[p + "moe_router"] = (pad_to(E, 64), Wp)
+                shapes[p + "moe_up"], shapes[p + "moe_down"] = (E, Fp, Wp), (E, Wp, Fp)
+                if Fs:
+                    shapes[p + "shared_up"], shapes[p + "shared_down"] = (Fs, Wp), (Wp, Fs)
+        shapes["final_norm"] = (Wp,)
+        if cfg.embed_norm:
+            shapes["embed_norm"] = (Wp,)
+        if not cfg.tie_word_embeddings:
+            shapes["lm_head"] = (Vp, Wp)
         return shapes
 
     # ------------------------------------------------------------------ mixers
@@ -220,20 +295,53 @@ class ComposedForward:
             parts.append(ops.head_linear(o, uv.view(H, vp, Rp), True).reshape(T - n, H * vp))
         return ops.linear(parts[0] if len(parts) == 1 else torch.cat(parts), p[pre + "lat_o"])
 
+    def _attention(self, i, h, b: SegmentBatch, cache: StackCache, tables: dict):
+        s, p, pre = self.cfg.layer_specs[i], self.p, f"layers.{i}."
+        dp, _, vo = self.attention_dims(i)
+        k_pool, v_pool = cache.kv[i]
+        qkv = ops.linear(h, p[pre + "attn_qkv"])
+        q = ops.attention_inputs(qkv, self._rope_table(s, b, tables), s.heads, s.kv_heads, s.dim, s.vdim, dp, s.rot_dims,
+                                 self.cfg.rms_norm_eps if s.qk_norm else 0.0, *((k_pool, v_pool) if s.own_kv else (None, None)), b.slots)
+        o = ops.paged_attention(q, k_pool, v_pool, b, cache.block_size, s.scale, p.get(pre + "attn_sink"), vo)
+        return ops.linear(o, p[pre + "attn_o"])
+
+    def _rope_table(self, s, b: SegmentBatch, tables: dict):
+        if not s.rot_dims:
+            return None
+        key = (s.rot_base, s.rot_dims)
+        if key not in tables:
+            tables[key] = ops.rope_table(b.ctx if b.pos is None else b.pos, -1 if b.pos is None else 0, self.rope_frequencies(s))
+        return tables[key]
+
+    # ------------------------------------------------------------------ feed-forwards
+    def _feed_forward(self, i, h):
+        """``(output rows or None, (expert rows, plan) or None)`` of layer ``i``'s feed-forward."""
+        s, p, pre = self.cfg.layer_specs[i], self.p, f"layers.{i}."
+        if s.moe is None:
+            return ops.linear(ops.linear_glu(h, p[pre + "gate_up"], s.act), p[pre + "down"]), None
+        plan = ops.moe_route(ops.linear_fp32(h, p[pre + "moe_router"]), s.moe)
+        rows = ops.moe_experts(h, plan, p[pre + "moe_up"], p[pre + "moe_down"], s.moe.act)
+        shared = ops.linear(ops.linear_act(h, p[pre + "shared_up"], s.moe.act), p[pre + "shared_down"]) if s.moe.shared_ff else None
+        return shared, (rows, plan)
+
     # ------------------------------------------------------------------ trunk
     def _run_composed(self, b: SegmentBatch, cache: StackCache, taps: Optional[list] = None):
         """Final-norm output of every row.  ``taps``: a list that receives the fp32 residual stream after every layer."""
         cfg, p = self.cfg, self.p
         W, G, eps = cfg.hidden_size, cfg.norm_groups, cfg.rms_norm_eps
-        res, h = ops.embed_rows(b.tokens, p["embed"])
+        res, h = ops.embed_rows(b.tokens, p["embed"], p.get("embed_norm"), W, G, eps)
+        tables: dict = {}
         for i, s in enumerate(cfg.layer_specs):
             pre = f"layers.{i}."
             final = p["final_norm"] if i + 1 == cfg.num_layers else None
-            a = self._hgrn2(i, h, b, cache) if s.mixer == "hgrn2" else self._latent(i, h, b, cache)
-            h = ops.norm_add(res, a, p[pre + "post_attn_norm"], W, G, eps, None if s.ff else final)
-            if s.ff:
-                m = ops.linear(ops.linear_glu(h, p[pre + "gate_up"], s.act), p[pre + "down"])
-                h = ops.norm_add(res, m, p[pre + "post_mlp_norm"], W, G, eps, final)
+            if s.mixer == "attention":
+                a = self._attention(i, h, b, cache, tables)
+            else:
+                a = self._hgrn2(i, h, b, cache) if s.mixer == "hgrn2" else self._latent(i, h, b, cache)
+            h = ops.norm_add(res, a, p[pre + "post_attn_norm"], W, G, eps, None if s.has_ff else final)
+            if s.has_ff:
+                m, experts = self._feed_forward(i, h)
+                h = ops.norm_add(res, m, p[pre + "post_mlp_norm"], W, G, eps, final, experts)
             if taps is not None:
                 taps.append(res[:, :W].clone())
         return h
@@ -246,7 +354,7 @@ class ComposedForward:
     def forward_step(self, tokens, block_tables, context_lens, slots, state_slot, cache: StackCache, tp):
         """One decoded token per sequence (the captured step): everything is read from device arrays."""
         b = SegmentBatch(tokens, slots, context_lens, block_tables, state_slot,
-                         max_ctx=block_tables.shape[1] * cache.block_size)
+                         max_ctx=block_tables.shape[1] * cache.block_size, max_ctx_one=block_tables.shape[1] * cache.block_size)
         return self._logits(self._run_composed(b, cache), tp)
 
 
@@ -280,8 +388,10 @@ class ComposedScheduler:
                 r.blocks.append(self.bm.alloc())
                 r._reserve = max(0, getattr(r, "_reserve", 0) - 1)
         long_ok = self._long_portions
-        order = sorted(range(len(parts)), key=lambda j: not (long_ok and parts[j][1] >= LONG_PORTION))      # stable: long ones first
-        n_long = sum(1 for r, n in parts if long_ok and n >= LONG_PORTION)
+        kind = lambda n: 0 if long_ok and n >= LONG_PORTION else (1 if n > 1 else 2)      # long portions, short ones, single rows
+        order = sorted(range(len(parts)), key=lambda j: kind(parts[j][1]))                # (stable)
+        n_long = sum(1 for r, n in parts if kind(n) == 0)
+        n_multi = sum(1 for r, n in parts if n > 1)
         toks, slots, cu, ctx, sslot, bt, rows_of = [], [], [0], [], [], [], {}
         for j in order:
             r, n = parts[j]
@@ -298,12 +408,20 @@ class ComposedScheduler:
         single = all(n == 1 for _, n in parts)
         i32, i64 = torch.int32, torch.int64
         arrays = {"tokens": (toks, i64), "slots": (slots, i64), "ctx": (ctx, i32), "block_tables": (bt, i32), "state_slot": (sslot, i32)}
-        host = {"long_segs": n_long, "long_rows": cu[n_long], "max_ctx": max(ctx[n_long:], default=0)}
-        heads = []
+        host = {"long_segs": n_long, "long_rows": cu[n_long], "max_ctx": max(ctx[n_long:], default=0),
+                "multi_segs": n_multi, "multi_rows": cu[n_multi], "max_ctx_one": max(ctx[n_multi:], default=0)}
+        heads, tiles = [], []
         if not single:
             arrays["cu"] = (cu, i32)
             lens = [b - a for a, b in zip(cu, cu[1:])]
             sl, sc = lens[n_long:], ctx[n_long:]
+            attn = [self.cfg.layer_specs[i] for i in self.cfg.layers_with("attention")]
+            if attn:
+                arrays["pos"] = ([c - n + k for n, c in zip(lens, ctx) for k in range(n)], i32)
+                arrays["seg_of"] = ([s for s, n in enumerate(lens) for _ in range(n)], i32)
+                tiles = sorted({tile_tokens(s) for s in attn})
+                for t in tiles:
+                    arrays[f"blocks{t}"] = (query_blocks(lens[:n_multi], ctx, t), i32)
             if n_long:
                 arrays["long_cu"] = (cu[:n_long + 1], i32)
                 ck = [0]
@@ -316,7 +434,7 @@ class ComposedScheduler:
             cuts = recurrent_spans(lens, max(rec)) if rec and self.device.type == "cuda" else None
             if cuts is not None:
                 arrays["spans"], arrays["span_first"] = (cuts[0], i32), (cuts[1], i32)
-            if sl:
+            if sl and self.cfg.layers_with("latent_attention"):
                 arrays["short_cu"] = ([c - cu[n_long] for c in cu[n_long:]], i32)
                 arrays["row_seg"] = ([s for s, n in enumerate(sl) for _ in range(n)], i32)
                 arrays["row_pos"] = ([c - n + k for n, c in zip(sl, sc) for k in range(n)], i32)
@@ -329,7 +447,8 @@ class ComposedScheduler:
         want_t = dev.pop("rows", None)
         spans = (dev.pop("spans"), dev.pop("span_first")) if "spans" in dev else None
         items = {H: dev.pop(f"items{H}") for H in heads}
-        batch = SegmentBatch(**dev, **host, items=items or None, spans=spans)
+        blocks = {t: dev.pop(f"blocks{t}") for t in tiles}
+        batch = SegmentBatch(**dev, **host, items=items or None, spans=spans, blocks=blocks or None)
         logits = self.weights.forward_segments(batch, self.kv, want_t, self.tp, taps)
         for r, n in parts:
             r.fed += n

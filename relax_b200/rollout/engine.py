@@ -54,7 +54,7 @@ class Request:
     finish_reason: Optional[str] = None
     weight_versions: list = field(default_factory=list)
     cached_tokens: int = 0
-    # composed stacks: tokens whose latent rows / states are in the cache, and the slot of the recurrent states
+    # composed stacks: tokens whose rows / states are in the cache, and the slot of the recurrent states
     fed: int = 0
     state_slot: Optional[int] = None
     # with ``return_routed_experts``: per context position that was fed to the model, the expert ids every MoE layer
@@ -130,7 +130,7 @@ class RolloutEngine(SpeculativeMixin, ComposedScheduler):
         self.cfg = cfg
         self.composed = cfg.is_composed
         if self.composed and (speculative or return_routed_experts):
-            raise NotImplementedError("composed stacks serve without speculative decoding and have no routed experts")
+            raise NotImplementedError("composed stacks serve without speculative decoding and do not record routed experts")
         # speculative decoding drafted by the model's multi-token-prediction block (rollout/speculative.py)
         self.speculative = bool(speculative)
         self.speculative_steps = max(1, int(speculative_steps))      # proposals per verify pass (the block is chained)
@@ -175,8 +175,9 @@ class RolloutEngine(SpeculativeMixin, ComposedScheduler):
             self.sm = SlotManager(self.max_running + 1)
             self._scratch_slot = self.sm.alloc()      # padding rows of a graph bucket; never handed to a request
             # flash attention on projected keys / values: the tensor-core kernel takes bf16 heads of up to 128 features
-            self._long_portions = self.device.type == "cuda" and all(
-                ops.flash_serves_dims(self.dtype, *self.weights.latent_dims(i)[:2]) for i in cfg.layers_with("latent_attention"))
+            latent = cfg.layers_with("latent_attention")
+            self._long_portions = self.device.type == "cuda" and bool(latent) and all(
+                ops.flash_serves_dims(self.dtype, *self.weights.latent_dims(i)[:2]) for i in latent)
         self._alloc_kv()
         self.use_cuda_graph = use_cuda_graph and self.device.type == "cuda"
         self.max_model_len = max_model_len
