@@ -153,6 +153,31 @@ int rb_gate_heads(const void* o, const void* gate, int ld_gate, void* out, int r
 int rb_glu(const void* in, void* out, long long rows, int F, int ld_in, int act, int fp32, cudaStream_t st);
 int rb_simt_gemm(const void* A, const void* B, void* C, int M, int N, int K, int lda, int ldb, int ldc, int b_kn, int batch, long long sa,
                  long long sb, long long sc, int fp32, cudaStream_t st);
+int rb_norm_add_experts(float* res, const void* y, const void* ex, const int* expert, const int* place, const int* offset, const float* weight,
+                        int top, const void* w, const void* next_w, void* h, int rows, int ldy, int pitch, int width, int groups, float eps,
+                        int fp32, cudaStream_t st);
+int rb_embed_norm(const long long* tok, const void* table, const void* w, float* res, void* h, int rows, int vocab, int pitch, int width, int groups,
+                  float eps, int fp32, cudaStream_t st);
+int rb_rope_table(const int* pos, int offset, const double* freq, float* out, int rows, int half, cudaStream_t st);
+int rb_attention_inputs(const void* qkv, int ld, const float* table, void* q, void* k_pool, void* v_pool, const long long* slots, long long pool_rows,
+                        int T, int H, int G, int dim, int vdim, int dp, int vp, int rot, float eps, int fp32, cudaStream_t st);
+int rb_gqa_attn(const void* q, const void* k_pool, const void* v_pool, const int* block_tables, const int* row_seg, const int* row_pos, const int* ctx,
+                const void* sink, void* out, int rows, int H, int G, int dp, int vp, int vo, int max_blocks, int block_size, float scale, int fp32,
+                cudaStream_t st);
+int rb_paged_flash(const void* q, const void* kc, const void* vc, const int* block_tables, const int* ctx, const int* blocks, const void* sink,
+                   void* out, int rows, int n, int Hq, int Hkv, int dk, int dv, int out_d, long long pool_rows, int page, int max_blocks,
+                   float scale, int* err, cudaStream_t st);
+int rb_paged_decode_tc(const void* q, const void* kc, const void* vc, const int* block_tables, const int* ctx_lens, const void* sink, void* out,
+                       float* part_o, float* part_ml, int B, int Hq, int Hkv, int dk, int dv, int out_d, long long pool_rows, int page,
+                       int max_blocks, int max_ctx, float scale, int splits, int* err, cudaStream_t st);
+int rb_moe_route(const float* logits, int ld, int* expert, float* weight, int* place, int* row_token, int* count, int* offset, int* tiles,
+                 int* n_tiles, int T, int E, int groups, int keep, int top, int tile_rows, int cap, int renormalize, float weight_scale,
+                 cudaStream_t st);
+int rb_relu2(void* x, long long n, int fp32, cudaStream_t st);
+int rb_moe_simt(const void* A, const void* B, void* C, const int* tiles, const int* n_tiles, const int* row_token, int capacity, int cap, int N, int K,
+                int act, int fp32, cudaStream_t st);
+int rb_moe_gemm(const void* X, const void* W, void* out, const int* tiles, const int* n_tiles, const int* row_token, int x_rows, int capacity,
+                int cap, int E, int N, int K, int act, int bn, int* err, cudaStream_t st);
 #ifdef __cplusplus
 }
 #endif

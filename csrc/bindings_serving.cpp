@@ -105,7 +105,8 @@ void decode_advance(torch::Tensor tok_new, torch::Tensor lp_new, torch::Tensor t
 // Weight-streaming decode GEMM; returns false when the shape is outside its range (the caller uses the split-K path).
 bool decode_gemm(torch::Tensor x, torch::Tensor W, torch::Tensor y, int64_t glu, int64_t splits, torch::Tensor err) {
   const c10::cuda::CUDAGuard guard(x.device());
-  TORCH_CHECK(x.scalar_type() == at::kBFloat16 && W.scalar_type() == at::kBFloat16 && y.scalar_type() == at::kBFloat16, "bf16 only");
+  TORCH_CHECK(x.scalar_type() == at::kBFloat16 && W.scalar_type() == at::kBFloat16, "bf16 only");
+  TORCH_CHECK(y.scalar_type() == (glu == 4 ? at::kFloat : at::kBFloat16), "decode_gemm: output type");
   TORCH_CHECK(x.dim() == 2 && W.dim() == 2 && x.stride(1) == 1 && W.stride(1) == 1 && y.is_contiguous(), "row-major operands");
   const int rc = rb_decode_gemm(x.data_ptr(), W.data_ptr(), y.data_ptr(), (int)x.size(0), (int)W.size(0), (int)x.size(1),
                                 (int)x.stride(0), (int)W.stride(0), (int)glu, (int)splits, err.data_ptr<int>(), cur_stream());
@@ -286,6 +287,163 @@ void simt_gemm(torch::Tensor A, torch::Tensor B, torch::Tensor C, bool b_kn) {
                      b_kn, (int)A.size(0), A.stride(0), B.stride(0), C.stride(0), is_fp32(A), cur_stream()),
         "rb_simt_gemm");
 }
+// ---- attention over cached keys and values, routed experts
+inline bool is_i32(const torch::Tensor& t) { return t.scalar_type() == at::kInt && t.is_contiguous(); }
+void embed_norm(torch::Tensor tok, torch::Tensor table, torch::Tensor w, torch::Tensor res, torch::Tensor h, int64_t width, int64_t groups, double eps) {
+  const c10::cuda::CUDAGuard guard(table.device());
+  check_same(table, h, "embed_norm");
+  check_same(table, w, "embed_norm");
+  TORCH_CHECK(tok.scalar_type() == at::kLong && tok.is_contiguous() && table.is_contiguous() && res.is_contiguous() && h.is_contiguous());
+  TORCH_CHECK(res.scalar_type() == at::kFloat && res.sizes() == h.sizes() && h.size(0) == tok.numel() && h.size(1) == table.size(1) && w.numel() == table.size(1));
+  check(rb_embed_norm((const long long*)tok.data_ptr<int64_t>(), table.data_ptr(), w.data_ptr(), res.data_ptr<float>(), h.data_ptr(), (int)tok.numel(),
+                      (int)table.size(0), (int)table.size(1), (int)width, (int)groups, (float)eps, is_fp32(table), cur_stream()),
+        "rb_embed_norm");
+}
+void norm_add_experts(torch::Tensor res, c10::optional<torch::Tensor> y, torch::Tensor ex, torch::Tensor expert, torch::Tensor place, torch::Tensor offset,
+                      torch::Tensor weight, torch::Tensor w, c10::optional<torch::Tensor> next_w, torch::Tensor h, int64_t width, int64_t groups, double eps) {
+  const c10::cuda::CUDAGuard guard(res.device());
+  check_same(ex, w, "norm_add_experts");
+  check_same(ex, h, "norm_add_experts");
+  TORCH_CHECK(res.scalar_type() == at::kFloat && res.is_contiguous() && h.is_contiguous() && res.sizes() == h.sizes() && w.numel() == res.size(1));
+  TORCH_CHECK(ex.dim() == 2 && ex.is_contiguous() && ex.size(1) == res.size(1) && ex.size(0) == expert.numel());
+  TORCH_CHECK(!y.has_value() || (y->scalar_type() == ex.scalar_type() && y->is_contiguous() && y->sizes() == res.sizes()));
+  TORCH_CHECK(is_i32(expert) && is_i32(place) && is_i32(offset) && weight.scalar_type() == at::kFloat && weight.is_contiguous());
+  TORCH_CHECK(expert.dim() == 2 && expert.size(0) == res.size(0) && place.sizes() == expert.sizes() && weight.sizes() == expert.sizes());
+  TORCH_CHECK(!next_w.has_value() || (next_w->numel() == w.numel() && next_w->scalar_type() == w.scalar_type()));
+  check(rb_norm_add_experts(res.data_ptr<float>(), optptr(y), ex.data_ptr(), expert.data_ptr<int>(), place.data_ptr<int>(), offset.data_ptr<int>(),
+                            weight.data_ptr<float>(), (int)expert.size(1), w.data_ptr(), optptr(next_w), h.data_ptr(), (int)res.size(0),
+                            (int)ex.size(1), (int)res.size(1), (int)width, (int)groups, (float)eps, is_fp32(ex), cur_stream()),
+        "rb_norm_add_experts");
+}
+void rope_table(torch::Tensor pos, int64_t offset, torch::Tensor freq, torch::Tensor out) {
+  const c10::cuda::CUDAGuard guard(pos.device());
+  TORCH_CHECK(is_i32(pos) && freq.scalar_type() == at::kDouble && freq.is_contiguous() && out.scalar_type() == at::kFloat && out.is_contiguous());
+  TORCH_CHECK(out.numel() == pos.numel() * freq.numel() * 2 && freq.device() == pos.device());
+  check(rb_rope_table(pos.data_ptr<int>(), (int)offset, freq.data_ptr<double>(), out.data_ptr<float>(), (int)pos.numel(), (int)freq.numel(), cur_stream()),
+        "rb_rope_table");
+}
+void attention_inputs(torch::Tensor qkv, c10::optional<torch::Tensor> table, torch::Tensor q, c10::optional<torch::Tensor> k_pool,
+                      c10::optional<torch::Tensor> v_pool, torch::Tensor slots, int64_t kv_heads, int64_t dim, int64_t vdim, int64_t rot, double eps) {
+  const c10::cuda::CUDAGuard guard(qkv.device());
+  check_same(qkv, q, "attention_inputs");
+  const int64_t T = qkv.size(0);
+  TORCH_CHECK(qkv.dim() == 2 && qkv.stride(1) == 1 && q.dim() == 3 && q.is_contiguous() && q.size(0) == T && k_pool.has_value() == v_pool.has_value());
+  TORCH_CHECK(qkv.size(1) >= q.size(1) * dim + (k_pool.has_value() ? kv_heads * (dim + vdim) : 0), "attention_inputs: columns");
+  TORCH_CHECK(rot == 0 || (table.has_value() && table->scalar_type() == at::kFloat && table->is_contiguous() && table->numel() == T * rot));
+  TORCH_CHECK(slots.scalar_type() == at::kLong && slots.is_contiguous() && slots.numel() == T);
+  if (k_pool.has_value()) {
+    check_same(qkv, *k_pool, "attention_inputs");
+    check_same(qkv, *v_pool, "attention_inputs");
+    TORCH_CHECK(k_pool->dim() == 3 && v_pool->dim() == 3 && k_pool->is_contiguous() && v_pool->is_contiguous() && k_pool->size(0) == v_pool->size(0));
+    TORCH_CHECK(k_pool->size(1) == kv_heads && v_pool->size(1) == kv_heads && k_pool->size(2) == q.size(2), "attention_inputs: pools");
+  }
+  check(rb_attention_inputs(qkv.data_ptr(), (int)qkv.stride(0), rot ? table->data_ptr<float>() : nullptr, q.data_ptr(),
+                            k_pool.has_value() ? k_pool->data_ptr() : nullptr, v_pool.has_value() ? v_pool->data_ptr() : nullptr,
+                            (const long long*)slots.data_ptr<int64_t>(), k_pool.has_value() ? k_pool->size(0) : 0, (int)T, (int)q.size(1), (int)kv_heads,
+                            (int)dim, (int)vdim, (int)q.size(2), v_pool.has_value() ? (int)v_pool->size(2) : 0, (int)rot, (float)eps, is_fp32(qkv),
+                            cur_stream()),
+        "rb_attention_inputs");
+}
+inline void check_pools(const torch::Tensor& q, const torch::Tensor& k, const torch::Tensor& v, const torch::Tensor& bt, const torch::Tensor& ctx,
+                        const c10::optional<torch::Tensor>& sink, const torch::Tensor& out) {
+  check_same(q, k, "paged attention");
+  check_same(q, v, "paged attention");
+  check_same(q, out, "paged attention");
+  TORCH_CHECK(q.dim() == 3 && k.dim() == 3 && v.dim() == 3 && q.is_contiguous() && k.is_contiguous() && v.is_contiguous() && out.is_contiguous());
+  TORCH_CHECK(k.size(2) == q.size(2) && v.size(0) == k.size(0) && v.size(1) == k.size(1) && q.size(1) % k.size(1) == 0, "paged attention: shapes");
+  TORCH_CHECK(out.dim() == 2 && out.size(0) == q.size(0) && out.size(1) % q.size(1) == 0 && out.size(1) / q.size(1) <= v.size(2), "paged attention: output");
+  TORCH_CHECK(is_i32(bt) && bt.dim() == 2 && is_i32(ctx) && ctx.numel() == bt.size(0), "paged attention: block tables");
+  TORCH_CHECK(!sink.has_value() || (sink->scalar_type() == q.scalar_type() && sink->is_contiguous() && sink->numel() == q.size(1)), "paged attention: sink");
+}
+void gqa_attn(torch::Tensor q, torch::Tensor k, torch::Tensor v, torch::Tensor bt, c10::optional<torch::Tensor> row_seg, c10::optional<torch::Tensor> row_pos,
+              torch::Tensor ctx, c10::optional<torch::Tensor> sink, torch::Tensor out, int64_t block_size, double scale) {
+  const c10::cuda::CUDAGuard guard(q.device());
+  check_pools(q, k, v, bt, ctx, sink, out);
+  const int64_t T = q.size(0), H = q.size(1);
+  TORCH_CHECK(row_seg.has_value() == row_pos.has_value());
+  TORCH_CHECK(row_seg.has_value() ? (is_i32(*row_seg) && is_i32(*row_pos) && row_seg->numel() == T && row_pos->numel() == T) : ctx.numel() == T,
+              "gqa_attn: row description");
+  check(rb_gqa_attn(q.data_ptr(), k.data_ptr(), v.data_ptr(), bt.data_ptr<int>(), optint(row_seg), optint(row_pos), ctx.data_ptr<int>(), optptr(sink),
+                    out.data_ptr(), (int)T, (int)H, (int)k.size(1), (int)q.size(2), (int)v.size(2), (int)(out.size(1) / H), (int)bt.size(1),
+                    (int)block_size, (float)scale, is_fp32(q), cur_stream()),
+        "rb_gqa_attn");
+}
+// Prompt portions; returns false for shapes the tensor-core kernel does not take.
+bool paged_flash(torch::Tensor q, torch::Tensor k, torch::Tensor v, torch::Tensor bt, torch::Tensor ctx, c10::optional<torch::Tensor> blocks,
+                 c10::optional<torch::Tensor> sink, torch::Tensor out, int64_t block_size, double scale, torch::Tensor err) {
+  const c10::cuda::CUDAGuard guard(q.device());
+  if (q.scalar_type() != at::kBFloat16) return false;
+  check_pools(q, k, v, bt, ctx, sink, out);
+  const int64_t T = q.size(0), H = q.size(1);
+  TORCH_CHECK(blocks.has_value() ? (is_i32(*blocks) && blocks->dim() == 2 && blocks->size(1) == 4) : ctx.numel() == T, "paged_flash: query tiles");
+  const int rc = rb_paged_flash(q.data_ptr(), k.data_ptr(), v.data_ptr(), bt.data_ptr<int>(), ctx.data_ptr<int>(), optint(blocks), optptr(sink), out.data_ptr(),
+                                (int)T, (int)(blocks.has_value() ? blocks->size(0) : T), (int)H, (int)k.size(1), (int)q.size(2), (int)v.size(2),
+                                (int)(out.size(1) / H), k.size(0), (int)block_size, (int)bt.size(1), (float)scale, err.data_ptr<int>(), cur_stream());
+  if (rc == -20) return false;
+  check(rc, "rb_paged_flash");
+  return true;
+}
+// One row per sequence; returns false for shapes the tensor-core kernel does not take.
+bool paged_decode(torch::Tensor q, torch::Tensor k, torch::Tensor v, torch::Tensor bt, torch::Tensor ctx, c10::optional<torch::Tensor> sink, torch::Tensor out,
+                  c10::optional<torch::Tensor> part_o, c10::optional<torch::Tensor> part_ml, int64_t block_size, int64_t max_ctx, int64_t splits,
+                  double scale, torch::Tensor err) {
+  const c10::cuda::CUDAGuard guard(q.device());
+  if (q.scalar_type() != at::kBFloat16) return false;
+  check_pools(q, k, v, bt, ctx, sink, out);
+  const int64_t B = q.size(0), H = q.size(1);
+  TORCH_CHECK(ctx.numel() == B, "paged_decode: one row per sequence");
+  TORCH_CHECK(splits == 1 || (part_o.has_value() && part_o->scalar_type() == at::kFloat && part_o->numel() >= splits * B * H * 128 && part_ml.has_value() &&
+                              part_ml->scalar_type() == at::kFloat && part_ml->numel() >= splits * B * H * 2), "paged_decode: scratch");
+  const int rc = rb_paged_decode_tc(q.data_ptr(), k.data_ptr(), v.data_ptr(), bt.data_ptr<int>(), ctx.data_ptr<int>(), optptr(sink), out.data_ptr(),
+                                    part_o.has_value() ? part_o->data_ptr<float>() : nullptr, part_ml.has_value() ? part_ml->data_ptr<float>() : nullptr,
+                                    (int)B, (int)H, (int)k.size(1), (int)q.size(2), (int)v.size(2), (int)(out.size(1) / H), k.size(0), (int)block_size,
+                                    (int)bt.size(1), (int)max_ctx, (float)scale, (int)splits, err.data_ptr<int>(), cur_stream());
+  if (rc == -20) return false;
+  check(rc, "rb_paged_decode_tc");
+  return true;
+}
+void moe_route(torch::Tensor logits, torch::Tensor expert, torch::Tensor weight, torch::Tensor place, torch::Tensor row_token, torch::Tensor count,
+               torch::Tensor offset, torch::Tensor tiles, torch::Tensor n_tiles, int64_t experts, int64_t groups, int64_t keep, int64_t tile_rows,
+               bool renormalize, double weight_scale) {
+  const c10::cuda::CUDAGuard guard(logits.device());
+  const int64_t T = logits.size(0), top = expert.size(1);
+  TORCH_CHECK(logits.dim() == 2 && logits.scalar_type() == at::kFloat && logits.stride(1) == 1 && logits.size(1) >= experts, "moe_route: logits");
+  TORCH_CHECK(is_i32(expert) && is_i32(place) && expert.size(0) == T && place.sizes() == expert.sizes() && weight.scalar_type() == at::kFloat &&
+              weight.is_contiguous() && weight.sizes() == expert.sizes());
+  TORCH_CHECK(is_i32(row_token) && row_token.numel() >= experts * T && is_i32(count) && count.numel() >= experts + 1 && is_i32(offset) &&
+              offset.numel() >= experts + 1 && is_i32(n_tiles) && is_i32(tiles) && tiles.dim() == 2 && tiles.size(1) == 4);
+  TORCH_CHECK(tiles.size(0) >= std::min(T * top, experts) + T * top / tile_rows, "moe_route: tile list");
+  check(rb_moe_route(logits.data_ptr<float>(), (int)logits.stride(0), expert.data_ptr<int>(), weight.data_ptr<float>(), place.data_ptr<int>(),
+                     row_token.data_ptr<int>(), count.data_ptr<int>(), offset.data_ptr<int>(), tiles.data_ptr<int>(), n_tiles.data_ptr<int>(), (int)T,
+                     (int)experts, (int)groups, (int)keep, (int)top, (int)tile_rows, (int)tiles.size(0), renormalize, (float)weight_scale, cur_stream()),
+        "rb_moe_route");
+}
+// out[sorted row] = act(x[its token, or the sorted row] * W[expert]^T); act: 0 none, 1 squared relu
+void moe_gemm(torch::Tensor x, torch::Tensor W, torch::Tensor out, torch::Tensor tiles, torch::Tensor n_tiles, c10::optional<torch::Tensor> row_token,
+              int64_t act, int64_t bn, torch::Tensor err) {
+  const c10::cuda::CUDAGuard guard(x.device());
+  check_same(x, W, "moe_gemm");
+  check_same(x, out, "moe_gemm");
+  const int64_t E = W.size(0), N = W.size(1), K = W.size(2);
+  TORCH_CHECK(x.dim() == 2 && W.dim() == 3 && out.dim() == 2 && x.is_contiguous() && W.is_contiguous() && out.is_contiguous() && x.size(1) == K && out.size(1) == N);
+  TORCH_CHECK(is_i32(tiles) && is_i32(n_tiles) && (!row_token.has_value() || is_i32(*row_token)));
+  TORCH_CHECK(row_token.has_value() ? row_token->numel() >= E * x.size(0) : x.size(0) == out.size(0), "moe_gemm: rows");
+  const int cap = (int)tiles.size(0);
+  if (is_fp32(x)) {
+    check(rb_moe_simt(x.data_ptr(), W.data_ptr(), out.data_ptr(), tiles.data_ptr<int>(), n_tiles.data_ptr<int>(), optint(row_token), (int)x.size(0), cap,
+                      (int)N, (int)K, (int)act, 1, cur_stream()),
+          "rb_moe_simt");
+    return;
+  }
+  check(rb_moe_gemm(x.data_ptr(), W.data_ptr(), out.data_ptr(), tiles.data_ptr<int>(), n_tiles.data_ptr<int>(), optint(row_token), (int)x.size(0),
+                    (int)x.size(0), cap, (int)E, (int)N, (int)K, (int)act, (int)bn, err.data_ptr<int>(), cur_stream()),
+        "rb_moe_gemm");
+}
+void relu2(torch::Tensor x) {
+  const c10::cuda::CUDAGuard guard(x.device());
+  TORCH_CHECK(x.is_contiguous());
+  check(rb_relu2(x.data_ptr(), x.numel(), is_fp32(x), cur_stream()), "rb_relu2");
+}
 }  // namespace
 
 void register_serving(pybind11::module_& m) {
@@ -309,4 +467,14 @@ void register_serving(pybind11::module_& m) {
   m.def("gate_heads", &gate_heads);
   m.def("glu", &glu);
   m.def("simt_gemm", &simt_gemm);
+  m.def("embed_norm", &embed_norm);
+  m.def("norm_add_experts", &norm_add_experts);
+  m.def("rope_table", &rope_table);
+  m.def("attention_inputs", &attention_inputs);
+  m.def("gqa_attn", &gqa_attn);
+  m.def("paged_flash", &paged_flash);
+  m.def("paged_decode", &paged_decode);
+  m.def("moe_route", &moe_route);
+  m.def("moe_gemm", &moe_gemm);
+  m.def("relu2", &relu2);
 }

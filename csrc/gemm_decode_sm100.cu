@@ -26,6 +26,7 @@ struct Params {
   int Mt, N, K;             // tokens, output features of W (rows), reduction length
   int S;                    // cluster size = k splits
   int glu;                  // W rows are [gate (N/2); up (N/2)], output is [Mt, N/2]: 1 silu(g) u, 2 gelu_tanh(g) u
+  int post;                 // without a gated unit: 0 bf16, 1 squared relu then bf16, 2 fp32
   void* out;
   int* err;
 };
@@ -258,7 +259,13 @@ decode_gemm_kernel(const __grid_constant__ CUtensorMap tma_w, const __grid_const
           if (!p.glu) {
             const int f = tile * BM + u_lo + 4 * g;
             __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(p.out) + static_cast<size_t>(tok) * p.N + f;
-            if (f + 3 < p.N) {
+            if (p.post == 1) {
+              acc.x = fmaxf(acc.x, 0.f); acc.y = fmaxf(acc.y, 0.f); acc.z = fmaxf(acc.z, 0.f); acc.w = fmaxf(acc.w, 0.f);
+              acc.x *= acc.x; acc.y *= acc.y; acc.z *= acc.z; acc.w *= acc.w;
+            }
+            if (p.post == 2) {       // N is a multiple of 4: a group of four is inside or outside
+              if (f < p.N) *reinterpret_cast<float4*>(reinterpret_cast<float*>(p.out) + static_cast<size_t>(tok) * p.N + f) = acc;
+            } else if (f + 3 < p.N) {
               store_bf16x4(o, acc);
             } else {
               const float v[4] = {acc.x, acc.y, acc.z, acc.w};
@@ -349,7 +356,7 @@ extern "C" int rb_decode_gemm_splits(int tiles, int k_iters) {
 }
 
 // y = x W^T (glu = 0, y [Mt, N]) or y = act(x Wg^T) * (x Wu^T) with W = [Wg; Wu] (glu = 1: silu, 2: tanh form of gelu;
-// y [Mt, N / 2]).
+// y [Mt, N / 2]); glu = 3: y = relu(x W^T)^2, glu = 4: y = x W^T in fp32.
 // x [Mt <= 256, K], W [N, K], all bf16 row-major; returns -20 when the shape is outside what this kernel covers.
 extern "C" int rb_decode_gemm(const void* x, const void* W, void* y, int Mt, int N, int K, int ldx, int ldw, int glu,
                               int splits, int* err, cudaStream_t st) {
@@ -358,13 +365,15 @@ extern "C" int rb_decode_gemm(const void* x, const void* W, void* y, int Mt, int
   if (Mt <= 0 || N <= 0 || K <= 0) return 0;
   if (Mt > 256 || (ldx % 8) || (ldw % 8) || (K % 8)) return -20;
   if ((reinterpret_cast<uintptr_t>(x) % 16) || (reinterpret_cast<uintptr_t>(W) % 16)) return -20;
+  const int post = glu == 3 ? 1 : (glu == 4 ? 2 : 0);
+  if (post) glu = 0;
   if (glu && ((N / 2) % 64)) return -20;
-  if ((N % 4) || (reinterpret_cast<uintptr_t>(y) % 8)) return -20;   // 4 features per store
+  if ((N % 4) || (reinterpret_cast<uintptr_t>(y) % (post == 2 ? 16 : 8))) return -20;   // 4 features per store
   const int nt = Mt <= 64 ? 64 : (Mt <= 128 ? 128 : 256);
   const int tiles = glu ? (N / 2) / 64 : (N + BM - 1) / BM;
   const int k_iters = (K + BK - 1) / BK;
   Params p{};
-  p.Mt = Mt; p.N = N; p.K = K; p.glu = glu; p.out = y; p.err = err;
+  p.Mt = Mt; p.N = N; p.K = K; p.glu = glu; p.post = post; p.out = y; p.err = err;
   p.S = splits > 0 ? splits : rb_decode_gemm_splits(tiles, k_iters);
   if (p.S > 8) p.S = 8;
   while (p.S & (p.S - 1)) p.S &= p.S - 1;       // the reduction slices the tile in powers of two

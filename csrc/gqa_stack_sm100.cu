@@ -1,0 +1,233 @@
+// Around the attention of composed stacks with cached keys and values: angles, rotation + norm + cache write, and a CUDA-core
+// attention for any sizes.  Compiled WITHOUT fast-math: the 32-bit mode of the engine uses these kernels as they are.
+//
+//  * rope_table        cos / sin of every row's angles, once per forward
+//  * attention_inputs  raw projections -> rotated and normed queries; keys and values into their pages
+//  * paged_attention   one (row, head) per CTA: 32-bit mode, and head sizes that the tensor-core kernels do not take
+#include "stack_common.cuh"
+
+namespace rb {
+namespace stack {
+
+__global__ void rope_table_kernel(const int* __restrict__ pos, int offset, const double* __restrict__ freq, float2* __restrict__ out, int rows,
+                                  int half) {
+  const int i = blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= rows * half) return;
+  const int t = i / half;
+  double s, c;
+  sincos(static_cast<double>(pos[t] + offset) * freq[i - t * half], &s, &c);      // late positions keep their low bits
+  out[i] = make_float2(static_cast<float>(c), static_cast<float>(s));
+}
+
+struct InputParams {
+  const void* qkv;           // [T][ld]: H query heads | G key heads | G value heads (keys and values only with k_pool)
+  const float2* table;       // [T][rot / 2] or null
+  void* q;                   // [T][H][dp]
+  void* k_pool;              // [rows][G][dp] or null
+  void* v_pool;              // [rows][G][vp]
+  const long long* slots;    // [T] pool rows
+  long long pool_rows;
+  int T, H, G, dim, vdim, dp, vp, rot, ld;
+  float eps;                 // <= 0: no norm
+};
+// One warp per (row, head); lane l holds the feature pairs l, l + 32, ...
+template <typename T, int NP, bool kPair>
+__global__ void __launch_bounds__(256) attention_inputs_kernel(const InputParams p) {
+  const int lane = threadIdx.x & 31;
+  const int per = p.H + (p.k_pool ? 2 * p.G : 0);
+  const long long u = static_cast<long long>(blockIdx.x) * 8 + (threadIdx.x >> 5);
+  if (u >= static_cast<long long>(p.T) * per) return;
+  const int t = static_cast<int>(u / per), hd = static_cast<int>(u - static_cast<long long>(t) * per);
+  const T* src = static_cast<const T*>(p.qkv) + static_cast<long long>(t) * p.ld;
+  const bool value = hd >= p.H + p.G;
+  const int n = value ? p.vdim : p.dim, pitch = value ? p.vp : p.dp;
+  T* dst;
+  if (hd < p.H) {
+    src += hd * p.dim;
+    dst = static_cast<T*>(p.q) + (static_cast<long long>(t) * p.H + hd) * p.dp;
+  } else {
+    const long long slot = p.slots[t];
+    if (slot < 0 || slot >= p.pool_rows) return;
+    const int g = hd - p.H - (value ? p.G : 0);
+    src += p.H * p.dim + (value ? p.G * p.dim + g * p.vdim : g * p.dim);
+    dst = static_cast<T*>(value ? p.v_pool : p.k_pool) + (slot * p.G + g) * pitch;
+  }
+  float a[NP], b[NP], ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < NP; ++i) {
+    const int e = 2 * (lane + 32 * i);
+    a[i] = b[i] = 0.f;
+    if constexpr (kPair) {
+      if (e < n) {
+        if constexpr (sizeof(T) == 4) {
+          const float2 x = *reinterpret_cast<const float2*>(src + e);
+          a[i] = x.x;
+          b[i] = x.y;
+        } else {
+          const uint32_t x = *reinterpret_cast<const uint32_t*>(src + e);
+          a[i] = __uint_as_float(x << 16);
+          b[i] = __uint_as_float(x & 0xffff0000u);
+        }
+      }
+    } else {
+      if (e < n) a[i] = ld(src + e);
+      if (e + 1 < n) b[i] = ld(src + e + 1);
+    }
+    if (!value && e < p.rot) {
+      const float2 cs = p.table[static_cast<long long>(t) * (p.rot >> 1) + (e >> 1)];
+      const float x = a[i] * cs.x - b[i] * cs.y;
+      b[i] = b[i] * cs.x + a[i] * cs.y;
+      a[i] = x;
+    }
+    ss += a[i] * a[i] + b[i] * b[i];
+  }
+  float r = 1.f;
+  if (!value && p.eps > 0.f) r = 1.f / sqrtf(wsum(ss) / p.dim + p.eps);
+#pragma unroll
+  for (int i = 0; i < NP; ++i) {      // columns behind the head's features are written as zeros
+    const int e = 2 * (lane + 32 * i);
+    if (e >= pitch) continue;
+    if constexpr (sizeof(T) == 4) {
+      *reinterpret_cast<float2*>(dst + e) = make_float2(a[i] * r, b[i] * r);
+    } else {
+      const __nv_bfloat162 v = __floats2bfloat162_rn(a[i] * r, b[i] * r);
+      *reinterpret_cast<__nv_bfloat162*>(dst + e) = v;
+    }
+  }
+}
+
+// CTA = (row, head), every warp walks every fourth visible position, a lane holds NR features of query, accumulator, key and
+// value; the four running softmaxes and the sink are merged at the end.
+struct GqaParams {
+  const void* q;            // [rows][H][dp]
+  const void* k_pool;       // [pool rows][G][dp]
+  const void* v_pool;       // [pool rows][G][vp]
+  const int* block_tables;
+  const int* row_seg;       // [rows] or null (row = segment)
+  const int* row_pos;       // [rows] last visible position; null: ctx[row] - 1
+  const int* ctx;
+  const void* sink;         // [H] or null
+  void* out;                // [rows][H][vo]
+  int H, G, dp, vp, vo, max_blocks, block_size;
+  float scale;
+};
+template <typename T, int NR>
+__global__ void __launch_bounds__(128) gqa_attn_kernel(const GqaParams p) {
+  extern __shared__ float sm[];                 // [4][vp] accumulators
+  __shared__ float sml[4][2];
+  const int row = blockIdx.x, hd = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int g = hd / (p.H / p.G);
+  const int seg = p.row_seg ? p.row_seg[row] : row;
+  const int n = (p.row_pos ? p.row_pos[row] : p.ctx[row] - 1) + 1;
+  const int* bt = p.block_tables + static_cast<long long>(seg) * p.max_blocks;
+  const T* qp = static_cast<const T*>(p.q) + (static_cast<long long>(row) * p.H + hd) * p.dp;
+  float q[NR], o[NR];
+#pragma unroll
+  for (int i = 0; i < NR; ++i) {
+    const int c = lane + 32 * i;
+    q[i] = c < p.dp ? ld(qp + c) : 0.f;
+    o[i] = 0.f;
+  }
+  float m = -INFINITY, l = 0.f;
+  for (int k = warp; k < n; k += 4) {
+    const long long at = (static_cast<long long>(bt[k / p.block_size]) * p.block_size + k % p.block_size) * p.G + g;
+    const T* kp = static_cast<const T*>(p.k_pool) + at * p.dp;
+    const T* vp = static_cast<const T*>(p.v_pool) + at * p.vp;
+    float x[NR], s = 0.f;
+#pragma unroll
+    for (int i = 0; i < NR; ++i) {
+      const int c = lane + 32 * i;
+      if (c < p.dp) s += q[i] * ld(kp + c);
+      x[i] = c < p.vp ? ld(vp + c) : 0.f;
+    }
+    s = wsum(s) * p.scale;
+    const float mn = fmaxf(m, s), a = expf(m - mn), e = expf(s - mn);
+    m = mn;
+    l = l * a + e;
+#pragma unroll
+    for (int i = 0; i < NR; ++i) o[i] = o[i] * a + e * x[i];
+  }
+  if (lane == 0) { sml[warp][0] = m; sml[warp][1] = l; }
+#pragma unroll
+  for (int i = 0; i < NR; ++i)
+    if (lane + 32 * i < p.vp) sm[warp * p.vp + lane + 32 * i] = o[i];
+  __syncthreads();
+  float M = fmaxf(fmaxf(sml[0][0], sml[1][0]), fmaxf(sml[2][0], sml[3][0]));
+  const float sink = p.sink ? ld(static_cast<const T*>(p.sink) + hd) : 0.f;
+  if (p.sink) M = fmaxf(M, sink);
+  float w[4], L = p.sink ? expf(sink - M) : 0.f;
+#pragma unroll
+  for (int k = 0; k < 4; ++k) {
+    w[k] = sml[k][0] == -INFINITY ? 0.f : expf(sml[k][0] - M);
+    L += w[k] * sml[k][1];
+  }
+  const float f = L > 0.f ? 1.f / L : 0.f;
+  T* out = static_cast<T*>(p.out) + (static_cast<long long>(row) * p.H + hd) * p.vo;
+  for (int c = threadIdx.x; c < p.vo; c += 128)
+    st(out + c, (w[0] * sm[c] + w[1] * sm[p.vp + c] + w[2] * sm[2 * p.vp + c] + w[3] * sm[3 * p.vp + c]) * f);
+}
+
+template <typename T, bool kPair>
+static int launch_inputs(const InputParams& p, cudaStream_t stm) {
+  const long long units = static_cast<long long>(p.T) * (p.H + (p.k_pool ? 2 * p.G : 0));
+  const unsigned grid = static_cast<unsigned>((units + 7) / 8);
+  const int w = p.k_pool ? (p.dp > p.vp ? p.dp : p.vp) : p.dp;
+  if (w <= 128) attention_inputs_kernel<T, 2, kPair><<<grid, 256, 0, stm>>>(p);
+  else if (w <= 256) attention_inputs_kernel<T, 4, kPair><<<grid, 256, 0, stm>>>(p);
+  else if (w <= 512) attention_inputs_kernel<T, 8, kPair><<<grid, 256, 0, stm>>>(p);
+  else return -2;
+  rb_note_launch(1);
+  return static_cast<int>(cudaGetLastError());
+}
+
+template <typename T>
+static int launch_gqa(const GqaParams& p, int rows, cudaStream_t stm) {
+  const size_t smem = 4 * static_cast<size_t>(p.vp) * 4;
+  const dim3 grid(rows, p.H);
+  const int w = p.dp > p.vp ? p.dp : p.vp;
+  if (w <= 64) gqa_attn_kernel<T, 2><<<grid, 128, smem, stm>>>(p);
+  else if (w <= 128) gqa_attn_kernel<T, 4><<<grid, 128, smem, stm>>>(p);
+  else if (w <= 256) gqa_attn_kernel<T, 8><<<grid, 128, smem, stm>>>(p);
+  else if (w <= 512) gqa_attn_kernel<T, 16><<<grid, 128, smem, stm>>>(p);
+  else return -2;
+  rb_note_launch(1);
+  return static_cast<int>(cudaGetLastError());
+}
+
+}  // namespace stack
+}  // namespace rb
+
+using namespace rb;
+using namespace rb::stack;
+typedef __nv_bfloat16 bf16;
+
+// out [rows][half] (cos, sin) of (pos + offset) * freq
+extern "C" int rb_rope_table(const int* pos, int offset, const double* freq, float* out, int rows, int half, cudaStream_t stm) {
+  if (rows <= 0 || half <= 0) return 0;
+  const long long n = static_cast<long long>(rows) * half;
+  if (n > (1ll << 30)) return -2;
+  rope_table_kernel<<<static_cast<unsigned>((n + 127) / 128), 128, 0, stm>>>(pos, offset, freq, reinterpret_cast<float2*>(out), rows, half);
+  rb_note_launch(1);
+  return static_cast<int>(cudaGetLastError());
+}
+
+extern "C" int rb_attention_inputs(const void* qkv, int ld, const float* table, void* q, void* k_pool, void* v_pool, const long long* slots,
+                                   long long pool_rows, int T, int H, int G, int dim, int vdim, int dp, int vp, int rot, float eps, int fp32,
+                                   cudaStream_t stm) {
+  if (T <= 0) return 0;
+  if (H < 1 || dim < 1 || dp < dim || dp % 2 || rot % 2 || rot < 0 || rot > dim || (rot && !table)) return -2;
+  if (ld < H * dim + (k_pool ? G * (dim + vdim) : 0) || (k_pool && (!v_pool || !slots || G < 1 || vdim < 1 || vp < vdim || vp % 2))) return -2;
+  InputParams p{qkv, reinterpret_cast<const float2*>(table), q, k_pool, v_pool, slots, pool_rows, T, H, G, dim, vdim, dp, vp, rot, ld, eps};
+  const bool pair = dim % 2 == 0 && (!k_pool || vdim % 2 == 0) && ld % 2 == 0 && reinterpret_cast<uintptr_t>(qkv) % 8 == 0;
+  if (fp32) return pair ? launch_inputs<float, true>(p, stm) : launch_inputs<float, false>(p, stm);
+  return pair ? launch_inputs<bf16, true>(p, stm) : launch_inputs<bf16, false>(p, stm);
+}
+
+extern "C" int rb_gqa_attn(const void* q, const void* k_pool, const void* v_pool, const int* block_tables, const int* row_seg, const int* row_pos,
+                           const int* ctx, const void* sink, void* out, int rows, int H, int G, int dp, int vp, int vo, int max_blocks,
+                           int block_size, float scale, int fp32, cudaStream_t stm) {
+  if (rows <= 0) return 0;
+  if (G < 1 || H % G || vo > vp || H > 65535) return -2;
+  GqaParams p{q, k_pool, v_pool, block_tables, row_seg, row_pos, ctx, sink, out, H, G, dp, vp, vo, max_blocks, block_size, scale};
+  return fp32 ? launch_gqa<float>(p, rows, stm) : launch_gqa<bf16>(p, rows, stm);
+}

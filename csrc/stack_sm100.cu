@@ -5,93 +5,17 @@
 // mode can afford the hardware approximations (relative error around 1e-6) the code asks for them by intrinsic.
 //
 //  * embed_rows     token rows -> fp32 residual stream and its 16-bit copy
-//  * norm_add       residual += group norm of a sublayer's output; writes the next sublayer's input (or its final norm)
+//  * norm_add       residual += group norm of a sublayer's output; writes the next sublayer's input (or its final norm); one form
+//                   first sums the weighted rows of a token's experts, one starts the stream with normed embeddings
 //  * hgrn2_step     one token per sequence: gates, state update, read-out and per-head norm in one pass over the state
 //  * hgrn2_scan     segments of any length: the state stays in registers while the tokens stream through shared memory
 //  * latent_write   norm of the latent projection, scattered into the paged latent cache
 //  * latent_attn    CUDA-core attention over paged latent rows (any sizes, fp32 or bf16)
 //  * glu, gate_heads, and a CUDA-core GEMM for fp32 and for shapes that no tensor-core kernel takes
-#include <cuda_bf16.h>
-#include <cuda_runtime.h>
-#include <stdint.h>
-
-#include "host_utils.h"
+#include "stack_common.cuh"
 
 namespace rb {
 namespace stack {
-
-__device__ __forceinline__ float ld(const float* p) { return *p; }
-__device__ __forceinline__ float ld(const __nv_bfloat16* p) { return __bfloat162float(*p); }
-__device__ __forceinline__ void st(float* p, float v) { *p = v; }
-__device__ __forceinline__ void st(__nv_bfloat16* p, float v) { *p = __float2bfloat16(v); }
-
-// eight consecutive elements, 16-byte aligned
-struct F8 { float v[8]; };
-__device__ __forceinline__ F8 unpack8(const uint4& u) {
-  F8 r;
-  const uint32_t w[4] = {u.x, u.y, u.z, u.w};
-#pragma unroll
-  for (int i = 0; i < 4; ++i) {
-    r.v[2 * i] = __uint_as_float(w[i] << 16);
-    r.v[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
-  }
-  return r;
-}
-__device__ __forceinline__ F8 ld8(const __nv_bfloat16* p) { return unpack8(*reinterpret_cast<const uint4*>(p)); }
-__device__ __forceinline__ F8 ld8(const float* p) {
-  F8 r;
-  *reinterpret_cast<float4*>(r.v) = reinterpret_cast<const float4*>(p)[0];
-  *reinterpret_cast<float4*>(r.v + 4) = reinterpret_cast<const float4*>(p)[1];
-  return r;
-}
-__device__ __forceinline__ void st8(float* p, const F8& r) {
-  reinterpret_cast<float4*>(p)[0] = *reinterpret_cast<const float4*>(r.v);
-  reinterpret_cast<float4*>(p)[1] = *reinterpret_cast<const float4*>(r.v + 4);
-}
-__device__ __forceinline__ void st8(__nv_bfloat16* p, const F8& r) {
-  uint4 u;
-  uint32_t* w = reinterpret_cast<uint32_t*>(&u);
-#pragma unroll
-  for (int i = 0; i < 4; ++i) {
-    const __nv_bfloat162 b = __floats2bfloat162_rn(r.v[2 * i], r.v[2 * i + 1]);
-    w[i] = *reinterpret_cast<const uint32_t*>(&b);
-  }
-  *reinterpret_cast<uint4*>(p) = u;
-}
-template <int V, typename T>
-__device__ __forceinline__ void ldv(const T* p, float* v) {
-  if constexpr (V == 8) {
-    const F8 r = ld8(p);
-#pragma unroll
-    for (int i = 0; i < 8; ++i) v[i] = r.v[i];
-  } else {
-    v[0] = ld(p);
-  }
-}
-template <int V, typename T>
-__device__ __forceinline__ void stv(T* p, const float* v) {
-  if constexpr (V == 8) {
-    F8 r;
-#pragma unroll
-    for (int i = 0; i < 8; ++i) r.v[i] = v[i];
-    st8(p, r);
-  } else {
-    st(p, v[0]);
-  }
-}
-
-__device__ __forceinline__ float wsum(float v) {
-#pragma unroll
-  for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-  return v;
-}
-// 1 / (1 + exp(-x)): IEEE expf and division in 32-bit mode, hardware approximations in 16-bit mode
-template <bool kExact>
-__device__ __forceinline__ float sigmoid(float x) {
-  if constexpr (kExact) return 1.f / (1.f + expf(-x));
-  else return __fdividef(1.f, 1.f + __expf(-x));      // x << 0: the denominator overflows to inf, the quotient is 0
-}
-template <typename T> struct IsExact { static constexpr bool v = sizeof(T) == 4; };
 
 // ------------------------------------------------------------------------------------------------- embedding
 template <typename T>
@@ -114,6 +38,8 @@ __global__ void embed_rows_kernel(const long long* __restrict__ tok, const T* __
 // One CTA per row.  `parts` consecutive sets of warps own one group at a time (wpg warps per group), so groups are
 // reduced side by side; sums of the warps of a group meet in shared memory.
 constexpr int NA_WARPS = 8;
+template <typename T, bool kSum> struct YType { typedef T type; };
+template <typename T> struct YType<T, true> { typedef float type; };
 struct NormAddParams {
   float* res;             // [rows][pitch] fp32, updated in place
   const void* y;          // [rows][ldy]
@@ -122,12 +48,63 @@ struct NormAddParams {
   void* h;                // [rows][pitch]
   int ldy, pitch, width, groups, wpg;
   float eps;
+  // NA_EMBED: y is the embedding table, row `tok[row]` of it is normed, and the stream starts with the result
+  const long long* tok;
+  int vocab;
+  // NA_SUM: y (or nothing, when null) plus the weighted rows of `top` experts per row; ex [sorted rows][ldy], row of a
+  // choice = offset[expert] + place
+  const void* ex;
+  const int* expert;      // [rows][top]
+  const int* place;       // [rows][top]
+  const int* offset;      // [experts + 1]
+  const float* weight;    // [rows][top]
+  int top;
 };
-template <typename T, int V>
+enum : int { NA_PLAIN = 0, NA_EMBED = 1, NA_SUM = 2 };
+constexpr int NA_MAX_TOP = 64;
+template <typename T, int V, int MODE>
 __global__ void __launch_bounds__(NA_WARPS * 32) norm_add_kernel(const NormAddParams p) {
   __shared__ float red[2][NA_WARPS];
+  extern __shared__ __align__(16) float ysum[];      // [width] (NA_SUM)
   const long long row = blockIdx.x;
-  const T* y = static_cast<const T*>(p.y) + row * p.ldy;
+  using Y = typename YType<T, MODE == NA_SUM>::type;
+  const Y* y;
+  bool known = true;
+  if constexpr (MODE == NA_SUM) {
+    __shared__ long long s_row[NA_MAX_TOP];
+    __shared__ float s_w[NA_MAX_TOP];
+    if (threadIdx.x < p.top) {
+      const long long i = row * p.top + threadIdx.x;
+      s_row[threadIdx.x] = (static_cast<long long>(p.offset[p.expert[i]]) + p.place[i]) * p.ldy;
+      s_w[threadIdx.x] = p.weight[i];
+    }
+    __syncthreads();
+    const T* base = p.y ? static_cast<const T*>(p.y) + row * p.ldy : nullptr;
+    const T* ex = static_cast<const T*>(p.ex);
+    for (int c = threadIdx.x * V; c < p.width; c += NA_WARPS * 32 * V) {
+      float a[V];
+#pragma unroll
+      for (int i = 0; i < V; ++i) a[i] = 0.f;
+      if (base) ldv<V>(base + c, a);
+#pragma unroll 4
+      for (int k = 0; k < p.top; ++k) {
+        float b[V];
+        ldv<V>(ex + s_row[k] + c, b);
+        const float w = s_w[k];
+#pragma unroll
+        for (int i = 0; i < V; ++i) a[i] += w * b[i];
+      }
+      stv<V>(ysum + c, a);
+    }
+    __syncthreads();
+    y = ysum;
+  } else if constexpr (MODE == NA_EMBED) {
+    const long long id = p.tok[row];
+    known = id >= 0 && id < p.vocab;
+    y = static_cast<const T*>(p.y) + (known ? id : 0) * p.ldy;
+  } else {
+    y = static_cast<const T*>(p.y) + row * p.ldy;
+  }
   const T* w = static_cast<const T*>(p.w);
   const T* nw = static_cast<const T*>(p.next_w);
   float* res = p.res + row * p.pitch;
@@ -155,13 +132,18 @@ __global__ void __launch_bounds__(NA_WARPS * 32) norm_add_kernel(const NormAddPa
       ss = 0.f;
       for (int k = 0; k < wpg; ++k) ss += red[0][first + k];
     }
-    const float r = 1.f / sqrtf(ss * inv_n + p.eps);
+    const float r = known ? 1.f / sqrtf(ss * inv_n + p.eps) : 0.f;
     float s2 = 0.f;
     for (int c = lo + l * V; c < hi; c += lanes * V) {
       float a[V], b[V], x[V];
       ldv<V>(y + c, a);
       ldv<V>(w + c, b);
-      ldv<V>(res + c, x);
+      if constexpr (MODE == NA_EMBED) {
+#pragma unroll
+        for (int i = 0; i < V; ++i) x[i] = 0.f;
+      } else {
+        ldv<V>(res + c, x);
+      }
 #pragma unroll
       for (int i = 0; i < V; ++i) {
         x[i] += a[i] * r * b[i];
@@ -190,7 +172,10 @@ __global__ void __launch_bounds__(NA_WARPS * 32) norm_add_kernel(const NormAddPa
     }
     if (wpg > 1) __syncthreads();      // the next pass rewrites the sums
   }
-  for (int c = p.width + threadIdx.x; c < p.pitch; c += blockDim.x) st(h + c, 0.f);
+  for (int c = p.width + threadIdx.x; c < p.pitch; c += blockDim.x) {
+    st(h + c, 0.f);
+    if constexpr (MODE == NA_EMBED) st(res + c, 0.f);
+  }
 }
 
 // ------------------------------------------------------------------------------------------------- HGRN2
@@ -742,22 +727,47 @@ extern "C" int rb_embed_rows(const long long* tok, const void* w, float* res, vo
   return static_cast<int>(cudaGetLastError());
 }
 
+template <int MODE>
+static int launch_norm_add(NormAddParams p, int rows, bool vec, int fp32, cudaStream_t stm) {
+  while (p.wpg < NA_WARPS && p.groups * p.wpg * 2 <= NA_WARPS) p.wpg *= 2;
+  const size_t smem = MODE == NA_SUM ? static_cast<size_t>(p.width) * 4 : 0;
+  auto k = fp32 ? (vec ? norm_add_kernel<float, 8, MODE> : norm_add_kernel<float, 1, MODE>)
+                : (vec ? norm_add_kernel<bf16, 8, MODE> : norm_add_kernel<bf16, 1, MODE>);
+  if (smem > 40 * 1024) {
+    if (smem > 200 * 1024) return -2;
+    const cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
+    if (e != cudaSuccess) return static_cast<int>(e);
+  }
+  k<<<rows, NA_WARPS * 32, smem, stm>>>(p);
+  rb_note_launch(1);
+  return static_cast<int>(cudaGetLastError());
+}
+
 extern "C" int rb_norm_add(float* res, const void* y, const void* w, const void* next_w, void* h, int rows, int ldy, int pitch, int width,
                            int groups, float eps, int fp32, cudaStream_t stm) {
   if (rows <= 0) return 0;
   if (groups < 1 || width % groups || pitch < width || pitch % 8 || ldy % 8) return -2;
   NormAddParams p{res, y, w, next_w, h, ldy, pitch, width, groups, 1, eps};
-  while (p.wpg < NA_WARPS && groups * p.wpg * 2 <= NA_WARPS) p.wpg *= 2;
-  const bool vec = (width / groups) % 8 == 0;
-  if (fp32) {
-    if (vec) norm_add_kernel<float, 8><<<rows, NA_WARPS * 32, 0, stm>>>(p);
-    else norm_add_kernel<float, 1><<<rows, NA_WARPS * 32, 0, stm>>>(p);
-  } else {
-    if (vec) norm_add_kernel<bf16, 8><<<rows, NA_WARPS * 32, 0, stm>>>(p);
-    else norm_add_kernel<bf16, 1><<<rows, NA_WARPS * 32, 0, stm>>>(p);
-  }
-  rb_note_launch(1);
-  return static_cast<int>(cudaGetLastError());
+  return launch_norm_add<NA_PLAIN>(p, rows, (width / groups) % 8 == 0, fp32, stm);
+}
+
+// y may be null; ex [sorted rows][ldy] are expert outputs (see NormAddParams), offset has one entry more than there are experts
+extern "C" int rb_norm_add_experts(float* res, const void* y, const void* ex, const int* expert, const int* place, const int* offset,
+                                   const float* weight, int top, const void* w, const void* next_w, void* h, int rows, int ldy, int pitch,
+                                   int width, int groups, float eps, int fp32, cudaStream_t stm) {
+  if (rows <= 0) return 0;
+  if (groups < 1 || width % groups || pitch < width || pitch % 8 || ldy % 8 || top < 1 || top > NA_MAX_TOP) return -2;
+  NormAddParams p{res, y, w, next_w, h, ldy, pitch, width, groups, 1, eps, nullptr, 0, ex, expert, place, offset, weight, top};
+  return launch_norm_add<NA_SUM>(p, rows, (width / groups) % 8 == 0, fp32, stm);
+}
+
+// the stream starts with the normed rows of the embedding table
+extern "C" int rb_embed_norm(const long long* tok, const void* table, const void* w, float* res, void* h, int rows, int vocab, int pitch, int width,
+                             int groups, float eps, int fp32, cudaStream_t stm) {
+  if (rows <= 0) return 0;
+  if (groups < 1 || width % groups || pitch < width || pitch % 8) return -2;
+  NormAddParams p{res, table, w, nullptr, h, pitch, pitch, width, groups, 1, eps, tok, vocab};
+  return launch_norm_add<NA_EMBED>(p, rows, (width / groups) % 8 == 0, fp32, stm);
 }
 
 // cu == null: one row per segment.  o_raw: scratch [rows][H][vdim] fp32, needed with cu.

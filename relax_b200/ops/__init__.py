@@ -102,9 +102,11 @@ def paged_attention(q, k_pool, v_pool, batch, block_size, scale, sink, out_width
     return ref.paged_attention(q, k_pool, v_pool, batch.block_tables, block_size, batch.ctx, batch.cu, scale, sink, out_width)
 
 
-def moe_route(logits, spec):
-    """Expert choice of every row (:class:`relax_b200.models.config.MoESpec`)."""
-    return (_cuda() if _use_cuda(logits) else ref).moe_route(logits, spec)
+def moe_route(logits, spec, dtype):
+    """Expert choice of every row (:class:`relax_b200.models.config.MoESpec`) from fp32 logits; ``dtype``: of the experts' operands."""
+    if _use_cuda(logits):
+        return _cuda().moe_route(logits, spec, 64 if dtype == torch.float32 else 128)      # rows per tile of the grouped GEMM
+    return ref.moe_route(logits, spec)
 
 
 def moe_experts(h, plan, up, down, act):

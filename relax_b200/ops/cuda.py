@@ -211,13 +211,14 @@ GLU_ACT = {"silu": 1, "gelu_tanh": 2}
 
 
 def _decode_gemm(x, w, glu_act: int):
-    """Weight-streaming decode GEMM (csrc/gemm_decode_sm100.cu) when the shape is in its range, else None."""
+    """Weight-streaming decode GEMM (csrc/gemm_decode_sm100.cu) when the shape is in its range, else None.  ``glu_act``: 0 none,
+    1 and 2 gated units (:data:`GLU_ACT`), 3 squared relu without a gate, 4 fp32 results."""
     if not _DECODE_GEMM or x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 or x.shape[0] > 128:
         return None     # above 128 rows the 2-stage ring of the 256-column variant loses to the other paths (measured)
     if w.stride(1) != 1 or w.stride(0) % 8 or w.data_ptr() % 16:
         return None
     N = w.shape[0]
-    out = torch.empty(x.shape[0], N // 2 if glu_act else N, dtype=x.dtype, device=x.device)
+    out = torch.empty(x.shape[0], N // 2 if glu_act in (1, 2) else N, dtype=torch.float32 if glu_act == 4 else x.dtype, device=x.device)
     if _load().decode_gemm(x, w, out, glu_act, 0, err_flag(x.device)):
         return out
     return None
@@ -303,20 +304,142 @@ def linear_glu(x, w, act: str = "silu"):
     return glu(linear(x, w), act)
 
 
+def linear_relu2(x, w):
+    """``relu(x @ w.T) ** 2``: the activation joins the decode GEMM's reduction for up to 128 rows."""
+    if x.dtype == torch.bfloat16 and x.shape[0] <= 128:
+        x, _ = _rowmajor_2d(x)
+        y = _decode_gemm(x, w, 3)
+        if y is not None:
+            return y
+    y = linear(x, w)
+    _load().relu2(y)
+    return y
+
+
+def linear_fp32(x, w):
+    """``x @ w.T`` with fp32 results from bf16 (or fp32) operands."""
+    if x.dtype == torch.float32:
+        return linear(x, w)
+    x, ld = _rowmajor_2d(x)
+    y = _decode_gemm(x, w, 4)
+    return matmul_nt(x, w, out_dtype=torch.float32) if y is None else y
+
+
 # --------------------------------------------------------------------------- composed stacks (inference)
 
 
-def embed_rows(tokens, w):
+def embed_rows(tokens, w, norm_w=None, width=0, groups=1, eps=0.0):
     res = torch.empty(tokens.shape[0], w.shape[1], dtype=torch.float32, device=w.device)
     h = torch.empty(tokens.shape[0], w.shape[1], dtype=w.dtype, device=w.device)
-    _load().embed_rows(tokens, w, res, h)
+    if norm_w is None:
+        _load().embed_rows(tokens, w, res, h)
+    else:
+        _load().embed_norm(tokens, w, norm_w, res, h, int(width), int(groups), float(eps))
     return res, h
 
 
-def norm_add(res, y, w, width, groups, eps, next_w=None):
+def norm_add(res, y, w, width, groups, eps, next_w=None, experts=None):
     h = torch.empty(res.shape, dtype=w.dtype, device=w.device)
-    _load().norm_add(res, y, w, next_w, h, int(width), int(groups), float(eps))
+    if experts is None:
+        _load().norm_add(res, y, w, next_w, h, int(width), int(groups), float(eps))
+    else:
+        rows, plan = experts
+        _load().norm_add_experts(res, y, rows, plan.expert, plan.place, plan.offset, plan.weight, w, next_w, h, int(width), int(groups), float(eps))
     return h
+
+
+def rope_table(positions, offset, inv_freq):
+    out = torch.empty(positions.shape[0], inv_freq.shape[0], 2, dtype=torch.float32, device=positions.device)
+    _load().rope_table(positions, int(offset), inv_freq, out)
+    return out
+
+
+def attention_inputs(qkv, table, heads, kv_heads, dim, vdim, dp, rot_dims, eps, k_pool, v_pool, slots):
+    q = torch.empty(qkv.shape[0], heads, dp, dtype=qkv.dtype, device=qkv.device)
+    _load().attention_inputs(qkv, table, q, k_pool, v_pool, slots, int(kv_heads), int(dim), int(vdim), int(rot_dims), float(eps))
+    return q
+
+
+def decode_splits(rows: int, kv_heads: int, max_ctx: int) -> int:
+    """Parts of the context that run side by side: enough CTAs to fill the machine twice, at least 512 positions each, none
+    when the batch alone fills it."""
+    ctas, splits = rows * kv_heads, 1
+    if ctas >= 148:
+        return 1
+    while ctas * splits < 296 and (max_ctx + splits - 1) // splits > 512 and splits < 32:
+        splits *= 2
+    return splits
+
+
+def paged_attention(q, k_pool, v_pool, b, block_size, scale, sink, out_width):
+    """bf16 heads of up to 128 features: segments of several rows on the flash kernel, single rows on the decode kernel (the
+    flash kernel when more than 16 heads share keys); anything else, and fp32, on CUDA cores."""
+    T, H, dp = q.shape
+    G = k_pool.shape[1]
+    L, err = _load(), err_flag(q.device)
+    out = torch.empty(T, H * out_width, dtype=q.dtype, device=q.device)
+    n, s = (0, 0) if b.cu is None else (b.multi_rows, b.multi_segs)
+    if q.dtype == torch.bfloat16 and max(dp, v_pool.shape[2]) <= 128 and H // G <= 128:
+        ok = n == 0 or L.paged_flash(q[:n], k_pool, v_pool, b.block_tables, b.ctx, b.blocks[128 // (H // G)], sink, out[:n], int(block_size),
+                                     float(scale), err)
+        if ok and n == T:
+            return out
+        if ok:
+            bt, ctx = b.block_tables[s:], b.ctx[s:]
+            if H // G <= 16:
+                splits = decode_splits(T - n, G, b.max_ctx_one)
+                po = ml = None
+                if splits > 1:
+                    po = torch.empty(splits * (T - n) * H * 128, dtype=torch.float32, device=q.device)
+                    ml = torch.empty(splits * (T - n) * H * 2, dtype=torch.float32, device=q.device)
+                ok = L.paged_decode(q[n:], k_pool, v_pool, bt, ctx, sink, out[n:], po, ml, int(block_size), int(b.max_ctx_one), splits, float(scale), err)
+            else:
+                ok = L.paged_flash(q[n:], k_pool, v_pool, bt, ctx, None, sink, out[n:], int(block_size), float(scale), err)
+            if ok:
+                return out
+    L.gqa_attn(q, k_pool, v_pool, b.block_tables, b.seg_of, b.pos, b.ctx, sink, out, int(block_size), float(scale))
+    return out
+
+
+class ExpertPlan:
+    """Device description of one layer's routing: per row and choice ``expert``, ``weight`` and ``place`` (its row among the expert's
+    rows), the token of every expert row, the experts' first sorted rows, and the tile list of the grouped GEMMs."""
+    __slots__ = ("expert", "weight", "place", "row_token", "offset", "tiles", "n_tiles")
+
+
+def moe_route(logits, spec, tile_rows):
+    T, E, k, dev = logits.shape[0], spec.experts, spec.top, logits.device
+    p = ExpertPlan()
+    i32 = lambda *s: torch.empty(*s, dtype=torch.int32, device=dev)
+    p.expert, p.place, p.row_token, p.offset, p.n_tiles = i32(T, k), i32(T, k), i32(E, T), i32(E + 1), i32(1)
+    p.weight = torch.empty(T, k, dtype=torch.float32, device=dev)
+    p.tiles = i32(min(T * k, E) + T * k // tile_rows, 4)
+    count = torch.zeros(E + 1, dtype=torch.int32, device=dev)
+    _load().moe_route(logits, p.expert, p.weight, p.place, p.row_token, count, p.offset, p.tiles, p.n_tiles, E, spec.groups, spec.keep, tile_rows,
+                      bool(spec.renormalize), float(spec.weight_scale))
+    return p
+
+
+def _moe_tile_width(rows: int, experts: int, n: int) -> int:
+    """Columns per tile: wide ones when every expert has full row tiles, narrow ones while they would leave SMs idle."""
+    tiles = min(rows, experts) + rows // 128
+    for bn in (256, 128):
+        if tiles * ((n + bn - 1) // bn) >= (296 if bn == 256 else 148) and (bn == 128 or rows >= 64 * experts):
+            return bn
+    return 64
+
+
+def moe_experts(h, plan, up, down, act):
+    """Sorted expert rows ``[T top, W]``: gather, up-projection and activation in one grouped GEMM, down-projection in a second."""
+    if act != "relu2":
+        raise ValueError(f"no ungated activation {act!r}")
+    R, E, err = plan.expert.numel(), up.shape[0], err_flag(h.device)
+    mid = torch.empty(R, up.shape[1], dtype=h.dtype, device=h.device)
+    out = torch.empty(R, down.shape[1], dtype=h.dtype, device=h.device)
+    L = _load()
+    L.moe_gemm(h, up, mid, plan.tiles, plan.n_tiles, plan.row_token, 1, _moe_tile_width(R, E, up.shape[1]), err)
+    L.moe_gemm(mid, down, out, plan.tiles, plan.n_tiles, None, 0, _moe_tile_width(R, E, down.shape[1]), err)
+    return out
 
 
 def hgrn2(qfv, f_bias, lower, norm_w, state, state_slot, ctx_lens, cu, heads, dim, vdim, eps, spans=None):

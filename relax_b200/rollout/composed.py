@@ -319,7 +319,7 @@ class ComposedForward:
         s, p, pre = self.cfg.layer_specs[i], self.p, f"layers.{i}."
         if s.moe is None:
             return ops.linear(ops.linear_glu(h, p[pre + "gate_up"], s.act), p[pre + "down"]), None
-        plan = ops.moe_route(ops.linear_fp32(h, p[pre + "moe_router"]), s.moe)
+        plan = ops.moe_route(ops.linear_fp32(h, p[pre + "moe_router"]), s.moe, h.dtype)
         rows = ops.moe_experts(h, plan, p[pre + "moe_up"], p[pre + "moe_down"], s.moe.act)
         shared = ops.linear(ops.linear_act(h, p[pre + "shared_up"], s.moe.act), p[pre + "shared_down"]) if s.moe.shared_ff else None
         return shared, (rows, plan)
