@@ -384,7 +384,7 @@ _reg(composed_config("tiny-ketolorn", shared_kv_layers(
     160, MoESpec(experts=8, top=2, ff=48, groups=4, keep=2, shared_ff=96)), hidden_size=160, vocab_size=320, eps=1e-6, embed_norm=True,
     tie_word_embeddings=True, dtype="fp32"))
 _reg(composed_config("ketolorn-16b", shared_kv_layers(
-    24, 12, LayerSpec("attention", heads=32, dim=128, vdim=128, kv_heads=4, scale=128 ** -0.5, rot_dims=64, rot_base=5e5, qk_norm=True, sink=True,
+    24, 12, LayerSpec("attention", heads=32, dim=128, vdim=128, kv_heads=4, scale=128 ** -0.5, rot_dims=64, rot_base=1e6, qk_norm=True, sink=True,
                       act="silu"),
     8192, MoESpec(experts=128, top=8, ff=1024, groups=8, keep=4, shared_ff=2048)), hidden_size=2048, vocab_size=64000, eps=1e-6, embed_norm=True,
     tie_word_embeddings=True))

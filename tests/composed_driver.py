@@ -1,17 +1,24 @@
 """Helpers of the composed-stack tests: engines on random models, and feeding sequences in portions."""
 import torch
 
-import oracle_composed as O
+import oracle_composed
+import oracle_ketolorn
+
+
+def oracle(cfg):
+    return oracle_ketolorn if cfg.get("architecture") == "Ketolorn" else oracle_composed
 
 
 def engine(cfg, tensors, device="cpu", dtype=torch.float32, blocks=64, block_size=16, **kw):
-    from relax_b200.models import talizen
+    from relax_b200.models.architectures import architecture_of
     from relax_b200.rollout.engine import RolloutEngine
 
-    mc = talizen.config_from_dict({"architecture": "Talizen", **cfg}, dtype="fp32" if dtype == torch.float32 else "bf16")
+    full = {"architecture": "Talizen", **cfg}
+    design = architecture_of(full)
+    mc = design.config_from_dict(full, dtype="fp32" if dtype == torch.float32 else "bf16")
     eng = RolloutEngine(mc, device=device, dtype=dtype, num_kv_blocks=blocks, block_size=block_size, memory_saver=False,
                         **{"state_slots": 4, "use_cuda_graph": False, **kw})
-    talizen.load_tensors(mc, tensors, eng.weights)
+    design.load_tensors(mc, tensors, eng.weights)
     return eng
 
 
@@ -72,5 +79,5 @@ def all_free(eng):
 def greedy(cfg, tensors, prompt, n):
     seq = list(prompt)
     for _ in range(n):
-        seq.append(int(O.model(cfg, tensors, seq)[-1].argmax()))
+        seq.append(int(oracle(cfg).model(cfg, tensors, seq)[-1].argmax()))
     return seq[len(prompt):]
