@@ -78,6 +78,7 @@ def parse():
     ap.add_argument("--stack-bench", choices=["1b", "5b"], default=None,
                     help="instead of the headline workload: serving kernels and engine throughput of a composed stack (Talizen) "
                          "beside the engine's existing models at the same layer sizes (1 GPU; plain-text table)")
+    ap.add_argument("--stack-design", choices=["talizen", "ketolorn"], default="talizen", help="design that --stack-bench measures")
     return ap.parse_args()
 
 
@@ -144,7 +145,7 @@ def main():
     if args.stack_bench:
         from relax_b200.rollout.bench_stack import main as stack_bench
 
-        return stack_bench(args.stack_bench, os.path.join(ROOT, "MEASURED_PEAKS.json"))
+        return stack_bench(args.stack_bench, os.path.join(ROOT, "MEASURED_PEAKS.json"), design=args.stack_design)
     os.environ.setdefault("PYTORCH_CUDA_ALLOC_CONF", "expandable_segments:True")
     if os.environ.get("RELAX_B200_HANG_DUMP_S"):
         # debugging aid: print every thread's Python stack and exit if the run is still going after this many seconds

@@ -177,7 +177,7 @@ int rb_relu2(void* x, long long n, int fp32, cudaStream_t st);
 int rb_moe_simt(const void* A, const void* B, void* C, const int* tiles, const int* n_tiles, const int* row_token, int capacity, int cap, int N, int K,
                 int act, int fp32, cudaStream_t st);
 int rb_moe_gemm(const void* X, const void* W, void* out, const int* tiles, const int* n_tiles, const int* row_token, int x_rows, int capacity,
-                int cap, int E, int N, int K, int act, int bn, int* err, cudaStream_t st);
+                int cap, int E, int N, int K, int act, int bn, int full, int* err, cudaStream_t st);
 #ifdef __cplusplus
 }
 #endif

@@ -420,7 +420,7 @@ void moe_route(torch::Tensor logits, torch::Tensor expert, torch::Tensor weight,
 }
 // out[sorted row] = act(x[its token, or the sorted row] * W[expert]^T); act: 0 none, 1 squared relu
 void moe_gemm(torch::Tensor x, torch::Tensor W, torch::Tensor out, torch::Tensor tiles, torch::Tensor n_tiles, c10::optional<torch::Tensor> row_token,
-              int64_t act, int64_t bn, torch::Tensor err) {
+              int64_t act, int64_t bn, bool full, torch::Tensor err) {
   const c10::cuda::CUDAGuard guard(x.device());
   check_same(x, W, "moe_gemm");
   check_same(x, out, "moe_gemm");
@@ -436,7 +436,7 @@ void moe_gemm(torch::Tensor x, torch::Tensor W, torch::Tensor out, torch::Tensor
     return;
   }
   check(rb_moe_gemm(x.data_ptr(), W.data_ptr(), out.data_ptr(), tiles.data_ptr<int>(), n_tiles.data_ptr<int>(), optint(row_token), (int)x.size(0),
-                    (int)x.size(0), cap, (int)E, (int)N, (int)K, (int)act, (int)bn, err.data_ptr<int>(), cur_stream()),
+                    (int)x.size(0), cap, (int)E, (int)N, (int)K, (int)act, (int)bn, full, err.data_ptr<int>(), cur_stream()),
         "rb_moe_gemm");
 }
 void relu2(torch::Tensor x) {

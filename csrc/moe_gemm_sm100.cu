@@ -19,11 +19,15 @@ namespace mg {
 constexpr int BM = 128;
 constexpr int BK = 64;
 constexpr int THREADS = 192;
+constexpr int COPIERS = 128;                   // threads of the row copies (kCopy)
+constexpr int LAG = 2;                         // stages whose row copies are in flight behind the newest one
 constexpr int kABytes = BM * BK * 2;
+enum : int { kSorted = 0, kGather4 = 1, kCopy = 2 };      // source of the A rows
 
 template <int BN>
 struct Cfg {
-  static constexpr int kStages = BN == 256 ? 4 : (BN == 128 ? 6 : 8);
+  static constexpr int kStages = BN == 256 ? 4 : 6;
+  static_assert(kStages > LAG, "the copiers arrive LAG stages late");
   static constexpr int kBBytes = BN * BK * 2;
   static constexpr int kStage = kABytes + kBBytes;
   static constexpr int kBar = kStages * kStage;
@@ -36,6 +40,7 @@ struct Params {
   const int* n_tiles;        // device counter
   const int* row_token;      // [E][capacity] token of an expert's rows; null: the sorted rows themselves
   int capacity, cap, N, K, act;
+  const __nv_bfloat16* x;    // [x_rows][K] (kCopy)
   __nv_bfloat16* out;        // [sorted rows][N]
   int* err;
 };
@@ -47,9 +52,15 @@ __device__ __forceinline__ void tma_gather4(void* dst, const CUtensorMap* m, uin
       : "memory");
 }
 
-// kGather: token rows by index (a box of one row); else 128 sorted rows per box
-template <int BN, bool kGather>
-__global__ void __launch_bounds__(THREADS, 1)
+__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
+}
+__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+
+template <int BN, int SRC>
+__global__ void __launch_bounds__(SRC == kCopy ? THREADS + COPIERS : THREADS, 1)
 moe_gemm_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constant__ CUtensorMap tma_b, const Params p) {
   using C = Cfg<BN>;
   constexpr int kStages = C::kStages;
@@ -68,7 +79,7 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constant
   const int k_iters = p.K / BK;
 
   if (threadIdx.x == 0) {
-    for (int s = 0; s < kStages; ++s) { mbar_init(&full_bar[s], 1); mbar_init(&empty_bar[s], 1); }
+    for (int s = 0; s < kStages; ++s) { mbar_init(&full_bar[s], SRC == kCopy ? 1 + COPIERS : 1); mbar_init(&empty_bar[s], 1); }
     for (int a = 0; a < 2; ++a) { mbar_init(&tfull_bar[a], 1); mbar_init(&tempty_bar[a], 4); }
     *abort_flag = 0;
     fence_barrier_init();
@@ -83,9 +94,9 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constant
   const uint32_t tmem_base = *tmem_slot;
 
   if (warp == 0) {
-    // ------------------------------------------------------------------ TMA producer (gather: the whole warp)
+    // ------------------------------------------------------------------ TMA producer (gather4: the whole warp)
     if (lane == 0) {
-      tma_prefetch_desc(&tma_a);
+      if constexpr (SRC != kCopy) tma_prefetch_desc(&tma_a);
       tma_prefetch_desc(&tma_b);
     }
     int s = 0;
@@ -96,7 +107,7 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constant
       const int4 tile = p.tiles[m];
       int4 src = make_int4(0, 0, 0, 0);
       const int quads = (tile.z + 3) >> 2;
-      if constexpr (kGather) {
+      if constexpr (SRC == kGather4) {
         // lane l brings rows 4 l .. 4 l + 3; behind the last row of the tile its token is repeated
         const int* tok = p.row_token + static_cast<long long>(tile.x) * p.capacity + tile.w * BM;
         const int last = tile.z - 1;
@@ -107,11 +118,11 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constant
         if (!__all_sync(0xffffffffu, ok)) { ok = false; break; }
         uint8_t* sa = smem + s * C::kStage;
         if (lane == 0) {
-          mbar_expect_tx(&full_bar[s], (kGather ? quads * 512 : kABytes) + C::kBBytes);
+          mbar_expect_tx(&full_bar[s], (SRC == kGather4 ? quads * 512 : (SRC == kSorted ? kABytes : 0)) + C::kBBytes);
           tma_load_2d(sa + kABytes, &tma_b, &full_bar[s], k * BK, tile.x * p.N + n0);
-          if constexpr (!kGather) tma_load_2d(sa, &tma_a, &full_bar[s], k * BK, tile.y);
+          if constexpr (SRC == kSorted) tma_load_2d(sa, &tma_a, &full_bar[s], k * BK, tile.y);
         }
-        if constexpr (kGather) {
+        if constexpr (SRC == kGather4) {
           __syncwarp();
           if (lane < quads) tma_gather4(sa + lane * 512, &tma_a, &full_bar[s], k * BK, src);
         }
@@ -146,6 +157,47 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constant
         acc ^= 1;
         if (acc == 0) acc_ph ^= 1;
       }
+    }
+  } else if (SRC == kCopy && warp >= 6) {
+    // ------------------------------------------------------------------ row copies: eight threads bring 128 bytes of one row
+    const int i = threadIdx.x - THREADS, c = i & 7, r0 = i >> 3;
+    const uint32_t sbase = smem_u32(smem);
+    int s = 0, done = 0;
+    uint32_t ph = 0;
+    int pending = 0;
+    bool ok = true;
+    for (int t = blockIdx.x; t < total && ok; t += gridDim.x) {
+      const int4 tile = p.tiles[t / tiles_n];
+      const int* tok = p.row_token + static_cast<long long>(tile.x) * p.capacity + tile.w * BM;
+      const __nv_bfloat16* src[BM / 16];
+#pragma unroll
+      for (int j = 0; j < BM / 16; ++j) {
+        const int r = r0 + 16 * j;
+        src[j] = r < tile.z ? p.x + static_cast<long long>(tok[r]) * p.K + c * 8 : nullptr;
+      }
+      for (int k = 0; k < k_iters; ++k) {
+        if (!mbar_wait(&empty_bar[s], ph ^ 1, abort_flag, p.err)) { ok = false; break; }
+        const uint32_t sa = sbase + s * C::kStage + ((c ^ (r0 & 7)) << 4);      // rows 16 apart share the swizzle
+#pragma unroll
+        for (int j = 0; j < BM / 16; ++j)
+          if (src[j]) cp_async16(sa + (r0 + 16 * j) * 128, src[j] + k * BK);
+        cp_async_commit();
+        if (pending == LAG) {          // the stage LAG behind has landed: hand it to the tensor core's proxy
+          cp_async_wait<LAG>();
+          fence_proxy_async();
+          mbar_arrive(&full_bar[done]);
+          if (++done == kStages) done = 0;
+        } else {
+          ++pending;
+        }
+        if (++s == kStages) { s = 0; ph ^= 1; }
+      }
+    }
+    cp_async_wait<0>();
+    fence_proxy_async();
+    for (; pending > 0; --pending) {
+      mbar_arrive(&full_bar[done]);
+      if (++done == kStages) done = 0;
     }
   } else {
     // ------------------------------------------------------------------ epilogue (warps 2..5)
@@ -207,15 +259,15 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constant
   }
 }
 
-template <int BN, bool kGather>
+template <int BN, int SRC>
 static int launch(const void* X, int x_rows, const void* W, int E, const Params& p, cudaStream_t st) {
   using C = Cfg<BN>;
   CUtensorMap ta, tb;
-  int rc = encode_tma_2d_bf16(&ta, X, p.K, x_rows, p.K, BK, kGather ? 1 : BM);
+  int rc = encode_tma_2d_bf16(&ta, X, p.K, x_rows, p.K, BK, SRC == kGather4 ? 1 : BM);
   if (rc) return rc;
   rc = encode_tma_2d_bf16(&tb, W, p.K, static_cast<uint64_t>(E) * p.N, p.K, BK, BN);
   if (rc) return rc;
-  auto kern = moe_gemm_kernel<BN, kGather>;
+  auto kern = moe_gemm_kernel<BN, SRC>;
   static bool attr = false;
   if (!attr) {
     const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, C::kTotal);
@@ -223,7 +275,7 @@ static int launch(const void* X, int x_rows, const void* W, int E, const Params&
     attr = true;
   }
   const long long work = static_cast<long long>(p.cap) * ((p.N + BN - 1) / BN);
-  kern<<<static_cast<unsigned>(work < num_sms() ? work : num_sms()), THREADS, C::kTotal, st>>>(ta, tb, p);
+  kern<<<static_cast<unsigned>(work < num_sms() ? work : num_sms()), SRC == kCopy ? THREADS + COPIERS : THREADS, C::kTotal, st>>>(ta, tb, p);
   rb_note_launch(1);
   return static_cast<int>(cudaGetLastError());
 }
@@ -232,20 +284,16 @@ static int launch(const void* X, int x_rows, const void* W, int E, const Params&
 }  // namespace rb
 
 // X [x_rows][K] (token rows with row_token [E][capacity], else sorted rows), W [E][N][K] -> out [sorted rows][N]; tiles hold at most
-// `cap` entries.  act: 0 none, 1 squared relu.  bn: 64, 128 or 256 columns per tile.  N and K are multiples of 64.
+// `cap` entries.  act: 0 none, 1 squared relu.  bn: 128 or 256 columns per tile.  full: most tiles have many rows (choice of the
+// gather only).  N and K are multiples of 64.
 extern "C" int rb_moe_gemm(const void* X, const void* W, void* out, const int* tiles, const int* n_tiles, const int* row_token, int x_rows,
-                           int capacity, int cap, int E, int N, int K, int act, int bn, int* err, cudaStream_t st) {
+                           int capacity, int cap, int E, int N, int K, int act, int bn, int full, int* err, cudaStream_t st) {
   using namespace rb;
   using namespace rb::mg;
   if (x_rows <= 0 || cap <= 0) return 0;
-  if (E < 1 || N < 64 || K < 64 || N % 64 || K % 64 || act < 0 || act > 1) return -2;
-  Params p{reinterpret_cast<const int4*>(tiles), n_tiles, row_token, capacity, cap, N, K, act, (__nv_bfloat16*)out, err};
-  if (row_token) {
-    if (bn == 256) return launch<256, true>(X, x_rows, W, E, p, st);
-    if (bn == 128) return launch<128, true>(X, x_rows, W, E, p, st);
-    return launch<64, true>(X, x_rows, W, E, p, st);
-  }
-  if (bn == 256) return launch<256, false>(X, x_rows, W, E, p, st);
-  if (bn == 128) return launch<128, false>(X, x_rows, W, E, p, st);
-  return launch<64, false>(X, x_rows, W, E, p, st);
+  if (E < 1 || N < 64 || K < 64 || N % 64 || K % 64 || act < 0 || act > 1 || reinterpret_cast<uintptr_t>(X) % 16) return -2;
+  Params p{reinterpret_cast<const int4*>(tiles), n_tiles, row_token, capacity, cap, N, K, act, (const __nv_bfloat16*)X, (__nv_bfloat16*)out, err};
+  if (row_token && full) return bn == 256 ? launch<256, kCopy>(X, x_rows, W, E, p, st) : launch<128, kCopy>(X, x_rows, W, E, p, st);
+  if (row_token) return bn == 256 ? launch<256, kGather4>(X, x_rows, W, E, p, st) : launch<128, kGather4>(X, x_rows, W, E, p, st);
+  return bn == 256 ? launch<256, kSorted>(X, x_rows, W, E, p, st) : launch<128, kSorted>(X, x_rows, W, E, p, st);
 }

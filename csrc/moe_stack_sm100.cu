@@ -20,18 +20,16 @@ struct RouteParams {
 };
 constexpr int RT_WARPS = 8;
 
-// index of the largest of x[0 .. n), the first one among equals; every lane returns it
+// index of the largest of x[0 .. n), the first one among equals; every lane returns it.  Scores are not negative, so their bits
+// order like integers; what is negative is taken already or not open.
 __device__ __forceinline__ int warp_argmax(const float* x, int n, int lane) {
-  float best = -2.f;
-  int at = n;
-  for (int i = lane; i < n; i += 32)
-    if (x[i] > best) { best = x[i]; at = i; }
-#pragma unroll
-  for (int o = 16; o > 0; o >>= 1) {
-    const float b = __shfl_xor_sync(0xffffffffu, best, o);
-    const int a = __shfl_xor_sync(0xffffffffu, at, o);
-    if (b > best || (b == best && a < at)) { best = b; at = a; }
+  int best = -1, at = n;
+  for (int i = lane; i < n; i += 32) {
+    const int b = __float_as_int(x[i]);
+    if (b > best) { best = b; at = i; }
   }
+  const int top = __reduce_max_sync(0xffffffffu, best);
+  at = __reduce_min_sync(0xffffffffu, best == top ? at : n);
   return at < n ? at : 0;
 }
 
@@ -39,7 +37,7 @@ __device__ __forceinline__ int warp_argmax(const float* x, int n, int lane) {
 __global__ void __launch_bounds__(RT_WARPS * 32) moe_route_kernel(const RouteParams p) {
   extern __shared__ float sm[];                 // [warps][E + groups]
   __shared__ int s_last;
-  __shared__ int s_sum[2][RT_WARPS * 32];
+  __shared__ int s_sum[2][RT_WARPS];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const long long t = static_cast<long long>(blockIdx.x) * RT_WARPS + warp;
   float* sc = sm + warp * (p.E + p.groups);
@@ -54,6 +52,7 @@ __global__ void __launch_bounds__(RT_WARPS * 32) moe_route_kernel(const RoutePar
     if (p.keep < p.groups) {
       for (int g = lane; g < p.groups; g += 32) {      // a group counts with its two best scores
         float a = 0.f, b = 0.f;
+#pragma unroll 4
         for (int i = 0; i < n; ++i) {
           const float s = sc[g * n + i];
           if (s > a) { b = a; a = s; }
@@ -65,7 +64,7 @@ __global__ void __launch_bounds__(RT_WARPS * 32) moe_route_kernel(const RoutePar
       for (int k = 0; k < p.keep; ++k) {
         const int g = warp_argmax(gs, p.groups, lane);
         __syncwarp();
-        if (lane == 0) gs[g] = -3.f;             // taken: below what warp_argmax accepts
+        if (lane == 0) gs[g] = -3.f;             // taken
         __syncwarp();
       }
       for (int e = lane; e < p.E; e += 32)
@@ -99,13 +98,15 @@ __global__ void __launch_bounds__(RT_WARPS * 32) moe_route_kernel(const RoutePar
     __threadfence();
   }
   __syncthreads();
-  if (threadIdx.x == 0) {
+  if (gridDim.x > 1) {
+    if (threadIdx.x == 0) {
+      __threadfence();
+      s_last = atomicAdd(p.count + p.E, 1) == static_cast<int>(gridDim.x) - 1;
+    }
+    __syncthreads();
+    if (!s_last) return;
     __threadfence();
-    s_last = atomicAdd(p.count + p.E, 1) == static_cast<int>(gridDim.x) - 1;
   }
-  __syncthreads();
-  if (!s_last) return;
-  __threadfence();
   // ---- rows and tiles in front of every expert: each thread takes a run of experts
   const int per = (p.E + RT_WARPS * 32 - 1) / (RT_WARPS * 32);
   const int e0 = min(p.E, static_cast<int>(threadIdx.x) * per), e1 = min(p.E, e0 + per);
@@ -115,27 +116,27 @@ __global__ void __launch_bounds__(RT_WARPS * 32) moe_route_kernel(const RoutePar
     rows += c;
     tiles += (c + p.tile_rows - 1) / p.tile_rows;
   }
-  s_sum[0][threadIdx.x] = rows;
-  s_sum[1][threadIdx.x] = tiles;
-  __syncthreads();
-  for (int o = 1; o < RT_WARPS * 32; o <<= 1) {
-    const int a = threadIdx.x >= o ? s_sum[0][threadIdx.x - o] : 0, b = threadIdx.x >= o ? s_sum[1][threadIdx.x - o] : 0;
-    __syncthreads();
-    s_sum[0][threadIdx.x] += a;
-    s_sum[1][threadIdx.x] += b;
-    __syncthreads();
+  int row = rows, tile = tiles;                  // inclusive sums over the warp, then over the warps
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) {
+    const int a = __shfl_up_sync(0xffffffffu, row, o), b = __shfl_up_sync(0xffffffffu, tile, o);
+    if (lane >= o) { row += a; tile += b; }
   }
-  int row = s_sum[0][threadIdx.x] - rows, tile = s_sum[1][threadIdx.x] - tiles;
+  if (lane == 31) { s_sum[0][warp] = row; s_sum[1][warp] = tile; }
+  __syncthreads();
+  for (int w = 0; w < warp; ++w) { row += s_sum[0][w]; tile += s_sum[1][w]; }
+  if (threadIdx.x == RT_WARPS * 32 - 1) {
+    p.offset[p.E] = row;
+    *p.n_tiles = tile;
+  }
+  row -= rows;
+  tile -= tiles;
   for (int e = e0; e < e1; ++e) {
     const int c = __ldcg(p.count + e);
     p.offset[e] = row;
     for (int i = 0; i * p.tile_rows < c; ++i, ++tile)
       if (tile < p.cap) p.tiles[tile] = make_int4(e, row + i * p.tile_rows, min(p.tile_rows, c - i * p.tile_rows), i);
     row += c;
-  }
-  if (threadIdx.x == RT_WARPS * 32 - 1) {
-    p.offset[p.E] = s_sum[0][threadIdx.x];
-    *p.n_tiles = s_sum[1][threadIdx.x];
   }
 }
 

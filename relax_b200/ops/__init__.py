@@ -102,10 +102,17 @@ def paged_attention(q, k_pool, v_pool, batch, block_size, scale, sink, out_width
     return ref.paged_attention(q, k_pool, v_pool, batch.block_tables, block_size, batch.ctx, batch.cu, scale, sink, out_width)
 
 
-def moe_route(logits, spec, dtype):
-    """Expert choice of every row (:class:`relax_b200.models.config.MoESpec`) from fp32 logits; ``dtype``: of the experts' operands."""
+def route_counters(layers: int, experts: int, device):
+    """Zeroed counters for ``layers`` calls of :func:`moe_route` with up to ``experts`` experts (one memset per forward)."""
+    on_gpu = torch.device(device).type == "cuda" and not _force_ref()
+    return _cuda().route_counters(layers, experts, device) if on_gpu else [None] * layers
+
+
+def moe_route(logits, spec, dtype, count=None):
+    """Expert choice of every row (:class:`relax_b200.models.config.MoESpec`) from fp32 logits; ``dtype``: of the experts' operands;
+    ``count``: an unused row of :func:`route_counters`."""
     if _use_cuda(logits):
-        return _cuda().moe_route(logits, spec, 64 if dtype == torch.float32 else 128)      # rows per tile of the grouped GEMM
+        return _cuda().moe_route(logits, spec, 64 if dtype == torch.float32 else 128, count)      # rows per tile of the grouped GEMM
     return ref.moe_route(logits, spec)
 
 

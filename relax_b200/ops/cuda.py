@@ -407,26 +407,28 @@ class ExpertPlan:
     __slots__ = ("expert", "weight", "place", "row_token", "offset", "tiles", "n_tiles")
 
 
-def moe_route(logits, spec, tile_rows):
+def route_counters(layers, experts, device):
+    return torch.zeros(layers, experts + 1, dtype=torch.int32, device=device)
+
+
+def moe_route(logits, spec, tile_rows, count=None):
     T, E, k, dev = logits.shape[0], spec.experts, spec.top, logits.device
     p = ExpertPlan()
     i32 = lambda *s: torch.empty(*s, dtype=torch.int32, device=dev)
     p.expert, p.place, p.row_token, p.offset, p.n_tiles = i32(T, k), i32(T, k), i32(E, T), i32(E + 1), i32(1)
     p.weight = torch.empty(T, k, dtype=torch.float32, device=dev)
     p.tiles = i32(min(T * k, E) + T * k // tile_rows, 4)
-    count = torch.zeros(E + 1, dtype=torch.int32, device=dev)
+    if count is None:
+        count = route_counters(1, E, dev)[0]
     _load().moe_route(logits, p.expert, p.weight, p.place, p.row_token, count, p.offset, p.tiles, p.n_tiles, E, spec.groups, spec.keep, tile_rows,
                       bool(spec.renormalize), float(spec.weight_scale))
     return p
 
 
-def _moe_tile_width(rows: int, experts: int, n: int) -> int:
-    """Columns per tile: wide ones when every expert has full row tiles, narrow ones while they would leave SMs idle."""
+def _moe_plan(rows: int, experts: int, n: int) -> tuple:
+    """``(columns per tile, whether most tiles have many rows)``: wide tiles when they fill the machine twice (measured)."""
     tiles = min(rows, experts) + rows // 128
-    for bn in (256, 128):
-        if tiles * ((n + bn - 1) // bn) >= (296 if bn == 256 else 148) and (bn == 128 or rows >= 64 * experts):
-            return bn
-    return 64
+    return (256 if tiles * ((n + 255) // 256) >= 296 else 128), rows >= 16 * experts
 
 
 def moe_experts(h, plan, up, down, act):
@@ -437,8 +439,8 @@ def moe_experts(h, plan, up, down, act):
     mid = torch.empty(R, up.shape[1], dtype=h.dtype, device=h.device)
     out = torch.empty(R, down.shape[1], dtype=h.dtype, device=h.device)
     L = _load()
-    L.moe_gemm(h, up, mid, plan.tiles, plan.n_tiles, plan.row_token, 1, _moe_tile_width(R, E, up.shape[1]), err)
-    L.moe_gemm(mid, down, out, plan.tiles, plan.n_tiles, None, 0, _moe_tile_width(R, E, down.shape[1]), err)
+    L.moe_gemm(h, up, mid, plan.tiles, plan.n_tiles, plan.row_token, 1, *_moe_plan(R, E, up.shape[1]), err)
+    L.moe_gemm(mid, down, out, plan.tiles, plan.n_tiles, None, 0, *_moe_plan(R, E, down.shape[1]), err)
     return out
 
 

@@ -4,8 +4,9 @@ Two tables, random weights, bf16, one GPU:
 
 * kernels: device time per launch, algorithmic bytes or FLOPs, fraction of the measured copy bandwidth / cuBLAS rate
   (``--peaks``), each kernel of the composed stack beside the like kernel of the existing models;
-* models: prefill and decode tokens/s through the engine's scheduler - a Talizen stack, the Gated-DeltaNet hybrid and
-  the dense softmax model with the same width, heads, feed-forward and depth.
+* models: prefill and decode tokens/s through the engine's scheduler - a Talizen stack beside the Gated-DeltaNet hybrid and
+  the dense softmax model, or a Ketolorn stack beside the mixture-of-experts model, with the same width, heads,
+  feed-forward bytes and depth.
 
 Times come from CUDA events after warm-up; every kernel rotates through inputs larger than the L2 cache.
 """
@@ -137,6 +138,131 @@ def kernel_rows(H=32, d=128, R=512, W=4096, F=12288, groups=8, only=""):
     return rows
 
 
+@torch.no_grad()
+def ketolorn_kernel_rows(W=2048, H=32, G=4, d=128, E=128, k=8, F=1152, only=""):
+    """The kernels of one real-sized Ketolorn layer, each beside the like kernel of the existing models."""
+    from .. import ops
+    from ..models.config import LayerSpec, MoESpec
+    from .composed import SegmentBatch, query_blocks, tile_tokens
+
+    dev, bf = "cuda", torch.bfloat16
+    rows = []
+    mk = lambda *s: torch.randn(*s, device=dev).to(bf)
+    i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
+    want = lambda section: not only or section in only.split(",")
+    sink, scale = mk(H), d ** -0.5
+    for B in (16, 128) if want("attn") else ():
+        for L in (2048, 8192):
+            nbytes = B * L * G * d * 4
+            cl = torch.full((B,), L, dtype=torch.int32, device=dev)
+            for page, like in ((64, False), (16, True)):
+                bt = torch.randperm(B * L // page, device=dev).to(torch.int32).view(B, L // page)
+                fns = []
+                for _ in range(_copies(nbytes)):
+                    kc, vc, q = mk(B * L, G, d), mk(B * L, G, d), mk(B, H, d)
+                    if like:
+                        kv = kc.view(-1, page, G, d), vc.view(-1, page, G, d)
+                        fns.append(_graph(lambda q=q, kv=kv: ops.paged_decode_attention(q, *kv, bt, cl)))
+                    else:
+                        b = SegmentBatch(None, None, cl, bt, None, max_ctx_one=L)
+                        fns.append(_graph(lambda q=q, kc=kc, vc=vc, b=b: ops.paged_attention(q, kc, vc, b, page, scale, sink, d)))
+                rows.append(("  like: paged decode attention" if like else "attention decode + sink", f"batch {B}, context {L}, pages of {page}", _time(fns), nbytes, None))
+                del fns, kc, vc, q
+    spec = LayerSpec("attention", heads=H, dim=d, vdim=d, kv_heads=G)
+    for S, n, L in ((1, 8192, 8192), (4, 2048, 2048), (32, 256, 256), (16, 64, 2048), (16, 4, 2048)) if want("prompt") else ():
+        T, page = S * n, 64
+        nb = L // page
+        bt = torch.randperm(S * nb, device=dev).to(torch.int32).view(S, nb)
+        q, kc, vc = mk(T, H, d), mk(S * L, G, d), mk(S * L, G, d)
+        t = tile_tokens(spec)
+        b = SegmentBatch(None, None, i32([L] * S), bt, None, cu=i32([i * n for i in range(S + 1)]), multi_segs=S, multi_rows=T,
+                         blocks={t: i32(query_blocks([n] * S, [L] * S, t))})
+        flops = 4.0 * S * H * d * sum(L - n + i + 1 for i in range(n))
+        rows.append(("paged flash + sink", f"{S} x {n} tokens, context {L}", _time([_graph(lambda: ops.paged_attention(q, kc, vc, b, page, scale, sink, d))], 10),
+                     T * H * d * 4 + S * L * G * d * 4, flops))
+        cq, ck = i32([i * n for i in range(S + 1)]), i32([i * L for i in range(S + 1)])
+        rows.append(("  like: flash attention", f"{S} x {n} tokens, context {L}", _time([_graph(lambda: ops.attention_varlen(q, kc, vc, cq, True, scale, ck, n))], 10),
+                     T * H * d * 4 + S * L * G * d * 4, flops))
+    for T in (128, 8192) if want("prep") else ():
+        n = _copies(T * (H + 2 * G) * d * 4)
+        freq = torch.tensor([1e6 ** (-2 * i / 64) for i in range(32)], dtype=torch.float64, device=dev)
+        pos, slots = torch.arange(T, device=dev).to(torch.int32), torch.randperm(T, device=dev)
+        tab, kp, vp = ops.rope_table(pos, 0, freq), mk(T, G, d), mk(T, G, d)
+        xs = [mk(T, (H + 2 * G) * d) for _ in range(n)]
+        nb = T * (H + 2 * G) * d * 4
+        rows.append(("rotation + norm + cache write", f"{T} rows", _time([_graph(lambda x=x: ops.attention_inputs(x, tab, H, G, d, d, d, 64, 1e-6, kp, vp, slots)) for x in xs]), nb, None))
+        cos, sin = torch.randn(T, d // 2, device=dev), torch.randn(T, d // 2, device=dev)
+        qw, kc, vc = mk(d), kp.view(-1, 16, G, d), vp.view(-1, 16, G, d)
+        rows.append(("  like: qkv_post", f"{T} rows", _time([_graph(lambda x=x: ops.qkv_post(x, H, G, qw, qw, cos, sin, 1e-6, kc, vc, slots, False)) for x in xs]), nb, None))
+        rows.append(("rope_table (once per forward)", f"{T} rows", _time([_graph(lambda: ops.rope_table(pos, 0, freq))]), T * 32 * 8, None))
+        del xs
+    moe = MoESpec(experts=E, top=k, ff=F, groups=8, keep=4)
+    for T in (1, 16, 128, 8192) if want("moe") else ():
+        R, h = T * k, mk(T, W)
+        up, down = mk(E, F, W), mk(E, W, F)
+        plans = [ops.moe_route(torch.randn(T, E, device=dev), moe, bf) for _ in range(1 if T > 1000 else 4)]      # each touches other experts
+        hit = [int((p.offset[1:] > p.offset[:-1]).sum()) for p in plans]
+        nb, fl = sum(hit) / len(hit) * 2 * F * W * 2 + R * (2 * W + 2 * F) * 2, 4.0 * R * F * W
+        rows.append(("expert products (gather, up, relu^2, down)", f"{T} rows", _time([_graph(lambda p=p: ops.moe_experts(h, p, up, down, "relu2")) for p in plans], 10), nb, fl if T > 1000 else None))
+        from ..models.moe import grouped_swiglu_mlp
+
+        w1, w2 = mk(E, 2 * 768, W), mk(E, W, 768)
+        sorts = [torch.rand(T, E, device=dev).topk(k, -1).indices for _ in range(len(plans))]
+        hit = [x.unique().numel() for x in sorts]
+        nb2, fl2 = sum(hit) / len(hit) * 3 * 768 * W * 2 + R * (2 * W + 3 * 768) * 2, 6.0 * R * 768 * W
+        rows.append(("  like: grouped SwiGLU experts with their permutation", f"{T} rows",
+                     _time([_graph(lambda i=i: grouped_swiglu_mlp(h.repeat_interleave(k, 0), i.reshape(-1), w1, w2)) for i in sorts], 10), nb2, fl2 if T > 1000 else None))
+        if T > 1000:      # the products alone: rows laid out beforehand
+            cap = R // E // 128 * 128 * E
+            x, te = mk(cap, W), torch.arange(E, device=dev).to(torch.int32).repeat_interleave(cap // E // 128)
+            er = (torch.arange(E + 1, device=dev) * (cap // E)).to(torch.int32)
+            rows.append(("  like: grouped GEMM alone", f"{cap} sorted rows", _time([_graph(lambda: ops.grouped_linear(x, w1, te, er))], 10), cap * (W + 1536) * 2 + E * 1536 * W * 2, 2.0 * cap * 1536 * W))
+            y = mk(cap, 768)
+            rows.append(("  like: grouped GEMM alone (down)", f"{cap} sorted rows", _time([_graph(lambda: ops.grouped_linear(y, w2, te, er))], 10), cap * (W + 768) * 2 + E * 768 * W * 2, 2.0 * cap * 768 * W))
+        z = torch.randn(T, E, device=dev)
+        rows.append(("routing and layout of the experts' rows", f"{T} rows", _time([_graph(lambda: ops.moe_route(z, moe, bf))]), T * E * 4 + R * 16, None))
+        rows.append(("  like: softmax top-k", f"{T} rows", _time([_graph(lambda: ops.topk_router(z, k))]), T * E * 8 + R * 12, None))
+        from ..models.moe import padded_expert_layout
+
+        rows.append(("  like: softmax top-k and padded_expert_layout", f"{T} rows",
+                     _time([_graph(lambda: padded_expert_layout(ops.topk_router(z, k)[1].reshape(-1), E))]), T * E * 8 + R * 28, None))
+        wr = mk(E, W)
+        rows.append(("router logits (fp32)", f"{T} rows", _time([_graph(lambda: ops.linear_fp32(h, wr))]), T * W * 2 + E * W * 2 + T * E * 4, None))
+        rows.append(("  like: GEMM of that size", f"{T} rows", _time([_graph(lambda: ops.linear(h, wr))]), T * W * 2 + E * W * 2 + T * E * 2, None))
+        del up, down, w1, w2
+    for T in (128, 8192) if want("norm") else ():
+        n = _copies(T * W * (12 + 2 * k))
+        w = mk(W)
+        plan = ops.moe_route(torch.randn(T, E, device=dev), moe, bf)
+        buf = [(torch.randn(T, W, device=dev), mk(T, W), mk(T * k, W)) for _ in range(n)]
+        rows.append(("norm_add with expert rows", f"{T} rows", _time([_graph(lambda r=r, y=y, e=e: ops.norm_add(r, y, w, W, 1, 1e-6, None, (e, plan))) for r, y, e in buf]), T * W * (12 + 2 * k), None))
+        rows.append(("norm_add", f"{T} rows", _time([_graph(lambda r=r, y=y: ops.norm_add(r, y, w, W, 1, 1e-6)) for r, y, _ in buf]), T * W * 12, None))
+        rows.append(("  like: add_rmsnorm (bf16 stream)", f"{T} rows", _time([_graph(lambda y=y, e=e: ops.add_rmsnorm(y, e[:T], w, 1e-6)) for _, y, e in buf]), T * W * 8, None))
+        del buf
+    for T in (16, 128, 8192) if want("gemm") else ():
+        x = mk(T, W)
+        wc = [mk(2 * F, W) for _ in range(_copies(2 * F * W * 2))]
+        fl = 4.0 * T * F * W if T > 1000 else None
+        rows.append(("GEMM + squared relu (shared expert)", f"{T} rows", _time([_graph(lambda w=w: ops.linear_act(x, w, "relu2")) for w in wc], 10), 2 * F * W * 2 + T * (W + 2 * F) * 2, fl))
+        rows.append(("  like: GEMM + SwiGLU", f"{T} rows", _time([_graph(lambda w=w: ops.linear_glu(x, w, "silu")) for w in wc], 10), 2 * F * W * 2 + T * (W + F) * 2, fl))
+        del wc
+    return rows
+
+
+def _ketolorn_models(layers: int, W: int, H: int, G: int, experts: int, top: int, ff: int, dense_ff: int, vocab: int):
+    """A Ketolorn stack (squared-relu experts of 3 / 2 the width: the same bytes as gated ones) and the mixture-of-experts model."""
+    from ..models.config import LayerSpec, ModelConfig, MoESpec, composed_config, shared_kv_layers
+
+    d = 128
+    att = LayerSpec("attention", heads=H, dim=d, vdim=d, kv_heads=G, scale=d ** -0.5, rot_dims=64, rot_base=1e6, qk_norm=True, sink=True, act="silu")
+    moe = MoESpec(experts=experts, top=top, ff=ff * 3 // 2, groups=8, keep=4, shared_ff=ff * 3)
+    return {"ketolorn": composed_config("ketolorn", shared_kv_layers(layers, layers // 2, att, dense_ff, moe), W, vocab, embed_norm=True, tie_word_embeddings=True),
+            "mixture of experts": ModelConfig(name="moe", num_layers=layers, hidden_size=W, num_attention_heads=H, num_query_groups=G, head_dim=d,
+                                              ffn_hidden_size=dense_ff, vocab_size=vocab, num_experts=experts, moe_top_k=top, moe_ffn_hidden_size=ff,
+                                              moe_first_dense_layers=1, moe_shared_expert_ffn=2 * ff, moe_router_score="sigmoid",
+                                              tie_word_embeddings=True)}
+
+
 def _models(layers: int, W: int, H: int, ff: int, vocab: int):
     from ..models.config import LayerSpec, ModelConfig, composed_config, talizen_layers
 
@@ -150,13 +276,16 @@ def _models(layers: int, W: int, H: int, ff: int, vocab: int):
 
 
 @torch.no_grad()
-def model_rows(size: str, only=None, decode_batches=(1, 32, 128), prompt=2048):
+def model_rows(size: str, only=None, decode_batches=(1, 32, 128), prompt=2048, design="talizen"):
     """``(model, workload, tokens/s, ms)`` through ``RolloutEngine.step``."""
     from .engine import RolloutEngine, SamplingParams
 
-    layers, W, H, ff = {"1b": (8, 2048, 16, 8192), "5b": (8, 4096, 32, 12288)}[size]
+    if design == "ketolorn":
+        models = _ketolorn_models(*{"1b": (8, 2048, 32, 4, 128, 8, 768, 6144), "5b": (8, 4096, 64, 4, 128, 8, 1536, 12288)}[size], 64000)
+    else:
+        models = _models(*{"1b": (8, 2048, 16, 8192), "5b": (8, 4096, 32, 12288)}[size], 64000)
     out = []
-    for name, cfg in _models(layers, W, H, ff, 64000).items():
+    for name, cfg in models.items():
         if only and name not in only:
             continue
         slow = name == "gdn hybrid"
@@ -202,7 +331,7 @@ def model_rows(size: str, only=None, decode_batches=(1, 32, 128), prompt=2048):
     return out
 
 
-def main(size: str = "5b", peaks: str = "MEASURED_PEAKS.json", kernels: bool = True, models: bool = True, only: str = "") -> int:
+def main(size: str = "5b", peaks: str = "MEASURED_PEAKS.json", kernels: bool = True, models: bool = True, only: str = "", design: str = "talizen") -> int:
     from ..ops import cuda as C
 
     assert C.available()
@@ -210,7 +339,7 @@ def main(size: str = "5b", peaks: str = "MEASURED_PEAKS.json", kernels: bool = T
     hbm, tf = pk.get("hbm_gbs"), pk.get("bf16_tflops")
     if kernels:
         print("kernel | case | us | GB/s (of measured copy) | TFLOP/s (of measured GEMM)")
-        for k, case, ms, nb, fl in kernel_rows(only=only):
+        for k, case, ms, nb, fl in (ketolorn_kernel_rows if design == "ketolorn" else kernel_rows)(only=only):
             gb = nb / ms / 1e6
             t = f"{gb:7.0f}" + (f" ({gb / hbm:.2f})" if hbm else "")
             if fl:
@@ -218,7 +347,7 @@ def main(size: str = "5b", peaks: str = "MEASURED_PEAKS.json", kernels: bool = T
                 t += f" | {v:7.1f}" + (f" ({v / tf:.2f})" if tf else "")
             print(f"{k} | {case} | {ms * 1e3:.1f} | {t}", flush=True)
     if models:
-        for name, what, tps, ms in model_rows(size):
+        for name, what, tps, ms in model_rows(size, design=design):
             print(f"[{size}] {name} | {what} | {tps:,.0f} tokens/s | {ms:.3f} ms", flush=True)
     C.check_error_flag()
     return 0
@@ -228,6 +357,8 @@ if __name__ == "__main__":
     import argparse
 
     ap = argparse.ArgumentParser(description="kernel table of composed stacks")
-    ap.add_argument("--only", default="", help="sections, with commas: step, attn, gemm, norm, prompt")
+    ap.add_argument("--design", choices=["talizen", "ketolorn"], default="talizen")
+    ap.add_argument("--only", default="", help="sections, with commas: step, attn, gemm, norm, prompt (talizen); attn, prompt, prep, moe, norm, gemm (ketolorn)")
     ap.add_argument("--peaks", default="MEASURED_PEAKS.json")
-    raise SystemExit(main(peaks=ap.parse_args().peaks, models=False, only=ap.parse_args().only))
+    a = ap.parse_args()
+    raise SystemExit(main(peaks=a.peaks, models=False, only=a.only, design=a.design))

@@ -314,12 +314,12 @@ class ComposedForward:
         return tables[key]
 
     # ------------------------------------------------------------------ feed-forwards
-    def _feed_forward(self, i, h):
-        """``(output rows or None, (expert rows, plan) or None)`` of layer ``i``'s feed-forward."""
+    def _feed_forward(self, i, h, count):
+        """``(output rows or None, (expert rows, plan) or None)`` of layer ``i``'s feed-forward; ``count``: the router's counters."""
         s, p, pre = self.cfg.layer_specs[i], self.p, f"layers.{i}."
         if s.moe is None:
             return ops.linear(ops.linear_glu(h, p[pre + "gate_up"], s.act), p[pre + "down"]), None
-        plan = ops.moe_route(ops.linear_fp32(h, p[pre + "moe_router"]), s.moe, h.dtype)
+        plan = ops.moe_route(ops.linear_fp32(h, p[pre + "moe_router"]), s.moe, h.dtype, count)
         rows = ops.moe_experts(h, plan, p[pre + "moe_up"], p[pre + "moe_down"], s.moe.act)
         shared = ops.linear(ops.linear_act(h, p[pre + "shared_up"], s.moe.act), p[pre + "shared_down"]) if s.moe.shared_ff else None
         return shared, (rows, plan)
@@ -331,6 +331,8 @@ class ComposedForward:
         W, G, eps = cfg.hidden_size, cfg.norm_groups, cfg.rms_norm_eps
         res, h = ops.embed_rows(b.tokens, p["embed"], p.get("embed_norm"), W, G, eps)
         tables: dict = {}
+        routed = [i for i, s in enumerate(cfg.layer_specs) if s.moe is not None]
+        counts = dict(zip(routed, ops.route_counters(len(routed), max(cfg.layer_specs[i].moe.experts for i in routed), res.device))) if routed else {}
         for i, s in enumerate(cfg.layer_specs):
             pre = f"layers.{i}."
             final = p["final_norm"] if i + 1 == cfg.num_layers else None
@@ -340,7 +342,7 @@ class ComposedForward:
                 a = self._hgrn2(i, h, b, cache) if s.mixer == "hgrn2" else self._latent(i, h, b, cache)
             h = ops.norm_add(res, a, p[pre + "post_attn_norm"], W, G, eps, None if s.has_ff else final)
             if s.has_ff:
-                m, experts = self._feed_forward(i, h)
+                m, experts = self._feed_forward(i, h, counts.get(i))
                 h = ops.norm_add(res, m, p[pre + "post_mlp_norm"], W, G, eps, final, experts)
             if taps is not None:
                 taps.append(res[:, :W].clone())

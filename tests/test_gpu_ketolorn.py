@@ -235,7 +235,7 @@ def test_router_and_layout(T, E, top, groups, keep):
 @BOTH
 @pytest.mark.parametrize("T,E,W,F", [(1, 8, 128, 64), (5, 16, 192, 128), (130, 4, 64, 320), (700, 3, 256, 192), (1000, 12, 128, 512)])
 def test_expert_products(dtype, T, E, W, F):
-    """Few rows per expert, experts without rows, and experts with several tiles of rows; every tile width."""
+    """Few rows per expert, experts without rows, and experts with several tiles of rows; every tile width and source of rows."""
     from relax_b200 import ops
     from relax_b200.models.config import MoESpec
     from relax_b200.ops import cuda as C
@@ -259,14 +259,14 @@ def test_expert_products(dtype, T, E, W, F):
         for e in range(E):
             t, j = (ex == e).nonzero(as_tuple=True)
             want[flat[t, j].long()] = O.expert(hc[t], upc[e], dc[e])
-    widths = (64, 128, 256) if dtype == BF else (0,)
-    keep = C._moe_tile_width
+    plans = [(bn, full) for bn in (128, 256) for full in (False, True)] if dtype == BF else [(128, False)]
+    keep = C._moe_plan
     try:
-        for bn in widths:
-            C._moe_tile_width = lambda *a, bn=bn: bn
+        for choice in plans:
+            C._moe_plan = lambda *a, choice=choice: choice
             _close(ops.moe_experts(h, plan, up, down, "relu2"), want, 2e-2 if dtype == BF else 1e-5)
     finally:
-        C._moe_tile_width = keep
+        C._moe_plan = keep
     _ok()
 
 
