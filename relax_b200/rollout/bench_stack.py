@@ -281,7 +281,7 @@ def model_rows(size: str, only=None, decode_batches=(1, 32, 128), prompt=2048, d
     from .engine import RolloutEngine, SamplingParams
 
     if design == "ketolorn":
-        models = _ketolorn_models(*{"1b": (8, 2048, 32, 4, 128, 8, 768, 6144), "5b": (8, 4096, 64, 4, 128, 8, 1536, 12288)}[size], 64000)
+        models = _ketolorn_models(*{"1b": (8, 2048, 32, 4, 128, 8, 768, 6144), "5b": (8, 4096, 64, 8, 128, 8, 1536, 12288)}[size], 64000)
     else:
         models = _models(*{"1b": (8, 2048, 16, 8192), "5b": (8, 4096, 32, 12288)}[size], 64000)
     out = []
