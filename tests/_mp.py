@@ -16,7 +16,7 @@ def _free_port():
     return p
 
 
-def _entry(rank, world, port, fn, args, q, backend="gloo"):
+def _entry(rank, world, port, fn, args, q, backend="gloo", received=None):
     os.environ["MASTER_ADDR"] = "127.0.0.1"
     os.environ["MASTER_PORT"] = str(port)
     torch.set_num_threads(1)
@@ -33,13 +33,15 @@ def _entry(rank, world, port, fn, args, q, backend="gloo"):
     finally:
         if dist.is_initialized():
             dist.destroy_process_group()
+    if received is not None:
+        received.wait(60)      # tensors in the result are fetched from this process: it must not leave before
 
 
 def run_distributed(fn, world, *args, timeout=300, backend="gloo"):
     ctx = mp.get_context("spawn")
-    q = ctx.Queue()
+    q, received = ctx.Queue(), ctx.Event()
     port = _free_port()
-    procs = [ctx.Process(target=_entry, args=(r, world, port, fn, args, q, backend)) for r in range(world)]
+    procs = [ctx.Process(target=_entry, args=(r, world, port, fn, args, q, backend, received)) for r in range(world)]
     for p in procs:
         p.start()
     res = {}
@@ -50,6 +52,7 @@ def run_distributed(fn, world, *args, timeout=300, backend="gloo"):
                 p.kill()
             raise RuntimeError(f"rank {rank} failed:\n{out}")
         res[rank] = out
+    received.set()
     for p in procs:
         p.join(timeout=30)
     return [res[r] for r in range(world)]
