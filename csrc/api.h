@@ -37,6 +37,12 @@ int rb_int4_fake_quant(const void* x, void* out, void* scale, void* zero, int M,
 int rb_fp8_block_cast(const void* w, void* q, float* scale, int M, int N, int block, int ue8m0, int dtype, cudaStream_t st);
 int rb_fp8_block_dequant(const void* q, const float* scale, void* out, int M, int N, int block, int dtype, cudaStream_t st);
 
+int rb_sum_norm(float* res, const void* y, const void* ex, const int* expert, const int* place, const int* offset, const float* weight, int top, int
+                experts, const void* w, const void* b, const void* next_w, const void* next_b, void* h, int rows, int ldy, int pitch, int width, int
+                centre, float alpha, float eps, float scale, int fp32, cudaStream_t st);
+int rb_projection_inputs(const void* qkv, int ld, const void* q_w, const void* k_w, const float* table, void* q, void* k_pool, void* v_pool, const
+                         long long* slots, long long pool_rows, int T, int H, int G, int dim, int vdim, int dp, int vp, int rot, int halves, float
+                         eps, int fp32, cudaStream_t st);
 #ifdef __cplusplus
 }
 #endif
@@ -130,7 +136,7 @@ int rb_lm_head_dlogits(const void* h, const void* W, const long long* targets, c
                        const float* g_ent, void* dlogits, int M, int N, int K, int ldh, int ldw, int ldd, int vocab_start,
                        float inv_temp, int* err, cudaStream_t stream);
 // ---- composed stacks (stack_sm100.cu); fp32 = 1: 32-bit operands, 0: bf16
-int rb_embed_rows(const long long* tok, const void* w, float* res, void* h, int rows, int vocab, int pitch, int fp32, cudaStream_t st);
+int rb_embed_rows(const long long* tok, const void* w, float* res, void* h, int rows, int vocab, int pitch, float scale, int fp32, cudaStream_t st);
 int rb_norm_add(float* res, const void* y, const void* w, const void* next_w, void* h, int rows, int ldy, int pitch, int width,
                 int groups, float eps, int fp32, cudaStream_t st);
 int rb_hgrn2(const void* qfv, const void* f_bias, const void* lower, const void* norm_w, float* state, const int* slot, const int* ctx,
@@ -139,45 +145,45 @@ int rb_hgrn2(const void* qfv, const void* f_bias, const void* lower, const void*
 int rb_hgrn2_chunk(const void* qfv, const void* f_bias, const void* lower, const void* norm_w, float* state, const int* slot, const int* ctx,
                    const int* cu, const int* spans, const int* first, float* span_state, float* span_gate, void* out, int rows, int segs,
                    int n_spans, int H, int dim, int vdim, int vp, int ld, int ldo, float eps, cudaStream_t st);
-int rb_latent_write(const void* raw, int ld_raw, const void* w, void* pool, const long long* slots, long long pool_rows, int rows,
-                    int rank, int pitch, float eps, int fp32, cudaStream_t st);
-int rb_latent_attn(const void* q, const void* pool, const int* block_tables, const int* row_seg, const int* row_pos, const int* ctx,
-                   const void* gate, void* out, int rows, int H, int R, int max_blocks, int block_size, int ld_gate, float scale,
-                   int fp32, cudaStream_t st);
-int rb_latent_attn_tc(const void* q, const void* pool, const int* block_tables, const int* items, const int* ctx, const void* gate,
-                      void* out, float* part_o, float* part_ml, int rows, int H, int R, long long pool_rows, int max_blocks, int page,
-                      int n_items, int width, int splits, int ld_gate, float scale, int* err, cudaStream_t st);
-int rb_head_gemm(const void* x, const void* w, void* out, int T, int H, int N, int K, long long x_tok, long long x_head, int kn, int* err,
-                 cudaStream_t st);
-int rb_gate_heads(const void* o, const void* gate, int ld_gate, void* out, int rows, int H, int dv, cudaStream_t st);
+int rb_latent_write(const void* raw, const void* k_rot, void* q, int ld, const void* w, void* pool, const long long* slots, const float* table, long
+                    long pool_rows, int rows, int rank, int pitch, int part, int rot, int H, int dk, int dim, float eps, int fp32, cudaStream_t st);
+int rb_latent_attn(const void* q, const void* pool, const int* block_tables, const int* row_seg, const int* row_pos, const int* ctx, const void* gate,
+                   void* out, int rows, int H, int R, int Rv, int max_blocks, int block_size, int ld_gate, float scale, int fp32, cudaStream_t st);
+int rb_latent_attn_tc(const void* q, const void* pool, const int* block_tables, const int* items, const int* ctx, const void* gate, void* out, float*
+                      part_o, float* part_ml, int rows, int H, int R, int Rv, long long pool_rows, int max_blocks, int page, int n_items, int width,
+                      int splits, int ld_gate, float scale, int* err, cudaStream_t st);
+int rb_head_gemm(const void* x, const void* w, const void* gate, int ld_gate, void* out, int T, int H, int N, int K, long long x_tok, long long
+                 x_head, int kn, int* err, cudaStream_t st);
+int rb_gate_heads(const void* o, const void* gate, int ld_gate, void* out, int rows, int H, int pitch, int dv, int features, int fp32, cudaStream_t
+                  st);
 int rb_glu(const void* in, void* out, long long rows, int F, int ld_in, int act, int fp32, cudaStream_t st);
 int rb_simt_gemm(const void* A, const void* B, void* C, int M, int N, int K, int lda, int ldb, int ldc, int b_kn, int batch, long long sa,
                  long long sb, long long sc, int fp32, cudaStream_t st);
-int rb_norm_add_experts(float* res, const void* y, const void* ex, const int* expert, const int* place, const int* offset, const float* weight,
-                        int top, const void* w, const void* next_w, void* h, int rows, int ldy, int pitch, int width, int groups, float eps,
+int rb_norm_add_experts(float* res, const void* y, const void* ex, const int* expert, const int* place, const int* offset, const float* weight, int
+                        top, int experts, const void* w, const void* next_w, void* h, int rows, int ldy, int pitch, int width, int groups, float eps,
                         int fp32, cudaStream_t st);
 int rb_embed_norm(const long long* tok, const void* table, const void* w, float* res, void* h, int rows, int vocab, int pitch, int width, int groups,
                   float eps, int fp32, cudaStream_t st);
 int rb_rope_table(const int* pos, int offset, const double* freq, float* out, int rows, int half, cudaStream_t st);
 int rb_attention_inputs(const void* qkv, int ld, const float* table, void* q, void* k_pool, void* v_pool, const long long* slots, long long pool_rows,
                         int T, int H, int G, int dim, int vdim, int dp, int vp, int rot, float eps, int fp32, cudaStream_t st);
-int rb_gqa_attn(const void* q, const void* k_pool, const void* v_pool, const int* block_tables, const int* row_seg, const int* row_pos, const int* ctx,
-                const void* sink, void* out, int rows, int H, int G, int dp, int vp, int vo, int max_blocks, int block_size, float scale, int fp32,
-                cudaStream_t st);
-int rb_paged_flash(const void* q, const void* kc, const void* vc, const int* block_tables, const int* ctx, const int* blocks, const void* sink,
-                   void* out, int rows, int n, int Hq, int Hkv, int dk, int dv, int out_d, long long pool_rows, int page, int max_blocks,
-                   float scale, int* err, cudaStream_t st);
-int rb_paged_decode_tc(const void* q, const void* kc, const void* vc, const int* block_tables, const int* ctx_lens, const void* sink, void* out,
-                       float* part_o, float* part_ml, int B, int Hq, int Hkv, int dk, int dv, int out_d, long long pool_rows, int page,
-                       int max_blocks, int max_ctx, float scale, int splits, int* err, cudaStream_t st);
-int rb_moe_route(const float* logits, int ld, int* expert, float* weight, int* place, int* row_token, int* count, int* offset, int* tiles,
-                 int* n_tiles, int T, int E, int groups, int keep, int top, int tile_rows, int cap, int renormalize, float weight_scale,
-                 cudaStream_t st);
+int rb_gqa_attn(const void* q, const void* k_pool, const void* v_pool, const int* block_tables, const int* row_seg, const int* row_pos, const int*
+                ctx, const void* sink, const void* gate, int ld_gate, void* out, int rows, int H, int G, int dp, int vp, int vo, int max_blocks, int
+                block_size, int window, float scale, int fp32, cudaStream_t st);
+int rb_paged_flash(const void* q, const void* kc, const void* vc, const int* block_tables, const int* ctx, const int* blocks, const void* sink, const
+                   void* gate, int ld_gate, void* out, int rows, int n, int Hq, int Hkv, int dk, int dv, int out_d, long long pool_rows, int page, int
+                   max_blocks, int window, float scale, int* err, cudaStream_t st);
+int rb_paged_decode_tc(const void* q, const void* kc, const void* vc, const int* block_tables, const int* ctx_lens, const void* sink, const void*
+                       gate, int ld_gate, void* out, float* part_o, float* part_ml, int B, int Hq, int Hkv, int dk, int dv, int out_d, long long
+                       pool_rows, int page, int max_blocks, int max_ctx, int window, float scale, int splits, int* err, cudaStream_t st);
+int rb_moe_route(const float* logits, int ld, const void* correction, int corr_fp32, int* expert, float* weight, int* place, int* row_token, int*
+                 count, int* offset, int* tiles, int* n_tiles, int T, int E, int N, int groups, int keep, int group_best, int top, int tile_rows, int
+                 cap, int renormalize, int softmax, float weight_scale, cudaStream_t st);
 int rb_relu2(void* x, long long n, int fp32, cudaStream_t st);
-int rb_moe_simt(const void* A, const void* B, void* C, const int* tiles, const int* n_tiles, const int* row_token, int capacity, int cap, int N, int K,
-                int act, int fp32, cudaStream_t st);
-int rb_moe_gemm(const void* X, const void* W, void* out, const int* tiles, const int* n_tiles, const int* row_token, int x_rows, int capacity,
-                int cap, int E, int N, int K, int act, int bn, int full, int* err, cudaStream_t st);
+int rb_moe_simt(const void* A, const void* B, void* C, const int* tiles, const int* n_tiles, const int* row_token, int capacity, int cap, int N, int
+                K, int act, float limit, int fp32, cudaStream_t st);
+int rb_moe_gemm(const void* X, const void* W, void* out, const int* tiles, const int* n_tiles, const int* row_token, int x_rows, int capacity, int
+                cap, int E, int N, int K, int act, float limit, int bn, int full, int* err, cudaStream_t st);
 #ifdef __cplusplus
 }
 #endif

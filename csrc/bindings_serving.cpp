@@ -29,6 +29,7 @@ inline int is_fp32(const torch::Tensor& t) {
   TORCH_CHECK(t.scalar_type() == at::kFloat || t.scalar_type() == at::kBFloat16, "bf16 or fp32 expected, got ", t.scalar_type());
   return t.scalar_type() == at::kFloat;
 }
+inline bool is_i32(const torch::Tensor& t) { return t.scalar_type() == at::kInt && t.is_contiguous(); }
 inline void check_same(const torch::Tensor& a, const torch::Tensor& b, const char* what) {
   TORCH_CHECK(a.scalar_type() == b.scalar_type() && a.device() == b.device(), what, ": operands differ in type or device");
 }
@@ -131,13 +132,13 @@ void gemm_splitk(torch::Tensor A, torch::Tensor B, torch::Tensor C, c10::optiona
 }
 
 // ---- composed stacks
-void embed_rows(torch::Tensor tok, torch::Tensor w, torch::Tensor res, torch::Tensor h) {
+void embed_rows(torch::Tensor tok, torch::Tensor w, torch::Tensor res, torch::Tensor h, double scale) {
   const c10::cuda::CUDAGuard guard(w.device());
   check_same(w, h, "embed_rows");
   TORCH_CHECK(tok.scalar_type() == at::kLong && tok.is_contiguous() && w.is_contiguous() && res.is_contiguous() && h.is_contiguous());
   TORCH_CHECK(res.scalar_type() == at::kFloat && res.sizes() == h.sizes() && h.size(0) == tok.numel() && h.size(1) == w.size(1));
   check(rb_embed_rows((const long long*)tok.data_ptr<int64_t>(), w.data_ptr(), res.data_ptr<float>(), h.data_ptr(), (int)tok.numel(),
-                      (int)w.size(0), (int)w.size(1), is_fp32(w), cur_stream()),
+                      (int)w.size(0), (int)w.size(1), (float)scale, is_fp32(w), cur_stream()),
         "rb_embed_rows");
 }
 void norm_add(torch::Tensor res, torch::Tensor y, torch::Tensor w, c10::optional<torch::Tensor> next_w, torch::Tensor h, int64_t width,
@@ -194,14 +195,29 @@ bool hgrn2(torch::Tensor qfv, torch::Tensor f_bias, torch::Tensor lower, torch::
         "rb_hgrn2");
   return true;
 }
-void latent_write(torch::Tensor raw, torch::Tensor w, torch::Tensor pool, torch::Tensor slots, int64_t rank, double eps) {
+// k_rot, q, table: the rotated key part and the query heads [T][H][dk] (features dim .. dim + rot turn in place) of the same projection
+void latent_write(torch::Tensor raw, c10::optional<torch::Tensor> k_rot, c10::optional<torch::Tensor> q, c10::optional<torch::Tensor> table, torch::Tensor w,
+                  torch::Tensor pool, torch::Tensor slots, int64_t rank, int64_t part, int64_t rot, int64_t dim, double eps) {
   const c10::cuda::CUDAGuard guard(raw.device());
+  TORCH_CHECK(rot == 0 || (k_rot.has_value() && q.has_value() && table.has_value()), "latent_write: rotated parts");
+  if (rot) {
+    check_same(raw, *k_rot, "latent_write");
+    check_same(raw, *q, "latent_write");
+    const bool one = raw.size(0) == 1;      // (a dimension of size one may have any stride)
+    TORCH_CHECK(k_rot->dim() == 2 && (one || k_rot->stride(0) == raw.stride(0)) && k_rot->stride(1) == 1 && k_rot->size(1) >= rot &&
+                k_rot->size(0) == raw.size(0), "latent_write: rotated key part");
+    TORCH_CHECK(q->dim() == 3 && q->size(0) == raw.size(0) && (one || q->stride(0) == raw.stride(0)) && q->stride(2) == 1 &&
+                (q->size(1) == 1 || q->stride(1) == q->size(2)), "latent_write: queries");
+    TORCH_CHECK(table->scalar_type() == at::kFloat && table->is_contiguous() && table->numel() == raw.size(0) * rot, "latent_write: angles");
+  }
   check_same(raw, w, "latent_write");
   check_same(raw, pool, "latent_write");
   TORCH_CHECK(raw.dim() == 2 && raw.stride(1) == 1 && raw.size(1) >= rank && w.numel() >= rank && pool.dim() == 2 && pool.is_contiguous());
   TORCH_CHECK(slots.scalar_type() == at::kLong && slots.is_contiguous() && slots.numel() == raw.size(0));
-  check(rb_latent_write(raw.data_ptr(), (int)raw.stride(0), w.data_ptr(), pool.data_ptr(), (const long long*)slots.data_ptr<int64_t>(), pool.size(0),
-                        (int)raw.size(0), (int)rank, (int)pool.size(1), (float)eps, is_fp32(raw), cur_stream()),
+  check(rb_latent_write(raw.data_ptr(), rot ? k_rot->data_ptr() : nullptr, rot ? q->data_ptr() : nullptr, (int)raw.stride(0), w.data_ptr(), pool.data_ptr(),
+                        (const long long*)slots.data_ptr<int64_t>(), rot ? table->data_ptr<float>() : nullptr, pool.size(0), (int)raw.size(0), (int)rank,
+                        (int)pool.size(1), (int)part, (int)rot, rot ? (int)q->size(1) : 0, rot ? (int)q->size(2) : 0, (int)dim, (float)eps, is_fp32(raw),
+                        cur_stream()),
         "rb_latent_write");
 }
 void latent_attn(torch::Tensor q, torch::Tensor pool, torch::Tensor bt, c10::optional<torch::Tensor> row_seg, c10::optional<torch::Tensor> row_pos,
@@ -210,7 +226,8 @@ void latent_attn(torch::Tensor q, torch::Tensor pool, torch::Tensor bt, c10::opt
   check_same(q, pool, "latent_attn");
   check_same(q, out, "latent_attn");
   const int64_t T = q.size(0);
-  TORCH_CHECK(q.dim() == 3 && q.is_contiguous() && out.is_contiguous() && out.sizes() == q.sizes() && pool.is_contiguous() && pool.size(1) == q.size(2));
+  TORCH_CHECK(q.dim() == 3 && q.is_contiguous() && out.dim() == 3 && out.is_contiguous() && pool.is_contiguous() && pool.size(1) == q.size(2));
+  TORCH_CHECK(out.size(0) == T && out.size(1) == q.size(1) && out.size(2) <= q.size(2), "latent_attn: output");
   TORCH_CHECK(bt.scalar_type() == at::kInt && bt.is_contiguous() && ctx.scalar_type() == at::kInt && ctx.is_contiguous());
   TORCH_CHECK(row_seg.has_value() == row_pos.has_value());
   TORCH_CHECK(row_seg.has_value() ? (row_seg->numel() == T && row_pos->numel() == T && row_seg->scalar_type() == at::kInt &&
@@ -218,7 +235,7 @@ void latent_attn(torch::Tensor q, torch::Tensor pool, torch::Tensor bt, c10::opt
                                   : (ctx.numel() == T && bt.size(0) == T), "latent_attn: row description");
   TORCH_CHECK(!gate.has_value() || (gate->scalar_type() == q.scalar_type() && gate->stride(1) == 1 && gate->size(0) == T));
   check(rb_latent_attn(q.data_ptr(), pool.data_ptr(), bt.data_ptr<int>(), optint(row_seg), optint(row_pos), ctx.data_ptr<int>(), optptr(gate),
-                       out.data_ptr(), (int)T, (int)q.size(1), (int)q.size(2), (int)bt.size(1), (int)block_size,
+                       out.data_ptr(), (int)T, (int)q.size(1), (int)q.size(2), (int)out.size(2), (int)bt.size(1), (int)block_size,
                        gate.has_value() ? (int)gate->stride(0) : 0, (float)scale, is_fp32(q), cur_stream()),
         "rb_latent_attn");
 }
@@ -227,9 +244,10 @@ bool latent_attn_tc(torch::Tensor q, torch::Tensor pool, torch::Tensor bt, c10::
                     c10::optional<torch::Tensor> gate, torch::Tensor out, c10::optional<torch::Tensor> part_o,
                     c10::optional<torch::Tensor> part_ml, int64_t block_size, int64_t width, int64_t splits, double scale, torch::Tensor err) {
   const c10::cuda::CUDAGuard guard(q.device());
-  const int64_t T = q.size(0), H = q.size(1), R = q.size(2);
+  const int64_t T = q.size(0), H = q.size(1), R = q.size(2), Rv = out.size(2);
   TORCH_CHECK(q.scalar_type() == at::kBFloat16 && pool.scalar_type() == at::kBFloat16 && out.scalar_type() == at::kBFloat16);
-  TORCH_CHECK(q.dim() == 3 && q.is_contiguous() && out.is_contiguous() && out.sizes() == q.sizes() && pool.is_contiguous() && pool.size(1) == R);
+  TORCH_CHECK(q.dim() == 3 && q.is_contiguous() && out.dim() == 3 && out.is_contiguous() && pool.is_contiguous() && pool.size(1) == R);
+  TORCH_CHECK(out.size(0) == T && out.size(1) == H && Rv <= R, "latent_attn_tc: output");
   TORCH_CHECK(bt.scalar_type() == at::kInt && bt.is_contiguous() && ctx.scalar_type() == at::kInt && ctx.is_contiguous());
   if (items.has_value()) {
     TORCH_CHECK(items->scalar_type() == at::kInt && items->dim() == 2 && items->size(1) == 4 && items->is_contiguous());
@@ -237,35 +255,44 @@ bool latent_attn_tc(torch::Tensor q, torch::Tensor pool, torch::Tensor bt, c10::
     TORCH_CHECK(ctx.numel() == T && bt.size(0) == T, "latent_attn_tc: one row per segment");
   }
   TORCH_CHECK(!gate.has_value() || (gate->scalar_type() == at::kBFloat16 && gate->stride(1) == 1 && gate->size(0) == T));
-  TORCH_CHECK(splits == 1 || (part_o.has_value() && part_o->numel() >= splits * T * H * R && part_ml.has_value() &&
+  TORCH_CHECK(splits == 1 || (part_o.has_value() && part_o->numel() >= splits * T * H * Rv && part_ml.has_value() &&
                               part_ml->numel() >= splits * T * H * 2), "latent_attn_tc: scratch");
   const int rc = rb_latent_attn_tc(q.data_ptr(), pool.data_ptr(), bt.data_ptr<int>(), optint(items), ctx.data_ptr<int>(), optptr(gate), out.data_ptr(),
                                    part_o.has_value() ? part_o->data_ptr<float>() : nullptr, part_ml.has_value() ? part_ml->data_ptr<float>() : nullptr,
-                                   (int)T, (int)H, (int)R, pool.size(0), (int)bt.size(1), (int)block_size,
+                                   (int)T, (int)H, (int)R, (int)Rv, pool.size(0), (int)bt.size(1), (int)block_size,
                                    items.has_value() ? (int)items->size(0) : 0, (int)width, (int)splits,
                                    gate.has_value() ? (int)gate->stride(0) : 0, (float)scale, err.data_ptr<int>(), cur_stream());
   if (rc == -20) return false;
   check(rc, "rb_latent_attn_tc");
   return true;
 }
-bool head_gemm(torch::Tensor x, torch::Tensor w, torch::Tensor out, bool kn, torch::Tensor err) {
+// gate: columns of a gate per output feature, [T, >= H N], or none
+inline int gate_pitch(const c10::optional<torch::Tensor>& gate, const torch::Tensor& like, int64_t rows, int64_t cols) {
+  if (!gate.has_value()) return 0;
+  TORCH_CHECK(gate->scalar_type() == like.scalar_type() && gate->device() == like.device() && gate->dim() == 2 && gate->stride(1) == 1, "output gate: layout");
+  TORCH_CHECK(gate->size(0) == rows && gate->size(1) >= cols, "output gate: shape");
+  return (int)gate->stride(0);
+}
+bool head_gemm(torch::Tensor x, torch::Tensor w, c10::optional<torch::Tensor> gate, torch::Tensor out, bool kn, torch::Tensor err) {
   const c10::cuda::CUDAGuard guard(x.device());
   TORCH_CHECK(x.scalar_type() == at::kBFloat16 && w.scalar_type() == at::kBFloat16 && out.scalar_type() == at::kBFloat16);
   TORCH_CHECK(x.dim() == 3 && w.dim() == 3 && out.dim() == 3 && x.stride(2) == 1 && w.is_contiguous() && out.is_contiguous());
   TORCH_CHECK(w.size(0) == x.size(1) && w.size(kn ? 1 : 2) == x.size(2) && out.size(0) == x.size(0) && out.size(1) == x.size(1) &&
               out.size(2) == w.size(kn ? 2 : 1), "head_gemm: shapes");
-  const int rc = rb_head_gemm(x.data_ptr(), w.data_ptr(), out.data_ptr(), (int)x.size(0), (int)x.size(1), (int)out.size(2), (int)x.size(2), x.stride(0),
+  const int rc = rb_head_gemm(x.data_ptr(), w.data_ptr(), optptr(gate), gate_pitch(gate, x, x.size(0), out.size(1) * out.size(2)), out.data_ptr(), (int)x.size(0), (int)x.size(1), (int)out.size(2), (int)x.size(2), x.stride(0),
                               x.stride(1), kn, err.data_ptr<int>(), cur_stream());
   if (rc == -20) return false;
   check(rc, "rb_head_gemm");
   return true;
 }
-void gate_heads(torch::Tensor o, torch::Tensor gate, torch::Tensor out, int64_t dv) {
+// features: a gate per output feature, else per head
+void gate_heads(torch::Tensor o, torch::Tensor gate, torch::Tensor out, int64_t dv, bool features) {
   const c10::cuda::CUDAGuard guard(o.device());
-  TORCH_CHECK(o.scalar_type() == at::kBFloat16 && gate.scalar_type() == at::kBFloat16 && out.scalar_type() == at::kBFloat16);
-  TORCH_CHECK(o.dim() == 3 && o.size(2) == 128 && o.is_contiguous() && out.is_contiguous() && gate.stride(1) == 1 && gate.size(0) == o.size(0));
-  TORCH_CHECK(out.numel() == o.size(0) * o.size(1) * dv);
-  check(rb_gate_heads(o.data_ptr(), gate.data_ptr(), (int)gate.stride(0), out.data_ptr(), (int)o.size(0), (int)o.size(1), (int)dv, cur_stream()),
+  check_same(o, out, "gate_heads");
+  TORCH_CHECK(o.dim() == 3 && o.is_contiguous() && out.is_contiguous() && out.numel() == o.size(0) * o.size(1) * dv);
+  const int ld = gate_pitch(gate, o, o.size(0), features ? o.size(1) * dv : o.size(1));
+  check(rb_gate_heads(o.data_ptr(), gate.data_ptr(), ld, out.data_ptr(), (int)o.size(0), (int)o.size(1), (int)o.size(2), (int)dv, features, is_fp32(o),
+                      cur_stream()),
         "rb_gate_heads");
 }
 void glu(torch::Tensor in, torch::Tensor out, int64_t act) {
@@ -288,7 +315,6 @@ void simt_gemm(torch::Tensor A, torch::Tensor B, torch::Tensor C, bool b_kn) {
         "rb_simt_gemm");
 }
 // ---- attention over cached keys and values, routed experts
-inline bool is_i32(const torch::Tensor& t) { return t.scalar_type() == at::kInt && t.is_contiguous(); }
 void embed_norm(torch::Tensor tok, torch::Tensor table, torch::Tensor w, torch::Tensor res, torch::Tensor h, int64_t width, int64_t groups, double eps) {
   const c10::cuda::CUDAGuard guard(table.device());
   check_same(table, h, "embed_norm");
@@ -299,19 +325,55 @@ void embed_norm(torch::Tensor tok, torch::Tensor table, torch::Tensor w, torch::
                       (int)table.size(0), (int)table.size(1), (int)width, (int)groups, (float)eps, is_fp32(table), cur_stream()),
         "rb_embed_norm");
 }
+// choices from `experts` on (= entries of offset - 1) are identity experts
+inline int check_experts(const torch::Tensor& res, const torch::Tensor& ex, const torch::Tensor& expert, const torch::Tensor& place,
+                         const torch::Tensor& offset, const torch::Tensor& weight) {
+  TORCH_CHECK(ex.dim() == 2 && ex.is_contiguous() && ex.size(1) == res.size(1) && ex.size(0) == expert.numel(), "expert rows");
+  TORCH_CHECK(is_i32(expert) && is_i32(place) && is_i32(offset) && weight.scalar_type() == at::kFloat && weight.is_contiguous(), "expert plan: types");
+  TORCH_CHECK(expert.dim() == 2 && expert.size(0) == res.size(0) && place.sizes() == expert.sizes() && weight.sizes() == expert.sizes(), "expert plan: shapes");
+  return (int)offset.numel() - 1;
+}
+// x <- norm(alpha x + y + weighted expert rows); y or the experts may be missing.  centre: layer norm (bias b), else RMS.  next_w: h is the
+// norm of the new stream with it, times scale.
+void sum_norm(torch::Tensor res, c10::optional<torch::Tensor> y, c10::optional<torch::Tensor> ex, c10::optional<torch::Tensor> expert,
+              c10::optional<torch::Tensor> place, c10::optional<torch::Tensor> offset, c10::optional<torch::Tensor> weight, torch::Tensor w,
+              c10::optional<torch::Tensor> b, c10::optional<torch::Tensor> next_w, c10::optional<torch::Tensor> next_b, torch::Tensor h, int64_t width,
+              bool centre, double alpha, double eps, double scale) {
+  const c10::cuda::CUDAGuard guard(res.device());
+  check_same(w, h, "sum_norm");
+  TORCH_CHECK(res.scalar_type() == at::kFloat && res.is_contiguous() && h.is_contiguous() && res.sizes() == h.sizes() && w.numel() == res.size(1));
+  for (const auto& t : {b, next_w, next_b})
+    if (t.has_value()) {
+      check_same(w, *t, "sum_norm");
+      TORCH_CHECK(t->numel() == w.numel() && t->is_contiguous(), "sum_norm: weights");
+    }
+  if (y.has_value()) {
+    check_same(w, *y, "sum_norm");
+    TORCH_CHECK(y->is_contiguous() && y->sizes() == res.sizes(), "sum_norm: input");
+  }
+  int top = 0, experts = 0;
+  if (ex.has_value()) {
+    check_same(w, *ex, "sum_norm");
+    TORCH_CHECK(expert.has_value() && place.has_value() && offset.has_value() && weight.has_value(), "sum_norm: expert plan");
+    experts = check_experts(res, *ex, *expert, *place, *offset, *weight);
+    top = (int)expert->size(1);
+  }
+  check(rb_sum_norm(res.data_ptr<float>(), optptr(y), optptr(ex), optint(expert), optint(place), optint(offset),
+                    weight.has_value() ? weight->data_ptr<float>() : nullptr, top, experts, w.data_ptr(), optptr(b), optptr(next_w), optptr(next_b), h.data_ptr(),
+                    (int)res.size(0), (int)res.size(1), (int)res.size(1), (int)width, centre, (float)alpha, (float)eps, (float)scale, is_fp32(w), cur_stream()),
+        "rb_sum_norm");
+}
 void norm_add_experts(torch::Tensor res, c10::optional<torch::Tensor> y, torch::Tensor ex, torch::Tensor expert, torch::Tensor place, torch::Tensor offset,
                       torch::Tensor weight, torch::Tensor w, c10::optional<torch::Tensor> next_w, torch::Tensor h, int64_t width, int64_t groups, double eps) {
   const c10::cuda::CUDAGuard guard(res.device());
   check_same(ex, w, "norm_add_experts");
   check_same(ex, h, "norm_add_experts");
   TORCH_CHECK(res.scalar_type() == at::kFloat && res.is_contiguous() && h.is_contiguous() && res.sizes() == h.sizes() && w.numel() == res.size(1));
-  TORCH_CHECK(ex.dim() == 2 && ex.is_contiguous() && ex.size(1) == res.size(1) && ex.size(0) == expert.numel());
+  const int experts = check_experts(res, ex, expert, place, offset, weight);
   TORCH_CHECK(!y.has_value() || (y->scalar_type() == ex.scalar_type() && y->is_contiguous() && y->sizes() == res.sizes()));
-  TORCH_CHECK(is_i32(expert) && is_i32(place) && is_i32(offset) && weight.scalar_type() == at::kFloat && weight.is_contiguous());
-  TORCH_CHECK(expert.dim() == 2 && expert.size(0) == res.size(0) && place.sizes() == expert.sizes() && weight.sizes() == expert.sizes());
   TORCH_CHECK(!next_w.has_value() || (next_w->numel() == w.numel() && next_w->scalar_type() == w.scalar_type()));
   check(rb_norm_add_experts(res.data_ptr<float>(), optptr(y), ex.data_ptr(), expert.data_ptr<int>(), place.data_ptr<int>(), offset.data_ptr<int>(),
-                            weight.data_ptr<float>(), (int)expert.size(1), w.data_ptr(), optptr(next_w), h.data_ptr(), (int)res.size(0),
+                            weight.data_ptr<float>(), (int)expert.size(1), experts, w.data_ptr(), optptr(next_w), h.data_ptr(), (int)res.size(0),
                             (int)ex.size(1), (int)res.size(1), (int)width, (int)groups, (float)eps, is_fp32(ex), cur_stream()),
         "rb_norm_add_experts");
 }
@@ -344,6 +406,38 @@ void attention_inputs(torch::Tensor qkv, c10::optional<torch::Tensor> table, tor
                             cur_stream()),
         "rb_attention_inputs");
 }
+// the same with weighted norms over the whole query and key projections (q_w, k_w; none: no norm when eps <= 0); halves: pairs rot / 2 apart
+void projection_inputs(torch::Tensor qkv, c10::optional<torch::Tensor> q_w, c10::optional<torch::Tensor> k_w, c10::optional<torch::Tensor> table, torch::Tensor q,
+                       c10::optional<torch::Tensor> k_pool, c10::optional<torch::Tensor> v_pool, torch::Tensor slots, int64_t kv_heads, int64_t dim, int64_t vdim,
+                       int64_t rot, bool halves, double eps) {
+  const c10::cuda::CUDAGuard guard(qkv.device());
+  check_same(qkv, q, "projection_inputs");
+  const int64_t T = qkv.size(0);
+  TORCH_CHECK(qkv.dim() == 2 && qkv.stride(1) == 1 && q.dim() == 3 && q.is_contiguous() && q.size(0) == T && k_pool.has_value() == v_pool.has_value());
+  TORCH_CHECK(qkv.size(1) >= q.size(1) * dim + (k_pool.has_value() ? kv_heads * (dim + vdim) : 0), "projection_inputs: columns");
+  TORCH_CHECK(rot == 0 || (table.has_value() && table->scalar_type() == at::kFloat && table->is_contiguous() && table->numel() == T * rot));
+  TORCH_CHECK(slots.scalar_type() == at::kLong && slots.is_contiguous() && slots.numel() == T);
+  if (q_w.has_value()) {
+    check_same(qkv, *q_w, "projection_inputs");
+    TORCH_CHECK(q_w->is_contiguous() && q_w->numel() == q.size(1) * dim, "projection_inputs: query norm");
+  }
+  if (k_pool.has_value()) {
+    check_same(qkv, *k_pool, "projection_inputs");
+    check_same(qkv, *v_pool, "projection_inputs");
+    TORCH_CHECK(k_pool->dim() == 3 && v_pool->dim() == 3 && k_pool->is_contiguous() && v_pool->is_contiguous() && k_pool->size(0) == v_pool->size(0));
+    TORCH_CHECK(k_pool->size(1) == kv_heads && v_pool->size(1) == kv_heads && k_pool->size(2) == q.size(2), "projection_inputs: pools");
+    if (k_w.has_value()) {
+      check_same(qkv, *k_w, "projection_inputs");
+      TORCH_CHECK(k_w->is_contiguous() && k_w->numel() == kv_heads * dim, "projection_inputs: key norm");
+    }
+  }
+  check(rb_projection_inputs(qkv.data_ptr(), (int)qkv.stride(0), optptr(q_w), optptr(k_w), rot ? table->data_ptr<float>() : nullptr, q.data_ptr(),
+                             k_pool.has_value() ? k_pool->data_ptr() : nullptr, v_pool.has_value() ? v_pool->data_ptr() : nullptr,
+                             (const long long*)slots.data_ptr<int64_t>(), k_pool.has_value() ? k_pool->size(0) : 0, (int)T, (int)q.size(1), (int)kv_heads,
+                             (int)dim, (int)vdim, (int)q.size(2), v_pool.has_value() ? (int)v_pool->size(2) : 0, (int)rot, halves, (float)eps, is_fp32(qkv),
+                             cur_stream()),
+        "rb_projection_inputs");
+}
 inline void check_pools(const torch::Tensor& q, const torch::Tensor& k, const torch::Tensor& v, const torch::Tensor& bt, const torch::Tensor& ctx,
                         const c10::optional<torch::Tensor>& sink, const torch::Tensor& out) {
   check_same(q, k, "paged attention");
@@ -356,7 +450,8 @@ inline void check_pools(const torch::Tensor& q, const torch::Tensor& k, const to
   TORCH_CHECK(!sink.has_value() || (sink->scalar_type() == q.scalar_type() && sink->is_contiguous() && sink->numel() == q.size(1)), "paged attention: sink");
 }
 void gqa_attn(torch::Tensor q, torch::Tensor k, torch::Tensor v, torch::Tensor bt, c10::optional<torch::Tensor> row_seg, c10::optional<torch::Tensor> row_pos,
-              torch::Tensor ctx, c10::optional<torch::Tensor> sink, torch::Tensor out, int64_t block_size, double scale) {
+              torch::Tensor ctx, c10::optional<torch::Tensor> sink, c10::optional<torch::Tensor> gate, torch::Tensor out, int64_t block_size, int64_t window,
+              double scale) {
   const c10::cuda::CUDAGuard guard(q.device());
   check_pools(q, k, v, bt, ctx, sink, out);
   const int64_t T = q.size(0), H = q.size(1);
@@ -364,29 +459,30 @@ void gqa_attn(torch::Tensor q, torch::Tensor k, torch::Tensor v, torch::Tensor b
   TORCH_CHECK(row_seg.has_value() ? (is_i32(*row_seg) && is_i32(*row_pos) && row_seg->numel() == T && row_pos->numel() == T) : ctx.numel() == T,
               "gqa_attn: row description");
   check(rb_gqa_attn(q.data_ptr(), k.data_ptr(), v.data_ptr(), bt.data_ptr<int>(), optint(row_seg), optint(row_pos), ctx.data_ptr<int>(), optptr(sink),
-                    out.data_ptr(), (int)T, (int)H, (int)k.size(1), (int)q.size(2), (int)v.size(2), (int)(out.size(1) / H), (int)bt.size(1),
-                    (int)block_size, (float)scale, is_fp32(q), cur_stream()),
+                    optptr(gate), gate_pitch(gate, q, T, out.size(1)), out.data_ptr(), (int)T, (int)H, (int)k.size(1), (int)q.size(2), (int)v.size(2),
+                    (int)(out.size(1) / H), (int)bt.size(1), (int)block_size, (int)window, (float)scale, is_fp32(q), cur_stream()),
         "rb_gqa_attn");
 }
 // Prompt portions; returns false for shapes the tensor-core kernel does not take.
 bool paged_flash(torch::Tensor q, torch::Tensor k, torch::Tensor v, torch::Tensor bt, torch::Tensor ctx, c10::optional<torch::Tensor> blocks,
-                 c10::optional<torch::Tensor> sink, torch::Tensor out, int64_t block_size, double scale, torch::Tensor err) {
+                 c10::optional<torch::Tensor> sink, c10::optional<torch::Tensor> gate, torch::Tensor out, int64_t block_size, int64_t window, double scale,
+                 torch::Tensor err) {
   const c10::cuda::CUDAGuard guard(q.device());
   if (q.scalar_type() != at::kBFloat16) return false;
   check_pools(q, k, v, bt, ctx, sink, out);
   const int64_t T = q.size(0), H = q.size(1);
   TORCH_CHECK(blocks.has_value() ? (is_i32(*blocks) && blocks->dim() == 2 && blocks->size(1) == 4) : ctx.numel() == T, "paged_flash: query tiles");
-  const int rc = rb_paged_flash(q.data_ptr(), k.data_ptr(), v.data_ptr(), bt.data_ptr<int>(), ctx.data_ptr<int>(), optint(blocks), optptr(sink), out.data_ptr(),
-                                (int)T, (int)(blocks.has_value() ? blocks->size(0) : T), (int)H, (int)k.size(1), (int)q.size(2), (int)v.size(2),
-                                (int)(out.size(1) / H), k.size(0), (int)block_size, (int)bt.size(1), (float)scale, err.data_ptr<int>(), cur_stream());
+  const int rc = rb_paged_flash(q.data_ptr(), k.data_ptr(), v.data_ptr(), bt.data_ptr<int>(), ctx.data_ptr<int>(), optint(blocks), optptr(sink),
+                                optptr(gate), gate_pitch(gate, q, T, out.size(1)), out.data_ptr(), (int)T, (int)(blocks.has_value() ? blocks->size(0) : T), (int)H, (int)k.size(1), (int)q.size(2), (int)v.size(2),
+                                (int)(out.size(1) / H), k.size(0), (int)block_size, (int)bt.size(1), (int)window, (float)scale, err.data_ptr<int>(), cur_stream());
   if (rc == -20) return false;
   check(rc, "rb_paged_flash");
   return true;
 }
 // One row per sequence; returns false for shapes the tensor-core kernel does not take.
-bool paged_decode(torch::Tensor q, torch::Tensor k, torch::Tensor v, torch::Tensor bt, torch::Tensor ctx, c10::optional<torch::Tensor> sink, torch::Tensor out,
-                  c10::optional<torch::Tensor> part_o, c10::optional<torch::Tensor> part_ml, int64_t block_size, int64_t max_ctx, int64_t splits,
-                  double scale, torch::Tensor err) {
+bool paged_decode(torch::Tensor q, torch::Tensor k, torch::Tensor v, torch::Tensor bt, torch::Tensor ctx, c10::optional<torch::Tensor> sink,
+                  c10::optional<torch::Tensor> gate, torch::Tensor out, c10::optional<torch::Tensor> part_o, c10::optional<torch::Tensor> part_ml,
+                  int64_t block_size, int64_t max_ctx, int64_t window, int64_t splits, double scale, torch::Tensor err) {
   const c10::cuda::CUDAGuard guard(q.device());
   if (q.scalar_type() != at::kBFloat16) return false;
   check_pools(q, k, v, bt, ctx, sink, out);
@@ -394,49 +490,55 @@ bool paged_decode(torch::Tensor q, torch::Tensor k, torch::Tensor v, torch::Tens
   TORCH_CHECK(ctx.numel() == B, "paged_decode: one row per sequence");
   TORCH_CHECK(splits == 1 || (part_o.has_value() && part_o->scalar_type() == at::kFloat && part_o->numel() >= splits * B * H * 128 && part_ml.has_value() &&
                               part_ml->scalar_type() == at::kFloat && part_ml->numel() >= splits * B * H * 2), "paged_decode: scratch");
-  const int rc = rb_paged_decode_tc(q.data_ptr(), k.data_ptr(), v.data_ptr(), bt.data_ptr<int>(), ctx.data_ptr<int>(), optptr(sink), out.data_ptr(),
-                                    part_o.has_value() ? part_o->data_ptr<float>() : nullptr, part_ml.has_value() ? part_ml->data_ptr<float>() : nullptr,
+  const int rc = rb_paged_decode_tc(q.data_ptr(), k.data_ptr(), v.data_ptr(), bt.data_ptr<int>(), ctx.data_ptr<int>(), optptr(sink), optptr(gate),
+                                    gate_pitch(gate, q, B, out.size(1)), out.data_ptr(), part_o.has_value() ? part_o->data_ptr<float>() : nullptr, part_ml.has_value() ? part_ml->data_ptr<float>() : nullptr,
                                     (int)B, (int)H, (int)k.size(1), (int)q.size(2), (int)v.size(2), (int)(out.size(1) / H), k.size(0), (int)block_size,
-                                    (int)bt.size(1), (int)max_ctx, (float)scale, (int)splits, err.data_ptr<int>(), cur_stream());
+                                    (int)bt.size(1), (int)max_ctx, (int)window, (float)scale, (int)splits, err.data_ptr<int>(), cur_stream());
   if (rc == -20) return false;
   check(rc, "rb_paged_decode_tc");
   return true;
 }
-void moe_route(torch::Tensor logits, torch::Tensor expert, torch::Tensor weight, torch::Tensor place, torch::Tensor row_token, torch::Tensor count,
-               torch::Tensor offset, torch::Tensor tiles, torch::Tensor n_tiles, int64_t experts, int64_t groups, int64_t keep, int64_t tile_rows,
-               bool renormalize, double weight_scale) {
+void moe_route(torch::Tensor logits, c10::optional<torch::Tensor> correction, torch::Tensor expert, torch::Tensor weight, torch::Tensor place, torch::Tensor row_token, torch::Tensor count,
+               torch::Tensor offset, torch::Tensor tiles, torch::Tensor n_tiles, int64_t experts, int64_t outputs, int64_t groups, int64_t keep,
+               int64_t group_best, int64_t tile_rows, bool renormalize, bool softmax, double weight_scale) {
   const c10::cuda::CUDAGuard guard(logits.device());
   const int64_t T = logits.size(0), top = expert.size(1);
-  TORCH_CHECK(logits.dim() == 2 && logits.scalar_type() == at::kFloat && logits.stride(1) == 1 && logits.size(1) >= experts, "moe_route: logits");
+  TORCH_CHECK(logits.dim() == 2 && logits.scalar_type() == at::kFloat && logits.stride(1) == 1 && logits.size(1) >= outputs, "moe_route: logits");
+  int corr_fp32 = 0;
+  if (correction.has_value()) {
+    TORCH_CHECK(correction->is_contiguous() && correction->numel() >= outputs && correction->device() == logits.device(), "moe_route: correction");
+    corr_fp32 = is_fp32(*correction);
+  }
   TORCH_CHECK(is_i32(expert) && is_i32(place) && expert.size(0) == T && place.sizes() == expert.sizes() && weight.scalar_type() == at::kFloat &&
               weight.is_contiguous() && weight.sizes() == expert.sizes());
   TORCH_CHECK(is_i32(row_token) && row_token.numel() >= experts * T && is_i32(count) && count.numel() >= experts + 1 && is_i32(offset) &&
-              offset.numel() >= experts + 1 && is_i32(n_tiles) && is_i32(tiles) && tiles.dim() == 2 && tiles.size(1) == 4);
+              offset.numel() == experts + 1 && is_i32(n_tiles) && is_i32(tiles) && tiles.dim() == 2 && tiles.size(1) == 4);
   TORCH_CHECK(tiles.size(0) >= std::min(T * top, experts) + T * top / tile_rows, "moe_route: tile list");
-  check(rb_moe_route(logits.data_ptr<float>(), (int)logits.stride(0), expert.data_ptr<int>(), weight.data_ptr<float>(), place.data_ptr<int>(),
+  check(rb_moe_route(logits.data_ptr<float>(), (int)logits.stride(0), optptr(correction), corr_fp32, expert.data_ptr<int>(), weight.data_ptr<float>(), place.data_ptr<int>(),
                      row_token.data_ptr<int>(), count.data_ptr<int>(), offset.data_ptr<int>(), tiles.data_ptr<int>(), n_tiles.data_ptr<int>(), (int)T,
-                     (int)experts, (int)groups, (int)keep, (int)top, (int)tile_rows, (int)tiles.size(0), renormalize, (float)weight_scale, cur_stream()),
+                     (int)experts, (int)outputs, (int)groups, (int)keep, (int)group_best, (int)top, (int)tile_rows, (int)tiles.size(0), renormalize, softmax,
+                     (float)weight_scale, cur_stream()),
         "rb_moe_route");
 }
-// out[sorted row] = act(x[its token, or the sorted row] * W[expert]^T); act: 0 none, 1 squared relu
+// out[sorted row] = act(x[its token, or the sorted row] * W[expert]^T); act: 0 none, 1 squared relu, 2 gated (half as many columns out)
 void moe_gemm(torch::Tensor x, torch::Tensor W, torch::Tensor out, torch::Tensor tiles, torch::Tensor n_tiles, c10::optional<torch::Tensor> row_token,
-              int64_t act, int64_t bn, bool full, torch::Tensor err) {
+              int64_t act, double limit, int64_t bn, bool full, torch::Tensor err) {
   const c10::cuda::CUDAGuard guard(x.device());
   check_same(x, W, "moe_gemm");
   check_same(x, out, "moe_gemm");
   const int64_t E = W.size(0), N = W.size(1), K = W.size(2);
-  TORCH_CHECK(x.dim() == 2 && W.dim() == 3 && out.dim() == 2 && x.is_contiguous() && W.is_contiguous() && out.is_contiguous() && x.size(1) == K && out.size(1) == N);
+  TORCH_CHECK(x.dim() == 2 && W.dim() == 3 && out.dim() == 2 && x.is_contiguous() && W.is_contiguous() && out.is_contiguous() && x.size(1) == K && out.size(1) == (act == 2 ? N / 2 : N));
   TORCH_CHECK(is_i32(tiles) && is_i32(n_tiles) && (!row_token.has_value() || is_i32(*row_token)));
   TORCH_CHECK(row_token.has_value() ? row_token->numel() >= E * x.size(0) : x.size(0) == out.size(0), "moe_gemm: rows");
   const int cap = (int)tiles.size(0);
   if (is_fp32(x)) {
     check(rb_moe_simt(x.data_ptr(), W.data_ptr(), out.data_ptr(), tiles.data_ptr<int>(), n_tiles.data_ptr<int>(), optint(row_token), (int)x.size(0), cap,
-                      (int)N, (int)K, (int)act, 1, cur_stream()),
+                      (int)N, (int)K, (int)act, (float)limit, 1, cur_stream()),
           "rb_moe_simt");
     return;
   }
   check(rb_moe_gemm(x.data_ptr(), W.data_ptr(), out.data_ptr(), tiles.data_ptr<int>(), n_tiles.data_ptr<int>(), optint(row_token), (int)x.size(0),
-                    (int)x.size(0), cap, (int)E, (int)N, (int)K, (int)act, (int)bn, full, err.data_ptr<int>(), cur_stream()),
+                    (int)x.size(0), cap, (int)E, (int)N, (int)K, (int)act, (float)limit, (int)bn, full, err.data_ptr<int>(), cur_stream()),
         "rb_moe_gemm");
 }
 void relu2(torch::Tensor x) {
@@ -469,7 +571,9 @@ void register_serving(pybind11::module_& m) {
   m.def("simt_gemm", &simt_gemm);
   m.def("embed_norm", &embed_norm);
   m.def("norm_add_experts", &norm_add_experts);
+  m.def("sum_norm", &sum_norm);
   m.def("rope_table", &rope_table);
+  m.def("projection_inputs", &projection_inputs);
   m.def("attention_inputs", &attention_inputs);
   m.def("gqa_attn", &gqa_attn);
   m.def("paged_flash", &paged_flash);

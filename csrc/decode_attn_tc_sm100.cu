@@ -13,6 +13,8 @@
 // token row of S^T (and one d row of O^T); the per-head running max is shared by the CTA
 // (lazy rescaling, threshold 2^8), per-thread partial sums are reduced once at the end.
 // CTA = (sequence, kv head, split); partial (m, l, o) go to scratch when splits > 1.
+#include <limits.h>
+
 #include "common.cuh"
 #include "host_utils.h"
 
@@ -51,10 +53,12 @@ struct DecodeTcParams {
   const int* block_tables;  // [B][max_blocks]
   const int* ctx_lens;      // [B]
   const __nv_bfloat16* sink;  // [Hq] logits that only join the denominator, or null
+  const __nv_bfloat16* gate;  // [B][ld_gate]: sigmoid(gate) of every output feature, head h's at h * out_d, or null
   __nv_bfloat16* out;       // [B][Hq][out_d]
   float* part_o;            // [B*Hq*splits][128]
   float* part_ml;           // [B*Hq*splits][2]
-  int Hq, Hkv, G, max_blocks, page, out_d, num_splits, split_tokens;
+  int Hq, Hkv, G, max_blocks, page, out_d, num_splits, split_tokens, ld_gate;
+  int window;               // positions a token sees (INT_MAX: all)
   float scale_log2;
   int* err;
 };
@@ -64,6 +68,9 @@ __device__ __forceinline__ void join_sink(float m, float sink, float& o, float& 
   const float z = sink * 1.4426950408889634f, top = fmaxf(m, z), f = exp2f(m - top);
   o *= f;
   l = l * f + exp2f(z - top);
+}
+__device__ __forceinline__ float open_gate(const __nv_bfloat16* gate, size_t i) {
+  return gate ? __fdividef(1.f, 1.f + __expf(-__bfloat162float(gate[i]))) : 1.f;
 }
 
 // NH: query heads per KV head that the softmax handles (8 or 16)
@@ -92,7 +99,8 @@ decode_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_k, const __grid_co
   const int b = blockIdx.x, kvh = blockIdx.y, split = blockIdx.z;
   const int G = p.G;
   const int ctx = p.ctx_lens[b];
-  const int t_begin = split * p.split_tokens;
+  const int seen_from = max(0, ctx - p.window);                             // first position in the window
+  const int t_begin = seen_from / p.page * p.page + split * p.split_tokens;    // (tiles start on a page)
   const int t_end = min(ctx, t_begin + p.split_tokens);
   const int n_tiles = t_end > t_begin ? (t_end - t_begin + DT_TILE - 1) / DT_TILE : 0;
   const int* bt = p.block_tables + static_cast<size_t>(b) * p.max_blocks;
@@ -216,7 +224,7 @@ decode_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_k, const __grid_co
       tmem_ld_32x32b_x16(tmem_base + DT_T_S + (j & 1) * 16 + lane_addr, raw);
       tmem_wait_ld();
       const int tok = t_begin + j * DT_TILE + r;
-      const bool valid = tok < t_end;
+      const bool valid = tok < t_end && tok >= seen_from;
       float s[NH];
 #pragma unroll
       for (int h = 0; h < NH; ++h) {
@@ -296,7 +304,9 @@ decode_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_k, const __grid_co
         float ov = __uint_as_float(o[h]);
         if (p.num_splits == 1) {
           if (p.sink) join_sink(m_ref[h], __bfloat162float(p.sink[hq]), ov, l);
-          if (r < p.out_d) p.out[(static_cast<size_t>(b) * p.Hq + hq) * p.out_d + r] = __float2bfloat16(l > 0.f ? ov / l : 0.f);
+          if (r < p.out_d)
+            p.out[(static_cast<size_t>(b) * p.Hq + hq) * p.out_d + r] =
+                __float2bfloat16(l > 0.f ? ov / l * open_gate(p.gate, static_cast<size_t>(b) * p.ld_gate + hq * p.out_d + r) : 0.f);
         } else {
           const size_t pidx = (static_cast<size_t>(b) * p.Hq + hq) * p.num_splits + split;
           p.part_o[pidx * DT_D + r] = ov;
@@ -316,8 +326,8 @@ decode_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_k, const __grid_co
 }
 
 __global__ void decode_attn_tc_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
-                                              const __nv_bfloat16* __restrict__ sink, __nv_bfloat16* __restrict__ out,
-                                              int num_splits, int Hq, int out_d) {
+                                              const __nv_bfloat16* __restrict__ sink, const __nv_bfloat16* __restrict__ gate,
+                                              __nv_bfloat16* __restrict__ out, int num_splits, int Hq, int out_d, int ld_gate) {
   const size_t bh = blockIdx.x;
   const int d = threadIdx.x;
   float m = -1e30f;
@@ -329,7 +339,7 @@ __global__ void decode_attn_tc_combine_kernel(const float* __restrict__ part_o, 
     o += w * part_o[(bh * num_splits + s) * DT_D + d];
   }
   if (sink) join_sink(m, __bfloat162float(sink[bh % Hq]), o, l);
-  if (d < out_d) out[bh * out_d + d] = __float2bfloat16(l > 0.f ? o / l : 0.f);
+  if (d < out_d) out[bh * out_d + d] = __float2bfloat16(l > 0.f ? o / l * open_gate(gate, bh / Hq * ld_gate + bh % Hq * out_d + d) : 0.f);
 }
 
 template <int DK, int DV, int NH>
@@ -349,7 +359,7 @@ static int launch_decode_tc(const void* kc, const void* vc, uint64_t slots, cons
   }
   launch_pdl(kern, dim3(B, p.Hkv, p.num_splits), dim3(DT_THREADS), L::kTotal, st, tk, tv, p);
   if (p.num_splits > 1)
-    decode_attn_tc_combine_kernel<<<B * p.Hq, DT_D, 0, st>>>(p.part_o, p.part_ml, p.sink, p.out, p.num_splits, p.Hq, p.out_d);
+    decode_attn_tc_combine_kernel<<<B * p.Hq, DT_D, 0, st>>>(p.part_o, p.part_ml, p.sink, p.gate, p.out, p.num_splits, p.Hq, p.out_d, p.ld_gate);
   rb_note_launch(p.num_splits > 1 ? 2 : 1);
   return (int)cudaGetLastError();
 }
@@ -360,7 +370,7 @@ static DecodeTcParams decode_tc_params(const void* q, const int* block_tables, c
   DecodeTcParams p{};
   p.q = (const __nv_bfloat16*)q; p.block_tables = block_tables; p.ctx_lens = ctx_lens; p.out = (__nv_bfloat16*)out;
   p.part_o = part_o; p.part_ml = part_ml; p.Hq = Hq; p.Hkv = Hkv; p.G = Hq / Hkv; p.max_blocks = max_blocks;
-  p.page = page; p.out_d = DT_D;
+  p.page = page; p.out_d = DT_D; p.window = INT_MAX;
   p.num_splits = splits;
   p.split_tokens = ((max_ctx + splits - 1) / splits + DT_TILE - 1) / DT_TILE * DT_TILE;
   p.scale_log2 = scale * 1.4426950408889634f;
@@ -384,19 +394,25 @@ extern "C" int rb_decode_attn_tc(const void* q, const void* kc, const void* vc, 
 }
 
 // The same over pools [rows][Hkv][dk] / [rows][Hkv][dv] (dk, dv: 64 or 128) with pages of 16 to 128 tokens, an optional sink
-// logit per head and outputs of out_d columns.  Returns -20 for shapes outside that.
+// logit per head, an optional window (positions a token sees, its own included; 0: all), an optional gate per output feature and
+// outputs of out_d columns.  max_ctx: most positions any row may see, rounded up by less than a page at a window's far end
+// (the splits share them out).  Returns -20 for shapes outside that.
 extern "C" int rb_paged_decode_tc(const void* q, const void* kc, const void* vc, const int* block_tables, const int* ctx_lens,
-                                  const void* sink, void* out, float* part_o, float* part_ml, int B, int Hq, int Hkv, int dk, int dv,
-                                  int out_d, long long pool_rows, int page, int max_blocks, int max_ctx, float scale, int splits, int* err,
-                                  cudaStream_t st) {
+                                  const void* sink, const void* gate, int ld_gate, void* out, float* part_o, float* part_ml, int B, int Hq,
+                                  int Hkv, int dk, int dv, int out_d, long long pool_rows, int page, int max_blocks, int max_ctx, int window,
+                                  float scale, int splits, int* err, cudaStream_t st) {
   using namespace rb;
   if (B == 0) return 0;
   if (Hkv < 1 || Hq % Hkv) return -2;
   const int G = Hq / Hkv;
   if (G > 16 || (dk != 64 && dk != 128) || (dv != 64 && dv != 128) || out_d > dv || out_d < 1) return -20;
   if ((page != 16 && page != 32 && page != 64 && page != 128) || Hkv > 65535 || splits < 1 || splits > 65535) return -20;
+  if (window < 0 || (gate && ld_gate < Hq * out_d)) return -2;
+  if (window && window + page < max_ctx) max_ctx = window + page;
   DecodeTcParams p = decode_tc_params(q, block_tables, ctx_lens, out, part_o, part_ml, Hq, Hkv, page, max_blocks, max_ctx, scale, splits, err);
   p.sink = (const __nv_bfloat16*)sink;
+  p.gate = (const __nv_bfloat16*)gate; p.ld_gate = ld_gate;
+  if (window) p.window = window;
   p.out_d = out_d;
   const uint64_t slots = static_cast<uint64_t>(pool_rows);
   if (G <= 8) {

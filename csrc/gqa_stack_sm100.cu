@@ -2,7 +2,9 @@
 // attention for any sizes.  Compiled WITHOUT fast-math: the 32-bit mode of the engine uses these kernels as they are.
 //
 //  * rope_table        cos / sin of every row's angles, once per forward
-//  * attention_inputs  raw projections -> rotated and normed queries; keys and values into their pages
+//  * attention_inputs  raw projections -> rotated and normed queries; keys and values into their pages (norms head by head, pairs
+//                      of neighbours)
+//  * projection_inputs the same with weighted norms over the whole query and key projections, and either pairing
 //  * paged_attention   one (row, head) per CTA: 32-bit mode, and head sizes that the tensor-core kernels do not take
 #include "stack_common.cuh"
 
@@ -96,6 +98,120 @@ __global__ void __launch_bounds__(256) attention_inputs_kernel(const InputParams
   }
 }
 
+// Norms over the whole projection: one CTA per row sums the squares of all query and all key columns, then every thread turns and
+// stores groups of V columns.  A feature's partner in its pair is `rot / 2` columns away, or its neighbour; it is read again
+// (from the cache) instead of being handed over.
+struct ProjectionParams {
+  const void* qkv;           // [T][ld]: H query heads | G key heads | G value heads (keys and values only with k_pool)
+  const void* q_w;           // [H * dim] or null
+  const void* k_w;           // [G * dim] or null
+  const float2* table;       // [T][rot / 2] or null
+  void* q;                   // [T][H][dp]
+  void* k_pool;              // [rows][G][dp] or null
+  void* v_pool;              // [rows][G][vp]
+  const long long* slots;    // [T] pool rows
+  long long pool_rows;
+  int H, G, dim, vdim, dp, vp, rot, halves, ld;
+  float eps;                 // <= 0: no norm
+};
+constexpr int PI_WARPS = 8;
+template <typename T, int V>
+__global__ void __launch_bounds__(PI_WARPS * 32) projection_inputs_kernel(const ProjectionParams p) {
+  __shared__ float red[2][PI_WARPS];
+  const long long t = blockIdx.x;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const T* row = static_cast<const T*>(p.qkv) + t * p.ld;
+  const int qd = p.H * p.dim, kd = p.k_pool ? p.G * p.dim : 0;
+  float r[2] = {1.f, 1.f};
+  if (p.eps > 0.f) {
+    float ss[2] = {0.f, 0.f};
+    for (int c = tid * V; c < qd + kd; c += PI_WARPS * 32 * V) {      // (qd is a multiple of V)
+      float a[V];
+      ldv<V>(row + c, a);
+      float s = 0.f;
+#pragma unroll
+      for (int i = 0; i < V; ++i) s += a[i] * a[i];
+      if (c < qd) ss[0] += s;
+      else ss[1] += s;
+    }
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+      ss[k] = wsum(ss[k]);
+      if (lane == 0) red[k][warp] = ss[k];
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+      float s = 0.f;
+#pragma unroll
+      for (int w = 0; w < PI_WARPS; ++w) s += red[k][w];
+      r[k] = 1.f / sqrtf(s / (k ? max(kd, 1) : qd) + p.eps);
+    }
+  }
+  long long slot = 0;
+  int heads = p.H;
+  if (p.k_pool) {
+    slot = p.slots[t];
+    if (slot >= 0 && slot < p.pool_rows) heads += 2 * p.G;
+  }
+  const int half = p.rot >> 1, per = (max(p.dp, p.k_pool ? p.vp : 0) + V - 1) / V;
+  for (int i = tid; i < heads * per; i += PI_WARPS * 32) {
+    const int hd = i / per, e = (i - hd * per) * V;
+    const int kind = hd < p.H ? 0 : (hd < p.H + p.G ? 1 : 2);
+    const int n = kind == 2 ? p.vdim : p.dim, pitch = kind == 2 ? p.vp : p.dp;
+    if (e >= pitch) continue;
+    const int g = kind == 0 ? hd : hd - p.H - (kind == 2 ? p.G : 0);
+    const T* src = row + (kind == 0 ? 0 : (kind == 1 ? qd : qd + p.G * p.dim)) + g * n;
+    float x[V];
+    if (e < n) {
+      ldv<V>(src + e, x);
+      if (kind < 2) {
+        const T* w = static_cast<const T*>(kind ? p.k_w : p.q_w);
+        const float f = r[kind];
+        if (w) {
+          float b[V];
+          ldv<V>(w + g * n + e, b);
+#pragma unroll
+          for (int k = 0; k < V; ++k) x[k] *= f * b[k];
+        } else {
+#pragma unroll
+          for (int k = 0; k < V; ++k) x[k] *= f;
+        }
+        if (e < p.rot) {
+          const float2* cs = p.table + t * half;
+          if (V > 1 && !p.halves) {      // both features of every pair are here
+#pragma unroll
+            for (int k = 0; k + 1 < V; k += 2) {
+              const float2 a = cs[(e + k) >> 1];
+              const float u = x[k] * a.x - x[k + 1] * a.y;
+              x[k + 1] = x[k + 1] * a.x + x[k] * a.y;
+              x[k] = u;
+            }
+          } else {
+            const bool second = p.halves ? e >= half : (e & 1) != 0;
+            const int at = p.halves ? (second ? e - half : e + half) : e ^ 1;
+            const int pair = p.halves ? (second ? e - half : e) : e >> 1;
+            float y[V], b[V];
+            ldv<V>(src + at, y);
+            if (w) ldv<V>(w + g * n + at, b);
+#pragma unroll
+            for (int k = 0; k < V; ++k) {
+              const float2 a = cs[pair + k];
+              const float o = y[k] * (w ? f * b[k] : f);
+              x[k] = second ? x[k] * a.x + o * a.y : x[k] * a.x - o * a.y;
+            }
+          }
+        }
+      }
+    } else {      // columns behind the head's features are written as zeros
+#pragma unroll
+      for (int k = 0; k < V; ++k) x[k] = 0.f;
+    }
+    T* dst = kind == 0 ? static_cast<T*>(p.q) + (t * p.H + g) * p.dp : static_cast<T*>(kind == 1 ? p.k_pool : p.v_pool) + (slot * p.G + g) * pitch;
+    stv<V>(dst + e, x);
+  }
+}
+
 // CTA = (row, head), every warp walks every fourth visible position, a lane holds NR features of query, accumulator, key and
 // value; the four running softmaxes and the sink are merged at the end.
 struct GqaParams {
@@ -107,8 +223,10 @@ struct GqaParams {
   const int* row_pos;       // [rows] last visible position; null: ctx[row] - 1
   const int* ctx;
   const void* sink;         // [H] or null
+  const void* gate;         // [rows][ld_gate]: sigmoid(gate) of every output feature, head h's at h * vo, or null
   void* out;                // [rows][H][vo]
-  int H, G, dp, vp, vo, max_blocks, block_size;
+  int H, G, dp, vp, vo, max_blocks, block_size, ld_gate;
+  int window;               // positions a row sees, its own included (0: all)
   float scale;
 };
 template <typename T, int NR>
@@ -129,7 +247,7 @@ __global__ void __launch_bounds__(128) gqa_attn_kernel(const GqaParams p) {
     o[i] = 0.f;
   }
   float m = -INFINITY, l = 0.f;
-  for (int k = warp; k < n; k += 4) {
+  for (int k = (p.window && n > p.window ? n - p.window : 0) + warp; k < n; k += 4) {
     const long long at = (static_cast<long long>(bt[k / p.block_size]) * p.block_size + k % p.block_size) * p.G + g;
     const T* kp = static_cast<const T*>(p.k_pool) + at * p.dp;
     const T* vp = static_cast<const T*>(p.v_pool) + at * p.vp;
@@ -163,8 +281,12 @@ __global__ void __launch_bounds__(128) gqa_attn_kernel(const GqaParams p) {
   }
   const float f = L > 0.f ? 1.f / L : 0.f;
   T* out = static_cast<T*>(p.out) + (static_cast<long long>(row) * p.H + hd) * p.vo;
-  for (int c = threadIdx.x; c < p.vo; c += 128)
-    st(out + c, (w[0] * sm[c] + w[1] * sm[p.vp + c] + w[2] * sm[2 * p.vp + c] + w[3] * sm[3 * p.vp + c]) * f);
+  const T* gate = p.gate ? static_cast<const T*>(p.gate) + static_cast<long long>(row) * p.ld_gate + hd * p.vo : nullptr;
+  for (int c = threadIdx.x; c < p.vo; c += 128) {
+    float o = (w[0] * sm[c] + w[1] * sm[p.vp + c] + w[2] * sm[2 * p.vp + c] + w[3] * sm[3 * p.vp + c]) * f;
+    if (gate) o *= sigmoid<true>(ld(gate + c));
+    st(out + c, o);
+  }
 }
 
 template <typename T, bool kPair>
@@ -223,11 +345,35 @@ extern "C" int rb_attention_inputs(const void* qkv, int ld, const float* table, 
   return pair ? launch_inputs<bf16, true>(p, stm) : launch_inputs<bf16, false>(p, stm);
 }
 
+// q_w, k_w: weights of the norms over all query / key columns (null: none); eps <= 0: no norms; halves: pairs are rot / 2 apart
+extern "C" int rb_projection_inputs(const void* qkv, int ld, const void* q_w, const void* k_w, const float* table, void* q, void* k_pool, void* v_pool,
+                                    const long long* slots, long long pool_rows, int T, int H, int G, int dim, int vdim, int dp, int vp, int rot,
+                                    int halves, float eps, int fp32, cudaStream_t stm) {
+  if (T <= 0) return 0;
+  if (H < 1 || dim < 1 || dp < dim || rot % 2 || rot < 0 || rot > dim || (rot && !table)) return -2;
+  if (ld < H * dim + (k_pool ? G * (dim + vdim) : 0) || (k_pool && (!v_pool || !slots || G < 1 || vdim < 1 || vp < vdim))) return -2;
+  ProjectionParams p{qkv, q_w, k_w, reinterpret_cast<const float2*>(table), q, k_pool, v_pool, slots, pool_rows, H, G, dim, vdim, dp, vp, rot, halves, ld,
+                     eps};
+  const uintptr_t bases = reinterpret_cast<uintptr_t>(qkv) | reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(q_w) |
+                          reinterpret_cast<uintptr_t>(k_w) | reinterpret_cast<uintptr_t>(k_pool) | reinterpret_cast<uintptr_t>(v_pool);
+  const bool vec = dim % 8 == 0 && dp % 8 == 0 && ld % 8 == 0 && rot % (halves ? 16 : 8) == 0 && bases % 16 == 0 &&
+                   (!k_pool || (vdim % 8 == 0 && vp % 8 == 0));
+  if (fp32) {
+    if (vec) projection_inputs_kernel<float, 8><<<T, PI_WARPS * 32, 0, stm>>>(p);
+    else projection_inputs_kernel<float, 1><<<T, PI_WARPS * 32, 0, stm>>>(p);
+  } else {
+    if (vec) projection_inputs_kernel<bf16, 8><<<T, PI_WARPS * 32, 0, stm>>>(p);
+    else projection_inputs_kernel<bf16, 1><<<T, PI_WARPS * 32, 0, stm>>>(p);
+  }
+  rb_note_launch(1);
+  return static_cast<int>(cudaGetLastError());
+}
+
 extern "C" int rb_gqa_attn(const void* q, const void* k_pool, const void* v_pool, const int* block_tables, const int* row_seg, const int* row_pos,
-                           const int* ctx, const void* sink, void* out, int rows, int H, int G, int dp, int vp, int vo, int max_blocks,
-                           int block_size, float scale, int fp32, cudaStream_t stm) {
+                           const int* ctx, const void* sink, const void* gate, int ld_gate, void* out, int rows, int H, int G, int dp, int vp, int vo,
+                           int max_blocks, int block_size, int window, float scale, int fp32, cudaStream_t stm) {
   if (rows <= 0) return 0;
-  if (G < 1 || H % G || vo > vp || H > 65535) return -2;
-  GqaParams p{q, k_pool, v_pool, block_tables, row_seg, row_pos, ctx, sink, out, H, G, dp, vp, vo, max_blocks, block_size, scale};
+  if (G < 1 || H % G || vo > vp || H > 65535 || window < 0 || (gate && ld_gate < H * vo)) return -2;
+  GqaParams p{q, k_pool, v_pool, block_tables, row_seg, row_pos, ctx, sink, gate, out, H, G, dp, vp, vo, max_blocks, block_size, ld_gate, window, scale};
   return fp32 ? launch_gqa<float>(p, rows, stm) : launch_gqa<bf16>(p, rows, stm);
 }

@@ -3,7 +3,7 @@
 // This folds a latent up-projection into the queries (W_h [K][N], read MN-major in place) and applies one to attended
 // latent rows (W_h [N][K]).  CTA = (128 output features, head, 128 tokens): TMA warp (64-deep stages, A through a
 // 3-D map so that x may be a strided slice of a wider projection), MMA warp, four epilogue warps that write rows of the
-// output directly.  The reductions are short (one to eight stages), so CTAs are small and several share an SM.
+// output directly, multiplied by the sigmoid of a gate per output feature when one is given.  The reductions are short (one to eight stages), so CTAs are small and several share an SM.
 #include "common.cuh"
 #include "host_utils.h"
 
@@ -19,7 +19,8 @@ constexpr int TOTAL = BAR + 256;
 
 struct Params {
   __nv_bfloat16* out;      // [T][H][N]
-  int T, H, N, K, kn;
+  const __nv_bfloat16* gate;      // [T][ld_gate], head h's features at h * N, or null
+  int T, H, N, K, kn, ld_gate;
   int* err;
 };
 
@@ -106,6 +107,15 @@ head_gemm_kernel(const __grid_constant__ CUtensorMap tma_x, const __grid_constan
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
           if (n0 + c + i * 8 < p.N) {      // N is a multiple of 8
+            if (p.gate) {
+              const uint4 g = *reinterpret_cast<const uint4*>(p.gate + static_cast<size_t>(t) * p.ld_gate + h * p.N + n0 + c + i * 8);
+              const uint32_t w[4] = {g.x, g.y, g.z, g.w};
+#pragma unroll
+              for (int k = 0; k < 4; ++k) {
+                r[8 * i + 2 * k] = __float_as_uint(__fdividef(__uint_as_float(r[8 * i + 2 * k]), 1.f + __expf(-__uint_as_float(w[k] << 16))));
+                r[8 * i + 2 * k + 1] = __float_as_uint(__fdividef(__uint_as_float(r[8 * i + 2 * k + 1]), 1.f + __expf(-__uint_as_float(w[k] & 0xffff0000u))));
+              }
+            }
             uint4 v;
             v.x = pack_bf16(__uint_as_float(r[8 * i]), __uint_as_float(r[8 * i + 1]));
             v.y = pack_bf16(__uint_as_float(r[8 * i + 2]), __uint_as_float(r[8 * i + 3]));
@@ -130,14 +140,15 @@ head_gemm_kernel(const __grid_constant__ CUtensorMap tma_x, const __grid_constan
 }  // namespace rb
 
 // x [T][H][K] bf16 with strides x_tok, x_head (elements, multiples of 8); w [H][N][K] (kn = 0) or [H][K][N] (kn = 1),
-// contiguous; out [T][H][N] contiguous.  N and K are multiples of 8; returns -20 otherwise.
-extern "C" int rb_head_gemm(const void* x, const void* w, void* out, int T, int H, int N, int K, long long x_tok, long long x_head, int kn, int* err,
-                            cudaStream_t st) {
+// contiguous; out [T][H][N] contiguous.  gate [T][ld_gate >= H N] or null.  N and K are multiples of 8; returns -20 otherwise.
+extern "C" int rb_head_gemm(const void* x, const void* w, const void* gate, int ld_gate, void* out, int T, int H, int N, int K, long long x_tok,
+                            long long x_head, int kn, int* err, cudaStream_t st) {
   using namespace rb;
   using namespace rb::hg;
   if (T <= 0 || H <= 0) return 0;
   if (N % 8 || K % 8 || x_tok % 8 || x_head % 8 || N < 8 || K < 8 || H > 65535 || (T + 127) / 128 > 65535) return -20;
   if ((reinterpret_cast<uintptr_t>(x) % 16) || (reinterpret_cast<uintptr_t>(w) % 16) || (reinterpret_cast<uintptr_t>(out) % 16)) return -20;
+  if (gate && (ld_gate % 8 || ld_gate < H * N || reinterpret_cast<uintptr_t>(gate) % 16)) return -2;
   CUtensorMap tx, tw;
   int rc = encode_tma_3d_16bit(&tx, x, K, H, T, x_head, x_tok, 64, 1, 128);
   if (rc) return rc;
@@ -149,7 +160,7 @@ extern "C" int rb_head_gemm(const void* x, const void* w, void* out, int T, int 
     if (e != cudaSuccess) return static_cast<int>(e);
     attr = true;
   }
-  Params p{static_cast<__nv_bfloat16*>(out), T, H, N, K, kn, err};
+  Params p{static_cast<__nv_bfloat16*>(out), static_cast<const __nv_bfloat16*>(gate), T, H, N, K, kn, ld_gate, err};
   head_gemm_kernel<<<dim3((N + 127) / 128, H, (T + 127) / 128), THREADS, TOTAL, st>>>(tx, tw, p);
   rb_note_launch(1);
   return static_cast<int>(cudaGetLastError());

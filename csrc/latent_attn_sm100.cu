@@ -5,8 +5,10 @@
 // once, so a CTA streams each row once and serves a group of up to N (token, head) query columns with it:
 //
 //   S^T[128 positions][N]   = C_tile[128][R]   * Q^T            (Q: N absorbed queries, K-major)
-//   O^T[R][N]              += C_tile^T[R][128] * P               (the same tile, read MN-major in place)
+//   O^T[Rv][N]             += C_tile^T[Rv][128] * P              (the same tile, read MN-major in place)
 //
+// Rows may end in features that only join the scores (a rotated key part: Rv < R): their slots are free again as soon as S has read
+// them.
 // The columns of a group belong to one sequence: the heads of one decoded token, or of several consecutive tokens of a
 // prompt portion, each with its own causal limit.  Rows are gathered page by page with TMA into the 128-byte swizzled
 // layout; a ring of 32 KB slots (128 positions x 128 latent features) keeps loads in flight while a tile is processed: a
@@ -32,10 +34,12 @@ struct Params {
   const int* block_tables;   // [S][max_blocks]
   const int* ctx;            // [S] (decode)
   const __nv_bfloat16* gate; // [rows][ld_gate] or null
-  __nv_bfloat16* out;        // [columns][R]
-  float* part_o;             // [splits][columns][R]
+  __nv_bfloat16* out;        // [columns][Rv]
+  float* part_o;             // [splits][columns][Rv]
   float* part_ml;            // [splits][columns][2]
-  int H, R, NC, NP, slots, max_blocks, page, splits, columns, groups_per_row, ld_gate, ahead;
+  int H, Rv;
+  int NC, NP, NV;            // 64-feature chunks of a row; slots per tile, the first NV of which hold values
+  int slots, max_blocks, page, splits, columns, groups_per_row, ld_gate, ahead;
   float scale_log2;
   int* err;
 };
@@ -97,7 +101,7 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
   int* s_lim = reinterpret_cast<int*>(s_gate + N);            // [N] positions a column sees
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  constexpr int kTmemCols = N == 16 ? 128 : (N == 32 ? 256 : 512);      // (2 + NP) * N columns, NP <= 4
+  constexpr int kTmemCols = N == 16 ? 128 : (N == 32 ? 256 : 512);      // (2 + NV) * N columns, NV <= 4
   constexpr int T_S = 0, T_O = 2 * N;
 
   int seg, col0, ncols, base;
@@ -220,6 +224,7 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
             for (int kk = 0; kk < 4; ++kk) umma_f16(d, da + (SLOT >> 5) + kk * 2, db + (N * 128 >> 4) + kk * 2, id_s, 1u);
           }
           db += 2 * (N * 128 >> 4);
+          if (pr >= p.NV) umma_commit(&empty[ss]);
           if (++ss == p.slots) { ss = 0; phase ^= 1; }
         }
         umma_commit(&bar_s[j & 1]);
@@ -237,7 +242,7 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
         tc_fence_after();
         const uint64_t db = p0 + static_cast<uint32_t>(j & 1) * (Layout<N>::kP >> 4);
         const uint32_t first = j > 0 ? 1u : 0u;
-        for (int pr = 0; pr < p.NP; ++pr) {
+        for (int pr = 0; pr < p.NV; ++pr) {
           // A: M = 128 latent features (two chunks SLOT / 2 apart), K = 16 positions (2048 bytes).  In the last slot of an odd
           // chunk count the upper 64 rows of the product come from stale data and are never read
           const uint64_t da = ring_mn + static_cast<uint32_t>(so) * (SLOT >> 4);
@@ -248,6 +253,8 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
           umma_commit(&empty[so]);
           if (++so == p.slots) so = 0;
         }
+        for (int pr = p.NV; pr < p.NP; ++pr)
+          if (++so == p.slots) so = 0;
         umma_commit(&bar_o[j & 1]);
         if (!p.ahead && j + 1 < n_tiles && !issue_s(j + 1)) break;
       }
@@ -314,7 +321,7 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
           __syncwarp();
           tc_fence_after();
 #pragma unroll 1
-          for (int pr = 0; pr < p.NP; ++pr) {
+          for (int pr = 0; pr < p.NV; ++pr) {
 #pragma unroll
             for (int c = 0; c < NH; c += CW) {
               uint32_t o[CW];
@@ -367,30 +374,30 @@ latent_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_co
     }
     if (have) {
 #pragma unroll 1
-      for (int pr = 0; pr < p.NP; ++pr) {
+      for (int pr = 0; pr < p.NV; ++pr) {
         const int d = pr * 128 + r;
 #pragma unroll
         for (int c = 0; c < NH; c += CW) {
           uint32_t o[CW];
           tmem_get<CW>(tmem_base + T_O + pr * N + c + lane_addr, o);
           tmem_wait_ld();
-          if (d < p.R) {
+          if (d < p.Rv) {
 #pragma unroll
             for (int i = 0; i < CW; ++i) {
               const int n = n0 + c + i;
               if (n < ncols) {
                 const float v = __uint_as_float(o[i]);
                 if (p.splits == 1)
-                  p.out[static_cast<size_t>(col0 + n) * p.R + d] = __float2bfloat16(ok && l_part[c + i] > 0.f ? v / l_part[c + i] * s_gate[n] : 0.f);
+                  p.out[static_cast<size_t>(col0 + n) * p.Rv + d] = __float2bfloat16(ok && l_part[c + i] > 0.f ? v / l_part[c + i] * s_gate[n] : 0.f);
                 else
-                  p.part_o[(static_cast<size_t>(split) * p.columns + col0 + n) * p.R + d] = v;
+                  p.part_o[(static_cast<size_t>(split) * p.columns + col0 + n) * p.Rv + d] = v;
               }
             }
           }
         }
       }
     } else if (p.splits == 1) {
-      for (int i = threadIdx.x; i < ncols * p.R; i += SOFTMAX) p.out[static_cast<size_t>(col0) * p.R + i] = __float2bfloat16(0.f);
+      for (int i = threadIdx.x; i < ncols * p.Rv; i += SOFTMAX) p.out[static_cast<size_t>(col0) * p.Rv + i] = __float2bfloat16(0.f);
     }
   }
 
@@ -453,28 +460,28 @@ static int launch(const CUtensorMap& tq, const CUtensorMap& tc, const Params& p,
 }  // namespace la
 }  // namespace rb
 
-// q [rows][H][R] bf16 (absorbed queries), pool [pool_rows][R] bf16 in pages of `page` rows (16, 32, 64 or 128), R a multiple
-// of 64 up to 512.  width: columns per group (16, 32 or 64).  items [n_items][4] or null (one row per segment: ctx is read
+// q [rows][H][R] bf16 (absorbed queries), pool [pool_rows][R] bf16 in pages of `page` rows (16, 32, 64 or 128), out [rows][H][Rv]: the
+// first Rv features are values, all R join the scores; both multiples of 64, Rv up to 512, R up to 640.  width: columns per group (16, 32 or 64).  items [n_items][4] or null (one row per segment: ctx is read
 // on the device).  part_o / part_ml: scratch for splits > 1.  Returns -20 for shapes outside this range.
 extern "C" int rb_latent_attn_tc(const void* q, const void* pool, const int* block_tables, const int* items, const int* ctx, const void* gate,
-                                 void* out, float* part_o, float* part_ml, int rows, int H, int R, long long pool_rows, int max_blocks, int page,
+                                 void* out, float* part_o, float* part_ml, int rows, int H, int R, int Rv, long long pool_rows, int max_blocks, int page,
                                  int n_items, int width, int splits, int ld_gate, float scale, int* err, cudaStream_t st) {
   using namespace rb;
   using namespace rb::la;
   if (rows <= 0) return 0;
   if (!(scale > 0.f)) return -20;            // masking relies on the sign
-  if (R % 64 || R > 512 || R < 64 || (page != 16 && page != 32 && page != 64 && page != 128)) return -20;
+  if (R % 64 || R > 640 || Rv % 64 || Rv > 512 || Rv > R || Rv < 64 || (page != 16 && page != 32 && page != 64 && page != 128)) return -20;
   if ((width != 16 && width != 32 && width != 64) || splits < 1 || splits > 32 || (splits > 1 && (!part_o || !part_ml))) return -2;
   if ((reinterpret_cast<uintptr_t>(q) % 16) || (reinterpret_cast<uintptr_t>(pool) % 16)) return -2;
   Params p{};
   p.items = items; p.block_tables = block_tables; p.ctx = ctx;
   p.gate = static_cast<const __nv_bfloat16*>(gate); p.out = static_cast<__nv_bfloat16*>(out); p.part_o = part_o; p.part_ml = part_ml;
-  p.H = H; p.R = R; p.NC = R / 64; p.NP = (p.NC + 1) / 2; p.max_blocks = max_blocks; p.page = page; p.splits = splits;
+  p.H = H; p.Rv = Rv; p.NC = R / 64; p.NP = (p.NC + 1) / 2; p.NV = (Rv / 64 + 1) / 2; p.max_blocks = max_blocks; p.page = page; p.splits = splits;
   p.columns = rows * H; p.groups_per_row = (H + width - 1) / width; p.ld_gate = ld_gate;
   p.scale_log2 = scale * 1.4426950408889634f; p.err = err;
   const int fixed = p.NC * width * 128 + 2 * (2 * width * 128) + SCRATCH;
   p.slots = p.NP == 1 ? 3 : MAX_SLOTS;       // one pair: a small CTA, so that two share an SM
-  while (p.slots * SLOT + fixed > 227 * 1024) --p.slots;
+  while (p.slots > 0 && p.slots * SLOT + fixed > 227 * 1024) --p.slots;
   if (p.slots < p.NP) return -20;
   p.ahead = p.slots >= 2 * p.NP;
   CUtensorMap tq, tc;
@@ -487,7 +494,7 @@ extern "C" int rb_latent_attn_tc(const void* q, const void* pool, const int* blo
   rc = width == 16 ? launch<16>(tq, tc, p, n, smem, st) : width == 32 ? launch<32>(tq, tc, p, n, smem, st) : launch<64>(tq, tc, p, n, smem, st);
   if (rc) return rc;
   if (splits > 1)
-    latent_combine_kernel<<<p.columns, 128, 0, st>>>(part_o, part_ml, p.gate, p.out, splits, p.columns, H, R, ld_gate);
+    latent_combine_kernel<<<p.columns, 128, 0, st>>>(part_o, part_ml, p.gate, p.out, splits, p.columns, H, Rv, ld_gate);
   rb_note_launch(splits > 1 ? 2 : 1);
   return static_cast<int>(cudaGetLastError());
 }

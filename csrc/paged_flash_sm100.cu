@@ -9,10 +9,13 @@
 //   O += P V       V is read in place from its [position][d] tile (MN-major)
 // Keys and values come straight from the pages (TMA, one box per page and 64 columns): new rows are written to the pages before
 // this kernel runs, and nothing is gathered into a dense copy.  The running softmax starts from the head's sink logit
-// (sum = 1 at reference = sink), or empty without one.  S is double buffered, so the product of block j + 1 runs while the
+// (sum = 1 at reference = sink), or empty without one.  With a window a tile starts at the block of the first position that its first
+// row sees, and every row masks what lies before its own.  A gate per output feature is applied in the epilogue.  S is double buffered, so the product of block j + 1 runs while the
 // softmax of block j does.  The accumulator is rescaled only when a row's maximum grows by more than 2^8 (decided per warp: TMEM
 // accesses are warp-wide).  Warps 0-3: softmax and epilogue, warp 4: TMA, warp 5: MMA.  Two CTAs share an SM.  Every wait is
 // bounded; no load uses cluster multicast.
+#include <limits.h>
+
 #include "common.cuh"
 #include "host_utils.h"
 
@@ -44,11 +47,24 @@ struct Params {
   const int* ctx;            // [S]
   const int* block_tables;   // [S][max_blocks]
   const __nv_bfloat16* sink; // [H] or null
+  const __nv_bfloat16* gate; // [rows][ld_gate], head h's features at h * out_d, or null
   __nv_bfloat16* out;        // [rows][H][out_d]
-  int H, G, tokens, max_blocks, page, out_d;
+  int H, G, tokens, max_blocks, page, out_d, ld_gate;
+  int window;                // positions a row sees (INT_MAX: all)
   float scale_log2;
   int* err;
 };
+
+// eight accumulators times sigmoid(gate)
+__device__ __forceinline__ void gate8(uint32_t* o, const __nv_bfloat16* gate) {
+  const uint4 g = *reinterpret_cast<const uint4*>(gate);
+  const uint32_t w[4] = {g.x, g.y, g.z, g.w};
+#pragma unroll
+  for (int k = 0; k < 4; ++k) {
+    o[2 * k] = __float_as_uint(__fdividef(__uint_as_float(o[2 * k]), 1.f + __expf(-__uint_as_float(w[k] << 16))));
+    o[2 * k + 1] = __float_as_uint(__fdividef(__uint_as_float(o[2 * k + 1]), 1.f + __expf(-__uint_as_float(w[k] & 0xffff0000u))));
+  }
+}
 
 template <int DK, int DV>
 __global__ void __launch_bounds__(THREADS, 2)
@@ -80,7 +96,8 @@ paged_flash_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_const
     pos0 = p.ctx[seg] - 1;
   }
   const int seen = pos0 + ntok;                    // positions that the last token of the tile sees
-  const int n_blocks = (seen + BKV - 1) / BKV;
+  const int block0 = max(0, pos0 - p.window + 1) / BKV;      // block of the first position that the first token sees
+  const int n_blocks = (seen + BKV - 1) / BKV - block0;
   const int* bt = p.block_tables + static_cast<size_t>(seg) * p.max_blocks;
 
   if (threadIdx.x == 0) {
@@ -128,7 +145,7 @@ paged_flash_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_const
         uint8_t* sk = smem + L::kK + s * L::kKBytes;
         mbar_expect_tx(&kfull[s], L::kKBytes);
         for (int r = 0; r < BKV; r += rows) {
-          const int pos = j * BKV + r;
+          const int pos = (block0 + j) * BKV + r;
           const int row = bt[min(pos / p.page, p.max_blocks - 1)] * p.page + pos % p.page;
           for (int c = 0; c < DK / 64; ++c) tma_load_3d(sk + c * L::kKVHalf + r * 128, &tma_k, &kfull[s], c * 64, kvh, row);
         }
@@ -136,7 +153,7 @@ paged_flash_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_const
         uint8_t* sv = smem + L::kV + s * L::kVBytes;
         mbar_expect_tx(&vfull[s], L::kVBytes);
         for (int r = 0; r < BKV; r += rows) {
-          const int pos = j * BKV + r;
+          const int pos = (block0 + j) * BKV + r;
           const int row = bt[min(pos / p.page, p.max_blocks - 1)] * p.page + pos % p.page;
           for (int c = 0; c < DV / 64; ++c) tma_load_3d(sv + c * L::kKVHalf + r * 128, &tma_v, &vfull[s], c * 64, kvh, row);
         }
@@ -189,7 +206,8 @@ paged_flash_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_const
     // ================================================================ softmax + epilogue (warps 0..3)
     const int r = warp * 32 + lane;                // row of the tile = TMEM lane
     const int t = r / p.G, head = kvh * p.G + r % p.G;
-    const int limit = pos0 + t + 1;                // positions this row sees
+    const int limit = pos0 + t + 1 - block0 * BKV;             // this row sees positions first .. limit - 1 of the tile's blocks
+    const int first = limit - min(p.window, pos0 + t + 1);
     const bool mine = t < ntok;
     const uint32_t lane_addr = static_cast<uint32_t>(warp * 32) << 16;
     float m_ref = -1e30f, l = 0.f;
@@ -208,15 +226,15 @@ paged_flash_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_const
       tmem_ld_32x32b_x32(tmem_base + T_S + s * BKV + lane_addr, raw);
       tmem_ld_32x32b_x32(tmem_base + T_S + s * BKV + lane_addr + 32, raw + 32);
       tmem_wait_ld();
-      const int lim = limit - j * BKV;             // columns < lim are seen
+      const int lim = limit - j * BKV, low = first - j * BKV;      // columns low .. lim - 1 are seen
       float mx = -1e30f;
-      if (__all_sync(0xffffffffu, lim >= BKV)) {
+      if (__all_sync(0xffffffffu, lim >= BKV && low <= 0)) {
 #pragma unroll
         for (int c = 0; c < 64; ++c) mx = fmaxf(mx, __uint_as_float(raw[c]));
       } else {
 #pragma unroll
         for (int c = 0; c < 64; ++c) {
-          if (c >= lim) raw[c] = 0xff800000u;      // -inf
+          if (c >= lim || c < low) raw[c] = 0xff800000u;      // -inf
           mx = fmaxf(mx, __uint_as_float(raw[c]));
         }
       }
@@ -284,6 +302,7 @@ paged_flash_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_const
 #pragma unroll
           for (int i = 0; i < 4; ++i) {
             if (c * 32 + i * 8 < p.out_d) {
+              if (p.gate) gate8(o + 8 * i, p.gate + static_cast<size_t>(row0 + t) * p.ld_gate + head * p.out_d + c * 32 + i * 8);
               uint4 pk;
               pk.x = pack_bf16(__uint_as_float(o[8 * i]) * inv_l, __uint_as_float(o[8 * i + 1]) * inv_l);
               pk.y = pack_bf16(__uint_as_float(o[8 * i + 2]) * inv_l, __uint_as_float(o[8 * i + 3]) * inv_l);
@@ -333,10 +352,11 @@ static int launch(const void* q, const void* kc, const void* vc, int rows, int H
 }  // namespace rb
 
 // q [rows][Hq][dk], pools [pool_rows][Hkv][dk / dv] (dk, dv: 64 or 128), out [rows][Hq][out_d].  blocks [n][4]: query tiles of at
-// most 128 / (Hq / Hkv) tokens, every row in exactly one (null: n = rows, one row per segment).  Returns -20 for shapes outside that.
+// most 128 / (Hq / Hkv) tokens, every row in exactly one (null: n = rows, one row per segment).  window: positions a row sees, its own
+// included (0: all).  gate [rows][ld_gate] or null.  Returns -20 for shapes outside that.
 extern "C" int rb_paged_flash(const void* q, const void* kc, const void* vc, const int* block_tables, const int* ctx, const int* blocks,
-                              const void* sink, void* out, int rows, int n, int Hq, int Hkv, int dk, int dv, int out_d, long long pool_rows,
-                              int page, int max_blocks, float scale, int* err, cudaStream_t st) {
+                              const void* sink, const void* gate, int ld_gate, void* out, int rows, int n, int Hq, int Hkv, int dk, int dv, int out_d,
+                              long long pool_rows, int page, int max_blocks, int window, float scale, int* err, cudaStream_t st) {
   using namespace rb;
   using namespace rb::pf;
   if (rows <= 0 || n <= 0) return 0;
@@ -344,8 +364,10 @@ extern "C" int rb_paged_flash(const void* q, const void* kc, const void* vc, con
   const int G = Hq / Hkv;
   if (G > BQ || Hkv > 65535 || (dk != 64 && dk != 128) || (dv != 64 && dv != 128) || out_d % 8 || out_d > dv || out_d < 1) return -20;
   if ((page != 16 && page != 32 && page % 64) || scale <= 0.f) return -20;
+  if (window < 0 || (gate && (ld_gate % 8 || ld_gate < Hq * out_d || reinterpret_cast<uintptr_t>(gate) % 16))) return -2;
   Params p{};
   p.blocks = blocks; p.ctx = ctx; p.block_tables = block_tables; p.sink = (const __nv_bfloat16*)sink; p.out = (__nv_bfloat16*)out;
+  p.gate = (const __nv_bfloat16*)gate; p.ld_gate = ld_gate; p.window = window ? window : INT_MAX;
   p.H = Hq; p.G = G; p.tokens = BQ / G; p.max_blocks = max_blocks; p.page = page; p.out_d = out_d;
   p.scale_log2 = scale * 1.4426950408889634f;
   p.err = err;

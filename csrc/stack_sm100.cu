@@ -6,12 +6,15 @@
 //
 //  * embed_rows     token rows -> fp32 residual stream and its 16-bit copy
 //  * norm_add       residual += group norm of a sublayer's output; writes the next sublayer's input (or its final norm); one form
-//                   first sums the weighted rows of a token's experts, one starts the stream with normed embeddings
+//                  first sums the weighted rows of a token's experts, one starts the stream with normed embeddings
+//  * sum_norm       residual = norm(alpha residual + a sublayer's output, weighted expert rows included); writes the next sublayer's input
+//                  (or its final norm)
 //  * hgrn2_step     one token per sequence: gates, state update, read-out and per-head norm in one pass over the state
 //  * hgrn2_scan     segments of any length: the state stays in registers while the tokens stream through shared memory
-//  * latent_write   norm of the latent projection, scattered into the paged latent cache
+//  * latent_write   norm of the latent projection, scattered into the paged latent cache, with the rotation of the part of queries and
+//                  rows that carries positions
 //  * latent_attn    CUDA-core attention over paged latent rows (any sizes, fp32 or bf16)
-//  * glu, gate_heads, and a CUDA-core GEMM for fp32 and for shapes that no tensor-core kernel takes
+//  * glu, gates of attention outputs, and a CUDA-core GEMM for fp32 and for shapes that no tensor-core kernel takes
 #include "stack_common.cuh"
 
 namespace rb {
@@ -20,7 +23,7 @@ namespace stack {
 // ------------------------------------------------------------------------------------------------- embedding
 template <typename T>
 __global__ void embed_rows_kernel(const long long* __restrict__ tok, const T* __restrict__ w, float* __restrict__ res,
-                                  T* __restrict__ h, int vocab, int pitch) {
+                                  T* __restrict__ h, int vocab, int pitch, float scale) {
   const long long t = blockIdx.x;
   const long long id = tok[t];
   const bool ok = id >= 0 && id < vocab;
@@ -29,6 +32,8 @@ __global__ void embed_rows_kernel(const long long* __restrict__ tok, const T* __
 #pragma unroll
     for (int i = 0; i < 8; ++i) v.v[i] = 0.f;
     if (ok) v = ld8(w + id * pitch + c);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) v.v[i] *= scale;
     st8(res + t * pitch + c, v);
     st8(h + t * pitch + c, v);
   }
@@ -58,10 +63,48 @@ struct NormAddParams {
   const int* place;       // [rows][top]
   const int* offset;      // [experts + 1]
   const float* weight;    // [rows][top]
-  int top;
+  int top, experts;       // choices from `experts` on are identity experts: their output is the stream itself
 };
 enum : int { NA_PLAIN = 0, NA_EMBED = 1, NA_SUM = 2 };
 constexpr int NA_MAX_TOP = 64;
+
+// Where the rows of a token's experts lie (shared memory, filled by the whole CTA).
+template <int MAX>
+struct ExpertRows {
+  long long at[MAX];      // first element of a choice's row, -1: identity expert
+  float w[MAX];
+  int top;
+  // returns the sum of the identity experts' weights
+  __device__ __forceinline__ float gather(const int* expert, const int* place, const int* offset, const float* weight, long long row, int n, int experts,
+                                          int pitch) {
+    if (static_cast<int>(threadIdx.x) < n) {
+      const long long i = row * n + threadIdx.x;
+      const int e = expert[i];
+      at[threadIdx.x] = e < experts ? (static_cast<long long>(offset[e]) + place[i]) * pitch : -1;
+      w[threadIdx.x] = weight[i];
+    }
+    if (threadIdx.x == 0) top = n;
+    __syncthreads();
+    float identity = 0.f;
+    for (int k = 0; k < n; ++k) identity += at[k] < 0 ? w[k] : 0.f;
+    return identity;
+  }
+  template <int V, typename T>
+  __device__ __forceinline__ void add(const T* ex, float* a) const {
+    const int n = top;
+#pragma unroll 4
+    for (int k = 0; k < n; ++k) {
+      float b[V];
+      const long long i = at[k];
+#pragma unroll
+      for (int j = 0; j < V; ++j) b[j] = 0.f;
+      if (i >= 0) ldv<V>(ex + i, b);
+      const float f = w[k];
+#pragma unroll
+      for (int j = 0; j < V; ++j) a[j] += f * b[j];
+    }
+  }
+};
 template <typename T, int V, int MODE>
 __global__ void __launch_bounds__(NA_WARPS * 32) norm_add_kernel(const NormAddParams p) {
   __shared__ float red[2][NA_WARPS];
@@ -71,28 +114,21 @@ __global__ void __launch_bounds__(NA_WARPS * 32) norm_add_kernel(const NormAddPa
   const Y* y;
   bool known = true;
   if constexpr (MODE == NA_SUM) {
-    __shared__ long long s_row[NA_MAX_TOP];
-    __shared__ float s_w[NA_MAX_TOP];
-    if (threadIdx.x < p.top) {
-      const long long i = row * p.top + threadIdx.x;
-      s_row[threadIdx.x] = (static_cast<long long>(p.offset[p.expert[i]]) + p.place[i]) * p.ldy;
-      s_w[threadIdx.x] = p.weight[i];
-    }
-    __syncthreads();
+    __shared__ ExpertRows<NA_MAX_TOP> s;
+    const float identity = s.gather(p.expert, p.place, p.offset, p.weight, row, p.top, p.experts, p.ldy);
+    const float* stream = p.res + row * p.pitch;
     const T* base = p.y ? static_cast<const T*>(p.y) + row * p.ldy : nullptr;
     const T* ex = static_cast<const T*>(p.ex);
     for (int c = threadIdx.x * V; c < p.width; c += NA_WARPS * 32 * V) {
-      float a[V];
+      float a[V], x[V];
 #pragma unroll
       for (int i = 0; i < V; ++i) a[i] = 0.f;
       if (base) ldv<V>(base + c, a);
-#pragma unroll 4
-      for (int k = 0; k < p.top; ++k) {
-        float b[V];
-        ldv<V>(ex + s_row[k] + c, b);
-        const float w = s_w[k];
+      s.add<V>(ex + c, a);
+      if (identity != 0.f) {
+        ldv<V>(stream + c, x);
 #pragma unroll
-        for (int i = 0; i < V; ++i) a[i] += w * b[i];
+        for (int i = 0; i < V; ++i) a[i] += identity * x[i];
       }
       stv<V>(ysum + c, a);
     }
@@ -176,6 +212,123 @@ __global__ void __launch_bounds__(NA_WARPS * 32) norm_add_kernel(const NormAddPa
     st(h + c, 0.f);
     if constexpr (MODE == NA_EMBED) st(res + c, 0.f);
   }
+}
+
+// ------------------------------------------------------------------------------------------------- norm of the sum
+// x <- norm(alpha x + y + weighted expert rows) over the whole width.  One CTA per row; the row waits in shared memory between the
+// passes, and every thread reads back only what it wrote itself.  Variances are means of squared deviations.
+struct SumNormParams {
+  float* res;             // [rows][pitch] fp32, updated in place
+  const void* y;          // [rows][ldy] or null
+  const void* ex;         // weighted expert rows as in NormAddParams, or null
+  const int* expert;
+  const int* place;
+  const int* offset;
+  const float* weight;
+  int top, experts;
+  const void* w;          // [pitch]
+  const void* b;          // [pitch] or null
+  const void* next_w;     // [pitch] or null: h is the stream itself
+  const void* next_b;     // [pitch] or null
+  void* h;                // [rows][pitch]
+  int ldy, pitch, width, centre;
+  float alpha, eps, scale;      // scale: factor on h when next_w is given
+};
+template <typename T, int V, bool kExperts>
+__global__ void __launch_bounds__(NA_WARPS * 32) sum_norm_kernel(const SumNormParams p) {
+  extern __shared__ __align__(16) float z[];      // [width]
+  __shared__ float red[4][NA_WARPS];
+  const long long row = blockIdx.x;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, step = NA_WARPS * 32 * V;
+  float* res = p.res + row * p.pitch;
+  const T* y = p.y ? static_cast<const T*>(p.y) + row * p.ldy : nullptr;
+  const T* ex = static_cast<const T*>(p.ex);
+  __shared__ ExpertRows<kExperts ? NA_MAX_TOP : 1> rows;
+  float alpha = p.alpha;
+  if constexpr (kExperts) {
+    alpha += rows.gather(p.expert, p.place, p.offset, p.weight, row, p.top, p.experts, p.ldy);
+  }
+  auto total = [&](float v, int k) {      // over the CTA; every k is used once
+    v = wsum(v);
+    if (lane == 0) red[k][warp] = v;
+    __syncthreads();
+    float s = 0.f;
+#pragma unroll
+    for (int i = 0; i < NA_WARPS; ++i) s += red[k][i];
+    return s;
+  };
+  float sum = 0.f;
+  for (int c = threadIdx.x * V; c < p.width; c += step) {
+    float x[V], a[V];
+    ldv<V>(res + c, x);
+#pragma unroll
+    for (int i = 0; i < V; ++i) x[i] *= alpha;
+    if (y) {
+      ldv<V>(y + c, a);
+#pragma unroll
+      for (int i = 0; i < V; ++i) x[i] += a[i];
+    }
+    if constexpr (kExperts) rows.template add<V>(ex + c, x);
+#pragma unroll
+    for (int i = 0; i < V; ++i) sum += x[i];
+    stv<V>(z + c, x);
+  }
+  const float inv_n = 1.f / p.width;
+  float mean = p.centre ? total(sum, 0) * inv_n : 0.f;
+  float ss = 0.f;
+  for (int c = threadIdx.x * V; c < p.width; c += step) {
+    float x[V];
+    ldv<V>(z + c, x);
+#pragma unroll
+    for (int i = 0; i < V; ++i) ss += (x[i] - mean) * (x[i] - mean);
+  }
+  float r = 1.f / sqrtf(total(ss, 1) * inv_n + p.eps);
+  const T* w = static_cast<const T*>(p.w);
+  const T* b = static_cast<const T*>(p.b);
+  const T* nw = static_cast<const T*>(p.next_w);
+  const T* nb = static_cast<const T*>(p.next_b);
+  T* h = static_cast<T*>(p.h) + row * p.pitch;
+  sum = 0.f;
+  for (int c = threadIdx.x * V; c < p.width; c += step) {
+    float x[V], f[V], g[V];
+    ldv<V>(z + c, x);
+    ldv<V>(w + c, f);
+    if (b) ldv<V>(b + c, g);
+#pragma unroll
+    for (int i = 0; i < V; ++i) {
+      x[i] = (x[i] - mean) * r * f[i];
+      if (b) x[i] += g[i];
+      sum += x[i];
+    }
+    stv<V>(res + c, x);
+    if (nw) stv<V>(z + c, x);
+    else stv<V>(h + c, x);
+  }
+  if (nw) {
+    mean = p.centre ? total(sum, 2) * inv_n : 0.f;
+    ss = 0.f;
+    for (int c = threadIdx.x * V; c < p.width; c += step) {
+      float x[V];
+      ldv<V>(z + c, x);
+#pragma unroll
+      for (int i = 0; i < V; ++i) ss += (x[i] - mean) * (x[i] - mean);
+    }
+    r = 1.f / sqrtf(total(ss, 3) * inv_n + p.eps);
+    for (int c = threadIdx.x * V; c < p.width; c += step) {
+      float x[V], f[V], g[V];
+      ldv<V>(z + c, x);
+      ldv<V>(nw + c, f);
+      if (nb) ldv<V>(nb + c, g);
+#pragma unroll
+      for (int i = 0; i < V; ++i) {
+        x[i] = (x[i] - mean) * r * f[i];
+        if (nb) x[i] += g[i];
+        x[i] *= p.scale;
+      }
+      stv<V>(h + c, x);
+    }
+  }
+  for (int c = p.width + threadIdx.x; c < p.pitch; c += blockDim.x) st(h + c, 0.f);
 }
 
 // ------------------------------------------------------------------------------------------------- HGRN2
@@ -501,26 +654,64 @@ __global__ void __launch_bounds__(256) head_norm_kernel(const float* __restrict_
 }
 
 // ------------------------------------------------------------------------------------------------- latent cache write
+// One CTA per row.  With rot > 0 the row's rotated key part follows the latent features in the pool (at `part`), and the rotated
+// features of every query head, which start at `dim` of its `dk`, turn in place.  Pairs are neighbours.
+struct LatentWriteParams {
+  const void* raw;           // [rows][ld]: latent projection
+  const void* k_rot;         // [rows][ld]: projection of the rotated key part
+  void* q;                   // [rows][ld]: query heads of dk features
+  const void* w;             // [rank]
+  void* pool;                // [pool rows][pitch]
+  const long long* slots;
+  const float2* table;       // [rows][rot / 2]
+  long long pool_rows;
+  int ld, rank, pitch, part, rot, H, dk, dim;
+  float eps;
+};
 template <typename T>
-__global__ void __launch_bounds__(128) latent_write_kernel(const T* __restrict__ raw, int ld_raw, const T* __restrict__ w, T* __restrict__ pool,
-                                                           const long long* __restrict__ slots, long long pool_rows, int rank, int pitch,
-                                                           float eps) {
+__global__ void __launch_bounds__(128) latent_write_kernel(const LatentWriteParams p) {
   __shared__ float red[4];
   const long long t = blockIdx.x;
-  const T* x = raw + t * ld_raw;
+  const T* x = static_cast<const T*>(p.raw) + t * p.ld;
+  const T* w = static_cast<const T*>(p.w);
   float ss = 0.f;
-  for (int c = threadIdx.x; c < rank; c += 128) {
+  for (int c = threadIdx.x; c < p.rank; c += 128) {
     const float v = ld(x + c);
     ss += v * v;
+  }
+  const float2* cs = p.table + t * (p.rot >> 1);
+  if (p.rot) {
+    const int half = p.rot >> 1;
+    T* q = static_cast<T*>(p.q) + t * p.ld + p.dim;
+    for (int i = threadIdx.x; i < p.H * half; i += 128) {
+      const int hd = i / half, k = i - hd * half;
+      T* a = q + hd * p.dk + 2 * k;
+      const float u = ld(a), v = ld(a + 1);
+      const float2 f = cs[k];
+      st(a, u * f.x - v * f.y);
+      st(a + 1, v * f.x + u * f.y);
+    }
   }
   ss = wsum(ss);
   if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
   __syncthreads();
-  const float r = 1.f / sqrtf((red[0] + red[1] + red[2] + red[3]) / rank + eps);
-  const long long s = slots[t];
-  if (s < 0 || s >= pool_rows) return;
-  T* d = pool + s * pitch;
-  for (int c = threadIdx.x; c < pitch; c += 128) st(d + c, c < rank ? ld(x + c) * r * ld(w + c) : 0.f);
+  const float r = 1.f / sqrtf((red[0] + red[1] + red[2] + red[3]) / p.rank + p.eps);
+  const long long s = p.slots[t];
+  if (s < 0 || s >= p.pool_rows) return;
+  T* d = static_cast<T*>(p.pool) + s * p.pitch;
+  const T* kr = static_cast<const T*>(p.k_rot) + t * p.ld;
+  for (int c = threadIdx.x; c < p.pitch; c += 128) {
+    float v = 0.f;
+    if (c < p.rank) {
+      v = ld(x + c) * r * ld(w + c);
+    } else if (c >= p.part && c - p.part < p.rot) {
+      const int i = c - p.part;
+      const float2 f = cs[i >> 1];
+      const float a = ld(kr + (i & ~1)), b = ld(kr + (i | 1));
+      v = (i & 1) ? b * f.x + a * f.y : a * f.x - b * f.y;
+    }
+    st(d + c, v);
+  }
 }
 
 // ------------------------------------------------------------------------------------------------- latent attention
@@ -528,19 +719,19 @@ __global__ void __launch_bounds__(128) latent_write_kernel(const T* __restrict__
 // latent features of query, accumulator and current row; the four running softmaxes are merged at the end.
 struct LatentParams {
   const void* q;          // [rows][H][R]
-  const void* pool;       // [pool rows][R]
+  const void* pool;       // [pool rows][R]; the first Rv features are the values
   const int* block_tables;
   const int* row_seg;     // [rows] or null (row = sequence)
   const int* row_pos;     // [rows] last visible position; null: ctx[row] - 1
   const int* ctx;
   const void* gate;       // [rows][ld_gate] or null
-  void* out;              // [rows][H][R]
-  int H, R, max_blocks, block_size, ld_gate;
+  void* out;              // [rows][H][Rv]
+  int H, R, Rv, max_blocks, block_size, ld_gate;
   float scale;
 };
 template <typename T, int NR>
 __global__ void __launch_bounds__(128) latent_attn_kernel(const LatentParams p) {
-  extern __shared__ float sm[];                 // [4][R] accumulators
+  extern __shared__ float sm[];                 // [4][Rv] accumulators
   __shared__ float sml[4][2];
   const int row = blockIdx.x, hd = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int seg = p.row_seg ? p.row_seg[row] : row;
@@ -575,7 +766,7 @@ __global__ void __launch_bounds__(128) latent_attn_kernel(const LatentParams p) 
   if (lane == 0) { sml[warp][0] = m; sml[warp][1] = l; }
 #pragma unroll
   for (int i = 0; i < NR; ++i)
-    if (lane + 32 * i < p.R) sm[warp * p.R + lane + 32 * i] = o[i];
+    if (lane + 32 * i < p.Rv) sm[warp * p.Rv + lane + 32 * i] = o[i];
   __syncthreads();
   const float M = fmaxf(fmaxf(sml[0][0], sml[1][0]), fmaxf(sml[2][0], sml[3][0]));
   float w[4], L = 0.f;
@@ -586,22 +777,30 @@ __global__ void __launch_bounds__(128) latent_attn_kernel(const LatentParams p) 
   }
   float f = L > 0.f ? 1.f / L : 0.f;
   if (p.gate) f *= sigmoid<true>(ld(static_cast<const T*>(p.gate) + static_cast<long long>(row) * p.ld_gate + hd));
-  T* out = static_cast<T*>(p.out) + (static_cast<long long>(row) * p.H + hd) * p.R;
-  for (int c = threadIdx.x; c < p.R; c += 128)
-    st(out + c, (w[0] * sm[c] + w[1] * sm[p.R + c] + w[2] * sm[2 * p.R + c] + w[3] * sm[3 * p.R + c]) * f);
+  T* out = static_cast<T*>(p.out) + (static_cast<long long>(row) * p.H + hd) * p.Rv;
+  for (int c = threadIdx.x; c < p.Rv; c += 128)
+    st(out + c, (w[0] * sm[c] + w[1] * sm[p.Rv + c] + w[2] * sm[2 * p.Rv + c] + w[3] * sm[3 * p.Rv + c]) * f);
 }
 
-// flash-attention output [T][H][128] -> [T][H * dv], scaled per head by sigmoid(gate)
+// attention output [T][H][pitch] -> [T][H * dv] (which may be the same memory), scaled by the sigmoid of a gate per head or (features)
+// per output feature
 template <typename T>
-__global__ void gate_heads_kernel(const T* __restrict__ o, const T* __restrict__ gate, int ld_gate, T* __restrict__ out, int H, int dv) {
+__global__ void gate_heads_kernel(const T* o, const T* __restrict__ gate, int ld_gate, T* out, int H, int pitch, int dv, int features) {
+  constexpr bool kExact = IsExact<T>::v;
   const long long t = blockIdx.x;
   const int per = dv / 8;
   for (int i = threadIdx.x; i < H * per; i += blockDim.x) {
     const int h = i / per, c = (i - h * per) * 8;
-    const float g = sigmoid<true>(ld(gate + t * ld_gate + h));
-    F8 v = ld8(o + (t * H + h) * 128 + c);
+    F8 v = ld8(o + (t * H + h) * pitch + c);
+    if (features) {
+      const F8 g = ld8(gate + t * ld_gate + h * dv + c);
 #pragma unroll
-    for (int k = 0; k < 8; ++k) v.v[k] *= g;
+      for (int k = 0; k < 8; ++k) v.v[k] *= sigmoid<kExact>(g.v[k]);
+    } else {
+      const float g = sigmoid<true>(ld(gate + t * ld_gate + h));
+#pragma unroll
+      for (int k = 0; k < 8; ++k) v.v[k] *= g;
+    }
     st8(out + (t * H + h) * dv + c, v);
   }
 }
@@ -681,7 +880,7 @@ __global__ void __launch_bounds__(256) simt_gemm_kernel(const GemmParams p) {
 
 template <typename T>
 static int launch_latent_attn(const LatentParams& p, int rows, cudaStream_t stm) {
-  const size_t smem = 4 * static_cast<size_t>(p.R) * 4;
+  const size_t smem = 4 * static_cast<size_t>(p.Rv) * 4;
   const dim3 grid(rows, p.H);
   if (p.R <= 128) latent_attn_kernel<T, 4><<<grid, 128, smem, stm>>>(p);
   else if (p.R <= 256) latent_attn_kernel<T, 8><<<grid, 128, smem, stm>>>(p);
@@ -717,12 +916,13 @@ using namespace rb;
 using namespace rb::stack;
 typedef __nv_bfloat16 bf16;
 
-extern "C" int rb_embed_rows(const long long* tok, const void* w, float* res, void* h, int rows, int vocab, int pitch, int fp32, cudaStream_t stm) {
+extern "C" int rb_embed_rows(const long long* tok, const void* w, float* res, void* h, int rows, int vocab, int pitch, float scale, int fp32,
+                             cudaStream_t stm) {
   if (rows <= 0) return 0;
   if (pitch % 8) return -2;
   const int thr = pitch / 8 < 256 ? (pitch / 8 + 31) / 32 * 32 : 256;
-  if (fp32) embed_rows_kernel<float><<<rows, thr, 0, stm>>>(tok, (const float*)w, res, (float*)h, vocab, pitch);
-  else embed_rows_kernel<bf16><<<rows, thr, 0, stm>>>(tok, (const bf16*)w, res, (bf16*)h, vocab, pitch);
+  if (fp32) embed_rows_kernel<float><<<rows, thr, 0, stm>>>(tok, (const float*)w, res, (float*)h, vocab, pitch, scale);
+  else embed_rows_kernel<bf16><<<rows, thr, 0, stm>>>(tok, (const bf16*)w, res, (bf16*)h, vocab, pitch, scale);
   rb_note_launch(1);
   return static_cast<int>(cudaGetLastError());
 }
@@ -753,12 +953,38 @@ extern "C" int rb_norm_add(float* res, const void* y, const void* w, const void*
 
 // y may be null; ex [sorted rows][ldy] are expert outputs (see NormAddParams), offset has one entry more than there are experts
 extern "C" int rb_norm_add_experts(float* res, const void* y, const void* ex, const int* expert, const int* place, const int* offset,
-                                   const float* weight, int top, const void* w, const void* next_w, void* h, int rows, int ldy, int pitch,
-                                   int width, int groups, float eps, int fp32, cudaStream_t stm) {
+                                   const float* weight, int top, int experts, const void* w, const void* next_w, void* h, int rows, int ldy,
+                                   int pitch, int width, int groups, float eps, int fp32, cudaStream_t stm) {
   if (rows <= 0) return 0;
   if (groups < 1 || width % groups || pitch < width || pitch % 8 || ldy % 8 || top < 1 || top > NA_MAX_TOP) return -2;
-  NormAddParams p{res, y, w, next_w, h, ldy, pitch, width, groups, 1, eps, nullptr, 0, ex, expert, place, offset, weight, top};
+  NormAddParams p{res, y, w, next_w, h, ldy, pitch, width, groups, 1, eps, nullptr, 0, ex, expert, place, offset, weight, top, experts};
   return launch_norm_add<NA_SUM>(p, rows, (width / groups) % 8 == 0, fp32, stm);
+}
+
+template <bool kExperts>
+static int launch_sum_norm(const SumNormParams& p, int rows, int fp32, cudaStream_t stm) {
+  const bool vec = p.width % 8 == 0;
+  const size_t smem = static_cast<size_t>(p.width) * 4;
+  auto k = fp32 ? (vec ? sum_norm_kernel<float, 8, kExperts> : sum_norm_kernel<float, 1, kExperts>)
+                : (vec ? sum_norm_kernel<bf16, 8, kExperts> : sum_norm_kernel<bf16, 1, kExperts>);
+  if (smem > 40 * 1024) {
+    if (smem > 200 * 1024) return -2;
+    const cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
+    if (e != cudaSuccess) return static_cast<int>(e);
+  }
+  k<<<rows, NA_WARPS * 32, smem, stm>>>(p);
+  rb_note_launch(1);
+  return static_cast<int>(cudaGetLastError());
+}
+
+// y may be null, and so may ex (see rb_norm_add_experts), b, next_w and next_b; centre: layer norm, else RMS
+extern "C" int rb_sum_norm(float* res, const void* y, const void* ex, const int* expert, const int* place, const int* offset, const float* weight,
+                           int top, int experts, const void* w, const void* b, const void* next_w, const void* next_b, void* h, int rows, int ldy,
+                           int pitch, int width, int centre, float alpha, float eps, float scale, int fp32, cudaStream_t stm) {
+  if (rows <= 0) return 0;
+  if (width < 1 || pitch < width || pitch % 8 || ldy % 8 || ldy < width || (!y && !ex) || (ex && (top < 1 || top > NA_MAX_TOP))) return -2;
+  SumNormParams p{res, y, ex, expert, place, offset, weight, top, experts, w, b, next_w, next_b, h, ldy, pitch, width, centre, alpha, eps, scale};
+  return ex ? launch_sum_norm<true>(p, rows, fp32, stm) : launch_sum_norm<false>(p, rows, fp32, stm);
 }
 
 // the stream starts with the normed rows of the embedding table
@@ -791,28 +1017,38 @@ extern "C" int rb_hgrn2(const void* qfv, const void* f_bias, const void* lower, 
   return static_cast<int>(cudaGetLastError());
 }
 
-extern "C" int rb_latent_write(const void* raw, int ld_raw, const void* w, void* pool, const long long* slots, long long pool_rows, int rows, int rank,
-                               int pitch, float eps, int fp32, cudaStream_t stm) {
+// rot > 0: k_rot and q (see LatentWriteParams) share the pitch ld of raw; part: column of the rotated key part in the pool
+extern "C" int rb_latent_write(const void* raw, const void* k_rot, void* q, int ld, const void* w, void* pool, const long long* slots,
+                               const float* table, long long pool_rows, int rows, int rank, int pitch, int part, int rot, int H, int dk, int dim,
+                               float eps, int fp32, cudaStream_t stm) {
   if (rows <= 0) return 0;
-  if (rank < 1 || pitch < rank) return -2;
-  if (fp32) latent_write_kernel<float><<<rows, 128, 0, stm>>>((const float*)raw, ld_raw, (const float*)w, (float*)pool, slots, pool_rows, rank, pitch, eps);
-  else latent_write_kernel<bf16><<<rows, 128, 0, stm>>>((const bf16*)raw, ld_raw, (const bf16*)w, (bf16*)pool, slots, pool_rows, rank, pitch, eps);
+  if (rank < 1 || pitch < rank || rot < 0 || rot % 2) return -2;
+  if (rot && (!k_rot || !q || !table || part < rank || pitch < part + rot || H < 1 || dim < 0 || dk < dim + rot)) return -2;
+  LatentWriteParams p{raw, k_rot, q, w, pool, slots, reinterpret_cast<const float2*>(table), pool_rows, ld, rank, pitch, part, rot, H, dk, dim, eps};
+  if (fp32) latent_write_kernel<float><<<rows, 128, 0, stm>>>(p);
+  else latent_write_kernel<bf16><<<rows, 128, 0, stm>>>(p);
   rb_note_launch(1);
   return static_cast<int>(cudaGetLastError());
 }
 
 extern "C" int rb_latent_attn(const void* q, const void* pool, const int* block_tables, const int* row_seg, const int* row_pos, const int* ctx,
-                              const void* gate, void* out, int rows, int H, int R, int max_blocks, int block_size, int ld_gate, float scale,
+                              const void* gate, void* out, int rows, int H, int R, int Rv, int max_blocks, int block_size, int ld_gate, float scale,
                               int fp32, cudaStream_t stm) {
   if (rows <= 0) return 0;
-  LatentParams p{q, pool, block_tables, row_seg, row_pos, ctx, gate, out, H, R, max_blocks, block_size, ld_gate, scale};
+  if (Rv < 1 || Rv > R) return -2;
+  LatentParams p{q, pool, block_tables, row_seg, row_pos, ctx, gate, out, H, R, Rv, max_blocks, block_size, ld_gate, scale};
   return fp32 ? launch_latent_attn<float>(p, rows, stm) : launch_latent_attn<bf16>(p, rows, stm);
 }
 
-extern "C" int rb_gate_heads(const void* o, const void* gate, int ld_gate, void* out, int rows, int H, int dv, cudaStream_t stm) {
+// o [rows][H][pitch] -> out [rows][H * dv]; features: a gate per output feature ([rows][ld_gate >= H dv]), else one per head.  o and out may be
+// the same memory when pitch == dv.
+extern "C" int rb_gate_heads(const void* o, const void* gate, int ld_gate, void* out, int rows, int H, int pitch, int dv, int features, int fp32,
+                             cudaStream_t stm) {
   if (rows <= 0) return 0;
-  if (dv % 8 || dv > 128) return -2;
-  gate_heads_kernel<bf16><<<rows, 256, 0, stm>>>((const bf16*)o, (const bf16*)gate, ld_gate, (bf16*)out, H, dv);
+  if (dv % 8 || dv > pitch || pitch % 8 || ld_gate < (features ? H * dv : H)) return -2;
+  if (features && (ld_gate % 8 || reinterpret_cast<uintptr_t>(gate) % 16)) return -2;
+  if (fp32) gate_heads_kernel<float><<<rows, 256, 0, stm>>>((const float*)o, (const float*)gate, ld_gate, (float*)out, H, pitch, dv, features);
+  else gate_heads_kernel<bf16><<<rows, 256, 0, stm>>>((const bf16*)o, (const bf16*)gate, ld_gate, (bf16*)out, H, pitch, dv, features);
   rb_note_launch(1);
   return static_cast<int>(cudaGetLastError());
 }

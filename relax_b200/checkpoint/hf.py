@@ -569,7 +569,8 @@ def validate_against_hf(cfg: ModelConfig, path: str) -> None:
         return
     hf = config_from_hf(path)
     if cfg.is_composed or hf.is_composed:
-        names = ("layer_specs", "hidden_size", "vocab_size", "norm_groups", "rms_norm_eps", "embed_norm", "tie_word_embeddings")
+        names = ("layer_specs", "hidden_size", "vocab_size", "norm_groups", "norm_sum", "sum_alpha", "rms_norm_eps", "embed_norm", "embed_scale",
+                 "logit_scale", "tie_word_embeddings")
         diff = [f"{n}: {getattr(cfg, n)} here, {getattr(hf, n)} in the checkpoint" for n in names if getattr(cfg, n) != getattr(hf, n)]
         if diff:
             raise ValueError("the model configuration does not match the checkpoint: " + "; ".join(diff))

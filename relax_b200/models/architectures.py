@@ -3,9 +3,9 @@ tensor names: ``name -> module`` with ``config_from_dict(d, name, dtype)`` and `
 Checkpoints without the key are read as Hugging Face layouts (:mod:`relax_b200.checkpoint.hf`)."""
 from __future__ import annotations
 
-from . import ketolorn, talizen
+from . import ketolorn, talizen, zupupel
 
-ARCHITECTURES = {m.ARCHITECTURE: m for m in (talizen, ketolorn)}
+ARCHITECTURES = {m.ARCHITECTURE: m for m in (talizen, ketolorn, zupupel)}
 
 
 def architecture_of(config_json: dict):

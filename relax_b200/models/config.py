@@ -30,10 +30,13 @@ class VisionConfig:
 
 @dataclass(frozen=True)
 class MoESpec:
-    """Routed feed-forward of a composed layer: ``experts`` ungated feed-forwards ``down(act(up h))`` of width ``ff``, of which
-    every token takes ``top`` by the sigmoid of its router logits.  The experts form ``groups`` equal groups of neighbours; only
-    those of the ``keep`` groups with the largest sums of their two best scores can be taken.  ``shared_ff``: width of one
-    more feed-forward of the same form that every token takes with weight one (0 = none)."""
+    """Routed feed-forward of a composed layer: ``experts`` small feed-forwards of width ``ff``, of which every token takes ``top`` by
+    the ``score`` (sigmoid or softmax) of its router logits.  ``act`` ``relu2``: ``down(relu(up h)^2)``; ``clamped_swish``:
+    ``down(g sigmoid(1.702 g) (u + 1))`` with ``g = min(gate h, limit)`` and ``u = up h`` clamped to ``+- limit``.  ``identity``
+    more router outputs stand for experts without weights whose output is ``h`` itself.  All outputs form ``groups`` equal
+    groups of neighbours; only those of the ``keep`` groups whose ``group_best`` best scores have the largest sums can be taken.
+    ``correction``: a learned offset per output that joins the scores for the choice, not for the weights.  ``shared_ff``: width of
+    one more (``relu2``) feed-forward that every token takes with weight one (0 = none)."""
     experts: int
     top: int
     ff: int
@@ -43,33 +46,55 @@ class MoESpec:
     act: str = "relu2"
     renormalize: bool = False    # weights divided by their sum over the taken experts
     weight_scale: float = 1.0    # factor on the weights
+    score: str = "sigmoid"
+    correction: bool = False
+    identity: int = 0
+    group_best: int = 2
+    limit: float = 0.0           # clamped_swish only
 
     def __post_init__(self):
-        if min(self.experts, self.top, self.ff, self.groups, self.keep) < 1 or self.shared_ff < 0 or self.act not in ACTIVATIONS:
+        if min(self.experts, self.top, self.ff, self.groups, self.keep) < 1 or min(self.shared_ff, self.identity) < 0 \
+                or self.act not in EXPERT_ACTIVATIONS or self.score not in ("sigmoid", "softmax") or self.group_best not in (1, 2):
             raise ValueError(f"bad expert layer: {self}")
-        if self.experts % self.groups or self.keep > self.groups or self.top > self.experts // self.groups * self.keep:
-            raise ValueError(f"{self.top} of {self.experts} experts cannot be taken from {self.keep} of {self.groups} groups")
+        if (self.act == "clamped_swish") != (self.limit > 0) or (self.gated and self.shared_ff):
+            raise ValueError(f"bad expert activation: {self}")
+        if self.outputs % self.groups or self.keep > self.groups or self.top > self.outputs // self.groups * self.keep:
+            raise ValueError(f"{self.top} of {self.outputs} experts cannot be taken from {self.keep} of {self.groups} groups")
+
+    @property
+    def outputs(self) -> int:
+        """Outputs of the router: experts, then identity experts."""
+        return self.experts + self.identity
+
+    @property
+    def gated(self) -> bool:
+        return self.act == "clamped_swish"
 
 
 @dataclass(frozen=True)
 class LayerSpec:
     """One layer of a composed stack (``ModelConfig.layer_specs``): its token mixer with the mixer's sizes and its
     feed-forward.  ``hgrn2``: gated linear recurrence with ``heads`` states of ``dim x vdim``.  ``latent_attention``:
-    softmax attention whose keys and values are projections of one cached latent row of ``kv_rank`` features per token.
-    ``attention``: softmax attention over cached keys and values of ``kv_heads`` heads."""
+    softmax attention whose keys and values are projections of one cached latent row of ``kv_rank`` features per token;
+    with ``rot_dims`` every head's query has that many rotated features more, which meet ONE rotated key part that the row
+    holds for all heads.  ``attention``: softmax attention over cached keys and values of ``kv_heads`` heads."""
     mixer: str
     heads: int
-    dim: int                     # query (and key / forget-gate) features per head
+    dim: int                     # query (and key / forget-gate) features per head (latent_attention: the unrotated ones)
     vdim: int                    # value features per head
     kv_rank: int = 0             # latent_attention only
     scale: float = 1.0           # attention mixers: factor on q . k
     ff: int = 0                  # width of the gated feed-forward; 0 = the layer has none
     act: str = "gelu_tanh"       # activation of the feed-forward's gate half
+    out_gate: bool = False       # attention mixers: a gate per output feature, sigmoid(W_g h); latent_attention without: one per head
+    rot_dims: int = 0            # rotated features of queries and keys (attention: the leading ones of a head)
+    rot_base: float = 0.0        # pair i turns by position * rot_base ** (-2 i / rot_dims)
     # attention only
     kv_heads: int = 0            # query head h reads key / value head h // (heads / kv_heads)
-    rot_dims: int = 0            # leading features of queries and keys that are rotated, in neighbouring pairs
-    rot_base: float = 0.0        # pair i turns by position * rot_base ** (-2 i / rot_dims)
-    qk_norm: bool = False        # rotated queries and keys divided by their root mean square
+    rot_halves: bool = False     # pairs are features i and i + rot_dims / 2 instead of neighbours
+    qk_norm: bool = False        # rotated queries and keys divided by their root mean square, head by head
+    proj_norm: bool = False      # weighted RMS norm over all query rows, and over all key rows, before heads and rotation
+    window: int = 0              # a position sees itself and the window - 1 before it; 0 = all before it
     sink: bool = False           # one learned logit per head in the softmax denominator, without key or value
     kv_from: int = -1            # >= 0: reads the keys and values that this earlier layer has cached, and has none of its own
     moe: Optional[MoESpec] = None  # routed feed-forward instead of the gated one
@@ -77,15 +102,19 @@ class LayerSpec:
     def __post_init__(self):
         if self.mixer not in MIXERS:
             raise ValueError(f"unknown mixer {self.mixer!r}; known: {MIXERS}")
-        if min(self.heads, self.dim, self.vdim) < 1 or (self.mixer == "latent_attention" and self.kv_rank < 1) or self.ff < 0:
+        if min(self.heads, self.dim, self.vdim) < 1 or (self.mixer == "latent_attention" and self.kv_rank < 1) or min(self.ff, self.window) < 0:
             raise ValueError(f"bad layer sizes: {self}")
         if self.act not in ACTIVATIONS[:2] or (self.moe is not None and self.ff):
             raise ValueError(f"bad feed-forward: {self}")
+        if self.rot_dims % 2 or self.rot_dims < 0 or (self.rot_dims and self.rot_base <= 0):
+            raise ValueError(f"bad rotation: {self.rot_dims} features, base {self.rot_base}")
         if self.mixer == "attention":
             if self.kv_heads < 1 or self.heads % self.kv_heads:
                 raise ValueError(f"{self.kv_heads} key / value heads do not divide {self.heads} heads")
-            if self.rot_dims % 2 or not 0 <= self.rot_dims <= self.dim or (self.rot_dims and self.rot_base <= 0):
+            if self.rot_dims > self.dim:
                 raise ValueError(f"bad rotation: {self.rot_dims} of {self.dim} features, base {self.rot_base}")
+            if self.qk_norm and (self.proj_norm or self.rot_halves):
+                raise ValueError("queries and keys normed head by head turn in neighbouring pairs and have no norm over the projection")
 
     @property
     def has_ff(self) -> bool:
@@ -99,6 +128,7 @@ class LayerSpec:
 
 MIXERS = ("hgrn2", "latent_attention", "attention")
 ACTIVATIONS = ("silu", "gelu_tanh", "relu2")
+EXPERT_ACTIVATIONS = ("relu2", "clamped_swish")
 
 
 @dataclass
@@ -164,12 +194,17 @@ class ModelConfig:
     dsa_index_heads: int = 4
     dsa_index_dim: int = 16
     dsa_indexer_loss_coef: float = 1.0
-    # composed stacks (Talizen, Ketolorn): every layer is spelled out - mixer, sizes, feed-forward.  The sublayers read the fp32
-    # residual stream itself and their OUTPUT is normed (RMS over each of `norm_groups` equal parts) before it is added.
+    # composed stacks (Talizen, Ketolorn, Zupupel): every layer is spelled out - mixer, sizes, feed-forward.  The sublayers read the
+    # fp32 residual stream itself.  Their OUTPUT is normed (RMS over each of `norm_groups` equal parts) before it is added, or,
+    # with `norm_sum`, the SUM is: x <- norm(sum_alpha * x + sublayer(x)), a layer norm with weight and bias (as is the final norm).
     # The fields above that describe one uniform layer (heads, head_dim, ffn, rotary, MoE, ...) do not apply then.
     layer_specs: Optional[tuple] = None
     norm_groups: int = 1
+    norm_sum: bool = False
+    sum_alpha: float = 1.0
     embed_norm: bool = False               # the embedded tokens are normed before the first layer
+    embed_scale: float = 1.0               # factor on the embedded tokens
+    logit_scale: float = 1.0               # factor on the logits
     dtype: str = "bf16"
 
     @property
@@ -203,17 +238,21 @@ class ModelConfig:
     def num_parameters(self) -> int:
         h, L = self.hidden_size, self.num_layers
         if self.is_composed:
-            n = (1 if self.tie_word_embeddings else 2) * self.vocab_size * h + h + (h if self.embed_norm else 0)
+            norm = 2 * h if self.norm_sum else h
+            n = (1 if self.tie_word_embeddings else 2) * self.vocab_size * h + norm + (h if self.embed_norm else 0)
             for s in self.layer_specs:
-                n += h + 3 * s.ff * h + (h if s.has_ff else 0) + s.heads * s.vdim * h
+                n += norm + 3 * s.ff * h + (norm if s.has_ff else 0) + s.heads * s.vdim * h
                 if s.moe is not None:
-                    n += s.moe.experts * (h + 2 * s.moe.ff * h) + 2 * s.moe.shared_ff * h
+                    n += s.moe.experts * (3 if s.moe.gated else 2) * s.moe.ff * h + 2 * s.moe.shared_ff * h
+                    n += s.moe.outputs * (h + (1 if s.moe.correction else 0))
                 if s.mixer == "hgrn2":
                     n += s.heads * (2 * s.dim + s.vdim) * h + 2 * s.heads * s.dim + s.vdim
                 elif s.mixer == "attention":
                     n += s.heads * s.dim * h + (s.heads if s.sink else 0) + (s.kv_heads * (s.dim + s.vdim) * h if s.own_kv else 0)
+                    n += (s.heads * s.vdim * h if s.out_gate else 0) + ((s.heads + (s.kv_heads if s.own_kv else 0)) * s.dim if s.proj_norm else 0)
                 else:
-                    n += (s.heads * (s.dim + 1) + s.kv_rank) * h + s.kv_rank * (1 + s.heads * (s.dim + s.vdim))
+                    n += (s.heads * (s.dim + s.rot_dims + (s.vdim if s.out_gate else 1)) + s.kv_rank + s.rot_dims) * h
+                    n += s.kv_rank * (1 + s.heads * (s.dim + s.vdim))
             return n
         attn = h * (self.q_size * (2 if self.attention_output_gate else 1) + 2 * self.kv_size) + self.q_size * h
         if self.qk_layernorm:
@@ -246,15 +285,30 @@ def composed_config(name: str, layers, hidden_size: int, vocab_size: int, norm_g
         raise ValueError("a composed stack needs at least one layer")
     if norm_groups < 1 or hidden_size % norm_groups:
         raise ValueError(f"{norm_groups} norm groups do not divide the width {hidden_size}")
+    if kw.get("norm_sum") and (norm_groups > 1 or kw.get("embed_norm")):
+        raise ValueError("norms after the sum span the whole width, and leave the embedded tokens as they are")
+    if not kw.get("norm_sum") and (kw.get("sum_alpha", 1.0) != 1.0 or kw.get("logit_scale", 1.0) != 1.0):
+        raise ValueError("factors on the stream and on the logits join the norm after the sum")
+    if kw.get("embed_norm") and kw.get("embed_scale", 1.0) != 1.0:
+        raise ValueError("embedded tokens are normed or scaled")
     for i, s in enumerate(layers):
         if s.mixer == "attention" and s.kv_from >= 0:
             if s.kv_from >= i or not layers[s.kv_from].own_kv:
                 raise ValueError(f"layer {i} reads keys and values of layer {s.kv_from}, which has none before it")
-            what = ("kv_heads", "dim", "vdim", "rot_dims", "rot_base", "qk_norm")
+            what = ("kv_heads", "dim", "vdim", "rot_dims", "rot_base", "rot_halves", "qk_norm", "proj_norm")
             if any(getattr(s, f) != getattr(layers[s.kv_from], f) for f in what):
                 raise ValueError(f"layer {i} and the layer {s.kv_from} whose keys and values it reads differ in {what}")
     return ModelConfig(name=name, num_layers=len(layers), hidden_size=hidden_size, vocab_size=vocab_size, rms_norm_eps=eps,
                        layer_specs=layers, norm_groups=norm_groups, qk_layernorm=False, **kw)
+
+
+def window_latent_layers(n_layers: int, att: LayerSpec, lat: LayerSpec, moe: Optional[MoESpec]) -> tuple:
+    """Runs of three layers: ``att``, ``lat``, and ``att`` on the keys and values of the run's first layer; ``moe`` in all of them."""
+    out = []
+    for i in range(n_layers):
+        s = lat if i % 3 == 1 else (att if i % 3 == 0 else replace(att, kv_from=i - 2))
+        out.append(replace(s, moe=moe))
+    return tuple(out)
 
 
 def talizen_layers(n_layers: int, every: int, rec: LayerSpec, att: LayerSpec) -> tuple:
@@ -388,6 +442,21 @@ _reg(composed_config("ketolorn-16b", shared_kv_layers(
                       act="silu"),
     8192, MoESpec(experts=128, top=8, ff=1024, groups=8, keep=4, shared_ff=2048)), hidden_size=2048, vocab_size=64000, eps=1e-6, embed_norm=True,
     tie_word_embeddings=True))
+
+# Zupupel: sliding-window attention, latent attention with a rotated key part, upper window layers on the keys and values of a lower
+# one, experts beside identity experts, norms after the sum
+_reg(composed_config("tiny-zupupel", window_latent_layers(
+    6, LayerSpec("attention", heads=6, dim=24, vdim=32, kv_heads=3, scale=0.2, rot_dims=12, rot_base=1e4, rot_halves=True, proj_norm=True, window=20,
+                 out_gate=True),
+    LayerSpec("latent_attention", heads=4, dim=24, vdim=20, kv_rank=40, scale=0.18, rot_dims=16, rot_base=1e4, out_gate=True),
+    MoESpec(experts=7, top=2, ff=40, groups=3, keep=2, act="clamped_swish", limit=2.0, renormalize=True, score="softmax", correction=True, identity=2,
+            group_best=1)), hidden_size=160, vocab_size=320, eps=1e-6, norm_sum=True, sum_alpha=1.8, embed_scale=2.0, logit_scale=0.5, dtype="fp32"))
+_reg(composed_config("zupupel-15b", window_latent_layers(
+    24, LayerSpec("attention", heads=32, dim=128, vdim=128, kv_heads=4, scale=128 ** -0.5, rot_dims=64, rot_base=1e6, rot_halves=True, proj_norm=True,
+                  window=1024, out_gate=True),
+    LayerSpec("latent_attention", heads=32, dim=128, vdim=128, kv_rank=512, scale=192 ** -0.5, rot_dims=64, rot_base=1e6, out_gate=True),
+    MoESpec(experts=128, top=8, ff=768, groups=8, keep=4, act="clamped_swish", limit=7.0, renormalize=True, score="softmax", correction=True, identity=16,
+            group_best=1)), hidden_size=2048, vocab_size=64000, eps=1e-6, norm_sum=True, sum_alpha=48 ** 0.25, embed_scale=45.0, logit_scale=1 / 45))
 
 
 def get_config(name: str, **overrides) -> ModelConfig:

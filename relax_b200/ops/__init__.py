@@ -73,15 +73,23 @@ def linear_fp32(x, w):
     return _cuda().linear_fp32(x, w) if _use_cuda(x) else ref.linear(x.float(), w.float())
 
 
-def embed_rows(tokens, w, norm_w=None, width=0, groups=1, eps=0.0):
-    """Embedded tokens as the fp32 residual stream and its copy in the weights' type, normed in groups with ``norm_w``."""
-    return (_cuda() if _use_cuda(w) else ref).embed_rows(tokens, w, norm_w, width, groups, eps)
+def embed_rows(tokens, w, norm_w=None, width=0, groups=1, eps=0.0, scale=1.0):
+    """Embedded tokens as the fp32 residual stream and its copy in the weights' type: normed in groups with ``norm_w``, or times
+    ``scale`` without."""
+    return (_cuda() if _use_cuda(w) else ref).embed_rows(tokens, w, norm_w, width, groups, eps, scale)
 
 
 def norm_add(res, y, w, width, groups, eps, next_w=None, experts=None):
     """Output norm in groups + add to the fp32 residual stream (in place) + the next sublayer's input, one kernel.
     ``experts``: ``(rows, plan)`` of :func:`moe_experts`, whose weighted sum joins ``y`` in the same pass."""
     return (_cuda() if _use_cuda(res) else ref).norm_add(res, y, w, width, groups, eps, next_w, experts)
+
+
+def sum_norm(res, y, w, b, width, alpha, eps, nxt=None, scale=1.0, experts=None):
+    """``res <- norm(alpha res + y)`` in place (fp32), a layer norm with weight and bias (RMS when ``b`` is None), and the next
+    sublayer's input, one kernel; ``nxt``: ``(weight, bias)`` of the model's last norm, which then gives the result, times ``scale``.
+    ``experts``: as for :func:`norm_add`."""
+    return (_cuda() if _use_cuda(res) else ref).sum_norm(res, y, w, b, width, alpha, eps, nxt, scale, experts)
 
 
 def rope_table(positions, offset, inv_freq):
@@ -94,12 +102,20 @@ def attention_inputs(qkv, table, heads, kv_heads, dim, vdim, dp, rot_dims, eps, 
     return (_cuda() if _use_cuda(qkv) else ref).attention_inputs(qkv, table, heads, kv_heads, dim, vdim, dp, rot_dims, eps, k_pool, v_pool, slots)
 
 
-def paged_attention(q, k_pool, v_pool, batch, block_size, scale, sink, out_width):
+def projection_inputs(qkv, q_w, k_w, table, heads, kv_heads, dim, vdim, dp, rot_dims, halves, eps, k_pool, v_pool, slots):
+    """The same with weighted RMS norms over ALL query columns and over all key columns (``eps`` <= 0: none), then the rotation, of
+    neighbours or (``halves``) of features ``rot_dims / 2`` apart."""
+    return (_cuda() if _use_cuda(qkv) else ref).projection_inputs(qkv, q_w, k_w, table, heads, kv_heads, dim, vdim, dp, rot_dims, halves, eps, k_pool,
+                                                                  v_pool, slots)
+
+
+def paged_attention(q, k_pool, v_pool, batch, block_size, scale, sink, out_width, window=0, gate=None):
     """Grouped-query attention over paged keys and values for every segment of a
-    :class:`relax_b200.rollout.composed.SegmentBatch`, with an optional sink logit per head."""
+    :class:`relax_b200.rollout.composed.SegmentBatch`, with an optional sink logit per head, an optional ``window`` (positions a
+    row sees, its own included; 0 = all) and an optional ``gate`` per output feature (``[T, heads * out_width]``, its sigmoid counts)."""
     if _use_cuda(q):
-        return _cuda().paged_attention(q, k_pool, v_pool, batch, block_size, scale, sink, out_width)
-    return ref.paged_attention(q, k_pool, v_pool, batch.block_tables, block_size, batch.ctx, batch.cu, scale, sink, out_width)
+        return _cuda().paged_attention(q, k_pool, v_pool, batch, block_size, scale, sink, out_width, window, gate)
+    return ref.paged_attention(q, k_pool, v_pool, batch.block_tables, block_size, batch.ctx, batch.cu, scale, sink, out_width, window, gate)
 
 
 def route_counters(layers: int, experts: int, device):
@@ -108,17 +124,28 @@ def route_counters(layers: int, experts: int, device):
     return _cuda().route_counters(layers, experts, device) if on_gpu else [None] * layers
 
 
-def moe_route(logits, spec, dtype, count=None):
+def moe_route(logits, spec, dtype, count=None, correction=None):
     """Expert choice of every row (:class:`relax_b200.models.config.MoESpec`) from fp32 logits; ``dtype``: of the experts' operands;
-    ``count``: an unused row of :func:`route_counters`."""
+    ``count``: an unused row of :func:`route_counters`; ``correction``: offsets of the scores for the choice."""
     if _use_cuda(logits):
-        return _cuda().moe_route(logits, spec, 64 if dtype == torch.float32 else 128, count)      # rows per tile of the grouped GEMM
-    return ref.moe_route(logits, spec)
+        return _cuda().moe_route(logits, spec, 64 if dtype == torch.float32 else 128, count, correction)      # rows per tile of the grouped GEMM
+    return ref.moe_route(logits, spec, correction)
 
 
-def moe_experts(h, plan, up, down, act):
-    """The chosen experts' outputs, unweighted, in an order :func:`norm_add` understands."""
-    return (_cuda() if _use_cuda(h) else ref).moe_experts(h, plan, up, down, act)
+GLU_RUN = 32      # rows of one half that lie side by side in a gated expert's up-projection
+
+
+def glu_rows(gate, up):
+    """Rows ``[..., F, K]`` of the two halves of gated experts in the order of the grouped GEMM's epilogue: runs of :data:`GLU_RUN`
+    gate rows, each followed by the up rows of the same features (``F`` is a multiple of it)."""
+    s = (*gate.shape[:-2], gate.shape[-2] // GLU_RUN, GLU_RUN, gate.shape[-1])
+    return torch.stack([gate.reshape(s), up.reshape(s)], -3).reshape(*gate.shape[:-2], 2 * gate.shape[-2], gate.shape[-1])
+
+
+def moe_experts(h, plan, up, down, act, limit=0.0):
+    """The chosen experts' outputs, unweighted, in an order :func:`norm_add` understands.  ``act`` ``clamped_swish``: ``up`` is made by
+    :func:`glu_rows`, and ``limit`` bounds both halves."""
+    return (_cuda() if _use_cuda(h) else ref).moe_experts(h, plan, up, down, act, limit)
 
 
 def hgrn2(qfv, f_bias, lower, norm_w, state, state_slot, ctx_lens, cu, heads, dim, vdim, eps, spans=None):
@@ -129,24 +156,33 @@ def hgrn2(qfv, f_bias, lower, norm_w, state, state_slot, ctx_lens, cu, heads, di
     return ref.hgrn2(qfv, f_bias, lower, norm_w, state, state_slot, ctx_lens, cu, heads, dim, vdim, eps)
 
 
-def latent_write(raw, w, rank, eps, pool, slots):
-    """Norm of the latent projection + write of the new rows into the paged latent cache."""
-    (_cuda() if _use_cuda(raw) else ref).latent_write(raw, w, rank, eps, pool, slots)
+def latent_write(raw, w, rank, eps, pool, slots, turned=None):
+    """Norm of the latent projection + write of the new rows into the paged latent cache.  ``turned``: ``(q, k_rot, table, part, rot,
+    dim)`` - the rotated key part ``k_rot`` goes to the rows' columns ``part ..``, and features ``dim .. dim + rot`` of every query head
+    ``q[T, H, dk]`` turn in place (both pair by pair of neighbours)."""
+    (_cuda() if _use_cuda(raw) else ref).latent_write(raw, w, rank, eps, pool, slots, turned)
 
 
-def head_linear(x, w, transposed):
-    """One small linear map per head (folds a latent up-projection into the queries / applies it to attended latents)."""
-    return (_cuda() if _use_cuda(x) else ref).head_linear(x, w, transposed)
+def head_linear(x, w, transposed, gate=None):
+    """One small linear map per head (folds a latent up-projection into the queries / applies it to attended latents), every output
+    feature scaled by ``sigmoid(gate)`` when given (``[T, heads * out]``)."""
+    return (_cuda() if _use_cuda(x) else ref).head_linear(x, w, transposed, gate)
 
 
-def latent_attention(q, pool, batch, block_size, scale, gate):
+def latent_columns(row: int, rank: int) -> int:
+    """Columns per group that :func:`relax_b200.rollout.composed.attention_items` makes for latent rows of this size."""
+    return _cuda().latent_columns(row, rank) or 64
+
+
+def latent_attention(q, pool, batch, block_size, scale, gate, rank=None):
     """Attention of absorbed queries over paged latent rows for the short segments of a
-    :class:`relax_b200.rollout.composed.SegmentBatch`, head outputs scaled by ``sigmoid(gate)``."""
+    :class:`relax_b200.rollout.composed.SegmentBatch`; the first ``rank`` features of a row (all of them) are also the values.  Head outputs are
+    scaled by ``sigmoid(gate)`` (``[T, H]``) when given."""
     if _use_cuda(q):
-        return _cuda().latent_attention(q, pool, batch, block_size, scale, gate)
+        return _cuda().latent_attention(q, pool, batch, block_size, scale, gate, rank)
     n = batch.long_segs
     cu = batch.short_cu if n else batch.cu
-    return ref.latent_attention(q, pool, batch.block_tables[n:], block_size, batch.ctx[n:], cu, scale, gate)
+    return ref.latent_attention(q, pool, batch.block_tables[n:], block_size, batch.ctx[n:], cu, scale, gate, rank)
 
 
 def flash_serves_dims(dtype, dk: int, dv: int) -> bool:
@@ -154,10 +190,10 @@ def flash_serves_dims(dtype, dk: int, dv: int) -> bool:
     return not _force_ref() and dtype == torch.bfloat16 and max(dk, dv) <= 128
 
 
-def flash_gated(q, k, v, cu_q, cu_k, scale, max_q, gate):
-    """Causal varlen attention on per-head keys / values whose widths may differ, every head's output scaled by
-    ``sigmoid(gate)``; returns ``[T, H * dv]``."""
-    return _cuda().flash_gated(q, k, v, cu_q, cu_k, scale, max_q, gate)
+def flash_gated(q, k, v, cu_q, cu_k, scale, max_q, gate, features=False):
+    """Causal varlen attention on per-head keys / values whose widths may differ, every head's output (``features``: every output
+    feature) scaled by ``sigmoid(gate)``; returns ``[T, H * dv]``."""
+    return _cuda().flash_gated(q, k, v, cu_q, cu_k, scale, max_q, gate, features)
 
 
 def linear(x, w, bias=None):

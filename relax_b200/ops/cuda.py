@@ -328,11 +328,11 @@ def linear_fp32(x, w):
 # --------------------------------------------------------------------------- composed stacks (inference)
 
 
-def embed_rows(tokens, w, norm_w=None, width=0, groups=1, eps=0.0):
+def embed_rows(tokens, w, norm_w=None, width=0, groups=1, eps=0.0, scale=1.0):
     res = torch.empty(tokens.shape[0], w.shape[1], dtype=torch.float32, device=w.device)
     h = torch.empty(tokens.shape[0], w.shape[1], dtype=w.dtype, device=w.device)
     if norm_w is None:
-        _load().embed_rows(tokens, w, res, h)
+        _load().embed_rows(tokens, w, res, h, float(scale))
     else:
         _load().embed_norm(tokens, w, norm_w, res, h, int(width), int(groups), float(eps))
     return res, h
@@ -348,6 +348,15 @@ def norm_add(res, y, w, width, groups, eps, next_w=None, experts=None):
     return h
 
 
+def sum_norm(res, y, w, b, width, alpha, eps, nxt=None, scale=1.0, experts=None):
+    h = torch.empty(res.shape, dtype=w.dtype, device=w.device)
+    rows, plan = experts if experts is not None else (None, None)
+    e = (None,) * 4 if plan is None else (plan.expert, plan.place, plan.offset, plan.weight)
+    _load().sum_norm(res, y, rows, *e, w, b, *(nxt if nxt is not None else (None, None)), h, int(width), b is not None, float(alpha), float(eps),
+                     float(scale))
+    return h
+
+
 def rope_table(positions, offset, inv_freq):
     out = torch.empty(positions.shape[0], inv_freq.shape[0], 2, dtype=torch.float32, device=positions.device)
     _load().rope_table(positions, int(offset), inv_freq, out)
@@ -357,6 +366,12 @@ def rope_table(positions, offset, inv_freq):
 def attention_inputs(qkv, table, heads, kv_heads, dim, vdim, dp, rot_dims, eps, k_pool, v_pool, slots):
     q = torch.empty(qkv.shape[0], heads, dp, dtype=qkv.dtype, device=qkv.device)
     _load().attention_inputs(qkv, table, q, k_pool, v_pool, slots, int(kv_heads), int(dim), int(vdim), int(rot_dims), float(eps))
+    return q
+
+
+def projection_inputs(qkv, q_w, k_w, table, heads, kv_heads, dim, vdim, dp, rot_dims, halves, eps, k_pool, v_pool, slots):
+    q = torch.empty(qkv.shape[0], heads, dp, dtype=qkv.dtype, device=qkv.device)
+    _load().projection_inputs(qkv, q_w, k_w, table, q, k_pool, v_pool, slots, int(kv_heads), int(dim), int(vdim), int(rot_dims), bool(halves), float(eps))
     return q
 
 
@@ -371,7 +386,7 @@ def decode_splits(rows: int, kv_heads: int, max_ctx: int) -> int:
     return splits
 
 
-def paged_attention(q, k_pool, v_pool, b, block_size, scale, sink, out_width):
+def paged_attention(q, k_pool, v_pool, b, block_size, scale, sink, out_width, window=0, gate=None):
     """bf16 heads of up to 128 features: segments of several rows on the flash kernel, single rows on the decode kernel (the
     flash kernel when more than 16 heads share keys); anything else, and fp32, on CUDA cores."""
     T, H, dp = q.shape
@@ -380,24 +395,26 @@ def paged_attention(q, k_pool, v_pool, b, block_size, scale, sink, out_width):
     out = torch.empty(T, H * out_width, dtype=q.dtype, device=q.device)
     n, s = (0, 0) if b.cu is None else (b.multi_rows, b.multi_segs)
     if q.dtype == torch.bfloat16 and max(dp, v_pool.shape[2]) <= 128 and H // G <= 128:
-        ok = n == 0 or L.paged_flash(q[:n], k_pool, v_pool, b.block_tables, b.ctx, b.blocks[128 // (H // G)], sink, out[:n], int(block_size),
-                                     float(scale), err)
+        ok = n == 0 or L.paged_flash(q[:n], k_pool, v_pool, b.block_tables, b.ctx, b.blocks[128 // (H // G)], sink,
+                                     None if gate is None else gate[:n], out[:n], int(block_size), int(window), float(scale), err)
         if ok and n == T:
             return out
         if ok:
-            bt, ctx = b.block_tables[s:], b.ctx[s:]
+            bt, ctx, g = b.block_tables[s:], b.ctx[s:], None if gate is None else gate[n:]
             if H // G <= 16:
-                splits = decode_splits(T - n, G, b.max_ctx_one)
+                most = min(b.max_ctx_one, window + block_size) if window else b.max_ctx_one
+                splits = decode_splits(T - n, G, most)
                 po = ml = None
                 if splits > 1:
                     po = torch.empty(splits * (T - n) * H * 128, dtype=torch.float32, device=q.device)
                     ml = torch.empty(splits * (T - n) * H * 2, dtype=torch.float32, device=q.device)
-                ok = L.paged_decode(q[n:], k_pool, v_pool, bt, ctx, sink, out[n:], po, ml, int(block_size), int(b.max_ctx_one), splits, float(scale), err)
+                ok = L.paged_decode(q[n:], k_pool, v_pool, bt, ctx, sink, g, out[n:], po, ml, int(block_size), int(most), int(window), splits,
+                                    float(scale), err)
             else:
-                ok = L.paged_flash(q[n:], k_pool, v_pool, bt, ctx, None, sink, out[n:], int(block_size), float(scale), err)
+                ok = L.paged_flash(q[n:], k_pool, v_pool, bt, ctx, None, sink, g, out[n:], int(block_size), int(window), float(scale), err)
             if ok:
                 return out
-    L.gqa_attn(q, k_pool, v_pool, b.block_tables, b.seg_of, b.pos, b.ctx, sink, out, int(block_size), float(scale))
+    L.gqa_attn(q, k_pool, v_pool, b.block_tables, b.seg_of, b.pos, b.ctx, sink, gate, out, int(block_size), int(window), float(scale))
     return out
 
 
@@ -411,7 +428,7 @@ def route_counters(layers, experts, device):
     return torch.zeros(layers, experts + 1, dtype=torch.int32, device=device)
 
 
-def moe_route(logits, spec, tile_rows, count=None):
+def moe_route(logits, spec, tile_rows, count=None, correction=None):
     T, E, k, dev = logits.shape[0], spec.experts, spec.top, logits.device
     p = ExpertPlan()
     i32 = lambda *s: torch.empty(*s, dtype=torch.int32, device=dev)
@@ -420,8 +437,8 @@ def moe_route(logits, spec, tile_rows, count=None):
     p.tiles = i32(min(T * k, E) + T * k // tile_rows, 4)
     if count is None:
         count = route_counters(1, E, dev)[0]
-    _load().moe_route(logits, p.expert, p.weight, p.place, p.row_token, count, p.offset, p.tiles, p.n_tiles, E, spec.groups, spec.keep, tile_rows,
-                      bool(spec.renormalize), float(spec.weight_scale))
+    _load().moe_route(logits, correction, p.expert, p.weight, p.place, p.row_token, count, p.offset, p.tiles, p.n_tiles, E, spec.outputs, spec.groups,
+                      spec.keep, spec.group_best, tile_rows, bool(spec.renormalize), spec.score == "softmax", float(spec.weight_scale))
     return p
 
 
@@ -431,16 +448,18 @@ def _moe_plan(rows: int, experts: int, n: int) -> tuple:
     return (256 if tiles * ((n + 255) // 256) >= 296 else 128), rows >= 16 * experts
 
 
-def moe_experts(h, plan, up, down, act):
-    """Sorted expert rows ``[T top, W]``: gather, up-projection and activation in one grouped GEMM, down-projection in a second."""
-    if act != "relu2":
-        raise ValueError(f"no ungated activation {act!r}")
-    R, E, err = plan.expert.numel(), up.shape[0], err_flag(h.device)
-    mid = torch.empty(R, up.shape[1], dtype=h.dtype, device=h.device)
+EXPERT_ACT = {"relu2": 1, "clamped_swish": 2}
+
+
+def moe_experts(h, plan, up, down, act, limit=0.0):
+    """Sorted expert rows ``[T top, W]``: gather, up-projection and activation in one grouped GEMM, down-projection in a second.
+    Gated experts: ``up`` holds gate and up rows in alternating runs (:func:`relax_b200.ops.glu_rows`)."""
+    R, E, err, code = plan.expert.numel(), up.shape[0], err_flag(h.device), EXPERT_ACT[act]
+    mid = torch.empty(R, up.shape[1] // code, dtype=h.dtype, device=h.device)
     out = torch.empty(R, down.shape[1], dtype=h.dtype, device=h.device)
     L = _load()
-    L.moe_gemm(h, up, mid, plan.tiles, plan.n_tiles, plan.row_token, 1, *_moe_plan(R, E, up.shape[1]), err)
-    L.moe_gemm(mid, down, out, plan.tiles, plan.n_tiles, None, 0, *_moe_plan(R, E, down.shape[1]), err)
+    L.moe_gemm(h, up, mid, plan.tiles, plan.n_tiles, plan.row_token, code, float(limit), *_moe_plan(R, E, up.shape[1]), err)
+    L.moe_gemm(mid, down, out, plan.tiles, plan.n_tiles, None, 0, 0.0, *_moe_plan(R, E, down.shape[1]), err)
     return out
 
 
@@ -460,39 +479,56 @@ def hgrn2(qfv, f_bias, lower, norm_w, state, state_slot, ctx_lens, cu, heads, di
     return out
 
 
-def latent_write(raw, w, rank, eps, pool, slots):
-    _load().latent_write(raw, w, pool, slots, int(rank), float(eps))
+def latent_write(raw, w, rank, eps, pool, slots, turned=None):
+    if turned is None:
+        _load().latent_write(raw, None, None, None, w, pool, slots, int(rank), 0, 0, 0, float(eps))
+    else:
+        q, k_rot, table, part, rot, dim = turned
+        _load().latent_write(raw, k_rot, q, table, w, pool, slots, int(rank), int(part), int(rot), int(dim), float(eps))
 
 
-def head_linear(x, w, transposed):
+def head_linear(x, w, transposed, gate=None):
     T, H, _ = x.shape
     out = torch.empty(T, H, w.shape[1] if transposed else w.shape[2], dtype=x.dtype, device=x.device)
-    if x.dtype == torch.bfloat16 and _load().head_gemm(x, w, out, not transposed, err_flag(x.device)):
+    if x.dtype == torch.bfloat16 and _load().head_gemm(x, w, gate, out, not transposed, err_flag(x.device)):
         return out
     _load().simt_gemm(x.transpose(0, 1), w, out.transpose(0, 1), not transposed)      # 32-bit mode
+    if gate is not None:
+        _load().gate_heads(out, gate, out, out.shape[2], True)
     return out
 
 
 LATENT_TILE = 128      # positions per tile of the tensor-core latent attention
 
 
-def latent_attention(q, pool, b, block_size, scale, gate):
+def latent_columns(row: int, rank: int) -> int:
+    """Most (token, head) columns a CTA of the tensor-core latent attention serves: 64, fewer when the queries of that many and the
+    tiles of one step (``row`` features, the first ``rank`` of them values) do not fit its shared memory together; 0: rows too wide."""
+    if row % 64 or rank % 64 or row > 640 or rank > 512:
+        return 0
+    pairs = (row // 64 + 1) // 2
+    return next((n for n in (64, 32, 16) if pairs * 32768 + row // 64 * n * 128 + 512 * n + 2560 <= 227 * 1024), 0)
+
+
+def latent_attention(q, pool, b, block_size, scale, gate, rank=None):
     """Tensor cores for bf16 with ranks up to 512 and pages of 16 to 128 tokens, CUDA cores otherwise (32-bit mode)."""
     q = q.contiguous()
-    out = torch.empty_like(q)
     T, H, R = q.shape
+    rank = rank or R
+    out = torch.empty(T, H, rank, dtype=q.dtype, device=q.device)
     n = b.long_segs
     bt, ctx = b.block_tables[n:], b.ctx[n:]
-    if q.dtype == torch.bfloat16 and R <= 512 and block_size in (16, 32, 64, 128):
+    most = latent_columns(R, rank) if q.dtype == torch.bfloat16 and block_size in (16, 32, 64, 128) else 0
+    if most:
         items = b.items[H] if b.items is not None else None
         if items is None and b.cu is not None:
             raise ValueError("a batch of segments needs its column groups (attention_items)")
-        width = 64 if items is not None or H > 32 else (16 if H <= 16 else 32)
+        width = (b.item_width or {}).get(H, 64) if items is not None else min(most, 64 if H > 32 else (16 if H <= 16 else 32))
         groups = items.shape[0] if items is not None else T * ((H + width - 1) // width)
         splits = max(1, min(148 // groups, (b.max_ctx + LATENT_TILE - 1) // LATENT_TILE, 32))
         po = ml = None
         if splits > 1:
-            po = torch.empty(splits * T * H * R, dtype=torch.float32, device=q.device)
+            po = torch.empty(splits * T * H * rank, dtype=torch.float32, device=q.device)
             ml = torch.empty(splits * T * H * 2, dtype=torch.float32, device=q.device)
         if _load().latent_attn_tc(q, pool, bt, items, ctx, gate, out, po, ml, int(block_size), width, splits, float(scale), err_flag(q.device)):
             return out
@@ -500,14 +536,14 @@ def latent_attention(q, pool, b, block_size, scale, gate):
     return out
 
 
-def flash_gated(q, k, v, cu_q, cu_k, scale, max_q, gate):
+def flash_gated(q, k, v, cu_q, cu_k, scale, max_q, gate, features=False):
     F = torch.nn.functional
     dk, dv = q.shape[-1], v.shape[-1]
     q, k = (t if dk == 128 else F.pad(t, (0, 128 - dk)) for t in (q, k))
     v = v if dv == 128 else F.pad(v, (0, 128 - dv))
     o = attention_varlen(q, k, v, cu_q, True, scale, cu_k, max_q)
     out = torch.empty(q.shape[0], q.shape[1] * dv, dtype=q.dtype, device=q.device)
-    _load().gate_heads(o, gate, out, int(dv))
+    _load().gate_heads(o, gate, out, int(dv), bool(features))
     return out
 
 

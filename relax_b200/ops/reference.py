@@ -57,11 +57,13 @@ def group_rms(x, w, width: int, groups: int, eps: float):
     return y
 
 
-def embed_rows(tokens, w, norm_w=None, width: int = 0, groups: int = 1, eps: float = 0.0):
-    """``(fp32 residual stream, its copy in the weights' type)`` of embedded tokens, group-normed when ``norm_w`` is given."""
+def embed_rows(tokens, w, norm_w=None, width: int = 0, groups: int = 1, eps: float = 0.0, scale: float = 1.0):
+    """``(fp32 residual stream, its copy in the weights' type)`` of embedded tokens, group-normed when ``norm_w`` is given, else times
+    ``scale``."""
     h = w[tokens]
     if norm_w is None:
-        return h.float(), h
+        res = h.float() * scale
+        return res, res.to(w.dtype, copy=True)
     res = group_rms(h.float(), norm_w, width, groups, eps)
     return res, res.to(w.dtype)
 
@@ -71,11 +73,37 @@ def norm_add(res, y, w, width: int, groups: int, eps: float, next_w=None, expert
     itself, or its own group norm with ``next_w`` when given.  ``experts = (rows, plan)``: the weighted rows of
     :func:`moe_experts` join ``y`` (which may be None) first."""
     if experts is not None:
-        rows, plan = experts
-        z = (rows.float() * plan.weight[..., None]).sum(1)
+        z = expert_sum(res, experts)
         y = z if y is None else y.float() + z
     res += group_rms(y, w, width, groups, eps)
     return (res if next_w is None else group_rms(res, next_w, width, groups, eps)).to(w.dtype)
+
+
+def expert_sum(res, experts):
+    """Weighted sum over a token's experts; identity experts (choices behind the last expert) give back the stream itself."""
+    rows, plan = experts
+    z = (rows.float() * plan.weight[..., None]).sum(1)
+    return z + res * (plan.weight * (plan.index >= plan.experts)).sum(1, keepdim=True)
+
+
+def sum_norm(res, y, w, b, width: int, alpha: float, eps: float, nxt=None, scale: float = 1.0, experts=None):
+    """``res <- norm(alpha res + y + experts)`` over the first ``width`` columns, in place (fp32): a layer norm with weight ``w`` and bias
+    ``b``, RMS when ``b`` is None.  Returns the new stream in ``w``'s type, or its norm with ``nxt = (weight, bias)`` times ``scale``."""
+    def norm(x, w, b):
+        if b is not None:
+            x = x - x.mean(-1, keepdim=True)
+        x = x / torch.sqrt(x.pow(2).mean(-1, keepdim=True) + eps) * w[:width].float()
+        return x if b is None else x + b[:width].float()
+
+    x = alpha * res[:, :width]
+    if y is not None:
+        x = x + y[:, :width].float()
+    if experts is not None:
+        x = x + expert_sum(res, experts)[:, :width]
+    res[:, :width] = norm(x, w, b)
+    h = torch.zeros(res.shape, dtype=w.dtype, device=res.device)
+    h[:, :width] = res[:, :width] if nxt is None else norm(res[:, :width], *nxt) * scale
+    return h
 
 
 def hgrn2(qfv, f_bias, lower, norm_w, state, state_slot, ctx_lens, cu, heads: int, dim: int, vdim: int, eps: float):
@@ -103,25 +131,42 @@ def hgrn2(qfv, f_bias, lower, norm_w, state, state_slot, ctx_lens, cu, heads: in
     return o.to(qfv.dtype)
 
 
-def latent_write(raw, w, rank: int, eps: float, pool, slots):
-    """RMS-normed latent rows -> ``pool[slots]`` (columns behind ``rank`` zero)."""
+def turn_neighbours(x, table):
+    """Pairs of neighbouring features ``x[T, ..., 2 n]`` turned by ``table[T, n, 2]`` (cos, sin)."""
+    c, s = (table[..., k].view(table.shape[0], *[1] * (x.dim() - 2), -1) for k in (0, 1))
+    u, v = x[..., 0::2], x[..., 1::2]
+    return torch.stack([u * c - v * s, v * c + u * s], -1).flatten(-2)
+
+
+def latent_write(raw, w, rank: int, eps: float, pool, slots, turned=None):
+    """RMS-normed latent rows -> ``pool[slots]`` (columns behind ``rank`` zero, but for the rotated key part of ``turned``, whose query
+    features turn in place)."""
     c = torch.zeros(raw.shape[0], pool.shape[1], dtype=torch.float32, device=raw.device)
     x = raw[:, :rank].float()
     c[:, :rank] = x / torch.sqrt(x.pow(2).mean(-1, keepdim=True) + eps) * w[:rank].float()
+    if turned is not None:
+        q, k_rot, table, part, rot, dim = turned
+        c[:, part:part + rot] = turn_neighbours(k_rot[:, :rot].float(), table)
+        q[..., dim:dim + rot] = turn_neighbours(q[..., dim:dim + rot].float(), table).to(q.dtype)
     pool[slots] = c.to(pool.dtype)
 
 
-def head_linear(x, w, transposed: bool):
-    """Per-head product ``x[T, H, a] -> [T, H, b]`` with ``w[H, a, b]`` (``transposed``: ``w[H, b, a]``)."""
-    return torch.einsum("tha,hba->thb" if transposed else "tha,hab->thb", x.float(), w.float()).to(w.dtype)
+def head_linear(x, w, transposed: bool, gate=None):
+    """Per-head product ``x[T, H, a] -> [T, H, b]`` with ``w[H, a, b]`` (``transposed``: ``w[H, b, a]``), times ``sigmoid(gate[T, H * b])``
+    when given."""
+    y = torch.einsum("tha,hba->thb" if transposed else "tha,hab->thb", x.float(), w.float())
+    if gate is not None:
+        y = y * torch.sigmoid(gate[:, : y.shape[1] * y.shape[2]].float()).view(y.shape)
+    return y.to(w.dtype)
 
 
-def latent_attention(q, pool, block_tables, block_size: int, ctx_lens, cu, scale: float, gate=None):
-    """Softmax attention of absorbed queries ``q[T, H, R]`` over the paged latent rows of their sequence (each row is key
-    and value of every head); row ``i`` of a segment of ``n`` rows sees the first ``ctx - n + i + 1`` of them.
-    ``gate[T, H]``: every head's output is multiplied by its sigmoid."""
+def latent_attention(q, pool, block_tables, block_size: int, ctx_lens, cu, scale: float, gate=None, rank: Optional[int] = None):
+    """Softmax attention of absorbed queries ``q[T, H, R]`` over the paged latent rows of their sequence (each row is key, and its
+    first ``rank`` features are the value, of every head); row ``i`` of a segment of ``n`` rows sees the first ``ctx - n + i + 1`` of
+    them.  ``gate[T, H]``: every head's output is multiplied by its sigmoid."""
     T, H, R = q.shape
-    out = torch.zeros(T, H, R, dtype=torch.float32, device=q.device)
+    rank = rank or R
+    out = torch.zeros(T, H, rank, dtype=torch.float32, device=q.device)
     bounds = list(range(T + 1)) if cu is None else cu.tolist()
     for s, (a, b) in enumerate(zip(bounds, bounds[1:])):
         L = int(ctx_lens[s])
@@ -130,7 +175,7 @@ def latent_attention(q, pool, block_tables, block_size: int, ctx_lens, cu, scale
         sc = torch.einsum("thr,lr->thl", q[a:b].float(), c) * scale
         lim = L - (b - a) + torch.arange(b - a, device=q.device)
         sc = sc.masked_fill(pos[None, None, :] > lim[:, None, None], float("-inf"))
-        out[a:b] = torch.einsum("thl,lr->thr", torch.softmax(sc, -1), c)
+        out[a:b] = torch.einsum("thl,lr->thr", torch.softmax(sc, -1), c[:, :rank])
     if gate is not None:
         out = out * torch.sigmoid(gate.float())[..., None]
     return out.to(q.dtype)
@@ -167,10 +212,42 @@ def attention_inputs(qkv, table, heads: int, kv_heads: int, dim: int, vdim: int,
     return q
 
 
-def paged_attention(q, k_pool, v_pool, block_tables, block_size: int, ctx_lens, cu, scale: float, sink, out_width: int):
+def projection_inputs(qkv, q_w, k_w, table, heads: int, kv_heads: int, dim: int, vdim: int, dp: int, rot_dims: int, halves: bool, eps: float, k_pool,
+                      v_pool, slots):
+    """Like :func:`attention_inputs` with RMS norms (weights ``q_w``, ``k_w``) over all query columns and over all key columns, before
+    heads and rotation; ``halves``: features ``i`` and ``i + rot_dims / 2`` turn together."""
+    def heads_of(x, w, n):
+        x = x.float()
+        if eps > 0:
+            x = x / torch.sqrt(x.pow(2).mean(-1, keepdim=True) + eps)
+            if w is not None:
+                x = x * w.float()
+        x = x.view(x.shape[0], n, dim)
+        if not rot_dims:
+            return x
+        r, half = x[..., :rot_dims], rot_dims // 2
+        if halves:
+            c, s = table[:, None, :, 0], table[:, None, :, 1]
+            u, v = r[..., :half], r[..., half:]
+            r = torch.cat([u * c - v * s, v * c + u * s], -1)
+        else:
+            r = turn_neighbours(r, table)
+        return torch.cat([r, x[..., rot_dims:]], -1)
+
+    T, qd, kd = qkv.shape[0], heads * dim, kv_heads * dim
+    q = torch.zeros(T, heads, dp, dtype=qkv.dtype, device=qkv.device)
+    q[..., :dim] = heads_of(qkv[:, :qd], q_w, heads).to(qkv.dtype)
+    if k_pool is not None:
+        k_pool[slots, :, :dim] = heads_of(qkv[:, qd:qd + kd], k_w, kv_heads).to(k_pool.dtype)
+        v_pool[slots, :, :vdim] = qkv[:, qd + kd:qd + kd + kv_heads * vdim].view(T, kv_heads, vdim).to(v_pool.dtype)
+    return q
+
+
+def paged_attention(q, k_pool, v_pool, block_tables, block_size: int, ctx_lens, cu, scale: float, sink, out_width: int, window: int = 0, gate=None):
     """Softmax attention of ``q[T, H, dp]`` over paged keys and values ``[rows, kv_heads, ...]`` of their sequence; row ``i`` of
-    a segment of ``n`` rows sees the first ``ctx - n + i + 1`` positions.  ``sink[H]``: a logit per head that only joins the
-    denominator.  Returns ``[T, H * out_width]``."""
+    a segment of ``n`` rows sees the first ``ctx - n + i + 1`` positions, with a ``window`` only the last ``window`` of those.
+    ``sink[H]``: a logit per head that only joins the denominator.  ``gate[T, H * out_width]``: its sigmoid multiplies the outputs.
+    Returns ``[T, H * out_width]``."""
     T, H, _ = q.shape
     G, rep = k_pool.shape[1], H // k_pool.shape[1]
     out = torch.zeros(T, H, out_width, dtype=torch.float32, device=q.device)
@@ -184,46 +261,60 @@ def paged_attention(q, k_pool, v_pool, block_tables, block_size: int, ctx_lens, 
         sc = torch.einsum("tgrd,lgd->tgrl", q[a:b].float().view(b - a, G, rep, -1), k).reshape(b - a, H, L) * scale
         lim = L - (b - a) + torch.arange(b - a, device=q.device)
         sc = sc.masked_fill(pos[None, None, :] > lim[:, None, None], float("-inf"))
+        if window:
+            sc = sc.masked_fill(pos[None, None, :] <= lim[:, None, None] - window, float("-inf"))
         if sink is not None:
             sc = torch.cat([sc, sink.float()[None, :, None].expand(b - a, H, 1)], -1)
         p = torch.softmax(sc, -1)[..., :L].reshape(b - a, G, rep, L)
         out[a:b, :, :w] = torch.einsum("tgrl,lgd->tgrd", p, v).reshape(b - a, H, w)
-    return out.reshape(T, H * out_width).to(q.dtype)
+    out = out.reshape(T, H * out_width)
+    return (out if gate is None else out * torch.sigmoid(gate[:, : H * out_width].float())).to(q.dtype)
 
 
 class ExpertPlan:
-    """Which experts every row takes, ``index [T, top]``, and with which ``weight [T, top]``."""
+    """Which experts every row takes, ``index [T, top]`` (from ``experts`` on: identity experts), and with which ``weight [T, top]``."""
 
-    def __init__(self, index, weight):
-        self.index, self.weight = index, weight
+    def __init__(self, index, weight, experts: int):
+        self.index, self.weight, self.experts = index, weight, experts
 
 
-def moe_route(logits, spec):
-    """Sigmoid scores; the ``spec.keep`` groups with the largest sums of their two best scores stay; of their experts the
-    ``spec.top`` best are taken."""
-    s = torch.sigmoid(logits[:, : spec.experts].float())
-    T, n = s.shape[0], spec.experts // spec.groups
-    best = s.view(T, spec.groups, n).topk(min(2, n), -1).values.sum(-1)
+def moe_route(logits, spec, correction=None):
+    """Sigmoid or softmax scores; with ``correction`` added, the ``spec.keep`` groups with the largest sums of their ``spec.group_best``
+    best scores stay, and of their outputs the ``spec.top`` best are taken."""
+    z = logits[:, : spec.outputs].float()
+    s = torch.softmax(z, -1) if spec.score == "softmax" else torch.sigmoid(z)
+    choice = s if correction is None else s + correction[: spec.outputs].float()
+    T, n = s.shape[0], spec.outputs // spec.groups
+    best = choice.view(T, spec.groups, n).topk(min(spec.group_best, n), -1).values.sum(-1)
     open_ = torch.zeros(T, spec.groups, dtype=torch.bool, device=s.device).scatter_(1, best.topk(spec.keep, -1).indices, True)
-    idx = s.masked_fill(~open_.repeat_interleave(n, 1), -1.0).topk(spec.top, -1).indices
+    idx = choice.masked_fill(~open_.repeat_interleave(n, 1), float("-inf")).topk(spec.top, -1).indices
     w = s.gather(-1, idx)
     if spec.renormalize:
-        w = w / w.sum(-1, keepdim=True)
-    return ExpertPlan(idx, w * spec.weight_scale)
+        w = w / (w.sum(-1, keepdim=True) + 1e-20)
+    return ExpertPlan(idx, w * spec.weight_scale, spec.experts)
 
 
 def relu2(x):
     return torch.relu(x.float()).pow(2).to(x.dtype)
 
 
-def moe_experts(h, plan, up, down, act: str):
-    """Outputs ``down_e act(up_e h)`` of every row's experts, unweighted: ``[T, top, W]``."""
-    assert act == "relu2"
+def clamped_swish(gate_up, limit: float):
+    """``g sigmoid(1.702 g) (u + 1)`` of bounded halves; columns alternate between 32 gates and the 32 units they belong to."""
+    g, u = gate_up.float().view(gate_up.shape[0], -1, 2, 32).unbind(2)
+    g, u = g.clamp(max=limit), u.clamp(min=-limit, max=limit)
+    return (g * torch.sigmoid(1.702 * g) * (u + 1)).flatten(1).to(gate_up.dtype)
+
+
+def moe_experts(h, plan, up, down, act: str, limit: float = 0.0):
+    """Outputs ``down_e act(up_e h)`` of every row's experts, unweighted: ``[T, top, W]`` (zero for identity experts)."""
     T, k = plan.index.shape
     out = torch.zeros(T, k, down.shape[1], dtype=h.dtype, device=h.device)
     for e in plan.index.unique().tolist():
+        if e >= plan.experts:
+            continue
         t, j = (plan.index == e).nonzero(as_tuple=True)
-        out[t, j] = F.linear(relu2(F.linear(h[t], up[e])), down[e])
+        y = F.linear(h[t], up[e])
+        out[t, j] = F.linear(relu2(y) if act == "relu2" else clamped_swish(y, limit), down[e])
     return out
 
 

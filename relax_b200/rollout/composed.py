@@ -3,7 +3,8 @@
 A composed stack (``ModelConfig.layer_specs``) mixes layers whose memory of the past differs in kind:
 
 * recurrent layers keep one fp32 matrix per head and sequence, in a STATE SLOT of a fixed pool (:class:`StackCache.state`);
-* latent-attention layers keep one row per token in PAGES of the engine's block manager (:class:`StackCache.latent`);
+* latent-attention layers keep one row per token in PAGES of the engine's block manager (:class:`StackCache.latent`): the latent
+  features and, where positions are rotated in, one rotated key part behind them;
 * attention layers keep a key and a value row per token and key / value head in the same pages (:class:`StackCache.kv`), unless
   they read the rows of an earlier layer.
 
@@ -37,6 +38,11 @@ def head_pitch(n: int) -> int:
     return 64 if n <= 64 else (128 if n <= 128 else pad_to(n, 8))
 
 
+def latent_row(spec) -> int:
+    """Columns of a cached latent row: latent features, then the rotated key part, each in whole 64-column chunks."""
+    return pad_to(spec.kv_rank, 64) + pad_to(spec.rot_dims, 64)
+
+
 class SlotManager:
     """Fixed pool of state slots, one per live sequence."""
 
@@ -62,7 +68,7 @@ class SlotManager:
 
 
 class StackCache:
-    """The pools of a composed stack.  ``latent[layer]``: ``[blocks * block_size, padded rank]`` rows in the model's type;
+    """The pools of a composed stack.  ``latent[layer]``: ``[blocks * block_size, latent_row]`` rows in the model's type;
     ``kv[layer]``: keys and values ``[blocks * block_size, kv heads, padded width]``, one pair for the layer that computes them and
     all that read them; ``state[layer]``: ``[slots, heads, dim, padded vdim]`` fp32.  All of it lives in ONE buffer."""
 
@@ -75,7 +81,7 @@ class StackCache:
             if s.mixer == "hgrn2":
                 pools = [("state", (num_slots, s.heads, s.dim, pad_to(s.vdim, 4)), torch.float32, 4)]
             elif s.mixer == "latent_attention":
-                pools = [("latent", (rows, pad_to(s.kv_rank, 64)), dtype, es)]
+                pools = [("latent", (rows, latent_row(s)), dtype, es)]
             else:
                 pools = [(k, (rows, s.kv_heads, head_pitch(d)), dtype, es) for k, d in (("k", s.dim), ("v", s.vdim))] if s.own_kv else []
             for kind, shape, dt, size in pools:
@@ -116,7 +122,8 @@ class SegmentBatch:
     """Device description of a batch of segments; the first ``long_segs`` of them (``long_rows`` rows) are long portions, those
     from ``multi_segs`` (row ``multi_rows``) on have a single row.
     ``cu`` is None when every segment is a single row.  ``short_*`` describe the segments behind the long ones, with row
-    numbers counted from ``long_rows``; ``items[heads]`` are their column groups (see :func:`attention_items`)."""
+    numbers counted from ``long_rows``; ``items[heads]`` are their column groups of up to ``item_width[heads]`` (64)
+    columns (see :func:`attention_items`)."""
     tokens: torch.Tensor
     slots: torch.Tensor                      # [T] row of the latent pools that each token's row goes to
     ctx: torch.Tensor                        # [S] int32: tokens of the sequence including this segment
@@ -134,8 +141,9 @@ class SegmentBatch:
     row_pos: Optional[torch.Tensor] = None
     max_ctx: int = 0                         # host upper bound of the short segments' contexts
     items: Optional[dict] = None
+    item_width: Optional[dict] = None
     spans: Optional[tuple] = None            # row ranges of recurrent spans and the first span of every segment
-    # attention layers
+    # attention layers (and positions for all that rotate)
     multi_segs: int = 0
     multi_rows: int = 0
     max_ctx_one: int = 0                     # host upper bound of the single-row segments' contexts
@@ -199,12 +207,19 @@ class ComposedForward:
     """The forward of composed stacks (mixed into :class:`relax_b200.rollout.weights.RolloutWeights`).
 
     The residual stream is fp32.  A sublayer reads its copy in the model's type, and one kernel norms the sublayer's
-    output, adds it and writes the next copy; at the last sublayer that kernel also applies the final norm."""
+    output, adds it and writes the next copy (or adds first and norms the sum); at the last sublayer that kernel also applies the
+    final norm."""
 
     def latent_dims(self, i: int) -> tuple:
-        """Padded ``(dim, vdim, rank)`` of latent layer ``i`` (16-byte rows per head, 64-column latent chunks)."""
+        """Padded ``(dim, vdim, rank)`` of latent layer ``i`` (16-byte rows per head, 64-column latent chunks); ``dim`` counts the
+        unrotated and the rotated features of a head."""
         s = self.cfg.layer_specs[i]
-        return pad_to(s.dim, 8), pad_to(s.vdim, 8), pad_to(s.kv_rank, 64)
+        return pad_to(s.dim + s.rot_dims, 8), pad_to(s.vdim, 8), pad_to(s.kv_rank, 64)
+
+    @staticmethod
+    def gate_column(s) -> int:
+        """First column of an attention layer's output gate behind its projections (16-byte aligned)."""
+        return pad_to(s.heads * s.dim + (s.kv_heads * (s.dim + s.vdim) if s.own_kv else 0), 8)
 
     def attention_dims(self, i: int) -> tuple:
         """Pitch of a head's queries and keys, of its values, and of its output in attention layer ``i``."""
@@ -234,34 +249,55 @@ class ComposedForward:
                 shapes[p + "rec_f_bias"], shapes[p + "rec_lower"], shapes[p + "rec_norm"] = (qd,), (qd,), (s.vdim,)
                 shapes[p + "rec_o"] = (Wp, pad_to(vd, 8))
             elif s.mixer == "attention":
-                shapes[p + "attn_qkv"] = (pad_to(H * s.dim + (s.kv_heads * (s.dim + s.vdim) if s.own_kv else 0), 64), Wp)
+                cols = ComposedForward.gate_column(s) + H * pad_to(s.vdim, 8) if s.out_gate else \
+                    H * s.dim + (s.kv_heads * (s.dim + s.vdim) if s.own_kv else 0)
+                shapes[p + "attn_qkv"] = (pad_to(cols, 64), Wp)
+                if s.proj_norm:
+                    shapes[p + "attn_q_norm"] = (H * s.dim,)
+                    if s.own_kv:
+                        shapes[p + "attn_k_norm"] = (s.kv_heads * s.dim,)
                 if s.sink:
                     shapes[p + "attn_sink"] = (H,)
                 shapes[p + "attn_o"] = (Wp, H * pad_to(s.vdim, 8))
             else:
-                dp, vp, Rp = pad_to(s.dim, 8), pad_to(s.vdim, 8), pad_to(s.kv_rank, 64)
-                shapes[p + "lat_qcg"] = (pad_to(H * dp + Rp + H, 64), Wp)
+                # rows of lat_qcg: queries (a head's unrotated, then its rotated features), latent, rotated key part, gates.  lat_uk maps
+                # a cached row to a head's key; its rows of rotated features are those of the identity (:meth:`pass_rotated_keys`)
+                dp, vp, Rp = pad_to(s.dim + s.rot_dims, 8), pad_to(s.vdim, 8), pad_to(s.kv_rank, 64)
+                shapes[p + "lat_qcg"] = (pad_to(H * dp + Rp + pad_to(s.rot_dims, 8) + (H * vp if s.out_gate else H), 64), Wp)
                 shapes[p + "lat_norm"] = (Rp,)
-                shapes[p + "lat_uk"], shapes[p + "lat_uv"] = (H * dp, Rp), (H * vp, Rp)
+                shapes[p + "lat_uk"], shapes[p + "lat_uv"] = (H * dp, latent_row(s)), (H * vp, Rp)
                 shapes[p + "lat_o"] = (Wp, H * vp)
-            shapes[p + "post_attn_norm"] = (Wp,)
-            if s.has_ff:
-                shapes[p + "post_mlp_norm"] = (Wp,)
+            for norm in ["post_attn_norm"] + (["post_mlp_norm"] if s.has_ff else []):
+                shapes[p + norm] = (Wp,)
+                if cfg.norm_sum:
+                    shapes[p + norm + "_b"] = (Wp,)
             if s.ff:
                 Fp = pad_to(s.ff, 64)
                 shapes[p + "gate_up"], shapes[p + "down"] = (2 * Fp, Wp), (Wp, Fp)
             if s.moe is not None:
                 E, Fp, Fs = s.moe.experts, pad_to(s.moe.ff, 64), pad_to(s.moe.shared_ff, 64)
-                shapes[p + "moe_router"] = (pad_to(E, 64), Wp)
-                shapes[p + "moe_up"], shapes[p + "moe_down"] = (E, Fp, Wp), (E, Wp, Fp)
+                shapes[p + "moe_router"] = (pad_to(s.moe.outputs, 64), Wp)
+                if s.moe.correction:
+                    shapes[p + "moe_correction"] = (s.moe.outputs,)
+                shapes[p + "moe_up"], shapes[p + "moe_down"] = (E, 2 * Fp if s.moe.gated else Fp, Wp), (E, Wp, Fp)
                 if Fs:
                     shapes[p + "shared_up"], shapes[p + "shared_down"] = (Fs, Wp), (Wp, Fs)
         shapes["final_norm"] = (Wp,)
+        if cfg.norm_sum:
+            shapes["final_norm_b"] = (Wp,)
         if cfg.embed_norm:
             shapes["embed_norm"] = (Wp,)
         if not cfg.tie_word_embeddings:
             shapes["lm_head"] = (Vp, Wp)
         return shapes
+
+    def pass_rotated_keys(self, i: int) -> None:
+        """Let the key map of latent layer ``i`` hand the rotated part of a cached row on to every head's key unchanged (a reader calls
+        this after it has filled the map's other rows)."""
+        s = self.cfg.layer_specs[i]
+        uk = self.p[f"layers.{i}.lat_uk"].view(s.heads, -1, latent_row(s))
+        k = torch.arange(s.rot_dims, device=uk.device)
+        uk[:, s.dim + k, pad_to(s.kv_rank, 64) + k] = 1.0
 
     # ------------------------------------------------------------------ mixers
     def _hgrn2(self, i, h, b: SegmentBatch, cache: StackCache):
@@ -271,28 +307,31 @@ class ComposedForward:
                       b.ctx, b.cu, s.heads, s.dim, s.vdim, self.cfg.rms_norm_eps, b.spans)
         return ops.linear(o, p[pre + "rec_o"])
 
-    def _latent(self, i, h, b: SegmentBatch, cache: StackCache):
+    def _latent(self, i, h, b: SegmentBatch, cache: StackCache, tables: dict):
         """Keys and values are products of the cached latent row ``c``: ``q . (W_uk c) = (W_uk^T q) . c`` and
         ``sum p (W_uv c) = W_uv (sum p c)``.  Single tokens and short portions therefore attend to the latent rows in
         place, with the up-projections folded around the attention; long portions project keys and values of their whole
-        context once and run the flash kernel on them."""
+        context once and run the flash kernel on them.  A rotated key part in the row passes both ways unchanged
+        (:meth:`pass_rotated_keys`)."""
         s, p, pre = self.cfg.layer_specs[i], self.p, f"layers.{i}."
-        H, (dp, vp, Rp), pool = s.heads, self.latent_dims(i), cache.latent[i]
-        T = h.shape[0]
+        H, (dp, vp, Rp), row, pool = s.heads, self.latent_dims(i), latent_row(s), cache.latent[i]
+        T, rp = h.shape[0], pad_to(s.rot_dims, 8)
         qcg = ops.linear(h, p[pre + "lat_qcg"])
-        q, gate = qcg[:, : H * dp].view(T, H, dp), qcg[:, H * dp + Rp: H * dp + Rp + H]
-        ops.latent_write(qcg[:, H * dp: H * dp + Rp], p[pre + "lat_norm"], s.kv_rank, self.cfg.rms_norm_eps, pool, b.slots)
+        q, c, k_rot, gate = qcg[:, : H * dp + Rp + rp + H * (vp if s.out_gate else 1)].split([H * dp, Rp, rp, H * (vp if s.out_gate else 1)], 1)
+        q = q.view(T, H, dp)
+        turned = (q, k_rot, self._rope_table(s, b, tables), Rp, s.rot_dims, s.dim) if s.rot_dims else None
+        ops.latent_write(c, p[pre + "lat_norm"], s.kv_rank, self.cfg.rms_norm_eps, pool, b.slots, turned)
         uk, uv = p[pre + "lat_uk"], p[pre + "lat_uv"]
         n = b.long_rows
         parts = []
         if n:
             c = pool[b.ctx_slots]
-            k, v = ops.linear(c, uk).view(-1, H, dp), ops.linear(c, uv).view(-1, H, vp)
-            parts.append(ops.flash_gated(q[:n], k, v, b.long_cu, b.long_cu_k, s.scale, b.long_max, gate[:n]))
+            k, v = ops.linear(c, uk).view(-1, H, dp), ops.linear(c[:, :Rp], uv).view(-1, H, vp)
+            parts.append(ops.flash_gated(q[:n], k, v, b.long_cu, b.long_cu_k, s.scale, b.long_max, gate[:n], s.out_gate))
         if n < T:
-            ql = ops.head_linear(q[n:], uk.view(H, dp, Rp), False)
-            o = ops.latent_attention(ql, pool, b, cache.block_size, s.scale, gate[n:])
-            parts.append(ops.head_linear(o, uv.view(H, vp, Rp), True).reshape(T - n, H * vp))
+            ql = ops.head_linear(q[n:], uk.view(H, dp, row), False)
+            o = ops.latent_attention(ql, pool, b, cache.block_size, s.scale, None if s.out_gate else gate[n:], Rp)
+            parts.append(ops.head_linear(o, uv.view(H, vp, Rp), True, gate[n:] if s.out_gate else None).reshape(T - n, H * vp))
         return ops.linear(parts[0] if len(parts) == 1 else torch.cat(parts), p[pre + "lat_o"])
 
     def _attention(self, i, h, b: SegmentBatch, cache: StackCache, tables: dict):
@@ -300,9 +339,15 @@ class ComposedForward:
         dp, _, vo = self.attention_dims(i)
         k_pool, v_pool = cache.kv[i]
         qkv = ops.linear(h, p[pre + "attn_qkv"])
-        q = ops.attention_inputs(qkv, self._rope_table(s, b, tables), s.heads, s.kv_heads, s.dim, s.vdim, dp, s.rot_dims,
-                                 self.cfg.rms_norm_eps if s.qk_norm else 0.0, *((k_pool, v_pool) if s.own_kv else (None, None)), b.slots)
-        o = ops.paged_attention(q, k_pool, v_pool, b, cache.block_size, s.scale, p.get(pre + "attn_sink"), vo)
+        table, eps, pools = self._rope_table(s, b, tables), self.cfg.rms_norm_eps, (k_pool, v_pool) if s.own_kv else (None, None)
+        if s.proj_norm or s.rot_halves:
+            q = ops.projection_inputs(qkv, p.get(pre + "attn_q_norm"), p.get(pre + "attn_k_norm"), table, s.heads, s.kv_heads, s.dim, s.vdim, dp, s.rot_dims,
+                                      s.rot_halves, eps if s.proj_norm else 0.0, *pools, b.slots)
+        else:
+            q = ops.attention_inputs(qkv, table, s.heads, s.kv_heads, s.dim, s.vdim, dp, s.rot_dims, eps if s.qk_norm else 0.0, *pools, b.slots)
+        g = self.gate_column(s)
+        o = ops.paged_attention(q, k_pool, v_pool, b, cache.block_size, s.scale, p.get(pre + "attn_sink"), vo, s.window,
+                                qkv[:, g:g + s.heads * vo] if s.out_gate else None)
         return ops.linear(o, p[pre + "attn_o"])
 
     def _rope_table(self, s, b: SegmentBatch, tables: dict):
@@ -319,8 +364,8 @@ class ComposedForward:
         s, p, pre = self.cfg.layer_specs[i], self.p, f"layers.{i}."
         if s.moe is None:
             return ops.linear(ops.linear_glu(h, p[pre + "gate_up"], s.act), p[pre + "down"]), None
-        plan = ops.moe_route(ops.linear_fp32(h, p[pre + "moe_router"]), s.moe, h.dtype, count)
-        rows = ops.moe_experts(h, plan, p[pre + "moe_up"], p[pre + "moe_down"], s.moe.act)
+        plan = ops.moe_route(ops.linear_fp32(h, p[pre + "moe_router"]), s.moe, h.dtype, count, p.get(pre + "moe_correction"))
+        rows = ops.moe_experts(h, plan, p[pre + "moe_up"], p[pre + "moe_down"], s.moe.act, s.moe.limit)
         shared = ops.linear(ops.linear_act(h, p[pre + "shared_up"], s.moe.act), p[pre + "shared_down"]) if s.moe.shared_ff else None
         return shared, (rows, plan)
 
@@ -329,21 +374,29 @@ class ComposedForward:
         """Final-norm output of every row.  ``taps``: a list that receives the fp32 residual stream after every layer."""
         cfg, p = self.cfg, self.p
         W, G, eps = cfg.hidden_size, cfg.norm_groups, cfg.rms_norm_eps
-        res, h = ops.embed_rows(b.tokens, p["embed"], p.get("embed_norm"), W, G, eps)
+        res, h = ops.embed_rows(b.tokens, p["embed"], p.get("embed_norm"), W, G, eps, cfg.embed_scale)
+
+        def join(y, norm, last, experts=None):
+            """The sublayer's output meets the stream; returns the next sublayer's input."""
+            if not cfg.norm_sum:
+                return ops.norm_add(res, y, p[norm], W, G, eps, p["final_norm"] if last else None, experts)
+            nxt = (p["final_norm"], p["final_norm_b"]) if last else None
+            return ops.sum_norm(res, y, p[norm], p[norm + "_b"], W, cfg.sum_alpha, eps, nxt, cfg.logit_scale if last else 1.0, experts)
+
         tables: dict = {}
         routed = [i for i, s in enumerate(cfg.layer_specs) if s.moe is not None]
         counts = dict(zip(routed, ops.route_counters(len(routed), max(cfg.layer_specs[i].moe.experts for i in routed), res.device))) if routed else {}
         for i, s in enumerate(cfg.layer_specs):
             pre = f"layers.{i}."
-            final = p["final_norm"] if i + 1 == cfg.num_layers else None
-            if s.mixer == "attention":
-                a = self._attention(i, h, b, cache, tables)
+            final = i + 1 == cfg.num_layers
+            if s.mixer == "hgrn2":
+                a = self._hgrn2(i, h, b, cache)
             else:
-                a = self._hgrn2(i, h, b, cache) if s.mixer == "hgrn2" else self._latent(i, h, b, cache)
-            h = ops.norm_add(res, a, p[pre + "post_attn_norm"], W, G, eps, None if s.has_ff else final)
+                a = (self._attention if s.mixer == "attention" else self._latent)(i, h, b, cache, tables)
+            h = join(a, pre + "post_attn_norm", final and not s.has_ff)
             if s.has_ff:
                 m, experts = self._feed_forward(i, h, counts.get(i))
-                h = ops.norm_add(res, m, p[pre + "post_mlp_norm"], W, G, eps, final, experts)
+                h = join(m, pre + "post_mlp_norm", final, experts)
             if taps is not None:
                 taps.append(res[:, :W].clone())
         return h
@@ -412,14 +465,15 @@ class ComposedScheduler:
         arrays = {"tokens": (toks, i64), "slots": (slots, i64), "ctx": (ctx, i32), "block_tables": (bt, i32), "state_slot": (sslot, i32)}
         host = {"long_segs": n_long, "long_rows": cu[n_long], "max_ctx": max(ctx[n_long:], default=0),
                 "multi_segs": n_multi, "multi_rows": cu[n_multi], "max_ctx_one": max(ctx[n_multi:], default=0)}
-        heads, tiles = [], []
+        widths, tiles = {}, []
         if not single:
             arrays["cu"] = (cu, i32)
             lens = [b - a for a, b in zip(cu, cu[1:])]
             sl, sc = lens[n_long:], ctx[n_long:]
             attn = [self.cfg.layer_specs[i] for i in self.cfg.layers_with("attention")]
-            if attn:
+            if attn or any(s.rot_dims for s in self.cfg.layer_specs):
                 arrays["pos"] = ([c - n + k for n, c in zip(lens, ctx) for k in range(n)], i32)
+            if attn:
                 arrays["seg_of"] = ([s for s, n in enumerate(lens) for _ in range(n)], i32)
                 tiles = sorted({tile_tokens(s) for s in attn})
                 for t in tiles:
@@ -440,17 +494,19 @@ class ComposedScheduler:
                 arrays["short_cu"] = ([c - cu[n_long] for c in cu[n_long:]], i32)
                 arrays["row_seg"] = ([s for s, n in enumerate(sl) for _ in range(n)], i32)
                 arrays["row_pos"] = ([c - n + k for n, c in zip(sl, sc) for k in range(n)], i32)
-                heads = sorted({self.cfg.layer_specs[i].heads for i in self.cfg.layers_with("latent_attention")})
-                for H in heads:
-                    arrays[f"items{H}"] = (attention_items(sl, sc, H), i32)
+                specs = [self.cfg.layer_specs[i] for i in self.cfg.layers_with("latent_attention")]
+                for s in specs:
+                    widths[s.heads] = min(widths.get(s.heads, 64), ops.latent_columns(latent_row(s), pad_to(s.kv_rank, 64)))
+                for H, width in widths.items():
+                    arrays[f"items{H}"] = (attention_items(sl, sc, H, width), i32)
         if rows:
             arrays["rows"] = (rows, i64)
         dev = dict(zip(arrays, self._stage(list(arrays.values()))))
         want_t = dev.pop("rows", None)
         spans = (dev.pop("spans"), dev.pop("span_first")) if "spans" in dev else None
-        items = {H: dev.pop(f"items{H}") for H in heads}
+        items = {H: dev.pop(f"items{H}") for H in widths}
         blocks = {t: dev.pop(f"blocks{t}") for t in tiles}
-        batch = SegmentBatch(**dev, **host, items=items or None, spans=spans, blocks=blocks or None)
+        batch = SegmentBatch(**dev, **host, items=items or None, item_width=widths or None, spans=spans, blocks=blocks or None)
         logits = self.weights.forward_segments(batch, self.kv, want_t, self.tp, taps)
         for r, n in parts:
             r.fed += n

@@ -3,10 +3,11 @@ import torch
 
 import oracle_composed
 import oracle_ketolorn
+import oracle_zupupel
 
 
 def oracle(cfg):
-    return oracle_ketolorn if cfg.get("architecture") == "Ketolorn" else oracle_composed
+    return {"Ketolorn": oracle_ketolorn, "Zupupel": oracle_zupupel}.get(cfg.get("architecture"), oracle_composed)
 
 
 def engine(cfg, tensors, device="cpu", dtype=torch.float32, blocks=64, block_size=16, **kw):
