@@ -186,7 +186,7 @@ CONFIGS = {
                                  att(6, 2, 18, 13, 0.22, 10, 1e3, 9, moe(4, 3, 33, 0.5, 3), 0), att(5, 5, 7, 9, 0.9, 4, 50.0, 33),
                                  att(6, 2, 18, 13, 0.4, 10, 1e3, 40, moe(6, 1, 12, 2.0, 0, 2, 2), 0)]),
     # whole heads turn; wide groups, narrow keys beside wide values, a whole latent layer between
-    "even": stack(128, 256, 1e-4, [lat(8, 64, 32, 64, 128, 0.11, 1e4, moe(12, 4, 64, 1.5, 4, 4, 2)), att(8, 1, 64, 128, 0.2, 64, 1e4, 48, moe(8, 2, 64, 1.0, 0, 4, 2)),
+    "even": stack(128, 256, 1e-4, [lat(8, 56, 24, 64, 128, 0.12, 1e4, moe(12, 4, 64, 1.5, 4, 4, 2)), att(8, 1, 64, 128, 0.2, 64, 1e4, 48, moe(8, 2, 64, 1.0, 0, 4, 2)),
                                    att(4, 4, 128, 32, 0.11, 32, 1e5, 100, moe(14, 3, 128, 0.8, 2, 2, 1)), att(4, 4, 128, 32, 0.2, 32, 1e5, 64, None, 2),
                                    lat(16, 96, 32, 128, 192, 0.1, 1e5)], 2.5, 3.0, 1.4),
     # one head, one feature pair, a window of one token, experts of one per group
