@@ -37,6 +37,8 @@ int rb_int4_fake_quant(const void* x, void* out, void* scale, void* zero, int M,
 int rb_fp8_block_cast(const void* w, void* q, float* scale, int M, int N, int block, int ue8m0, int dtype, cudaStream_t st);
 int rb_fp8_block_dequant(const void* q, const float* scale, void* out, int M, int N, int block, int dtype, cudaStream_t st);
 
+int rb_dense_flash(const void* q, long long q_pitch, const void* k, const void* v, const int* first, const int* blocks, const void* gate, int ld_gate,
+                   int head_gate, void* out, int rows, int n, int H, int dk, int dv, long long k_rows, float scale, int* err, cudaStream_t st);
 int rb_sum_norm(float* res, const void* y, const void* ex, const int* expert, const int* place, const int* offset, const float* weight, int top, int
                 experts, const void* w, const void* b, const void* next_w, const void* next_b, void* h, int rows, int ldy, int pitch, int width, int
                 centre, float alpha, float eps, float scale, int fp32, cudaStream_t st);
@@ -154,8 +156,7 @@ int rb_latent_attn_tc(const void* q, const void* pool, const int* block_tables, 
                       int splits, int ld_gate, float scale, int* err, cudaStream_t st);
 int rb_head_gemm(const void* x, const void* w, const void* gate, int ld_gate, void* out, int T, int H, int N, int K, long long x_tok, long long
                  x_head, int kn, int* err, cudaStream_t st);
-int rb_gate_heads(const void* o, const void* gate, int ld_gate, void* out, int rows, int H, int pitch, int dv, int features, int fp32, cudaStream_t
-                  st);
+int rb_gate_outputs(void* o, const void* gate, int ld_gate, int rows, int n, int fp32, cudaStream_t st);
 int rb_glu(const void* in, void* out, long long rows, int F, int ld_in, int act, int fp32, cudaStream_t st);
 int rb_simt_gemm(const void* A, const void* B, void* C, int M, int N, int K, int lda, int ldb, int ldc, int b_kn, int batch, long long sa,
                  long long sb, long long sc, int fp32, cudaStream_t st);

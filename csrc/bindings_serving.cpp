@@ -285,15 +285,13 @@ bool head_gemm(torch::Tensor x, torch::Tensor w, c10::optional<torch::Tensor> ga
   check(rc, "rb_head_gemm");
   return true;
 }
-// features: a gate per output feature, else per head
-void gate_heads(torch::Tensor o, torch::Tensor gate, torch::Tensor out, int64_t dv, bool features) {
+// o [T, ...] times the sigmoid of a gate per feature, in place
+void gate_outputs(torch::Tensor o, torch::Tensor gate) {
   const c10::cuda::CUDAGuard guard(o.device());
-  check_same(o, out, "gate_heads");
-  TORCH_CHECK(o.dim() == 3 && o.is_contiguous() && out.is_contiguous() && out.numel() == o.size(0) * o.size(1) * dv);
-  const int ld = gate_pitch(gate, o, o.size(0), features ? o.size(1) * dv : o.size(1));
-  check(rb_gate_heads(o.data_ptr(), gate.data_ptr(), ld, out.data_ptr(), (int)o.size(0), (int)o.size(1), (int)o.size(2), (int)dv, features, is_fp32(o),
-                      cur_stream()),
-        "rb_gate_heads");
+  TORCH_CHECK(o.is_contiguous() && o.size(0) > 0, "gate_outputs: layout");
+  const int64_t n = o.numel() / o.size(0);
+  const int ld = gate_pitch(gate, o, o.size(0), n);
+  check(rb_gate_outputs(o.data_ptr(), gate.data_ptr(), ld, (int)o.size(0), (int)n, is_fp32(o), cur_stream()), "rb_gate_outputs");
 }
 void glu(torch::Tensor in, torch::Tensor out, int64_t act) {
   const c10::cuda::CUDAGuard guard(in.device());
@@ -479,6 +477,27 @@ bool paged_flash(torch::Tensor q, torch::Tensor k, torch::Tensor v, torch::Tenso
   check(rc, "rb_paged_flash");
   return true;
 }
+// Keys and values that lie side by side, segment by segment: k, v [rows][H][d], those of segment s from row first[s] on.  q [T][H][dk] may be
+// a strided slice.  gate: [T, H] or (features) [T, >= H dv].  Returns false for shapes the kernel does not take.
+bool dense_flash(torch::Tensor q, torch::Tensor k, torch::Tensor v, torch::Tensor first, torch::Tensor blocks, c10::optional<torch::Tensor> gate, bool features,
+                 torch::Tensor out, double scale, torch::Tensor err) {
+  const c10::cuda::CUDAGuard guard(q.device());
+  if (q.scalar_type() != at::kBFloat16) return false;
+  check_same(q, k, "dense_flash");
+  check_same(q, v, "dense_flash");
+  check_same(q, out, "dense_flash");
+  const int64_t T = q.size(0), H = q.size(1);
+  TORCH_CHECK(q.dim() == 3 && k.dim() == 3 && v.dim() == 3 && q.stride(2) == 1 && (H == 1 || q.stride(1) == q.size(2)) && k.is_contiguous() && v.is_contiguous());
+  TORCH_CHECK(k.size(1) == H && v.size(1) == H && k.size(0) == v.size(0) && k.size(2) == q.size(2), "dense_flash: shapes");
+  TORCH_CHECK(out.dim() == 2 && out.is_contiguous() && out.size(0) == T && out.size(1) == H * v.size(2), "dense_flash: output");
+  TORCH_CHECK(is_i32(first) && is_i32(blocks) && blocks.dim() == 2 && blocks.size(1) == 4, "dense_flash: tiles");
+  const int rc = rb_dense_flash(q.data_ptr(), T > 1 ? q.stride(0) : H * q.size(2), k.data_ptr(), v.data_ptr(), first.data_ptr<int>(), blocks.data_ptr<int>(),
+                                optptr(gate), gate_pitch(gate, q, T, features ? out.size(1) : H), !features, out.data_ptr(), (int)T, (int)blocks.size(0), (int)H,
+                                (int)q.size(2), (int)v.size(2), k.size(0), (float)scale, err.data_ptr<int>(), cur_stream());
+  if (rc == -20) return false;
+  check(rc, "rb_dense_flash");
+  return true;
+}
 // One row per sequence; returns false for shapes the tensor-core kernel does not take.
 bool paged_decode(torch::Tensor q, torch::Tensor k, torch::Tensor v, torch::Tensor bt, torch::Tensor ctx, c10::optional<torch::Tensor> sink,
                   c10::optional<torch::Tensor> gate, torch::Tensor out, c10::optional<torch::Tensor> part_o, c10::optional<torch::Tensor> part_ml,
@@ -566,7 +585,7 @@ void register_serving(pybind11::module_& m) {
   m.def("latent_attn", &latent_attn);
   m.def("latent_attn_tc", &latent_attn_tc);
   m.def("head_gemm", &head_gemm);
-  m.def("gate_heads", &gate_heads);
+  m.def("gate_outputs", &gate_outputs);
   m.def("glu", &glu);
   m.def("simt_gemm", &simt_gemm);
   m.def("embed_norm", &embed_norm);
@@ -577,6 +596,7 @@ void register_serving(pybind11::module_& m) {
   m.def("attention_inputs", &attention_inputs);
   m.def("gqa_attn", &gqa_attn);
   m.def("paged_flash", &paged_flash);
+  m.def("dense_flash", &dense_flash);
   m.def("paged_decode", &paged_decode);
   m.def("moe_route", &moe_route);
   m.def("moe_gemm", &moe_gemm);

@@ -8,12 +8,14 @@
 //                  into shared memory (128-byte swizzle)
 //   O += P V       V is read in place from its [position][d] tile (MN-major)
 // Keys and values come straight from the pages (TMA, one box per page and 64 columns): new rows are written to the pages before
-// this kernel runs, and nothing is gathered into a dense copy.  The running softmax starts from the head's sink logit
+// this kernel runs, and nothing is gathered into a dense copy.  Keys and values that were projected for one call (of a latent cache's
+// rows) lie side by side instead, every segment from a row of its own on.  Heads may be narrower than the 64-column boxes: what a box
+// reads behind them is zero.  The running softmax starts from the head's sink logit
 // (sum = 1 at reference = sink), or empty without one.  With a window a tile starts at the block of the first position that its first
 // row sees, and every row masks what lies before its own.  A gate per output feature is applied in the epilogue.  S is double buffered, so the product of block j + 1 runs while the
 // softmax of block j does.  The accumulator is rescaled only when a row's maximum grows by more than 2^8 (decided per warp: TMEM
-// accesses are warp-wide).  Warps 0-3: softmax and epilogue, warp 4: TMA, warp 5: MMA.  Two CTAs share an SM.  Every wait is
-// bounded; no load uses cluster multicast.
+// accesses are warp-wide).  Warps 0-3: softmax and epilogue, warp 4: TMA, warp 5: MMA.  Two CTAs share an SM; keys of more than 128
+// columns leave room for one stage of keys and values instead of two.  Every wait is bounded; no load uses cluster multicast.
 #include <limits.h>
 
 #include "common.cuh"
@@ -31,13 +33,14 @@ constexpr int T_O = 128;
 
 template <int DK, int DV>
 struct Tile {
-  static_assert((DK == 64 || DK == 128) && (DV == 64 || DV == 128), "key / value rows of 64 or 128 columns");
+  static_assert((DK == 64 || DK == 128 || DK == 192) && (DV == 64 || DV == 128), "key / value rows of 64, 128 or (keys) 192 columns");
+  static constexpr int kStages = DK > 128 ? 1 : 2;
   static constexpr int kQHalf = BQ * 128, kKVHalf = BKV * 128;      // bytes of 64 columns
   static constexpr int kQBytes = DK / 64 * kQHalf;
   static constexpr int kKBytes = DK / 64 * kKVHalf, kVBytes = DV / 64 * kKVHalf;
-  static constexpr int kK = kQBytes;                                // 2 stages
-  static constexpr int kV = kK + 2 * kKBytes;                       // 2 stages
-  static constexpr int kP = kV + 2 * kVBytes;
+  static constexpr int kK = kQBytes;
+  static constexpr int kV = kK + kStages * kKBytes;
+  static constexpr int kP = kV + kStages * kVBytes;
   static constexpr int kBar = kP + BQ * BKV * 2;
   static constexpr int kTotal = kBar + 256;
 };
@@ -46,8 +49,10 @@ struct Params {
   const int* blocks;         // [n][4]: segment, first row, rows, position of the first row; null: row i is segment i, at ctx[i] - 1
   const int* ctx;            // [S]
   const int* block_tables;   // [S][max_blocks]
+  const int* first_row;      // [S]: rows of a segment's positions lie side by side from here on (then there are no pages), or null
   const __nv_bfloat16* sink; // [H] or null
-  const __nv_bfloat16* gate; // [rows][ld_gate], head h's features at h * out_d, or null
+  const __nv_bfloat16* gate; // [rows][ld_gate], head h's features at h * out_d (head_gate: one for all of them at h), or null
+  int head_gate;
   __nv_bfloat16* out;        // [rows][H][out_d]
   int H, G, tokens, max_blocks, page, out_d, ld_gate;
   int window;                // positions a row sees (INT_MAX: all)
@@ -98,7 +103,9 @@ paged_flash_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_const
   const int seen = pos0 + ntok;                    // positions that the last token of the tile sees
   const int block0 = max(0, pos0 - p.window + 1) / BKV;      // block of the first position that the first token sees
   const int n_blocks = (seen + BKV - 1) / BKV - block0;
-  const int* bt = p.block_tables + static_cast<size_t>(seg) * p.max_blocks;
+  const int base = p.first_row ? p.first_row[seg] : -1;
+  const int* bt = p.block_tables + static_cast<size_t>(p.first_row ? 0 : seg) * p.max_blocks;
+  constexpr int ST = L::kStages;
 
   if (threadIdx.x == 0) {
     mbar_init(bar_q, 1);
@@ -139,22 +146,21 @@ paged_flash_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_const
       for (int c = 0; c < DK / 64; ++c) tma_load_3d(smem + c * L::kQHalf, &tma_q, bar_q, c * 64, kvh * p.G, row0);
       const int rows = p.page < BKV ? p.page : BKV;          // rows per box
       for (int j = 0; j < n_blocks; ++j) {
-        const int s = j & 1;
-        const uint32_t ph = (static_cast<uint32_t>(j >> 1) & 1) ^ 1;
+        const int s = j % ST;
+        const uint32_t ph = (static_cast<uint32_t>(j / ST) & 1) ^ 1;
+        auto pool_row = [&](int pos) { return base >= 0 ? base + pos : bt[min(pos / p.page, p.max_blocks - 1)] * p.page + pos % p.page; };
         if (!mbar_wait(&kempty[s], ph, abort_flag, p.err)) break;
         uint8_t* sk = smem + L::kK + s * L::kKBytes;
         mbar_expect_tx(&kfull[s], L::kKBytes);
         for (int r = 0; r < BKV; r += rows) {
-          const int pos = (block0 + j) * BKV + r;
-          const int row = bt[min(pos / p.page, p.max_blocks - 1)] * p.page + pos % p.page;
+          const int row = pool_row((block0 + j) * BKV + r);
           for (int c = 0; c < DK / 64; ++c) tma_load_3d(sk + c * L::kKVHalf + r * 128, &tma_k, &kfull[s], c * 64, kvh, row);
         }
         if (!mbar_wait(&vempty[s], ph, abort_flag, p.err)) break;
         uint8_t* sv = smem + L::kV + s * L::kVBytes;
         mbar_expect_tx(&vfull[s], L::kVBytes);
         for (int r = 0; r < BKV; r += rows) {
-          const int pos = (block0 + j) * BKV + r;
-          const int row = bt[min(pos / p.page, p.max_blocks - 1)] * p.page + pos % p.page;
+          const int row = pool_row((block0 + j) * BKV + r);
           for (int c = 0; c < DV / 64; ++c) tma_load_3d(sv + c * L::kKVHalf + r * 128, &tma_v, &vfull[s], c * 64, kvh, row);
         }
       }
@@ -166,17 +172,17 @@ paged_flash_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_const
       const uint32_t idesc_o = make_idesc_f16(BQ, DV, true, false, true);
       const uint32_t sq = smem_u32(smem), sp = smem_u32(smem + L::kP);
       auto issue_s = [&](int j) -> bool {
-        const int s = j & 1;
-        if (!mbar_wait(&kfull[s], static_cast<uint32_t>(j >> 1) & 1, abort_flag, p.err)) return false;
+        const int s = j & 1, st = j % ST;
+        if (!mbar_wait(&kfull[st], static_cast<uint32_t>(j / ST) & 1, abort_flag, p.err)) return false;
         tc_fence_after();
-        const uint32_t sk = smem_u32(smem + L::kK + s * L::kKBytes);
+        const uint32_t sk = smem_u32(smem + L::kK + st * L::kKBytes);
 #pragma unroll
         for (int kk = 0; kk < DK / 16; ++kk) {
           const uint64_t da = make_smem_desc(sq + (kk >> 2) * L::kQHalf + (kk & 3) * 32, 16, 1024, kSwizzle128B);
           const uint64_t db = make_smem_desc(sk + (kk >> 2) * L::kKVHalf + (kk & 3) * 32, 16, 1024, kSwizzle128B);
           umma_f16(tmem_base + T_S + s * BKV, da, db, idesc_s, kk > 0 ? 1u : 0u);
         }
-        umma_commit(&kempty[s]);
+        umma_commit(&kempty[st]);
         umma_commit(&bar_s[s]);
         return true;
       };
@@ -184,12 +190,11 @@ paged_flash_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_const
       if (ok) ok = issue_s(0);
       if (ok && n_blocks > 1) ok = issue_s(1);
       for (int j = 0; j < n_blocks && ok; ++j) {
-        const int s = j & 1;
-        const uint32_t ph = static_cast<uint32_t>(j >> 1) & 1;
-        if (!mbar_wait(&bar_p[s], ph, abort_flag, p.err)) break;
-        if (!mbar_wait(&vfull[s], ph, abort_flag, p.err)) break;
+        const int s = j & 1, st = j % ST;
+        if (!mbar_wait(&bar_p[s], static_cast<uint32_t>(j >> 1) & 1, abort_flag, p.err)) break;
+        if (!mbar_wait(&vfull[st], static_cast<uint32_t>(j / ST) & 1, abort_flag, p.err)) break;
         tc_fence_after();
-        const uint32_t sv = smem_u32(smem + L::kV + s * L::kVBytes);
+        const uint32_t sv = smem_u32(smem + L::kV + st * L::kVBytes);
 #pragma unroll
         for (int kk = 0; kk < BKV / 16; ++kk) {
           const uint64_t da = make_smem_desc(sp + kk * 32, 16, 1024, kSwizzle128B);
@@ -197,7 +202,7 @@ paged_flash_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_const
           const uint64_t db = make_smem_desc(sv + kk * 2048, L::kKVHalf, 1024, kSwizzle128B);
           umma_f16(tmem_base + T_O, da, db, idesc_o, (j > 0 || kk > 0) ? 1u : 0u);
         }
-        umma_commit(&vempty[s]);
+        umma_commit(&vempty[st]);
         umma_commit(&bar_o[s]);
         if (j + 2 < n_blocks && !issue_s(j + 2)) break;      // S of block j was read before bar_p completed
       }
@@ -289,7 +294,9 @@ paged_flash_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_const
     if (ok) ok = mbar_wait(&bar_o[(n_blocks - 1) & 1], static_cast<uint32_t>((n_blocks - 1) >> 1) & 1, abort_flag, p.err);
     const bool all_ok = __all_sync(0xffffffffu, ok);
     tc_fence_after();
-    const float inv_l = l > 0.f ? 1.f / l : 0.f;
+    float inv_l = l > 0.f ? 1.f / l : 0.f;
+    if (p.gate && p.head_gate && mine)
+      inv_l = __fdividef(inv_l, 1.f + __expf(-__bfloat162float(p.gate[static_cast<size_t>(row0 + t) * p.ld_gate + head])));
     __nv_bfloat16* out = p.out + (static_cast<size_t>(row0 + t) * p.H + head) * p.out_d;
     if (all_ok) {
 #pragma unroll 1
@@ -302,7 +309,7 @@ paged_flash_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_const
 #pragma unroll
           for (int i = 0; i < 4; ++i) {
             if (c * 32 + i * 8 < p.out_d) {
-              if (p.gate) gate8(o + 8 * i, p.gate + static_cast<size_t>(row0 + t) * p.ld_gate + head * p.out_d + c * 32 + i * 8);
+              if (p.gate && !p.head_gate) gate8(o + 8 * i, p.gate + static_cast<size_t>(row0 + t) * p.ld_gate + head * p.out_d + c * 32 + i * 8);
               uint4 pk;
               pk.x = pack_bf16(__uint_as_float(o[8 * i]) * inv_l, __uint_as_float(o[8 * i + 1]) * inv_l);
               pk.y = pack_bf16(__uint_as_float(o[8 * i + 2]) * inv_l, __uint_as_float(o[8 * i + 3]) * inv_l);
@@ -325,16 +332,25 @@ paged_flash_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_const
   }
 }
 
+struct Operands {      // widths dk, dv <= DK, DV; q_pitch: elements between two rows of q
+  const void* q;
+  const void* k;
+  const void* v;
+  int rows, n, Hkv, dk, dv;
+  long long q_pitch;
+  uint64_t pool_rows;
+};
+
 template <int DK, int DV>
-static int launch(const void* q, const void* kc, const void* vc, int rows, int Hkv, uint64_t pool_rows, int n, const Params& p, cudaStream_t st) {
+static int launch(const Operands& o, const Params& p, cudaStream_t st) {
   using L = Tile<DK, DV>;
   CUtensorMap tq, tk, tv;
-  int rc = encode_tma_3d_16bit(&tq, q, DK, p.H, rows, DK, static_cast<uint64_t>(p.H) * DK, 64, p.G, p.tokens);
+  int rc = encode_tma_3d_16bit(&tq, o.q, o.dk, p.H, o.rows, o.dk, o.q_pitch, 64, p.G, p.tokens);
   if (rc) return rc;
-  const uint32_t box = p.page < BKV ? p.page : BKV;
-  rc = encode_tma_3d_16bit(&tk, kc, DK, Hkv, pool_rows, DK, static_cast<uint64_t>(Hkv) * DK, 64, 1, box);
+  const uint32_t box = p.first_row || p.page >= BKV ? BKV : p.page;
+  rc = encode_tma_3d_16bit(&tk, o.k, o.dk, o.Hkv, o.pool_rows, o.dk, static_cast<uint64_t>(o.Hkv) * o.dk, 64, 1, box);
   if (rc) return rc;
-  rc = encode_tma_3d_16bit(&tv, vc, DV, Hkv, pool_rows, DV, static_cast<uint64_t>(Hkv) * DV, 64, 1, box);
+  rc = encode_tma_3d_16bit(&tv, o.v, o.dv, o.Hkv, o.pool_rows, o.dv, static_cast<uint64_t>(o.Hkv) * o.dv, 64, 1, box);
   if (rc) return rc;
   auto kern = paged_flash_kernel<DK, DV>;
   static bool attr_set = false;
@@ -343,15 +359,22 @@ static int launch(const void* q, const void* kc, const void* vc, int rows, int H
     if (e != cudaSuccess) return static_cast<int>(e);
     attr_set = true;
   }
-  kern<<<dim3(n, Hkv), THREADS, L::kTotal, st>>>(tq, tk, tv, p);
+  kern<<<dim3(o.n, o.Hkv), THREADS, L::kTotal, st>>>(tq, tk, tv, p);
   rb_note_launch(1);
   return static_cast<int>(cudaGetLastError());
+}
+
+static int dispatch(const Operands& o, const Params& p, cudaStream_t st) {
+  const bool wide = o.dv > 64;
+  if (o.dk > 128) return wide ? launch<192, 128>(o, p, st) : launch<192, 64>(o, p, st);
+  if (o.dk > 64) return wide ? launch<128, 128>(o, p, st) : launch<128, 64>(o, p, st);
+  return wide ? launch<64, 128>(o, p, st) : launch<64, 64>(o, p, st);
 }
 
 }  // namespace pf
 }  // namespace rb
 
-// q [rows][Hq][dk], pools [pool_rows][Hkv][dk / dv] (dk, dv: 64 or 128), out [rows][Hq][out_d].  blocks [n][4]: query tiles of at
+// q [rows][Hq][dk], pools [pool_rows][Hkv][dk / dv] (dk, dv: 64 or 128, dk also 192), out [rows][Hq][out_d].  blocks [n][4]: query tiles of at
 // most 128 / (Hq / Hkv) tokens, every row in exactly one (null: n = rows, one row per segment).  window: positions a row sees, its own
 // included (0: all).  gate [rows][ld_gate] or null.  Returns -20 for shapes outside that.
 extern "C" int rb_paged_flash(const void* q, const void* kc, const void* vc, const int* block_tables, const int* ctx, const int* blocks,
@@ -362,7 +385,7 @@ extern "C" int rb_paged_flash(const void* q, const void* kc, const void* vc, con
   if (rows <= 0 || n <= 0) return 0;
   if (Hkv < 1 || Hq % Hkv) return -2;
   const int G = Hq / Hkv;
-  if (G > BQ || Hkv > 65535 || (dk != 64 && dk != 128) || (dv != 64 && dv != 128) || out_d % 8 || out_d > dv || out_d < 1) return -20;
+  if (G > BQ || Hkv > 65535 || dk % 64 || dk < 64 || dk > 192 || (dv != 64 && dv != 128) || out_d % 8 || out_d > dv || out_d < 1) return -20;
   if ((page != 16 && page != 32 && page % 64) || scale <= 0.f) return -20;
   if (window < 0 || (gate && (ld_gate % 8 || ld_gate < Hq * out_d || reinterpret_cast<uintptr_t>(gate) % 16))) return -2;
   Params p{};
@@ -371,8 +394,28 @@ extern "C" int rb_paged_flash(const void* q, const void* kc, const void* vc, con
   p.H = Hq; p.G = G; p.tokens = BQ / G; p.max_blocks = max_blocks; p.page = page; p.out_d = out_d;
   p.scale_log2 = scale * 1.4426950408889634f;
   p.err = err;
-  if (dk == 128 && dv == 128) return launch<128, 128>(q, kc, vc, rows, Hkv, pool_rows, n, p, st);
-  if (dk == 128) return launch<128, 64>(q, kc, vc, rows, Hkv, pool_rows, n, p, st);
-  if (dv == 128) return launch<64, 128>(q, kc, vc, rows, Hkv, pool_rows, n, p, st);
-  return launch<64, 64>(q, kc, vc, rows, Hkv, pool_rows, n, p, st);
+  return dispatch({q, kc, vc, rows, n, Hkv, dk, dv, static_cast<long long>(Hq) * dk, static_cast<uint64_t>(pool_rows)}, p, st);
+}
+
+// The same without pages: segment s has its keys and values [rows][H][dk / dv] (dk up to 192, dv up to 128, multiples of 8) from row first[s] on, every
+// head its own.  q [rows][H][dk] with q_pitch elements between rows; out [rows][H][dv]; blocks: query tiles of at most 128 tokens; gate
+// [rows][ld_gate]: one per head (head_gate) or per output feature, or null.  Returns -20 for shapes outside that.
+extern "C" int rb_dense_flash(const void* q, long long q_pitch, const void* k, const void* v, const int* first, const int* blocks, const void* gate,
+                              int ld_gate, int head_gate, void* out, int rows, int n, int H, int dk, int dv, long long k_rows, float scale, int* err,
+                              cudaStream_t st) {
+  using namespace rb;
+  using namespace rb::pf;
+  if (rows <= 0 || n <= 0) return 0;
+  if (H < 1 || H > 65535 || dk % 8 || dk < 8 || dk > 192 || dv % 8 || dv < 8 || dv > 128 || q_pitch % 8 || q_pitch < static_cast<long long>(H) * dk || scale <= 0.f)
+    return -20;
+  const uintptr_t bases = reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(k) | reinterpret_cast<uintptr_t>(v);
+  if (bases % 16 || !first || !blocks) return -2;
+  if (gate && !head_gate && (ld_gate % 8 || ld_gate < H * dv || reinterpret_cast<uintptr_t>(gate) % 16)) return -2;
+  Params p{};
+  p.blocks = blocks; p.first_row = first; p.out = (__nv_bfloat16*)out;
+  p.gate = (const __nv_bfloat16*)gate; p.ld_gate = ld_gate; p.head_gate = head_gate; p.window = INT_MAX;
+  p.H = H; p.G = 1; p.tokens = BQ; p.max_blocks = 1; p.page = BKV; p.out_d = dv;
+  p.scale_log2 = scale * 1.4426950408889634f;
+  p.err = err;
+  return dispatch({q, k, v, rows, n, H, dk, dv, q_pitch, static_cast<uint64_t>(k_rows)}, p, st);
 }

@@ -14,7 +14,7 @@
 //  * latent_write   norm of the latent projection, scattered into the paged latent cache, with the rotation of the part of queries and
 //                  rows that carries positions
 //  * latent_attn    CUDA-core attention over paged latent rows (any sizes, fp32 or bf16)
-//  * glu, gates of attention outputs, and a CUDA-core GEMM for fp32 and for shapes that no tensor-core kernel takes
+//  * glu, gate_outputs, and a CUDA-core GEMM for fp32 and for shapes that no tensor-core kernel takes
 #include "stack_common.cuh"
 
 namespace rb {
@@ -782,26 +782,17 @@ __global__ void __launch_bounds__(128) latent_attn_kernel(const LatentParams p) 
     st(out + c, (w[0] * sm[c] + w[1] * sm[p.Rv + c] + w[2] * sm[2 * p.Rv + c] + w[3] * sm[3 * p.Rv + c]) * f);
 }
 
-// attention output [T][H][pitch] -> [T][H * dv] (which may be the same memory), scaled by the sigmoid of a gate per head or (features)
-// per output feature
+// attention output [T][n] times the sigmoid of a gate per feature, in place
 template <typename T>
-__global__ void gate_heads_kernel(const T* o, const T* __restrict__ gate, int ld_gate, T* out, int H, int pitch, int dv, int features) {
+__global__ void gate_outputs_kernel(T* o, const T* __restrict__ gate, int n, int ld_gate) {
   constexpr bool kExact = IsExact<T>::v;
   const long long t = blockIdx.x;
-  const int per = dv / 8;
-  for (int i = threadIdx.x; i < H * per; i += blockDim.x) {
-    const int h = i / per, c = (i - h * per) * 8;
-    F8 v = ld8(o + (t * H + h) * pitch + c);
-    if (features) {
-      const F8 g = ld8(gate + t * ld_gate + h * dv + c);
+  for (int c = threadIdx.x * 8; c < n; c += blockDim.x * 8) {
+    F8 v = ld8(o + t * n + c);
+    const F8 g = ld8(gate + t * ld_gate + c);
 #pragma unroll
-      for (int k = 0; k < 8; ++k) v.v[k] *= sigmoid<kExact>(g.v[k]);
-    } else {
-      const float g = sigmoid<true>(ld(gate + t * ld_gate + h));
-#pragma unroll
-      for (int k = 0; k < 8; ++k) v.v[k] *= g;
-    }
-    st8(out + (t * H + h) * dv + c, v);
+    for (int k = 0; k < 8; ++k) v.v[k] *= sigmoid<kExact>(g.v[k]);
+    st8(o + t * n + c, v);
   }
 }
 
@@ -1040,15 +1031,12 @@ extern "C" int rb_latent_attn(const void* q, const void* pool, const int* block_
   return fp32 ? launch_latent_attn<float>(p, rows, stm) : launch_latent_attn<bf16>(p, rows, stm);
 }
 
-// o [rows][H][pitch] -> out [rows][H * dv]; features: a gate per output feature ([rows][ld_gate >= H dv]), else one per head.  o and out may be
-// the same memory when pitch == dv.
-extern "C" int rb_gate_heads(const void* o, const void* gate, int ld_gate, void* out, int rows, int H, int pitch, int dv, int features, int fp32,
-                             cudaStream_t stm) {
+// o [rows][n] *= sigmoid(gate [rows][ld_gate])
+extern "C" int rb_gate_outputs(void* o, const void* gate, int ld_gate, int rows, int n, int fp32, cudaStream_t stm) {
   if (rows <= 0) return 0;
-  if (dv % 8 || dv > pitch || pitch % 8 || ld_gate < (features ? H * dv : H)) return -2;
-  if (features && (ld_gate % 8 || reinterpret_cast<uintptr_t>(gate) % 16)) return -2;
-  if (fp32) gate_heads_kernel<float><<<rows, 256, 0, stm>>>((const float*)o, (const float*)gate, ld_gate, (float*)out, H, pitch, dv, features);
-  else gate_heads_kernel<bf16><<<rows, 256, 0, stm>>>((const bf16*)o, (const bf16*)gate, ld_gate, (bf16*)out, H, pitch, dv, features);
+  if (n % 8 || ld_gate % 8 || ld_gate < n || (reinterpret_cast<uintptr_t>(o) | reinterpret_cast<uintptr_t>(gate)) % 16) return -2;
+  if (fp32) gate_outputs_kernel<float><<<rows, 256, 0, stm>>>((float*)o, (const float*)gate, n, ld_gate);
+  else gate_outputs_kernel<bf16><<<rows, 256, 0, stm>>>((bf16*)o, (const bf16*)gate, n, ld_gate);
   rb_note_launch(1);
   return static_cast<int>(cudaGetLastError());
 }

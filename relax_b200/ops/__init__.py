@@ -185,15 +185,16 @@ def latent_attention(q, pool, batch, block_size, scale, gate, rank=None):
     return ref.latent_attention(q, pool, batch.block_tables[n:], block_size, batch.ctx[n:], cu, scale, gate, rank)
 
 
-def flash_serves_dims(dtype, dk: int, dv: int) -> bool:
-    """Whether the flash kernel takes heads of ``dk`` query / key and ``dv`` value features (zero-padded to 128)."""
-    return not _force_ref() and dtype == torch.bfloat16 and max(dk, dv) <= 128
+def dense_flash_serves(dtype, dk: int, dv: int) -> bool:
+    """Whether :func:`dense_flash` takes heads of ``dk`` query / key and ``dv`` value features."""
+    return not _force_ref() and dtype == torch.bfloat16 and dk <= 192 and dv <= 128
 
 
-def flash_gated(q, k, v, cu_q, cu_k, scale, max_q, gate, features=False):
-    """Causal varlen attention on per-head keys / values whose widths may differ, every head's output (``features``: every output
-    feature) scaled by ``sigmoid(gate)``; returns ``[T, H * dv]``."""
-    return _cuda().flash_gated(q, k, v, cu_q, cu_k, scale, max_q, gate, features)
+def dense_flash(q, k, v, first, blocks, scale, gate=None, features=False):
+    """Causal attention on per-head keys and values ``[rows, H, dk / dv]`` (multiples of 8 that may differ), those of segment ``s`` from row
+    ``first[s]`` on; ``blocks``: query tiles of up to 128 rows.  Every head's output (``features``: every output feature) is scaled by
+    ``sigmoid(gate)``.  Returns ``[T, H * dv]``."""
+    return _cuda().dense_flash(q, k, v, first, blocks, scale, gate, features)
 
 
 def linear(x, w, bias=None):

@@ -494,7 +494,7 @@ def head_linear(x, w, transposed, gate=None):
         return out
     _load().simt_gemm(x.transpose(0, 1), w, out.transpose(0, 1), not transposed)      # 32-bit mode
     if gate is not None:
-        _load().gate_heads(out, gate, out, out.shape[2], True)
+        _load().gate_outputs(out, gate)
     return out
 
 
@@ -536,14 +536,10 @@ def latent_attention(q, pool, b, block_size, scale, gate, rank=None):
     return out
 
 
-def flash_gated(q, k, v, cu_q, cu_k, scale, max_q, gate, features=False):
-    F = torch.nn.functional
-    dk, dv = q.shape[-1], v.shape[-1]
-    q, k = (t if dk == 128 else F.pad(t, (0, 128 - dk)) for t in (q, k))
-    v = v if dv == 128 else F.pad(v, (0, 128 - dv))
-    o = attention_varlen(q, k, v, cu_q, True, scale, cu_k, max_q)
-    out = torch.empty(q.shape[0], q.shape[1] * dv, dtype=q.dtype, device=q.device)
-    _load().gate_heads(o, gate, out, int(dv), bool(features))
+def dense_flash(q, k, v, first, blocks, scale, gate=None, features=False):
+    out = torch.empty(q.shape[0], q.shape[1] * v.shape[2], dtype=q.dtype, device=q.device)
+    if not _load().dense_flash(q, k, v, first, blocks, gate, bool(features), out, float(scale), err_flag(q.device)):
+        raise ValueError(f"no kernel for heads of {q.shape[2]} / {v.shape[2]} features, {q.dtype}")
     return out
 
 

@@ -5,8 +5,8 @@ Two tables, random weights, bf16, one GPU:
 * kernels: device time per launch, algorithmic bytes or FLOPs, fraction of the measured copy bandwidth / cuBLAS rate
   (``--peaks``), each kernel of the composed stack beside the like kernel of the existing models;
 * models: prefill and decode tokens/s through the engine's scheduler - a Talizen stack beside the Gated-DeltaNet hybrid and
-  the dense softmax model, or a Ketolorn stack beside the mixture-of-experts model, with the same width, heads,
-  feed-forward bytes and depth.
+  the dense softmax model, a Ketolorn stack beside the mixture-of-experts model, or a Zupupel stack beside a Ketolorn stack, with
+  the same width, heads, feed-forward bytes and depth.
 
 Times come from CUDA events after warm-up; every kernel rotates through inputs larger than the L2 cache.
 """
@@ -52,7 +52,7 @@ def _graph(fn):
 def kernel_rows(H=32, d=128, R=512, W=4096, F=12288, groups=8, only=""):
     """``(kernel, case, ms, bytes, flops)`` for decode batches and prompts of one real-sized layer."""
     from .. import ops
-    from .composed import SegmentBatch, recurrent_spans
+    from .composed import SegmentBatch, query_blocks, recurrent_spans
 
     dev, bf = "cuda", torch.bfloat16
     rows = []
@@ -123,7 +123,8 @@ def kernel_rows(H=32, d=128, R=512, W=4096, F=12288, groups=8, only=""):
         cu, ctx, sl = i32([i * L for i in range(S + 1)]), i32([L] * S), i32(list(range(S)))
         rows.append(("hgrn2 prompt", f"{S} x {L}", _time([lambda: ops.hgrn2(x, fb, lo, nw, st, sl, ctx, cu, H, d, d, 1e-5, spans)], 10), T * H * d * 4 * 2, 6.0 * T * H * d * d))
         q, k, v, g = mk(T, H, d), mk(T, H, d), mk(T, H, d), mk(T, H)
-        rows.append(("flash + gate (prompt)", f"{S} x {L}", _time([lambda: ops.flash_gated(q, k, v, cu, cu, 0.08, L, g)], 10), T * H * d * 8, 2.0 * T * L * H * d))
+        first, tiles = i32([i * L for i in range(S)]), i32(query_blocks([L] * S, [L] * S, 128))
+        rows.append(("flash + gate (prompt)", f"{S} x {L}", _time([lambda: ops.dense_flash(q, k, v, first, tiles, 0.08, g)], 10), T * H * d * 8, 2.0 * T * L * H * d))
         rows.append(("  like: flash attention", f"{S} x {L}", _time([lambda: ops.attention_varlen(q, k, v, cu, True, 0.08, cu, L)], 10), T * H * d * 8, 2.0 * T * L * H * d))
     for n, L in ((4, 2048), (64, 2048)) if want("attn") else ():
         from .composed import attention_items
@@ -249,6 +250,167 @@ def ketolorn_kernel_rows(W=2048, H=32, G=4, d=128, E=128, k=8, F=1152, only=""):
     return rows
 
 
+@torch.no_grad()
+def zupupel_kernel_rows(W=2048, H=32, G=4, d=128, window=1024, R=512, rot=64, E=128, I=16, k=8, F=768, only=""):
+    """The kernels of one real-sized Zupupel layer of each kind, each beside the like kernel of Ketolorn or Talizen stacks."""
+    from dataclasses import replace
+
+    from .. import ops
+    from ..models.config import LayerSpec, MoESpec
+    from .composed import SegmentBatch, attention_items, query_blocks, tile_tokens
+
+    dev, bf = "cuda", torch.bfloat16
+    rows = []
+    mk = lambda *s: torch.randn(*s, device=dev).to(bf)
+    i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
+    want = lambda section: not only or section in only.split(",")
+    freq = torch.tensor([1e6 ** (-2 * i / rot) for i in range(rot // 2)], dtype=torch.float64, device=dev)
+    sink, scale, page = mk(H), d ** -0.5, 64
+    for B in (16, 128) if want("attn") else ():
+        for L, win in ((8192, window), (window, 0)):
+            seen = min(L, window)
+            nbytes = B * seen * G * d * 4
+            bt = torch.randperm(B * L // page, device=dev).to(torch.int32).view(B, L // page)
+            b = SegmentBatch(None, None, torch.full((B,), L, dtype=torch.int32, device=dev), bt, None, max_ctx_one=L)
+            fns = []
+            for _ in range(_copies(nbytes) if B * L < 1 << 20 else 2):
+                kc, vc, q, g = mk(B * L, G, d), mk(B * L, G, d), mk(B, H, d), mk(B, H * d)
+                extra = dict(window=win, gate=g) if win else {}
+                fns.append(_graph(lambda q=q, kc=kc, vc=vc, extra=extra: ops.paged_attention(q, kc, vc, b, page, scale, None if win else sink, d, **extra)))
+            name = f"attention decode, window {win}, gate" if win else "  like: attention decode + sink (Ketolorn)"
+            rows.append((name, f"batch {B}, context {L}", _time(fns), nbytes, None))
+            del fns, kc, vc, q
+    spec = LayerSpec("attention", heads=H, dim=d, vdim=d, kv_heads=G)
+    for S, n, L in ((1, 8192, 8192), (4, 2048, 2048), (32, 256, 256), (16, 64, 2048), (16, 4, 2048)) if want("prompt") else ():
+        T, nb, t = S * n, L // page, tile_tokens(spec)
+        bt = torch.randperm(S * nb, device=dev).to(torch.int32).view(S, nb)
+        q, kc, vc, g = mk(T, H, d), mk(S * L, G, d), mk(S * L, G, d), mk(T, H * d)
+        b = SegmentBatch(None, None, i32([L] * S), bt, None, cu=i32([i * n for i in range(S + 1)]), multi_segs=S, multi_rows=T,
+                         blocks={t: i32(query_blocks([n] * S, [L] * S, t))})
+        for win in (window, 0):
+            flops = 4.0 * S * H * d * sum(min(win or L, L - n + i + 1) for i in range(n))
+            extra = dict(window=win, gate=g) if win else {}
+            rows.append((f"paged flash, window {win}, gate" if win else "  like: paged flash + sink (Ketolorn)", f"{S} x {n} tokens, context {L}",
+                         _time([_graph(lambda: ops.paged_attention(q, kc, vc, b, page, scale, None if win else sink, d, **extra))], 10),
+                         T * H * d * (6 if win else 4) + S * min(L, (win or L) + n) * G * d * 4, flops))
+    for B, L in ((16, 2048), (16, 8192), (128, 2048), (128, 8192)) if want("latent") else ():
+        bt = torch.randperm(B * L // page, device=dev).to(torch.int32).view(B, L // page)
+        b = SegmentBatch(None, None, torch.full((B,), L, dtype=torch.int32, device=dev), bt, None, max_ctx=L)
+        for r, name in ((rot, "latent decode, rotated part"), (0, "  like: latent decode + gate (Talizen)")):
+            fns = []
+            for _ in range(_copies(B * L * (R + r) * 2)):
+                pool, q, g = mk(B * L, R + r), mk(B, H, R + r), mk(B, H)
+                fns.append(_graph(lambda pool=pool, q=q, g=g, r=r: ops.latent_attention(q, pool, b, page, 0.05, None if r else g, R)))
+            rows.append((name, f"batch {B}, context {L}", _time(fns), B * L * (R + r) * 2, None))
+            del fns, pool
+    for n, L in ((4, 2048), (64, 2048)) if want("latent") else ():
+        S = 16
+        bt = torch.randperm(S * L // page, device=dev).to(torch.int32).view(S, L // page)
+        for r, name in ((rot, "latent portions, rotated part"), (0, "  like: latent portions + gate (Talizen)")):
+            width = ops.latent_columns(R + r, R)
+            q, pool, g = mk(S * n, H, R + r), mk(S * L, R + r), mk(S * n, H)
+            b = SegmentBatch(None, None, i32([L] * S), bt, None, cu=i32([0]), max_ctx=L, items={H: i32(attention_items([n] * S, [L] * S, H, width))},
+                             item_width={H: width})
+            rows.append((name, f"{S} x {n} tokens, context {L}", _time([_graph(lambda r=r: ops.latent_attention(q, pool, b, page, 0.05, None if r else g, R))]),
+                         S * L * (R + r) * 2, 2.0 * S * n * L * (2 * R + r) * H))
+    for S, L in ((1, 8192), (4, 2048), (32, 256)) if want("latent") else ():
+        T = S * L
+        first, tiles = i32([i * L for i in range(S)]), i32(query_blocks([L] * S, [L] * S, 128))
+        for r, name in ((rot, "flash of a latent prompt, rotated part, feature gate"), (0, "  like: flash + head gate (Talizen)")):
+            q, kk, v, g = mk(T, H, d + r), mk(T, H, d + r), mk(T, H, d), mk(T, H * d if r else H)
+            rows.append((name, f"{S} x {L}", _time([_graph(lambda r=r: ops.dense_flash(q, kk, v, first, tiles, 0.08, g, bool(r)))], 10),
+                         T * H * (4 * d + 2 * r) * 2, 1.0 * S * L * (L + 1) * H * (2 * d + r)))
+    for T in (16, 128, 8192) if want("prep") else ():
+        n = _copies(T * (H + 2 * G) * d * 4)
+        pos, slots = torch.arange(T, device=dev).to(torch.int32), torch.randperm(T, device=dev)
+        tab, kp, vp, qw, kw = ops.rope_table(pos, 0, freq), mk(T, G, d), mk(T, G, d), mk(H * d), mk(G * d)
+        xs = [mk(T, (H + 2 * G) * d) for _ in range(n)]
+        nb = T * (H + 2 * G) * d * 4
+        rows.append(("projection norms + rotation + cache write", f"{T} rows",
+                     _time([_graph(lambda x=x: ops.projection_inputs(x, qw, kw, tab, H, G, d, d, d, rot, True, 1e-6, kp, vp, slots)) for x in xs]), nb, None))
+        rows.append(("  like: rotation + head norm + cache write (Ketolorn)", f"{T} rows",
+                     _time([_graph(lambda x=x: ops.attention_inputs(x, tab, H, G, d, d, d, rot, 1e-6, kp, vp, slots)) for x in xs]), nb, None))
+        del xs
+        pool, w = mk(T, R + rot), mk(R)
+        xs = [mk(T, H * (d + rot) + R + rot) for _ in range(n)]
+        parts = lambda x: x.split([H * (d + rot), R, rot], 1)
+        rows.append(("latent row: norm, rotation, queries' rotation", f"{T} rows",
+                     _time([_graph(lambda x=x: ops.latent_write(parts(x)[1], w, R, 1e-6, pool, slots, (parts(x)[0].view(T, H, d + rot), parts(x)[2], tab, R, rot, d)))
+                            for x in xs]), T * (R * 4 + rot * 4 + H * rot * 4), None))
+        plain = mk(T, R)
+        rows.append(("  like: latent row: norm (Talizen)", f"{T} rows", _time([_graph(lambda x=x: ops.latent_write(parts(x)[1], w, R, 1e-6, plain, slots)) for x in xs]),
+                     T * R * 4, None))
+        del xs
+    for B in (16, 128) if want("gemm") else ():
+        x, o, g = mk(B, H, d + rot), mk(B, H, R), mk(B, H * d)
+        wide, narrow = [mk(H, d + rot, R + rot) for _ in range(_copies(H * d * R * 2))], [mk(H, d, R) for _ in range(_copies(H * d * R * 2))]
+        alg = H * d * R * 2 + B * H * (d + R + 2 * rot) * 2      # (the identity rows of the key map are not counted)
+        rows.append(("head_gemm fold with the rotated part", f"batch {B}", _time([_graph(lambda w=w: ops.head_linear(x, w, False)) for w in wide]), alg, None))
+        y = x[..., :d].contiguous()
+        rows.append(("  like: head_gemm fold (Talizen)", f"batch {B}", _time([_graph(lambda w=w: ops.head_linear(y, w, False)) for w in narrow]),
+                     H * d * R * 2 + B * H * (d + R) * 2, None))
+        rows.append(("head_gemm unfold + feature gate", f"batch {B}", _time([_graph(lambda w=w: ops.head_linear(o, w, True, g)) for w in narrow]),
+                     H * d * R * 2 + B * H * (2 * d + R) * 2, None))
+        rows.append(("  like: head_gemm unfold (Talizen)", f"batch {B}", _time([_graph(lambda w=w: ops.head_linear(o, w, True)) for w in narrow]),
+                     H * d * R * 2 + B * H * (d + R) * 2, None))
+    mine = MoESpec(experts=E, top=k, ff=F, groups=8, keep=4, act="clamped_swish", limit=7.0, renormalize=True, score="softmax", correction=True, identity=I,
+                   group_best=1)
+    like = MoESpec(experts=E, top=k, ff=F * 3 // 2, groups=8, keep=4)
+    corr = torch.zeros(E + I, device=dev, dtype=bf)
+    route = lambda spec, z: ops.moe_route(z, spec, bf, None, corr if spec.correction else None)
+    for T in (1, 16, 128, 8192) if want("moe") else ():
+        h = mk(T, W)
+        for spec, name in ((mine, "gated expert products (gather, both halves, unit, down)"), (like, "  like: squared-relu expert products (Ketolorn)")):
+            up, down = mk(E, 2 * F if spec.gated else F * 3 // 2, W), mk(E, W, spec.ff)
+            plans = [route(spec, torch.randn(T, spec.outputs, device=dev)) for _ in range(1 if T > 1000 else 4)]      # each touches other experts
+            hit = [int((p.offset[1:] > p.offset[:-1]).sum()) for p in plans]
+            used = sum(int(p.offset[-1]) for p in plans) / len(plans)
+            nb = sum(hit) / len(hit) * 3 * F * W * 2 + used * (2 * W + 2 * spec.ff) * 2
+            rows.append((name, f"{T} rows ({used:.0f} expert rows)",
+                         _time([_graph(lambda p=p: ops.moe_experts(h, p, up, down, spec.act, spec.limit)) for p in plans], 10), nb,
+                         6.0 * used * F * W if T > 1000 else None))
+            del up, down
+        for spec, name in ((mine, "routing (softmax, correction, identity) and layout"), (like, "  like: routing and layout (Ketolorn)")):
+            z = torch.randn(T, spec.outputs, device=dev)
+            rows.append((name, f"{T} rows", _time([_graph(lambda: route(spec, z))]), T * spec.outputs * 4 + T * k * 16, None))
+    for T in (16, 128, 8192) if want("norm") else ():
+        n = _copies(T * W * (12 + 2 * k))
+        w, bias = mk(W), mk(W)
+        plans = {s: route(s, torch.randn(T, s.outputs, device=dev)) for s in (mine, replace(like, shared_ff=8))}
+        buf = [(torch.randn(T, W, device=dev), mk(T, W), mk(T * k, W)) for _ in range(n)]
+        pm, pl = plans.values()
+        used = int(pm.offset[-1])
+        rows.append(("sum_norm with expert rows", f"{T} rows", _time([_graph(lambda r=r, e=e: ops.sum_norm(r, None, w, bias, W, 1.5, 1e-6, None, 1.0, (e, pm))) for r, _, e in buf]),
+                     T * W * 10 + used * W * 2, None))
+        rows.append(("  like: norm_add with expert rows (Ketolorn)", f"{T} rows",
+                     _time([_graph(lambda r=r, e=e: ops.norm_add(r, None, w, W, 1, 1e-6, None, (e, pl))) for r, _, e in buf]), T * W * (10 + 2 * k), None))
+        rows.append(("sum_norm", f"{T} rows", _time([_graph(lambda r=r, y=y: ops.sum_norm(r, y, w, bias, W, 1.5, 1e-6)) for r, y, _ in buf]), T * W * 12, None))
+        rows.append(("  like: norm_add", f"{T} rows", _time([_graph(lambda r=r, y=y: ops.norm_add(r, y, w, W, 1, 1e-6)) for r, y, _ in buf]), T * W * 12, None))
+        rows.append(("sum_norm and the final norm", f"{T} rows", _time([_graph(lambda r=r, y=y: ops.sum_norm(r, y, w, bias, W, 1.5, 1e-6, (w, bias), 0.1)) for r, y, _ in buf]),
+                     T * W * 12, None))
+        rows.append(("  like: norm_add and the final norm", f"{T} rows", _time([_graph(lambda r=r, y=y: ops.norm_add(r, y, w, W, 1, 1e-6, w)) for r, y, _ in buf]),
+                     T * W * 12, None))
+        del buf
+    return rows
+
+
+def _zupupel_models(layers: int, W: int, H: int, G: int, experts: int, top: int, ff: int, vocab: int):
+    """A Zupupel stack and a Ketolorn stack with experts of the same bytes in every layer (no shared expert)."""
+    from dataclasses import replace
+
+    from ..models.config import LayerSpec, MoESpec, composed_config, window_latent_layers
+
+    d = 128
+    att = LayerSpec("attention", heads=H, dim=d, vdim=d, kv_heads=G, scale=d ** -0.5, rot_dims=64, rot_base=1e6)
+    lat = LayerSpec("latent_attention", heads=H, dim=d, vdim=d, kv_rank=512, scale=192 ** -0.5, rot_dims=64, rot_base=1e6, out_gate=True)
+    mine = MoESpec(experts=experts, top=top, ff=ff, groups=8, keep=4, act="clamped_swish", limit=7.0, renormalize=True, score="softmax", correction=True,
+                   identity=experts // 8, group_best=1)
+    like = MoESpec(experts=experts, top=top, ff=ff * 3 // 2, groups=8, keep=4)
+    return {"zupupel": composed_config("zupupel", window_latent_layers(layers, replace(att, rot_halves=True, proj_norm=True, window=1024, out_gate=True), lat, mine), W,
+                                       vocab, norm_sum=True, sum_alpha=2.0, embed_scale=W ** 0.5, logit_scale=W ** -0.5),
+            "ketolorn": composed_config("ketolorn", [replace(att, qk_norm=True, sink=True, moe=like) for _ in range(layers)], W, vocab, embed_norm=True)}
+
+
 def _ketolorn_models(layers: int, W: int, H: int, G: int, experts: int, top: int, ff: int, dense_ff: int, vocab: int):
     """A Ketolorn stack (squared-relu experts of 3 / 2 the width: the same bytes as gated ones) and the mixture-of-experts model."""
     from ..models.config import LayerSpec, ModelConfig, MoESpec, composed_config, shared_kv_layers
@@ -280,7 +442,9 @@ def model_rows(size: str, only=None, decode_batches=(1, 32, 128), prompt=2048, d
     """``(model, workload, tokens/s, ms)`` through ``RolloutEngine.step``."""
     from .engine import RolloutEngine, SamplingParams
 
-    if design == "ketolorn":
+    if design == "zupupel":
+        models = _zupupel_models(*{"1b": (9, 2048, 32, 4, 128, 8, 768), "5b": (9, 4096, 64, 8, 128, 8, 1536)}[size], 64000)
+    elif design == "ketolorn":
         models = _ketolorn_models(*{"1b": (8, 2048, 32, 4, 128, 8, 768, 6144), "5b": (8, 4096, 64, 8, 128, 8, 1536, 12288)}[size], 64000)
     else:
         models = _models(*{"1b": (8, 2048, 16, 8192), "5b": (8, 4096, 32, 12288)}[size], 64000)
@@ -339,7 +503,7 @@ def main(size: str = "5b", peaks: str = "MEASURED_PEAKS.json", kernels: bool = T
     hbm, tf = pk.get("hbm_gbs"), pk.get("bf16_tflops")
     if kernels:
         print("kernel | case | us | GB/s (of measured copy) | TFLOP/s (of measured GEMM)")
-        for k, case, ms, nb, fl in (ketolorn_kernel_rows if design == "ketolorn" else kernel_rows)(only=only):
+        for k, case, ms, nb, fl in {"talizen": kernel_rows, "ketolorn": ketolorn_kernel_rows, "zupupel": zupupel_kernel_rows}[design](only=only):
             gb = nb / ms / 1e6
             t = f"{gb:7.0f}" + (f" ({gb / hbm:.2f})" if hbm else "")
             if fl:
@@ -357,8 +521,9 @@ if __name__ == "__main__":
     import argparse
 
     ap = argparse.ArgumentParser(description="kernel table of composed stacks")
-    ap.add_argument("--design", choices=["talizen", "ketolorn"], default="talizen")
-    ap.add_argument("--only", default="", help="sections, with commas: step, attn, gemm, norm, prompt (talizen); attn, prompt, prep, moe, norm, gemm (ketolorn)")
+    ap.add_argument("--design", choices=["talizen", "ketolorn", "zupupel"], default="talizen")
+    ap.add_argument("--only", default="", help="sections, with commas: step, attn, gemm, norm, prompt (talizen); attn, prompt, prep, moe, norm, gemm (ketolorn); "
+                                               "attn, prompt, latent, prep, gemm, moe, norm (zupupel)")
     ap.add_argument("--peaks", default="MEASURED_PEAKS.json")
     a = ap.parse_args()
     raise SystemExit(main(peaks=a.peaks, models=False, only=a.only, design=a.design))

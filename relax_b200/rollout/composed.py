@@ -132,9 +132,8 @@ class SegmentBatch:
     cu: Optional[torch.Tensor] = None        # [S + 1] int32
     long_segs: int = 0
     long_rows: int = 0
-    long_cu: Optional[torch.Tensor] = None   # [long + 1] int32 rows / context rows of the long segments
-    long_cu_k: Optional[torch.Tensor] = None
-    long_max: int = 0
+    long_first: Optional[torch.Tensor] = None   # [long] int32 first row of a long segment's context among ``ctx_slots``
+    long_blocks: Optional[torch.Tensor] = None  # [n, 4] int32 query tiles of the long segments (see :func:`query_blocks`)
     ctx_slots: Optional[torch.Tensor] = None  # pool rows of the long segments' whole contexts
     short_cu: Optional[torch.Tensor] = None
     row_seg: Optional[torch.Tensor] = None   # [short rows] int32: segment (among the short ones) and last visible position
@@ -327,7 +326,7 @@ class ComposedForward:
         if n:
             c = pool[b.ctx_slots]
             k, v = ops.linear(c, uk).view(-1, H, dp), ops.linear(c[:, :Rp], uv).view(-1, H, vp)
-            parts.append(ops.flash_gated(q[:n], k, v, b.long_cu, b.long_cu_k, s.scale, b.long_max, gate[:n], s.out_gate))
+            parts.append(ops.dense_flash(q[:n], k, v, b.long_first, b.long_blocks, s.scale, gate[:n], s.out_gate))
         if n < T:
             ql = ops.head_linear(q[n:], uk.view(H, dp, row), False)
             o = ops.latent_attention(ql, pool, b, cache.block_size, s.scale, None if s.out_gate else gate[n:], Rp)
@@ -479,13 +478,9 @@ class ComposedScheduler:
                 for t in tiles:
                     arrays[f"blocks{t}"] = (query_blocks(lens[:n_multi], ctx, t), i32)
             if n_long:
-                arrays["long_cu"] = (cu[:n_long + 1], i32)
-                ck = [0]
-                for c in ctx[:n_long]:
-                    ck.append(ck[-1] + c)
-                arrays["long_cu_k"] = (ck, i32)
+                arrays["long_first"] = ([sum(ctx[:s]) for s in range(n_long)], i32)
+                arrays["long_blocks"] = (query_blocks(lens[:n_long], ctx, QUERY_ROWS), i32)
                 arrays["ctx_slots"] = ([x for j in order[:n_long] for x in self._slots(parts[j][0], 0, parts[j][0].fed + parts[j][1])], i64)
-                host["long_max"] = max(lens[:n_long])
             rec = [self.cfg.layer_specs[i].heads for i in self.cfg.layers_with("hgrn2")]
             cuts = recurrent_spans(lens, max(rec)) if rec and self.device.type == "cuda" else None
             if cuts is not None:

@@ -174,10 +174,10 @@ class RolloutEngine(SpeculativeMixin, ComposedScheduler):
             self.max_running = min(max_running, state_slots or max_running)
             self.sm = SlotManager(self.max_running + 1)
             self._scratch_slot = self.sm.alloc()      # padding rows of a graph bucket; never handed to a request
-            # flash attention on projected keys / values: the tensor-core kernel takes bf16 heads of up to 128 features
+            # flash attention on projected keys / values: the tensor-core kernel takes bf16 heads of up to 192 / 128 features
             latent = cfg.layers_with("latent_attention")
             self._long_portions = self.device.type == "cuda" and bool(latent) and all(
-                ops.flash_serves_dims(self.dtype, *self.weights.latent_dims(i)[:2]) for i in latent)
+                ops.dense_flash_serves(self.dtype, *self.weights.latent_dims(i)[:2]) for i in latent)
         self._alloc_kv()
         self.use_cuda_graph = use_cuda_graph and self.device.type == "cuda"
         self.max_model_len = max_model_len

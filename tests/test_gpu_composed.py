@@ -321,14 +321,19 @@ def test_latent_attention_single_keys(dtype, n):
 
 def test_flash_with_unequal_widths_and_gate():
     from relax_b200 import ops
+    from relax_b200.rollout.composed import query_blocks
 
     bf = torch.bfloat16
-    for H, dk, dv in ((3, 24, 16), (2, 128, 128), (4, 56, 72)):
+    for H, dk, dv in ((3, 24, 16), (2, 128, 128), (4, 56, 72), (2, 192, 128), (1, 136, 40)):
         lens, ctx = [200, 300], [450, 300]
         q, k, v = _rand(1, 500, H, dk, dtype=bf), _rand(2, 750, H, dk, dtype=bf), _rand(3, 750, H, dv, dtype=bf)
         g = _rand(4, 500, H, dtype=bf)
-        cq, ck = (torch.tensor(x, dtype=torch.int32, device="cuda") for x in ([0, 200, 500], [0, 450, 750]))
-        got = ops.flash_gated(q, k, v, cq, ck, 0.3, 300, g).view(500, H, dv)
+        cq, ck, tiles = (torch.tensor(x, dtype=torch.int32, device="cuda") for x in ([0, 200, 500], [0, 450, 750], query_blocks(lens, ctx, 128)))
+        got = ops.dense_flash(q, k, v, ck[:2].contiguous(), tiles, 0.3, g).view(500, H, dv)
+        wide = _rand(5, 500, H * dv + 24, dtype=bf)[:, 8:8 + H * dv]
+        fine = ops.dense_flash(q, k, v, ck[:2].contiguous(), tiles, 0.3, wide, True).view(500, H, dv)
+        bare = ops.dense_flash(q, k, v, ck[:2].contiguous(), tiles, 0.3).view(500, H, dv)
+        _close(fine, bare.to(F64) * torch.sigmoid(wide.to(F64)).view(500, H, dv), 2e-2)
         o = 0
         for s in range(2):
             kk, vv, qq = k[ck[s]:ck[s + 1]].to(F64), v[ck[s]:ck[s + 1]].to(F64), q[cq[s]:cq[s + 1]].to(F64)
