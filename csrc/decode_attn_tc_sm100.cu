@@ -278,6 +278,10 @@ decode_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_k, const __grid_co
       tc_fence_before();
       mbar_arrive(&bar_p[j & 1]);
     }
+    float opened[NH];                 // gates, fetched while the last products run
+#pragma unroll
+    for (int h = 0; h < NH; ++h)
+      opened[h] = p.num_splits == 1 && h < G && r < p.out_d ? open_gate(p.gate, static_cast<size_t>(b) * p.ld_gate + (kvh * G + h) * p.out_d + r) : 1.f;
     if (ok && n_tiles > 1) ok = mbar_wait(&bar_o[(n_tiles - 2) & 1], static_cast<uint32_t>((n_tiles - 2) >> 1) & 1, abort_flag, p.err);
     if (ok && n_tiles > 0) ok = mbar_wait(&bar_o[(n_tiles - 1) & 1], static_cast<uint32_t>((n_tiles - 1) >> 1) & 1, abort_flag, p.err);
     tc_fence_after();
@@ -304,9 +308,7 @@ decode_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_k, const __grid_co
         float ov = __uint_as_float(o[h]);
         if (p.num_splits == 1) {
           if (p.sink) join_sink(m_ref[h], __bfloat162float(p.sink[hq]), ov, l);
-          if (r < p.out_d)
-            p.out[(static_cast<size_t>(b) * p.Hq + hq) * p.out_d + r] =
-                __float2bfloat16(l > 0.f ? ov / l * open_gate(p.gate, static_cast<size_t>(b) * p.ld_gate + hq * p.out_d + r) : 0.f);
+          if (r < p.out_d) p.out[(static_cast<size_t>(b) * p.Hq + hq) * p.out_d + r] = __float2bfloat16(l > 0.f ? ov / l * opened[h] : 0.f);
         } else {
           const size_t pidx = (static_cast<size_t>(b) * p.Hq + hq) * p.num_splits + split;
           p.part_o[pidx * DT_D + r] = ov;

@@ -93,6 +93,15 @@ head_gemm_kernel(const __grid_constant__ CUtensorMap tma_x, const __grid_constan
     }
   } else {
     const int t = t0 + warp * 32 + lane;
+    // gates of 32 columns at a time are fetched ahead of their use
+    const __nv_bfloat16* gate = p.gate && t < p.T ? p.gate + static_cast<size_t>(t) * p.ld_gate + h * p.N + n0 : nullptr;
+    uint4 g[4];
+    auto fetch = [&](int c) {
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+        if (gate && c < 128 && n0 + c + i * 8 < p.N) g[i] = *reinterpret_cast<const uint4*>(gate + c + i * 8);
+    };
+    fetch(0);
     const bool ok = !dead && mbar_wait(done, 0, abort_flag, p.err);
     __syncwarp();
     tc_fence_after();
@@ -107,9 +116,8 @@ head_gemm_kernel(const __grid_constant__ CUtensorMap tma_x, const __grid_constan
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
           if (n0 + c + i * 8 < p.N) {      // N is a multiple of 8
-            if (p.gate) {
-              const uint4 g = *reinterpret_cast<const uint4*>(p.gate + static_cast<size_t>(t) * p.ld_gate + h * p.N + n0 + c + i * 8);
-              const uint32_t w[4] = {g.x, g.y, g.z, g.w};
+            if (gate) {
+              const uint32_t w[4] = {g[i].x, g[i].y, g[i].z, g[i].w};
 #pragma unroll
               for (int k = 0; k < 4; ++k) {
                 r[8 * i + 2 * k] = __float_as_uint(__fdividef(__uint_as_float(r[8 * i + 2 * k]), 1.f + __expf(-__uint_as_float(w[k] << 16))));
@@ -125,6 +133,7 @@ head_gemm_kernel(const __grid_constant__ CUtensorMap tma_x, const __grid_constan
           }
         }
       }
+      fetch(c + 32);
     }
   }
   if (*abort_flag) __nanosleep(50000);

@@ -61,8 +61,7 @@ struct Params {
 };
 
 // eight accumulators times sigmoid(gate)
-__device__ __forceinline__ void gate8(uint32_t* o, const __nv_bfloat16* gate) {
-  const uint4 g = *reinterpret_cast<const uint4*>(gate);
+__device__ __forceinline__ void gate8(uint32_t* o, const uint4& g) {
   const uint32_t w[4] = {g.x, g.y, g.z, g.w};
 #pragma unroll
   for (int k = 0; k < 4; ++k) {
@@ -291,6 +290,15 @@ paged_flash_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_const
       tc_fence_before();
       mbar_arrive(&bar_p[s]);
     }
+    // gates of 32 columns at a time are fetched ahead of their use
+    const __nv_bfloat16* gate = p.gate && !p.head_gate && mine ? p.gate + static_cast<size_t>(row0 + t) * p.ld_gate + head * p.out_d : nullptr;
+    uint4 g[4];
+    auto fetch = [&](int c) {
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+        if (gate && c + i * 8 < p.out_d) g[i] = *reinterpret_cast<const uint4*>(gate + c + i * 8);
+    };
+    fetch(0);
     if (ok) ok = mbar_wait(&bar_o[(n_blocks - 1) & 1], static_cast<uint32_t>((n_blocks - 1) >> 1) & 1, abort_flag, p.err);
     const bool all_ok = __all_sync(0xffffffffu, ok);
     tc_fence_after();
@@ -305,11 +313,15 @@ paged_flash_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_const
         uint32_t o[32];
         tmem_ld_32x32b_x32(tmem_base + T_O + lane_addr + c * 32, o);
         tmem_wait_ld();
+        if (gate) {
+#pragma unroll
+          for (int i = 0; i < 4; ++i) gate8(o + 8 * i, g[i]);
+          fetch(c * 32 + 32);
+        }
         if (mine) {
 #pragma unroll
           for (int i = 0; i < 4; ++i) {
             if (c * 32 + i * 8 < p.out_d) {
-              if (p.gate && !p.head_gate) gate8(o + 8 * i, p.gate + static_cast<size_t>(row0 + t) * p.ld_gate + head * p.out_d + c * 32 + i * 8);
               uint4 pk;
               pk.x = pack_bf16(__uint_as_float(o[8 * i]) * inv_l, __uint_as_float(o[8 * i + 1]) * inv_l);
               pk.y = pack_bf16(__uint_as_float(o[8 * i + 2]) * inv_l, __uint_as_float(o[8 * i + 3]) * inv_l);

@@ -73,32 +73,38 @@ template <int MAX>
 struct ExpertRows {
   long long at[MAX];      // first element of a choice's row, -1: identity expert
   float w[MAX];
-  int top;
-  // returns the sum of the identity experts' weights
-  __device__ __forceinline__ float gather(const int* expert, const int* place, const int* offset, const float* weight, long long row, int n, int experts,
+  // returns whether the token took identity experts
+  __device__ __forceinline__ bool gather(const int* expert, const int* place, const int* offset, const float* weight, long long row, int n, int experts,
                                           int pitch) {
+    bool identity = false;
     if (static_cast<int>(threadIdx.x) < n) {
       const long long i = row * n + threadIdx.x;
       const int e = expert[i];
-      at[threadIdx.x] = e < experts ? (static_cast<long long>(offset[e]) + place[i]) * pitch : -1;
+      identity = e >= experts;
+      at[threadIdx.x] = identity ? -1 : (static_cast<long long>(offset[e]) + place[i]) * pitch;
       w[threadIdx.x] = weight[i];
     }
-    if (threadIdx.x == 0) top = n;
-    __syncthreads();
-    float identity = 0.f;
-    for (int k = 0; k < n; ++k) identity += at[k] < 0 ? w[k] : 0.f;
-    return identity;
+    return __syncthreads_or(identity) != 0;
   }
-  template <int V, typename T>
-  __device__ __forceinline__ void add(const T* ex, float* a) const {
-    const int n = top;
+  // sum of the identity experts' weights
+  __device__ __forceinline__ float identity(int n) const {
+    float s = 0.f;
+    for (int k = 0; k < n; ++k) s += at[k] < 0 ? w[k] : 0.f;
+    return s;
+  }
+  template <int V, bool kIdentity, typename T>
+  __device__ __forceinline__ void add(const T* ex, int n, float* a) const {
 #pragma unroll 4
     for (int k = 0; k < n; ++k) {
       float b[V];
       const long long i = at[k];
+      if constexpr (kIdentity) {
 #pragma unroll
-      for (int j = 0; j < V; ++j) b[j] = 0.f;
-      if (i >= 0) ldv<V>(ex + i, b);
+        for (int j = 0; j < V; ++j) b[j] = 0.f;
+        if (i >= 0) ldv<V>(ex + i, b);
+      } else {
+        ldv<V>(ex + i, b);
+      }
       const float f = w[k];
 #pragma unroll
       for (int j = 0; j < V; ++j) a[j] += f * b[j];
@@ -115,7 +121,8 @@ __global__ void __launch_bounds__(NA_WARPS * 32) norm_add_kernel(const NormAddPa
   bool known = true;
   if constexpr (MODE == NA_SUM) {
     __shared__ ExpertRows<NA_MAX_TOP> s;
-    const float identity = s.gather(p.expert, p.place, p.offset, p.weight, row, p.top, p.experts, p.ldy);
+    const bool some = s.gather(p.expert, p.place, p.offset, p.weight, row, p.top, p.experts, p.ldy);
+    const float identity = some ? s.identity(p.top) : 0.f;
     const float* stream = p.res + row * p.pitch;
     const T* base = p.y ? static_cast<const T*>(p.y) + row * p.ldy : nullptr;
     const T* ex = static_cast<const T*>(p.ex);
@@ -124,11 +131,13 @@ __global__ void __launch_bounds__(NA_WARPS * 32) norm_add_kernel(const NormAddPa
 #pragma unroll
       for (int i = 0; i < V; ++i) a[i] = 0.f;
       if (base) ldv<V>(base + c, a);
-      s.add<V>(ex + c, a);
-      if (identity != 0.f) {
+      if (some) {
+        s.add<V, true>(ex + c, p.top, a);
         ldv<V>(stream + c, x);
 #pragma unroll
         for (int i = 0; i < V; ++i) a[i] += identity * x[i];
+      } else {
+        s.add<V, false>(ex + c, p.top, a);
       }
       stv<V>(ysum + c, a);
     }
@@ -245,8 +254,10 @@ __global__ void __launch_bounds__(NA_WARPS * 32) sum_norm_kernel(const SumNormPa
   const T* ex = static_cast<const T*>(p.ex);
   __shared__ ExpertRows<kExperts ? NA_MAX_TOP : 1> rows;
   float alpha = p.alpha;
+  bool some = false;
   if constexpr (kExperts) {
-    alpha += rows.gather(p.expert, p.place, p.offset, p.weight, row, p.top, p.experts, p.ldy);
+    some = rows.gather(p.expert, p.place, p.offset, p.weight, row, p.top, p.experts, p.ldy);
+    if (some) alpha += rows.identity(p.top);      // their output is the stream
   }
   auto total = [&](float v, int k) {      // over the CTA; every k is used once
     v = wsum(v);
@@ -268,7 +279,10 @@ __global__ void __launch_bounds__(NA_WARPS * 32) sum_norm_kernel(const SumNormPa
 #pragma unroll
       for (int i = 0; i < V; ++i) x[i] += a[i];
     }
-    if constexpr (kExperts) rows.template add<V>(ex + c, x);
+    if constexpr (kExperts) {
+      if (some) rows.template add<V, true>(ex + c, p.top, x);
+      else rows.template add<V, false>(ex + c, p.top, x);
+    }
 #pragma unroll
     for (int i = 0; i < V; ++i) sum += x[i];
     stv<V>(z + c, x);

@@ -458,6 +458,12 @@ def model_rows(size: str, only=None, decode_batches=(1, 32, 128), prompt=2048, d
                             block_size=page, max_running=136,
                             max_model_len=prompt + 256, memory_saver=False)
         eng.weights.flat.normal_(0, 0.02)
+        if design == "zupupel":      # rows of unit size and no bias of the choice: tokens spread over the experts
+            for key, t in eng.weights.p.items():
+                if key.endswith("norm"):
+                    t.fill_(1.0)
+                elif key.endswith(("norm_b", "moe_correction")):
+                    t.zero_()
         g = torch.Generator().manual_seed(0)
         prm = lambda n: torch.randint(0, cfg.vocab_size, (n,), generator=g).tolist()
 
