@@ -437,6 +437,17 @@ def save_hf_checkpoint(directory: str, cfg: ModelConfig, hf_state: dict, max_sha
         post_hook(directory)
 
 
+def checkpoint_shapes(directory: str) -> dict:
+    """Tensor name -> shape of the safetensors files in a folder (their headers only; empty without files)."""
+    from safetensors import safe_open
+
+    out = {}
+    for fn in sorted(f for f in os.listdir(directory) if f.endswith(".safetensors")):
+        with safe_open(os.path.join(directory, fn), framework="pt") as f:
+            out.update({k: tuple(f.get_slice(k).get_shape()) for k in f.keys()})
+    return out
+
+
 def load_hf_checkpoint(directory: str, dequantize: bool = True, dtype=None) -> dict:
     from safetensors import safe_open
 
@@ -522,7 +533,7 @@ def config_from_hf(path: str) -> ModelConfig:
         d = json.load(f)
     own = architecture_of(d)
     if own is not None:
-        return own.config_from_dict(d, os.path.basename(os.path.normpath(path)) or "model")
+        return own.config_from_dict(d, os.path.basename(os.path.normpath(path)) or "model", shapes=checkpoint_shapes(path))
     arch = (d.get("architectures") or [""])[0]
     heads = d["num_attention_heads"]
     kw = dict(name=os.path.basename(os.path.normpath(path)) or "hf", num_layers=d["num_hidden_layers"], hidden_size=d["hidden_size"],
@@ -570,7 +581,7 @@ def validate_against_hf(cfg: ModelConfig, path: str) -> None:
     hf = config_from_hf(path)
     if cfg.is_composed or hf.is_composed:
         names = ("layer_specs", "hidden_size", "vocab_size", "norm_groups", "norm_sum", "sum_alpha", "rms_norm_eps", "embed_norm", "embed_scale",
-                 "logit_scale", "tie_word_embeddings")
+                 "logit_scale", "logit_softcap", "pre_norm", "token_shift", "side_dim", "tie_word_embeddings")
         diff = [f"{n}: {getattr(cfg, n)} here, {getattr(hf, n)} in the checkpoint" for n in names if getattr(cfg, n) != getattr(hf, n)]
         if diff:
             raise ValueError("the model configuration does not match the checkpoint: " + "; ".join(diff))

@@ -1,11 +1,12 @@
 """Model designs that name themselves with an ``architecture`` key in ``config.json`` and bring their own configuration keys and
-tensor names: ``name -> module`` with ``config_from_dict(d, name, dtype)`` and ``load_tensors(cfg, tensors, rollout_weights)``.
+tensor names: ``name -> module`` with ``config_from_dict(d, name, dtype, shapes)`` and ``load_tensors(cfg, tensors, rollout_weights)``
+(``shapes``: tensor name -> shape of the checkpoint, for sizes that ``config.json`` leaves out).
 Checkpoints without the key are read as Hugging Face layouts (:mod:`relax_b200.checkpoint.hf`)."""
 from __future__ import annotations
 
-from . import ketolorn, talizen, zupupel
+from . import ketolorn, talizen, zoguzen, zupupel
 
-ARCHITECTURES = {m.ARCHITECTURE: m for m in (talizen, ketolorn, zupupel)}
+ARCHITECTURES = {m.ARCHITECTURE: m for m in (talizen, ketolorn, zupupel, zoguzen)}
 
 
 def architecture_of(config_json: dict):

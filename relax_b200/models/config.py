@@ -31,8 +31,9 @@ class VisionConfig:
 @dataclass(frozen=True)
 class MoESpec:
     """Routed feed-forward of a composed layer: ``experts`` small feed-forwards of width ``ff``, of which every token takes ``top`` by
-    the ``score`` (sigmoid or softmax) of its router logits.  ``act`` ``relu2``: ``down(relu(up h)^2)``; ``clamped_swish``:
-    ``down(g sigmoid(1.702 g) (u + 1))`` with ``g = min(gate h, limit)`` and ``u = up h`` clamped to ``+- limit``.  ``identity``
+    the ``score`` (sigmoid or softmax) of its router logits.  ``act`` ``relu2``: ``down(relu(up h)^2)``; ``swiglu``:
+    ``down(silu(gate h) * up h)``; ``clamped_swish``: ``down(g sigmoid(1.702 g) (u + 1))`` with ``g = min(gate h, limit)`` and
+    ``u = up h`` clamped to ``+- limit``.  ``identity``
     more router outputs stand for experts without weights whose output is ``h`` itself.  All outputs form ``groups`` equal
     groups of neighbours; only those of the ``keep`` groups whose ``group_best`` best scores have the largest sums can be taken.
     ``correction``: a learned offset per output that joins the scores for the choice, not for the weights.  ``shared_ff``: width of
@@ -68,7 +69,7 @@ class MoESpec:
 
     @property
     def gated(self) -> bool:
-        return self.act == "clamped_swish"
+        return self.act in ("clamped_swish", "swiglu")
 
 
 @dataclass(frozen=True)
@@ -77,11 +78,14 @@ class LayerSpec:
     feed-forward.  ``hgrn2``: gated linear recurrence with ``heads`` states of ``dim x vdim``.  ``latent_attention``:
     softmax attention whose keys and values are projections of one cached latent row of ``kv_rank`` features per token;
     with ``rot_dims`` every head's query has that many rotated features more, which meet ONE rotated key part that the row
-    holds for all heads.  ``attention``: softmax attention over cached keys and values of ``kv_heads`` heads."""
+    holds for all heads.  ``attention``: softmax attention over cached keys and values of ``kv_heads`` heads.  ``mingru``: ``vdim``
+    channels that each follow a gated running mean.  ``gla``: linear attention with ``heads`` states of ``dim x vdim`` whose rows decay by
+    gates of their own, read-outs normed head by head and gated.  ``pair``: the mixers of ``pair`` side by side on the same input;
+    the layer's output is half the sum of theirs, each RMS-normed over the model width with a weight."""
     mixer: str
-    heads: int
-    dim: int                     # query (and key / forget-gate) features per head (latent_attention: the unrotated ones)
-    vdim: int                    # value features per head
+    heads: int = 1
+    dim: int = 1                 # query (and key / forget-gate) features per head (latent_attention: the unrotated ones)
+    vdim: int = 1                # value features per head
     kv_rank: int = 0             # latent_attention only
     scale: float = 1.0           # attention mixers: factor on q . k
     ff: int = 0                  # width of the gated feed-forward; 0 = the layer has none
@@ -96,7 +100,20 @@ class LayerSpec:
     proj_norm: bool = False      # weighted RMS norm over all query rows, and over all key rows, before heads and rotation
     window: int = 0              # a position sees itself and the window - 1 before it; 0 = all before it
     sink: bool = False           # one learned logit per head in the softmax denominator, without key or value
+    unit_sink: bool = False      # a sink whose logit is 0 (one more in the softmax denominator)
     kv_from: int = -1            # >= 0: reads the keys and values that this earlier layer has cached, and has none of its own
+    keep_first: int = 0          # with a window: the first positions of a sequence stay visible
+    chunk: int = 0               # > 0: a position sees only those of its own chunk of this many, counted from the sequence's start
+    softcap: float = 0.0         # > 0: scores s become softcap * tanh(s / softcap)
+    talk: bool = False           # the heads' weights are mixed by a learned [heads, heads] matrix before they meet the values
+    qkv_bias: bool = False       # biases of the query, key and value projections
+    conv: int = 0                # > 0: taps of a causal convolution over time on every channel of the projected q, k and v
+    head_norm: bool = False      # queries and keys RMS-normed head by head with a weight (shared by heads), before they turn
+    rot_scaling: Optional[tuple] = None   # (factor, low, high, original): long wavelengths stretched as in Llama 3.1
+    # gla only
+    decay_rank: int = 0          # rank of the gates' projection
+    decay_root: float = 1.0      # gates are sigmoid(z) ** (1 / decay_root)
+    pair: Optional[tuple] = None          # pair only: two LayerSpecs without feed-forwards
     moe: Optional[MoESpec] = None  # routed feed-forward instead of the gated one
 
     def __post_init__(self):
@@ -115,6 +132,20 @@ class LayerSpec:
                 raise ValueError(f"bad rotation: {self.rot_dims} of {self.dim} features, base {self.rot_base}")
             if self.qk_norm and (self.proj_norm or self.rot_halves):
                 raise ValueError("queries and keys normed head by head turn in neighbouring pairs and have no norm over the projection")
+            if (self.conv or self.qkv_bias or self.head_norm) and (self.qk_norm or self.proj_norm or self.rot_halves):
+                raise ValueError("projections with biases, convolutions or weighted head norms turn in neighbouring pairs and have no other norm")
+            if not 0 <= self.conv <= MAX_TAPS or min(self.keep_first, self.chunk) < 0 or self.softcap < 0:
+                raise ValueError(f"bad attention: {self}")
+            if (self.window and self.chunk) or (self.keep_first and not self.window) or (self.sink and self.unit_sink) or (self.talk and self.out_gate):
+                raise ValueError(f"attention layers see a window (with or without first positions) or a chunk, have one sink, and gates or mixed heads: {self}")
+        if self.rot_scaling is not None and (len(self.rot_scaling) != 4 or min(self.rot_scaling) <= 0 or self.rot_scaling[1] >= self.rot_scaling[2]):
+            raise ValueError(f"bad rotation scaling: {self.rot_scaling}")
+        if self.mixer == "gla" and (self.decay_rank < 1 or self.decay_root <= 0):
+            raise ValueError(f"bad decay: {self}")
+        if (self.mixer == "pair") != (self.pair is not None):
+            raise ValueError(f"a pair has two mixers: {self}")
+        if self.pair is not None and (len(self.pair) != 2 or any(s.mixer == "pair" or s.has_ff or s.kv_from >= 0 for s in self.pair)):
+            raise ValueError("a pair is made of two plain mixers with inputs of their own and without feed-forwards")
 
     @property
     def has_ff(self) -> bool:
@@ -126,9 +157,10 @@ class LayerSpec:
         return self.mixer == "attention" and self.kv_from < 0
 
 
-MIXERS = ("hgrn2", "latent_attention", "attention")
+MIXERS = ("hgrn2", "latent_attention", "attention", "mingru", "gla", "pair")
+MAX_TAPS = 8           # of a short convolution
 ACTIVATIONS = ("silu", "gelu_tanh", "relu2")
-EXPERT_ACTIVATIONS = ("relu2", "clamped_swish")
+EXPERT_ACTIVATIONS = ("relu2", "clamped_swish", "swiglu")
 
 
 @dataclass
@@ -194,9 +226,12 @@ class ModelConfig:
     dsa_index_heads: int = 4
     dsa_index_dim: int = 16
     dsa_indexer_loss_coef: float = 1.0
-    # composed stacks (Talizen, Ketolorn, Zupupel): every layer is spelled out - mixer, sizes, feed-forward.  The sublayers read the
+    # composed stacks (Talizen, Ketolorn, Zupupel, Zoguzen): every layer is spelled out - mixer, sizes, feed-forward.  The sublayers read the
     # fp32 residual stream itself.  Their OUTPUT is normed (RMS over each of `norm_groups` equal parts) before it is added, or,
     # with `norm_sum`, the SUM is: x <- norm(sum_alpha * x + sublayer(x)), a layer norm with weight and bias (as is the final norm).
+    # With `pre_norm` the sublayers read norms of the stream instead (layer norms with a weight), and both join it at once:
+    # x <- x + mixer(norm1(x)) + ff(norm2(x)).  `token_shift`: what the mixer reads has moved towards the row before, by a weight per
+    # feature.  `side_dim`: every layer then adds the norm of a projection of gelu(gate x) times its own part of a second embedding.
     # The fields above that describe one uniform layer (heads, head_dim, ffn, rotary, MoE, ...) do not apply then.
     layer_specs: Optional[tuple] = None
     norm_groups: int = 1
@@ -205,15 +240,26 @@ class ModelConfig:
     embed_norm: bool = False               # the embedded tokens are normed before the first layer
     embed_scale: float = 1.0               # factor on the embedded tokens
     logit_scale: float = 1.0               # factor on the logits
+    logit_softcap: float = 0.0             # > 0: logits z become logit_softcap * tanh(z / logit_softcap)
+    pre_norm: bool = False
+    token_shift: bool = False
+    side_dim: int = 0                      # features per layer and token of the second embedding
     dtype: str = "bf16"
 
     @property
     def is_composed(self) -> bool:
         return self.layer_specs is not None
 
-    def layers_with(self, mixer: str) -> list:
-        """Indices of the layers of a composed stack that use ``mixer``."""
-        return [i for i, s in enumerate(self.layer_specs or ()) if s.mixer == mixer]
+    def mixers(self) -> list:
+        """``(key, spec)`` of every mixer of a composed stack: ``i`` for layer ``i``, ``(i, 0)`` and ``(i, 1)`` for the two of a pair."""
+        out = []
+        for i, s in enumerate(self.layer_specs or ()):
+            out += [((i, k), m) for k, m in enumerate(s.pair)] if s.pair is not None else [(i, s)]
+        return out
+
+    def specs_with(self, *mixers: str) -> list:
+        """Specs of the mixers of these kinds, those inside pairs included."""
+        return [s for _, s in self.mixers() if s.mixer in mixers]
 
     @property
     def is_moe(self) -> bool:
@@ -240,19 +286,13 @@ class ModelConfig:
         if self.is_composed:
             norm = 2 * h if self.norm_sum else h
             n = (1 if self.tie_word_embeddings else 2) * self.vocab_size * h + norm + (h if self.embed_norm else 0)
+            n += self.side_dim * self.num_layers * self.vocab_size
             for s in self.layer_specs:
-                n += norm + 3 * s.ff * h + (norm if s.has_ff else 0) + s.heads * s.vdim * h
+                n += norm + 3 * s.ff * h + (norm if s.has_ff else 0) + (h if self.token_shift else 0) + ((2 * self.side_dim + 1) * h if self.side_dim else 0)
                 if s.moe is not None:
                     n += s.moe.experts * (3 if s.moe.gated else 2) * s.moe.ff * h + 2 * s.moe.shared_ff * h
                     n += s.moe.outputs * (h + (1 if s.moe.correction else 0))
-                if s.mixer == "hgrn2":
-                    n += s.heads * (2 * s.dim + s.vdim) * h + 2 * s.heads * s.dim + s.vdim
-                elif s.mixer == "attention":
-                    n += s.heads * s.dim * h + (s.heads if s.sink else 0) + (s.kv_heads * (s.dim + s.vdim) * h if s.own_kv else 0)
-                    n += (s.heads * s.vdim * h if s.out_gate else 0) + ((s.heads + (s.kv_heads if s.own_kv else 0)) * s.dim if s.proj_norm else 0)
-                else:
-                    n += (s.heads * (s.dim + s.rot_dims + (s.vdim if s.out_gate else 1)) + s.kv_rank + s.rot_dims) * h
-                    n += s.kv_rank * (1 + s.heads * (s.dim + s.vdim))
+                n += self._mixer_parameters(s) if s.pair is None else 2 * h + sum(self._mixer_parameters(m) for m in s.pair)
             return n
         attn = h * (self.q_size * (2 if self.attention_output_gate else 1) + 2 * self.kv_size) + self.q_size * h
         if self.qk_layernorm:
@@ -265,6 +305,23 @@ class ModelConfig:
         emb = self.vocab_size * h
         out = 0 if self.tie_word_embeddings else self.vocab_size * h
         return L * per_layer + emb + out + h
+
+    def _mixer_parameters(self, s: LayerSpec) -> int:
+        h = self.hidden_size
+        n = s.heads * s.vdim * h
+        if s.mixer == "hgrn2":
+            return n + s.heads * (2 * s.dim + s.vdim) * h + 2 * s.heads * s.dim + s.vdim
+        if s.mixer == "mingru":
+            return n + 3 * s.vdim * h + 2 * s.vdim
+        if s.mixer == "gla":
+            return n + s.heads * (2 * s.dim + 2 * s.vdim) * h + s.decay_rank * (h + s.heads * s.dim) + s.heads * s.dim + s.vdim
+        if s.mixer == "attention":
+            cols = s.heads * s.dim + (s.kv_heads * (s.dim + s.vdim) if s.own_kv else 0)
+            n += cols * (h + s.conv + (1 if s.qkv_bias else 0)) + (s.heads if s.sink else 0) + (s.heads ** 2 if s.talk else 0)
+            n += (2 if s.own_kv else 1) * s.dim if s.head_norm else 0
+            return n + (s.heads * s.vdim * h if s.out_gate else 0) + ((s.heads + (s.kv_heads if s.own_kv else 0)) * s.dim if s.proj_norm else 0)
+        n += (s.heads * (s.dim + s.rot_dims + (s.vdim if s.out_gate else 1)) + s.kv_rank + s.rot_dims) * h
+        return n + s.kv_rank * (1 + s.heads * (s.dim + s.vdim))
 
     def to_dict(self):
         return asdict(self)
@@ -291,11 +348,16 @@ def composed_config(name: str, layers, hidden_size: int, vocab_size: int, norm_g
         raise ValueError("factors on the stream and on the logits join the norm after the sum")
     if kw.get("embed_norm") and kw.get("embed_scale", 1.0) != 1.0:
         raise ValueError("embedded tokens are normed or scaled")
+    if kw.get("pre_norm") and (norm_groups > 1 or kw.get("norm_sum") or kw.get("embed_norm") or kw.get("embed_scale", 1.0) != 1.0 or any(
+            s.ff or (s.moe and s.moe.shared_ff) for s in layers)):
+        raise ValueError("sublayers that read norms of the stream come with routed feed-forwards and without norms of their outputs or of embedded tokens")
+    if not kw.get("pre_norm") and (kw.get("token_shift") or kw.get("side_dim") or any(s.pair is not None for s in layers)):
+        raise ValueError("shifted tokens, a second embedding and pairs of mixers join sublayers that read norms of the stream")
     for i, s in enumerate(layers):
         if s.mixer == "attention" and s.kv_from >= 0:
             if s.kv_from >= i or not layers[s.kv_from].own_kv:
                 raise ValueError(f"layer {i} reads keys and values of layer {s.kv_from}, which has none before it")
-            what = ("kv_heads", "dim", "vdim", "rot_dims", "rot_base", "rot_halves", "qk_norm", "proj_norm")
+            what = ("kv_heads", "dim", "vdim", "rot_dims", "rot_base", "rot_scaling", "rot_halves", "qk_norm", "proj_norm", "head_norm")
             if any(getattr(s, f) != getattr(layers[s.kv_from], f) for f in what):
                 raise ValueError(f"layer {i} and the layer {s.kv_from} whose keys and values it reads differ in {what}")
     return ModelConfig(name=name, num_layers=len(layers), hidden_size=hidden_size, vocab_size=vocab_size, rms_norm_eps=eps,

@@ -29,7 +29,7 @@ def _feed_forward(i: int, mlp) -> dict:
                            keep=int(g["keep"]), shared_ff=int(shared["ff"]) if shared else 0)}
 
 
-def config_from_dict(d: dict, name: str = "ketolorn", dtype: str = "bf16") -> ModelConfig:
+def config_from_dict(d: dict, name: str = "ketolorn", dtype: str = "bf16", shapes=None) -> ModelConfig:
     layers = []
     for i, entry in enumerate(d["layers"]):
         m = entry["mixer"]
@@ -96,7 +96,7 @@ def load_tensors(cfg: ModelConfig, tensors: dict, weights) -> None:
         put(p[o + "post_attn_norm"], tensors[a + "norm1"])
         put(p[o + "attn_qkv"], torch.cat([tensors[m + k] for k in ("q", "k", "v") if m + k in tensors]))
         put(p[o + "attn_sink"], tensors[m + "sink"])
-        put(p[o + "attn_o"].view(-1, s.heads, weights.attention_dims(i)[2]), tensors[m + "o"].view(W, s.heads, s.vdim))
+        put(p[o + "attn_o"].view(-1, s.heads, weights.attention_dims(s)[2]), tensors[m + "o"].view(W, s.heads, s.vdim))
         if s.has_ff:
             put(p[o + "post_mlp_norm"], tensors[a + "norm2"])
         if s.ff:

@@ -6,6 +6,10 @@ import json
 import os
 
 
+def pad_to(n: int, m: int) -> int:
+    return (n + m - 1) // m * m
+
+
 def check_tensors(want: dict, tensors: dict) -> None:
     """Names and shapes must match exactly."""
     extra, missing = sorted(set(tensors) - set(want)), sorted(set(want) - set(tensors))

@@ -15,7 +15,7 @@ from .native import check_tensors, put, save_folder
 ARCHITECTURE = "Talizen"
 
 
-def config_from_dict(d: dict, name: str = "talizen", dtype: str = "bf16") -> ModelConfig:
+def config_from_dict(d: dict, name: str = "talizen", dtype: str = "bf16", shapes=None) -> ModelConfig:
     layers = []
     for i, entry in enumerate(d["layers"]):
         kind, m, mlp = entry["type"], entry["mixer"], entry.get("mlp")
@@ -82,7 +82,7 @@ def load_tensors(cfg: ModelConfig, tensors: dict, weights) -> None:
             put(p[o + "rec_norm"], tensors[m + "norm"])
             put(p[o + "rec_o"], tensors[m + "o"])
         else:
-            R, (dp, vp, Rp) = s.kv_rank, weights.latent_dims(i)
+            R, (dp, vp, Rp) = s.kv_rank, weights.latent_dims(s)
             w = p[o + "lat_qcg"]
             put(w[: H * dp].view(H, dp, -1), tensors[m + "q"].view(H, s.dim, W))
             put(w[H * dp:], tensors[m + "dkv"])

@@ -30,7 +30,7 @@ def _feed_forward(i: int, mlp) -> dict:
                            identity=int(r.get("identity") or 0), group_best=1)}
 
 
-def config_from_dict(d: dict, name: str = "zupupel", dtype: str = "bf16") -> ModelConfig:
+def config_from_dict(d: dict, name: str = "zupupel", dtype: str = "bf16", shapes=None) -> ModelConfig:
     layers = []
     for i, entry in enumerate(d["layers"]):
         m = entry["mixer"]
@@ -115,13 +115,13 @@ def load_tensors(cfg: ModelConfig, tensors: dict, weights) -> None:
         H = s.heads
         norm(o + "post_attn_norm", a + "norm1")
         if s.mixer == "attention":
-            w, vp = p[o + "attn_qkv"], weights.attention_dims(i)[2]
+            w, vp = p[o + "attn_qkv"], weights.attention_dims(s)[2]
             put(w, torch.cat([tensors[m + k] for k in ("q", "k", "v") if m + k in tensors]))
             for k in ("q", "k") if s.own_kv else ("q",):
                 put(p[f"{o}attn_{k}_norm"], tensors[f"{m}{k}.norm"])
             gate, out = weights.gate_column(s), p[o + "attn_o"]
         else:
-            dp, vp, Rp = weights.latent_dims(i)
+            dp, vp, Rp = weights.latent_dims(s)
             w, dkv = p[o + "lat_qcg"], tensors[m + "dkv"]
             put_heads(w[: H * dp], tensors[m + "q"], H)
             put(w[H * dp:], dkv[: s.kv_rank])

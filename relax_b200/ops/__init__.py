@@ -109,13 +109,23 @@ def projection_inputs(qkv, q_w, k_w, table, heads, kv_heads, dim, vdim, dp, rot_
                                                                   v_pool, slots)
 
 
-def paged_attention(q, k_pool, v_pool, batch, block_size, scale, sink, out_width, window=0, gate=None):
+def conv_inputs(qkv, bias, taps, state, batch, q_w, k_w, table, heads, kv_heads, dim, vdim, dp, rot_dims, eps, k_pool, v_pool):
+    """The same with biases, a causal convolution over time on every channel (its last rows carried in ``state`` by slot), and weighted
+    norms head by head (``eps`` <= 0: none) before neighbours turn."""
+    return (_cuda() if _use_cuda(qkv) else ref).conv_inputs(qkv, bias, taps, state, batch, q_w, k_w, table, heads, kv_heads, dim, vdim, dp, rot_dims, eps,
+                                                            k_pool, v_pool)
+
+
+def paged_attention(q, k_pool, v_pool, batch, block_size, scale, sink, out_width, window=0, gate=None, keep=0, chunk=0, softcap=0.0, talk=None):
     """Grouped-query attention over paged keys and values for every segment of a
     :class:`relax_b200.rollout.composed.SegmentBatch`, with an optional sink logit per head, an optional ``window`` (positions a
-    row sees, its own included; 0 = all) and an optional ``gate`` per output feature (``[T, heads * out_width]``, its sigmoid counts)."""
+    row sees, its own included; 0 = all) that leaves the first ``keep`` positions visible, or chunks of ``chunk`` positions, optionally capped
+    scores, an optional ``gate`` per output feature (``[T, heads * out_width]``, its sigmoid counts), and optionally heads whose weights
+    are mixed by ``talk[H, H]`` before they meet the values."""
     if _use_cuda(q):
-        return _cuda().paged_attention(q, k_pool, v_pool, batch, block_size, scale, sink, out_width, window, gate)
-    return ref.paged_attention(q, k_pool, v_pool, batch.block_tables, block_size, batch.ctx, batch.cu, scale, sink, out_width, window, gate)
+        return _cuda().paged_attention(q, k_pool, v_pool, batch, block_size, scale, sink, out_width, window, gate, keep, chunk, softcap, talk)
+    return ref.paged_attention(q, k_pool, v_pool, batch.block_tables, block_size, batch.ctx, batch.cu, scale, sink, out_width, window, gate, keep, chunk,
+                               softcap, talk)
 
 
 def route_counters(layers: int, experts: int, device):
@@ -154,6 +164,37 @@ def hgrn2(qfv, f_bias, lower, norm_w, state, state_slot, ctx_lens, cu, heads, di
     if _use_cuda(qfv):
         return _cuda().hgrn2(qfv, f_bias, lower, norm_w, state, state_slot, ctx_lens, cu, heads, dim, vdim, eps, spans)
     return ref.hgrn2(qfv, f_bias, lower, norm_w, state, state_slot, ctx_lens, cu, heads, dim, vdim, eps)
+
+
+def mingru(zxg, z_b, x_b, state, batch, width):
+    """Gated running means per channel, read out through ``silu`` gates, with the state carried in slots."""
+    return (_cuda() if _use_cuda(zxg) else ref).mingru(zxg, z_b, x_b, state, batch, width)
+
+
+def gla(rows, z, a2_b, norm_w, state, state_slot, ctx_lens, cu, heads, dim, vdim, gate_col, eps, root, spans=None):
+    """Linear attention whose state rows decay by gates of their own (recurrence, per-head norm, output gates), with the state carried in
+    slots; ``spans`` as for :func:`hgrn2`."""
+    if _use_cuda(rows):
+        return _cuda().gla(rows, z, a2_b, norm_w, state, state_slot, ctx_lens, cu, heads, dim, vdim, gate_col, eps, root, spans)
+    return ref.gla(rows, z, a2_b, norm_w, state, state_slot, ctx_lens, cu, heads, dim, vdim, gate_col, eps, root)
+
+
+def stream_step(res, width, eps, y=None, norm_w=None, experts=None, norms=(), shift=None):
+    """One pass over the fp32 stream ``res``: adds the mean of the rows in ``y`` (a list of one or two; with ``norm_w`` each is RMS-normed with
+    its weight first) and the weighted expert rows ``experts``, in place; returns a list with the stream's layer norm for every weight in
+    ``norms``, or with its copy in the weights' type.  ``shift``: ``(weights mu, state, batch)`` - the first norm's rows ``n`` become
+    ``n + (before - n) mu`` with ``before`` the row in front in the same sequence, from ``state`` (by slot) for a segment's first row."""
+    return (_cuda() if _use_cuda(res) else ref).stream_step(res, width, eps, y, norm_w, experts, norms, shift)
+
+
+def side_gate(z, embed, tokens, first, dim):
+    """``gelu_tanh(z)`` times a layer's own features of the tokens in a second embedding table."""
+    return (_cuda() if _use_cuda(z) else ref).side_gate(z, embed, tokens, first, dim)
+
+
+def softcap(z, cap):
+    """``cap * tanh(z / cap)`` of fp32 logits (in place on the GPU)."""
+    return (_cuda() if _use_cuda(z) else ref).softcap(z, cap)
 
 
 def latent_write(raw, w, rank, eps, pool, slots, turned=None):

@@ -243,11 +243,13 @@ def projection_inputs(qkv, q_w, k_w, table, heads: int, kv_heads: int, dim: int,
     return q
 
 
-def paged_attention(q, k_pool, v_pool, block_tables, block_size: int, ctx_lens, cu, scale: float, sink, out_width: int, window: int = 0, gate=None):
+def paged_attention(q, k_pool, v_pool, block_tables, block_size: int, ctx_lens, cu, scale: float, sink, out_width: int, window: int = 0, gate=None,
+                    keep: int = 0, chunk: int = 0, softcap: float = 0.0, talk=None):
     """Softmax attention of ``q[T, H, dp]`` over paged keys and values ``[rows, kv_heads, ...]`` of their sequence; row ``i`` of
-    a segment of ``n`` rows sees the first ``ctx - n + i + 1`` positions, with a ``window`` only the last ``window`` of those.
-    ``sink[H]``: a logit per head that only joins the denominator.  ``gate[T, H * out_width]``: its sigmoid multiplies the outputs.
-    Returns ``[T, H * out_width]``."""
+    a segment of ``n`` rows sees the first ``ctx - n + i + 1`` positions, with a ``window`` only the last ``window`` of those and the first
+    ``keep`` of the sequence, with a ``chunk`` only those of its own chunk.  ``softcap``: scores ``s`` become ``softcap tanh(s / softcap)``.
+    ``sink[H]``: a logit per head that only joins the denominator.  ``talk[H, H]``: mixes the heads' weights before they meet the values.
+    ``gate[T, H * out_width]``: its sigmoid multiplies the outputs.  Returns ``[T, H * out_width]``."""
     T, H, _ = q.shape
     G, rep = k_pool.shape[1], H // k_pool.shape[1]
     out = torch.zeros(T, H, out_width, dtype=torch.float32, device=q.device)
@@ -259,13 +261,20 @@ def paged_attention(q, k_pool, v_pool, block_tables, block_size: int, ctx_lens, 
         rows = block_tables[s].long()[pos // block_size] * block_size + pos % block_size
         k, v = k_pool[rows].float(), v_pool[rows].float()[..., :w]
         sc = torch.einsum("tgrd,lgd->tgrl", q[a:b].float().view(b - a, G, rep, -1), k).reshape(b - a, H, L) * scale
-        lim = L - (b - a) + torch.arange(b - a, device=q.device)
-        sc = sc.masked_fill(pos[None, None, :] > lim[:, None, None], float("-inf"))
+        if softcap:
+            sc = softcap * torch.tanh(sc / softcap)
+        lim = (L - (b - a) + torch.arange(b - a, device=q.device))[:, None, None]
+        sc = sc.masked_fill(pos > lim, float("-inf"))
         if window:
-            sc = sc.masked_fill(pos[None, None, :] <= lim[:, None, None] - window, float("-inf"))
+            sc = sc.masked_fill((pos <= lim - window) & (pos >= keep), float("-inf"))
+        if chunk:
+            sc = sc.masked_fill(pos < lim // chunk * chunk, float("-inf"))
         if sink is not None:
             sc = torch.cat([sc, sink.float()[None, :, None].expand(b - a, H, 1)], -1)
-        p = torch.softmax(sc, -1)[..., :L].reshape(b - a, G, rep, L)
+        p = torch.softmax(sc, -1)[..., :L]
+        if talk is not None:
+            p = torch.einsum("hg,tgl->thl", talk.float(), p)
+        p = p.reshape(b - a, G, rep, L)
         out[a:b, :, :w] = torch.einsum("tgrl,lgd->tgrd", p, v).reshape(b - a, H, w)
     out = out.reshape(T, H * out_width)
     return (out if gate is None else out * torch.sigmoid(gate[:, : H * out_width].float())).to(q.dtype)
@@ -305,6 +314,12 @@ def clamped_swish(gate_up, limit: float):
     return (g * torch.sigmoid(1.702 * g) * (u + 1)).flatten(1).to(gate_up.dtype)
 
 
+def swiglu_runs(gate_up):
+    """``silu(g) u`` of halves in alternating runs of 32 columns."""
+    g, u = gate_up.float().view(gate_up.shape[0], -1, 2, 32).unbind(2)
+    return (F.silu(g) * u).flatten(1).to(gate_up.dtype)
+
+
 def moe_experts(h, plan, up, down, act: str, limit: float = 0.0):
     """Outputs ``down_e act(up_e h)`` of every row's experts, unweighted: ``[T, top, W]`` (zero for identity experts)."""
     T, k = plan.index.shape
@@ -314,8 +329,130 @@ def moe_experts(h, plan, up, down, act: str, limit: float = 0.0):
             continue
         t, j = (plan.index == e).nonzero(as_tuple=True)
         y = F.linear(h[t], up[e])
-        out[t, j] = F.linear(relu2(y) if act == "relu2" else clamped_swish(y, limit), down[e])
+        out[t, j] = F.linear(relu2(y) if act == "relu2" else swiglu_runs(y) if act == "swiglu" else clamped_swish(y, limit), down[e])
     return out
+
+
+def _segments(b, T: int) -> list:
+    """``(first row, last row + 1, position of the first row, state slot)`` of a batch's segments."""
+    bounds = list(range(T + 1)) if b.cu is None else b.cu.tolist()
+    return [(a, e, int(n) - (e - a), int(s)) for a, e, n, s in zip(bounds, bounds[1:], b.ctx.tolist(), b.state_slot.tolist())]
+
+
+def conv_inputs(qkv, bias, taps, state, b, q_w, k_w, table, heads: int, kv_heads: int, dim: int, vdim: int, dp: int, rot_dims: int, eps: float, k_pool,
+                v_pool):
+    """Like :func:`attention_inputs` with biases ``bias[channels]``, then a causal convolution over a sequence's rows (``taps[channels, n]``,
+    the last tap on the row itself; ``state[slot, n - 1, channels]``: the rows before a segment, without biases, replaced by its last
+    ones), then RMS norms head by head with weights (``eps`` > 0), then the rotation of neighbours."""
+    T, C = qkv.shape[0], heads * dim + (kv_heads * (dim + vdim) if k_pool is not None else 0)
+    add = 0.0 if bias is None else bias[:C].float()
+    y = torch.empty(T, C, dtype=torch.float32, device=qkv.device)
+    n = 1 if taps is None else taps.shape[1]
+    for lo, hi, pos, slot in _segments(b, T):
+        u = qkv[lo:hi, :C]
+        if n == 1:
+            y[lo:hi] = (u.float() + add) * (1.0 if taps is None else taps[:, 0].float())
+            continue
+        before = state[slot] if pos else torch.zeros_like(state[slot])
+        rows = torch.cat([before, u.to(state.dtype)])
+        x = rows.float() + add
+        x[: max(0, n - 1 - pos)] = 0.0               # rows before the sequence's start have no bias either
+        y[lo:hi] = sum(taps[:, j].float() * x[j:j + hi - lo] for j in range(n))
+        state[slot] = rows[hi - lo:]
+
+    def head(x, w):
+        if eps > 0:
+            x = x / torch.sqrt(x.pow(2).mean(-1, keepdim=True) + eps) * w.float()
+        return torch.cat([turn_neighbours(x[..., :rot_dims], table), x[..., rot_dims:]], -1) if rot_dims else x
+
+    qd, kd = heads * dim, kv_heads * dim
+    q = torch.zeros(T, heads, dp, dtype=qkv.dtype, device=qkv.device)
+    q[..., :dim] = head(y[:, :qd].view(T, heads, dim), q_w).to(qkv.dtype)
+    if k_pool is not None:
+        k_pool[b.slots, :, :dim] = head(y[:, qd:qd + kd].view(T, kv_heads, dim), k_w).to(k_pool.dtype)
+        v_pool[b.slots, :, :vdim] = y[:, qd + kd:].view(T, kv_heads, vdim).to(v_pool.dtype)
+    return q
+
+
+def mingru(zxg, z_b, x_b, state, b, width: int):
+    """Gated running means ``S <- (1 - z) S + z c`` per channel, ``z = sigmoid(z_t + z_b)`` and ``c`` = ``u + 1/2`` or (``u`` < 0)
+    ``sigmoid(u)`` of ``u = x_t + x_b``; rows ``[z | x | g]`` whose parts are padded to 8 columns.  Returns ``S silu(g)``, padded alike."""
+    T, n = zxg.shape[0], (width + 7) // 8 * 8
+    z, u, g = (zxg[:, k * n:k * n + width].float() for k in range(3))
+    z, u = torch.sigmoid(z + z_b[:width].float()), u + x_b[:width].float()
+    c = torch.where(u >= 0, u + 0.5, torch.sigmoid(u))
+    out = torch.zeros(T, n, dtype=torch.float32, device=zxg.device)
+    for lo, hi, pos, slot in _segments(b, T):
+        S = state[slot].view(-1)[:width]
+        S = S.clone() if pos else torch.zeros_like(S)
+        for t in range(lo, hi):
+            S = (1 - z[t]) * S + z[t] * c[t]
+            out[t, :width] = S * F.silu(g[t])
+        state[slot].view(-1)[:width] = S
+    return out.to(zxg.dtype)
+
+
+def gla(rows, z, a2_b, norm_w, state, state_slot, ctx_lens, cu, heads: int, dim: int, vdim: int, gate_col: int, eps: float, root: float):
+    """Linear attention ``S <- diag(alpha) S + k v^T``, read-outs ``S^T q dim^-1/2``, with ``alpha = sigmoid(z + a2_b) ** (1 / root)`` per key
+    channel; read-outs normed head by head, times ``silu`` of the gates.  Rows ``[q | k | v | .. gate_col: g]``."""
+    T, qd, vd = rows.shape[0], heads * dim, heads * vdim
+    q, k, v = rows[:, : 2 * qd + vd].float().split([qd, qd, vd], 1)
+    q, k, v = q.view(T, heads, dim) * dim ** -0.5, k.view(T, heads, dim), v.view(T, heads, vdim)
+    alpha = torch.exp(F.logsigmoid(z[:, :qd].float() + a2_b.float()) / root).view(T, heads, dim)
+    o = torch.zeros(T, heads, vdim, dtype=torch.float32, device=rows.device)
+    bounds = list(range(T + 1)) if cu is None else cu.tolist()
+    for s, (a, b) in enumerate(zip(bounds, bounds[1:])):
+        S = state[state_slot[s], :, :, :vdim]
+        cur = torch.zeros_like(S) if int(ctx_lens[s]) == b - a else S.clone()
+        for t in range(a, b):
+            cur = alpha[t][..., None] * cur + k[t][..., None] * v[t][:, None, :]
+            o[t] = torch.einsum("hdv,hd->hv", cur, q[t])
+        S.copy_(cur)
+    o = o / torch.sqrt(o.pow(2).mean(-1, keepdim=True) + eps) * norm_w.float()
+    out = torch.zeros(T, (vd + 7) // 8 * 8, dtype=torch.float32, device=rows.device)
+    out[:, :vd] = o.reshape(T, vd) * F.silu(rows[:, gate_col:gate_col + vd].float())
+    return out.to(rows.dtype)
+
+
+def stream_step(res, width: int, eps: float, y=None, norm_w=None, experts=None, norms=(), shift=None):
+    """``res += ...`` (see :func:`relax_b200.ops.stream_step`)."""
+    dt = norms[0].dtype if norms else y[0].dtype
+    x = res[:, :width]
+    if y is not None:
+        parts = [a[:, :width].float() for a in y]
+        if norm_w is not None:
+            parts = [a / torch.sqrt(a.pow(2).mean(-1, keepdim=True) + eps) * w[:width].float() for a, w in zip(parts, norm_w)]
+        x += sum(parts) / len(parts)
+    if experts is not None:
+        rows, plan = experts
+        x += (rows[..., :width].float() * plan.weight[..., None]).sum(1)
+    out = []
+    for w in norms or (None,):
+        h = torch.zeros(res.shape, dtype=torch.float32, device=res.device)
+        d = x - x.mean(-1, keepdim=True)
+        h[:, :width] = x if w is None else d / torch.sqrt(d.pow(2).mean(-1, keepdim=True) + eps) * w[:width].float()
+        out.append(h.to(dt))
+    if shift is not None:
+        mu, state, b = shift
+        n, mixed = out[0], torch.empty_like(out[0])
+        for lo, hi, pos, slot in _segments(b, n.shape[0]):
+            first = state[slot] if pos else torch.zeros_like(state[slot])
+            before = torch.cat([first[None], n[lo:hi - 1]]).float()
+            mixed[lo:hi] = (n[lo:hi].float() + (before - n[lo:hi].float()) * mu.float()).to(dt)
+            state[slot] = n[hi - 1]
+        out[0] = mixed
+    return out
+
+
+def side_gate(z, embed, tokens, first: int, dim: int):
+    """``gelu_tanh(z) * e`` of the tokens' features ``first .. first + dim`` in a second embedding, padded to 8 columns."""
+    out = torch.zeros(z.shape[0], (dim + 7) // 8 * 8, dtype=torch.float32, device=z.device)
+    out[:, :dim] = F.gelu(z[:, :dim].float(), approximate="tanh") * embed[tokens, first:first + dim].float()
+    return out.to(z.dtype)
+
+
+def softcap(z, cap: float):
+    return cap * torch.tanh(z.float() / cap)
 
 
 # --------------------------------------------------------------------------- rotary embedding

@@ -2,7 +2,9 @@
 
 A composed stack (``ModelConfig.layer_specs``) mixes layers whose memory of the past differs in kind:
 
-* recurrent layers keep one fp32 matrix per head and sequence, in a STATE SLOT of a fixed pool (:class:`StackCache.state`);
+* recurrent layers keep one fp32 matrix per head and sequence (running means: one row), in a STATE SLOT of a fixed pool
+  (:class:`StackCache.state`);
+* short convolutions and shifted tokens keep the last rows they have read in the same slots (:class:`StackCache.conv`, ``shift``);
 * latent-attention layers keep one row per token in PAGES of the engine's block manager (:class:`StackCache.latent`): the latent
   features and, where positions are rotated in, one rotated key part behind them;
 * attention layers keep a key and a value row per token and key / value head in the same pages (:class:`StackCache.kv`), unless
@@ -24,12 +26,9 @@ import torch
 
 from .. import ops
 from ..models.config import ModelConfig
+from ..models.native import pad_to
 
 LONG_PORTION = 192     # portions of at least this many rows attend through projected keys / values (flash attention)
-
-
-def pad_to(n: int, m: int) -> int:
-    return (n + m - 1) // m * m
 
 
 def head_pitch(n: int) -> int:
@@ -41,6 +40,11 @@ def head_pitch(n: int) -> int:
 def latent_row(spec) -> int:
     """Columns of a cached latent row: latent features, then the rotated key part, each in whole 64-column chunks."""
     return pad_to(spec.kv_rank, 64) + pad_to(spec.rot_dims, 64)
+
+
+def projected(spec) -> int:
+    """Columns of an attention layer's query, key and value projections."""
+    return spec.heads * spec.dim + (spec.kv_heads * (spec.dim + spec.vdim) if spec.own_kv else 0)
 
 
 class SlotManager:
@@ -68,25 +72,36 @@ class SlotManager:
 
 
 class StackCache:
-    """The pools of a composed stack.  ``latent[layer]``: ``[blocks * block_size, latent_row]`` rows in the model's type;
-    ``kv[layer]``: keys and values ``[blocks * block_size, kv heads, padded width]``, one pair for the layer that computes them and
-    all that read them; ``state[layer]``: ``[slots, heads, dim, padded vdim]`` fp32.  All of it lives in ONE buffer."""
+    """The pools of a composed stack, by mixer (:meth:`ModelConfig.mixers`).  ``latent[key]``: ``[blocks * block_size, latent_row]`` rows in
+    the model's type; ``kv[key]``: keys and values ``[blocks * block_size, kv heads, padded width]``, one pair for the layer that computes
+    them and all that read them; ``state[key]``: ``[slots, heads, dim, padded vdim]`` fp32; ``conv[key]``: the last ``taps - 1`` projected
+    rows ``[slots, taps - 1, channels]``; ``shift[layer]``: the mixer's last input row ``[slots, width]``.  All of it lives in ONE buffer."""
 
     def __init__(self, cfg: ModelConfig, num_blocks: int, block_size: int, num_slots: int, dtype, device, memory_saver: bool):
         self.block_size = block_size
         views, n = [], 0
         es = torch.empty(0, dtype=dtype).element_size()
         rows = num_blocks * block_size
-        for i, s in enumerate(cfg.layer_specs):
-            if s.mixer == "hgrn2":
-                pools = [("state", (num_slots, s.heads, s.dim, pad_to(s.vdim, 4)), torch.float32, 4)]
+
+        def room(key, kind, shape, dt, size):
+            nonlocal n
+            views.append((key, kind, shape, dt, n))
+            n += pad_to(math.prod(shape) * size, 1024)
+
+        for key, s in cfg.mixers():
+            if s.mixer in ("hgrn2", "gla", "mingru"):
+                room(key, "state", (num_slots, s.heads, s.dim, pad_to(s.vdim, 4)), torch.float32, 4)
             elif s.mixer == "latent_attention":
-                pools = [("latent", (rows, latent_row(s)), dtype, es)]
+                room(key, "latent", (rows, latent_row(s)), dtype, es)
             else:
-                pools = [(k, (rows, s.kv_heads, head_pitch(d)), dtype, es) for k, d in (("k", s.dim), ("v", s.vdim))] if s.own_kv else []
-            for kind, shape, dt, size in pools:
-                views.append((i, kind, shape, dt, n))
-                n += pad_to(math.prod(shape) * size, 1024)
+                if s.own_kv:
+                    for k, d in (("k", s.dim), ("v", s.vdim)):
+                        room(key, k, (rows, s.kv_heads, head_pitch(d)), dtype, es)
+                if s.conv > 1:
+                    room(key, "conv", (num_slots, s.conv - 1, projected(s)), dtype, es)
+        if cfg.token_shift:
+            for i in range(cfg.num_layers):
+                room(i, "shift", (num_slots, pad_to(cfg.hidden_size, 64)), dtype, es)
         self.nbytes = n
         self.buf = None
         if memory_saver:
@@ -97,15 +112,16 @@ class StackCache:
         else:
             flat = torch.zeros(max(n, 1), dtype=torch.uint8, device=device)
             make = lambda shape, dt, off: flat[off:off + math.prod(shape) * torch.empty(0, dtype=dt).element_size()].view(dt).view(shape)
-        made = {"latent": {}, "state": {}, "k": {}, "v": {}}
-        for i, kind, shape, dt, off in views:
-            made[kind][i] = make(shape, dt, off)
-        self.latent, self.state = made["latent"], made["state"]
-        self.kv = {i: (made["k"][i], made["v"][i]) for i in made["k"]}
-        for i, s in enumerate(cfg.layer_specs):
+        made = {k: {} for k in ("latent", "state", "k", "v", "conv", "shift")}
+        for key, kind, shape, dt, off in views:
+            made[kind][key] = make(shape, dt, off)
+        self.latent, self.state, self.conv, self.shift = (made[k] for k in ("latent", "state", "conv", "shift"))
+        self.kv = {key: (made["k"][key], made["v"][key]) for key in made["k"]}
+        for key, s in cfg.mixers():
             if s.kv_from >= 0:
-                self.kv[i] = self.kv[s.kv_from]
-        self.paged = list(made["latent"].values()) + list(made["k"].values()) + list(made["v"].values())
+                self.kv[key] = self.kv[s.kv_from]
+        self.paged = [p for k in ("latent", "k", "v") for p in made[k].values()]
+        self.slotted = [p for k in ("state", "conv", "shift") for p in made[k].values()]
 
     def copy_sequence(self, src_blocks: Sequence[int], dst_blocks: Sequence[int], src_slot: int, dst_slot: int):
         """Pages ``src -> dst`` pairwise and the whole state slot."""
@@ -113,7 +129,7 @@ class StackCache:
             v = pool.view(-1, self.block_size, *pool.shape[1:])
             for a, b in zip(src_blocks, dst_blocks):
                 v[b] = v[a]
-        for st in self.state.values():
+        for st in self.slotted:
             st[dst_slot] = st[src_slot]
 
 
@@ -142,6 +158,7 @@ class SegmentBatch:
     items: Optional[dict] = None
     item_width: Optional[dict] = None
     spans: Optional[tuple] = None            # row ranges of recurrent spans and the first span of every segment
+    mean_spans: Optional[tuple] = None       # the same for running means
     # attention layers (and positions for all that rotate)
     multi_segs: int = 0
     multi_rows: int = 0
@@ -202,37 +219,114 @@ def recurrent_spans(lens: Sequence[int], heads: int, ctas: int = 296, shortest: 
     return (spans, first) if len(spans) > len(lens) else None
 
 
+MEAN_SPAN = 64         # tokens of a span of a running mean
+
+
+def mean_spans(lens: Sequence[int], span: int = MEAN_SPAN) -> Optional[tuple]:
+    """Cut segments of more than four spans' tokens into spans for running means; ``(row ranges, first span of every segment)``, None when
+    no segment is that long."""
+    if max(lens) <= 4 * span:
+        return None
+    spans, first, row = [], [0], 0
+    for n in lens:
+        step = span if n > 4 * span else n
+        spans += [[row + a, row + min(n, a + step)] for a in range(0, n, step)]
+        first.append(len(spans))
+        row += n
+    return spans, first
+
+
 class ComposedForward:
     """The forward of composed stacks (mixed into :class:`relax_b200.rollout.weights.RolloutWeights`).
 
     The residual stream is fp32.  A sublayer reads its copy in the model's type, and one kernel norms the sublayer's
     output, adds it and writes the next copy (or adds first and norms the sum); at the last sublayer that kernel also applies the
-    final norm."""
+    final norm.  With norms in front of the sublayers, one kernel adds the outputs of both and of the second embedding and writes
+    the norms that the next layer reads."""
 
-    def latent_dims(self, i: int) -> tuple:
-        """Padded ``(dim, vdim, rank)`` of latent layer ``i`` (16-byte rows per head, 64-column latent chunks); ``dim`` counts the
+    @staticmethod
+    def latent_dims(s) -> tuple:
+        """Padded ``(dim, vdim, rank)`` of a latent layer (16-byte rows per head, 64-column latent chunks); ``dim`` counts the
         unrotated and the rotated features of a head."""
-        s = self.cfg.layer_specs[i]
         return pad_to(s.dim + s.rot_dims, 8), pad_to(s.vdim, 8), pad_to(s.kv_rank, 64)
 
     @staticmethod
     def gate_column(s) -> int:
         """First column of an attention layer's output gate behind its projections (16-byte aligned)."""
-        return pad_to(s.heads * s.dim + (s.kv_heads * (s.dim + s.vdim) if s.own_kv else 0), 8)
+        return pad_to(projected(s), 8)
 
-    def attention_dims(self, i: int) -> tuple:
-        """Pitch of a head's queries and keys, of its values, and of its output in attention layer ``i``."""
-        s = self.cfg.layer_specs[i]
+    @staticmethod
+    def gla_columns(s) -> dict:
+        """First columns of queries, keys, values, output gates and the decay's inner projection, and the number of columns."""
+        qd, vd = s.heads * s.dim, s.heads * s.vdim
+        g = pad_to(2 * qd + vd, 8)
+        a1 = pad_to(g + vd, 8)
+        return {"q": 0, "k": qd, "v": 2 * qd, "g": g, "a1": a1, "end": a1 + pad_to(s.decay_rank, 8)}
+
+    @staticmethod
+    def attention_dims(s) -> tuple:
+        """Pitch of a head's queries and keys, of its values, and of its output in an attention layer."""
         return head_pitch(s.dim), head_pitch(s.vdim), pad_to(s.vdim, 8)
 
     def rope_frequencies(self, spec) -> torch.Tensor:
-        """``rot_base ** (-2 i / rot_dims)`` in fp64, kept on the device."""
+        """``rot_base ** (-2 i / rot_dims)`` in fp64, kept on the device; with ``rot_scaling`` frequencies whose wavelength exceeds
+        ``original / low`` are divided by ``factor``, and those down to ``original / high`` partly."""
         made = self.__dict__.setdefault("_rope_freq", {})
-        key = (spec.rot_base, spec.rot_dims)
+        key = (spec.rot_base, spec.rot_dims, spec.rot_scaling)
         if key not in made:
             i = torch.arange(spec.rot_dims // 2, dtype=torch.float64)
-            made[key] = (float(spec.rot_base) ** (-2.0 * i / spec.rot_dims)).to(self.device)
+            f = float(spec.rot_base) ** (-2.0 * i / spec.rot_dims)
+            if spec.rot_scaling is not None:
+                factor, low, high, original = spec.rot_scaling
+                kept = ((original * f / (2 * math.pi) - low) / (high - low)).clamp(0.0, 1.0)      # share that stays as it is
+                f = (1 - kept) * f / factor + kept * f
+            made[key] = f.to(self.device)
         return made[key]
+
+    INPUT = {"hgrn2": "rec_qfv", "attention": "attn_qkv", "latent_attention": "lat_qcg", "mingru": "gru_zxg", "gla": "gla_in"}
+
+    @staticmethod
+    def mixer_param_shapes(s, p: str, Wp: int) -> dict:
+        shapes, H = {}, s.heads
+        if s.mixer == "hgrn2":
+            qd, vd = H * s.dim, H * s.vdim
+            shapes[p + "rec_qfv"] = (pad_to(2 * qd + vd, 64), Wp)
+            shapes[p + "rec_f_bias"], shapes[p + "rec_lower"], shapes[p + "rec_norm"] = (qd,), (qd,), (s.vdim,)
+            shapes[p + "rec_o"] = (Wp, pad_to(vd, 8))
+        elif s.mixer == "mingru":
+            n = pad_to(s.vdim, 8)
+            shapes[p + "gru_zxg"], shapes[p + "gru_o"] = (pad_to(3 * n, 64), Wp), (Wp, n)
+            shapes[p + "gru_z_b"], shapes[p + "gru_x_b"] = (n,), (n,)
+        elif s.mixer == "gla":
+            qd, vd = H * s.dim, H * s.vdim
+            shapes[p + "gla_in"] = (pad_to(ComposedForward.gla_columns(s)["end"], 64), Wp)
+            shapes[p + "gla_a2"], shapes[p + "gla_a2_b"] = (pad_to(qd, 64), pad_to(s.decay_rank, 8)), (qd,)
+            shapes[p + "gla_norm"], shapes[p + "gla_o"] = (s.vdim,), (Wp, pad_to(vd, 8))
+        elif s.mixer == "attention":
+            cols = ComposedForward.gate_column(s) + H * pad_to(s.vdim, 8) if s.out_gate else projected(s)
+            shapes[p + "attn_qkv"] = (pad_to(cols, 64), Wp)
+            if s.qkv_bias:
+                shapes[p + "attn_qkv_b"] = (projected(s),)
+            if s.conv:
+                shapes[p + "attn_conv"] = (projected(s), s.conv)
+            if s.proj_norm or s.head_norm:
+                shapes[p + "attn_q_norm"] = (H * s.dim if s.proj_norm else s.dim,)
+                if s.own_kv:
+                    shapes[p + "attn_k_norm"] = (s.kv_heads * s.dim if s.proj_norm else s.dim,)
+            if s.sink or s.unit_sink:      # (a unit sink's logits stay zero)
+                shapes[p + "attn_sink"] = (H,)
+            if s.talk:
+                shapes[p + "attn_talk"] = (H, H)
+            shapes[p + "attn_o"] = (Wp, H * pad_to(s.vdim, 8))
+        else:
+            # rows of lat_qcg: queries (a head's unrotated, then its rotated features), latent, rotated key part, gates.  lat_uk maps
+            # a cached row to a head's key; its rows of rotated features are those of the identity (:meth:`pass_rotated_keys`)
+            dp, vp, Rp = pad_to(s.dim + s.rot_dims, 8), pad_to(s.vdim, 8), pad_to(s.kv_rank, 64)
+            shapes[p + "lat_qcg"] = (pad_to(H * dp + Rp + pad_to(s.rot_dims, 8) + (H * vp if s.out_gate else H), 64), Wp)
+            shapes[p + "lat_norm"] = (Rp,)
+            shapes[p + "lat_uk"], shapes[p + "lat_uv"] = (H * dp, latent_row(s)), (H * vp, Rp)
+            shapes[p + "lat_o"] = (Wp, H * vp)
+        return shapes
 
     @staticmethod
     def composed_param_shapes(cfg: ModelConfig) -> dict:
@@ -240,36 +334,30 @@ class ComposedForward:
         padding is zero and stays zero through every layer."""
         Wp, Vp = pad_to(cfg.hidden_size, 64), pad_to(cfg.vocab_size, 64)
         shapes = {"embed": (Vp, Wp)}
+        if cfg.side_dim:
+            shapes["side_embed"] = (Vp, pad_to(cfg.num_layers * cfg.side_dim, 8))
         for i, s in enumerate(cfg.layer_specs):
-            p, H = f"layers.{i}.", s.heads
-            if s.mixer == "hgrn2":
-                qd, vd = H * s.dim, H * s.vdim
-                shapes[p + "rec_qfv"] = (pad_to(2 * qd + vd, 64), Wp)
-                shapes[p + "rec_f_bias"], shapes[p + "rec_lower"], shapes[p + "rec_norm"] = (qd,), (qd,), (s.vdim,)
-                shapes[p + "rec_o"] = (Wp, pad_to(vd, 8))
-            elif s.mixer == "attention":
-                cols = ComposedForward.gate_column(s) + H * pad_to(s.vdim, 8) if s.out_gate else \
-                    H * s.dim + (s.kv_heads * (s.dim + s.vdim) if s.own_kv else 0)
-                shapes[p + "attn_qkv"] = (pad_to(cols, 64), Wp)
-                if s.proj_norm:
-                    shapes[p + "attn_q_norm"] = (H * s.dim,)
-                    if s.own_kv:
-                        shapes[p + "attn_k_norm"] = (s.kv_heads * s.dim,)
-                if s.sink:
-                    shapes[p + "attn_sink"] = (H,)
-                shapes[p + "attn_o"] = (Wp, H * pad_to(s.vdim, 8))
+            p = f"layers.{i}."
+            if s.pair is None:
+                shapes.update(ComposedForward.mixer_param_shapes(s, p, Wp))
+            else:      # the input projections of both lie one behind the other (:meth:`pair_views`)
+                rows = 0
+                for k, m in enumerate(s.pair):
+                    own = ComposedForward.mixer_param_shapes(m, f"{p}{k}.", Wp)
+                    rows += own.pop(f"{p}{k}.{ComposedForward.INPUT[m.mixer]}")[0]
+                    shapes.update({**own, f"{p}{k}.out_norm": (Wp,)})
+                shapes[p + "pair_in"] = (rows, Wp)
+            if cfg.pre_norm:
+                norms = ["norm1"] + (["norm2"] if s.has_ff else []) + (["shift"] if cfg.token_shift else [])
             else:
-                # rows of lat_qcg: queries (a head's unrotated, then its rotated features), latent, rotated key part, gates.  lat_uk maps
-                # a cached row to a head's key; its rows of rotated features are those of the identity (:meth:`pass_rotated_keys`)
-                dp, vp, Rp = pad_to(s.dim + s.rot_dims, 8), pad_to(s.vdim, 8), pad_to(s.kv_rank, 64)
-                shapes[p + "lat_qcg"] = (pad_to(H * dp + Rp + pad_to(s.rot_dims, 8) + (H * vp if s.out_gate else H), 64), Wp)
-                shapes[p + "lat_norm"] = (Rp,)
-                shapes[p + "lat_uk"], shapes[p + "lat_uv"] = (H * dp, latent_row(s)), (H * vp, Rp)
-                shapes[p + "lat_o"] = (Wp, H * vp)
-            for norm in ["post_attn_norm"] + (["post_mlp_norm"] if s.has_ff else []):
+                norms = ["post_attn_norm"] + (["post_mlp_norm"] if s.has_ff else [])
+            for norm in norms:
                 shapes[p + norm] = (Wp,)
                 if cfg.norm_sum:
                     shapes[p + norm + "_b"] = (Wp,)
+            if cfg.side_dim:
+                shapes[p + "side_gate"], shapes[p + "side_proj"] = (pad_to(cfg.side_dim, 64), Wp), (Wp, pad_to(cfg.side_dim, 8))
+                shapes[p + "side_norm"] = (Wp,)
             if s.ff:
                 Fp = pad_to(s.ff, 64)
                 shapes[p + "gate_up"], shapes[p + "down"] = (2 * Fp, Wp), (Wp, Fp)
@@ -290,6 +378,19 @@ class ComposedForward:
             shapes["lm_head"] = (Vp, Wp)
         return shapes
 
+    @staticmethod
+    def pair_views(cfg: ModelConfig, params: dict) -> dict:
+        """The input projections of a pair's mixers as parameters of their own."""
+        out = {}
+        for i, s in enumerate(cfg.layer_specs):
+            at = 0
+            for k, m in enumerate(s.pair or ()):
+                name, w = f"layers.{i}.{k}.{ComposedForward.INPUT[m.mixer]}", params[f"layers.{i}.pair_in"]
+                n = ComposedForward.mixer_param_shapes(m, f"layers.{i}.{k}.", w.shape[1])[name][0]
+                out[name] = w[at:at + n]
+                at += n
+        return out
+
     def pass_rotated_keys(self, i: int) -> None:
         """Let the key map of latent layer ``i`` hand the rotated part of a cached row on to every head's key unchanged (a reader calls
         this after it has filled the map's other rows)."""
@@ -299,23 +400,33 @@ class ComposedForward:
         uk[:, s.dim + k, pad_to(s.kv_rank, 64) + k] = 1.0
 
     # ------------------------------------------------------------------ mixers
-    def _hgrn2(self, i, h, b: SegmentBatch, cache: StackCache):
-        s, p, pre = self.cfg.layer_specs[i], self.p, f"layers.{i}."
-        qfv = ops.linear(h, p[pre + "rec_qfv"])
-        o = ops.hgrn2(qfv, p[pre + "rec_f_bias"], p[pre + "rec_lower"], p[pre + "rec_norm"], cache.state[i], b.state_slot,
+    # every mixer: (cache key, spec, prefix of its parameters, rows of its input projection, batch, cache, angle tables) -> output rows
+    def _hgrn2(self, key, s, pre, qfv, b: SegmentBatch, cache: StackCache, tables: dict):
+        p = self.p
+        o = ops.hgrn2(qfv, p[pre + "rec_f_bias"], p[pre + "rec_lower"], p[pre + "rec_norm"], cache.state[key], b.state_slot,
                       b.ctx, b.cu, s.heads, s.dim, s.vdim, self.cfg.rms_norm_eps, b.spans)
         return ops.linear(o, p[pre + "rec_o"])
 
-    def _latent(self, i, h, b: SegmentBatch, cache: StackCache, tables: dict):
+    def _mingru(self, key, s, pre, zxg, b: SegmentBatch, cache: StackCache, tables: dict):
+        p = self.p
+        return ops.linear(ops.mingru(zxg, p[pre + "gru_z_b"], p[pre + "gru_x_b"], cache.state[key], b, s.vdim), p[pre + "gru_o"])
+
+    def _gla(self, key, s, pre, rows, b: SegmentBatch, cache: StackCache, tables: dict):
+        p, at = self.p, self.gla_columns(s)
+        z = ops.linear_fp32(rows[:, at["a1"]:at["end"]], p[pre + "gla_a2"])
+        o = ops.gla(rows, z, p[pre + "gla_a2_b"], p[pre + "gla_norm"], cache.state[key], b.state_slot, b.ctx, b.cu, s.heads, s.dim, s.vdim, at["g"],
+                    self.cfg.rms_norm_eps, s.decay_root, b.spans)
+        return ops.linear(o, p[pre + "gla_o"])
+
+    def _latent(self, key, s, pre, qcg, b: SegmentBatch, cache: StackCache, tables: dict):
         """Keys and values are products of the cached latent row ``c``: ``q . (W_uk c) = (W_uk^T q) . c`` and
         ``sum p (W_uv c) = W_uv (sum p c)``.  Single tokens and short portions therefore attend to the latent rows in
         place, with the up-projections folded around the attention; long portions project keys and values of their whole
         context once and run the flash kernel on them.  A rotated key part in the row passes both ways unchanged
         (:meth:`pass_rotated_keys`)."""
-        s, p, pre = self.cfg.layer_specs[i], self.p, f"layers.{i}."
-        H, (dp, vp, Rp), row, pool = s.heads, self.latent_dims(i), latent_row(s), cache.latent[i]
-        T, rp = h.shape[0], pad_to(s.rot_dims, 8)
-        qcg = ops.linear(h, p[pre + "lat_qcg"])
+        p = self.p
+        H, (dp, vp, Rp), row, pool = s.heads, self.latent_dims(s), latent_row(s), cache.latent[key]
+        T, rp = qcg.shape[0], pad_to(s.rot_dims, 8)
         q, c, k_rot, gate = qcg[:, : H * dp + Rp + rp + H * (vp if s.out_gate else 1)].split([H * dp, Rp, rp, H * (vp if s.out_gate else 1)], 1)
         q = q.view(T, H, dp)
         turned = (q, k_rot, self._rope_table(s, b, tables), Rp, s.rot_dims, s.dim) if s.rot_dims else None
@@ -333,26 +444,41 @@ class ComposedForward:
             parts.append(ops.head_linear(o, uv.view(H, vp, Rp), True, gate[n:] if s.out_gate else None).reshape(T - n, H * vp))
         return ops.linear(parts[0] if len(parts) == 1 else torch.cat(parts), p[pre + "lat_o"])
 
-    def _attention(self, i, h, b: SegmentBatch, cache: StackCache, tables: dict):
-        s, p, pre = self.cfg.layer_specs[i], self.p, f"layers.{i}."
-        dp, _, vo = self.attention_dims(i)
-        k_pool, v_pool = cache.kv[i]
-        qkv = ops.linear(h, p[pre + "attn_qkv"])
+    def _attention(self, key, s, pre, qkv, b: SegmentBatch, cache: StackCache, tables: dict):
+        p = self.p
+        dp, _, vo = self.attention_dims(s)
+        k_pool, v_pool = cache.kv[key]
         table, eps, pools = self._rope_table(s, b, tables), self.cfg.rms_norm_eps, (k_pool, v_pool) if s.own_kv else (None, None)
-        if s.proj_norm or s.rot_halves:
+        if s.conv or s.qkv_bias or s.head_norm:
+            q = ops.conv_inputs(qkv, p.get(pre + "attn_qkv_b"), p.get(pre + "attn_conv"), cache.conv.get(key), b, p.get(pre + "attn_q_norm"),
+                                p.get(pre + "attn_k_norm"), table, s.heads, s.kv_heads, s.dim, s.vdim, dp, s.rot_dims, eps if s.head_norm else 0.0, *pools)
+        elif s.proj_norm or s.rot_halves:
             q = ops.projection_inputs(qkv, p.get(pre + "attn_q_norm"), p.get(pre + "attn_k_norm"), table, s.heads, s.kv_heads, s.dim, s.vdim, dp, s.rot_dims,
                                       s.rot_halves, eps if s.proj_norm else 0.0, *pools, b.slots)
         else:
             q = ops.attention_inputs(qkv, table, s.heads, s.kv_heads, s.dim, s.vdim, dp, s.rot_dims, eps if s.qk_norm else 0.0, *pools, b.slots)
         g = self.gate_column(s)
         o = ops.paged_attention(q, k_pool, v_pool, b, cache.block_size, s.scale, p.get(pre + "attn_sink"), vo, s.window,
-                                qkv[:, g:g + s.heads * vo] if s.out_gate else None)
+                                qkv[:, g:g + s.heads * vo] if s.out_gate else None, s.keep_first, s.chunk, s.softcap, p.get(pre + "attn_talk"))
         return ops.linear(o, p[pre + "attn_o"])
+
+    def _mix(self, i, h, b: SegmentBatch, cache: StackCache, tables: dict) -> list:
+        """Outputs of layer ``i``'s mixer, or of the two of a pair, on rows ``h``."""
+        s, pre = self.cfg.layer_specs[i], f"layers.{i}."
+        run = lambda key, m, at, x: getattr(self, "_latent" if m.mixer == "latent_attention" else "_" + m.mixer)(key, m, at, x, b, cache, tables)
+        if s.pair is None:
+            return [run(i, s, pre, ops.linear(h, self.p[pre + self.INPUT[s.mixer]]))]
+        rows, at, out = ops.linear(h, self.p[pre + "pair_in"]), 0, []
+        for k, m in enumerate(s.pair):
+            n = self.p[f"{pre}{k}.{self.INPUT[m.mixer]}"].shape[0]
+            out.append(run((i, k), m, f"{pre}{k}.", rows[:, at:at + n]))
+            at += n
+        return out
 
     def _rope_table(self, s, b: SegmentBatch, tables: dict):
         if not s.rot_dims:
             return None
-        key = (s.rot_base, s.rot_dims)
+        key = (s.rot_base, s.rot_dims, s.rot_scaling)
         if key not in tables:
             tables[key] = ops.rope_table(b.ctx if b.pos is None else b.pos, -1 if b.pos is None else 0, self.rope_frequencies(s))
         return tables[key]
@@ -369,10 +495,18 @@ class ComposedForward:
         return shared, (rows, plan)
 
     # ------------------------------------------------------------------ trunk
+    def _route_counts(self, device) -> dict:
+        """Counters of every routed layer's :func:`ops.moe_route`, zeroed at once."""
+        specs = self.cfg.layer_specs
+        routed = [i for i, s in enumerate(specs) if s.moe is not None]
+        return dict(zip(routed, ops.route_counters(len(routed), max(specs[i].moe.experts for i in routed), device))) if routed else {}
+
     def _run_composed(self, b: SegmentBatch, cache: StackCache, taps: Optional[list] = None):
         """Final-norm output of every row.  ``taps``: a list that receives the fp32 residual stream after every layer."""
         cfg, p = self.cfg, self.p
         W, G, eps = cfg.hidden_size, cfg.norm_groups, cfg.rms_norm_eps
+        if cfg.pre_norm:
+            return self._run_pre_norm(b, cache, taps)
         res, h = ops.embed_rows(b.tokens, p["embed"], p.get("embed_norm"), W, G, eps, cfg.embed_scale)
 
         def join(y, norm, last, experts=None):
@@ -383,22 +517,51 @@ class ComposedForward:
             return ops.sum_norm(res, y, p[norm], p[norm + "_b"], W, cfg.sum_alpha, eps, nxt, cfg.logit_scale if last else 1.0, experts)
 
         tables: dict = {}
-        routed = [i for i, s in enumerate(cfg.layer_specs) if s.moe is not None]
-        counts = dict(zip(routed, ops.route_counters(len(routed), max(cfg.layer_specs[i].moe.experts for i in routed), res.device))) if routed else {}
+        counts = self._route_counts(res.device)
         for i, s in enumerate(cfg.layer_specs):
             pre = f"layers.{i}."
             final = i + 1 == cfg.num_layers
-            if s.mixer == "hgrn2":
-                a = self._hgrn2(i, h, b, cache)
-            else:
-                a = (self._attention if s.mixer == "attention" else self._latent)(i, h, b, cache, tables)
-            h = join(a, pre + "post_attn_norm", final and not s.has_ff)
+            h = join(self._mix(i, h, b, cache, tables)[0], pre + "post_attn_norm", final and not s.has_ff)
             if s.has_ff:
                 m, experts = self._feed_forward(i, h, counts.get(i))
                 h = join(m, pre + "post_mlp_norm", final, experts)
             if taps is not None:
                 taps.append(res[:, :W].clone())
         return h
+
+    def _run_pre_norm(self, b: SegmentBatch, cache: StackCache, taps: Optional[list] = None):
+        """The same for sublayers that read norms of the stream: ``x <- x + mixer(norm1 x) + ff(norm2 x)``, then the second
+        embedding's part."""
+        cfg, p = self.cfg, self.p
+        W, eps = cfg.hidden_size, cfg.rms_norm_eps
+
+        def reads(i):
+            """``(norms of the stream that layer i reads, what shifts the first of them)``; behind the last layer: the final norm."""
+            if i == cfg.num_layers:
+                return (p["final_norm"],), None
+            pre = f"layers.{i}."
+            norms = (p[pre + "norm1"],) + ((p[pre + "norm2"],) if cfg.layer_specs[i].has_ff else ())
+            return norms, (p[pre + "shift"], cache.shift[i], b) if cfg.token_shift else None
+
+        tables: dict = {}
+        counts = self._route_counts(b.tokens.device)
+        res, _ = ops.embed_rows(b.tokens, p["embed"])
+        h = ops.stream_step(res, W, eps, norms=reads(0)[0], shift=reads(0)[1])
+        for i, s in enumerate(cfg.layer_specs):
+            pre = f"layers.{i}."
+            y = self._mix(i, h[0], b, cache, tables)
+            pair = (p[pre + "0.out_norm"], p[pre + "1.out_norm"]) if s.pair is not None else None
+            experts = self._feed_forward(i, h[1], counts.get(i))[1] if s.has_ff else None
+            norms, shift = reads(i + 1)
+            if cfg.side_dim:
+                x, = ops.stream_step(res, W, eps, y, pair, experts)
+                g = ops.side_gate(ops.linear(x, p[pre + "side_gate"]), p["side_embed"], b.tokens, i * cfg.side_dim, cfg.side_dim)
+                h = ops.stream_step(res, W, eps, [ops.linear(g, p[pre + "side_proj"])], (p[pre + "side_norm"],), norms=norms, shift=shift)
+            else:
+                h = ops.stream_step(res, W, eps, y, pair, experts, norms, shift)
+            if taps is not None:
+                taps.append(res[:, :W].clone())
+        return h[0]
 
     def forward_segments(self, b: SegmentBatch, cache: StackCache, rows: Optional[torch.Tensor], tp, taps: Optional[list] = None):
         """Logits of the given rows (None: no row is asked for, only slots and pages are advanced)."""
@@ -469,11 +632,12 @@ class ComposedScheduler:
             arrays["cu"] = (cu, i32)
             lens = [b - a for a, b in zip(cu, cu[1:])]
             sl, sc = lens[n_long:], ctx[n_long:]
-            attn = [self.cfg.layer_specs[i] for i in self.cfg.layers_with("attention")]
-            if attn or any(s.rot_dims for s in self.cfg.layer_specs):
+            attn = self.cfg.specs_with("attention")
+            if attn or self.cfg.token_shift or any(s.rot_dims for _, s in self.cfg.mixers()):
                 arrays["pos"] = ([c - n + k for n, c in zip(lens, ctx) for k in range(n)], i32)
-            if attn:
+            if attn or self.cfg.token_shift:
                 arrays["seg_of"] = ([s for s, n in enumerate(lens) for _ in range(n)], i32)
+            if attn:
                 tiles = sorted({tile_tokens(s) for s in attn})
                 for t in tiles:
                     arrays[f"blocks{t}"] = (query_blocks(lens[:n_multi], ctx, t), i32)
@@ -481,15 +645,18 @@ class ComposedScheduler:
                 arrays["long_first"] = ([sum(ctx[:s]) for s in range(n_long)], i32)
                 arrays["long_blocks"] = (query_blocks(lens[:n_long], ctx, QUERY_ROWS), i32)
                 arrays["ctx_slots"] = ([x for j in order[:n_long] for x in self._slots(parts[j][0], 0, parts[j][0].fed + parts[j][1])], i64)
-            rec = [self.cfg.layer_specs[i].heads for i in self.cfg.layers_with("hgrn2")]
+            rec = [s.heads for s in self.cfg.specs_with("hgrn2", "gla")]
             cuts = recurrent_spans(lens, max(rec)) if rec and self.device.type == "cuda" else None
             if cuts is not None:
                 arrays["spans"], arrays["span_first"] = (cuts[0], i32), (cuts[1], i32)
-            if sl and self.cfg.layers_with("latent_attention"):
+            cuts = mean_spans(lens) if self.cfg.specs_with("mingru") and self.device.type == "cuda" else None
+            if cuts is not None:
+                arrays["mean"], arrays["mean_first"] = (cuts[0], i32), (cuts[1], i32)
+            specs = self.cfg.specs_with("latent_attention")
+            if sl and specs:
                 arrays["short_cu"] = ([c - cu[n_long] for c in cu[n_long:]], i32)
                 arrays["row_seg"] = ([s for s, n in enumerate(sl) for _ in range(n)], i32)
                 arrays["row_pos"] = ([c - n + k for n, c in zip(sl, sc) for k in range(n)], i32)
-                specs = [self.cfg.layer_specs[i] for i in self.cfg.layers_with("latent_attention")]
                 for s in specs:
                     widths[s.heads] = min(widths.get(s.heads, 64), ops.latent_columns(latent_row(s), pad_to(s.kv_rank, 64)))
                 for H, width in widths.items():
@@ -499,9 +666,10 @@ class ComposedScheduler:
         dev = dict(zip(arrays, self._stage(list(arrays.values()))))
         want_t = dev.pop("rows", None)
         spans = (dev.pop("spans"), dev.pop("span_first")) if "spans" in dev else None
+        mean = (dev.pop("mean"), dev.pop("mean_first")) if "mean" in dev else None
         items = {H: dev.pop(f"items{H}") for H in widths}
         blocks = {t: dev.pop(f"blocks{t}") for t in tiles}
-        batch = SegmentBatch(**dev, **host, items=items or None, item_width=widths or None, spans=spans, blocks=blocks or None)
+        batch = SegmentBatch(**dev, **host, items=items or None, item_width=widths or None, spans=spans, mean_spans=mean, blocks=blocks or None)
         logits = self.weights.forward_segments(batch, self.kv, want_t, self.tp, taps)
         for r, n in parts:
             r.fed += n

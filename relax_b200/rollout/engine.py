@@ -175,9 +175,9 @@ class RolloutEngine(SpeculativeMixin, ComposedScheduler):
             self.sm = SlotManager(self.max_running + 1)
             self._scratch_slot = self.sm.alloc()      # padding rows of a graph bucket; never handed to a request
             # flash attention on projected keys / values: the tensor-core kernel takes bf16 heads of up to 192 / 128 features
-            latent = cfg.layers_with("latent_attention")
+            latent = cfg.specs_with("latent_attention")
             self._long_portions = self.device.type == "cuda" and bool(latent) and all(
-                ops.dense_flash_serves(self.dtype, *self.weights.latent_dims(i)[:2]) for i in latent)
+                ops.dense_flash_serves(self.dtype, *self.weights.latent_dims(s)[:2]) for s in latent)
         self._alloc_kv()
         self.use_cuda_graph = use_cuda_graph and self.device.type == "cuda"
         self.max_model_len = max_model_len

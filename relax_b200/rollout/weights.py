@@ -181,6 +181,8 @@ class RolloutWeights(ComposedForward):
         self.p = {k: self.flat[o:o + math.prod(self.shapes[k])].view(self.shapes[k]) for k, o in self.offsets.items()}
         if self.cfg.tie_word_embeddings:
             self.p["lm_head"] = self.p["embed"]
+        if self.cfg.is_composed:
+            self.p.update(self.pair_views(self.cfg, self.p))
         self.p.update(self.lora)
 
     def enable_lora(self, rank: int, scale: float, targets=("linear_qkv", "linear_proj", "linear_fc1", "linear_fc2")):
@@ -229,6 +231,8 @@ class RolloutWeights(ComposedForward):
         return x
 
     def _logits(self, h, tp: GroupInfo):
+        if self.cfg.logit_softcap > 0:
+            return ops.softcap(ops.linear_fp32(h, self.p["lm_head"]), self.cfg.logit_softcap)
         z = ops.linear(h, self.p["lm_head"])
         if not z.is_cuda:
             z = z.float()       # the sampling kernel reads bf16 rows directly; the CPU statement wants fp32

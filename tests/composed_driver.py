@@ -3,11 +3,12 @@ import torch
 
 import oracle_composed
 import oracle_ketolorn
+import oracle_zoguzen
 import oracle_zupupel
 
 
 def oracle(cfg):
-    return {"Ketolorn": oracle_ketolorn, "Zupupel": oracle_zupupel}.get(cfg.get("architecture"), oracle_composed)
+    return {"Ketolorn": oracle_ketolorn, "Zupupel": oracle_zupupel, "Zoguzen": oracle_zoguzen}.get(cfg.get("architecture"), oracle_composed)
 
 
 def engine(cfg, tensors, device="cpu", dtype=torch.float32, blocks=64, block_size=16, **kw):
@@ -16,7 +17,7 @@ def engine(cfg, tensors, device="cpu", dtype=torch.float32, blocks=64, block_siz
 
     full = {"architecture": "Talizen", **cfg}
     design = architecture_of(full)
-    mc = design.config_from_dict(full, dtype="fp32" if dtype == torch.float32 else "bf16")
+    mc = design.config_from_dict(full, dtype="fp32" if dtype == torch.float32 else "bf16", shapes={k: tuple(v.shape) for k, v in tensors.items()})
     eng = RolloutEngine(mc, device=device, dtype=dtype, num_kv_blocks=blocks, block_size=block_size, memory_saver=False,
                         **{"state_slots": 4, "use_cuda_graph": False, **kw})
     design.load_tensors(mc, tensors, eng.weights)
