@@ -147,6 +147,27 @@ int rb_hgrn2(const void* qfv, const void* f_bias, const void* lower, const void*
 int rb_hgrn2_chunk(const void* qfv, const void* f_bias, const void* lower, const void* norm_w, float* state, const int* slot, const int* ctx,
                    const int* cu, const int* spans, const int* first, float* span_state, float* span_gate, void* out, int rows, int segs,
                    int n_spans, int H, int dim, int vdim, int vp, int ld, int ldo, float eps, cudaStream_t st);
+int rb_gla(const void* in, const float* z, int ldz, const void* z_bias, const void* norm_w, float* state, const int* slot, const int* ctx, const int* cu,
+           float* o_raw, void* out, int rows, int segs, int H, int dim, int vdim, int vp, int ld, int ldo, int gate_col, float eps, float q_scale,
+           float inv_root, int fp32, cudaStream_t st);
+int rb_gla_chunk(const void* in, const float* z, int ldz, const void* z_bias, const void* norm_w, float* state, const int* slot, const int* ctx,
+                 const int* cu, const int* spans, const int* first, float* span_state, float* span_gate, void* out, int rows, int segs, int n_spans,
+                 int H, int dim, int vdim, int vp, int ld, int ldo, int gate_col, float eps, float q_scale, float inv_root, cudaStream_t st);
+int rb_mingru(const void* rows, const void* z_b, const void* x_b, float* state, const int* slot, const int* ctx, const int* cu, const int* spans, const
+              int* first, float* span_sum, float* span_keep, void* out, int segs, int n_spans, int width, int ld, int sp, int fp32, cudaStream_t st);
+int rb_stream_step(float* res, const void* y0, int ldy0, const void* y1, int ldy1, const void* w0, const void* w1, const void* ex, int ldx, const int*
+                   expert, const int* place, const int* offset, const float* weight, int top, const void* n0, const void* n1, void* h0, void* h1, const
+                   void* mu, void* state, const int* slot, const int* ctx, int rows, int pitch, int width, float eps, int fp32, cudaStream_t st);
+int rb_token_shift(const void* n, const void* mu, void* state, void* out, const int* slot, const int* ctx, const int* cu, const int* seg_of, int rows,
+                   int pitch, int fp32, cudaStream_t st);
+int rb_side_gate(const void* z, int ldz, const void* embed, long long lde, const long long* tok, int vocab, void* out, int rows, int dim, int pitch,
+                 int fp32, cudaStream_t st);
+int rb_softcap(float* z, long long n, float cap, cudaStream_t st);
+int rb_conv_inputs(const void* qkv, int ld, const void* bias, const void* taps, int n, void* state, const void* q_w, const void* k_w, const float* table,
+                   void* q, void* k_pool, void* v_pool, const long long* slots, const int* ctx, const int* state_slot, const int* cu, const int* seg_of,
+                   const int* pos, long long pool_rows, int T, int segs, int H, int G, int dim, int vdim, int dp, int vp, int rot, float eps, int fp32,
+                   cudaStream_t st);
+int rb_mix_heads(const void* wide, const void* mix, void* out, int rows, int H, int G, int vo, int fp32, cudaStream_t st);
 int rb_latent_write(const void* raw, const void* k_rot, void* q, int ld, const void* w, void* pool, const long long* slots, const float* table, long
                     long pool_rows, int rows, int rank, int pitch, int part, int rot, int H, int dk, int dim, float eps, int fp32, cudaStream_t st);
 int rb_latent_attn(const void* q, const void* pool, const int* block_tables, const int* row_seg, const int* row_pos, const int* ctx, const void* gate,
@@ -170,13 +191,14 @@ int rb_attention_inputs(const void* qkv, int ld, const float* table, void* q, vo
                         int T, int H, int G, int dim, int vdim, int dp, int vp, int rot, float eps, int fp32, cudaStream_t st);
 int rb_gqa_attn(const void* q, const void* k_pool, const void* v_pool, const int* block_tables, const int* row_seg, const int* row_pos, const int*
                 ctx, const void* sink, const void* gate, int ld_gate, void* out, int rows, int H, int G, int dp, int vp, int vo, int max_blocks, int
-                block_size, int window, float scale, int fp32, cudaStream_t st);
+                block_size, int window, int keep, int chunk, int wide, float scale, float cap, int fp32, cudaStream_t st);
 int rb_paged_flash(const void* q, const void* kc, const void* vc, const int* block_tables, const int* ctx, const int* blocks, const void* sink, const
                    void* gate, int ld_gate, void* out, int rows, int n, int Hq, int Hkv, int dk, int dv, int out_d, long long pool_rows, int page, int
-                   max_blocks, int window, float scale, int* err, cudaStream_t st);
+                   max_blocks, int window, int keep, int chunk, int wide, float scale, float cap, int* err, cudaStream_t st);
 int rb_paged_decode_tc(const void* q, const void* kc, const void* vc, const int* block_tables, const int* ctx_lens, const void* sink, const void*
                        gate, int ld_gate, void* out, float* part_o, float* part_ml, int B, int Hq, int Hkv, int dk, int dv, int out_d, long long
-                       pool_rows, int page, int max_blocks, int max_ctx, int window, float scale, int splits, int* err, cudaStream_t st);
+                       pool_rows, int page, int max_blocks, int max_ctx, int window, int keep, int chunk, float scale, float cap, int splits, int* err,
+                       cudaStream_t st);
 int rb_moe_route(const float* logits, int ld, const void* correction, int corr_fp32, int* expert, float* weight, int* place, int* row_token, int*
                  count, int* offset, int* tiles, int* n_tiles, int T, int E, int N, int groups, int keep, int group_best, int top, int tile_rows, int
                  cap, int renormalize, int softmax, float weight_scale, cudaStream_t st);

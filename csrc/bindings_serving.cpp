@@ -437,42 +437,45 @@ void projection_inputs(torch::Tensor qkv, c10::optional<torch::Tensor> q_w, c10:
         "rb_projection_inputs");
 }
 inline void check_pools(const torch::Tensor& q, const torch::Tensor& k, const torch::Tensor& v, const torch::Tensor& bt, const torch::Tensor& ctx,
-                        const c10::optional<torch::Tensor>& sink, const torch::Tensor& out) {
+                        const c10::optional<torch::Tensor>& sink, const torch::Tensor& out, bool wide = false) {
   check_same(q, k, "paged attention");
   check_same(q, v, "paged attention");
   check_same(q, out, "paged attention");
   TORCH_CHECK(q.dim() == 3 && k.dim() == 3 && v.dim() == 3 && q.is_contiguous() && k.is_contiguous() && v.is_contiguous() && out.is_contiguous());
   TORCH_CHECK(k.size(2) == q.size(2) && v.size(0) == k.size(0) && v.size(1) == k.size(1) && q.size(1) % k.size(1) == 0, "paged attention: shapes");
-  TORCH_CHECK(out.dim() == 2 && out.size(0) == q.size(0) && out.size(1) % q.size(1) == 0 && out.size(1) / q.size(1) <= v.size(2), "paged attention: output");
+  const int64_t outs = q.size(1) * (wide ? k.size(1) : 1);      // out: every head's columns, wide: for every group
+  TORCH_CHECK(out.dim() == 2 && out.size(0) == q.size(0) && out.size(1) % outs == 0 && out.size(1) / outs <= v.size(2), "paged attention: output");
   TORCH_CHECK(is_i32(bt) && bt.dim() == 2 && is_i32(ctx) && ctx.numel() == bt.size(0), "paged attention: block tables");
   TORCH_CHECK(!sink.has_value() || (sink->scalar_type() == q.scalar_type() && sink->is_contiguous() && sink->numel() == q.size(1)), "paged attention: sink");
 }
 void gqa_attn(torch::Tensor q, torch::Tensor k, torch::Tensor v, torch::Tensor bt, c10::optional<torch::Tensor> row_seg, c10::optional<torch::Tensor> row_pos,
               torch::Tensor ctx, c10::optional<torch::Tensor> sink, c10::optional<torch::Tensor> gate, torch::Tensor out, int64_t block_size, int64_t window,
-              double scale) {
+              int64_t keep, int64_t chunk, bool wide, double scale, double cap) {
   const c10::cuda::CUDAGuard guard(q.device());
-  check_pools(q, k, v, bt, ctx, sink, out);
+  check_pools(q, k, v, bt, ctx, sink, out, wide);
   const int64_t T = q.size(0), H = q.size(1);
   TORCH_CHECK(row_seg.has_value() == row_pos.has_value());
   TORCH_CHECK(row_seg.has_value() ? (is_i32(*row_seg) && is_i32(*row_pos) && row_seg->numel() == T && row_pos->numel() == T) : ctx.numel() == T,
               "gqa_attn: row description");
   check(rb_gqa_attn(q.data_ptr(), k.data_ptr(), v.data_ptr(), bt.data_ptr<int>(), optint(row_seg), optint(row_pos), ctx.data_ptr<int>(), optptr(sink),
                     optptr(gate), gate_pitch(gate, q, T, out.size(1)), out.data_ptr(), (int)T, (int)H, (int)k.size(1), (int)q.size(2), (int)v.size(2),
-                    (int)(out.size(1) / H), (int)bt.size(1), (int)block_size, (int)window, (float)scale, is_fp32(q), cur_stream()),
+                    (int)(out.size(1) / H / (wide ? k.size(1) : 1)), (int)bt.size(1), (int)block_size, (int)window, (int)keep, (int)chunk, wide, (float)scale,
+                    (float)cap, is_fp32(q), cur_stream()),
         "rb_gqa_attn");
 }
 // Prompt portions; returns false for shapes the tensor-core kernel does not take.
 bool paged_flash(torch::Tensor q, torch::Tensor k, torch::Tensor v, torch::Tensor bt, torch::Tensor ctx, c10::optional<torch::Tensor> blocks,
-                 c10::optional<torch::Tensor> sink, c10::optional<torch::Tensor> gate, torch::Tensor out, int64_t block_size, int64_t window, double scale,
-                 torch::Tensor err) {
+                 c10::optional<torch::Tensor> sink, c10::optional<torch::Tensor> gate, torch::Tensor out, int64_t block_size, int64_t window, int64_t keep,
+                 int64_t chunk, bool wide, double scale, double cap, torch::Tensor err) {
   const c10::cuda::CUDAGuard guard(q.device());
   if (q.scalar_type() != at::kBFloat16) return false;
-  check_pools(q, k, v, bt, ctx, sink, out);
+  check_pools(q, k, v, bt, ctx, sink, out, wide);
   const int64_t T = q.size(0), H = q.size(1);
   TORCH_CHECK(blocks.has_value() ? (is_i32(*blocks) && blocks->dim() == 2 && blocks->size(1) == 4) : ctx.numel() == T, "paged_flash: query tiles");
   const int rc = rb_paged_flash(q.data_ptr(), k.data_ptr(), v.data_ptr(), bt.data_ptr<int>(), ctx.data_ptr<int>(), optint(blocks), optptr(sink),
                                 optptr(gate), gate_pitch(gate, q, T, out.size(1)), out.data_ptr(), (int)T, (int)(blocks.has_value() ? blocks->size(0) : T), (int)H, (int)k.size(1), (int)q.size(2), (int)v.size(2),
-                                (int)(out.size(1) / H), k.size(0), (int)block_size, (int)bt.size(1), (int)window, (float)scale, err.data_ptr<int>(), cur_stream());
+                                (int)(out.size(1) / H / (wide ? k.size(1) : 1)), k.size(0), (int)block_size, (int)bt.size(1), (int)window, (int)keep, (int)chunk, wide,
+                                (float)scale, (float)cap, err.data_ptr<int>(), cur_stream());
   if (rc == -20) return false;
   check(rc, "rb_paged_flash");
   return true;
@@ -501,7 +504,7 @@ bool dense_flash(torch::Tensor q, torch::Tensor k, torch::Tensor v, torch::Tenso
 // One row per sequence; returns false for shapes the tensor-core kernel does not take.
 bool paged_decode(torch::Tensor q, torch::Tensor k, torch::Tensor v, torch::Tensor bt, torch::Tensor ctx, c10::optional<torch::Tensor> sink,
                   c10::optional<torch::Tensor> gate, torch::Tensor out, c10::optional<torch::Tensor> part_o, c10::optional<torch::Tensor> part_ml,
-                  int64_t block_size, int64_t max_ctx, int64_t window, int64_t splits, double scale, torch::Tensor err) {
+                  int64_t block_size, int64_t max_ctx, int64_t window, int64_t keep, int64_t chunk, int64_t splits, double scale, double cap, torch::Tensor err) {
   const c10::cuda::CUDAGuard guard(q.device());
   if (q.scalar_type() != at::kBFloat16) return false;
   check_pools(q, k, v, bt, ctx, sink, out);
@@ -512,10 +515,207 @@ bool paged_decode(torch::Tensor q, torch::Tensor k, torch::Tensor v, torch::Tens
   const int rc = rb_paged_decode_tc(q.data_ptr(), k.data_ptr(), v.data_ptr(), bt.data_ptr<int>(), ctx.data_ptr<int>(), optptr(sink), optptr(gate),
                                     gate_pitch(gate, q, B, out.size(1)), out.data_ptr(), part_o.has_value() ? part_o->data_ptr<float>() : nullptr, part_ml.has_value() ? part_ml->data_ptr<float>() : nullptr,
                                     (int)B, (int)H, (int)k.size(1), (int)q.size(2), (int)v.size(2), (int)(out.size(1) / H), k.size(0), (int)block_size,
-                                    (int)bt.size(1), (int)max_ctx, (int)window, (float)scale, (int)splits, err.data_ptr<int>(), cur_stream());
+                                    (int)bt.size(1), (int)max_ctx, (int)window, (int)keep, (int)chunk, (float)scale, (float)cap, (int)splits, err.data_ptr<int>(), cur_stream());
   if (rc == -20) return false;
   check(rc, "rb_paged_decode_tc");
   return true;
+}
+// wide [T][H G vo]: what every head's weights make of every group's values; mix [H][H]; out [T][H vo]
+void mix_heads(torch::Tensor wide, torch::Tensor mix, torch::Tensor out, int64_t kv_heads) {
+  const c10::cuda::CUDAGuard guard(wide.device());
+  check_same(wide, mix, "mix_heads");
+  check_same(wide, out, "mix_heads");
+  const int64_t T = out.size(0), H = mix.size(0);
+  TORCH_CHECK(mix.dim() == 2 && mix.size(1) == H && wide.is_contiguous() && mix.is_contiguous() && out.is_contiguous() && out.dim() == 2 && out.size(1) % H == 0);
+  TORCH_CHECK(kv_heads > 0 && wide.dim() == 2 && wide.size(0) == T && wide.size(1) == out.size(1) * kv_heads, "mix_heads: shapes");
+  check(rb_mix_heads(wide.data_ptr(), mix.data_ptr(), out.data_ptr(), (int)T, (int)H, (int)kv_heads, (int)(out.size(1) / H), is_fp32(wide), cur_stream()),
+        "rb_mix_heads");
+}
+inline void check_segments(const torch::Tensor& slot, const torch::Tensor& ctx, const c10::optional<torch::Tensor>& cu, int64_t rows, const char* what) {
+  TORCH_CHECK(is_i32(slot) && is_i32(ctx) && slot.numel() == ctx.numel(), what, ": segments");
+  TORCH_CHECK(cu.has_value() ? (is_i32(*cu) && cu->numel() == slot.numel() + 1) : slot.numel() == rows, what, ": segment bounds");
+}
+inline int64_t check_spans(const c10::optional<torch::Tensor>& spans, const c10::optional<torch::Tensor>& first, int64_t segs, const char* what) {
+  if (!spans.has_value()) return 0;
+  TORCH_CHECK(is_i32(*spans) && spans->dim() == 2 && spans->size(1) == 2 && first.has_value() && is_i32(*first) && first->numel() == segs + 1, what, ": spans");
+  return spans->size(0);
+}
+void conv_inputs(torch::Tensor qkv, c10::optional<torch::Tensor> bias, c10::optional<torch::Tensor> taps, c10::optional<torch::Tensor> state,
+                 c10::optional<torch::Tensor> q_w, c10::optional<torch::Tensor> k_w, c10::optional<torch::Tensor> table, torch::Tensor q,
+                 c10::optional<torch::Tensor> k_pool, c10::optional<torch::Tensor> v_pool, torch::Tensor slots, torch::Tensor ctx, torch::Tensor state_slot,
+                 c10::optional<torch::Tensor> cu, c10::optional<torch::Tensor> seg_of, c10::optional<torch::Tensor> pos, int64_t kv_heads, int64_t dim,
+                 int64_t vdim, int64_t rot, double eps) {
+  const c10::cuda::CUDAGuard guard(qkv.device());
+  check_same(qkv, q, "conv_inputs");
+  const int64_t T = qkv.size(0), C = q.size(1) * dim + (k_pool.has_value() ? kv_heads * (dim + vdim) : 0);
+  TORCH_CHECK(qkv.dim() == 2 && qkv.stride(1) == 1 && qkv.size(1) >= C && q.dim() == 3 && q.is_contiguous() && q.size(0) == T && k_pool.has_value() == v_pool.has_value());
+  TORCH_CHECK(rot == 0 || (table.has_value() && table->scalar_type() == at::kFloat && table->is_contiguous() && table->numel() == T * rot));
+  TORCH_CHECK(slots.scalar_type() == at::kLong && slots.is_contiguous() && slots.numel() == T);
+  check_segments(state_slot, ctx, cu, T, "conv_inputs");
+  TORCH_CHECK(!cu.has_value() || (seg_of.has_value() && is_i32(*seg_of) && seg_of->numel() == T && pos.has_value() && is_i32(*pos) && pos->numel() == T));
+  const int64_t n = taps.has_value() ? taps->size(1) : 1;
+  for (const auto& o : {bias, taps, q_w, k_w, state})
+    if (o.has_value()) {
+      check_same(qkv, *o, "conv_inputs");
+      TORCH_CHECK(o->is_contiguous());
+    }
+  TORCH_CHECK((!bias.has_value() || bias->numel() >= C) && (!taps.has_value() || (taps->dim() == 2 && taps->size(0) >= C)), "conv_inputs: weights");
+  TORCH_CHECK(n == 1 || (state.has_value() && state->dim() == 3 && state->size(1) == n - 1 && state->size(2) == C), "conv_inputs: state");
+  TORCH_CHECK((!q_w.has_value() || q_w->numel() >= dim) && (!k_w.has_value() || k_w->numel() >= dim), "conv_inputs: norms");
+  if (k_pool.has_value()) {
+    check_same(qkv, *k_pool, "conv_inputs");
+    check_same(qkv, *v_pool, "conv_inputs");
+    TORCH_CHECK(k_pool->dim() == 3 && v_pool->dim() == 3 && k_pool->is_contiguous() && v_pool->is_contiguous() && k_pool->size(0) == v_pool->size(0));
+    TORCH_CHECK(k_pool->size(1) == kv_heads && v_pool->size(1) == kv_heads && k_pool->size(2) == q.size(2), "conv_inputs: pools");
+  }
+  check(rb_conv_inputs(qkv.data_ptr(), (int)qkv.stride(0), optptr(bias), optptr(taps), (int)n, state.has_value() ? state->data_ptr() : nullptr, optptr(q_w),
+                       optptr(k_w), rot ? table->data_ptr<float>() : nullptr, q.data_ptr(), k_pool.has_value() ? k_pool->data_ptr() : nullptr,
+                       v_pool.has_value() ? v_pool->data_ptr() : nullptr, (const long long*)slots.data_ptr<int64_t>(), ctx.data_ptr<int>(),
+                       state_slot.data_ptr<int>(), optint(cu), cu.has_value() ? optint(seg_of) : nullptr, cu.has_value() ? optint(pos) : nullptr,
+                       k_pool.has_value() ? k_pool->size(0) : 0, (int)T, (int)ctx.numel(), (int)q.size(1), (int)kv_heads, (int)dim, (int)vdim, (int)q.size(2),
+                       v_pool.has_value() ? (int)v_pool->size(2) : 0, (int)rot, (float)eps, is_fp32(qkv), cur_stream()),
+        "rb_conv_inputs");
+}
+void mingru(torch::Tensor rows, torch::Tensor z_b, torch::Tensor x_b, torch::Tensor state, torch::Tensor slot, torch::Tensor ctx, c10::optional<torch::Tensor> cu,
+            c10::optional<torch::Tensor> spans, c10::optional<torch::Tensor> first, c10::optional<torch::Tensor> span_sum,
+            c10::optional<torch::Tensor> span_keep, torch::Tensor out, int64_t width) {
+  const c10::cuda::CUDAGuard guard(rows.device());
+  const int64_t pitch = (width + 7) / 8 * 8, T = rows.size(0);
+  for (const auto& t : {z_b, x_b, out}) {
+    check_same(rows, t, "mingru");
+    TORCH_CHECK(t.is_contiguous());
+  }
+  TORCH_CHECK(rows.dim() == 2 && rows.stride(1) == 1 && rows.size(1) >= 3 * pitch && out.dim() == 2 && out.size(0) == T && out.size(1) == pitch && z_b.numel() >= pitch &&
+              x_b.numel() >= pitch && reinterpret_cast<uintptr_t>(rows.data_ptr()) % 8 == 0, "mingru: rows");
+  TORCH_CHECK(state.scalar_type() == at::kFloat && state.is_contiguous() && state.dim() >= 2, "mingru: state");
+  check_segments(slot, ctx, cu, T, "mingru");
+  const int64_t n = cu.has_value() ? check_spans(spans, first, slot.numel(), "mingru") : 0;
+  if (n)
+    for (const auto& o : {span_sum, span_keep}) TORCH_CHECK(o.has_value() && o->scalar_type() == at::kFloat && o->numel() >= n * pitch, "mingru: scratch");
+  check(rb_mingru(rows.data_ptr(), z_b.data_ptr(), x_b.data_ptr(), state.data_ptr<float>(), slot.data_ptr<int>(), ctx.data_ptr<int>(), optint(cu),
+                  n ? spans->data_ptr<int>() : nullptr, n ? first->data_ptr<int>() : nullptr, n ? span_sum->data_ptr<float>() : nullptr,
+                  n ? span_keep->data_ptr<float>() : nullptr, out.data_ptr(), (int)slot.numel(), (int)n, (int)width, (int)rows.stride(0), (int)state.stride(0),
+                  is_fp32(rows), cur_stream()),
+        "rb_mingru");
+}
+// o_raw: scratch of the CUDA-core scan; without it segments run on the tensor cores.  Returns false for shapes those do not take.
+bool gla(torch::Tensor rows, torch::Tensor z, torch::Tensor z_bias, torch::Tensor norm_w, torch::Tensor state, torch::Tensor slot, torch::Tensor ctx,
+         c10::optional<torch::Tensor> cu, c10::optional<torch::Tensor> o_raw, c10::optional<torch::Tensor> spans, c10::optional<torch::Tensor> first,
+         c10::optional<torch::Tensor> span_state, c10::optional<torch::Tensor> span_gate, torch::Tensor out, int64_t dim, int64_t vdim, int64_t gate_col,
+         double eps, double root) {
+  const c10::cuda::CUDAGuard guard(rows.device());
+  for (const auto& t : {z_bias, norm_w, out}) {
+    check_same(rows, t, "gla");
+    TORCH_CHECK(t.is_contiguous());
+  }
+  const int64_t H = state.size(1), T = rows.size(0), segs = slot.numel();
+  TORCH_CHECK(state.dim() == 4 && state.scalar_type() == at::kFloat && state.is_contiguous() && state.size(2) == dim, "gla: state");
+  TORCH_CHECK(rows.dim() == 2 && rows.stride(1) == 1 && rows.size(1) >= gate_col + H * vdim && gate_col >= H * (2 * dim + vdim) && out.size(0) == T, "gla: rows");
+  TORCH_CHECK(z.dim() == 2 && z.scalar_type() == at::kFloat && z.stride(1) == 1 && z.size(0) == T && z.size(1) >= H * dim, "gla: decay");
+  TORCH_CHECK(z_bias.numel() == H * dim && norm_w.numel() == vdim && root > 0, "gla: weights");
+  check_segments(slot, ctx, cu, T, "gla");
+  const float q_scale = 1.f / std::sqrt((float)dim), inv_root = (float)(1.0 / root);
+  if (cu.has_value() && !o_raw.has_value()) {
+    TORCH_CHECK(rows.scalar_type() == at::kBFloat16, "gla: the 32-bit scan needs its scratch");
+    const int64_t n = check_spans(spans, first, segs, "gla");
+    if (n) {
+      TORCH_CHECK(span_state.has_value() && span_state->scalar_type() == at::kFloat && span_state->numel() >= n * state.stride(0));
+      TORCH_CHECK(span_gate.has_value() && span_gate->scalar_type() == at::kFloat && span_gate->numel() >= n * H * dim);
+    }
+    const int rc = rb_gla_chunk(rows.data_ptr(), z.data_ptr<float>(), (int)z.stride(0), z_bias.data_ptr(), norm_w.data_ptr(), state.data_ptr<float>(),
+                                slot.data_ptr<int>(), ctx.data_ptr<int>(), cu->data_ptr<int>(), n ? spans->data_ptr<int>() : nullptr,
+                                n ? first->data_ptr<int>() : nullptr, n ? span_state->data_ptr<float>() : nullptr, n ? span_gate->data_ptr<float>() : nullptr,
+                                out.data_ptr(), (int)T, (int)segs, (int)n, (int)H, (int)dim, (int)vdim, (int)state.size(3), (int)rows.stride(0),
+                                (int)out.size(1), (int)gate_col, (float)eps, q_scale, inv_root, cur_stream());
+    if (rc == -20) return false;
+    check(rc, "rb_gla_chunk");
+    return true;
+  }
+  TORCH_CHECK(!cu.has_value() || (o_raw->scalar_type() == at::kFloat && o_raw->numel() >= T * H * vdim), "gla: scratch");
+  check(rb_gla(rows.data_ptr(), z.data_ptr<float>(), (int)z.stride(0), z_bias.data_ptr(), norm_w.data_ptr(), state.data_ptr<float>(), slot.data_ptr<int>(),
+               ctx.data_ptr<int>(), optint(cu), o_raw.has_value() ? o_raw->data_ptr<float>() : nullptr, out.data_ptr(), (int)T, (int)segs, (int)H, (int)dim,
+               (int)vdim, (int)state.size(3), (int)rows.stride(0), (int)out.size(1), (int)gate_col, (float)eps, q_scale, inv_root, is_fp32(rows), cur_stream()),
+        "rb_gla");
+  return true;
+}
+// y: none, one or two sublayer outputs; yw: weights of their norms or none; norms: one or two weights, or none (h[0] is a copy of the stream)
+void stream_step(torch::Tensor res, std::vector<torch::Tensor> y, std::vector<torch::Tensor> yw, c10::optional<torch::Tensor> ex,
+                 c10::optional<torch::Tensor> expert, c10::optional<torch::Tensor> place, c10::optional<torch::Tensor> offset,
+                 c10::optional<torch::Tensor> weight, std::vector<torch::Tensor> norms, std::vector<torch::Tensor> h, c10::optional<torch::Tensor> mu,
+                 c10::optional<torch::Tensor> state, c10::optional<torch::Tensor> slot, c10::optional<torch::Tensor> ctx, int64_t width, double eps) {
+  const c10::cuda::CUDAGuard guard(res.device());
+  const int64_t T = res.size(0), pitch = res.size(1);
+  TORCH_CHECK(res.dim() == 2 && res.is_contiguous() && res.scalar_type() == at::kFloat && y.size() <= 2 && (yw.empty() || yw.size() == y.size()) &&
+              norms.size() <= 2 && h.size() == (norms.empty() ? 1 : norms.size()), "stream_step: operands");
+  for (const auto& t : h) {
+    check_same(h[0], t, "stream_step");
+    TORCH_CHECK(t.is_contiguous() && t.sizes() == res.sizes());
+  }
+  for (const auto& t : y) {
+    check_same(h[0], t, "stream_step");
+    TORCH_CHECK(t.dim() == 2 && t.size(0) == T && t.stride(1) == 1 && t.size(1) >= width && reinterpret_cast<uintptr_t>(t.data_ptr()) % 16 == 0, "stream_step: outputs");
+  }
+  for (const auto* v : {&yw, &norms})
+    for (const auto& t : *v) {
+      check_same(h[0], t, "stream_step");
+      TORCH_CHECK(t.is_contiguous() && t.numel() == pitch, "stream_step: weights");
+    }
+  int top = 0;
+  if (ex.has_value()) {
+    check_same(h[0], *ex, "stream_step");
+    TORCH_CHECK(expert.has_value() && place.has_value() && offset.has_value() && weight.has_value() && is_i32(*expert) && is_i32(*place) && is_i32(*offset) &&
+                weight->scalar_type() == at::kFloat && weight->is_contiguous() && expert->dim() == 2 && expert->size(0) == T && ex->is_contiguous() && ex->dim() == 2,
+                "stream_step: experts");
+    top = (int)expert->size(1);
+  }
+  if (mu.has_value()) {
+    check_same(h[0], *mu, "stream_step");
+    TORCH_CHECK(mu->numel() == pitch && state.has_value() && state->is_contiguous() && state->dim() == 2 && state->size(1) == pitch, "stream_step: shift");
+    check_same(h[0], *state, "stream_step");
+    check_segments(*slot, *ctx, c10::nullopt, T, "stream_step");
+  }
+  check(rb_stream_step(res.data_ptr<float>(), y.size() > 0 ? y[0].data_ptr() : nullptr, y.size() > 0 ? (int)y[0].stride(0) : 0,
+                       y.size() > 1 ? y[1].data_ptr() : nullptr, y.size() > 1 ? (int)y[1].stride(0) : 0, yw.size() > 0 ? yw[0].data_ptr() : nullptr,
+                       yw.size() > 1 ? yw[1].data_ptr() : nullptr, optptr(ex), ex.has_value() ? (int)ex->size(1) : 0, optint(expert), optint(place),
+                       optint(offset), weight.has_value() ? weight->data_ptr<float>() : nullptr, top, norms.size() > 0 ? norms[0].data_ptr() : nullptr,
+                       norms.size() > 1 ? norms[1].data_ptr() : nullptr, h[0].data_ptr(), h.size() > 1 ? h[1].data_ptr() : nullptr, optptr(mu),
+                       state.has_value() ? state->data_ptr() : nullptr, optint(slot), optint(ctx), (int)T, (int)pitch, (int)width, (float)eps, is_fp32(h[0]),
+                       cur_stream()),
+        "rb_stream_step");
+}
+void token_shift(torch::Tensor n, torch::Tensor mu, torch::Tensor state, torch::Tensor out, torch::Tensor slot, torch::Tensor ctx, torch::Tensor cu,
+                 torch::Tensor seg_of) {
+  const c10::cuda::CUDAGuard guard(n.device());
+  for (const auto& t : {mu, state, out}) {
+    check_same(n, t, "token_shift");
+    TORCH_CHECK(t.is_contiguous());
+  }
+  const int64_t T = n.size(0), pitch = n.size(1);
+  TORCH_CHECK(n.is_contiguous() && n.dim() == 2 && out.sizes() == n.sizes() && mu.numel() == pitch && state.dim() == 2 && state.size(1) == pitch, "token_shift: rows");
+  check_segments(slot, ctx, cu, T, "token_shift");
+  TORCH_CHECK(is_i32(seg_of) && seg_of.numel() == T, "token_shift: rows");
+  check(rb_token_shift(n.data_ptr(), mu.data_ptr(), state.data_ptr(), out.data_ptr(), slot.data_ptr<int>(), ctx.data_ptr<int>(), cu.data_ptr<int>(),
+                       seg_of.data_ptr<int>(), (int)T, (int)pitch, is_fp32(n), cur_stream()),
+        "rb_token_shift");
+}
+// embed [vocab][..]: a layer's own columns start at `first`
+void side_gate(torch::Tensor z, torch::Tensor embed, torch::Tensor tokens, torch::Tensor out, int64_t first, int64_t dim) {
+  const c10::cuda::CUDAGuard guard(z.device());
+  check_same(z, embed, "side_gate");
+  check_same(z, out, "side_gate");
+  const int64_t T = z.size(0);
+  TORCH_CHECK(z.dim() == 2 && z.stride(1) == 1 && z.size(1) >= dim && embed.dim() == 2 && embed.is_contiguous() && first >= 0 && first + dim <= embed.size(1));
+  TORCH_CHECK(out.dim() == 2 && out.is_contiguous() && out.size(0) == T && out.size(1) >= dim && tokens.scalar_type() == at::kLong && tokens.is_contiguous() &&
+              tokens.numel() == T, "side_gate: rows");
+  const char* e = static_cast<const char*>(embed.data_ptr()) + first * embed.element_size();
+  check(rb_side_gate(z.data_ptr(), (int)z.stride(0), e, embed.size(1), (const long long*)tokens.data_ptr<int64_t>(), (int)embed.size(0), out.data_ptr(), (int)T,
+                     (int)dim, (int)out.size(1), is_fp32(z), cur_stream()),
+        "rb_side_gate");
+}
+void softcap(torch::Tensor z, double cap) {
+  const c10::cuda::CUDAGuard guard(z.device());
+  TORCH_CHECK(z.is_contiguous() && z.scalar_type() == at::kFloat);
+  check(rb_softcap(z.data_ptr<float>(), z.numel(), (float)cap, cur_stream()), "rb_softcap");
 }
 void moe_route(torch::Tensor logits, c10::optional<torch::Tensor> correction, torch::Tensor expert, torch::Tensor weight, torch::Tensor place, torch::Tensor row_token, torch::Tensor count,
                torch::Tensor offset, torch::Tensor tiles, torch::Tensor n_tiles, int64_t experts, int64_t outputs, int64_t groups, int64_t keep,
@@ -539,14 +739,14 @@ void moe_route(torch::Tensor logits, c10::optional<torch::Tensor> correction, to
                      (float)weight_scale, cur_stream()),
         "rb_moe_route");
 }
-// out[sorted row] = act(x[its token, or the sorted row] * W[expert]^T); act: 0 none, 1 squared relu, 2 gated (half as many columns out)
+// out[sorted row] = act(x[its token, or the sorted row] * W[expert]^T); act: 0 none, 1 squared relu, 2 and 3 gated (half as many columns out)
 void moe_gemm(torch::Tensor x, torch::Tensor W, torch::Tensor out, torch::Tensor tiles, torch::Tensor n_tiles, c10::optional<torch::Tensor> row_token,
               int64_t act, double limit, int64_t bn, bool full, torch::Tensor err) {
   const c10::cuda::CUDAGuard guard(x.device());
   check_same(x, W, "moe_gemm");
   check_same(x, out, "moe_gemm");
   const int64_t E = W.size(0), N = W.size(1), K = W.size(2);
-  TORCH_CHECK(x.dim() == 2 && W.dim() == 3 && out.dim() == 2 && x.is_contiguous() && W.is_contiguous() && out.is_contiguous() && x.size(1) == K && out.size(1) == (act == 2 ? N / 2 : N));
+  TORCH_CHECK(x.dim() == 2 && W.dim() == 3 && out.dim() == 2 && x.is_contiguous() && W.is_contiguous() && out.is_contiguous() && x.size(1) == K && out.size(1) == (act >= 2 ? N / 2 : N));
   TORCH_CHECK(is_i32(tiles) && is_i32(n_tiles) && (!row_token.has_value() || is_i32(*row_token)));
   TORCH_CHECK(row_token.has_value() ? row_token->numel() >= E * x.size(0) : x.size(0) == out.size(0), "moe_gemm: rows");
   const int cap = (int)tiles.size(0);
@@ -598,6 +798,14 @@ void register_serving(pybind11::module_& m) {
   m.def("paged_flash", &paged_flash);
   m.def("dense_flash", &dense_flash);
   m.def("paged_decode", &paged_decode);
+  m.def("mix_heads", &mix_heads);
+  m.def("conv_inputs", &conv_inputs);
+  m.def("mingru", &mingru);
+  m.def("gla", &gla);
+  m.def("stream_step", &stream_step);
+  m.def("token_shift", &token_shift);
+  m.def("side_gate", &side_gate);
+  m.def("softcap", &softcap);
   m.def("moe_route", &moe_route);
   m.def("moe_gemm", &moe_gemm);
   m.def("relu2", &relu2);

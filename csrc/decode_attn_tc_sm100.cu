@@ -59,8 +59,24 @@ struct DecodeTcParams {
   float* part_ml;           // [B*Hq*splits][2]
   int Hq, Hkv, G, max_blocks, page, out_d, num_splits, split_tokens, ld_gate;
   int window;               // positions a token sees (INT_MAX: all)
+  int keep;                 // first positions that stay visible outside the window
+  int chunk;                // > 0: a token sees its own chunk of this many positions
   float scale_log2;
+  float cap_in, cap_log2;   // cap_log2 > 0: scores are cap_log2 tanh(cap_in q . k), in log2 units
   int* err;
+};
+
+// Pages that a token at the end of a context of `ctx` positions sees: the first `kept` pages of its sequence, then those from page
+// `first` on.  A position counts from 0 through these pages.
+struct SeenPages {
+  int from, first, kept, total;      // first position of the window or chunk; total: positions of all these pages
+  __device__ __forceinline__ SeenPages(const DecodeTcParams& p, int ctx) {
+    from = p.chunk ? (ctx - 1) / p.chunk * p.chunk : max(0, ctx - p.window);
+    first = from / p.page;
+    kept = min((p.keep + p.page - 1) / p.page, first);
+    total = kept * p.page + ctx - first * p.page;
+  }
+  __device__ __forceinline__ int page(int i) const { return i < kept ? i : first + i - kept; }
 };
 
 // the sink's term joins numerator and denominator (m: the reference of both, in log2 units)
@@ -99,9 +115,9 @@ decode_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_k, const __grid_co
   const int b = blockIdx.x, kvh = blockIdx.y, split = blockIdx.z;
   const int G = p.G;
   const int ctx = p.ctx_lens[b];
-  const int seen_from = max(0, ctx - p.window);                             // first position in the window
-  const int t_begin = seen_from / p.page * p.page + split * p.split_tokens;    // (tiles start on a page)
-  const int t_end = min(ctx, t_begin + p.split_tokens);
+  const SeenPages seen(p, ctx);
+  const int t_begin = split * p.split_tokens;                               // positions of the seen pages (tiles start on a page)
+  const int t_end = min(seen.total, t_begin + p.split_tokens);
   const int n_tiles = t_end > t_begin ? (t_end - t_begin + DT_TILE - 1) / DT_TILE : 0;
   const int* bt = p.block_tables + static_cast<size_t>(b) * p.max_blocks;
 
@@ -156,7 +172,7 @@ decode_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_k, const __grid_co
         const int page0 = (t_begin + (u >> 1) * DT_TILE) / p.page;
         mbar_expect_tx(&full[s], two ? 2 * DT_HALF : DT_HALF);
         for (int pg = 0; pg < DT_TILE / p.page; ++pg) {
-          const int idx = min(page0 + pg, p.max_blocks - 1);
+          const int idx = min(seen.page(page0 + pg), p.max_blocks - 1);
           const int row = bt[idx] * p.page;
           tma_load_3d(dst + pg * p.page * 128, map, &full[s], 0, kvh, row);
           if (two) tma_load_3d(dst + DT_HALF + pg * p.page * 128, map, &full[s], 64, kvh, row);
@@ -223,12 +239,17 @@ decode_attn_tc_kernel(const __grid_constant__ CUtensorMap tma_k, const __grid_co
       uint32_t raw[16];
       tmem_ld_32x32b_x16(tmem_base + DT_T_S + (j & 1) * 16 + lane_addr, raw);
       tmem_wait_ld();
-      const int tok = t_begin + j * DT_TILE + r;
-      const bool valid = tok < t_end && tok >= seen_from;
+      const int i = t_begin + j * DT_TILE + r, tok = seen.page(i / p.page) * p.page + i % p.page;
+      const bool valid = i < t_end && (tok >= seen.from || tok < p.keep);
       float s[NH];
 #pragma unroll
       for (int h = 0; h < NH; ++h) {
-        s[h] = (valid && h < G) ? __uint_as_float(raw[h]) * p.scale_log2 : -1e30f;
+        s[h] = -1e30f;
+        if (valid && h < G) {
+          const float x = __uint_as_float(raw[h]);
+          // tanh in fp32 up to about 1e-7 (2 / ln 2)
+          s[h] = p.cap_log2 > 0.f ? p.cap_log2 * (1.f - __fdividef(2.f, 1.f + exp2f(2.8853900817779268f * fminf(p.cap_in * x, 20.f)))) : x * p.scale_log2;
+        }
         const float wm = warp_max(s[h]);
         if (lane == 0) red_max[warp * 16 + h] = wm;
       }
@@ -396,26 +417,32 @@ extern "C" int rb_decode_attn_tc(const void* q, const void* kc, const void* vc, 
 }
 
 // The same over pools [rows][Hkv][dk] / [rows][Hkv][dv] (dk, dv: 64 or 128) with pages of 16 to 128 tokens, an optional sink
-// logit per head, an optional window (positions a token sees, its own included; 0: all), an optional gate per output feature and
-// outputs of out_d columns.  max_ctx: most positions any row may see, rounded up by less than a page at a window's far end
-// (the splits share them out).  Returns -20 for shapes outside that.
+// logit per head, an optional window (positions a token sees, its own included; 0: all) that leaves the first `keep` positions visible or
+// chunks of `chunk` positions, optionally capped scores, an optional gate per output feature and outputs of out_d columns.  max_ctx: most
+// positions any row may see, pages that count in part as a whole (the splits share them out).  Returns -20 for shapes outside that.
 extern "C" int rb_paged_decode_tc(const void* q, const void* kc, const void* vc, const int* block_tables, const int* ctx_lens,
                                   const void* sink, const void* gate, int ld_gate, void* out, float* part_o, float* part_ml, int B, int Hq,
                                   int Hkv, int dk, int dv, int out_d, long long pool_rows, int page, int max_blocks, int max_ctx, int window,
-                                  float scale, int splits, int* err, cudaStream_t st) {
+                                  int keep, int chunk, float scale, float cap, int splits, int* err, cudaStream_t st) {
   using namespace rb;
   if (B == 0) return 0;
   if (Hkv < 1 || Hq % Hkv) return -2;
   const int G = Hq / Hkv;
   if (G > 16 || (dk != 64 && dk != 128) || (dv != 64 && dv != 128) || out_d > dv || out_d < 1) return -20;
   if ((page != 16 && page != 32 && page != 64 && page != 128) || Hkv > 65535 || splits < 1 || splits > 65535) return -20;
-  if (window < 0 || (gate && ld_gate < Hq * out_d)) return -2;
-  if (window && window + page < max_ctx) max_ctx = window + page;
+  if (window < 0 || keep < 0 || chunk < 0 || cap < 0.f || (chunk && window) || (keep && !window) || (gate && ld_gate < Hq * out_d)) return -2;
+  const long long most = chunk ? static_cast<long long>(chunk) + page : window + static_cast<long long>(keep) + 2 * page;
+  if ((chunk || window) && most < max_ctx) max_ctx = static_cast<int>(most);
   DecodeTcParams p = decode_tc_params(q, block_tables, ctx_lens, out, part_o, part_ml, Hq, Hkv, page, max_blocks, max_ctx, scale, splits, err);
   p.sink = (const __nv_bfloat16*)sink;
   p.gate = (const __nv_bfloat16*)gate; p.ld_gate = ld_gate;
   if (window) p.window = window;
   p.out_d = out_d;
+  p.keep = keep; p.chunk = chunk;
+  if (cap > 0.f) {
+    p.cap_in = scale / cap;
+    p.cap_log2 = cap * 1.4426950408889634f;
+  }
   const uint64_t slots = static_cast<uint64_t>(pool_rows);
   if (G <= 8) {
     if (dk == 128 && dv == 128) return launch_decode_tc<128, 128, 8>(kc, vc, slots, p, B, st);

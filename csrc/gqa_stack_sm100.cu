@@ -5,6 +5,9 @@
 //  * attention_inputs  raw projections -> rotated and normed queries; keys and values into their pages (norms head by head, pairs
 //                      of neighbours)
 //  * projection_inputs the same with weighted norms over the whole query and key projections, and either pairing
+//  * conv_inputs       the same with biases, a short causal convolution over time on every channel (the last rows of a sequence wait in a
+//                      state slot) and weighted norms head by head
+//  * mix_heads         outputs of every head's weights on every group's values -> heads whose weights were mixed
 //  * paged_attention   one (row, head) per CTA: 32-bit mode, and head sizes that the tensor-core kernels do not take
 #include "stack_common.cuh"
 
@@ -212,6 +215,226 @@ __global__ void __launch_bounds__(PI_WARPS * 32) projection_inputs_kernel(const 
   }
 }
 
+// One warp per (head, run of RUN rows): raw rows slide through registers, so a run reads every row once.  Lane l holds the feature pairs
+// l, l + 32, ...  With one row per sequence the warp also moves the state on; otherwise conv_state_kernel does, afterwards.
+struct ConvParams {
+  const void* qkv;           // [T][ld]: H query heads | G key heads | G value heads (keys and values only with k_pool)
+  const void* bias;          // [C] or null
+  const void* taps;          // [C][n], the last one on the row itself; null: none
+  void* state;               // [slots][n - 1][C] raw rows before a segment, the newest last
+  const void* q_w;           // [dim] weights of the norms (eps > 0)
+  const void* k_w;
+  const float2* table;       // [T][rot / 2] or null
+  void* q;                   // [T][H][dp]
+  void* k_pool;              // [rows][G][dp] or null
+  void* v_pool;              // [rows][G][vp]
+  const long long* slots;    // [T] pool rows
+  const int* ctx;            // [segments]
+  const int* state_slot;     // [segments]
+  const int* cu;             // [segments + 1]; null: one row per segment
+  const int* seg_of;         // [T] (with cu)
+  const int* pos;            // [T] (with cu)
+  long long pool_rows;
+  int T, H, G, dim, vdim, dp, vp, rot, ld, n, C;
+  float eps;                 // <= 0: no norm
+};
+template <typename T, bool kPair>
+__device__ __forceinline__ void load_pair(const T* p, int left, float& a, float& b) {      // `left` elements from here on
+  a = b = 0.f;
+  if constexpr (kPair) {
+    if (left > 0) {
+      if constexpr (sizeof(T) == 4) {
+        const float2 x = *reinterpret_cast<const float2*>(p);
+        a = x.x;
+        b = x.y;
+      } else {
+        const uint32_t x = *reinterpret_cast<const uint32_t*>(p);
+        a = __uint_as_float(x << 16);
+        b = __uint_as_float(x & 0xffff0000u);
+      }
+    }
+  } else {
+    if (left > 0) a = ld(p);
+    if (left > 1) b = ld(p + 1);
+  }
+}
+template <typename T, bool kPair>
+__device__ __forceinline__ void store_pair(T* p, int left, float a, float b) {
+  if constexpr (kPair) {
+    if (left > 0) {
+      if constexpr (sizeof(T) == 4) *reinterpret_cast<float2*>(p) = make_float2(a, b);
+      else *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(a, b);
+    }
+  } else {
+    if (left > 0) st(p, a);
+    if (left > 1) st(p + 1, b);
+  }
+}
+template <typename T, int NP, int NT, int RUN, bool kPair>
+__global__ void __launch_bounds__(256) conv_inputs_kernel(const ConvParams p) {
+  const int lane = threadIdx.x & 31;
+  const int per = p.H + (p.k_pool ? 2 * p.G : 0);
+  const long long u = static_cast<long long>(blockIdx.x) * 8 + (threadIdx.x >> 5);
+  const long long run = u / per;
+  const int hd = static_cast<int>(u - run * per);
+  const int t0 = static_cast<int>(run) * RUN, t1 = min(p.T, t0 + RUN);
+  if (t0 >= t1) return;
+  const bool value = hd >= p.H + p.G;
+  const int n = value ? p.vdim : p.dim, pitch = value ? p.vp : p.dp;
+  const int g = hd - (hd < p.H ? 0 : p.H + (value ? p.G : 0));
+  const int ch = (hd < p.H ? 0 : p.H * p.dim + (value ? p.G * p.dim : 0)) + g * n;      // first channel of the head
+  const T* src = static_cast<const T*>(p.qkv) + ch;
+  const bool normed = !value && p.eps > 0.f;
+  float w[NP][2][NT], bias[NP][2], nw[NP][2];
+#pragma unroll
+  for (int i = 0; i < NP; ++i) {
+    const int e = 2 * (lane + 32 * i), left = n - e;
+#pragma unroll
+    for (int k = 0; k < NT; ++k) w[i][0][k] = w[i][1][k] = 0.f;
+    if (p.taps) {
+      const T* tp = static_cast<const T*>(p.taps) + static_cast<long long>(ch + e) * p.n;
+#pragma unroll
+      for (int k = 0; k < NT; ++k)
+        if (k < p.n) {
+          if (left > 0) w[i][0][k] = ld(tp + p.n - 1 - k);
+          if (left > 1) w[i][1][k] = ld(tp + 2 * p.n - 1 - k);
+        }
+    } else {
+      w[i][0][0] = w[i][1][0] = 1.f;
+    }
+    bias[i][0] = bias[i][1] = 0.f;
+    nw[i][0] = nw[i][1] = 1.f;
+    if (p.bias) load_pair<T, false>(static_cast<const T*>(p.bias) + ch + e, left, bias[i][0], bias[i][1]);
+    if (normed) load_pair<T, false>(static_cast<const T*>(hd < p.H ? p.q_w : p.k_w) + e, left, nw[i][0], nw[i][1]);
+  }
+  float past[NP][2][NT > 1 ? NT - 1 : 1];      // raw rows t - 1, t - 2, ...
+  int seg = -1;
+  for (int t = t0; t < t1; ++t) {
+    const int s = p.cu ? p.seg_of[t] : t, at = p.cu ? p.pos[t] : p.ctx[t] - 1, local = p.cu ? t - p.cu[s] : 0;
+    T* state = p.n > 1 ? static_cast<T*>(p.state) + static_cast<long long>(p.state_slot[s]) * (p.n - 1) * p.C + ch : nullptr;
+    if (s != seg) {
+      seg = s;
+#pragma unroll
+      for (int k = 1; k < NT; ++k) {
+        const T* from = k <= local ? src + static_cast<long long>(t - k) * p.ld : state + static_cast<long long>(p.n - 1 - (k - local)) * p.C;
+#pragma unroll
+        for (int i = 0; i < NP; ++i) {
+          const int e = 2 * (lane + 32 * i);
+          past[i][0][k - 1] = past[i][1][k - 1] = 0.f;
+          if (k < p.n && k <= at) load_pair<T, kPair>(from + e, n - e, past[i][0][k - 1], past[i][1][k - 1]);
+        }
+      }
+    }
+    float y[NP][2], ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < NP; ++i) {
+      const int e = 2 * (lane + 32 * i);
+      float x[2];
+      load_pair<T, kPair>(src + static_cast<long long>(t) * p.ld + e, n - e, x[0], x[1]);
+      if (!p.cu && p.n > 1) {      // the state moves on by one row
+#pragma unroll
+        for (int k = NT - 1; k >= 1; --k)
+          if (k < p.n) store_pair<T, kPair>(state + static_cast<long long>(p.n - 1 - k) * p.C + e, n - e, k > 1 ? past[i][0][k > 1 ? k - 2 : 0] : x[0],
+                                            k > 1 ? past[i][1][k > 1 ? k - 2 : 0] : x[1]);
+      }
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        float a = w[i][h][0] * (x[h] + bias[i][h]);
+#pragma unroll
+        for (int k = 1; k < NT; ++k)
+          if (k <= at) a += w[i][h][k] * (past[i][h][k - 1] + bias[i][h]);      // (taps behind the last one are zero)
+#pragma unroll
+        for (int k = NT - 1; k > 1; --k) past[i][h][k - 1] = past[i][h][k - 2];
+        if (NT > 1) past[i][h][0] = x[h];
+        y[i][h] = a;
+        ss += a * a;
+      }
+    }
+    if (normed) {
+      const float r = 1.f / sqrtf(wsum(ss) / p.dim + p.eps);
+#pragma unroll
+      for (int i = 0; i < NP; ++i) {
+        y[i][0] *= r * nw[i][0];
+        y[i][1] *= r * nw[i][1];
+      }
+    }
+    T* dst;
+    if (hd < p.H) {
+      dst = static_cast<T*>(p.q) + (static_cast<long long>(t) * p.H + hd) * p.dp;
+    } else {
+      const long long slot = p.slots[t];
+      if (slot < 0 || slot >= p.pool_rows) continue;
+      dst = static_cast<T*>(value ? p.v_pool : p.k_pool) + (slot * p.G + g) * pitch;
+    }
+#pragma unroll
+    for (int i = 0; i < NP; ++i) {      // columns behind the head's features are written as zeros
+      const int e = 2 * (lane + 32 * i);
+      if (!value && e < p.rot) {
+        const float2 cs = p.table[static_cast<long long>(t) * (p.rot >> 1) + (e >> 1)];
+        const float a = y[i][0] * cs.x - y[i][1] * cs.y;
+        y[i][1] = y[i][1] * cs.x + y[i][0] * cs.y;
+        y[i][0] = a;
+      }
+      store_pair<T, true>(dst + e, pitch - e, y[i][0], y[i][1]);
+    }
+  }
+}
+
+// The last n - 1 raw rows of every segment, or of what was before it and the segment together, become its state.
+template <typename T>
+__global__ void __launch_bounds__(256) conv_state_kernel(const ConvParams p) {
+  const int s = blockIdx.x, c = blockIdx.y * 256 + threadIdx.x;
+  if (c >= p.C) return;
+  const int lo = p.cu[s], len = p.cu[s + 1] - lo;
+  const bool fresh = p.ctx[s] == len;
+  T* state = static_cast<T*>(p.state) + static_cast<long long>(p.state_slot[s]) * (p.n - 1) * p.C + c;
+  const T* src = static_cast<const T*>(p.qkv) + c;
+  for (int j = 0; j < p.n - 1; ++j) {      // (what is read lies behind what has been written)
+    const int i = len + j;
+    float v;
+    if (i >= p.n - 1) v = ld(src + static_cast<long long>(lo + i - (p.n - 1)) * p.ld);
+    else v = fresh ? 0.f : ld(state + static_cast<long long>(i) * p.C);
+    st(state + static_cast<long long>(j) * p.C, v);
+  }
+}
+
+// out[t][h] = sum over g of mix[h][g] wide[t][g][group of h]: `wide` holds what every head's weights make of every group's values.
+// Thread = (token, four heads of one group, V columns).
+template <typename T, int V>
+__global__ void __launch_bounds__(128) mix_heads_kernel(const T* __restrict__ wide, const T* __restrict__ mix, T* __restrict__ out, long long units, int H,
+                                                        int G, int vo) {
+  const long long u = static_cast<long long>(blockIdx.x) * 128 + threadIdx.x;
+  if (u >= units) return;
+  const int cols = vo / V, rep = H / G, quads = (rep + 3) / 4;
+  const int c = static_cast<int>(u % cols) * V;
+  long long r = u / cols;
+  const int quad = static_cast<int>(r % quads) * 4;
+  r /= quads;
+  const int grp = static_cast<int>(r % G);
+  const long long t = r / G;
+  const T* src = wide + (t * H * G + grp) * vo + c;
+  const T* m = mix + static_cast<long long>(grp * rep + quad) * H;
+  float acc[4][V];
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int j = 0; j < V; ++j) acc[i][j] = 0.f;
+#pragma unroll 4
+  for (int g = 0; g < H; ++g) {
+    float a[V];
+    ldv<V>(src + static_cast<long long>(g) * G * vo, a);
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const float f = quad + i < rep ? ld(m + i * H + g) : 0.f;
+#pragma unroll
+      for (int j = 0; j < V; ++j) acc[i][j] += f * a[j];
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+    if (quad + i < rep) stv<V>(out + (t * H + grp * rep + quad + i) * vo + c, acc[i]);
+}
+
 // CTA = (row, head), every warp walks every fourth visible position, a lane holds NR features of query, accumulator, key and
 // value; the four running softmaxes and the sink are merged at the end.
 struct GqaParams {
@@ -227,7 +450,11 @@ struct GqaParams {
   void* out;                // [rows][H][vo]
   int H, G, dp, vp, vo, max_blocks, block_size, ld_gate;
   int window;               // positions a row sees, its own included (0: all)
+  int keep;                 // with a window: the first positions that stay visible
+  int chunk;                // > 0: a row sees its own chunk of this many positions
+  int wide;                 // the head's weights meet the values of every group (blockIdx.z): out [rows][H][G][vo], no gate
   float scale;
+  float cap;                // > 0: scores s become cap tanh(s / cap)
 };
 template <typename T, int NR>
 __global__ void __launch_bounds__(128) gqa_attn_kernel(const GqaParams p) {
@@ -247,10 +474,13 @@ __global__ void __launch_bounds__(128) gqa_attn_kernel(const GqaParams p) {
     o[i] = 0.f;
   }
   float m = -INFINITY, l = 0.f;
-  for (int k = (p.window && n > p.window ? n - p.window : 0) + warp; k < n; k += 4) {
-    const long long at = (static_cast<long long>(bt[k / p.block_size]) * p.block_size + k % p.block_size) * p.G + g;
-    const T* kp = static_cast<const T*>(p.k_pool) + at * p.dp;
-    const T* vp = static_cast<const T*>(p.v_pool) + at * p.vp;
+  const int first = p.chunk ? (n - 1) / p.chunk * p.chunk : (p.window && n > p.window ? n - p.window : 0);
+  const int kept = min(p.keep, first);          // positions 0 .. kept - 1, then first .. n - 1
+  for (int i = warp; i < kept + n - first; i += 4) {
+    const int k = i < kept ? i : first + i - kept;
+    const long long row_at = (static_cast<long long>(bt[k / p.block_size]) * p.block_size + k % p.block_size) * p.G;
+    const T* kp = static_cast<const T*>(p.k_pool) + (row_at + g) * p.dp;
+    const T* vp = static_cast<const T*>(p.v_pool) + (row_at + (p.wide ? blockIdx.z : g)) * p.vp;
     float x[NR], s = 0.f;
 #pragma unroll
     for (int i = 0; i < NR; ++i) {
@@ -259,6 +489,7 @@ __global__ void __launch_bounds__(128) gqa_attn_kernel(const GqaParams p) {
       x[i] = c < p.vp ? ld(vp + c) : 0.f;
     }
     s = wsum(s) * p.scale;
+    if (p.cap > 0.f) s = p.cap * tanhf(s / p.cap);
     const float mn = fmaxf(m, s), a = expf(m - mn), e = expf(s - mn);
     m = mn;
     l = l * a + e;
@@ -280,7 +511,7 @@ __global__ void __launch_bounds__(128) gqa_attn_kernel(const GqaParams p) {
     L += w[k] * sml[k][1];
   }
   const float f = L > 0.f ? 1.f / L : 0.f;
-  T* out = static_cast<T*>(p.out) + (static_cast<long long>(row) * p.H + hd) * p.vo;
+  T* out = static_cast<T*>(p.out) + ((static_cast<long long>(row) * p.H + hd) * gridDim.z + blockIdx.z) * p.vo;
   const T* gate = p.gate ? static_cast<const T*>(p.gate) + static_cast<long long>(row) * p.ld_gate + hd * p.vo : nullptr;
   for (int c = threadIdx.x; c < p.vo; c += 128) {
     float o = (w[0] * sm[c] + w[1] * sm[p.vp + c] + w[2] * sm[2 * p.vp + c] + w[3] * sm[3 * p.vp + c]) * f;
@@ -302,10 +533,37 @@ static int launch_inputs(const InputParams& p, cudaStream_t stm) {
   return static_cast<int>(cudaGetLastError());
 }
 
+template <typename T, int NP, int NT>
+static int launch_conv_np(const ConvParams& p, bool pair, int segs, cudaStream_t stm) {
+  const int run = p.cu ? 8 : 1;
+  const long long units = static_cast<long long>((p.T + run - 1) / run) * (p.H + (p.k_pool ? 2 * p.G : 0));
+  const unsigned grid = static_cast<unsigned>((units + 7) / 8);
+  if (p.cu) {
+    if (pair) conv_inputs_kernel<T, NP, NT, 8, true><<<grid, 256, 0, stm>>>(p);
+    else conv_inputs_kernel<T, NP, NT, 8, false><<<grid, 256, 0, stm>>>(p);
+    if (p.n > 1) conv_state_kernel<T><<<dim3(segs, (p.C + 255) / 256), 256, 0, stm>>>(p);
+    rb_note_launch(p.n > 1 ? 2 : 1);
+  } else {
+    if (pair) conv_inputs_kernel<T, NP, NT, 1, true><<<grid, 256, 0, stm>>>(p);
+    else conv_inputs_kernel<T, NP, NT, 1, false><<<grid, 256, 0, stm>>>(p);
+    rb_note_launch(1);
+  }
+  return static_cast<int>(cudaGetLastError());
+}
+template <typename T, int NT>
+static int launch_conv(const ConvParams& p, bool pair, int segs, cudaStream_t stm) {
+  const int w = p.k_pool ? (p.dp > p.vp ? p.dp : p.vp) : p.dp;
+  if (w <= 64) return launch_conv_np<T, 1, NT>(p, pair, segs, stm);
+  if (w <= 128) return launch_conv_np<T, 2, NT>(p, pair, segs, stm);
+  if (w <= 256) return launch_conv_np<T, 4, NT>(p, pair, segs, stm);
+  if (w <= 512) return launch_conv_np<T, 8, NT>(p, pair, segs, stm);
+  return -2;
+}
+
 template <typename T>
 static int launch_gqa(const GqaParams& p, int rows, cudaStream_t stm) {
   const size_t smem = 4 * static_cast<size_t>(p.vp) * 4;
-  const dim3 grid(rows, p.H);
+  const dim3 grid(rows, p.H, p.wide ? p.G : 1);
   const int w = p.dp > p.vp ? p.dp : p.vp;
   if (w <= 64) gqa_attn_kernel<T, 2><<<grid, 128, smem, stm>>>(p);
   else if (w <= 128) gqa_attn_kernel<T, 4><<<grid, 128, smem, stm>>>(p);
@@ -369,11 +627,43 @@ extern "C" int rb_projection_inputs(const void* qkv, int ld, const void* q_w, co
   return static_cast<int>(cudaGetLastError());
 }
 
+// C = H dim (+ G (dim + vdim) with k_pool) channels; taps [C][n] (n up to 8) or null; state [slots][n - 1][C] (n > 1); cu, seg_of, pos: segments of any
+// length, or null: one row per segment.  q_w, k_w: weights of the norms (eps > 0)
+extern "C" int rb_conv_inputs(const void* qkv, int ld, const void* bias, const void* taps, int n, void* state, const void* q_w, const void* k_w,
+                              const float* table, void* q, void* k_pool, void* v_pool, const long long* slots, const int* ctx, const int* state_slot,
+                              const int* cu, const int* seg_of, const int* pos, long long pool_rows, int T, int segs, int H, int G, int dim, int vdim,
+                              int dp, int vp, int rot, float eps, int fp32, cudaStream_t stm) {
+  if (T <= 0) return 0;
+  if (H < 1 || dim < 1 || dp < dim || dp % 2 || rot % 2 || rot < 0 || rot > dim || (rot && !table) || n < 1 || n > 8 || (n > 1 && (!taps || !state))) return -2;
+  const int C = H * dim + (k_pool ? G * (dim + vdim) : 0);
+  if (ld < C || (k_pool && (!v_pool || !slots || G < 1 || vdim < 1 || vp < vdim || vp % 2)) || (cu && (!seg_of || !pos)) || !ctx || !state_slot) return -2;
+  if (eps > 0.f && (!q_w || (k_pool && !k_w))) return -2;
+  ConvParams p{qkv, bias, taps, state, q_w, k_w, reinterpret_cast<const float2*>(table), q, k_pool, v_pool, slots, ctx, state_slot, cu, seg_of, pos,
+               pool_rows, T, H, G, dim, vdim, dp, vp, rot, ld, n, C, eps};
+  const bool pair = dim % 2 == 0 && (!k_pool || vdim % 2 == 0) && ld % 2 == 0 && (reinterpret_cast<uintptr_t>(qkv) | reinterpret_cast<uintptr_t>(state)) % 8 == 0;
+  if (fp32) return n <= 4 ? launch_conv<float, 4>(p, pair, segs, stm) : launch_conv<float, 8>(p, pair, segs, stm);
+  return n <= 4 ? launch_conv<bf16, 4>(p, pair, segs, stm) : launch_conv<bf16, 8>(p, pair, segs, stm);
+}
+
+// wide [rows][H][G][vo], mix [H][H], out [rows][H][vo]
+extern "C" int rb_mix_heads(const void* wide, const void* mix, void* out, int rows, int H, int G, int vo, int fp32, cudaStream_t stm) {
+  if (rows <= 0) return 0;
+  if (G < 1 || H % G || vo % 8 || vo < 8) return -2;
+  const long long units = static_cast<long long>(rows) * G * ((H / G + 3) / 4) * (vo / 8);
+  const unsigned grid = static_cast<unsigned>((units + 127) / 128);
+  if (fp32) mix_heads_kernel<float, 8><<<grid, 128, 0, stm>>>((const float*)wide, (const float*)mix, (float*)out, units, H, G, vo);
+  else mix_heads_kernel<bf16, 8><<<grid, 128, 0, stm>>>((const bf16*)wide, (const bf16*)mix, (bf16*)out, units, H, G, vo);
+  rb_note_launch(1);
+  return static_cast<int>(cudaGetLastError());
+}
+
 extern "C" int rb_gqa_attn(const void* q, const void* k_pool, const void* v_pool, const int* block_tables, const int* row_seg, const int* row_pos,
                            const int* ctx, const void* sink, const void* gate, int ld_gate, void* out, int rows, int H, int G, int dp, int vp, int vo,
-                           int max_blocks, int block_size, int window, float scale, int fp32, cudaStream_t stm) {
+                           int max_blocks, int block_size, int window, int keep, int chunk, int wide, float scale, float cap, int fp32,
+                           cudaStream_t stm) {
   if (rows <= 0) return 0;
-  if (G < 1 || H % G || vo > vp || H > 65535 || window < 0 || (gate && ld_gate < H * vo)) return -2;
-  GqaParams p{q, k_pool, v_pool, block_tables, row_seg, row_pos, ctx, sink, gate, out, H, G, dp, vp, vo, max_blocks, block_size, ld_gate, window, scale};
+  if (G < 1 || G > 65535 || H % G || vo > vp || H > 65535 || window < 0 || keep < 0 || chunk < 0 || (gate && (wide || ld_gate < H * vo))) return -2;
+  GqaParams p{q, k_pool, v_pool, block_tables, row_seg, row_pos, ctx, sink, gate, out, H, G, dp, vp, vo, max_blocks, block_size, ld_gate, window, keep,
+              chunk, wide, scale, cap};
   return fp32 ? launch_gqa<float>(p, rows, stm) : launch_gqa<bf16>(p, rows, stm);
 }

@@ -16,6 +16,8 @@
 // q~, S and a (17 bits).  CTA = (segment, head), all value columns: gates and a_ts are computed once, half of the warps
 // build the products along time while the other half builds a_ts, and the per-head norm is applied before the output is
 // written.
+// The same kernel serves linear attention whose rows decay by gates of their own (kGla): k and q are projections, the gates
+// g = sigmoid(z) ^ r come from an fp32 projection, and the normed output is multiplied by silu of a gate per feature.
 #include "common.cuh"
 #include "host_utils.h"
 
@@ -43,6 +45,10 @@ struct Params {
   float* span_gate;              // [n][H][dim]
   int H, dim, vdim, vp, ld, ldo;
   float eps;
+  // kGla: qfv is q (H*dim) | k (H*dim) | v (H*vdim) and, from column gate_col on, output gates (H*vdim); f_bias joins z
+  const float* z;                // [T][ldz]
+  int ldz, gate_col;
+  float q_scale, inv_root;
 };
 
 __device__ __forceinline__ void mma_bf16(float* c, const uint32_t* a, uint32_t b0, uint32_t b1) {
@@ -101,7 +107,7 @@ __device__ __forceinline__ void copy16(void* dst, const void* src, bool in) {
 }
 __device__ __forceinline__ void copies_landed() { asm volatile("cp.async.wait_all;" ::: "memory"); }
 
-template <int DK, int NW>
+template <int DK, int NW, bool kGla>
 struct Smem {
   static constexpr int GP = DK + 4;                  // fp32 row pitch
   static constexpr int DP = DK + 8;                  // bf16 row pitch of the products (conflict-free ldmatrix)
@@ -114,13 +120,16 @@ struct Smem {
   __nv_bfloat16 ah[CH][24], al[CH][24];              // a_ts
   __nv_bfloat16 v[CH][VP], o[CH][VP];
   __nv_bfloat16 rq[CH][DK], rf[CH][DK], rv[CH][NW * 16];   // raw projections on their way in
+  float rz[kGla ? CH : 1][DK];
+  __nv_bfloat16 rg[kGla ? CH : 1][NW * 16];
 };
 
-template <int DK, int NW, int kMode>
+template <int DK, int NW, int kMode, bool kGla>
 __global__ void __launch_bounds__(NW * 32, NW == 8 ? 2 : 3) hgrn2_chunk_kernel(const Params p) {
   constexpr int NT = NW * 32, UQ = (2 * DK + NT - 1) / NT, TILES = DK / 8;
   extern __shared__ __align__(16) uint8_t raw_smem[];
-  Smem<DK, NW>& sm = *reinterpret_cast<Smem<DK, NW>*>(raw_smem);
+  using S_ = Smem<DK, NW, kGla>;
+  S_& sm = *reinterpret_cast<S_*>(raw_smem);
   const int seg = blockIdx.x, hd = blockIdx.y;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int lo = kMode == kWhole ? p.cu[seg] : p.spans[2 * seg], hi = kMode == kWhole ? p.cu[seg + 1] : p.spans[2 * seg + 1];
@@ -155,15 +164,22 @@ __global__ void __launch_bounds__(NW * 32, NW == 8 ? 2 : 3) hgrn2_chunk_kernel(c
         const __nv_bfloat16* a = in ? p.qfv + static_cast<long long>(t0 + t) * p.ld + hd * p.dim + d : p.qfv;
         if (kMode != kStates) copy16(&sm.rq[t][d], a, in);
         copy16(&sm.rf[t][d], in ? a + qd : a, in);
+        if constexpr (kGla) {
+          const float* z = in ? p.z + static_cast<long long>(t0 + t) * p.ldz + hd * p.dim + d : p.z;
+          copy16(&sm.rz[t][d], z, in);
+          copy16(&sm.rz[t][d + 4], in ? z + 4 : z, in);
+        }
       }
     }
     const int t = tid / (NW * 2), c = (tid % (NW * 2)) * 8;
     const bool in = t0 + t < hi && c < p.vdim;
     copy16(&sm.rv[t][c], in ? p.qfv + static_cast<long long>(t0 + t) * p.ld + 2 * qd + hd * p.vdim + c : p.qfv, in);
+    if constexpr (kGla && kMode != kStates)
+      copy16(&sm.rg[t][c], in ? p.qfv + static_cast<long long>(t0 + t) * p.ld + p.gate_col + hd * p.vdim + c : p.qfv, in);
   };
   for (int d = tid; d < DK; d += NT) {      // padding channels: gate 1, nothing is written
     sm.fb[d] = d < p.dim ? __bfloat162float(p.f_bias[hd * p.dim + d]) : 0.f;
-    sm.fl[d] = d < p.dim ? __bfloat162float(p.lower[hd * p.dim + d]) : 1.f;
+    if constexpr (!kGla) sm.fl[d] = d < p.dim ? __bfloat162float(p.lower[hd * p.dim + d]) : 1.f;
   }
   __syncthreads();
   float gate0 = 1.f, gate1 = 1.f;             // kStates: product of the span's gates (threads DK / 2 .. DK - 1)
@@ -184,6 +200,16 @@ __global__ void __launch_bounds__(NW * 32, NW == 8 ? 2 : 3) hgrn2_chunk_kernel(c
 #pragma unroll
         for (int c = 0; c < 8; ++c) {
           const float x = (c & 1) ? hi16(wq[c >> 1]) : lo16(wq[c >> 1]);
+          if constexpr (kGla) {      // tokens and channels behind the last one: gate 1, k = 0
+            const float z = sm.rz[t][dpre + c] + sm.fb[dpre + c], e = __expf(-fabsf(z));
+            // log(1 + e) of small e keeps its leading digits
+            const float l = fminf(z, 0.f) - (e < 1e-3f ? e * (1.f - 0.5f * e) : __logf(1.f + e));
+            const bool in = t < n && dpre + c < p.dim;
+            g[c] = in ? __expf(l * p.inv_root) : 1.f;
+            k[c] = in ? ((c & 1) ? hi16(wf[c >> 1]) : lo16(wf[c >> 1])) : 0.f;
+            q[c] = x * p.q_scale;
+            continue;
+          }
           const float f = ((c & 1) ? hi16(wf[c >> 1]) : lo16(wf[c >> 1])) + sm.fb[dpre + c];
           // one exponential of -|f| gives both halves of the gate without overflow or cancellation
           // (and likewise for silu; the two denominators lie in [1, 2] and share one reciprocal)
@@ -203,6 +229,8 @@ __global__ void __launch_bounds__(NW * 32, NW == 8 ? 2 : 3) hgrn2_chunk_kernel(c
       }
     }
     *reinterpret_cast<uint4*>(&sm.v[tid / (NW * 2)][(tid % (NW * 2)) * 8]) = *reinterpret_cast<const uint4*>(&sm.rv[tid / (NW * 2)][(tid % (NW * 2)) * 8]);
+    uint4 out_gate = make_uint4(0, 0, 0, 0);      // of the eight output columns that this thread stores
+    if constexpr (kGla && kMode != kStates) out_gate = *reinterpret_cast<const uint4*>(&sm.rg[tid / (NW * 2)][(tid % (NW * 2)) * 8]);
     __syncthreads();
     if (t0 + CH < hi) fetch(t0 + CH);
     // ---------------------------------------------------------------- products along time: one thread per channel pair
@@ -400,8 +428,19 @@ __global__ void __launch_bounds__(NW * 32, NW == 8 ? 2 : 3) hgrn2_chunk_kernel(c
     __syncthreads();
     {
       const int t = tid / (NW * 2), c = (tid % (NW * 2)) * 8;
-      if (t < n && c < p.vdim)
-        *reinterpret_cast<uint4*>(p.out + static_cast<long long>(t0 + t) * p.ldo + hd * p.vdim + c) = *reinterpret_cast<const uint4*>(&sm.o[t][c]);
+      if (t < n && c < p.vdim) {
+        uint4 o = *reinterpret_cast<const uint4*>(&sm.o[t][c]);
+        if constexpr (kGla) {
+          uint32_t* w = reinterpret_cast<uint32_t*>(&o);
+          const uint32_t gw[4] = {out_gate.x, out_gate.y, out_gate.z, out_gate.w};
+#pragma unroll
+          for (int i = 0; i < 4; ++i) {
+            const float a = lo16(gw[i]), b = hi16(gw[i]);
+            w[i] = pack_bf16(lo16(w[i]) * __fdividef(a, 1.f + __expf(-a)), hi16(w[i]) * __fdividef(b, 1.f + __expf(-b)));
+          }
+        }
+        *reinterpret_cast<uint4*>(p.out + static_cast<long long>(t0 + t) * p.ldo + hd * p.vdim + c) = o;
+      }
     }
     }
   }
@@ -446,10 +485,10 @@ __global__ void __launch_bounds__(256) span_scan_kernel(const Params p, const in
   *S = s;
 }
 
-template <int DK, int NW, int kMode>
+template <int DK, int NW, int kMode, bool kGla>
 static int launch_mode(const Params& p, int n, cudaStream_t st) {
-  auto k = hgrn2_chunk_kernel<DK, NW, kMode>;
-  const int smem = static_cast<int>(sizeof(Smem<DK, NW>));
+  auto k = hgrn2_chunk_kernel<DK, NW, kMode, kGla>;
+  const int smem = static_cast<int>(sizeof(Smem<DK, NW, kGla>));
   static bool attr = false;
   if (!attr) {
     const cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
@@ -460,14 +499,20 @@ static int launch_mode(const Params& p, int n, cudaStream_t st) {
   rb_note_launch(1);
   return static_cast<int>(cudaGetLastError());
 }
-template <int DK, int NW>
+template <int DK, int NW, bool kGla>
 static int launch(const Params& p, int segs, int spans, const int* first, cudaStream_t st) {
-  if (!spans) return launch_mode<DK, NW, kWhole>(p, segs, st);
-  int rc = launch_mode<DK, NW, kStates>(p, spans, st);
+  if (!spans) return launch_mode<DK, NW, kWhole, kGla>(p, segs, st);
+  int rc = launch_mode<DK, NW, kStates, kGla>(p, spans, st);
   if (rc) return rc;
   span_scan_kernel<<<dim3(segs, p.H, (p.dim * (p.vp / 4) + 255) / 256), 256, 0, st>>>(p, first);
   rb_note_launch(1);
-  return launch_mode<DK, NW, kFromScratch>(p, spans, st);
+  return launch_mode<DK, NW, kFromScratch, kGla>(p, spans, st);
+}
+
+template <bool kGla>
+static int dispatch(const Params& p, int segs, int n_spans, const int* first, cudaStream_t st) {
+  if (p.dim <= 64) return p.vdim <= 64 ? launch<64, 4, kGla>(p, segs, n_spans, first, st) : launch<64, 8, kGla>(p, segs, n_spans, first, st);
+  return p.vdim <= 64 ? launch<128, 4, kGla>(p, segs, n_spans, first, st) : launch<128, 8, kGla>(p, segs, n_spans, first, st);
 }
 
 }  // namespace hc
@@ -488,6 +533,21 @@ extern "C" int rb_hgrn2_chunk(const void* qfv, const void* f_bias, const void* l
   Params p{static_cast<const __nv_bfloat16*>(qfv), static_cast<const __nv_bfloat16*>(f_bias), static_cast<const __nv_bfloat16*>(lower),
            static_cast<const __nv_bfloat16*>(norm_w), state, slot, ctx, cu, static_cast<__nv_bfloat16*>(out), spans, span_state, span_gate,
            H, dim, vdim, vp, ld, ldo, eps};
-  if (dim <= 64) return vdim <= 64 ? launch<64, 4>(p, segs, n_spans, first, st) : launch<64, 8>(p, segs, n_spans, first, st);
-  return vdim <= 64 ? launch<128, 4>(p, segs, n_spans, first, st) : launch<128, 8>(p, segs, n_spans, first, st);
+  return dispatch<false>(p, segs, n_spans, first, st);
+}
+
+// The same for linear attention with decaying rows: in [T][ld] is q | k | v and, from gate_col on, output gates; z [T][ldz] fp32.
+extern "C" int rb_gla_chunk(const void* in, const float* z, int ldz, const void* z_bias, const void* norm_w, float* state, const int* slot, const int* ctx,
+                            const int* cu, const int* spans, const int* first, float* span_state, float* span_gate, void* out, int rows, int segs,
+                            int n_spans, int H, int dim, int vdim, int vp, int ld, int ldo, int gate_col, float eps, float q_scale, float inv_root,
+                            cudaStream_t st) {
+  using namespace rb;
+  using namespace rb::hc;
+  if (rows <= 0 || segs <= 0) return 0;
+  if (dim % 8 || vdim % 8 || dim > 128 || vdim > 128 || ld % 8 || ldo != H * vdim || vp < vdim || vp % 4 || H > 65535 || ldz % 4 || gate_col % 8) return -20;
+  if ((reinterpret_cast<uintptr_t>(in) | reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(z)) % 16) return -20;
+  if (n_spans && (!spans || !first || !span_state || !span_gate)) return -2;
+  Params p{static_cast<const __nv_bfloat16*>(in), static_cast<const __nv_bfloat16*>(z_bias), nullptr, static_cast<const __nv_bfloat16*>(norm_w), state, slot,
+           ctx, cu, static_cast<__nv_bfloat16*>(out), spans, span_state, span_gate, H, dim, vdim, vp, ld, ldo, eps, z, ldz, gate_col, q_scale, inv_root};
+  return dispatch<true>(p, segs, n_spans, first, st);
 }

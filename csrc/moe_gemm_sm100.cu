@@ -41,7 +41,7 @@ struct Params {
   const int* n_tiles;        // device counter
   const int* row_token;      // [E][capacity] token of an expert's rows; null: the sorted rows themselves
   int capacity, cap, N, K, act;
-  float limit;               // act 2 (gated): g = min(gate, limit), u = unit clamped to +- limit, g sigmoid(1.702 g) (u + 1)
+  float limit;               // act 2 (gated): g = min(gate, limit), u = unit clamped to +- limit, g sigmoid(1.702 g) (u + 1); act 3: silu(gate) unit
   const __nv_bfloat16* x;    // [x_rows][K] (kCopy)
   __nv_bfloat16* out;        // [sorted rows][N], act 2: [N / 2]
   int* err;
@@ -217,7 +217,7 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constant
       const bool live = row < tile.z;
       if (grp * 32 < tile.z) {
         const uint32_t taddr = tmem_base + acc * BN + (static_cast<uint32_t>(grp * 32) << 16);
-        const bool gated = p.act == 2;
+        const bool gated = p.act >= 2;
         const int shift = gated ? 1 : 0, step = 1 + shift;
         __nv_bfloat16* out = p.out + static_cast<size_t>(tile.y + row) * (p.N >> shift) + (n0 >> shift);
 #pragma unroll 1
@@ -229,10 +229,18 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constant
             uint32_t v[32];
             tmem_ld_32x32b_x32(taddr + c * 32 + 32, v);
             tmem_wait_ld();
+            if (p.act == 3) {
+#pragma unroll
+              for (int i = 0; i < 32; ++i) {
+                const float g = __uint_as_float(r[i]);
+                r[i] = __float_as_uint(__fdividef(g, 1.f + __expf(-g)) * __uint_as_float(v[i]));
+              }
+            } else {
 #pragma unroll
             for (int i = 0; i < 32; ++i) {
               const float g = fminf(__uint_as_float(r[i]), p.limit), u = fminf(fmaxf(__uint_as_float(v[i]), -p.limit), p.limit);
               r[i] = __float_as_uint(__fdividef(g, 1.f + __expf(-1.702f * g)) * (u + 1.f));
+            }
             }
           } else {
             tmem_wait_ld();
@@ -299,14 +307,14 @@ static int launch(const void* X, int x_rows, const void* W, int E, const Params&
 }  // namespace rb
 
 // X [x_rows][K] (token rows with row_token [E][capacity], else sorted rows), W [E][N][K] -> out [sorted rows][N]; tiles hold at most
-// `cap` entries.  act: 0 none, 1 squared relu, 2 gated (see Params::limit; out [sorted rows][N / 2]).  bn: 128 or 256 columns per tile.  full: most tiles have many rows (choice of the
+// `cap` entries.  act: 0 none, 1 squared relu, 2 and 3 gated (see Params::limit; out [sorted rows][N / 2]).  bn: 128 or 256 columns per tile.  full: most tiles have many rows (choice of the
 // gather only).  N and K are multiples of 64.
 extern "C" int rb_moe_gemm(const void* X, const void* W, void* out, const int* tiles, const int* n_tiles, const int* row_token, int x_rows,
                            int capacity, int cap, int E, int N, int K, int act, float limit, int bn, int full, int* err, cudaStream_t st) {
   using namespace rb;
   using namespace rb::mg;
   if (x_rows <= 0 || cap <= 0) return 0;
-  if (E < 1 || N < 64 || K < 64 || N % 64 || K % 64 || act < 0 || act > 2 || (act == 2 && N % 128) || reinterpret_cast<uintptr_t>(X) % 16) return -2;
+  if (E < 1 || N < 64 || K < 64 || N % 64 || K % 64 || act < 0 || act > 3 || (act >= 2 && N % 128) || reinterpret_cast<uintptr_t>(X) % 16) return -2;
   Params p{reinterpret_cast<const int4*>(tiles), n_tiles, row_token, capacity, cap, N, K, act, limit, (const __nv_bfloat16*)X, (__nv_bfloat16*)out, err};
   if (row_token && full) return bn == 256 ? launch<256, kCopy>(X, x_rows, W, E, p, st) : launch<128, kCopy>(X, x_rows, W, E, p, st);
   if (row_token) return bn == 256 ? launch<256, kGather4>(X, x_rows, W, E, p, st) : launch<128, kGather4>(X, x_rows, W, E, p, st);

@@ -187,7 +187,7 @@ __global__ void relu2_kernel(T* __restrict__ x, long long n8) {
 }
 
 // C[sorted row] = act(A[token or sorted row] * B[expert]^T); one tile of the list (up to 64 rows) x 64 columns per CTA.  act 0: none,
-// 1: squared relu, 2: gated (columns of B alternate between 32 gates and the 32 units they belong to; C has half as many)
+// 1: squared relu, 2 and 3: gated (columns of B alternate between 32 gates and the 32 units they belong to; C has half as many)
 struct MoeSimtParams {
   const void* A;
   const void* B;             // [E][N][K]
@@ -196,7 +196,7 @@ struct MoeSimtParams {
   const int* n_tiles;
   const int* row_token;      // [E][capacity] or null
   int capacity, cap, N, K, act;
-  float limit;               // act 2: g = min(gate, limit), u = unit clamped to +- limit, g sigmoid(1.702 g) (u + 1)
+  float limit;               // act 2: g = min(gate, limit), u = unit clamped to +- limit, g sigmoid(1.702 g) (u + 1); act 3: silu(gate) unit
 };
 template <typename T>
 __global__ void __launch_bounds__(256) moe_simt_kernel(const MoeSimtParams p) {
@@ -235,14 +235,20 @@ __global__ void __launch_bounds__(256) moe_simt_kernel(const MoeSimtParams p) {
     __syncthreads();
   }
   T* C = static_cast<T*>(p.C);
-  if (p.act == 2) {
+  if (p.act >= 2) {
 #pragma unroll
     for (int i = 0; i < 4; ++i)
 #pragma unroll
       for (int j = 0; j < 4; ++j) {      // the thread eight lanes on holds the units of this thread's gates
-        const float u = fminf(fmaxf(__shfl_down_sync(0xffffffffu, acc[i][j], 8), -p.limit), p.limit), g = fminf(acc[i][j], p.limit);
-        if (tn < 32 && tm + i < tile.z)
-          st(C + static_cast<long long>(tile.y + tm + i) * (p.N >> 1) + (n0 >> 1) + tn + j, g * sigmoid<true>(1.702f * g) * (u + 1.f));
+        float u = __shfl_down_sync(0xffffffffu, acc[i][j], 8), g = acc[i][j];
+        if (p.act == 2) {
+          u = fminf(fmaxf(u, -p.limit), p.limit) + 1.f;
+          g = fminf(g, p.limit);
+          g *= sigmoid<true>(1.702f * g);
+        } else {
+          g *= sigmoid<true>(g);
+        }
+        if (tn < 32 && tm + i < tile.z) st(C + static_cast<long long>(tile.y + tm + i) * (p.N >> 1) + (n0 >> 1) + tn + j, g * u);
       }
     return;
   }
@@ -304,7 +310,7 @@ extern "C" int rb_relu2(void* x, long long n, int fp32, cudaStream_t stm) {
 extern "C" int rb_moe_simt(const void* A, const void* B, void* C, const int* tiles, const int* n_tiles, const int* row_token, int capacity, int cap,
                            int N, int K, int act, float limit, int fp32, cudaStream_t stm) {
   if (cap <= 0) return 0;
-  if (cap > 65535 || N < 1 || K < 1 || act < 0 || act > 2 || (act == 2 && N % 64)) return -2;
+  if (cap > 65535 || N < 1 || K < 1 || act < 0 || act > 3 || (act >= 2 && N % 64)) return -2;
   MoeSimtParams p{A, B, C, reinterpret_cast<const int4*>(tiles), n_tiles, row_token, capacity, cap, N, K, act, limit};
   const dim3 grid((N + 63) / 64, cap);
   if (fp32) moe_simt_kernel<float><<<grid, 256, 0, stm>>>(p);

@@ -13,7 +13,9 @@
 // reads behind them is zero.  The running softmax starts from the head's sink logit
 // (sum = 1 at reference = sink), or empty without one.  With a window a tile starts at the block of the first position that its first
 // row sees, and every row masks what lies before its own.  A gate per output feature is applied in the epilogue.  S is double buffered, so the product of block j + 1 runs while the
-// softmax of block j does.  The accumulator is rescaled only when a row's maximum grows by more than 2^8 (decided per warp: TMEM
+// softmax of block j does.  Positions at a sequence's start may stay visible outside a window (their blocks come first), rows may see
+// only their own chunk of positions, scores may be capped, and a head's weights may meet the values of every group (one group per
+// blockIdx.z), for heads whose weights are mixed afterwards.  The accumulator is rescaled only when a row's maximum grows by more than 2^8 (decided per warp: TMEM
 // accesses are warp-wide).  Warps 0-3: softmax and epilogue, warp 4: TMA, warp 5: MMA.  Two CTAs share an SM; keys of more than 128
 // columns leave room for one stage of keys and values instead of two.  Every wait is bounded; no load uses cluster multicast.
 #include <limits.h>
@@ -56,9 +58,17 @@ struct Params {
   __nv_bfloat16* out;        // [rows][H][out_d]
   int H, G, tokens, max_blocks, page, out_d, ld_gate;
   int window;                // positions a row sees (INT_MAX: all)
-  float scale_log2;
+  int keep;                  // first positions that stay visible outside the window
+  int chunk;                 // > 0: a row sees its own chunk of this many positions
+  float scale_log2;          // kCap: 1, scores come out of the cap in log2 units
+  float cap_in, cap_log2;    // kCap: s <- cap_log2 tanh(cap_in q . k)
   int* err;
 };
+
+// tanh in fp32 up to about 1e-7
+__device__ __forceinline__ float bounded(float x) {
+  return 1.f - __fdividef(2.f, 1.f + exp2f(2.8853900817779268f * fminf(x, 20.f)));      // 2 / ln 2
+}
 
 // eight accumulators times sigmoid(gate)
 __device__ __forceinline__ void gate8(uint32_t* o, const uint4& g) {
@@ -70,7 +80,7 @@ __device__ __forceinline__ void gate8(uint32_t* o, const uint4& g) {
   }
 }
 
-template <int DK, int DV>
+template <int DK, int DV, bool kCap>
 __global__ void __launch_bounds__(THREADS, 2)
 paged_flash_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant__ CUtensorMap tma_k,
                    const __grid_constant__ CUtensorMap tma_v, const Params p) {
@@ -89,7 +99,7 @@ paged_flash_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_const
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int kvh = blockIdx.y;
+  const int kvh = blockIdx.y, vh = gridDim.z > 1 ? blockIdx.z : blockIdx.y;      // group of the keys, and of the values
   int seg, row0, ntok, pos0;
   if (p.blocks) {
     const int4 b = reinterpret_cast<const int4*>(p.blocks)[blockIdx.x];
@@ -100,8 +110,11 @@ paged_flash_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_const
     pos0 = p.ctx[seg] - 1;
   }
   const int seen = pos0 + ntok;                    // positions that the last token of the tile sees
-  const int block0 = max(0, pos0 - p.window + 1) / BKV;      // block of the first position that the first token sees
-  const int n_blocks = (seen + BKV - 1) / BKV - block0;
+  // block of the first position that the first token sees, kept ones aside; the blocks of kept positions in front of it come first
+  const int block0 = (p.chunk ? pos0 / p.chunk * p.chunk : max(0, pos0 - p.window + 1)) / BKV;
+  const int n_kept = min((p.keep + BKV - 1) / BKV, block0);
+  const int n_blocks = n_kept + (seen + BKV - 1) / BKV - block0;
+  auto block_at = [&](int j) { return j < n_kept ? j : block0 + j - n_kept; };
   const int base = p.first_row ? p.first_row[seg] : -1;
   const int* bt = p.block_tables + static_cast<size_t>(p.first_row ? 0 : seg) * p.max_blocks;
   constexpr int ST = L::kStages;
@@ -152,15 +165,15 @@ paged_flash_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_const
         uint8_t* sk = smem + L::kK + s * L::kKBytes;
         mbar_expect_tx(&kfull[s], L::kKBytes);
         for (int r = 0; r < BKV; r += rows) {
-          const int row = pool_row((block0 + j) * BKV + r);
+          const int row = pool_row(block_at(j) * BKV + r);
           for (int c = 0; c < DK / 64; ++c) tma_load_3d(sk + c * L::kKVHalf + r * 128, &tma_k, &kfull[s], c * 64, kvh, row);
         }
         if (!mbar_wait(&vempty[s], ph, abort_flag, p.err)) break;
         uint8_t* sv = smem + L::kV + s * L::kVBytes;
         mbar_expect_tx(&vfull[s], L::kVBytes);
         for (int r = 0; r < BKV; r += rows) {
-          const int row = pool_row((block0 + j) * BKV + r);
-          for (int c = 0; c < DV / 64; ++c) tma_load_3d(sv + c * L::kKVHalf + r * 128, &tma_v, &vfull[s], c * 64, kvh, row);
+          const int row = pool_row(block_at(j) * BKV + r);
+          for (int c = 0; c < DV / 64; ++c) tma_load_3d(sv + c * L::kKVHalf + r * 128, &tma_v, &vfull[s], c * 64, vh, row);
         }
       }
     }
@@ -210,8 +223,8 @@ paged_flash_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_const
     // ================================================================ softmax + epilogue (warps 0..3)
     const int r = warp * 32 + lane;                // row of the tile = TMEM lane
     const int t = r / p.G, head = kvh * p.G + r % p.G;
-    const int limit = pos0 + t + 1 - block0 * BKV;             // this row sees positions first .. limit - 1 of the tile's blocks
-    const int first = limit - min(p.window, pos0 + t + 1);
+    const int limit = pos0 + t + 1;                // this row sees positions first .. limit - 1, and those in front of p.keep
+    const int first = p.chunk ? (pos0 + t) / p.chunk * p.chunk : limit - min(p.window, limit);
     const bool mine = t < ntok;
     const uint32_t lane_addr = static_cast<uint32_t>(warp * 32) << 16;
     float m_ref = -1e30f, l = 0.f;
@@ -230,15 +243,20 @@ paged_flash_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_const
       tmem_ld_32x32b_x32(tmem_base + T_S + s * BKV + lane_addr, raw);
       tmem_ld_32x32b_x32(tmem_base + T_S + s * BKV + lane_addr + 32, raw + 32);
       tmem_wait_ld();
-      const int lim = limit - j * BKV, low = first - j * BKV;      // columns low .. lim - 1 are seen
+      if constexpr (kCap) {
+#pragma unroll
+        for (int c = 0; c < 64; ++c) raw[c] = __float_as_uint(p.cap_log2 * bounded(p.cap_in * __uint_as_float(raw[c])));
+      }
+      const int at = block_at(j) * BKV;
+      const int lim = limit - at, low = first - at, kept = p.keep - at;      // columns low .. lim - 1 are seen, and those in front of `kept`
       float mx = -1e30f;
-      if (__all_sync(0xffffffffu, lim >= BKV && low <= 0)) {
+      if (__all_sync(0xffffffffu, lim >= BKV && (low <= 0 || kept >= BKV))) {
 #pragma unroll
         for (int c = 0; c < 64; ++c) mx = fmaxf(mx, __uint_as_float(raw[c]));
       } else {
 #pragma unroll
         for (int c = 0; c < 64; ++c) {
-          if (c >= lim || c < low) raw[c] = 0xff800000u;      // -inf
+          if (c >= lim || (c < low && c >= kept)) raw[c] = 0xff800000u;      // -inf
           mx = fmaxf(mx, __uint_as_float(raw[c]));
         }
       }
@@ -305,7 +323,7 @@ paged_flash_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_const
     float inv_l = l > 0.f ? 1.f / l : 0.f;
     if (p.gate && p.head_gate && mine)
       inv_l = __fdividef(inv_l, 1.f + __expf(-__bfloat162float(p.gate[static_cast<size_t>(row0 + t) * p.ld_gate + head])));
-    __nv_bfloat16* out = p.out + (static_cast<size_t>(row0 + t) * p.H + head) * p.out_d;
+    __nv_bfloat16* out = p.out + ((static_cast<size_t>(row0 + t) * p.H + head) * gridDim.z + blockIdx.z) * p.out_d;
     if (all_ok) {
 #pragma unroll 1
       for (int c = 0; c < DV / 32; ++c) {
@@ -351,9 +369,10 @@ struct Operands {      // widths dk, dv <= DK, DV; q_pitch: elements between two
   int rows, n, Hkv, dk, dv;
   long long q_pitch;
   uint64_t pool_rows;
+  bool wide;                // every head's weights meet the values of every group
 };
 
-template <int DK, int DV>
+template <int DK, int DV, bool kCap>
 static int launch(const Operands& o, const Params& p, cudaStream_t st) {
   using L = Tile<DK, DV>;
   CUtensorMap tq, tk, tv;
@@ -364,23 +383,27 @@ static int launch(const Operands& o, const Params& p, cudaStream_t st) {
   if (rc) return rc;
   rc = encode_tma_3d_16bit(&tv, o.v, o.dv, o.Hkv, o.pool_rows, o.dv, static_cast<uint64_t>(o.Hkv) * o.dv, 64, 1, box);
   if (rc) return rc;
-  auto kern = paged_flash_kernel<DK, DV>;
+  auto kern = paged_flash_kernel<DK, DV, kCap>;
   static bool attr_set = false;
   if (!attr_set) {
     const cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, L::kTotal);
     if (e != cudaSuccess) return static_cast<int>(e);
     attr_set = true;
   }
-  kern<<<dim3(o.n, o.Hkv), THREADS, L::kTotal, st>>>(tq, tk, tv, p);
+  kern<<<dim3(o.n, o.Hkv, o.wide ? o.Hkv : 1), THREADS, L::kTotal, st>>>(tq, tk, tv, p);
   rb_note_launch(1);
   return static_cast<int>(cudaGetLastError());
 }
 
+template <bool kCap>
 static int dispatch(const Operands& o, const Params& p, cudaStream_t st) {
   const bool wide = o.dv > 64;
-  if (o.dk > 128) return wide ? launch<192, 128>(o, p, st) : launch<192, 64>(o, p, st);
-  if (o.dk > 64) return wide ? launch<128, 128>(o, p, st) : launch<128, 64>(o, p, st);
-  return wide ? launch<64, 128>(o, p, st) : launch<64, 64>(o, p, st);
+  if (o.dk > 128) {
+    if constexpr (kCap) return -20;
+    else return wide ? launch<192, 128, kCap>(o, p, st) : launch<192, 64, kCap>(o, p, st);
+  }
+  if (o.dk > 64) return wide ? launch<128, 128, kCap>(o, p, st) : launch<128, 64, kCap>(o, p, st);
+  return wide ? launch<64, 128, kCap>(o, p, st) : launch<64, 64, kCap>(o, p, st);
 }
 
 }  // namespace pf
@@ -388,14 +411,17 @@ static int dispatch(const Operands& o, const Params& p, cudaStream_t st) {
 
 // q [rows][Hq][dk], pools [pool_rows][Hkv][dk / dv] (dk, dv: 64 or 128, dk also 192), out [rows][Hq][out_d].  blocks [n][4]: query tiles of at
 // most 128 / (Hq / Hkv) tokens, every row in exactly one (null: n = rows, one row per segment).  window: positions a row sees, its own
-// included (0: all).  gate [rows][ld_gate] or null.  Returns -20 for shapes outside that.
+// included (0: all), besides the first `keep` of the sequence; chunk > 0: only its own chunk of that many positions; cap > 0: scores s become
+// cap tanh(s / cap); wide: every head's weights meet the values of every group, out [rows][Hq][Hkv][out_d], no gate.  gate [rows][ld_gate] or
+// null.  Returns -20 for shapes outside that.
 extern "C" int rb_paged_flash(const void* q, const void* kc, const void* vc, const int* block_tables, const int* ctx, const int* blocks,
                               const void* sink, const void* gate, int ld_gate, void* out, int rows, int n, int Hq, int Hkv, int dk, int dv, int out_d,
-                              long long pool_rows, int page, int max_blocks, int window, float scale, int* err, cudaStream_t st) {
+                              long long pool_rows, int page, int max_blocks, int window, int keep, int chunk, int wide, float scale, float cap, int* err,
+                              cudaStream_t st) {
   using namespace rb;
   using namespace rb::pf;
   if (rows <= 0 || n <= 0) return 0;
-  if (Hkv < 1 || Hq % Hkv) return -2;
+  if (Hkv < 1 || Hq % Hkv || keep < 0 || chunk < 0 || cap < 0.f || (wide && gate) || (keep && !window) || (chunk && window)) return -2;
   const int G = Hq / Hkv;
   if (G > BQ || Hkv > 65535 || dk % 64 || dk < 64 || dk > 192 || (dv != 64 && dv != 128) || out_d % 8 || out_d > dv || out_d < 1) return -20;
   if ((page != 16 && page != 32 && page % 64) || scale <= 0.f) return -20;
@@ -404,9 +430,15 @@ extern "C" int rb_paged_flash(const void* q, const void* kc, const void* vc, con
   p.blocks = blocks; p.ctx = ctx; p.block_tables = block_tables; p.sink = (const __nv_bfloat16*)sink; p.out = (__nv_bfloat16*)out;
   p.gate = (const __nv_bfloat16*)gate; p.ld_gate = ld_gate; p.window = window ? window : INT_MAX;
   p.H = Hq; p.G = G; p.tokens = BQ / G; p.max_blocks = max_blocks; p.page = page; p.out_d = out_d;
+  p.keep = keep; p.chunk = chunk;
   p.scale_log2 = scale * 1.4426950408889634f;
   p.err = err;
-  return dispatch({q, kc, vc, rows, n, Hkv, dk, dv, static_cast<long long>(Hq) * dk, static_cast<uint64_t>(pool_rows)}, p, st);
+  const Operands o{q, kc, vc, rows, n, Hkv, dk, dv, static_cast<long long>(Hq) * dk, static_cast<uint64_t>(pool_rows), wide != 0};
+  if (cap <= 0.f) return dispatch<false>(o, p, st);
+  p.scale_log2 = 1.f;
+  p.cap_in = scale / cap;
+  p.cap_log2 = cap * 1.4426950408889634f;
+  return dispatch<true>(o, p, st);
 }
 
 // The same without pages: segment s has its keys and values [rows][H][dk / dv] (dk up to 192, dv up to 128, multiples of 8) from row first[s] on, every
@@ -429,5 +461,5 @@ extern "C" int rb_dense_flash(const void* q, long long q_pitch, const void* k, c
   p.H = H; p.G = 1; p.tokens = BQ; p.max_blocks = 1; p.page = BKV; p.out_d = dv;
   p.scale_log2 = scale * 1.4426950408889634f;
   p.err = err;
-  return dispatch({q, k, v, rows, n, H, dk, dv, q_pitch, static_cast<uint64_t>(k_rows)}, p, st);
+  return dispatch<false>({q, k, v, rows, n, H, dk, dv, q_pitch, static_cast<uint64_t>(k_rows), false}, p, st);
 }

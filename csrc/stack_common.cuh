@@ -80,6 +80,12 @@ __device__ __forceinline__ float sigmoid(float x) {
   if constexpr (kExact) return 1.f / (1.f + expf(-x));
   else return __fdividef(1.f, 1.f + __expf(-x));      // x << 0: the denominator overflows to inf, the quotient is 0
 }
+// the value that an element of type T keeps of x
+template <typename T>
+__device__ __forceinline__ float round_to(float x) {
+  if constexpr (sizeof(T) == 4) return x;
+  else return __bfloat162float(__float2bfloat16(x));
+}
 template <typename T> struct IsExact { static constexpr bool v = sizeof(T) == 4; };
 
 }  // namespace stack

@@ -10,6 +10,7 @@
 //  * sum_norm       residual = norm(alpha residual + a sublayer's output, weighted expert rows included); writes the next sublayer's input
 //                  (or its final norm)
 //  * hgrn2_step     one token per sequence: gates, state update, read-out and per-head norm in one pass over the state
+//                  (and the same for linear attention whose rows decay by gates of their own, here and in hgrn2_scan)
 //  * hgrn2_scan     segments of any length: the state stays in registers while the tokens stream through shared memory
 //  * latent_write   norm of the latent projection, scattered into the paged latent cache, with the rotation of the part of queries and
 //                  rows that carries positions
@@ -359,12 +360,19 @@ struct HgrnParams {
   void* out;              // [T][ldo]
   int H, dim, vdim, vp, ld, ldo;
   float eps;
+  // kGla (linear attention with decaying rows): qfv is q (H*dim) | k (H*dim) | v (H*vdim) and, from column gate_col on, output gates
+  // (H*vdim); f_bias joins z, and a row decays by sigmoid(z) ^ inv_root
+  const float* z;         // [T][ldz]
+  int ldz, gate_col;
+  float q_scale, inv_root;
 };
+// sigmoid(z) ^ r from its logarithm, min(z, 0) - log(1 + exp(-|z|))
+__device__ __forceinline__ float decay(float z, float r) { return expf((fminf(z, 0.f) - log1pf(expf(-fabsf(z)))) * r); }
 
 // One new token per sequence.  CTA = (sequence, head); a thread owns four value columns of every ng-th state row, so a
 // warp reads and writes whole rows; eight rows per thread are in flight at a time.
 constexpr int HS_THREADS = 256;
-template <typename T>
+template <typename T, bool kGla>
 __global__ void __launch_bounds__(HS_THREADS) hgrn2_step_kernel(const HgrnParams p) {
   constexpr bool kExact = IsExact<T>::v;
   extern __shared__ __align__(16) float sm[];
@@ -380,6 +388,12 @@ __global__ void __launch_bounds__(HS_THREADS) hgrn2_step_kernel(const HgrnParams
   const int qd = p.H * p.dim;
   for (int d = tid; d < p.dim; d += HS_THREADS) {
     const int c = hd * p.dim + d;
+    if constexpr (kGla) {
+      sq[d] = ld(row + c) * p.q_scale;
+      sk[d] = ld(row + qd + c);
+      sg[d] = decay(p.z[static_cast<long long>(s) * p.ldz + c] + ld(static_cast<const T*>(p.f_bias) + c), p.inv_root);
+      continue;
+    }
     const float q = ld(row + c), f = ld(row + qd + c) + ld(static_cast<const T*>(p.f_bias) + c);
     const float lo = ld(static_cast<const T*>(p.lower) + c);
     const float sf = sigmoid<kExact>(f), sn = sigmoid<kExact>(-f);
@@ -440,7 +454,14 @@ __global__ void __launch_bounds__(HS_THREADS) hgrn2_step_kernel(const HgrnParams
   for (int k = 0; k < HS_THREADS / 32; ++k) ss += wred[k];
   const float r = 1.f / sqrtf(ss / p.vdim + p.eps);
   T* out = static_cast<T*>(p.out) + static_cast<long long>(s) * p.ldo;
-  for (int j = tid; j < p.vdim; j += HS_THREADS) st(out + hd * p.vdim + j, red[j] * r * ld(static_cast<const T*>(p.norm_w) + j));
+  for (int j = tid; j < p.vdim; j += HS_THREADS) {
+    float o = red[j] * r * ld(static_cast<const T*>(p.norm_w) + j);
+    if constexpr (kGla) {
+      const float g = ld(row + p.gate_col + hd * p.vdim + j);
+      o *= g * sigmoid<kExact>(g);
+    }
+    st(out + hd * p.vdim + j, o);
+  }
   if (hd == p.H - 1)
     for (int j = p.H * p.vdim + tid; j < p.ldo; j += HS_THREADS) st(out + j, 0.f);
 }
@@ -493,7 +514,7 @@ __device__ __forceinline__ Raw8<T> raw_load(const T* p, int valid) {      // `va
   return r;
 }
 
-template <typename T, bool kVec>
+template <typename T, bool kVec, bool kGla>
 __global__ void __launch_bounds__(512) hgrn2_scan_kernel(const HgrnParams p, int NG) {
   constexpr bool kExact = IsExact<T>::v;
   extern __shared__ __align__(16) float sm[];
@@ -531,6 +552,7 @@ __global__ void __launch_bounds__(512) hgrn2_scan_kernel(const HgrnParams p, int
   // raw data of the next chunk: this thread prepares features dpre .. dpre + 7 of the tokens tpre and tpre + 8
   const int tpre = tid / NG, dpre = (tid - tpre * NG) * 8;
   Raw8<T> rq[2], rf[2], rv;
+  Raw8<float> rz[kGla ? 2 : 1];
   auto fetch = [&](int t0) {
 #pragma unroll
     for (int k = 0; k < 2; ++k) {
@@ -539,6 +561,7 @@ __global__ void __launch_bounds__(512) hgrn2_scan_kernel(const HgrnParams p, int
       const T* a = base + static_cast<long long>(t0 + t) * p.ld + hd * p.dim + dpre;
       rq[k] = raw_load<T, kVec>(a, valid);
       rf[k] = raw_load<T, kVec>(a + qd, valid);
+      if constexpr (kGla) rz[k] = raw_load<float, kVec>(p.z + static_cast<long long>(t0 + t) * p.ldz + hd * p.dim + dpre, valid);
     }
     if (tid < SC_CH * 4) {
       const int t = tid >> 2, j = (tid & 3) * 8;
@@ -550,7 +573,7 @@ __global__ void __launch_bounds__(512) hgrn2_scan_kernel(const HgrnParams p, int
   for (int i = 0; i < 8; ++i) {
     const bool in = dpre + i < p.dim;
     fb[i] = in ? ld(static_cast<const T*>(p.f_bias) + hd * p.dim + dpre + i) : 0.f;
-    fl[i] = in ? ld(static_cast<const T*>(p.lower) + hd * p.dim + dpre + i) : 1.f;       // padding rows: 1 - gate = 0
+    if constexpr (!kGla) fl[i] = in ? ld(static_cast<const T*>(p.lower) + hd * p.dim + dpre + i) : 1.f;       // padding rows: 1 - gate = 0
   }
   fetch(lo);
   for (int t0 = lo; t0 < hi; t0 += SC_CH) {
@@ -562,6 +585,12 @@ __global__ void __launch_bounds__(512) hgrn2_scan_kernel(const HgrnParams p, int
 #pragma unroll
       for (int i = 0; i < 8; ++i) {
         const float q = raw_get<T>(rq[k], i), f = raw_get<T>(rf[k], i) + fb[i];
+        if constexpr (kGla) {      // padding rows: k = 0
+          a.v[i] = decay(raw_get<float>(rz[k], i) + fb[i], p.inv_root);
+          b.v[i] = raw_get<T>(rf[k], i);
+          c.v[i] = q * p.q_scale;
+          continue;
+        }
         if constexpr (kExact) {
           a.v[i] = fl[i] + (1.f - fl[i]) * sigmoid<true>(f);
           b.v[i] = (1.f - fl[i]) * sigmoid<true>(-f);
@@ -647,10 +676,11 @@ __global__ void __launch_bounds__(512) hgrn2_scan_kernel(const HgrnParams p, int
   }
 }
 
-// per-head RMS norm of the scan's read-outs; one warp per (token, head)
+// per-head RMS norm of the scan's read-outs, times silu of a gate per feature when given; one warp per (token, head)
 template <typename T>
 __global__ void __launch_bounds__(256) head_norm_kernel(const float* __restrict__ o_raw, const T* __restrict__ w, T* __restrict__ out,
-                                                        long long units, int H, int vdim, int ldo, float eps) {
+                                                        const T* __restrict__ gate, int ld_gate, long long units, int H, int vdim, int ldo, float eps) {
+  constexpr bool kExact = IsExact<T>::v;
   const long long u = static_cast<long long>(blockIdx.x) * 8 + (threadIdx.x >> 5);
   const int lane = threadIdx.x & 31;
   if (u >= units) return;
@@ -662,7 +692,14 @@ __global__ void __launch_bounds__(256) head_norm_kernel(const float* __restrict_
   ss = wsum(ss);
   const float r = 1.f / sqrtf(ss / vdim + eps);
   T* d = out + t * ldo;
-  for (int j = lane; j < vdim; j += 32) st(d + hd * vdim + j, o[j] * r * ld(w + j));
+  for (int j = lane; j < vdim; j += 32) {
+    float x = o[j] * r * ld(w + j);
+    if (gate) {
+      const float g = ld(gate + t * ld_gate + hd * vdim + j);
+      x *= g * sigmoid<kExact>(g);
+    }
+    st(d + hd * vdim + j, x);
+  }
   if (hd == H - 1)
     for (int j = H * vdim + lane; j < ldo; j += 32) st(d + j, 0.f);
 }
@@ -896,20 +933,21 @@ static int launch_latent_attn(const LatentParams& p, int rows, cudaStream_t stm)
   return static_cast<int>(cudaGetLastError());
 }
 
-template <typename T>
+template <typename T, bool kGla>
 static int launch_scan(const HgrnParams& p, int segs, int rows, bool vec, cudaStream_t stm) {
   int NG = (p.dim + 31) / 32 * 4;                 // row groups of 8; whole warps (8 lanes per group)
   if (NG < 8) NG = 8;                             // at least 64 threads: they also fetch the values of a chunk
   if (NG * 8 > 512) return -2;
   const size_t smem = (static_cast<size_t>(SC_CH) * (3 * NG * 8 + 2 * SC_V + NG * SC_V)) * 4;
   if (smem > 227 * 1024) return -2;
-  auto k = vec ? hgrn2_scan_kernel<T, true> : hgrn2_scan_kernel<T, false>;
+  auto k = vec ? hgrn2_scan_kernel<T, true, kGla> : hgrn2_scan_kernel<T, false, kGla>;
   const cudaError_t e = cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
   if (e != cudaSuccess) return static_cast<int>(e);
   k<<<dim3(segs, p.H, (p.vdim + SC_V - 1) / SC_V), NG * 8, smem, stm>>>(p, NG);
   const long long units = static_cast<long long>(rows) * p.H;
-  head_norm_kernel<T><<<static_cast<unsigned>((units + 7) / 8), 256, 0, stm>>>(p.o_raw, static_cast<const T*>(p.norm_w), static_cast<T*>(p.out), units,
-                                                                             p.H, p.vdim, p.ldo, p.eps);
+  head_norm_kernel<T><<<static_cast<unsigned>((units + 7) / 8), 256, 0, stm>>>(p.o_raw, static_cast<const T*>(p.norm_w), static_cast<T*>(p.out),
+                                                                             kGla ? static_cast<const T*>(p.qfv) + p.gate_col : nullptr, p.ld, units, p.H, p.vdim,
+                                                                             p.ldo, p.eps);
   rb_note_launch(2);
   return static_cast<int>(cudaGetLastError());
 }
@@ -1001,6 +1039,22 @@ extern "C" int rb_embed_norm(const long long* tok, const void* table, const void
   return launch_norm_add<NA_EMBED>(p, rows, (width / groups) % 8 == 0, fp32, stm);
 }
 
+template <typename T, bool kGla>
+static int launch_recurrence(const HgrnParams& p, int rows, int segs, cudaStream_t stm) {
+  if (p.cu) {
+    if (!p.o_raw) return -3;
+    const bool vec = p.dim % 8 == 0 && p.vdim % 8 == 0 && p.ld % 8 == 0 && p.ldz % 4 == 0 &&
+                     (reinterpret_cast<uintptr_t>(p.qfv) | reinterpret_cast<uintptr_t>(p.z)) % 16 == 0;
+    return launch_scan<T, kGla>(p, segs, rows, vec, stm);
+  }
+  const int lpr = p.vp / 4, ng = HS_THREADS / lpr;
+  const size_t smem = (3 * static_cast<size_t>((p.dim + 3) & ~3) + p.vp + static_cast<size_t>(ng) * p.vp) * 4;
+  if (smem > 48 * 1024) return -2;
+  hgrn2_step_kernel<T, kGla><<<dim3(segs, p.H), HS_THREADS, smem, stm>>>(p);
+  rb_note_launch(1);
+  return static_cast<int>(cudaGetLastError());
+}
+
 // cu == null: one row per segment.  o_raw: scratch [rows][H][vdim] fp32, needed with cu.
 extern "C" int rb_hgrn2(const void* qfv, const void* f_bias, const void* lower, const void* norm_w, float* state, const int* slot, const int* ctx,
                         const int* cu, float* o_raw, void* out, int rows, int segs, int H, int dim, int vdim, int vp, int ld, int ldo, float eps,
@@ -1008,18 +1062,17 @@ extern "C" int rb_hgrn2(const void* qfv, const void* f_bias, const void* lower, 
   if (rows <= 0 || segs <= 0) return 0;
   if (vp % 4 || vp < vdim || vp > 4 * HS_THREADS || ld < H * (2 * dim + vdim) || ldo < H * vdim) return -2;
   HgrnParams p{qfv, f_bias, lower, norm_w, state, slot, ctx, cu, o_raw, out, H, dim, vdim, vp, ld, ldo, eps};
-  if (cu) {
-    if (!o_raw) return -3;
-    const bool vec = dim % 8 == 0 && vdim % 8 == 0 && ld % 8 == 0 && reinterpret_cast<uintptr_t>(qfv) % 16 == 0;
-    return fp32 ? launch_scan<float>(p, segs, rows, vec, stm) : launch_scan<bf16>(p, segs, rows, vec, stm);
-  }
-  const int lpr = vp / 4, ng = HS_THREADS / lpr;
-  const size_t smem = (3 * static_cast<size_t>((dim + 3) & ~3) + vp + static_cast<size_t>(ng) * vp) * 4;
-  if (smem > 48 * 1024) return -2;
-  if (fp32) hgrn2_step_kernel<float><<<dim3(segs, H), HS_THREADS, smem, stm>>>(p);
-  else hgrn2_step_kernel<bf16><<<dim3(segs, H), HS_THREADS, smem, stm>>>(p);
-  rb_note_launch(1);
-  return static_cast<int>(cudaGetLastError());
+  return fp32 ? launch_recurrence<float, false>(p, rows, segs, stm) : launch_recurrence<bf16, false>(p, rows, segs, stm);
+}
+
+// rows [T][ld]: q | k | v, from gate_col on output gates; z [T][ldz] fp32, to which z_bias is added; q_scale: factor on q
+extern "C" int rb_gla(const void* in, const float* z, int ldz, const void* z_bias, const void* norm_w, float* state, const int* slot, const int* ctx,
+                      const int* cu, float* o_raw, void* out, int rows, int segs, int H, int dim, int vdim, int vp, int ld, int ldo, int gate_col, float eps,
+                      float q_scale, float inv_root, int fp32, cudaStream_t stm) {
+  if (rows <= 0 || segs <= 0) return 0;
+  if (vp % 4 || vp < vdim || vp > 4 * HS_THREADS || gate_col < H * (2 * dim + vdim) || ld < gate_col + H * vdim || ldo < H * vdim || ldz < H * dim) return -2;
+  HgrnParams p{in, z_bias, nullptr, norm_w, state, slot, ctx, cu, o_raw, out, H, dim, vdim, vp, ld, ldo, eps, z, ldz, gate_col, q_scale, inv_root};
+  return fp32 ? launch_recurrence<float, true>(p, rows, segs, stm) : launch_recurrence<bf16, true>(p, rows, segs, stm);
 }
 
 // rot > 0: k_rot and q (see LatentWriteParams) share the pitch ld of raw; part: column of the rotated key part in the pool

@@ -375,6 +375,13 @@ def projection_inputs(qkv, q_w, k_w, table, heads, kv_heads, dim, vdim, dp, rot_
     return q
 
 
+def conv_inputs(qkv, bias, taps, state, b, q_w, k_w, table, heads, kv_heads, dim, vdim, dp, rot_dims, eps, k_pool, v_pool):
+    q = torch.empty(qkv.shape[0], heads, dp, dtype=qkv.dtype, device=qkv.device)
+    _load().conv_inputs(qkv, bias, taps, state, q_w, k_w, table, q, k_pool, v_pool, b.slots, b.ctx, b.state_slot, b.cu, b.seg_of, b.pos, int(kv_heads),
+                        int(dim), int(vdim), int(rot_dims), float(eps))
+    return q
+
+
 def decode_splits(rows: int, kv_heads: int, max_ctx: int) -> int:
     """Parts of the context that run side by side: enough CTAs to fill the machine twice, at least 512 positions each, none
     when the batch alone fills it."""
@@ -386,36 +393,42 @@ def decode_splits(rows: int, kv_heads: int, max_ctx: int) -> int:
     return splits
 
 
-def paged_attention(q, k_pool, v_pool, b, block_size, scale, sink, out_width, window=0, gate=None):
+def paged_attention(q, k_pool, v_pool, b, block_size, scale, sink, out_width, window=0, gate=None, keep=0, chunk=0, softcap=0.0, talk=None):
     """bf16 heads of up to 128 features: segments of several rows on the flash kernel, single rows on the decode kernel (the
-    flash kernel when more than 16 heads share keys); anything else, and fp32, on CUDA cores."""
+    flash kernel when more than 16 heads share keys); anything else, and fp32, on CUDA cores.  With ``talk`` every head's weights meet the
+    values of every group, and the outputs are mixed: ``sum_g T[h, g] (P_g V) = (sum_g T[h, g] P_g) V``."""
     T, H, dp = q.shape
     G = k_pool.shape[1]
-    L, err = _load(), err_flag(q.device)
-    out = torch.empty(T, H * out_width, dtype=q.dtype, device=q.device)
+    L, err, wide = _load(), err_flag(q.device), talk is not None
+    out = torch.empty(T, H * out_width * (G if wide else 1), dtype=q.dtype, device=q.device)
     n, s = (0, 0) if b.cu is None else (b.multi_rows, b.multi_segs)
-    if q.dtype == torch.bfloat16 and max(dp, v_pool.shape[2]) <= 128 and H // G <= 128:
-        ok = n == 0 or L.paged_flash(q[:n], k_pool, v_pool, b.block_tables, b.ctx, b.blocks[128 // (H // G)], sink,
-                                     None if gate is None else gate[:n], out[:n], int(block_size), int(window), float(scale), err)
-        if ok and n == T:
-            return out
-        if ok:
-            bt, ctx, g = b.block_tables[s:], b.ctx[s:], None if gate is None else gate[n:]
-            if H // G <= 16:
-                most = min(b.max_ctx_one, window + block_size) if window else b.max_ctx_one
-                splits = decode_splits(T - n, G, most)
-                po = ml = None
-                if splits > 1:
-                    po = torch.empty(splits * (T - n) * H * 128, dtype=torch.float32, device=q.device)
-                    ml = torch.empty(splits * (T - n) * H * 2, dtype=torch.float32, device=q.device)
-                ok = L.paged_decode(q[n:], k_pool, v_pool, bt, ctx, sink, g, out[n:], po, ml, int(block_size), int(most), int(window), splits,
-                                    float(scale), err)
-            else:
-                ok = L.paged_flash(q[n:], k_pool, v_pool, bt, ctx, None, sink, g, out[n:], int(block_size), int(window), float(scale), err)
-            if ok:
-                return out
-    L.gqa_attn(q, k_pool, v_pool, b.block_tables, b.seg_of, b.pos, b.ctx, sink, gate, out, int(block_size), int(window), float(scale))
-    return out
+    see = (int(window), int(keep), int(chunk))
+
+    def tensor_cores() -> bool:
+        if n and not L.paged_flash(q[:n], k_pool, v_pool, b.block_tables, b.ctx, b.blocks[128 // (H // G)], sink, None if gate is None else gate[:n], out[:n],
+                                   int(block_size), *see, wide, float(scale), float(softcap), err):
+            return False
+        if n == T:
+            return True
+        bt, ctx, g = b.block_tables[s:], b.ctx[s:], None if gate is None else gate[n:]
+        if H // G > 16 or wide:
+            return L.paged_flash(q[n:], k_pool, v_pool, bt, ctx, None, sink, g, out[n:], int(block_size), *see, wide, float(scale), float(softcap), err)
+        most = min(b.max_ctx_one, chunk + block_size if chunk else window + keep + 2 * block_size if window else b.max_ctx_one)
+        splits = decode_splits(T - n, G, most)
+        po = ml = None
+        if splits > 1:
+            po = torch.empty(splits * (T - n) * H * 128, dtype=torch.float32, device=q.device)
+            ml = torch.empty(splits * (T - n) * H * 2, dtype=torch.float32, device=q.device)
+        return L.paged_decode(q[n:], k_pool, v_pool, bt, ctx, sink, g, out[n:], po, ml, int(block_size), int(most), *see, splits, float(scale),
+                              float(softcap), err)
+
+    if not (q.dtype == torch.bfloat16 and max(dp, v_pool.shape[2]) <= 128 and H // G <= 128 and tensor_cores()):
+        L.gqa_attn(q, k_pool, v_pool, b.block_tables, b.seg_of, b.pos, b.ctx, sink, gate, out, int(block_size), *see, wide, float(scale), float(softcap))
+    if not wide:
+        return out
+    mixed = torch.empty(T, H * out_width, dtype=q.dtype, device=q.device)
+    L.mix_heads(out, talk, mixed, G)
+    return mixed
 
 
 class ExpertPlan:
@@ -448,14 +461,14 @@ def _moe_plan(rows: int, experts: int, n: int) -> tuple:
     return (256 if tiles * ((n + 255) // 256) >= 296 else 128), rows >= 16 * experts
 
 
-EXPERT_ACT = {"relu2": 1, "clamped_swish": 2}
+EXPERT_ACT = {"relu2": 1, "clamped_swish": 2, "swiglu": 3}
 
 
 def moe_experts(h, plan, up, down, act, limit=0.0):
     """Sorted expert rows ``[T top, W]``: gather, up-projection and activation in one grouped GEMM, down-projection in a second.
     Gated experts: ``up`` holds gate and up rows in alternating runs (:func:`relax_b200.ops.glu_rows`)."""
     R, E, err, code = plan.expert.numel(), up.shape[0], err_flag(h.device), EXPERT_ACT[act]
-    mid = torch.empty(R, up.shape[1] // code, dtype=h.dtype, device=h.device)
+    mid = torch.empty(R, up.shape[1] // (2 if code >= 2 else 1), dtype=h.dtype, device=h.device)
     out = torch.empty(R, down.shape[1], dtype=h.dtype, device=h.device)
     L = _load()
     L.moe_gemm(h, up, mid, plan.tiles, plan.n_tiles, plan.row_token, code, float(limit), *_moe_plan(R, E, up.shape[1]), err)
@@ -477,6 +490,59 @@ def hgrn2(qfv, f_bias, lower, norm_w, state, state_slot, ctx_lens, cu, heads, di
         return out
     run(torch.empty(T, heads, vdim, dtype=torch.float32, device=qfv.device))      # 32-bit mode and head sizes of odd shape
     return out
+
+
+def mingru(zxg, z_b, x_b, state, b, width):
+    T, n = zxg.shape[0], (width + 7) // 8 * 8
+    out = torch.empty(T, n, dtype=zxg.dtype, device=zxg.device)
+    spans, first = b.mean_spans if b.mean_spans is not None else (None, None)
+    total = keep = None
+    if spans is not None:
+        total, keep = (torch.empty(spans.shape[0], n, dtype=torch.float32, device=zxg.device) for _ in range(2))
+    _load().mingru(zxg, z_b, x_b, state, b.state_slot, b.ctx, b.cu, spans, first, total, keep, out, int(width))
+    return out
+
+
+def gla(rows, z, a2_b, norm_w, state, state_slot, ctx_lens, cu, heads, dim, vdim, gate_col, eps, root, spans=None):
+    T = rows.shape[0]
+    sp, first = spans if spans is not None else (None, None)
+    out = torch.empty(T, (heads * vdim + 7) // 8 * 8, dtype=rows.dtype, device=rows.device)
+    st = gt = None
+    if sp is not None and rows.dtype == torch.bfloat16:
+        st = torch.empty(sp.shape[0], *state.shape[1:], dtype=torch.float32, device=rows.device)
+        gt = torch.empty(sp.shape[0], heads, dim, dtype=torch.float32, device=rows.device)
+    run = lambda raw: _load().gla(rows, z, a2_b, norm_w, state, state_slot, ctx_lens, cu, raw, sp, first, st, gt, out, int(dim), int(vdim), int(gate_col),
+                                  float(eps), float(root))
+    if (cu is None or rows.dtype == torch.bfloat16) and run(None):      # decode step, or segments on the tensor cores
+        return out
+    run(torch.empty(T, heads, vdim, dtype=torch.float32, device=rows.device))      # 32-bit mode and head sizes of odd shape
+    return out
+
+
+def stream_step(res, width, eps, y=None, norm_w=None, experts=None, norms=(), shift=None):
+    dt = norms[0].dtype if norms else y[0].dtype
+    h = [torch.empty(res.shape, dtype=dt, device=res.device) for _ in norms or (None,)]
+    rows, plan = experts if experts is not None else (None, None)
+    e = (None,) * 4 if plan is None else (plan.expert, plan.place, plan.offset, plan.weight)
+    mu, state, b = shift if shift is not None else (None, None, None)
+    one = b is not None and b.cu is None      # one row per sequence: shifted in the same pass
+    _load().stream_step(res, list(y or ()), list(norm_w or ()), rows, *e, list(norms), h, mu if one else None, state if one else None,
+                        b.state_slot if one else None, b.ctx if one else None, int(width), float(eps))
+    if b is not None and not one:
+        n, h[0] = h[0], torch.empty_like(h[0])
+        _load().token_shift(n, mu, state, h[0], b.state_slot, b.ctx, b.cu, b.seg_of)
+    return h
+
+
+def side_gate(z, embed, tokens, first, dim):
+    out = torch.empty(z.shape[0], (dim + 7) // 8 * 8, dtype=z.dtype, device=z.device)
+    _load().side_gate(z, embed, tokens, out, int(first), int(dim))
+    return out
+
+
+def softcap(z, cap):
+    _load().softcap(z, float(cap))
+    return z
 
 
 def latent_write(raw, w, rank, eps, pool, slots, turned=None):
