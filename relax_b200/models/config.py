@@ -373,6 +373,14 @@ def window_latent_layers(n_layers: int, att: LayerSpec, lat: LayerSpec, moe: Opt
     return tuple(out)
 
 
+def chunk_mean_pair_layers(n_layers: int, att: LayerSpec, mean: LayerSpec, pair: LayerSpec, moe: Optional[MoESpec]) -> tuple:
+    """Runs of four layers: ``att``, ``mean``, ``pair``, and ``att`` on the keys and values of the run's first layer; ``moe`` in all of them."""
+    out = []
+    for i in range(n_layers):
+        out.append(replace((att, mean, pair, replace(att, kv_from=i - 3))[i % 4], moe=moe))
+    return tuple(out)
+
+
 def talizen_layers(n_layers: int, every: int, rec: LayerSpec, att: LayerSpec) -> tuple:
     """``every - 1`` recurrent layers, then one latent-attention layer, repeated."""
     return tuple(att if (i + 1) % every == 0 else rec for i in range(n_layers))
@@ -519,6 +527,28 @@ _reg(composed_config("zupupel-15b", window_latent_layers(
     LayerSpec("latent_attention", heads=32, dim=128, vdim=128, kv_rank=512, scale=192 ** -0.5, rot_dims=64, rot_base=1e6, out_gate=True),
     MoESpec(experts=128, top=8, ff=768, groups=8, keep=4, act="clamped_swish", limit=7.0, renormalize=True, score="softmax", correction=True, identity=16,
             group_best=1)), hidden_size=2048, vocab_size=64000, eps=1e-6, norm_sum=True, sum_alpha=48 ** 0.25, embed_scale=45.0, logit_scale=1 / 45))
+
+
+# Zoguzen: attention inside chunks with mixed heads, running means, sliding-window attention beside linear attention, upper chunk layers
+# on the keys and values of a lower one; sublayers on norms of the stream, a second embedding, gated experts
+_reg(composed_config("tiny-zoguzen", chunk_mean_pair_layers(
+    5, LayerSpec("attention", heads=6, dim=24, vdim=32, kv_heads=3, scale=0.2, chunk=24, softcap=9.0, unit_sink=True, talk=True, qkv_bias=True, conv=3,
+                 head_norm=True),
+    LayerSpec("mingru", vdim=72),
+    LayerSpec("pair", pair=(LayerSpec("attention", heads=4, dim=16, vdim=24, kv_heads=2, scale=0.3, window=20, keep_first=3, rot_dims=8, rot_base=1e4,
+                                      rot_scaling=(2.0, 1.0, 4.0, 64.0), conv=3, out_gate=True),
+                            LayerSpec("gla", heads=3, dim=16, vdim=24, decay_rank=8, decay_root=8.0))),
+    MoESpec(experts=6, top=2, ff=40, act="swiglu", score="softmax", renormalize=True)), hidden_size=160, vocab_size=320, eps=1e-6, pre_norm=True,
+    token_shift=True, side_dim=12, logit_softcap=15.0, tie_word_embeddings=True, dtype="fp32"))
+_reg(composed_config("zoguzen-15b", chunk_mean_pair_layers(
+    24, LayerSpec("attention", heads=32, dim=128, vdim=128, kv_heads=4, scale=128 ** -0.5, chunk=1024, softcap=30.0, unit_sink=True, talk=True, qkv_bias=True,
+                  conv=4, head_norm=True),
+    LayerSpec("mingru", vdim=4096),
+    LayerSpec("pair", pair=(LayerSpec("attention", heads=16, dim=128, vdim=128, kv_heads=4, scale=128 ** -0.5, window=1024, keep_first=16, rot_dims=128,
+                                      rot_base=5e5, rot_scaling=(8.0, 1.0, 4.0, 8192.0), conv=4, out_gate=True),
+                            LayerSpec("gla", heads=16, dim=64, vdim=128, decay_rank=16, decay_root=16.0))),
+    MoESpec(experts=128, top=8, ff=768, act="swiglu", score="softmax", renormalize=True)), hidden_size=2048, vocab_size=64000, eps=1e-6, pre_norm=True,
+    token_shift=True, side_dim=256, logit_softcap=30.0, tie_word_embeddings=True))
 
 
 def get_config(name: str, **overrides) -> ModelConfig:

@@ -226,3 +226,106 @@ def run(cfg, tensors, tokens):
 
 def model(cfg, tensors, tokens):
     return run(cfg, tensors, tokens)[0]
+
+
+# ---------------------------------------------------------------------------------------------------- random models
+
+
+def moe(experts, top, ff):
+    return {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top}}
+
+
+def att(heads, kv_heads, dim, vdim, scale, chunk, cap, conv, mlp=None, kv_from=None):
+    m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale, "mask": {"size": chunk}, "softcap": cap, "conv": conv}
+    if kv_from is not None:
+        m["kv_from"] = kv_from
+    return {"type": "attention", "mixer": m, "mlp": mlp}
+
+
+def gru(width, mlp=None):
+    return {"type": "mingru", "mixer": {"width": width}, "mlp": mlp}
+
+
+def left(heads, kv_heads, dim, vdim, scale, window, keep, conv, rot, base, scaling=None):
+    r = {"dims": rot, "base": base}
+    if scaling is not None:
+        r["scaling"] = dict(zip(("factor", "low", "high", "original"), scaling))
+    return {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale, "mask": {"size": window, "keep_first": keep}, "conv": conv, "rot": r}
+
+
+def right(heads, dim, vdim, tau, rank):
+    """(the rank is no key of a configuration: :func:`random_model` takes it out)"""
+    return {"heads": heads, "dim": dim, "vdim": vdim, "tau": tau, "rank": rank}
+
+
+def pair(a, b, mlp=None):
+    return {"type": "parallel", "mixer": {"left": a, "right": b}, "mlp": mlp}
+
+
+def stack(width, vocab, eps, layers, side, cap):
+    return {"architecture": "Zoguzen", "width": width, "vocab": vocab, "norm": {"eps": eps}, "token_side": {"dim": side}, "logit_softcap": cap, "layers": layers}
+
+
+CONFIGS = {
+    # every padding rule at once: nothing is a multiple of anything; readers with chunks and caps other than their source's
+    "odd": stack(74, 131, 3e-5, [att(6, 2, 18, 13, 0.31, 21, 5.0, 3, moe(7, 2, 20)), gru(37, moe(5, 1, 9)), att(6, 2, 18, 13, 0.22, 9, 3.0, 4, moe(4, 3, 33), 0),
+                                 pair(left(4, 2, 10, 7, 0.5, 12, 5, 2, 6, 300.0, (3.0, 1.0, 3.0, 60.0)), right(3, 6, 5, 3.0, 3), moe(6, 3, 12)),
+                                 att(5, 5, 7, 9, 0.9, 33, 2.0, 5), pair(left(3, 3, 8, 11, 0.6, 20, 2, 3, 8, 50.0), right(2, 9, 12, 5.0, 20))], 5, 7.0),
+    # whole heads turn; wide groups, narrow keys beside wide values, more groups than two
+    "even": stack(128, 256, 1e-4, [pair(left(8, 2, 64, 64, 0.15, 48, 16, 4, 64, 1e4, (8.0, 1.0, 4.0, 64.0)), right(4, 32, 64, 12.0, 8), moe(8, 2, 64)),
+                                   att(8, 1, 64, 128, 0.2, 40, 15.0, 4, moe(6, 3, 64)), gru(192, moe(8, 2, 32)), att(16, 4, 128, 32, 0.11, 64, 25.0, 2, moe(14, 4, 128)),
+                                   att(16, 4, 128, 32, 0.2, 100, 10.0, 4, None, 3), pair(left(4, 4, 128, 40, 0.1, 33, 70, 4, 32, 1e5), right(3, 64, 32, 16.0, 24))], 16, 20.0),
+    # one head, one feature pair, one tap, a window of one token without kept ones, chunks of one token, all experts taken
+    "single": stack(64, 65, 1e-3, [att(1, 1, 16, 40, 0.7, 1, 4.0, 1, moe(2, 2, 8)), gru(8, moe(3, 1, 8)),
+                                   pair(left(1, 1, 16, 8, 0.7, 1, 0, 1, 2, 10.0), right(1, 8, 8, 1.0, 1)), att(1, 1, 16, 40, 0.5, 500, 9.0, 6, None, 0)], 1, 3.0),
+    # more heads per group than the decode tile takes; heads wider than the tensor-core kernels take; a decay of odd shape
+    "wide": stack(256, 320, 1e-5, [att(40, 2, 24, 16, 0.3, 17, 8.0, 4, moe(8, 3, 96)), pair(left(20, 1, 24, 16, 0.4, 19, 3, 4, 8, 1e4), right(2, 128, 96, 20.0, 40)),
+                                   att(3, 1, 144, 136, 0.1, 70, 12.0, 3, moe(6, 2, 64)), gru(300, moe(9, 5, 40)),
+                                   pair(left(2, 2, 144, 136, 0.1, 30, 9, 2, 96, 1e6, (2.0, 0.5, 5.0, 100.0)), right(5, 20, 28, 2.0, 6))], 40, 12.0),
+}
+
+
+def random_model(cfg, seed=0, sharp=1.0):
+    """bf16-representable random tensors; ``sharp`` multiplies the attention scales of the configuration that comes back."""
+    cfg = copy.deepcopy(cfg)
+    g = torch.Generator().manual_seed(seed)
+    W, V, S = cfg["width"], cfg["vocab"], cfg["token_side"]["dim"]
+    n = lambda *s, std=1.0: torch.randn(*s, generator=g) * std
+    lin = lambda out, fan: n(out, fan, std=fan ** -0.5)
+    t = {"embed": n(V, W, std=0.4), "side.embed": n(V, S * len(cfg["layers"])), "final.norm": 1 + n(W, std=0.2)}
+
+    def attention(m, p, extras):
+        m["scale"] *= sharp
+        for k, rows in (("q", m["heads"] * m["dim"]), ("k", m["kv_heads"] * m["dim"]), ("v", m["kv_heads"] * m["vdim"]))[:1 if "kv_from" in m else 3]:
+            t.update({p + k: lin(rows, W), p + k + ".conv": n(rows, m["conv"], std=m["conv"] ** -0.5)})
+            if extras:
+                t[p + k + ".b"] = n(rows, std=0.3)
+                if k != "v":
+                    t[p + k + ".norm"] = 1.2 + n(m["dim"], std=0.3)
+        t[p + "o"] = lin(W, m["heads"] * m["vdim"])
+
+    for i, layer in enumerate(cfg["layers"]):
+        m, a, p, f, mlp = layer["mixer"], f"l{i}.", f"l{i}.mix.", f"l{i}.mlp.", layer["mlp"]
+        t.update({a + "norm1": 1 + n(W, std=0.2), a + "shift": torch.rand(W, generator=g), a + "side.gate": lin(S, W) * 0.7, a + "side.proj": lin(W, S),
+                  a + "side.norm": 0.5 + n(W, std=0.2)})
+        if layer["type"] == "attention":
+            attention(m, p, True)
+            t[p + "talk"] = torch.eye(m["heads"]) + n(m["heads"], m["heads"], std=0.4)
+        elif layer["type"] == "mingru":
+            w = m["width"]
+            t.update({p + "z": lin(w, W), p + "z.b": n(w) - 1, p + "x": lin(w, W), p + "x.b": n(w, std=0.5), p + "g": lin(w, W), p + "o": lin(W, w) * 2})
+        else:
+            r = m["right"]
+            rank, qd, vd = r.pop("rank"), r["heads"] * r["dim"], r["heads"] * r["vdim"]
+            attention(m["left"], p + "left.", False)
+            q = p + "right."
+            t.update({p + "left.g": lin(m["left"]["heads"] * m["left"]["vdim"], W), p + "left.out": 1 + n(W, std=0.2), q + "out": 1 + n(W, std=0.2),
+                      q + "q": lin(qd, W), q + "k": lin(qd, W), q + "v": lin(vd, W), q + "g": lin(vd, W), q + "o": lin(W, vd), q + "norm": 1 + n(r["vdim"], std=0.2),
+                      q + "a1": lin(rank, W), q + "a2": lin(qd, rank) * 2, q + "a2.b": n(qd) + 1})
+        if mlp is None:
+            continue
+        E, ff = mlp["router"]["experts"], mlp["expert"]["ff"]
+        t.update({a + "norm2": 1 + n(W, std=0.2), f + "router": lin(E, W) * 1.5})
+        for e in range(E):
+            t.update({f"{f}e{e}.gate": lin(ff, W) * 1.5, f"{f}e{e}.up": lin(ff, W), f"{f}e{e}.down": lin(W, ff) * 2})
+    return cfg, {k: v.to(torch.bfloat16) for k, v in t.items()}
