@@ -78,7 +78,7 @@ def parse():
     ap.add_argument("--stack-bench", choices=["1b", "5b"], default=None,
                     help="instead of the headline workload: serving kernels and engine throughput of a composed stack (Talizen) "
                          "beside the engine's existing models at the same layer sizes (1 GPU; plain-text table)")
-    ap.add_argument("--stack-design", choices=["talizen", "ketolorn", "zupupel"], default="talizen", help="design that --stack-bench measures")
+    ap.add_argument("--stack-design", choices=["talizen", "ketolorn", "zupupel", "zoguzen"], default="talizen", help="design that --stack-bench measures")
     return ap.parse_args()
 
 

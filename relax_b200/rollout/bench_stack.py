@@ -5,8 +5,8 @@ Two tables, random weights, bf16, one GPU:
 * kernels: device time per launch, algorithmic bytes or FLOPs, fraction of the measured copy bandwidth / cuBLAS rate
   (``--peaks``), each kernel of the composed stack beside the like kernel of the existing models;
 * models: prefill and decode tokens/s through the engine's scheduler - a Talizen stack beside the Gated-DeltaNet hybrid and
-  the dense softmax model, a Ketolorn stack beside the mixture-of-experts model, or a Zupupel stack beside a Ketolorn stack, with
-  the same width, heads, feed-forward bytes and depth.
+  the dense softmax model, a Ketolorn stack beside the mixture-of-experts model, a Zupupel stack beside a Ketolorn stack, or a Zoguzen
+  stack beside a Zupupel stack, with the same width, heads, feed-forward bytes and depth.
 
 Times come from CUDA events after warm-up; every kernel rotates through inputs larger than the L2 cache.
 """
@@ -394,6 +394,163 @@ def zupupel_kernel_rows(W=2048, H=32, G=4, d=128, window=1024, R=512, rot=64, E=
     return rows
 
 
+def zoguzen_kernel_rows(W=2048, H=32, G=4, d=128, chunk=1024, Hl=16, Hr=16, dk=64, width=4096, side=256, E=128, k=8, F=768, only=""):
+    """The kernels of one real-sized Zoguzen layer of each kind, each beside the like kernel of Zupupel or Talizen stacks."""
+    from .. import ops
+    from ..models.config import LayerSpec, MoESpec
+    from .composed import ComposedForward, SegmentBatch, mean_spans, query_blocks, recurrent_spans, tile_tokens
+
+    dev, bf = "cuda", torch.bfloat16
+    rows = []
+    mk = lambda *s: torch.randn(*s, device=dev).to(bf)
+    i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
+    want = lambda section: not only or section in only.split(",")
+    one, talk, scale, page = torch.zeros(H, device=dev, dtype=bf), mk(H, H), d ** -0.5, 64
+    chunked = dict(chunk=chunk, softcap=30.0, talk=talk)
+    for B in (16, 128) if want("attn") else ():
+        L = 8 * chunk
+        bt = torch.randperm(B * L // page, device=dev).to(torch.int32).view(B, L // page)
+        b = SegmentBatch(None, None, torch.full((B,), L, dtype=torch.int32, device=dev), bt, None, max_ctx_one=L)
+        for heads, name, kw, s in ((H, "attention decode, chunk, cap, mixed heads", chunked, one), (H, "  like: attention decode, window, gate (Zupupel)", dict(window=chunk), None),
+                                   (Hl, "attention decode, window, first tokens, gate", dict(window=chunk, keep=16), None),
+                                   (Hl, "  like: attention decode, window, gate (Zupupel)", dict(window=chunk), None)):
+            fns = []
+            for _ in range(2 if B * L >= 1 << 20 else _copies(B * chunk * G * d * 4)):
+                kc, vc, q, g = mk(B * L, G, d), mk(B * L, G, d), mk(B, heads, d), mk(B, heads * d)
+                extra = dict(kw, gate=None if "talk" in kw else g)
+                fns.append(_graph(lambda q=q, kc=kc, vc=vc, extra=extra, s=s: ops.paged_attention(q, kc, vc, b, page, scale, s, d, **extra)))
+            rows.append((name, f"batch {B}, {heads} heads, {chunk} of {L} positions", _time(fns), B * chunk * G * d * 4, None))
+            del fns, kc, vc, q
+    for S, n, L in ((1, 8192, 8192), (4, 2048, 2048), (32, 256, 256), (16, 64, 2048), (16, 4, 2048)) if want("prompt") else ():
+        T, nb = S * n, L // page
+        bt = torch.randperm(S * nb, device=dev).to(torch.int32).view(S, nb)
+        for heads, name, kw, s in ((H, "paged flash, chunk, cap, mixed heads", chunked, one), (H, "  like: paged flash, window, gate (Zupupel)", dict(window=chunk), None),
+                                   (Hl, "paged flash, window, first tokens, gate", dict(window=chunk, keep=16), None),
+                                   (Hl, "  like: paged flash, window, gate (Zupupel)", dict(window=chunk), None)):
+            t = tile_tokens(LayerSpec("attention", heads=heads, dim=d, vdim=d, kv_heads=G))
+            q, kc, vc, g = mk(T, heads, d), mk(S * L, G, d), mk(S * L, G, d), mk(T, heads * d)
+            b = SegmentBatch(None, None, i32([L] * S), bt, None, cu=i32([i * n for i in range(S + 1)]), multi_segs=S, multi_rows=T,
+                             blocks={t: i32(query_blocks([n] * S, [L] * S, t))})
+            mixes = "talk" in kw
+            seen = lambda p: p % chunk + 1 if mixes else min(chunk, p + 1)
+            pairs = S * heads * sum(seen(L - n + i) for i in range(n))
+            extra = dict(kw, gate=None if mixes else g)
+            rows.append((name, f"{S} x {n} tokens, context {L}, {heads} heads", _time([_graph(lambda: ops.paged_attention(q, kc, vc, b, page, scale, s, d, **extra))], 10),
+                         T * heads * d * (4 if mixes else 6) + S * min(L, chunk + n) * G * d * 4, pairs * (4.0 * d + (2.0 * heads if mixes else 0.0))))
+    rot, freq = d, torch.tensor([1e6 ** (-2 * i / d) for i in range(d // 2)], dtype=torch.float64, device=dev)
+    for T in (16, 128, 8192) if want("prep") else ():
+        C = (H + 2 * G) * d
+        n = _copies(T * C * 4)
+        pos, slots = torch.arange(T, device=dev).to(torch.int32), torch.randperm(T, device=dev)
+        tab, kp, vp, qw, kw, bias, taps = ops.rope_table(pos, 0, freq), mk(T, G, d), mk(T, G, d), mk(H * d), mk(G * d), mk(C), mk(C, 4)
+        if T > 1000:
+            b = SegmentBatch(None, slots, i32([T // 4] * 4), None, i32([0, 1, 2, 3]), cu=i32([i * T // 4 for i in range(5)]),
+                             seg_of=(torch.arange(T, device=dev) // (T // 4)).to(torch.int32), pos=(torch.arange(T, device=dev) % (T // 4)).to(torch.int32))
+        else:
+            b = SegmentBatch(None, slots, i32([900] * T), None, torch.arange(T, device=dev).to(torch.int32))
+        xs, nb = [mk(T, C) for _ in range(n)], T * C * 4
+        state = mk(T if T < 1000 else 4, 3, C)
+        rows.append(("bias, convolution, head norm, cache write", f"{T} rows", _time([_graph(lambda x=x: ops.conv_inputs(
+            x, bias, taps, state, b, qw[:d], kw[:d], None, H, G, d, d, d, 0, 1e-6, kp, vp)) for x in xs]), nb + (T * 6 * C * 2 if T < 1000 else 0), None))
+        rows.append(("convolution, rotation, cache write", f"{T} rows", _time([_graph(lambda x=x: ops.conv_inputs(
+            x, None, taps, state, b, None, None, tab, H, G, d, d, d, rot, 0.0, kp, vp)) for x in xs]), nb + (T * 6 * C * 2 if T < 1000 else 0), None))
+        rows.append(("  like: projection norms, rotation, cache write (Zupupel)", f"{T} rows",
+                     _time([_graph(lambda x=x: ops.projection_inputs(x, qw, kw, tab, H, G, d, d, d, rot, True, 1e-6, kp, vp, slots)) for x in xs]), nb, None))
+        del xs, state
+    gla = LayerSpec("gla", heads=Hr, dim=dk, vdim=d, decay_rank=16)
+    at = ComposedForward.gla_columns(gla)
+    zb, zw, fb, lower, nw = mk(width), mk(width), mk(Hr * dk), torch.rand(Hr * dk, device=dev).to(bf), mk(d)
+    for B in (16, 128) if want("step") else ():
+        ids, ctx = torch.arange(B, device=dev).to(torch.int32), i32([900] * B)
+        n = _copies(B * Hr * dk * d * 8)
+        states = [torch.randn(B, Hr, dk, d, device=dev) for _ in range(n)]
+        x, z, q = mk(B, at["end"]), torch.randn(B, Hr * dk, device=dev), mk(B, Hr * (2 * dk + d))
+        nb = B * Hr * dk * d * 8
+        rows.append(("linear attention step", f"batch {B}", _time([_graph(lambda s=s: ops.gla(x, z, fb, nw, s, ids, ctx, None, Hr, dk, d, at["g"], 1e-6, 16.0)) for s in states]),
+                     nb, None))
+        rows.append(("  like: hgrn2 step (Talizen)", f"batch {B}", _time([_graph(lambda s=s: ops.hgrn2(q, fb, lower, nw, s, ids, ctx, None, Hr, dk, d, 1e-6)) for s in states]),
+                     nb, None))
+        del states
+        n = _copies(B * width * 16)
+        states, xs = [torch.randn(B, 1, 1, width, device=dev) for _ in range(n)], [mk(B, 3 * width) for _ in range(n)]
+        b = SegmentBatch(None, None, ctx, None, ids)
+        rows.append(("running mean step", f"batch {B}", _time([_graph(lambda s=s, x=x: ops.mingru(x, zb, zw, s, b, width)) for s, x in zip(states, xs)]), B * width * 16, None))
+        del states, xs
+    for S, L in ((1, 8192), (4, 2048), (32, 256)) if want("step") else ():
+        T = S * L
+        cu, ids, ctx = i32([i * L for i in range(S + 1)]), torch.arange(S, device=dev).to(torch.int32), i32([L] * S)
+        both = lambda c: None if c is None else (i32(c[0]), i32(c[1]))
+        spans = both(recurrent_spans([L] * S, Hr))
+        state, x, z, q = torch.zeros(S, Hr, dk, d, device=dev), mk(T, at["end"]), torch.randn(T, Hr * dk, device=dev), mk(T, Hr * (2 * dk + d))
+        rows.append(("linear attention of a prompt", f"{S} x {L}", _time([_graph(lambda: ops.gla(x, z, fb, nw, state, ids, ctx, cu, Hr, dk, d, at["g"], 1e-6, 16.0, spans))], 10),
+                     T * (at["a1"] * 2 + Hr * (dk * 4 + d * 2)), 6.0 * T * Hr * dk * d))
+        rows.append(("  like: hgrn2 of a prompt (Talizen)", f"{S} x {L}", _time([_graph(lambda: ops.hgrn2(q, fb, lower, nw, state, ids, ctx, cu, Hr, dk, d, 1e-6, spans))], 10),
+                     T * Hr * (2 * dk + 2 * d) * 2, 6.0 * T * Hr * dk * d))
+        xs, mean = [mk(T, 3 * width) for _ in range(2)], torch.zeros(S, 1, 1, width, device=dev)
+        b = SegmentBatch(None, None, ctx, None, ids, cu=cu, mean_spans=both(mean_spans([L] * S)))
+        rows.append(("running mean of a prompt", f"{S} x {L}", _time([_graph(lambda x=x: ops.mingru(x, zb, zw, mean, b, width)) for x in xs], 10), T * width * 8, None))
+        del xs
+    mine = MoESpec(experts=E, top=k, ff=F, act="swiglu", score="softmax", renormalize=True)
+    like = MoESpec(experts=E, top=k, ff=F, groups=8, keep=4, act="clamped_swish", limit=7.0, renormalize=True, score="softmax", correction=True, group_best=1)
+    corr = torch.zeros(E, device=dev, dtype=bf)
+    route = lambda spec, z: ops.moe_route(z, spec, bf, None, corr if spec.correction else None)
+    for T in (1, 16, 128, 8192) if want("moe") else ():
+        h, up, down = mk(T, W), mk(E, 2 * F, W), mk(E, W, F)
+        zs = [torch.randn(T, E, device=dev) for _ in range(1 if T > 1000 else 4)]      # each touches other experts
+        for spec, name in ((mine, "expert products (gather, both halves, silu unit, down)"), (like, "  like: bounded units (Zupupel)")):
+            plans = [route(spec, z) for z in zs]
+            hit = sum(int((p.offset[1:] > p.offset[:-1]).sum()) for p in plans) / len(plans)
+            rows.append((name, f"{T} rows", _time([_graph(lambda p=p: ops.moe_experts(h, p, up, down, spec.act, spec.limit)) for p in plans], 10),
+                         hit * 3 * F * W * 2 + T * k * (2 * W + 2 * F) * 2, 6.0 * T * k * F * W if T > 1000 else None))
+        for spec, name in ((mine, "routing and layout"), (like, "  like: routing and layout, groups and correction (Zupupel)")):
+            rows.append((name, f"{T} rows", _time([_graph(lambda: route(spec, zs[0]))]), T * E * 4 + T * k * 16, None))
+        del up, down
+    for T in (16, 128, 8192) if want("norm") else ():
+        n = _copies(T * W * (12 + 2 * k))
+        w, mu, bias = mk(W), mk(W), mk(W)
+        plan, other = (route(s, torch.randn(T, E, device=dev)) for s in (mine, like))
+        buf = [(torch.randn(T, W, device=dev), mk(T, W), mk(T, W), mk(T * k, W)) for _ in range(n)]
+        many = T > 1000
+        b = SegmentBatch(None, None, i32([T // 4] * 4) if many else i32([900] * T), None, torch.arange(4 if many else T, device=dev).to(torch.int32),
+                         cu=i32([i * T // 4 for i in range(5)]) if many else None, seg_of=(torch.arange(T, device=dev) // max(1, T // 4)).to(torch.int32))
+        state = mk(4 if many else T, W)
+        run = lambda f: _time([_graph(lambda a=a: f(*a)) for a in buf])
+        rows.append(("stream step: mixer, expert rows", f"{T} rows", run(lambda r, y, _, e: ops.stream_step(r, W, 1e-6, [y], None, (e, plan))), T * W * (12 + 2 * k), None))
+        rows.append(("stream step: pair of normed mixers, expert rows", f"{T} rows", run(lambda r, y, x, e: ops.stream_step(r, W, 1e-6, [y, x], (w, bias), (e, plan))),
+                     T * W * (14 + 2 * k), None))
+        rows.append(("stream step: second embedding, two norms, shift", f"{T} rows", run(lambda r, y, _, e: ops.stream_step(r, W, 1e-6, [y], (w,), None, (w, bias), (mu, state, b))),
+                     T * W * (18 if many else 18), None))
+        rows.append(("  like: sum_norm with expert rows (Zupupel)", f"{T} rows", run(lambda r, y, _, e: ops.sum_norm(r, y, w, bias, W, 1.5, 1e-6, None, 1.0, (e, other))),
+                     T * W * (12 + 2 * k), None))
+        rows.append(("  like: sum_norm and the final norm (Zupupel)", f"{T} rows", run(lambda r, y, _, e: ops.sum_norm(r, y, w, bias, W, 1.5, 1e-6, (w, bias), 0.1)), T * W * 12, None))
+        ids, table = torch.randint(0, 64000, (T,), device=dev), mk(64000, 4 * side)
+        zs = [mk(T, side) for _ in range(n)]
+        rows.append(("second embedding: gelu and product", f"{T} rows", _time([_graph(lambda z=z: ops.side_gate(z, table, ids, side, side)) for z in zs]), T * side * 6, None))
+        xs = [mk(T, 2 * side) for _ in range(n)]
+        rows.append(("  like: gated unit", f"{T} rows", _time([_graph(lambda x=x: ops.glu(x, "gelu_tanh")) for x in xs]), T * side * 6, None))
+        if not many:
+            zs = [torch.randn(T, 64000, device=dev) for _ in range(_copies(T * 64000 * 8))]
+            rows.append(("capped logits", f"{T} rows of 64000", _time([_graph(lambda z=z: ops.softcap(z, 30.0)) for z in zs]), T * 64000 * 8, None))
+        del buf, zs, xs
+    return rows
+
+
+def _zoguzen_models(layers: int, W: int, H: int, G: int, experts: int, top: int, ff: int, vocab: int):
+    """A Zoguzen stack and a Zupupel stack of the same width, heads, window, depth and experts."""
+    from ..models.config import LayerSpec, MoESpec, chunk_mean_pair_layers, composed_config
+
+    d = 128
+    att = LayerSpec("attention", heads=H, dim=d, vdim=d, kv_heads=G, scale=d ** -0.5, chunk=1024, softcap=30.0, unit_sink=True, talk=True, qkv_bias=True, conv=4,
+                    head_norm=True)
+    pair = LayerSpec("pair", pair=(LayerSpec("attention", heads=H // 2, dim=d, vdim=d, kv_heads=G, scale=d ** -0.5, window=1024, keep_first=16, rot_dims=d, rot_base=5e5,
+                                             rot_scaling=(8.0, 1.0, 4.0, 8192.0), conv=4, out_gate=True),
+                                   LayerSpec("gla", heads=H // 2, dim=64, vdim=d, decay_rank=16, decay_root=16.0)))
+    mine = MoESpec(experts=experts, top=top, ff=ff, act="swiglu", score="softmax", renormalize=True)
+    return {"zoguzen": composed_config("zoguzen", chunk_mean_pair_layers(layers, att, LayerSpec("mingru", vdim=2 * W), pair, mine), W, vocab, pre_norm=True,
+                                       token_shift=True, side_dim=256, logit_softcap=30.0, tie_word_embeddings=True),
+            "zupupel": _zupupel_models(layers, W, H, G, experts, top, ff, vocab)["zupupel"]}
+
+
 def _zupupel_models(layers: int, W: int, H: int, G: int, experts: int, top: int, ff: int, vocab: int):
     """A Zupupel stack and a Ketolorn stack with experts of the same bytes in every layer (no shared expert)."""
     from dataclasses import replace
@@ -442,7 +599,9 @@ def model_rows(size: str, only=None, decode_batches=(1, 32, 128), prompt=2048, d
     """``(model, workload, tokens/s, ms)`` through ``RolloutEngine.step``."""
     from .engine import RolloutEngine, SamplingParams
 
-    if design == "zupupel":
+    if design == "zoguzen":
+        models = _zoguzen_models(*{"1b": (8, 2048, 32, 4, 128, 8, 768), "5b": (8, 4096, 64, 8, 128, 8, 1536)}[size], 64000)
+    elif design == "zupupel":
         models = _zupupel_models(*{"1b": (9, 2048, 32, 4, 128, 8, 768), "5b": (9, 4096, 64, 8, 128, 8, 1536)}[size], 64000)
     elif design == "ketolorn":
         models = _ketolorn_models(*{"1b": (8, 2048, 32, 4, 128, 8, 768, 6144), "5b": (8, 4096, 64, 8, 128, 8, 1536, 12288)}[size], 64000)
@@ -458,9 +617,9 @@ def model_rows(size: str, only=None, decode_batches=(1, 32, 128), prompt=2048, d
                             block_size=page, max_running=136,
                             max_model_len=prompt + 256, memory_saver=False)
         eng.weights.flat.normal_(0, 0.02)
-        if design == "zupupel":      # rows of unit size and no bias of the choice: tokens spread over the experts
+        if design in ("zupupel", "zoguzen"):      # rows of unit size and no bias of the choice: tokens spread over the experts
             for key, t in eng.weights.p.items():
-                if key.endswith("norm"):
+                if key.endswith(("norm", "norm1", "norm2")):
                     t.fill_(1.0)
                 elif key.endswith(("norm_b", "moe_correction")):
                     t.zero_()
@@ -509,7 +668,7 @@ def main(size: str = "5b", peaks: str = "MEASURED_PEAKS.json", kernels: bool = T
     hbm, tf = pk.get("hbm_gbs"), pk.get("bf16_tflops")
     if kernels:
         print("kernel | case | us | GB/s (of measured copy) | TFLOP/s (of measured GEMM)")
-        for k, case, ms, nb, fl in {"talizen": kernel_rows, "ketolorn": ketolorn_kernel_rows, "zupupel": zupupel_kernel_rows}[design](only=only):
+        for k, case, ms, nb, fl in {"talizen": kernel_rows, "ketolorn": ketolorn_kernel_rows, "zupupel": zupupel_kernel_rows, "zoguzen": zoguzen_kernel_rows}[design](only=only):
             gb = nb / ms / 1e6
             t = f"{gb:7.0f}" + (f" ({gb / hbm:.2f})" if hbm else "")
             if fl:
@@ -527,9 +686,9 @@ if __name__ == "__main__":
     import argparse
 
     ap = argparse.ArgumentParser(description="kernel table of composed stacks")
-    ap.add_argument("--design", choices=["talizen", "ketolorn", "zupupel"], default="talizen")
+    ap.add_argument("--design", choices=["talizen", "ketolorn", "zupupel", "zoguzen"], default="talizen")
     ap.add_argument("--only", default="", help="sections, with commas: step, attn, gemm, norm, prompt (talizen); attn, prompt, prep, moe, norm, gemm (ketolorn); "
-                                               "attn, prompt, latent, prep, gemm, moe, norm (zupupel)")
+                                               "attn, prompt, latent, prep, gemm, moe, norm (zupupel); attn, prompt, prep, step, moe, norm (zoguzen)")
     ap.add_argument("--peaks", default="MEASURED_PEAKS.json")
     a = ap.parse_args()
     raise SystemExit(main(peaks=a.peaks, models=False, only=a.only, design=a.design))
