@@ -153,8 +153,8 @@ int rb_gla(const void* in, const float* z, int ldz, const void* z_bias, const vo
 int rb_gla_chunk(const void* in, const float* z, int ldz, const void* z_bias, const void* norm_w, float* state, const int* slot, const int* ctx,
                  const int* cu, const int* spans, const int* first, float* span_state, float* span_gate, void* out, int rows, int segs, int n_spans,
                  int H, int dim, int vdim, int vp, int ld, int ldo, int gate_col, float eps, float q_scale, float inv_root, cudaStream_t st);
-int rb_mingru(const void* rows, const void* z_b, const void* x_b, float* state, const int* slot, const int* ctx, const int* cu, const int* spans, const
-              int* first, float* span_sum, float* span_keep, void* out, int segs, int n_spans, int width, int ld, int sp, int fp32, cudaStream_t st);
+int rb_mingru(const void* rows, const void* z_b, const void* x_b, float* state, const int* slot, const int* ctx, const int* cu, void* out, int segs, int
+              width, int ld, int sp, int fp32, cudaStream_t st);
 int rb_stream_step(float* res, const void* y0, int ldy0, const void* y1, int ldy1, const void* w0, const void* w1, const void* ex, int ldx, const int*
                    expert, const int* place, const int* offset, const float* weight, int top, const void* n0, const void* n1, void* h0, void* h1, const
                    void* mu, void* state, const int* slot, const int* ctx, int rows, int pitch, int width, float eps, int fp32, cudaStream_t st);
@@ -167,6 +167,13 @@ int rb_conv_inputs(const void* qkv, int ld, const void* bias, const void* taps, 
                    void* q, void* k_pool, void* v_pool, const long long* slots, const int* ctx, const int* state_slot, const int* cu, const int* seg_of,
                    const int* pos, long long pool_rows, int T, int segs, int H, int G, int dim, int vdim, int dp, int vp, int rot, float eps, int fp32,
                    cudaStream_t st);
+int rb_talk_decode_plan(int H, int G, int dk, int dv, int* value_groups);
+int rb_talk_decode(const void* q, const void* kc, const void* vc, const int* block_tables, const int* ctx_lens, const void* sink, const void* mix, void* out,
+                   float* part_o, float* part_l, int B, int H, int G, int dk, int dv, int out_d, long long pool_rows, int page, int max_blocks, int max_ctx,
+                   int window, int keep, int chunk, float scale, float cap, int splits, int* err, cudaStream_t st);
+int rb_talk_flash(const void* q, const void* kc, const void* vc, const int* block_tables, const int* ctx, const int* blocks, const void* sink, void* out,
+                  int rows, int n, int Hq, int Hkv, int dk, int dv, int out_d, long long pool_rows, int page, int max_blocks, int window, int keep, int
+                  chunk, float scale, float cap, int* err, cudaStream_t st);
 int rb_mix_heads(const void* wide, const void* mix, void* out, int rows, int H, int G, int vo, int fp32, cudaStream_t st);
 int rb_latent_write(const void* raw, const void* k_rot, void* q, int ld, const void* w, void* pool, const long long* slots, const float* table, long
                     long pool_rows, int rows, int rank, int pitch, int part, int rot, int H, int dk, int dim, float eps, int fp32, cudaStream_t st);

@@ -520,6 +520,52 @@ bool paged_decode(torch::Tensor q, torch::Tensor k, torch::Tensor v, torch::Tens
   check(rc, "rb_paged_decode_tc");
   return true;
 }
+// (packed head columns, value groups per CTA) of talk_decode for these heads; columns 0: it does not take them
+std::tuple<int64_t, int64_t> talk_decode_plan(int64_t H, int64_t G, int64_t dk, int64_t dv) {
+  int groups = 0;
+  const int cols = rb_talk_decode_plan((int)H, (int)G, (int)dk, (int)dv, &groups);
+  return {cols, groups};
+}
+// One row per sequence with mixed heads; returns false for shapes the kernel does not take.
+bool talk_decode(torch::Tensor q, torch::Tensor k, torch::Tensor v, torch::Tensor bt, torch::Tensor ctx, c10::optional<torch::Tensor> sink, torch::Tensor mix,
+                 torch::Tensor out, torch::Tensor part_o, torch::Tensor part_l, int64_t block_size, int64_t max_ctx, int64_t window, int64_t keep,
+                 int64_t chunk, int64_t splits, double scale, double cap, torch::Tensor err) {
+  const c10::cuda::CUDAGuard guard(q.device());
+  if (q.scalar_type() != at::kBFloat16) return false;
+  check_pools(q, k, v, bt, ctx, sink, out);
+  check_same(q, mix, "talk_decode");
+  const int64_t B = q.size(0), H = q.size(1), G = k.size(1);
+  int groups = 0;
+  const int64_t cols = rb_talk_decode_plan((int)H, (int)G, (int)q.size(2), (int)v.size(2), &groups);
+  if (!cols) return false;
+  TORCH_CHECK(ctx.numel() == B && mix.is_contiguous() && mix.numel() == H * H, "talk_decode: one row per sequence");
+  TORCH_CHECK(part_o.scalar_type() == at::kFloat && part_o.numel() >= B * splits * G * cols * 128 && part_l.scalar_type() == at::kFloat &&
+              part_l.numel() >= B * splits * cols, "talk_decode: scratch");
+  const int rc = rb_talk_decode(q.data_ptr(), k.data_ptr(), v.data_ptr(), bt.data_ptr<int>(), ctx.data_ptr<int>(), optptr(sink), mix.data_ptr(), out.data_ptr(),
+                                part_o.data_ptr<float>(), part_l.data_ptr<float>(), (int)B, (int)H, (int)G, (int)q.size(2), (int)v.size(2),
+                                (int)(out.size(1) / H), k.size(0), (int)block_size, (int)bt.size(1), (int)max_ctx, (int)window, (int)keep, (int)chunk,
+                                (float)scale, (float)cap, (int)splits, err.data_ptr<int>(), cur_stream());
+  if (rc == -20) return false;
+  check(rc, "rb_talk_decode");
+  return true;
+}
+// Prompt portions: every head's weights on every group's values, out [T][H G vo]; returns false for shapes the kernel does not take.
+bool talk_flash(torch::Tensor q, torch::Tensor k, torch::Tensor v, torch::Tensor bt, torch::Tensor ctx, c10::optional<torch::Tensor> blocks,
+                c10::optional<torch::Tensor> sink, torch::Tensor out, int64_t block_size, int64_t window, int64_t keep, int64_t chunk, double scale, double cap,
+                torch::Tensor err) {
+  const c10::cuda::CUDAGuard guard(q.device());
+  if (q.scalar_type() != at::kBFloat16) return false;
+  check_pools(q, k, v, bt, ctx, sink, out, true);
+  const int64_t T = q.size(0), H = q.size(1), G = k.size(1);
+  TORCH_CHECK(blocks.has_value() ? (is_i32(*blocks) && blocks->dim() == 2 && blocks->size(1) == 4) : ctx.numel() == T, "talk_flash: query tiles");
+  const int rc = rb_talk_flash(q.data_ptr(), k.data_ptr(), v.data_ptr(), bt.data_ptr<int>(), ctx.data_ptr<int>(), optint(blocks), optptr(sink), out.data_ptr(),
+                               (int)T, (int)(blocks.has_value() ? blocks->size(0) : T), (int)H, (int)G, (int)q.size(2), (int)v.size(2),
+                               (int)(out.size(1) / H / G), k.size(0), (int)block_size, (int)bt.size(1), (int)window, (int)keep, (int)chunk, (float)scale,
+                               (float)cap, err.data_ptr<int>(), cur_stream());
+  if (rc == -20) return false;
+  check(rc, "rb_talk_flash");
+  return true;
+}
 // wide [T][H G vo]: what every head's weights make of every group's values; mix [H][H]; out [T][H vo]
 void mix_heads(torch::Tensor wide, torch::Tensor mix, torch::Tensor out, int64_t kv_heads) {
   const c10::cuda::CUDAGuard guard(wide.device());
@@ -577,8 +623,7 @@ void conv_inputs(torch::Tensor qkv, c10::optional<torch::Tensor> bias, c10::opti
         "rb_conv_inputs");
 }
 void mingru(torch::Tensor rows, torch::Tensor z_b, torch::Tensor x_b, torch::Tensor state, torch::Tensor slot, torch::Tensor ctx, c10::optional<torch::Tensor> cu,
-            c10::optional<torch::Tensor> spans, c10::optional<torch::Tensor> first, c10::optional<torch::Tensor> span_sum,
-            c10::optional<torch::Tensor> span_keep, torch::Tensor out, int64_t width) {
+            torch::Tensor out, int64_t width) {
   const c10::cuda::CUDAGuard guard(rows.device());
   const int64_t pitch = (width + 7) / 8 * 8, T = rows.size(0);
   for (const auto& t : {z_b, x_b, out}) {
@@ -589,13 +634,8 @@ void mingru(torch::Tensor rows, torch::Tensor z_b, torch::Tensor x_b, torch::Ten
               x_b.numel() >= pitch && reinterpret_cast<uintptr_t>(rows.data_ptr()) % 8 == 0, "mingru: rows");
   TORCH_CHECK(state.scalar_type() == at::kFloat && state.is_contiguous() && state.dim() >= 2, "mingru: state");
   check_segments(slot, ctx, cu, T, "mingru");
-  const int64_t n = cu.has_value() ? check_spans(spans, first, slot.numel(), "mingru") : 0;
-  if (n)
-    for (const auto& o : {span_sum, span_keep}) TORCH_CHECK(o.has_value() && o->scalar_type() == at::kFloat && o->numel() >= n * pitch, "mingru: scratch");
   check(rb_mingru(rows.data_ptr(), z_b.data_ptr(), x_b.data_ptr(), state.data_ptr<float>(), slot.data_ptr<int>(), ctx.data_ptr<int>(), optint(cu),
-                  n ? spans->data_ptr<int>() : nullptr, n ? first->data_ptr<int>() : nullptr, n ? span_sum->data_ptr<float>() : nullptr,
-                  n ? span_keep->data_ptr<float>() : nullptr, out.data_ptr(), (int)slot.numel(), (int)n, (int)width, (int)rows.stride(0), (int)state.stride(0),
-                  is_fp32(rows), cur_stream()),
+                  out.data_ptr(), (int)slot.numel(), (int)width, (int)rows.stride(0), (int)state.stride(0), is_fp32(rows), cur_stream()),
         "rb_mingru");
 }
 // o_raw: scratch of the CUDA-core scan; without it segments run on the tensor cores.  Returns false for shapes those do not take.
@@ -798,6 +838,9 @@ void register_serving(pybind11::module_& m) {
   m.def("paged_flash", &paged_flash);
   m.def("dense_flash", &dense_flash);
   m.def("paged_decode", &paged_decode);
+  m.def("talk_decode_plan", &talk_decode_plan);
+  m.def("talk_decode", &talk_decode);
+  m.def("talk_flash", &talk_flash);
   m.def("mix_heads", &mix_heads);
   m.def("conv_inputs", &conv_inputs);
   m.def("mingru", &mingru);

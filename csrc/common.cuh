@@ -316,5 +316,15 @@ __device__ __forceinline__ bool sys_wait_ge(const unsigned* addr, unsigned targe
 __device__ __forceinline__ void named_bar_sync(int id, int threads) {
   asm volatile("bar.sync %0, %1;" ::"r"(id), "r"(threads) : "memory");
 }
+// the same barrier; every thread learns whether `v` held in all of them
+__device__ __forceinline__ bool named_bar_and(int id, int threads, bool v) {
+  uint32_t all;
+  asm volatile(
+      "{\n\t.reg .pred p, q;\n\tsetp.ne.u32 p, %3, 0;\n\tbar.red.and.pred q, %1, %2, p;\n\tselp.u32 %0, 1, 0, q;\n\t}"
+      : "=r"(all)
+      : "r"(id), "r"(threads), "r"(static_cast<uint32_t>(v))
+      : "memory");
+  return all != 0;
+}
 
 }  // namespace rb

@@ -215,8 +215,9 @@ __global__ void __launch_bounds__(PI_WARPS * 32) projection_inputs_kernel(const 
   }
 }
 
-// One warp per (head, run of RUN rows): raw rows slide through registers, so a run reads every row once.  Lane l holds the feature pairs
-// l, l + 32, ...  With one row per sequence the warp also moves the state on; otherwise conv_state_kernel does, afterwards.
+// One warp per (head, run of RUN rows).  Lane l holds 2 NP consecutive features; a run's raw rows and what is known about them are fetched
+// at once, and the rows slide through registers.  With one row per sequence the warp also moves the state on; otherwise
+// conv_state_kernel does, afterwards.
 struct ConvParams {
   const void* qkv;           // [T][ld]: H query heads | G key heads | G value heads (keys and values only with k_pool)
   const void* bias;          // [C] or null
@@ -238,145 +239,182 @@ struct ConvParams {
   int T, H, G, dim, vdim, dp, vp, rot, ld, n, C;
   float eps;                 // <= 0: no norm
 };
-template <typename T, bool kPair>
-__device__ __forceinline__ void load_pair(const T* p, int left, float& a, float& b) {      // `left` elements from here on
-  a = b = 0.f;
-  if constexpr (kPair) {
-    if (left > 0) {
-      if constexpr (sizeof(T) == 4) {
-        const float2 x = *reinterpret_cast<const float2*>(p);
-        a = x.x;
-        b = x.y;
+// N consecutive elements of which `left` exist (kVec: all or none, N * sizeof(T) aligned)
+template <typename T, int N, bool kVec>
+__device__ __forceinline__ void load_run(const T* p, int left, float* v) {
+#pragma unroll
+  for (int i = 0; i < N; ++i) v[i] = 0.f;
+  if constexpr (kVec) {
+    if (left <= 0) return;
+    if constexpr (sizeof(T) == 4) {
+#pragma unroll
+      for (int i = 0; i < N; i += 2) *reinterpret_cast<float2*>(v + i) = *reinterpret_cast<const float2*>(p + i);
+    } else {
+      uint32_t u[N / 2];
+      if constexpr (N % 8 == 0) {
+#pragma unroll
+        for (int i = 0; i < N / 2; i += 4) *reinterpret_cast<uint4*>(u + i) = *reinterpret_cast<const uint4*>(p + 2 * i);
+      } else if constexpr (N == 4) {
+        *reinterpret_cast<uint2*>(u) = *reinterpret_cast<const uint2*>(p);
       } else {
-        const uint32_t x = *reinterpret_cast<const uint32_t*>(p);
-        a = __uint_as_float(x << 16);
-        b = __uint_as_float(x & 0xffff0000u);
+#pragma unroll
+        for (int i = 0; i < N / 2; ++i) u[i] = *reinterpret_cast<const uint32_t*>(p + 2 * i);
+      }
+#pragma unroll
+      for (int i = 0; i < N / 2; ++i) {
+        v[2 * i] = __uint_as_float(u[i] << 16);
+        v[2 * i + 1] = __uint_as_float(u[i] & 0xffff0000u);
       }
     }
   } else {
-    if (left > 0) a = ld(p);
-    if (left > 1) b = ld(p + 1);
+#pragma unroll
+    for (int i = 0; i < N; ++i)
+      if (i < left) v[i] = ld(p + i);
   }
 }
-template <typename T, bool kPair>
-__device__ __forceinline__ void store_pair(T* p, int left, float a, float b) {
-  if constexpr (kPair) {
-    if (left > 0) {
-      if constexpr (sizeof(T) == 4) *reinterpret_cast<float2*>(p) = make_float2(a, b);
-      else *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(a, b);
+template <typename T, int N, bool kVec>
+__device__ __forceinline__ void store_run(T* p, int left, const float* v) {
+  if constexpr (kVec) {
+    if (left <= 0) return;
+    if constexpr (sizeof(T) == 4) {
+#pragma unroll
+      for (int i = 0; i < N; i += 2) *reinterpret_cast<float2*>(p + i) = *reinterpret_cast<const float2*>(v + i);
+    } else {
+      uint32_t u[N / 2];
+#pragma unroll
+      for (int i = 0; i < N / 2; ++i) {
+        const __nv_bfloat162 b = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
+        u[i] = *reinterpret_cast<const uint32_t*>(&b);
+      }
+      if constexpr (N % 8 == 0) {
+#pragma unroll
+        for (int i = 0; i < N / 2; i += 4) *reinterpret_cast<uint4*>(p + 2 * i) = *reinterpret_cast<const uint4*>(u + i);
+      } else if constexpr (N == 4) {
+        *reinterpret_cast<uint2*>(p) = *reinterpret_cast<const uint2*>(u);
+      } else {
+#pragma unroll
+        for (int i = 0; i < N / 2; ++i) *reinterpret_cast<uint32_t*>(p + 2 * i) = u[i];
+      }
     }
   } else {
-    if (left > 0) st(p, a);
-    if (left > 1) st(p + 1, b);
+#pragma unroll
+    for (int i = 0; i < N; ++i)
+      if (i < left) st(p + i, v[i]);
   }
 }
-template <typename T, int NP, int NT, int RUN, bool kPair>
+// kVec: heads, their pitches, rows and the state split into aligned runs of 2 NP features
+template <typename T, int NP, int NT, int RUN, bool kVec>
 __global__ void __launch_bounds__(256) conv_inputs_kernel(const ConvParams p) {
+  constexpr int N = 2 * NP;
   const int lane = threadIdx.x & 31;
   const int per = p.H + (p.k_pool ? 2 * p.G : 0);
   const long long u = static_cast<long long>(blockIdx.x) * 8 + (threadIdx.x >> 5);
   const long long run = u / per;
   const int hd = static_cast<int>(u - run * per);
-  const int t0 = static_cast<int>(run) * RUN, t1 = min(p.T, t0 + RUN);
-  if (t0 >= t1) return;
+  const int t0 = static_cast<int>(run) * RUN, rows = min(p.T - t0, RUN);
+  if (rows <= 0) return;
   const bool value = hd >= p.H + p.G;
   const int n = value ? p.vdim : p.dim, pitch = value ? p.vp : p.dp;
   const int g = hd - (hd < p.H ? 0 : p.H + (value ? p.G : 0));
   const int ch = (hd < p.H ? 0 : p.H * p.dim + (value ? p.G * p.dim : 0)) + g * n;      // first channel of the head
-  const T* src = static_cast<const T*>(p.qkv) + ch;
+  const int e = N * lane, left = n - e;
+  const T* src = static_cast<const T*>(p.qkv) + ch + e;
   const bool normed = !value && p.eps > 0.f;
-  float w[NP][2][NT], bias[NP][2], nw[NP][2];
-#pragma unroll
-  for (int i = 0; i < NP; ++i) {
-    const int e = 2 * (lane + 32 * i), left = n - e;
-#pragma unroll
-    for (int k = 0; k < NT; ++k) w[i][0][k] = w[i][1][k] = 0.f;
-    if (p.taps) {
-      const T* tp = static_cast<const T*>(p.taps) + static_cast<long long>(ch + e) * p.n;
-#pragma unroll
-      for (int k = 0; k < NT; ++k)
-        if (k < p.n) {
-          if (left > 0) w[i][0][k] = ld(tp + p.n - 1 - k);
-          if (left > 1) w[i][1][k] = ld(tp + 2 * p.n - 1 - k);
-        }
-    } else {
-      w[i][0][0] = w[i][1][0] = 1.f;
-    }
-    bias[i][0] = bias[i][1] = 0.f;
-    nw[i][0] = nw[i][1] = 1.f;
-    if (p.bias) load_pair<T, false>(static_cast<const T*>(p.bias) + ch + e, left, bias[i][0], bias[i][1]);
-    if (normed) load_pair<T, false>(static_cast<const T*>(hd < p.H ? p.q_w : p.k_w) + e, left, nw[i][0], nw[i][1]);
+  // what is known about the rows: lane i holds it for row t0 + i
+  int m_seg = 0, m_at = 0, m_first = 0, m_state = 0;
+  long long m_slot = 0;
+  if (lane < rows) {
+    const int t = t0 + lane;
+    m_seg = p.cu ? p.seg_of[t] : t;
+    m_at = p.cu ? p.pos[t] : p.ctx[t] - 1;
+    m_first = p.cu ? p.cu[m_seg] : t;
+    m_state = p.state_slot[m_seg];
+    if (hd >= p.H) m_slot = p.slots[t];
   }
-  float past[NP][2][NT > 1 ? NT - 1 : 1];      // raw rows t - 1, t - 2, ...
+  float x[RUN][N];
+#pragma unroll
+  for (int k = 0; k < RUN; ++k) {
+    if (k < rows) load_run<T, N, kVec>(src + static_cast<long long>(t0 + k) * p.ld, left, x[k]);
+  }
+  float w[NT][N], bias[N], nw[N];
+#pragma unroll
+  for (int i = 0; i < N; ++i) {
+#pragma unroll
+    for (int k = 0; k < NT; ++k) w[k][i] = 0.f;
+    w[0][i] = 1.f;
+    bias[i] = 0.f;
+    nw[i] = 1.f;
+    if (i < left) {
+      if (p.taps) {
+        const T* tp = static_cast<const T*>(p.taps) + static_cast<long long>(ch + e + i) * p.n;
+#pragma unroll
+        for (int k = 0; k < NT; ++k)
+          if (k < p.n) w[k][i] = ld(tp + p.n - 1 - k);
+      }
+      if (p.bias) bias[i] = ld(static_cast<const T*>(p.bias) + ch + e + i);
+      if (normed) nw[i] = ld(static_cast<const T*>(hd < p.H ? p.q_w : p.k_w) + e + i);
+    }
+  }
+  float past[NT > 1 ? NT - 1 : 1][N];      // raw rows t - 1, t - 2, ...
   int seg = -1;
-  for (int t = t0; t < t1; ++t) {
-    const int s = p.cu ? p.seg_of[t] : t, at = p.cu ? p.pos[t] : p.ctx[t] - 1, local = p.cu ? t - p.cu[s] : 0;
-    T* state = p.n > 1 ? static_cast<T*>(p.state) + static_cast<long long>(p.state_slot[s]) * (p.n - 1) * p.C + ch : nullptr;
+#pragma unroll
+  for (int k = 0; k < RUN; ++k) {
+    if (k >= rows) break;
+    const int t = t0 + k;
+    const int s = __shfl_sync(0xffffffffu, m_seg, k), at = __shfl_sync(0xffffffffu, m_at, k), local = t - __shfl_sync(0xffffffffu, m_first, k);
+    const int place = __shfl_sync(0xffffffffu, m_state, k);
+    const long long slot = __shfl_sync(0xffffffffu, m_slot, k);
+    T* state = p.n > 1 ? static_cast<T*>(p.state) + static_cast<long long>(place) * (p.n - 1) * p.C + ch + e : nullptr;
     if (s != seg) {
       seg = s;
 #pragma unroll
-      for (int k = 1; k < NT; ++k) {
-        const T* from = k <= local ? src + static_cast<long long>(t - k) * p.ld : state + static_cast<long long>(p.n - 1 - (k - local)) * p.C;
-#pragma unroll
-        for (int i = 0; i < NP; ++i) {
-          const int e = 2 * (lane + 32 * i);
-          past[i][0][k - 1] = past[i][1][k - 1] = 0.f;
-          if (k < p.n && k <= at) load_pair<T, kPair>(from + e, n - e, past[i][0][k - 1], past[i][1][k - 1]);
-        }
+      for (int b = 1; b < NT; ++b) {
+        const T* from = b <= local ? src + static_cast<long long>(t - b) * p.ld : state + static_cast<long long>(p.n - 1 - (b - local)) * p.C;
+        load_run<T, N, kVec>(from, b < p.n && b <= at ? left : 0, past[b - 1]);
       }
     }
-    float y[NP][2], ss = 0.f;
+    if (!p.cu && p.n > 1) {      // the state moves on by one row
 #pragma unroll
-    for (int i = 0; i < NP; ++i) {
-      const int e = 2 * (lane + 32 * i);
-      float x[2];
-      load_pair<T, kPair>(src + static_cast<long long>(t) * p.ld + e, n - e, x[0], x[1]);
-      if (!p.cu && p.n > 1) {      // the state moves on by one row
+      for (int b = NT - 1; b >= 1; --b)
+        if (b < p.n) store_run<T, N, kVec>(state + static_cast<long long>(p.n - 1 - b) * p.C, left, b > 1 ? past[b > 1 ? b - 2 : 0] : x[k]);
+    }
+    float y[N], ss = 0.f;
 #pragma unroll
-        for (int k = NT - 1; k >= 1; --k)
-          if (k < p.n) store_pair<T, kPair>(state + static_cast<long long>(p.n - 1 - k) * p.C + e, n - e, k > 1 ? past[i][0][k > 1 ? k - 2 : 0] : x[0],
-                                            k > 1 ? past[i][1][k > 1 ? k - 2 : 0] : x[1]);
-      }
+    for (int i = 0; i < N; ++i) {
+      float a = w[0][i] * (x[k][i] + bias[i]);
 #pragma unroll
-      for (int h = 0; h < 2; ++h) {
-        float a = w[i][h][0] * (x[h] + bias[i][h]);
+      for (int b = 1; b < NT; ++b)
+        if (b <= at) a += w[b][i] * (past[b - 1][i] + bias[i]);      // (taps behind the last one are zero)
 #pragma unroll
-        for (int k = 1; k < NT; ++k)
-          if (k <= at) a += w[i][h][k] * (past[i][h][k - 1] + bias[i][h]);      // (taps behind the last one are zero)
-#pragma unroll
-        for (int k = NT - 1; k > 1; --k) past[i][h][k - 1] = past[i][h][k - 2];
-        if (NT > 1) past[i][h][0] = x[h];
-        y[i][h] = a;
-        ss += a * a;
-      }
+      for (int b = NT - 1; b > 1; --b) past[b - 1][i] = past[b - 2][i];
+      if (NT > 1) past[0][i] = x[k][i];
+      y[i] = a;
+      ss += a * a;
     }
     if (normed) {
       const float r = 1.f / sqrtf(wsum(ss) / p.dim + p.eps);
 #pragma unroll
-      for (int i = 0; i < NP; ++i) {
-        y[i][0] *= r * nw[i][0];
-        y[i][1] *= r * nw[i][1];
-      }
+      for (int i = 0; i < N; ++i) y[i] *= r * nw[i];
     }
     T* dst;
     if (hd < p.H) {
       dst = static_cast<T*>(p.q) + (static_cast<long long>(t) * p.H + hd) * p.dp;
     } else {
-      const long long slot = p.slots[t];
       if (slot < 0 || slot >= p.pool_rows) continue;
       dst = static_cast<T*>(value ? p.v_pool : p.k_pool) + (slot * p.G + g) * pitch;
     }
+    if (!value && e < p.rot) {
+      const float2* cs = p.table + static_cast<long long>(t) * (p.rot >> 1) + (e >> 1);
 #pragma unroll
-    for (int i = 0; i < NP; ++i) {      // columns behind the head's features are written as zeros
-      const int e = 2 * (lane + 32 * i);
-      if (!value && e < p.rot) {
-        const float2 cs = p.table[static_cast<long long>(t) * (p.rot >> 1) + (e >> 1)];
-        const float a = y[i][0] * cs.x - y[i][1] * cs.y;
-        y[i][1] = y[i][1] * cs.x + y[i][0] * cs.y;
-        y[i][0] = a;
-      }
-      store_pair<T, true>(dst + e, pitch - e, y[i][0], y[i][1]);
+      for (int i = 0; i < N; i += 2)
+        if (e + i < p.rot) {
+          const float2 f = cs[i >> 1];
+          const float a = y[i] * f.x - y[i + 1] * f.y;
+          y[i + 1] = y[i + 1] * f.x + y[i] * f.y;
+          y[i] = a;
+        }
     }
+    store_run<T, N, kVec>(dst + e, pitch - e, y);      // columns behind the head's features are written as zeros
   }
 }
 
@@ -399,14 +437,14 @@ __global__ void __launch_bounds__(256) conv_state_kernel(const ConvParams p) {
 }
 
 // out[t][h] = sum over g of mix[h][g] wide[t][g][group of h]: `wide` holds what every head's weights make of every group's values.
-// Thread = (token, four heads of one group, V columns).
-template <typename T, int V>
+// Any type: thread = (token, four heads of one group, eight columns).
+template <typename T>
 __global__ void __launch_bounds__(128) mix_heads_kernel(const T* __restrict__ wide, const T* __restrict__ mix, T* __restrict__ out, long long units, int H,
                                                         int G, int vo) {
   const long long u = static_cast<long long>(blockIdx.x) * 128 + threadIdx.x;
   if (u >= units) return;
-  const int cols = vo / V, rep = H / G, quads = (rep + 3) / 4;
-  const int c = static_cast<int>(u % cols) * V;
+  const int cols = vo / 8, rep = H / G, quads = (rep + 3) / 4;
+  const int c = static_cast<int>(u % cols) * 8;
   long long r = u / cols;
   const int quad = static_cast<int>(r % quads) * 4;
   r /= quads;
@@ -414,25 +452,90 @@ __global__ void __launch_bounds__(128) mix_heads_kernel(const T* __restrict__ wi
   const long long t = r / G;
   const T* src = wide + (t * H * G + grp) * vo + c;
   const T* m = mix + static_cast<long long>(grp * rep + quad) * H;
-  float acc[4][V];
+  float acc[4][8];
 #pragma unroll
   for (int i = 0; i < 4; ++i)
 #pragma unroll
-    for (int j = 0; j < V; ++j) acc[i][j] = 0.f;
+    for (int j = 0; j < 8; ++j) acc[i][j] = 0.f;
 #pragma unroll 4
   for (int g = 0; g < H; ++g) {
-    float a[V];
-    ldv<V>(src + static_cast<long long>(g) * G * vo, a);
+    float a[8];
+    ldv<8>(src + static_cast<long long>(g) * G * vo, a);
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
       const float f = quad + i < rep ? ld(m + i * H + g) : 0.f;
 #pragma unroll
-      for (int j = 0; j < V; ++j) acc[i][j] += f * a[j];
+      for (int j = 0; j < 8; ++j) acc[i][j] += f * a[j];
     }
   }
 #pragma unroll
   for (int i = 0; i < 4; ++i)
-    if (quad + i < rep) stv<V>(out + (t * H + grp * rep + quad + i) * vo + c, acc[i]);
+    if (quad + i < rep) stv<8>(out + (t * H + grp * rep + quad + i) * vo + c, acc[i]);
+}
+
+// bf16, up to 16 heads per group: warp = (token, group, 64 columns), one m16n8k16 product per 16 heads g and 8 columns.  This pass is bound by
+// reading `wide`, and what its products need of the tensor cores is a few of these per 16-byte load.  A lane fetches 8 consecutive columns of
+// the rows g that its fragments hold; which columns form a product's eight is free, so column j of every lane quarter's run goes to product j.
+template <int KS>
+__global__ void __launch_bounds__(256) mix_heads_mma_kernel(const __nv_bfloat16* __restrict__ wide, const __nv_bfloat16* __restrict__ mix,
+                                                            __nv_bfloat16* __restrict__ out, int tokens, int H, int G, int vo) {
+  const int lane = threadIdx.x & 31, q = lane >> 2, k2 = (lane & 3) * 2;
+  const int runs = (vo + 63) / 64, rep = H / G;
+  const int grp = blockIdx.y / runs, c = (blockIdx.y % runs) * 64 + q * 8;
+  const long long row = static_cast<long long>(G) * vo;      // elements between two heads g
+  uint32_t a[KS][4];                                         // rows: heads of the group, columns: heads g
+#pragma unroll
+  for (int s = 0; s < KS; ++s)
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int h = q + (i & 1) * 8, g = s * 16 + k2 + (i >> 1) * 8;
+      const __nv_bfloat16* m = mix + static_cast<long long>(grp * rep + h) * H + g;
+      const uint32_t lo = h < rep && g < H ? __bfloat16_as_ushort(m[0]) : 0, hi = h < rep && g + 1 < H ? __bfloat16_as_ushort(m[1]) : 0;
+      a[s][i] = lo | hi << 16;
+    }
+  for (int t = blockIdx.x * 8 + (threadIdx.x >> 5); t < tokens; t += gridDim.x * 8) {
+    const __nv_bfloat16* src = wide + static_cast<long long>(t) * H * row + static_cast<long long>(grp) * vo + c;
+    uint4 x[KS][4];
+#pragma unroll
+    for (int s = 0; s < KS; ++s)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const int g = s * 16 + k2 + (i & 1) + (i >> 1) * 8;
+        x[s][i] = make_uint4(0, 0, 0, 0);
+        if (g < H && c < vo) x[s][i] = __ldcs(reinterpret_cast<const uint4*>(src + g * row));
+      }
+    float d[8][4];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) d[j][e] = 0.f;
+#pragma unroll
+      for (int s = 0; s < KS; ++s) {
+        const uint32_t* w0 = reinterpret_cast<const uint32_t*>(&x[s][0]) + (j >> 1);
+        uint32_t b[2];
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {      // heads g and g + 1 of column j
+          const uint32_t lo = w0[i * 8], hi = w0[i * 8 + 4];
+          b[i] = (j & 1) ? __byte_perm(lo, hi, 0x7632) : __byte_perm(lo, hi, 0x5410);
+        }
+        asm volatile(
+            "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+            : "+f"(d[j][0]), "+f"(d[j][1]), "+f"(d[j][2]), "+f"(d[j][3])
+            : "r"(a[s][0]), "r"(a[s][1]), "r"(a[s][2]), "r"(a[s][3]), "r"(b[0]), "r"(b[1]));
+      }
+    }
+    // d[j][e]: head q + (e / 2) 8, column j of the run of lane quarter k2 + (e & 1)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int h = q + (e >> 1) * 8, col = (blockIdx.y % runs) * 64 + (k2 + (e & 1)) * 8;
+      if (h < rep && col < vo) {
+        F8 o;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) o.v[j] = d[j][e];
+        st8(out + (static_cast<long long>(t) * H + grp * rep + h) * vo + col, o);
+      }
+    }
+  }
 }
 
 // CTA = (row, head), every warp walks every fourth visible position, a lane holds NR features of query, accumulator, key and
@@ -534,7 +637,12 @@ static int launch_inputs(const InputParams& p, cudaStream_t stm) {
 }
 
 template <typename T, int NP, int NT>
-static int launch_conv_np(const ConvParams& p, bool pair, int segs, cudaStream_t stm) {
+static int launch_conv_np(const ConvParams& p, int segs, cudaStream_t stm) {
+  constexpr int N = 2 * NP, bytes = sizeof(T) == 4 ? 8 : (N % 8 == 0 ? 16 : 2 * N);      // what a lane loads at once
+  const bool pair = p.dim % N == 0 && p.dp % N == 0 && p.ld * sizeof(T) % bytes == 0 && p.C * sizeof(T) % bytes == 0 &&
+                    (!p.k_pool || (p.vdim % N == 0 && p.vp % N == 0)) &&
+                    (reinterpret_cast<uintptr_t>(p.qkv) | reinterpret_cast<uintptr_t>(p.state) | reinterpret_cast<uintptr_t>(p.q) |
+                     reinterpret_cast<uintptr_t>(p.k_pool) | reinterpret_cast<uintptr_t>(p.v_pool)) % 16 == 0;
   const int run = p.cu ? 8 : 1;
   const long long units = static_cast<long long>((p.T + run - 1) / run) * (p.H + (p.k_pool ? 2 * p.G : 0));
   const unsigned grid = static_cast<unsigned>((units + 7) / 8);
@@ -551,12 +659,12 @@ static int launch_conv_np(const ConvParams& p, bool pair, int segs, cudaStream_t
   return static_cast<int>(cudaGetLastError());
 }
 template <typename T, int NT>
-static int launch_conv(const ConvParams& p, bool pair, int segs, cudaStream_t stm) {
+static int launch_conv(const ConvParams& p, int segs, cudaStream_t stm) {
   const int w = p.k_pool ? (p.dp > p.vp ? p.dp : p.vp) : p.dp;
-  if (w <= 64) return launch_conv_np<T, 1, NT>(p, pair, segs, stm);
-  if (w <= 128) return launch_conv_np<T, 2, NT>(p, pair, segs, stm);
-  if (w <= 256) return launch_conv_np<T, 4, NT>(p, pair, segs, stm);
-  if (w <= 512) return launch_conv_np<T, 8, NT>(p, pair, segs, stm);
+  if (w <= 64) return launch_conv_np<T, 1, NT>(p, segs, stm);
+  if (w <= 128) return launch_conv_np<T, 2, NT>(p, segs, stm);
+  if (w <= 256) return launch_conv_np<T, 4, NT>(p, segs, stm);
+  if (w <= 512) return launch_conv_np<T, 8, NT>(p, segs, stm);
   return -2;
 }
 
@@ -640,19 +748,27 @@ extern "C" int rb_conv_inputs(const void* qkv, int ld, const void* bias, const v
   if (eps > 0.f && (!q_w || (k_pool && !k_w))) return -2;
   ConvParams p{qkv, bias, taps, state, q_w, k_w, reinterpret_cast<const float2*>(table), q, k_pool, v_pool, slots, ctx, state_slot, cu, seg_of, pos,
                pool_rows, T, H, G, dim, vdim, dp, vp, rot, ld, n, C, eps};
-  const bool pair = dim % 2 == 0 && (!k_pool || vdim % 2 == 0) && ld % 2 == 0 && (reinterpret_cast<uintptr_t>(qkv) | reinterpret_cast<uintptr_t>(state)) % 8 == 0;
-  if (fp32) return n <= 4 ? launch_conv<float, 4>(p, pair, segs, stm) : launch_conv<float, 8>(p, pair, segs, stm);
-  return n <= 4 ? launch_conv<bf16, 4>(p, pair, segs, stm) : launch_conv<bf16, 8>(p, pair, segs, stm);
+  if (fp32) return n <= 4 ? launch_conv<float, 4>(p, segs, stm) : launch_conv<float, 8>(p, segs, stm);
+  return n <= 4 ? launch_conv<bf16, 4>(p, segs, stm) : launch_conv<bf16, 8>(p, segs, stm);
 }
 
 // wide [rows][H][G][vo], mix [H][H], out [rows][H][vo]
 extern "C" int rb_mix_heads(const void* wide, const void* mix, void* out, int rows, int H, int G, int vo, int fp32, cudaStream_t stm) {
   if (rows <= 0) return 0;
   if (G < 1 || H % G || vo % 8 || vo < 8) return -2;
+  const int ks = (H + 15) / 16, groups = G * ((vo + 63) / 64);
+  if (!fp32 && H / G <= 16 && ks <= 4 && groups <= 65535) {
+    const int blocks = (rows + 7) / 8, most = (num_sms() * 16 + groups - 1) / groups;
+    const dim3 grid(blocks < most ? blocks : most, groups);
+    auto k = ks == 1 ? mix_heads_mma_kernel<1> : ks == 2 ? mix_heads_mma_kernel<2> : ks == 3 ? mix_heads_mma_kernel<3> : mix_heads_mma_kernel<4>;
+    k<<<grid, 256, 0, stm>>>((const bf16*)wide, (const bf16*)mix, (bf16*)out, rows, H, G, vo);
+    rb_note_launch(1);
+    return static_cast<int>(cudaGetLastError());
+  }
   const long long units = static_cast<long long>(rows) * G * ((H / G + 3) / 4) * (vo / 8);
   const unsigned grid = static_cast<unsigned>((units + 127) / 128);
-  if (fp32) mix_heads_kernel<float, 8><<<grid, 128, 0, stm>>>((const float*)wide, (const float*)mix, (float*)out, units, H, G, vo);
-  else mix_heads_kernel<bf16, 8><<<grid, 128, 0, stm>>>((const bf16*)wide, (const bf16*)mix, (bf16*)out, units, H, G, vo);
+  if (fp32) mix_heads_kernel<float><<<grid, 128, 0, stm>>>((const float*)wide, (const float*)mix, (float*)out, units, H, G, vo);
+  else mix_heads_kernel<bf16><<<grid, 128, 0, stm>>>((const bf16*)wide, (const bf16*)mix, (bf16*)out, units, H, G, vo);
   rb_note_launch(1);
   return static_cast<int>(cudaGetLastError());
 }

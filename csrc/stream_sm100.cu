@@ -204,22 +204,27 @@ __global__ void __launch_bounds__(256) token_shift_kernel(const TokenShiftParams
   }
 }
 
-template <typename T>
-__global__ void side_gate_kernel(const T* __restrict__ z, int ldz, const T* __restrict__ embed, long long lde, const long long* __restrict__ tok, int vocab,
-                                 T* __restrict__ out, int rows, int dim, int pitch) {
+template <typename T, int V>
+__global__ void __launch_bounds__(256) side_gate_kernel(const T* __restrict__ z, int ldz, const T* __restrict__ embed, long long lde, const long long* __restrict__ tok,
+                                                        int vocab, T* __restrict__ out, int rows, int dim, int pitch) {
   constexpr bool kExact = IsExact<T>::v;
-  const long long i = static_cast<long long>(blockIdx.x) * blockDim.x + threadIdx.x;
+  const long long i = (static_cast<long long>(blockIdx.x) * 256 + threadIdx.x) * V;
   if (i >= static_cast<long long>(rows) * pitch) return;
   const long long t = i / pitch;
   const int c = static_cast<int>(i - t * pitch);
   const long long id = tok[t];
-  float v = 0.f;
+  float v[V];
+#pragma unroll
+  for (int k = 0; k < V; ++k) v[k] = 0.f;
   if (c < dim && id >= 0 && id < vocab) {
-    const float g = ld(z + t * ldz + c);
-    // 0.5 (1 + tanh(u)) = sigmoid(2 u)
-    v = g * sigmoid<kExact>(1.5957691216057308f * (g + 0.044715f * g * g * g)) * ld(embed + id * lde + c);      // 2 sqrt(2 / pi)
+    float g[V], e[V];
+    ldv<V>(z + t * ldz + c, g);
+    ldv<V>(embed + id * lde + c, e);
+#pragma unroll
+    for (int k = 0; k < V; ++k)      // 0.5 (1 + tanh(u)) = sigmoid(2 u); 2 sqrt(2 / pi)
+      v[k] = g[k] * sigmoid<kExact>(1.5957691216057308f * (g[k] + 0.044715f * g[k] * g[k] * g[k])) * e[k];
   }
-  st(out + i, v);
+  stv<V>(out + i, v);
 }
 
 __global__ void softcap_kernel(float* __restrict__ z, long long n4, float cap) {
@@ -282,10 +287,16 @@ extern "C" int rb_side_gate(const void* z, int ldz, const void* embed, long long
                             int pitch, int fp32, cudaStream_t stm) {
   if (rows <= 0) return 0;
   if (dim < 1 || pitch < dim || ldz < dim || lde < dim) return -2;
-  const long long n = static_cast<long long>(rows) * pitch;
+  const bool vec = dim % 8 == 0 && ldz % 8 == 0 && lde % 8 == 0 &&
+                   (reinterpret_cast<uintptr_t>(z) | reinterpret_cast<uintptr_t>(embed) | reinterpret_cast<uintptr_t>(out)) % 16 == 0;
+  const long long n = static_cast<long long>(rows) * pitch / (vec ? 8 : 1);
   const unsigned grid = static_cast<unsigned>((n + 255) / 256);
-  if (fp32) side_gate_kernel<float><<<grid, 256, 0, stm>>>((const float*)z, ldz, (const float*)embed, lde, tok, vocab, (float*)out, rows, dim, pitch);
-  else side_gate_kernel<bf16><<<grid, 256, 0, stm>>>((const bf16*)z, ldz, (const bf16*)embed, lde, tok, vocab, (bf16*)out, rows, dim, pitch);
+  auto run = [&](auto kernel, auto type) {
+    using T = decltype(type);
+    kernel<<<grid, 256, 0, stm>>>((const T*)z, ldz, (const T*)embed, lde, tok, vocab, (T*)out, rows, dim, pitch);
+  };
+  if (fp32) vec ? run(side_gate_kernel<float, 8>, float()) : run(side_gate_kernel<float, 1>, float());
+  else vec ? run(side_gate_kernel<bf16, 8>, bf16()) : run(side_gate_kernel<bf16, 1>, bf16());
   rb_note_launch(1);
   return static_cast<int>(cudaGetLastError());
 }

@@ -22,7 +22,8 @@ SO_PATH = os.path.join(ROOT, "relax_b200", "_C.so")
 SERVING_SO_PATH = os.path.join(ROOT, "relax_b200", "_C_serving.so")
 SERVING_SOURCES = ["attention_fwd_sm100.cu", "decode_attn_tc_sm100.cu", "decode_step_sm100.cu", "gemm2_sm100.cu", "gemm_decode_sm100.cu", "gemm_sm100.cu",
                    "gqa_stack_sm100.cu", "head_gemm_sm100.cu", "hgrn2_chunk_sm100.cu", "latent_attn_sm100.cu", "mingru_sm100.cu", "moe_gemm_sm100.cu",
-                   "moe_stack_sm100.cu", "paged_flash_sm100.cu", "stack_sm100.cu", "stream_sm100.cu", "bindings_serving.cpp", "launch_count.cpp", "module_serving.cpp"]
+                   "moe_stack_sm100.cu", "paged_flash_sm100.cu", "stack_sm100.cu", "stream_sm100.cu", "talk_decode_sm100.cu", "talk_flash_sm100.cu",
+                   "bindings_serving.cpp", "launch_count.cpp", "module_serving.cpp"]
 # fp32 results of these kernels are compared at fp32 rounding: IEEE division, square root and library exponentials
 PRECISE_SOURCES = {"stack_sm100.cu", "gqa_stack_sm100.cu", "mingru_sm100.cu", "moe_stack_sm100.cu", "stream_sm100.cu"}
 

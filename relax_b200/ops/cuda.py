@@ -395,25 +395,26 @@ def decode_splits(rows: int, kv_heads: int, max_ctx: int) -> int:
 
 def paged_attention(q, k_pool, v_pool, b, block_size, scale, sink, out_width, window=0, gate=None, keep=0, chunk=0, softcap=0.0, talk=None):
     """bf16 heads of up to 128 features: segments of several rows on the flash kernel, single rows on the decode kernel (the
-    flash kernel when more than 16 heads share keys); anything else, and fp32, on CUDA cores.  With ``talk`` every head's weights meet the
-    values of every group, and the outputs are mixed: ``sum_g T[h, g] (P_g V) = (sum_g T[h, g] P_g) V``."""
+    flash kernel when more than 16 heads share keys); anything else, and fp32, on CUDA cores."""
+    if talk is not None:
+        return _mixed_attention(q, k_pool, v_pool, b, block_size, scale, sink, out_width, window, keep, chunk, softcap, talk)
     T, H, dp = q.shape
     G = k_pool.shape[1]
-    L, err, wide = _load(), err_flag(q.device), talk is not None
-    out = torch.empty(T, H * out_width * (G if wide else 1), dtype=q.dtype, device=q.device)
+    L, err = _load(), err_flag(q.device)
+    out = torch.empty(T, H * out_width, dtype=q.dtype, device=q.device)
     n, s = (0, 0) if b.cu is None else (b.multi_rows, b.multi_segs)
     see = (int(window), int(keep), int(chunk))
 
     def tensor_cores() -> bool:
         if n and not L.paged_flash(q[:n], k_pool, v_pool, b.block_tables, b.ctx, b.blocks[128 // (H // G)], sink, None if gate is None else gate[:n], out[:n],
-                                   int(block_size), *see, wide, float(scale), float(softcap), err):
+                                   int(block_size), *see, False, float(scale), float(softcap), err):
             return False
         if n == T:
             return True
         bt, ctx, g = b.block_tables[s:], b.ctx[s:], None if gate is None else gate[n:]
-        if H // G > 16 or wide:
-            return L.paged_flash(q[n:], k_pool, v_pool, bt, ctx, None, sink, g, out[n:], int(block_size), *see, wide, float(scale), float(softcap), err)
-        most = min(b.max_ctx_one, chunk + block_size if chunk else window + keep + 2 * block_size if window else b.max_ctx_one)
+        if H // G > 16:
+            return L.paged_flash(q[n:], k_pool, v_pool, bt, ctx, None, sink, g, out[n:], int(block_size), *see, False, float(scale), float(softcap), err)
+        most = _most_seen(b.max_ctx_one, block_size, *see)
         splits = decode_splits(T - n, G, most)
         po = ml = None
         if splits > 1:
@@ -423,12 +424,54 @@ def paged_attention(q, k_pool, v_pool, b, block_size, scale, sink, out_width, wi
                               float(softcap), err)
 
     if not (q.dtype == torch.bfloat16 and max(dp, v_pool.shape[2]) <= 128 and H // G <= 128 and tensor_cores()):
-        L.gqa_attn(q, k_pool, v_pool, b.block_tables, b.seg_of, b.pos, b.ctx, sink, gate, out, int(block_size), *see, wide, float(scale), float(softcap))
-    if not wide:
+        L.gqa_attn(q, k_pool, v_pool, b.block_tables, b.seg_of, b.pos, b.ctx, sink, gate, out, int(block_size), *see, False, float(scale), float(softcap))
+    return out
+
+
+def _most_seen(max_ctx: int, page: int, window: int, keep: int, chunk: int) -> int:
+    """Most positions that a single row sees, pages that count in part as a whole."""
+    return min(max_ctx, chunk + page if chunk else window + keep + 2 * page if window else max_ctx)
+
+
+def _mixed_attention(q, k_pool, v_pool, b, block_size, scale, sink, out_width, window, keep, chunk, softcap, talk):
+    """Heads whose weights are mixed: ``sum_g T[h, g] (P_g V) = (sum_g T[h, g] P_g) V``, so every head's weights meet the values of every
+    group, and the outputs are mixed (single rows: when the splits are merged).  Capped scores (caps up to 80) have kernels that keep
+    several groups' accumulators; the others take the flash kernel once per group."""
+    T, H, dp = q.shape
+    G, dv = k_pool.shape[1], v_pool.shape[2]
+    L, err = _load(), err_flag(q.device)
+    out = torch.empty(T, H * out_width, dtype=q.dtype, device=q.device)
+    n, s = (0, 0) if b.cu is None else (b.multi_rows, b.multi_segs)
+    see, fl = (int(window), int(keep), int(chunk)), (float(scale), float(softcap))
+    tensor = q.dtype == torch.bfloat16 and max(dp, dv) <= 128 and H // G <= 128
+    done = T                                     # rows that are still to do: in front of here
+    if tensor and n < T and 0 < softcap <= 80:
+        cols, groups = L.talk_decode_plan(H, G, dp, dv)
+        if cols:
+            most = _most_seen(b.max_ctx_one, block_size, *see)
+            splits = max(1, min(148 // ((T - n) * -(-G // groups)), -(-most // 128)))      # one CTA per SM; tiles of 128 positions
+            po = torch.empty((T - n) * splits * G * cols * 128, dtype=torch.float32, device=q.device)
+            pl = torch.empty((T - n) * splits * cols, dtype=torch.float32, device=q.device)
+            if L.talk_decode(q[n:], k_pool, v_pool, b.block_tables[s:], b.ctx[s:], sink, talk, out[n:], po, pl, int(block_size), int(most), *see, splits, *fl, err):
+                done = n
+    if done == 0:
         return out
-    mixed = torch.empty(T, H * out_width, dtype=q.dtype, device=q.device)
-    L.mix_heads(out, talk, mixed, G)
-    return mixed
+    wide = torch.empty(done, H * G * out_width, dtype=q.dtype, device=q.device)
+
+    def flash(lo, hi, bt, ctx, blocks) -> bool:
+        a = (q[lo:hi], k_pool, v_pool, bt, ctx, blocks, sink)
+        if 0 < softcap <= 80 and L.talk_flash(*a, wide[lo:hi], int(block_size), *see, *fl, err):
+            return True
+        return L.paged_flash(*a, None, wide[lo:hi], int(block_size), *see, True, *fl, err)
+
+    if not (tensor and (n == 0 or flash(0, n, b.block_tables, b.ctx, b.blocks[128 // (H // G)])) and
+            (done == n or flash(n, done, b.block_tables[s:], b.ctx[s:], None))):
+        if done < T:      # (single rows are done, the segments of several rows are not)
+            L.gqa_attn(q[:n], k_pool, v_pool, b.block_tables, b.seg_of[:n], b.pos[:n], b.ctx, sink, None, wide, int(block_size), *see, True, *fl)
+        else:
+            L.gqa_attn(q, k_pool, v_pool, b.block_tables, b.seg_of, b.pos, b.ctx, sink, None, wide, int(block_size), *see, True, *fl)
+    L.mix_heads(wide, talk, out[:done], G)
+    return out
 
 
 class ExpertPlan:
@@ -493,13 +536,8 @@ def hgrn2(qfv, f_bias, lower, norm_w, state, state_slot, ctx_lens, cu, heads, di
 
 
 def mingru(zxg, z_b, x_b, state, b, width):
-    T, n = zxg.shape[0], (width + 7) // 8 * 8
-    out = torch.empty(T, n, dtype=zxg.dtype, device=zxg.device)
-    spans, first = b.mean_spans if b.mean_spans is not None else (None, None)
-    total = keep = None
-    if spans is not None:
-        total, keep = (torch.empty(spans.shape[0], n, dtype=torch.float32, device=zxg.device) for _ in range(2))
-    _load().mingru(zxg, z_b, x_b, state, b.state_slot, b.ctx, b.cu, spans, first, total, keep, out, int(width))
+    out = torch.empty(zxg.shape[0], (width + 7) // 8 * 8, dtype=zxg.dtype, device=zxg.device)
+    _load().mingru(zxg, z_b, x_b, state, b.state_slot, b.ctx, b.cu, out, int(width))
     return out
 
 

@@ -398,7 +398,7 @@ def zoguzen_kernel_rows(W=2048, H=32, G=4, d=128, chunk=1024, Hl=16, Hr=16, dk=6
     """The kernels of one real-sized Zoguzen layer of each kind, each beside the like kernel of Zupupel or Talizen stacks."""
     from .. import ops
     from ..models.config import LayerSpec, MoESpec
-    from .composed import ComposedForward, SegmentBatch, mean_spans, query_blocks, recurrent_spans, tile_tokens
+    from .composed import ComposedForward, SegmentBatch, query_blocks, recurrent_spans, tile_tokens
 
     dev, bf = "cuda", torch.bfloat16
     rows = []
@@ -487,7 +487,7 @@ def zoguzen_kernel_rows(W=2048, H=32, G=4, d=128, chunk=1024, Hl=16, Hr=16, dk=6
         rows.append(("  like: hgrn2 of a prompt (Talizen)", f"{S} x {L}", _time([_graph(lambda: ops.hgrn2(q, fb, lower, nw, state, ids, ctx, cu, Hr, dk, d, 1e-6, spans))], 10),
                      T * Hr * (2 * dk + 2 * d) * 2, 6.0 * T * Hr * dk * d))
         xs, mean = [mk(T, 3 * width) for _ in range(2)], torch.zeros(S, 1, 1, width, device=dev)
-        b = SegmentBatch(None, None, ctx, None, ids, cu=cu, mean_spans=both(mean_spans([L] * S)))
+        b = SegmentBatch(None, None, ctx, None, ids, cu=cu)
         rows.append(("running mean of a prompt", f"{S} x {L}", _time([_graph(lambda x=x: ops.mingru(x, zb, zw, mean, b, width)) for x in xs], 10), T * width * 8, None))
         del xs
     mine = MoESpec(experts=E, top=k, ff=F, act="swiglu", score="softmax", renormalize=True)

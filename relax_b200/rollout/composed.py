@@ -158,7 +158,6 @@ class SegmentBatch:
     items: Optional[dict] = None
     item_width: Optional[dict] = None
     spans: Optional[tuple] = None            # row ranges of recurrent spans and the first span of every segment
-    mean_spans: Optional[tuple] = None       # the same for running means
     # attention layers (and positions for all that rotate)
     multi_segs: int = 0
     multi_rows: int = 0
@@ -217,23 +216,6 @@ def recurrent_spans(lens: Sequence[int], heads: int, ctas: int = 296, shortest: 
         first.append(len(spans))
         row += n
     return (spans, first) if len(spans) > len(lens) else None
-
-
-MEAN_SPAN = 64         # tokens of a span of a running mean
-
-
-def mean_spans(lens: Sequence[int], span: int = MEAN_SPAN) -> Optional[tuple]:
-    """Cut segments of more than four spans' tokens into spans for running means; ``(row ranges, first span of every segment)``, None when
-    no segment is that long."""
-    if max(lens) <= 4 * span:
-        return None
-    spans, first, row = [], [0], 0
-    for n in lens:
-        step = span if n > 4 * span else n
-        spans += [[row + a, row + min(n, a + step)] for a in range(0, n, step)]
-        first.append(len(spans))
-        row += n
-    return spans, first
 
 
 class ComposedForward:
@@ -649,9 +631,6 @@ class ComposedScheduler:
             cuts = recurrent_spans(lens, max(rec)) if rec and self.device.type == "cuda" else None
             if cuts is not None:
                 arrays["spans"], arrays["span_first"] = (cuts[0], i32), (cuts[1], i32)
-            cuts = mean_spans(lens) if self.cfg.specs_with("mingru") and self.device.type == "cuda" else None
-            if cuts is not None:
-                arrays["mean"], arrays["mean_first"] = (cuts[0], i32), (cuts[1], i32)
             specs = self.cfg.specs_with("latent_attention")
             if sl and specs:
                 arrays["short_cu"] = ([c - cu[n_long] for c in cu[n_long:]], i32)
@@ -666,10 +645,9 @@ class ComposedScheduler:
         dev = dict(zip(arrays, self._stage(list(arrays.values()))))
         want_t = dev.pop("rows", None)
         spans = (dev.pop("spans"), dev.pop("span_first")) if "spans" in dev else None
-        mean = (dev.pop("mean"), dev.pop("mean_first")) if "mean" in dev else None
         items = {H: dev.pop(f"items{H}") for H in widths}
         blocks = {t: dev.pop(f"blocks{t}") for t in tiles}
-        batch = SegmentBatch(**dev, **host, items=items or None, item_width=widths or None, spans=spans, mean_spans=mean, blocks=blocks or None)
+        batch = SegmentBatch(**dev, **host, items=items or None, item_width=widths or None, spans=spans, blocks=blocks or None)
         logits = self.weights.forward_segments(batch, self.kv, want_t, self.tp, taps)
         for r, n in parts:
             r.fed += n

@@ -67,7 +67,7 @@ def _tables(ctx, page, seed):
 def _batch(lens, ctx, bt=None, H=1, G=1, slots=None, pools=None):
     """Segments of several rows first, as the engine orders them."""
     from relax_b200.models.config import LayerSpec
-    from relax_b200.rollout.composed import SegmentBatch, mean_spans, query_blocks, recurrent_spans, tile_tokens
+    from relax_b200.rollout.composed import SegmentBatch, query_blocks, recurrent_spans, tile_tokens
 
     slots = _i32(list(range(len(lens))) if slots is None else slots)
     if all(n == 1 for n in lens):
@@ -78,7 +78,7 @@ def _batch(lens, ctx, bt=None, H=1, G=1, slots=None, pools=None):
     both = lambda x: None if x is None else (_i32(x[0]), _i32(x[1]))
     return SegmentBatch(None, pools, _i32(ctx), bt, slots, cu=_i32(cu), multi_segs=m, multi_rows=cu[m], max_ctx_one=max(ctx[m:], default=0),
                         seg_of=_i32([s for s, n in enumerate(lens) for _ in range(n)]), blocks={t: _i32(query_blocks(lens[:m], ctx, t))},
-                        pos=_i32([c - n + k for n, c in zip(lens, ctx) for k in range(n)]), mean_spans=both(mean_spans(lens)),
+                        pos=_i32([c - n + k for n, c in zip(lens, ctx) for k in range(n)]),
                         spans=both(recurrent_spans(lens, H)))
 
 

@@ -1,7 +1,6 @@
 """Zoguzen stacks: every mechanism, the reader, cache, scheduler and generation on the CPU against plain float64 statements."""
 import io
 import json
-import math
 import os
 import sys
 from types import SimpleNamespace
@@ -33,7 +32,7 @@ def _batch(lens, starts, slots):
     cu = [0]
     for n in lens:
         cu.append(cu[-1] + n)
-    return SimpleNamespace(cu=torch.tensor(cu), ctx=torch.tensor([a + n for a, n in zip(starts, lens)]), state_slot=torch.tensor(slots), mean_spans=None)
+    return SimpleNamespace(cu=torch.tensor(cu), ctx=torch.tensor([a + n for a, n in zip(starts, lens)]), state_slot=torch.tensor(slots))
 
 
 # ---------------------------------------------------------------------------------------------------- mechanisms alone
@@ -530,12 +529,3 @@ def test_engine_server_serves_a_zoguzen_folder():
         assert list(out[0].output) == D.greedy(cfg, t, p, 4)
     finally:
         srv.close() if hasattr(srv, "close") else srv.httpd.shutdown()
-
-
-def test_spans_of_running_means_cover_every_row():
-    from relax_b200.rollout.composed import MEAN_SPAN, mean_spans
-
-    assert mean_spans([4 * MEAN_SPAN, 1]) is None
-    spans, first = mean_spans([3, 5 * MEAN_SPAN + 7, 1])
-    assert [b - a for a, b in spans] == [3] + [MEAN_SPAN] * 5 + [7, 1] and first == [0, 1, 7, 8]
-    assert all(a == b for (_, a), (b, _) in zip(spans, spans[1:])) and math.isclose(spans[-1][1], 11 + 5 * MEAN_SPAN)
