@@ -151,4 +151,19 @@ inline int encode_tma_3d_16bit(CUtensorMap* map, const void* ptr, uint64_t d0, u
   return r == CUDA_SUCCESS ? 0 : -11;
 }
 
+// 4-D bf16 tensor d0 x d1 x d2 x d3 whose dimensions lie dense behind one another; box b0 x b1 x b2 x b3, 128-byte swizzle.
+inline int encode_tma_4d_dense_bf16(CUtensorMap* map, const void* ptr, uint64_t d0, uint64_t d1, uint64_t d2, uint64_t d3, uint32_t b0, uint32_t b1,
+                                    uint32_t b2, uint32_t b3) {
+  ensure_context();
+  EncodeTiledFn fn = encode_fn();
+  if (!fn) return -10;
+  cuuint64_t dims[4] = {d0, d1, d2, d3};
+  cuuint64_t strides[3] = {d0 * 2, d0 * d1 * 2, d0 * d1 * d2 * 2};
+  cuuint32_t box[4] = {b0, b1, b2, b3};
+  cuuint32_t estr[4] = {1, 1, 1, 1};
+  CUresult r = fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 4, const_cast<void*>(ptr), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                  CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  return r == CUDA_SUCCESS ? 0 : -11;
+}
+
 }  // namespace rb

@@ -2,12 +2,15 @@
 // values of every group (see talk_decode_sm100.cu), out [rows][H][G][out_d].
 //
 // Tiles are those of paged_flash_sm100.cu (128 (token, head) rows of one key group, blocks of 64 positions straight from the pages), but a CTA
-// keeps the accumulators of several groups' values (up to 384 columns of TMEM), so scores and softmax are computed once for all of
-// them.  Scores are capped: the softmax has a fixed reference and nothing is rescaled; what a score costs is a polynomial and one
-// exponential.  Two sets of eight warps (two threads per row) take the blocks in turn, so one set's latencies hide behind the other's
-// arithmetic.  The CTAs are persistent: their blocks form one sequence across tiles, and the scores of the next tile are on their way
-// while the last one's accumulators are read.  Warps 0-15: softmax and epilogue, warp 16: TMA, warp 17: MMA.  Every wait is bounded; no load
-// uses cluster multicast.
+// keeps the accumulators of several groups' values (256 columns of TMEM), so scores and softmax are computed once for all of them.
+// Scores are capped: the softmax has a fixed reference and nothing is rescaled; what a score costs is a polynomial and one
+// exponential.  The CTAs are persistent and their blocks form one sequence across tiles.  Scores run four blocks ahead of the products; two
+// sets of eight warps (two threads per row) take the blocks in turn, and P replaces S in TMEM, where the products read it.  Warps of
+// their own read the accumulators of a finished tile while the softmax is at the next one; whole tiles leave through shared memory and TMA
+// stores.  Keys and values have three stages each and a producer of their own: a block's arithmetic is shorter than the way of its tiles
+// through the L2.  Issuing a block's products, with the waits around them, takes one thread longer than the tensor cores need for them, so scores
+// and output products are issued by two.  Warps 0-15: softmax, warp 16: TMA of queries and keys, warp 17: scores, warps 18-21: outputs, warp
+// 22: TMA of values, warp 23: products with the values.  Every wait is bounded; no load uses cluster multicast.
 #include <limits.h>
 
 #include "common.cuh"
@@ -19,12 +22,17 @@ namespace tf {
 constexpr int BQ = 128;
 constexpr int BKV = 64;
 constexpr int SOFT = 512;                 // softmax threads: two sets of two per row
-constexpr int THREADS = SOFT + 64;
+constexpr int kWarpK = 16, kWarpS = 17, kWarpOut = 18, kWarpV = 22, kWarpPv = 23;      // (four warps for the outputs)
+constexpr int THREADS = 24 * 32;
+constexpr int ST = 3;                     // stages of keys and of values
+constexpr int NS = 4;                     // buffers of scores
+static_assert(ST < NS, "a producer is never two phases behind");
+constexpr int RING = 8;                   // items whose sums are kept: the softmax is at most NS of them ahead of the outputs
 constexpr int kTmemCols = 512;
-constexpr int T_S = 0;                    // two buffers of 64 columns
-constexpr int T_O = 128;
+constexpr int T_S = 0;                    // NS buffers of 64 columns; P takes the first 16 of every 32
+constexpr int T_O = NS * 64;
 constexpr int kQHalf = BQ * 128, kKVHalf = BKV * 128;      // bytes of 64 columns
-constexpr int kPBytes = BQ * BKV * 2;
+constexpr int kStage = BQ * 128;          // 64 columns of outputs on their way out; two of them
 
 struct Params {
   const int* blocks;         // [n][4]: segment, first row, rows, position of the first row; null: row i is segment i, at ctx[i] - 1
@@ -35,7 +43,8 @@ struct Params {
   int H, Hkv, G, tokens, max_blocks, page, out_d, nv;      // G: heads per group; nv: value groups per item
   int n_items, slices;       // items: query tile, key group, slice of value groups (the last one fastest)
   int window, keep, chunk;   // as in paged_flash
-  int v_at, p_at, bar_at;    // bytes into shared memory
+  int v_at, out_at, bar_at;  // bytes into shared memory
+  int stores;                // whole tiles leave by TMA
   float cap_in;              // s = cap_log2 tanh(cap_in q . k), in log2 units
   float cap_log2;
   int* err;
@@ -89,39 +98,42 @@ struct Item {
 template <int DK, int DV>
 __global__ void __launch_bounds__(THREADS, 1)
 talk_flash_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_constant__ CUtensorMap tma_k, const __grid_constant__ CUtensorMap tma_v,
-                  const Params p) {
+                  const __grid_constant__ CUtensorMap tma_o, const Params p) {
   constexpr int kQBytes = DK / 64 * kQHalf, kKBytes = DK / 64 * kKVHalf, kVBytes = DV / 64 * kKVHalf;
   extern __shared__ __align__(1024) uint8_t smem[];
   uint64_t* bars = reinterpret_cast<uint64_t*>(smem + p.bar_at);
-  // blocks are numbered across items (g): index of a pair = g & 1, phase = g / 2; queries and accumulators by item
-  uint64_t* qfull = bars;          // [2]
-  uint64_t* qempty = bars + 2;     // [2] the scores of an item are complete
-  uint64_t* bar_s = bars + 4;      // [2] S of block g is complete
-  uint64_t* bar_p = bars + 6;      // [2] P of block g is written, S of block g is read
-  uint64_t* bar_o = bars + 8;      // [2] the products of block g are in the accumulators
-  uint64_t* kfull = bars + 10;     // [2]
-  uint64_t* vfull = bars + 12;     // [2]
-  uint64_t* kempty = bars + 14;    // [2]
-  uint64_t* vempty = bars + 16;    // [2]
-  uint64_t* bar_free = bars + 18;  // the accumulators of an item have been read
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 19);
+  // blocks are numbered across items (g): S and P of block g are buffer g % NS, its keys and values stage g % ST; queries and accumulators
+  // go by item (n)
+  uint64_t* qfull = bars;
+  uint64_t* qempty = bars + 1;     // the scores of an item are complete
+  uint64_t* bar_done = bars + 2;   // the products of an item are in the accumulators
+  uint64_t* bar_free = bars + 3;   // the accumulators of an item have been read
+  uint64_t* bar_s = bars + 4;      // [NS] S of a block is complete, and the stage of its keys free
+  uint64_t* bar_pv = bar_s + NS;   // [NS] its products are: the buffer and the stage of its values are free
+  uint64_t* bar_p = bar_pv + NS;   // [NS] P of a block is written
+  uint64_t* bar_l = bar_p + NS;    // [RING] the sums of an item are written
+  uint64_t* kfull = bar_l + RING;  // [ST]
+  uint64_t* vfull = kfull + ST;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(vfull + ST);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
-  float* sums = reinterpret_cast<float*>(tmem_slot + 2);      // [2][4][128]
+  float* sums = reinterpret_cast<float*>(smem + p.bar_at + 512);      // [RING][4][128]
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   if (threadIdx.x == 0) {
-    for (int i = 0; i < 2; ++i) {
-      mbar_init(&qfull[i], 1);
-      mbar_init(&qempty[i], 1);
+    mbar_init(qfull, 1);
+    mbar_init(qempty, 1);
+    mbar_init(bar_done, 1);
+    mbar_init(bar_free, 128);
+    for (int i = 0; i < NS; ++i) {
       mbar_init(&bar_s[i], 1);
+      mbar_init(&bar_pv[i], 1);
       mbar_init(&bar_p[i], SOFT / 2);
-      mbar_init(&bar_o[i], 1);
+    }
+    for (int i = 0; i < RING; ++i) mbar_init(&bar_l[i], SOFT);
+    for (int i = 0; i < ST; ++i) {
       mbar_init(&kfull[i], 1);
       mbar_init(&vfull[i], 1);
-      mbar_init(&kempty[i], 1);
-      mbar_init(&vempty[i], 1);
     }
-    mbar_init(bar_free, SOFT);
     *abort_flag = 0;
     if ((smem_u32(smem) & 1023u) != 0) {           // swizzled tiles need 1 KB alignment
       *abort_flag = 1;
@@ -129,7 +141,7 @@ talk_flash_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
     }
     fence_barrier_init();
   }
-  if (warp == 17) {
+  if (warp == kWarpS) {
     tmem_alloc<kTmemCols>(tmem_slot);
     tmem_relinquish();
   }
@@ -140,118 +152,183 @@ talk_flash_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
   const bool dead = *abort_flag != 0;
   const int step = gridDim.x;
 
-  if (warp == 16) {
-    // ================================================================ TMA producer
+  if (warp == kWarpK || warp == kWarpV) {
+  // ================================================================ TMA producers: queries and keys; values
     if (lane == 0 && !dead) {
-      tma_prefetch_desc(&tma_q);
-      tma_prefetch_desc(&tma_k);
-      tma_prefetch_desc(&tma_v);
+      const bool values = warp == kWarpV;
+      tma_prefetch_desc(values ? &tma_v : &tma_k);
+      if (!values) tma_prefetch_desc(&tma_q);
       const int rows = p.page < BKV ? p.page : BKV;          // rows per box
+      uint64_t* full = values ? vfull : kfull;
+      uint64_t* freed = values ? bar_pv : bar_s;
       bool ok = true;
-      int g = 0, n = 0;
+      int s = 0, n = 0, g = 0;
       for (int i = blockIdx.x; i < p.n_items && ok; i += step, ++n) {
         const Item w(p, i);
         const int* bt = p.block_tables + static_cast<size_t>(w.seg) * p.max_blocks;
-        auto pool_row = [&](int pos) { return bt[min(pos / p.page, p.max_blocks - 1)] * p.page + pos % p.page; };
-        ok = mbar_wait(&qempty[n & 1], (static_cast<uint32_t>(n >> 1) & 1) ^ 1, abort_flag, p.err);
-        if (!ok) break;
-        // the box holds `tokens` tokens of G heads: row = token * G + head; rows behind it are never stored
-        mbar_expect_tx(&qfull[n & 1], static_cast<uint32_t>(p.tokens * p.G) * DK * 2);
-        for (int c = 0; c < DK / 64; ++c) tma_load_3d(smem + (n & 1) * kQBytes + c * kQHalf, &tma_q, &qfull[n & 1], c * 64, w.kvh * p.G, w.row0);
+        if (!values) {
+          ok = mbar_wait(qempty, (static_cast<uint32_t>(n) & 1) ^ 1, abort_flag, p.err);
+          if (!ok) break;
+          // the box holds `tokens` tokens of G heads: row = token * G + head; rows behind it are never stored
+          mbar_expect_tx(qfull, static_cast<uint32_t>(p.tokens * p.G) * DK * 2);
+          for (int c = 0; c < DK / 64; ++c) tma_load_3d(smem + c * kQHalf, &tma_q, qfull, c * 64, w.kvh * p.G, w.row0);
+        }
         for (int j = 0; j < w.n_blocks; ++j, ++g) {
-          const int s = g & 1, at = w.first_position(j);
-          const uint32_t ph = (static_cast<uint32_t>(g >> 1) & 1) ^ 1;
-          ok = mbar_wait(&kempty[s], ph, abort_flag, p.err);
+          const int at = w.first_position(j);
+          if (g >= ST) ok = mbar_wait(&freed[(g - ST) % NS], static_cast<uint32_t>((g - ST) / NS) & 1, abort_flag, p.err);
           if (!ok) break;
-          uint8_t* sk = smem + 2 * kQBytes + s * kKBytes;
-          mbar_expect_tx(&kfull[s], kKBytes);
+          mbar_expect_tx(&full[s], values ? w.nv * kVBytes : kKBytes);
           for (int r = 0; r < BKV; r += rows) {
-            const int row = pool_row(at + r);
-            for (int c = 0; c < DK / 64; ++c) tma_load_3d(sk + c * kKVHalf + r * 128, &tma_k, &kfull[s], c * 64, w.kvh, row);
-          }
-          ok = mbar_wait(&vempty[s], ph, abort_flag, p.err);
-          if (!ok) break;
-          uint8_t* sv = smem + p.v_at + s * p.nv * kVBytes;
-          mbar_expect_tx(&vfull[s], w.nv * kVBytes);
-          for (int r = 0; r < BKV; r += rows) {
-            const int row = pool_row(at + r);
-            for (int v = 0; v < w.nv; ++v)
-              for (int c = 0; c < DV / 64; ++c) tma_load_3d(sv + v * kVBytes + c * kKVHalf + r * 128, &tma_v, &vfull[s], c * 64, w.v0 + v, row);
-          }
-        }
-      }
-    }
-  } else if (warp == 17) {
-    // ================================================================ MMA issuer
-    if (lane == 0 && !dead) {
-      const uint32_t idesc_s = make_idesc_f16(BQ, BKV, true, false, false);
-      const uint32_t idesc_o = make_idesc_f16(BQ, DV, true, false, true);
-      const uint32_t sq = smem_u32(smem), sp = smem_u32(smem + p.p_at);
-      // scores run two blocks ahead of the products, across items
-      int si = blockIdx.x, sn = 0, sj = 0, sg = 0;
-      int s_blocks = si < p.n_items ? Item(p, si).n_blocks : 0;
-      auto issue_s = [&]() -> bool {
-        if (si >= p.n_items) return true;
-        const int s = sg & 1;
-        if (sj == 0 && !mbar_wait(&qfull[sn & 1], static_cast<uint32_t>(sn >> 1) & 1, abort_flag, p.err)) return false;
-        if (!mbar_wait(&kfull[s], static_cast<uint32_t>(sg >> 1) & 1, abort_flag, p.err)) return false;
-        tc_fence_after();
-        const uint32_t q = sq + (sn & 1) * kQBytes, sk = smem_u32(smem + 2 * kQBytes + s * kKBytes);
-#pragma unroll
-        for (int kk = 0; kk < DK / 16; ++kk) {
-          const uint64_t da = make_smem_desc(q + (kk >> 2) * kQHalf + (kk & 3) * 32, 16, 1024, kSwizzle128B);
-          const uint64_t db = make_smem_desc(sk + (kk >> 2) * kKVHalf + (kk & 3) * 32, 16, 1024, kSwizzle128B);
-          umma_f16(tmem_base + T_S + s * BKV, da, db, idesc_s, kk > 0 ? 1u : 0u);
-        }
-        umma_commit(&kempty[s]);
-        umma_commit(&bar_s[s]);
-        ++sg;
-        if (++sj == s_blocks) {
-          umma_commit(&qempty[sn & 1]);
-          sj = 0;
-          ++sn;
-          si += step;
-          if (si < p.n_items) s_blocks = Item(p, si).n_blocks;
-        }
-        return true;
-      };
-      bool ok = issue_s() && issue_s();
-      int g = 0, n = 0;
-      for (int i = blockIdx.x; i < p.n_items && ok; i += step, ++n) {
-        const Item w(p, i);
-        if (n > 0) ok = mbar_wait(bar_free, static_cast<uint32_t>(n - 1) & 1, abort_flag, p.err);
-        for (int j = 0; j < w.n_blocks && ok; ++j, ++g) {
-          const int s = g & 1;
-          const uint32_t ph = static_cast<uint32_t>(g >> 1) & 1;
-          ok = mbar_wait(&bar_p[s], ph, abort_flag, p.err) && mbar_wait(&vfull[s], ph, abort_flag, p.err);
-          if (!ok) break;
-          tc_fence_after();
-          for (int v = 0; v < w.nv; ++v) {
-            const uint32_t sv = smem_u32(smem + p.v_at + (s * p.nv + v) * kVBytes);
-#pragma unroll
-            for (int kk = 0; kk < BKV / 16; ++kk) {
-              const uint64_t da = make_smem_desc(sp + s * kPBytes + kk * 32, 16, 1024, kSwizzle128B);
-              const uint64_t db = make_smem_desc(sv + kk * 2048, kKVHalf, 1024, kSwizzle128B);      // V tile [position][d]
-              umma_f16(tmem_base + T_O + v * DV, da, db, idesc_o, (j > 0 || kk > 0) ? 1u : 0u);
+            const int pos = at + r, row = bt[min(pos / p.page, p.max_blocks - 1)] * p.page + pos % p.page;
+            if (values) {
+              uint8_t* sv = smem + p.v_at + s * p.nv * kVBytes + r * 128;
+              for (int v = 0; v < w.nv; ++v)
+                for (int c = 0; c < DV / 64; ++c) tma_load_3d(sv + v * kVBytes + c * kKVHalf, &tma_v, &full[s], c * 64, w.v0 + v, row);
+            } else {
+              uint8_t* sk = smem + kQBytes + s * kKBytes + r * 128;
+              for (int c = 0; c < DK / 64; ++c) tma_load_3d(sk + c * kKVHalf, &tma_k, &full[s], c * 64, w.kvh, row);
             }
           }
-          umma_commit(&vempty[s]);
-          umma_commit(&bar_o[s]);
-          ok = issue_s();      // S of block g was read before bar_p completed
+          if (++s == ST) s = 0;
         }
       }
     }
-  } else {
-    // ================================================================ softmax + epilogue (warps 0..15)
-    const int set = warp >> 3, half = (warp >> 2) & 1;           // the set takes blocks set, set + 2, ..; columns half * 32 .. + 31 of a block
+  } else if (warp == kWarpS) {
+    // ================================================================ scores, up to NS blocks ahead of the products
+    if (lane == 0 && !dead) {
+      const uint32_t idesc = make_idesc_f16(BQ, BKV, true, false, false);
+      const uint32_t sq = smem_u32(smem);
+      bool ok = true;
+      int g = 0, n = 0, stage = 0;
+      uint32_t ph = 0;
+      for (int i = blockIdx.x; i < p.n_items && ok; i += step, ++n) {
+        const int blocks = Item(p, i).n_blocks;
+        ok = mbar_wait(qfull, static_cast<uint32_t>(n) & 1, abort_flag, p.err);
+        for (int j = 0; j < blocks && ok; ++j, ++g) {
+          const int s = g % NS;
+          ok = mbar_wait(&kfull[stage], ph, abort_flag, p.err);
+          if (ok && g >= NS) ok = mbar_wait(&bar_pv[s], static_cast<uint32_t>(g / NS - 1) & 1, abort_flag, p.err);
+          if (!ok) break;
+          tc_fence_after();
+          const uint32_t sk = smem_u32(smem + kQBytes + stage * kKBytes);
+#pragma unroll
+          for (int kk = 0; kk < DK / 16; ++kk) {
+            const uint64_t da = make_smem_desc(sq + (kk >> 2) * kQHalf + (kk & 3) * 32, 16, 1024, kSwizzle128B);
+            const uint64_t db = make_smem_desc(sk + (kk >> 2) * kKVHalf + (kk & 3) * 32, 16, 1024, kSwizzle128B);
+            umma_f16(tmem_base + T_S + s * BKV, da, db, idesc, kk > 0 ? 1u : 0u);
+          }
+          umma_commit(&bar_s[s]);
+          if (++stage == ST) {
+            stage = 0;
+            ph ^= 1;
+          }
+        }
+        if (ok) umma_commit(qempty);
+      }
+      if (ok && n > 0) mbar_wait(qempty, static_cast<uint32_t>(n - 1) & 1, abort_flag, p.err);      // (no commit outlives the CTA)
+    }
+  } else if (warp == kWarpPv) {
+    // ================================================================ products with the values, all groups of an item at once
+    if (lane == 0 && !dead) {
+      bool ok = true;
+      int g = 0, n = 0, stage = 0;
+      uint32_t ph = 0;
+      for (int i = blockIdx.x; i < p.n_items && ok; i += step, ++n) {
+        const Item w(p, i);
+        const uint32_t idesc = make_idesc_f16(BQ, w.nv * DV, true, false, true);
+        if (n > 0) ok = mbar_wait(bar_free, static_cast<uint32_t>(n - 1) & 1, abort_flag, p.err);
+        for (int j = 0; j < w.n_blocks && ok; ++j, ++g) {
+          const int s = g % NS;
+          ok = mbar_wait(&vfull[stage], ph, abort_flag, p.err) && mbar_wait(&bar_p[s], static_cast<uint32_t>(g / NS) & 1, abort_flag, p.err);
+          if (!ok) break;
+          tc_fence_after();
+          const uint32_t sv = smem_u32(smem + p.v_at + stage * p.nv * kVBytes);
+#pragma unroll
+          for (int kk = 0; kk < BKV / 16; ++kk) {
+            const uint64_t db = make_smem_desc(sv + kk * 2048, kKVHalf, 1024, kSwizzle128B);      // V tiles [position][d], 64 columns kKVHalf apart
+            umma_f16_ts(tmem_base + T_O, tmem_base + T_S + s * BKV + (kk >> 1) * 32 + (kk & 1) * 8, db, idesc, (j > 0 || kk > 0) ? 1u : 0u);
+          }
+          umma_commit(&bar_pv[s]);
+          if (++stage == ST) {
+            stage = 0;
+            ph ^= 1;
+          }
+        }
+        if (ok) umma_commit(bar_done);
+      }
+      if (ok && n > 0) mbar_wait(bar_done, static_cast<uint32_t>(n - 1) & 1, abort_flag, p.err);
+    }
+  } else if (warp >= kWarpOut && warp < kWarpV) {
+    // ================================================================ outputs (four warps)
     const int r = (warp & 3) * 32 + lane;                        // row of the tile = TMEM lane
     const int t = r / p.G;
     const uint32_t lane_addr = static_cast<uint32_t>((warp & 3) * 32) << 16;
+    const bool issues = warp == kWarpOut && lane == 0;
+    bool ok = !dead;
+    int n = 0, buffer = 0;
+    for (int i = blockIdx.x; i < p.n_items && ok; i += step, ++n) {
+      const Item w(p, i);
+      ok = mbar_wait(&bar_l[n % RING], static_cast<uint32_t>(n / RING) & 1, abort_flag, p.err) &&
+           mbar_wait(bar_done, static_cast<uint32_t>(n) & 1, abort_flag, p.err);
+      ok = named_bar_and(1, 128, ok);                            // (all leave together when a wait ran out)
+      if (!ok) break;
+      tc_fence_after();
+      const float* sum = sums + (n % RING) * 4 * BQ + r;
+      const float l = sum[0] + sum[BQ] + sum[2 * BQ] + sum[3 * BQ];
+      const float inv_l = l > 0.f ? 1.f / l : 0.f;
+      const int chunks = w.nv * (DV / 64);                       // of 64 columns; two buffers on their way out
+      const bool whole = p.stores && w.ntok == p.tokens, mine = t < w.ntok;
+      __nv_bfloat16* out = p.out + ((static_cast<size_t>(w.row0 + t) * p.H + w.kvh * p.G + r % p.G) * p.Hkv + w.v0) * p.out_d;
+#pragma unroll 1
+      for (int ch = 0; ch < chunks; ++ch) {
+        const int v = ch / (DV / 64), c = (ch % (DV / 64)) * 64;
+        uint8_t* dst = smem + p.out_at + buffer * kStage + r * 128;
+        if (whole) {
+          if (issues) tma_store_wait_read<1>();                  // the store before the last one has left shared memory
+          named_bar_sync(1, 128);
+        }
+#pragma unroll
+        for (int part = 0; part < 2; ++part) {
+          uint32_t o[32];
+          tmem_ld_32x32b_x32(tmem_base + T_O + v * DV + c + part * 32 + lane_addr, o);
+          tmem_wait_ld();
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            uint4 pk;
+            pk.x = pack_bf16(__uint_as_float(o[8 * e]) * inv_l, __uint_as_float(o[8 * e + 1]) * inv_l);
+            pk.y = pack_bf16(__uint_as_float(o[8 * e + 2]) * inv_l, __uint_as_float(o[8 * e + 3]) * inv_l);
+            pk.z = pack_bf16(__uint_as_float(o[8 * e + 4]) * inv_l, __uint_as_float(o[8 * e + 5]) * inv_l);
+            pk.w = pack_bf16(__uint_as_float(o[8 * e + 6]) * inv_l, __uint_as_float(o[8 * e + 7]) * inv_l);
+            if (whole) *reinterpret_cast<uint4*>(dst + (((part * 4 + e) ^ (r & 7)) << 4)) = pk;
+            else if (mine && c + part * 32 + e * 8 < p.out_d) *reinterpret_cast<uint4*>(out + static_cast<size_t>(v) * p.out_d + c + part * 32 + e * 8) = pk;
+          }
+        }
+        if (ch + 1 == chunks) {
+          tc_fence_before();
+          mbar_arrive(bar_free);
+        }
+        if (whole) {
+          fence_proxy_async();
+          named_bar_sync(1, 128);
+          if (issues) {
+            tma_store_4d(&tma_o, smem + p.out_at + buffer * kStage, c, w.v0 + v, w.kvh * p.G, w.row0);
+            tma_store_commit();
+          }
+          buffer ^= 1;
+        }
+      }
+    }
+    if (issues) tma_store_wait<0>();
+  } else {
+    // ================================================================ softmax (warps 0..15)
+    const int set = warp >> 3, half = (warp >> 2) & 1;           // the set takes every other block; columns half * 32 .. + 31 of a block
+    const int r = (warp & 3) * 32 + lane;                        // row of the tile = TMEM lane
+    const int t = r / p.G;
+    const uint32_t mine_at = tmem_base + T_S + half * 32 + (static_cast<uint32_t>((warp & 3) * 32) << 16);
     unsigned long long poly[7];
 #pragma unroll
     for (int k = 0; k < 7; ++k) poly[k] = pair2(kTanh[k] * p.cap_log2, kTanh[k] * p.cap_log2);
     const unsigned long long cin = pair2(p.cap_in, p.cap_in);
-    uint8_t* sp = smem + p.p_at + set * kPBytes + r * 128;
     bool ok = !dead;
     int g = 0, n = 0;
     for (int i = blockIdx.x; i < p.n_items && ok; i += step, ++n) {
@@ -263,12 +340,12 @@ talk_flash_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
       float l = 0.f;
       if (p.sink && mine && warp < 4) l = exp2f(__bfloat162float(p.sink[head]) * 1.4426950408889634f);
       for (int j = (g ^ set) & 1; j < w.n_blocks; j += 2) {
-        const uint32_t turn = static_cast<uint32_t>(g + j) >> 1;
-        if (ok) ok = mbar_wait(&bar_s[set], turn & 1, abort_flag, p.err);
+        const int s = (g + j) % NS;
+        if (ok) ok = mbar_wait(&bar_s[s], static_cast<uint32_t>((g + j) / NS) & 1, abort_flag, p.err);
         if (!__all_sync(0xffffffffu, ok)) { ok = false; break; }
         tc_fence_after();
         uint32_t raw[32];
-        tmem_ld_32x32b_x32(tmem_base + T_S + set * BKV + half * 32 + lane_addr, raw);
+        tmem_ld_32x32b_x32(mine_at + s * BKV, raw);
         tmem_wait_ld();
         float big = 0.f;
 #pragma unroll
@@ -308,61 +385,21 @@ talk_flash_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
           raw[c >> 1] = pack_bf16(a, b);
         }
         l += sum0 + sum1;
-        if (turn > 0) {      // the products of the set's block before have read this P buffer
-          if (ok) ok = mbar_wait(&bar_o[set], (turn - 1) & 1, abort_flag, p.err);
-          if (!__all_sync(0xffffffffu, ok)) { ok = false; break; }
-        }
-#pragma unroll
-        for (int k = 0; k < 4; ++k)
-          *reinterpret_cast<uint4*>(sp + (((half * 4 + k) ^ (r & 7)) << 4)) = make_uint4(raw[4 * k], raw[4 * k + 1], raw[4 * k + 2], raw[4 * k + 3]);
-        fence_proxy_async();
+        tmem_st_32x32b_x16(mine_at + s * BKV, raw);
+        tmem_wait_st();
         tc_fence_before();
-        mbar_arrive(&bar_p[set]);
+        mbar_arrive(&bar_p[s]);
       }
       g += w.n_blocks;
-      float* sum = sums + (n & 1) * 4 * BQ;      // (two buffers: a warp may be one item ahead)
-      sum[(set * 2 + half) * BQ + r] = l;
-      // The set without the last block waits for its own last one first: products complete in order, so the other barrier is then at most
-      // one phase behind and its parity says which.
-      if (ok && ((g - 1) & 1) != set && w.n_blocks > 1) ok = mbar_wait(&bar_o[set], static_cast<uint32_t>((g - 2) >> 1) & 1, abort_flag, p.err);
-      if (ok) ok = mbar_wait(&bar_o[(g - 1) & 1], static_cast<uint32_t>((g - 1) >> 1) & 1, abort_flag, p.err);
-      ok = named_bar_and(1, SOFT, ok);      // (all leave together when a wait ran out)
-      tc_fence_after();
-      l = sum[r] + sum[BQ + r] + sum[2 * BQ + r] + sum[3 * BQ + r];
-      const float inv_l = l > 0.f ? 1.f / l : 0.f;
-      __nv_bfloat16* out = p.out + ((static_cast<size_t>(w.row0 + t) * p.H + head) * p.Hkv + w.v0) * p.out_d;
-      if (ok) {
-#pragma unroll 1
-        for (int k = warp >> 2; k < w.nv * (DV / 32); k += 4) {      // the four warps of a lane quarter share the columns
-          const int v = k / (DV / 32), c = (k % (DV / 32)) * 32;
-          if (c >= p.out_d) continue;
-          uint32_t o[32];
-          tmem_ld_32x32b_x32(tmem_base + T_O + v * DV + c + lane_addr, o);
-          tmem_wait_ld();
-          if (mine) {
-#pragma unroll
-            for (int e = 0; e < 4; ++e) {
-              if (c + e * 8 < p.out_d) {
-                uint4 pk;
-                pk.x = pack_bf16(__uint_as_float(o[8 * e]) * inv_l, __uint_as_float(o[8 * e + 1]) * inv_l);
-                pk.y = pack_bf16(__uint_as_float(o[8 * e + 2]) * inv_l, __uint_as_float(o[8 * e + 3]) * inv_l);
-                pk.z = pack_bf16(__uint_as_float(o[8 * e + 4]) * inv_l, __uint_as_float(o[8 * e + 5]) * inv_l);
-                pk.w = pack_bf16(__uint_as_float(o[8 * e + 6]) * inv_l, __uint_as_float(o[8 * e + 7]) * inv_l);
-                reinterpret_cast<uint4*>(out + static_cast<size_t>(v) * p.out_d + c)[e] = pk;
-              }
-            }
-          }
-        }
-      }
-      tc_fence_before();
-      mbar_arrive(bar_free);
+      sums[((n % RING) * 4 + set * 2 + half) * BQ + r] = l;
+      mbar_arrive(&bar_l[n % RING]);
     }
   }
 
   if (*abort_flag) __nanosleep(50000);
   tc_fence_before();
   __syncthreads();
-  if (warp == 17) {
+  if (warp == kWarpS) {
     tc_fence_after();
     tmem_dealloc<kTmemCols>(tmem_base);
   }
@@ -378,19 +415,27 @@ static int launch(const void* q, const void* kc, const void* vc, int rows, int n
   if (rc) return rc;
   rc = encode_tma_3d_16bit(&tv, vc, DV, p.Hkv, pool_rows, DV, static_cast<uint64_t>(p.Hkv) * DV, 64, 1, box);
   if (rc) return rc;
-  // value groups whose accumulators fit (3 of 128 columns, 6 of 64), one less where two stages of their tiles do not
-  constexpr int most = (kTmemCols - T_O) / DV - (DK == 128 ? 1 : 0);
-  const int slices = (p.Hkv + most - 1) / most;
-  p.nv = (p.Hkv + slices - 1) / slices;
-  p.slices = (p.Hkv + p.nv - 1) / p.nv;
+  // value groups per item: as many as their accumulators and the stages of their tiles leave room for, shared out evenly
+  int total = 0;
+  for (int most = (kTmemCols - T_O) / DV;; --most) {
+    if (most < 1) return -20;
+    p.slices = (p.Hkv + most - 1) / most;
+    p.nv = (p.Hkv + p.slices - 1) / p.slices;
+    p.v_at = DK / 64 * (kQHalf + ST * kKVHalf);
+    p.out_at = p.v_at + ST * p.nv * (DV / 64) * kKVHalf;
+    p.bar_at = p.out_at + 2 * kStage;
+    total = p.bar_at + 512 + RING * 4 * BQ * 4;
+    if (total <= 227 * 1024) break;
+  }
   const long long items = static_cast<long long>(n) * p.Hkv * p.slices;
   if (items > 1 << 30) return -20;
   p.n_items = static_cast<int>(items);
-  p.v_at = DK / 64 * 2 * (kQHalf + kKVHalf);
-  p.p_at = p.v_at + 2 * p.nv * (DV / 64) * kKVHalf;
-  p.bar_at = p.p_at + 2 * kPBytes;
-  const int total = p.bar_at + 256 + 8 * BQ * 4;
-  if (total > 227 * 1024) return -20;
+  CUtensorMap to = tq;
+  p.stores = p.out_d % 64 == 0 && reinterpret_cast<uintptr_t>(p.out) % 16 == 0;
+  if (p.stores) {
+    rc = encode_tma_4d_dense_bf16(&to, p.out, p.out_d, p.Hkv, p.H, rows, 64, 1, p.G, p.tokens);
+    if (rc) return rc;
+  }
   auto kern = talk_flash_kernel<DK, DV>;
   static bool attr = false;
   if (!attr) {
@@ -399,7 +444,7 @@ static int launch(const void* q, const void* kc, const void* vc, int rows, int n
     attr = true;
   }
   // two CTAs of an SM would take turns with all of its TMEM columns: ask for more than half of the shared memory
-  kern<<<p.n_items < num_sms() ? p.n_items : num_sms(), THREADS, total < 116 * 1024 ? 116 * 1024 : total, st>>>(tq, tk, tv, p);
+  kern<<<p.n_items < num_sms() ? p.n_items : num_sms(), THREADS, total < 116 * 1024 ? 116 * 1024 : total, st>>>(tq, tk, tv, to, p);
   rb_note_launch(1);
   return static_cast<int>(cudaGetLastError());
 }

@@ -285,6 +285,25 @@ def test_scores_at_their_cap_do_not_overflow(dtype):
     _ok()
 
 
+@pytest.mark.parametrize("H,G,dim,vdim,chunk,cap", [(32, 4, 128, 128, 1024, 30.0), (16, 2, 64, 64, 300, 10.0), (24, 6, 128, 64, 0, 25.0), (12, 3, 64, 128, 700, 50.0)])
+def test_mixed_heads_of_long_prompts(H, G, dim, vdim, chunk, cap):
+    """Many tiles per CTA: the tensor-core kernels against the CUDA-core ones, prompts and single rows behind them."""
+    from relax_b200 import ops
+    from relax_b200.ops import cuda as C
+
+    lens, ctx, page = [1500, 700, 130, 1, 1], [1500, 2000, 130, 1999, 640], 64
+    bt, rows, total = _tables(ctx, page, 3)
+    k, v, q = _rand(1, total, G, dim, dtype=BF), _rand(2, total, G, vdim, dtype=BF), _rand(5, sum(lens), H, dim, dtype=BF)
+    mix, one = torch.eye(H, device="cuda").to(BF) + _rand(8, H, H, dtype=BF) * 0.3, torch.zeros(H, dtype=BF, device="cuda")
+    b = _batch(lens, ctx, bt, H, G)
+    args = (b, page, 2.0 / dim ** 0.5, one, vdim, 0, None, 0, chunk, cap, mix)
+    got = ops.paged_attention(q, k, v, *args)
+    want = C.paged_attention(q.float(), k.float(), v.float(), b, page, 2.0 / dim ** 0.5, one.float(), vdim, 0, None, 0, chunk, cap, mix.float())
+    _close(got, want, 1.5e-2)
+    assert torch.equal(got, ops.paged_attention(q, k, v, *args))      # nothing races
+    _ok()
+
+
 # ---------------------------------------------------------------------------------------------------- recurrences
 
 
