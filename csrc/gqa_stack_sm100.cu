@@ -215,9 +215,9 @@ __global__ void __launch_bounds__(PI_WARPS * 32) projection_inputs_kernel(const 
   }
 }
 
-// One warp per (head, run of RUN rows).  Lane l holds 2 NP consecutive features; a run's raw rows and what is known about them are fetched
-// at once, and the rows slide through registers.  With one row per sequence the warp also moves the state on; otherwise
-// conv_state_kernel does, afterwards.
+// One warp per head and `runs` runs of RUN rows.  Lane l holds 2 NP consecutive features with their weights; a run's raw rows and what is
+// known about them are fetched at once, and the rows slide through registers.  With one row per sequence the warp also moves the state on;
+// otherwise conv_state_kernel does, afterwards.
 struct ConvParams {
   const void* qkv;           // [T][ld]: H query heads | G key heads | G value heads (keys and values only with k_pool)
   const void* bias;          // [C] or null
@@ -236,7 +236,7 @@ struct ConvParams {
   const int* seg_of;         // [T] (with cu)
   const int* pos;            // [T] (with cu)
   long long pool_rows;
-  int T, H, G, dim, vdim, dp, vp, rot, ld, n, C;
+  int T, H, G, dim, vdim, dp, vp, rot, ld, n, C, runs;
   float eps;                 // <= 0: no norm
 };
 // N consecutive elements of which `left` exist (kVec: all or none, N * sizeof(T) aligned)
@@ -309,10 +309,9 @@ __global__ void __launch_bounds__(256) conv_inputs_kernel(const ConvParams p) {
   const int lane = threadIdx.x & 31;
   const int per = p.H + (p.k_pool ? 2 * p.G : 0);
   const long long u = static_cast<long long>(blockIdx.x) * 8 + (threadIdx.x >> 5);
-  const long long run = u / per;
-  const int hd = static_cast<int>(u - run * per);
-  const int t0 = static_cast<int>(run) * RUN, rows = min(p.T - t0, RUN);
-  if (rows <= 0) return;
+  const long long part = u / per;
+  const int hd = static_cast<int>(u - part * per);
+  if (part * p.runs * RUN >= p.T) return;
   const bool value = hd >= p.H + p.G;
   const int n = value ? p.vdim : p.dim, pitch = value ? p.vp : p.dp;
   const int g = hd - (hd < p.H ? 0 : p.H + (value ? p.G : 0));
@@ -320,22 +319,6 @@ __global__ void __launch_bounds__(256) conv_inputs_kernel(const ConvParams p) {
   const int e = N * lane, left = n - e;
   const T* src = static_cast<const T*>(p.qkv) + ch + e;
   const bool normed = !value && p.eps > 0.f;
-  // what is known about the rows: lane i holds it for row t0 + i
-  int m_seg = 0, m_at = 0, m_first = 0, m_state = 0;
-  long long m_slot = 0;
-  if (lane < rows) {
-    const int t = t0 + lane;
-    m_seg = p.cu ? p.seg_of[t] : t;
-    m_at = p.cu ? p.pos[t] : p.ctx[t] - 1;
-    m_first = p.cu ? p.cu[m_seg] : t;
-    m_state = p.state_slot[m_seg];
-    if (hd >= p.H) m_slot = p.slots[t];
-  }
-  float x[RUN][N];
-#pragma unroll
-  for (int k = 0; k < RUN; ++k) {
-    if (k < rows) load_run<T, N, kVec>(src + static_cast<long long>(t0 + k) * p.ld, left, x[k]);
-  }
   float w[NT][N], bias[N], nw[N];
 #pragma unroll
   for (int i = 0; i < N; ++i) {
@@ -344,77 +327,112 @@ __global__ void __launch_bounds__(256) conv_inputs_kernel(const ConvParams p) {
     w[0][i] = 1.f;
     bias[i] = 0.f;
     nw[i] = 1.f;
-    if (i < left) {
-      if (p.taps) {
-        const T* tp = static_cast<const T*>(p.taps) + static_cast<long long>(ch + e + i) * p.n;
+  }
+  if (p.taps) {
+    const T* tp = static_cast<const T*>(p.taps) + static_cast<long long>(ch + e) * p.n;
+    if (kVec && NT == 4 && p.n == NT) {
+      float v[N * NT];
+      load_run<T, N * NT, kVec>(tp, left, v);
+#pragma unroll
+      for (int i = 0; i < N; ++i)
+#pragma unroll
+        for (int k = 0; k < NT; ++k) w[k][i] = v[i * NT + NT - 1 - k];
+    } else {
+#pragma unroll
+      for (int i = 0; i < N; ++i)
 #pragma unroll
         for (int k = 0; k < NT; ++k)
-          if (k < p.n) w[k][i] = ld(tp + p.n - 1 - k);
-      }
-      if (p.bias) bias[i] = ld(static_cast<const T*>(p.bias) + ch + e + i);
-      if (normed) nw[i] = ld(static_cast<const T*>(hd < p.H ? p.q_w : p.k_w) + e + i);
+          if (i < left && k < p.n) w[k][i] = ld(tp + i * p.n + p.n - 1 - k);
     }
   }
-  float past[NT > 1 ? NT - 1 : 1][N];      // raw rows t - 1, t - 2, ...
+  if (p.bias) load_run<T, N, kVec>(static_cast<const T*>(p.bias) + ch + e, left, bias);
+  if (normed) load_run<T, N, kVec>(static_cast<const T*>(hd < p.H ? p.q_w : p.k_w) + e, left, nw);
+  float past[NT > 1 ? NT - 1 : 1][N];      // rows t - 1, t - 2, .. with their biases, zeros before the sequence's start
   int seg = -1;
-#pragma unroll
-  for (int k = 0; k < RUN; ++k) {
-    if (k >= rows) break;
-    const int t = t0 + k;
-    const int s = __shfl_sync(0xffffffffu, m_seg, k), at = __shfl_sync(0xffffffffu, m_at, k), local = t - __shfl_sync(0xffffffffu, m_first, k);
-    const int place = __shfl_sync(0xffffffffu, m_state, k);
-    const long long slot = __shfl_sync(0xffffffffu, m_slot, k);
-    T* state = p.n > 1 ? static_cast<T*>(p.state) + static_cast<long long>(place) * (p.n - 1) * p.C + ch + e : nullptr;
-    if (s != seg) {
-      seg = s;
-#pragma unroll
-      for (int b = 1; b < NT; ++b) {
-        const T* from = b <= local ? src + static_cast<long long>(t - b) * p.ld : state + static_cast<long long>(p.n - 1 - (b - local)) * p.C;
-        load_run<T, N, kVec>(from, b < p.n && b <= at ? left : 0, past[b - 1]);
-      }
+  for (int r = 0; r < p.runs; ++r) {
+    const int t0 = (static_cast<int>(part) * p.runs + r) * RUN, rows = min(p.T - t0, RUN);
+    if (rows <= 0) break;
+    // what is known about the rows: lane i holds it for row t0 + i
+    int m_seg = 0, m_at = 0, m_first = 0, m_state = 0;
+    long long m_slot = 0;
+    if (lane < rows) {
+      const int t = t0 + lane;
+      m_seg = p.cu ? p.seg_of[t] : t;
+      m_at = p.cu ? p.pos[t] : p.ctx[t] - 1;
+      m_first = p.cu ? p.cu[m_seg] : t;
+      m_state = p.state_slot[m_seg];
+      if (hd >= p.H) m_slot = p.slots[t];
     }
-    if (!p.cu && p.n > 1) {      // the state moves on by one row
+    float x[RUN][N];
 #pragma unroll
-      for (int b = NT - 1; b >= 1; --b)
-        if (b < p.n) store_run<T, N, kVec>(state + static_cast<long long>(p.n - 1 - b) * p.C, left, b > 1 ? past[b > 1 ? b - 2 : 0] : x[k]);
+    for (int k = 0; k < RUN; ++k) {
+      if (k < rows) load_run<T, N, kVec>(src + static_cast<long long>(t0 + k) * p.ld, left, x[k]);
     }
-    float y[N], ss = 0.f;
 #pragma unroll
-    for (int i = 0; i < N; ++i) {
-      float a = w[0][i] * (x[k][i] + bias[i]);
+    for (int k = 0; k < RUN; ++k) {
+      if (k >= rows) break;
+      const int t = t0 + k;
+      const int s = __shfl_sync(0xffffffffu, m_seg, k);
+      const long long slot = __shfl_sync(0xffffffffu, m_slot, k);
+      if (s != seg) {      // the rows in front of this one
+        seg = s;
+        const int at = __shfl_sync(0xffffffffu, m_at, k), local = t - __shfl_sync(0xffffffffu, m_first, k);
+        const int place = __shfl_sync(0xffffffffu, m_state, k);
+        T* state = p.n > 1 ? static_cast<T*>(p.state) + static_cast<long long>(place) * (p.n - 1) * p.C + ch + e : nullptr;
 #pragma unroll
-      for (int b = 1; b < NT; ++b)
-        if (b <= at) a += w[b][i] * (past[b - 1][i] + bias[i]);      // (taps behind the last one are zero)
-#pragma unroll
-      for (int b = NT - 1; b > 1; --b) past[b - 1][i] = past[b - 2][i];
-      if (NT > 1) past[0][i] = x[k][i];
-      y[i] = a;
-      ss += a * a;
-    }
-    if (normed) {
-      const float r = 1.f / sqrtf(wsum(ss) / p.dim + p.eps);
-#pragma unroll
-      for (int i = 0; i < N; ++i) y[i] *= r * nw[i];
-    }
-    T* dst;
-    if (hd < p.H) {
-      dst = static_cast<T*>(p.q) + (static_cast<long long>(t) * p.H + hd) * p.dp;
-    } else {
-      if (slot < 0 || slot >= p.pool_rows) continue;
-      dst = static_cast<T*>(value ? p.v_pool : p.k_pool) + (slot * p.G + g) * pitch;
-    }
-    if (!value && e < p.rot) {
-      const float2* cs = p.table + static_cast<long long>(t) * (p.rot >> 1) + (e >> 1);
-#pragma unroll
-      for (int i = 0; i < N; i += 2)
-        if (e + i < p.rot) {
-          const float2 f = cs[i >> 1];
-          const float a = y[i] * f.x - y[i + 1] * f.y;
-          y[i + 1] = y[i + 1] * f.x + y[i] * f.y;
-          y[i] = a;
+        for (int b = 1; b < NT; ++b) {
+          const bool there = b < p.n && b <= at;
+          const T* from = b <= local ? src + static_cast<long long>(t - b) * p.ld : state + static_cast<long long>(p.n - 1 - (b - local)) * p.C;
+          load_run<T, N, kVec>(from, there ? left : 0, past[b - 1]);
         }
+        if (!p.cu && p.n > 1) {      // the state moves on by one row
+#pragma unroll
+          for (int b = NT - 1; b >= 1; --b)
+            if (b < p.n) store_run<T, N, kVec>(state + static_cast<long long>(p.n - 1 - b) * p.C, left, b > 1 ? past[b > 1 ? b - 2 : 0] : x[k]);
+        }
+#pragma unroll
+        for (int b = 1; b < NT; ++b)
+#pragma unroll
+          for (int i = 0; i < N; ++i) past[b - 1][i] += b < p.n && b <= at ? bias[i] : 0.f;
+      }
+      float y[N], ss = 0.f;
+#pragma unroll
+      for (int i = 0; i < N; ++i) {
+        const float now = x[k][i] + bias[i];
+        float a = w[0][i] * now;
+#pragma unroll
+        for (int b = 1; b < NT; ++b) a += w[b][i] * past[b - 1][i];      // (taps behind the last one are zero)
+#pragma unroll
+        for (int b = NT - 1; b > 1; --b) past[b - 1][i] = past[b - 2][i];
+        if (NT > 1) past[0][i] = now;
+        y[i] = a;
+        ss += a * a;
+      }
+      if (normed) {
+        const float f = 1.f / sqrtf(wsum(ss) / p.dim + p.eps);
+#pragma unroll
+        for (int i = 0; i < N; ++i) y[i] *= f * nw[i];
+      }
+      T* dst;
+      if (hd < p.H) {
+        dst = static_cast<T*>(p.q) + (static_cast<long long>(t) * p.H + hd) * p.dp;
+      } else {
+        if (slot < 0 || slot >= p.pool_rows) continue;
+        dst = static_cast<T*>(value ? p.v_pool : p.k_pool) + (slot * p.G + g) * pitch;
+      }
+      if (!value && e < p.rot) {
+        const float2* cs = p.table + static_cast<long long>(t) * (p.rot >> 1) + (e >> 1);
+#pragma unroll
+        for (int i = 0; i < N; i += 2)
+          if (e + i < p.rot) {
+            const float2 f = cs[i >> 1];
+            const float a = y[i] * f.x - y[i + 1] * f.y;
+            y[i + 1] = y[i + 1] * f.x + y[i] * f.y;
+            y[i] = a;
+          }
+      }
+      store_run<T, N, kVec>(dst + e, pitch - e, y);      // columns behind the head's features are written as zeros
     }
-    store_run<T, N, kVec>(dst + e, pitch - e, y);      // columns behind the head's features are written as zeros
   }
 }
 
@@ -637,13 +655,15 @@ static int launch_inputs(const InputParams& p, cudaStream_t stm) {
 }
 
 template <typename T, int NP, int NT>
-static int launch_conv_np(const ConvParams& p, int segs, cudaStream_t stm) {
+static int launch_conv_np(ConvParams p, int segs, cudaStream_t stm) {
   constexpr int N = 2 * NP, bytes = sizeof(T) == 4 ? 8 : (N % 8 == 0 ? 16 : 2 * N);      // what a lane loads at once
   const bool pair = p.dim % N == 0 && p.dp % N == 0 && p.ld * sizeof(T) % bytes == 0 && p.C * sizeof(T) % bytes == 0 &&
                     (!p.k_pool || (p.vdim % N == 0 && p.vp % N == 0)) &&
                     (reinterpret_cast<uintptr_t>(p.qkv) | reinterpret_cast<uintptr_t>(p.state) | reinterpret_cast<uintptr_t>(p.q) |
-                     reinterpret_cast<uintptr_t>(p.k_pool) | reinterpret_cast<uintptr_t>(p.v_pool)) % 16 == 0;
-  const int run = p.cu ? 8 : 1;
+                     reinterpret_cast<uintptr_t>(p.k_pool) | reinterpret_cast<uintptr_t>(p.v_pool) | reinterpret_cast<uintptr_t>(p.bias) |
+                     reinterpret_cast<uintptr_t>(p.taps) | reinterpret_cast<uintptr_t>(p.q_w) | reinterpret_cast<uintptr_t>(p.k_w)) % 16 == 0;
+  p.runs = p.cu && p.T >= 2048 ? 4 : 1;      // (fewer rows: more warps instead)
+  const int run = (p.cu ? 8 : 1) * p.runs;
   const long long units = static_cast<long long>((p.T + run - 1) / run) * (p.H + (p.k_pool ? 2 * p.G : 0));
   const unsigned grid = static_cast<unsigned>((units + 7) / 8);
   if (p.cu) {
@@ -747,7 +767,7 @@ extern "C" int rb_conv_inputs(const void* qkv, int ld, const void* bias, const v
   if (ld < C || (k_pool && (!v_pool || !slots || G < 1 || vdim < 1 || vp < vdim || vp % 2)) || (cu && (!seg_of || !pos)) || !ctx || !state_slot) return -2;
   if (eps > 0.f && (!q_w || (k_pool && !k_w))) return -2;
   ConvParams p{qkv, bias, taps, state, q_w, k_w, reinterpret_cast<const float2*>(table), q, k_pool, v_pool, slots, ctx, state_slot, cu, seg_of, pos,
-               pool_rows, T, H, G, dim, vdim, dp, vp, rot, ld, n, C, eps};
+               pool_rows, T, H, G, dim, vdim, dp, vp, rot, ld, n, C, 1, eps};
   if (fp32) return n <= 4 ? launch_conv<float, 4>(p, segs, stm) : launch_conv<float, 8>(p, segs, stm);
   return n <= 4 ? launch_conv<bf16, 4>(p, segs, stm) : launch_conv<bf16, 8>(p, segs, stm);
 }

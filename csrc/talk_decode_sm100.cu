@@ -298,40 +298,57 @@ struct MergeParams {
   __nv_bfloat16* out;             // [B][H][out_d]
   int H, G, rep, repp, cols, splits, out_d;
 };
+constexpr int MG_WARPS = 8;      // every warp takes every eighth head g; a lane has four features
 template <int REPP>
-__global__ void __launch_bounds__(128) talk_merge_kernel(const MergeParams p) {
+__global__ void __launch_bounds__(MG_WARPS * 32) talk_merge_kernel(const MergeParams p) {
   __shared__ float inv[kMaxCols];
-  extern __shared__ float mix[];      // [H][REPP]: what head i of this group takes of head g
-  const int b = blockIdx.x, c = blockIdx.y, d = threadIdx.x;
-  for (int g = d; g < p.H; g += 128) {
+  extern __shared__ __align__(16) float sm[];      // [H][REPP]: what head i of this group takes of head g; then [MG_WARPS][REPP][128] sums
+  float* sums = sm + p.H * REPP;
+  const int b = blockIdx.x, c = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, d = (tid & 31) * 4;
+  for (int g = tid; g < p.H; g += MG_WARPS * 32) {
     const int col = g / p.rep * REPP + g % p.rep;
     float l = p.sink ? exp2f(__bfloat162float(p.sink[g]) * 1.4426950408889634f) : 0.f;
+#pragma unroll 4
     for (int s = 0; s < p.splits; ++s) l += p.part_l[(static_cast<size_t>(b) * p.splits + s) * p.cols + col];
     inv[g] = l > 0.f ? 1.f / l : 0.f;
   }
-  for (int i = d; i < p.H * REPP; i += 128) {
+  for (int i = tid; i < p.H * REPP; i += MG_WARPS * 32) {
     const int g = i / REPP, h = i - g * REPP;
-    mix[i] = h < p.rep ? __bfloat162float(p.mix[static_cast<size_t>(c * p.rep + h) * p.H + g]) : 0.f;
+    sm[i] = h < p.rep ? __bfloat162float(p.mix[static_cast<size_t>(c * p.rep + h) * p.H + g]) : 0.f;
   }
   __syncthreads();
-  if (d >= p.out_d) return;
-  float acc[REPP];
+  float4 acc[REPP];
 #pragma unroll
-  for (int i = 0; i < REPP; ++i) acc[i] = 0.f;
+  for (int i = 0; i < REPP; ++i) acc[i] = make_float4(0.f, 0.f, 0.f, 0.f);
   const float* base = p.part_o + (static_cast<size_t>(b) * p.splits * p.G + c) * p.cols * 128 + d;
   const size_t step = static_cast<size_t>(p.G) * p.cols * 128;
-#pragma unroll 4
-  for (int g = 0; g < p.H; ++g) {
-    const float* src = base + static_cast<size_t>(g / p.rep * REPP + g % p.rep) * 128;
-    float a = 0.f;
-    for (int s = 0; s < p.splits; ++s) a += src[s * step];
-    a *= inv[g];
+  if (d < p.out_d) {      // (features behind the values' columns were never written)
+    for (int g = warp; g < p.H; g += MG_WARPS) {
+      const float* src = base + static_cast<size_t>(g / p.rep * REPP + g % p.rep) * 128;
+      float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
+      for (int s = 0; s < p.splits; ++s) {
+        const float4 x = *reinterpret_cast<const float4*>(src + s * step);
+        a.x += x.x; a.y += x.y; a.z += x.z; a.w += x.w;
+      }
+      const float f = inv[g];
 #pragma unroll
-    for (int i = 0; i < REPP; ++i) acc[i] += mix[g * REPP + i] * a;
+      for (int i = 0; i < REPP; ++i) {
+        const float m = sm[g * REPP + i] * f;
+        acc[i].x += m * a.x; acc[i].y += m * a.y; acc[i].z += m * a.z; acc[i].w += m * a.w;
+      }
+    }
   }
 #pragma unroll
-  for (int i = 0; i < REPP; ++i)
-    if (i < p.rep) p.out[(static_cast<size_t>(b) * p.H + c * p.rep + i) * p.out_d + d] = __float2bfloat16(acc[i]);
+  for (int i = 0; i < REPP; ++i) *reinterpret_cast<float4*>(sums + (warp * REPP + i) * 128 + d) = acc[i];
+  __syncthreads();
+  for (int i = tid; i < p.rep * 128; i += MG_WARPS * 32) {
+    const int h = i >> 7, k = i & 127;
+    float o = 0.f;
+#pragma unroll
+    for (int w = 0; w < MG_WARPS; ++w) o += sums[(w * REPP + h) * 128 + k];
+    if (k < p.out_d) p.out[(static_cast<size_t>(b) * p.H + c * p.rep + h) * p.out_d + k] = __float2bfloat16(o);
+  }
 }
 
 struct Plan {
@@ -386,8 +403,14 @@ static int dispatch(int dk, int dv, const void* kc, const void* vc, uint64_t slo
   if (dk == 128) rc = dv == 128 ? launch<128, 128, REPP>(kc, vc, slots, p, o, B, st) : launch<128, 64, REPP>(kc, vc, slots, p, o, B, st);
   else rc = dv == 128 ? launch<64, 128, REPP>(kc, vc, slots, p, o, B, st) : launch<64, 64, REPP>(kc, vc, slots, p, o, B, st);
   if (rc) return rc;
-  const size_t smem = static_cast<size_t>(m.H) * REPP * 4;
-  talk_merge_kernel<REPP><<<dim3(B, m.G), 128, smem, st>>>(m);
+  const int smem = (m.H + MG_WARPS * 128) * REPP * 4;
+  static bool attr = false;
+  if (!attr) {
+    const cudaError_t e = cudaFuncSetAttribute(talk_merge_kernel<REPP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (kMaxCols + MG_WARPS * 128) * REPP * 4);
+    if (e != cudaSuccess) return static_cast<int>(e);
+    attr = true;
+  }
+  talk_merge_kernel<REPP><<<dim3(B, m.G), MG_WARPS * 32, smem, st>>>(m);
   rb_note_launch(1);
   return static_cast<int>(cudaGetLastError());
 }

@@ -7,7 +7,7 @@
 // exponential.  The CTAs are persistent and their blocks form one sequence across tiles.  Scores run four blocks ahead of the products; two
 // sets of eight warps (two threads per row) take the blocks in turn, and P replaces S in TMEM, where the products read it.  Warps of
 // their own read the accumulators of a finished tile while the softmax is at the next one; whole tiles leave through shared memory and TMA
-// stores.  Keys and values have three stages each and a producer of their own: a block's arithmetic is shorter than the way of its tiles
+// stores.  Keys (three stages) and values (two) have producers of their own: a block's arithmetic is shorter than the way of its tiles
 // through the L2.  Issuing a block's products, with the waits around them, takes one thread longer than the tensor cores need for them, so scores
 // and output products are issued by two.  Warps 0-15: softmax, warp 16: TMA of queries and keys, warp 17: scores, warps 18-21: outputs, warp
 // 22: TMA of values, warp 23: products with the values.  Every wait is bounded; no load uses cluster multicast.
@@ -24,15 +24,15 @@ constexpr int BKV = 64;
 constexpr int SOFT = 512;                 // softmax threads: two sets of two per row
 constexpr int kWarpK = 16, kWarpS = 17, kWarpOut = 18, kWarpV = 22, kWarpPv = 23;      // (four warps for the outputs)
 constexpr int THREADS = 24 * 32;
-constexpr int ST = 3;                     // stages of keys and of values
+constexpr int KST = 3, VST = 2;           // stages of keys and of values
 constexpr int NS = 4;                     // buffers of scores
-static_assert(ST < NS, "a producer is never two phases behind");
+static_assert(KST < NS && VST < NS, "a producer is never two phases behind");
 constexpr int RING = 8;                   // items whose sums are kept: the softmax is at most NS of them ahead of the outputs
 constexpr int kTmemCols = 512;
 constexpr int T_S = 0;                    // NS buffers of 64 columns; P takes the first 16 of every 32
 constexpr int T_O = NS * 64;
 constexpr int kQHalf = BQ * 128, kKVHalf = BKV * 128;      // bytes of 64 columns
-constexpr int kStage = BQ * 128;          // 64 columns of outputs on their way out; two of them
+constexpr int kStage = BQ * 128;          // 64 columns of outputs on their way out
 
 struct Params {
   const int* blocks;         // [n][4]: segment, first row, rows, position of the first row; null: row i is segment i, at ctx[i] - 1
@@ -102,7 +102,7 @@ talk_flash_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
   constexpr int kQBytes = DK / 64 * kQHalf, kKBytes = DK / 64 * kKVHalf, kVBytes = DV / 64 * kKVHalf;
   extern __shared__ __align__(1024) uint8_t smem[];
   uint64_t* bars = reinterpret_cast<uint64_t*>(smem + p.bar_at);
-  // blocks are numbered across items (g): S and P of block g are buffer g % NS, its keys and values stage g % ST; queries and accumulators
+  // blocks are numbered across items (g): S and P of block g are buffer g % NS, its keys and values a stage each; queries and accumulators
   // go by item (n)
   uint64_t* qfull = bars;
   uint64_t* qempty = bars + 1;     // the scores of an item are complete
@@ -112,9 +112,9 @@ talk_flash_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
   uint64_t* bar_pv = bar_s + NS;   // [NS] its products are: the buffer and the stage of its values are free
   uint64_t* bar_p = bar_pv + NS;   // [NS] P of a block is written
   uint64_t* bar_l = bar_p + NS;    // [RING] the sums of an item are written
-  uint64_t* kfull = bar_l + RING;  // [ST]
-  uint64_t* vfull = kfull + ST;
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(vfull + ST);
+  uint64_t* kfull = bar_l + RING;  // [KST]
+  uint64_t* vfull = kfull + KST;   // [VST]
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(vfull + VST);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
   float* sums = reinterpret_cast<float*>(smem + p.bar_at + 512);      // [RING][4][128]
 
@@ -130,10 +130,8 @@ talk_flash_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
       mbar_init(&bar_p[i], SOFT / 2);
     }
     for (int i = 0; i < RING; ++i) mbar_init(&bar_l[i], SOFT);
-    for (int i = 0; i < ST; ++i) {
-      mbar_init(&kfull[i], 1);
-      mbar_init(&vfull[i], 1);
-    }
+    for (int i = 0; i < KST; ++i) mbar_init(&kfull[i], 1);
+    for (int i = 0; i < VST; ++i) mbar_init(&vfull[i], 1);
     *abort_flag = 0;
     if ((smem_u32(smem) & 1023u) != 0) {           // swizzled tiles need 1 KB alignment
       *abort_flag = 1;
@@ -161,6 +159,7 @@ talk_flash_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
       const int rows = p.page < BKV ? p.page : BKV;          // rows per box
       uint64_t* full = values ? vfull : kfull;
       uint64_t* freed = values ? bar_pv : bar_s;
+      const int stages = values ? VST : KST;
       bool ok = true;
       int s = 0, n = 0, g = 0;
       for (int i = blockIdx.x; i < p.n_items && ok; i += step, ++n) {
@@ -175,7 +174,7 @@ talk_flash_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
         }
         for (int j = 0; j < w.n_blocks; ++j, ++g) {
           const int at = w.first_position(j);
-          if (g >= ST) ok = mbar_wait(&freed[(g - ST) % NS], static_cast<uint32_t>((g - ST) / NS) & 1, abort_flag, p.err);
+          if (g >= stages) ok = mbar_wait(&freed[(g - stages) % NS], static_cast<uint32_t>((g - stages) / NS) & 1, abort_flag, p.err);
           if (!ok) break;
           mbar_expect_tx(&full[s], values ? w.nv * kVBytes : kKBytes);
           for (int r = 0; r < BKV; r += rows) {
@@ -189,7 +188,7 @@ talk_flash_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
               for (int c = 0; c < DK / 64; ++c) tma_load_3d(sk + c * kKVHalf, &tma_k, &full[s], c * 64, w.kvh, row);
             }
           }
-          if (++s == ST) s = 0;
+          if (++s == stages) s = 0;
         }
       }
     }
@@ -218,7 +217,7 @@ talk_flash_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
             umma_f16(tmem_base + T_S + s * BKV, da, db, idesc, kk > 0 ? 1u : 0u);
           }
           umma_commit(&bar_s[s]);
-          if (++stage == ST) {
+          if (++stage == KST) {
             stage = 0;
             ph ^= 1;
           }
@@ -249,7 +248,7 @@ talk_flash_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
             umma_f16_ts(tmem_base + T_O, tmem_base + T_S + s * BKV + (kk >> 1) * 32 + (kk & 1) * 8, db, idesc, (j > 0 || kk > 0) ? 1u : 0u);
           }
           umma_commit(&bar_pv[s]);
-          if (++stage == ST) {
+          if (++stage == VST) {
             stage = 0;
             ph ^= 1;
           }
@@ -265,56 +264,50 @@ talk_flash_kernel(const __grid_constant__ CUtensorMap tma_q, const __grid_consta
     const uint32_t lane_addr = static_cast<uint32_t>((warp & 3) * 32) << 16;
     const bool issues = warp == kWarpOut && lane == 0;
     bool ok = !dead;
-    int n = 0, buffer = 0;
+    int n = 0;
     for (int i = blockIdx.x; i < p.n_items && ok; i += step, ++n) {
       const Item w(p, i);
       ok = mbar_wait(&bar_l[n % RING], static_cast<uint32_t>(n / RING) & 1, abort_flag, p.err) &&
            mbar_wait(bar_done, static_cast<uint32_t>(n) & 1, abort_flag, p.err);
+      if (issues) tma_store_wait_read<0>();                      // the item before has left shared memory
       ok = named_bar_and(1, 128, ok);                            // (all leave together when a wait ran out)
       if (!ok) break;
       tc_fence_after();
       const float* sum = sums + (n % RING) * 4 * BQ + r;
       const float l = sum[0] + sum[BQ] + sum[2 * BQ] + sum[3 * BQ];
       const float inv_l = l > 0.f ? 1.f / l : 0.f;
-      const int chunks = w.nv * (DV / 64);                       // of 64 columns; two buffers on their way out
       const bool whole = p.stores && w.ntok == p.tokens, mine = t < w.ntok;
       __nv_bfloat16* out = p.out + ((static_cast<size_t>(w.row0 + t) * p.H + w.kvh * p.G + r % p.G) * p.Hkv + w.v0) * p.out_d;
+      const int parts = w.nv * (DV / 32);                        // of 32 columns
 #pragma unroll 1
-      for (int ch = 0; ch < chunks; ++ch) {
-        const int v = ch / (DV / 64), c = (ch % (DV / 64)) * 64;
-        uint8_t* dst = smem + p.out_at + buffer * kStage + r * 128;
-        if (whole) {
-          if (issues) tma_store_wait_read<1>();                  // the store before the last one has left shared memory
-          named_bar_sync(1, 128);
-        }
-#pragma unroll
-        for (int part = 0; part < 2; ++part) {
-          uint32_t o[32];
-          tmem_ld_32x32b_x32(tmem_base + T_O + v * DV + c + part * 32 + lane_addr, o);
-          tmem_wait_ld();
-#pragma unroll
-          for (int e = 0; e < 4; ++e) {
-            uint4 pk;
-            pk.x = pack_bf16(__uint_as_float(o[8 * e]) * inv_l, __uint_as_float(o[8 * e + 1]) * inv_l);
-            pk.y = pack_bf16(__uint_as_float(o[8 * e + 2]) * inv_l, __uint_as_float(o[8 * e + 3]) * inv_l);
-            pk.z = pack_bf16(__uint_as_float(o[8 * e + 4]) * inv_l, __uint_as_float(o[8 * e + 5]) * inv_l);
-            pk.w = pack_bf16(__uint_as_float(o[8 * e + 6]) * inv_l, __uint_as_float(o[8 * e + 7]) * inv_l);
-            if (whole) *reinterpret_cast<uint4*>(dst + (((part * 4 + e) ^ (r & 7)) << 4)) = pk;
-            else if (mine && c + part * 32 + e * 8 < p.out_d) *reinterpret_cast<uint4*>(out + static_cast<size_t>(v) * p.out_d + c + part * 32 + e * 8) = pk;
-          }
-        }
-        if (ch + 1 == chunks) {
+      for (int part = 0; part < parts; ++part) {
+        uint32_t o[32];
+        tmem_ld_32x32b_x32(tmem_base + T_O + part * 32 + lane_addr, o);
+        tmem_wait_ld();
+        if (part + 1 == parts) {
           tc_fence_before();
           mbar_arrive(bar_free);
         }
-        if (whole) {
-          fence_proxy_async();
-          named_bar_sync(1, 128);
-          if (issues) {
-            tma_store_4d(&tma_o, smem + p.out_at + buffer * kStage, c, w.v0 + v, w.kvh * p.G, w.row0);
-            tma_store_commit();
-          }
-          buffer ^= 1;
+        const int v = part / (DV / 32), c = (part % (DV / 32)) * 32;
+        uint8_t* dst = smem + p.out_at + (part >> 1) * kStage + r * 128;
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          uint4 pk;
+          pk.x = pack_bf16(__uint_as_float(o[8 * e]) * inv_l, __uint_as_float(o[8 * e + 1]) * inv_l);
+          pk.y = pack_bf16(__uint_as_float(o[8 * e + 2]) * inv_l, __uint_as_float(o[8 * e + 3]) * inv_l);
+          pk.z = pack_bf16(__uint_as_float(o[8 * e + 4]) * inv_l, __uint_as_float(o[8 * e + 5]) * inv_l);
+          pk.w = pack_bf16(__uint_as_float(o[8 * e + 6]) * inv_l, __uint_as_float(o[8 * e + 7]) * inv_l);
+          if (whole) *reinterpret_cast<uint4*>(dst + ((((part & 1) * 4 + e) ^ (r & 7)) << 4)) = pk;
+          else if (mine && c + e * 8 < p.out_d) *reinterpret_cast<uint4*>(out + static_cast<size_t>(v) * p.out_d + c + e * 8) = pk;
+        }
+      }
+      if (whole) {
+        fence_proxy_async();
+        named_bar_sync(1, 128);
+        if (issues) {
+          for (int k = 0; k < parts / 2; ++k)
+            tma_store_4d(&tma_o, smem + p.out_at + k * kStage, (k % (DV / 64)) * 64, w.v0 + k / (DV / 64), w.kvh * p.G, w.row0);
+          tma_store_commit();
         }
       }
     }
@@ -421,9 +414,9 @@ static int launch(const void* q, const void* kc, const void* vc, int rows, int n
     if (most < 1) return -20;
     p.slices = (p.Hkv + most - 1) / most;
     p.nv = (p.Hkv + p.slices - 1) / p.slices;
-    p.v_at = DK / 64 * (kQHalf + ST * kKVHalf);
-    p.out_at = p.v_at + ST * p.nv * (DV / 64) * kKVHalf;
-    p.bar_at = p.out_at + 2 * kStage;
+    p.v_at = DK / 64 * (kQHalf + KST * kKVHalf);
+    p.out_at = p.v_at + VST * p.nv * (DV / 64) * kKVHalf;
+    p.bar_at = p.out_at + p.nv * (DV / 64) * kStage;
     total = p.bar_at + 512 + RING * 4 * BQ * 4;
     if (total <= 227 * 1024) break;
   }
