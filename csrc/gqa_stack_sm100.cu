@@ -241,36 +241,42 @@ struct ConvParams {
 };
 // N consecutive elements of which `left` exist (kVec: all or none, N * sizeof(T) aligned)
 template <typename T, int N, bool kVec>
-__device__ __forceinline__ void load_run(const T* p, int left, float* v) {
+struct Run {      // as loaded: 16-bit pairs stay packed until they are used
+  static constexpr bool kPacked = kVec && sizeof(T) == 2;
+  static constexpr int W = kPacked ? N / 2 : N;
+  uint32_t u[W];
+  __device__ __forceinline__ void load(const T* p, int left) {
 #pragma unroll
-  for (int i = 0; i < N; ++i) v[i] = 0.f;
-  if constexpr (kVec) {
-    if (left <= 0) return;
-    if constexpr (sizeof(T) == 4) {
+    for (int i = 0; i < W; ++i) u[i] = 0u;
+    if constexpr (kVec) {
+      if (left <= 0) return;
+      const uint32_t* w = reinterpret_cast<const uint32_t*>(p);
+      if constexpr (W % 4 == 0 && kPacked) {
 #pragma unroll
-      for (int i = 0; i < N; i += 2) *reinterpret_cast<float2*>(v + i) = *reinterpret_cast<const float2*>(p + i);
-    } else {
-      uint32_t u[N / 2];
-      if constexpr (N % 8 == 0) {
+        for (int i = 0; i < W; i += 4) *reinterpret_cast<uint4*>(u + i) = *reinterpret_cast<const uint4*>(w + i);
+      } else if constexpr (W % 2 == 0) {
 #pragma unroll
-        for (int i = 0; i < N / 2; i += 4) *reinterpret_cast<uint4*>(u + i) = *reinterpret_cast<const uint4*>(p + 2 * i);
-      } else if constexpr (N == 4) {
-        *reinterpret_cast<uint2*>(u) = *reinterpret_cast<const uint2*>(p);
+        for (int i = 0; i < W; i += 2) *reinterpret_cast<uint2*>(u + i) = *reinterpret_cast<const uint2*>(w + i);
       } else {
-#pragma unroll
-        for (int i = 0; i < N / 2; ++i) u[i] = *reinterpret_cast<const uint32_t*>(p + 2 * i);
+        u[0] = *w;
       }
+    } else {
 #pragma unroll
-      for (int i = 0; i < N / 2; ++i) {
-        v[2 * i] = __uint_as_float(u[i] << 16);
-        v[2 * i + 1] = __uint_as_float(u[i] & 0xffff0000u);
-      }
+      for (int i = 0; i < N; ++i)
+        if (i < left) u[i] = __float_as_uint(ld(p + i));
     }
-  } else {
-#pragma unroll
-    for (int i = 0; i < N; ++i)
-      if (i < left) v[i] = ld(p + i);
   }
+  __device__ __forceinline__ float at(int i) const {
+    if constexpr (kPacked) return __uint_as_float(i & 1 ? u[i >> 1] & 0xffff0000u : u[i >> 1] << 16);
+    else return __uint_as_float(u[i]);
+  }
+};
+template <typename T, int N, bool kVec>
+__device__ __forceinline__ void load_run(const T* p, int left, float* v) {
+  Run<T, N, kVec> r;
+  r.load(p, left);
+#pragma unroll
+  for (int i = 0; i < N; ++i) v[i] = r.at(i);
 }
 template <typename T, int N, bool kVec>
 __device__ __forceinline__ void store_run(T* p, int left, const float* v) {
@@ -304,7 +310,7 @@ __device__ __forceinline__ void store_run(T* p, int left, const float* v) {
 }
 // kVec: heads, their pitches, rows and the state split into aligned runs of 2 NP features
 template <typename T, int NP, int NT, int RUN, bool kVec>
-__global__ void __launch_bounds__(256) conv_inputs_kernel(const ConvParams p) {
+__global__ void __launch_bounds__(256, NP <= 2 && NT <= 4 ? 2 : 1) conv_inputs_kernel(const ConvParams p) {
   constexpr int N = 2 * NP;
   const int lane = threadIdx.x & 31;
   const int per = p.H + (p.k_pool ? 2 * p.G : 0);
@@ -363,10 +369,16 @@ __global__ void __launch_bounds__(256) conv_inputs_kernel(const ConvParams p) {
       m_state = p.state_slot[m_seg];
       if (hd >= p.H) m_slot = p.slots[t];
     }
-    float x[RUN][N];
+    Run<T, N, kVec> x[RUN];
+    float2 cs[RUN][NP];
 #pragma unroll
     for (int k = 0; k < RUN; ++k) {
-      if (k < rows) load_run<T, N, kVec>(src + static_cast<long long>(t0 + k) * p.ld, left, x[k]);
+      if (k < rows) x[k].load(src + static_cast<long long>(t0 + k) * p.ld, left);
+#pragma unroll
+      for (int i = 0; i < NP; ++i) {
+        cs[k][i] = make_float2(1.f, 0.f);
+        if (k < rows && !value && e + 2 * i < p.rot) cs[k][i] = p.table[static_cast<long long>(t0 + k) * (p.rot >> 1) + (e >> 1) + i];
+      }
     }
 #pragma unroll
     for (int k = 0; k < RUN; ++k) {
@@ -388,7 +400,12 @@ __global__ void __launch_bounds__(256) conv_inputs_kernel(const ConvParams p) {
         if (!p.cu && p.n > 1) {      // the state moves on by one row
 #pragma unroll
           for (int b = NT - 1; b >= 1; --b)
-            if (b < p.n) store_run<T, N, kVec>(state + static_cast<long long>(p.n - 1 - b) * p.C, left, b > 1 ? past[b > 1 ? b - 2 : 0] : x[k]);
+            if (b < p.n) {
+              float moved[N];
+#pragma unroll
+              for (int i = 0; i < N; ++i) moved[i] = b > 1 ? past[b > 1 ? b - 2 : 0][i] : x[k].at(i);
+              store_run<T, N, kVec>(state + static_cast<long long>(p.n - 1 - b) * p.C, left, moved);
+            }
         }
 #pragma unroll
         for (int b = 1; b < NT; ++b)
@@ -398,7 +415,7 @@ __global__ void __launch_bounds__(256) conv_inputs_kernel(const ConvParams p) {
       float y[N], ss = 0.f;
 #pragma unroll
       for (int i = 0; i < N; ++i) {
-        const float now = x[k][i] + bias[i];
+        const float now = x[k].at(i) + bias[i];
         float a = w[0][i] * now;
 #pragma unroll
         for (int b = 1; b < NT; ++b) a += w[b][i] * past[b - 1][i];      // (taps behind the last one are zero)
@@ -420,16 +437,12 @@ __global__ void __launch_bounds__(256) conv_inputs_kernel(const ConvParams p) {
         if (slot < 0 || slot >= p.pool_rows) continue;
         dst = static_cast<T*>(value ? p.v_pool : p.k_pool) + (slot * p.G + g) * pitch;
       }
-      if (!value && e < p.rot) {
-        const float2* cs = p.table + static_cast<long long>(t) * (p.rot >> 1) + (e >> 1);
 #pragma unroll
-        for (int i = 0; i < N; i += 2)
-          if (e + i < p.rot) {
-            const float2 f = cs[i >> 1];
-            const float a = y[i] * f.x - y[i + 1] * f.y;
-            y[i + 1] = y[i + 1] * f.x + y[i] * f.y;
-            y[i] = a;
-          }
+      for (int i = 0; i < N; i += 2) {
+        const float2 f = cs[k][i >> 1];
+        const float a = y[i] * f.x - y[i + 1] * f.y;
+        y[i + 1] = y[i + 1] * f.x + y[i] * f.y;
+        y[i] = a;
       }
       store_run<T, N, kVec>(dst + e, pitch - e, y);      // columns behind the head's features are written as zeros
     }
@@ -662,13 +675,14 @@ static int launch_conv_np(ConvParams p, int segs, cudaStream_t stm) {
                     (reinterpret_cast<uintptr_t>(p.qkv) | reinterpret_cast<uintptr_t>(p.state) | reinterpret_cast<uintptr_t>(p.q) |
                      reinterpret_cast<uintptr_t>(p.k_pool) | reinterpret_cast<uintptr_t>(p.v_pool) | reinterpret_cast<uintptr_t>(p.bias) |
                      reinterpret_cast<uintptr_t>(p.taps) | reinterpret_cast<uintptr_t>(p.q_w) | reinterpret_cast<uintptr_t>(p.k_w)) % 16 == 0;
-  p.runs = p.cu && p.T >= 2048 ? 4 : 1;      // (fewer rows: more warps instead)
-  const int run = (p.cu ? 8 : 1) * p.runs;
+  constexpr int RUN = NP <= 4 ? 4 : 2;
+  p.runs = p.cu ? (p.T >= 2048 ? 32 : 8) / RUN : 1;      // (fewer rows: more warps instead)
+  const int run = p.cu ? RUN * p.runs : 1;
   const long long units = static_cast<long long>((p.T + run - 1) / run) * (p.H + (p.k_pool ? 2 * p.G : 0));
   const unsigned grid = static_cast<unsigned>((units + 7) / 8);
   if (p.cu) {
-    if (pair) conv_inputs_kernel<T, NP, NT, 8, true><<<grid, 256, 0, stm>>>(p);
-    else conv_inputs_kernel<T, NP, NT, 8, false><<<grid, 256, 0, stm>>>(p);
+    if (pair) conv_inputs_kernel<T, NP, NT, RUN, true><<<grid, 256, 0, stm>>>(p);
+    else conv_inputs_kernel<T, NP, NT, RUN, false><<<grid, 256, 0, stm>>>(p);
     if (p.n > 1) conv_state_kernel<T><<<dim3(segs, (p.C + 255) / 256), 256, 0, stm>>>(p);
     rb_note_launch(p.n > 1 ? 2 : 1);
   } else {
